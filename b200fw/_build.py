@@ -50,13 +50,22 @@ def sources():
     return sorted(CSRC.glob("*.cu"))
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
-    """Compile (if stale) and return the path of the shared library."""
+def partial_path(only) -> Path:
+    return LIB_DIR / ("libb200fw_" + "_".join(sorted(only)) + ".so")
+
+
+def build(verbose: bool = False, force: bool = False, only=None) -> Path:
+    """Compile (if stale) and return the path of the shared library.  ``only``: stems of the sources to put into a smaller
+    library of their own (for a process that needs few kernels and should not wait for the others)."""
+    chosen = [p for p in sources() if only is None or p.stem in only]
+    if only is not None and len(chosen) != len(set(only)):
+        raise ValueError(f"unknown sources: {sorted(set(only) - {p.stem for p in chosen})}")
+    lib_path = LIB_PATH if only is None else partial_path(only)
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
     headers = sorted(list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h")))
     nvcc = _nvcc()
     jobs = []
-    for src in sources():
+    for src in chosen:
         obj = OBJ_DIR / (src.stem + ".o")
         stamp = OBJ_DIR / (src.stem + ".sha")
         dig = _digest([src] + headers)
@@ -80,13 +89,13 @@ def build(verbose: bool = False, force: bool = False) -> Path:
     if jobs:
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(compile_one, jobs))
-    objs = [OBJ_DIR / (s.stem + ".o") for s in sources()]
-    if jobs or not LIB_PATH.exists():
-        cmd = [nvcc, "-shared", "-o", str(LIB_PATH), *map(str, objs), "-cudart", "static"]
+    objs = [OBJ_DIR / (s.stem + ".o") for s in chosen]
+    if jobs or not lib_path.exists():
+        cmd = [nvcc, "-shared", "-o", str(lib_path), *map(str, objs), "-cudart", "static"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-    return LIB_PATH
+    return lib_path
 
 
 if __name__ == "__main__":

@@ -14,10 +14,18 @@ import torch
 
 _lock = threading.Lock()
 _lib: Optional[ctypes.CDLL] = None
+_sources = None      # see need_only()
 
 
 class NativeError(RuntimeError):
     """A launcher rejected its arguments, a launch failed, or a kernel recorded an error status."""
+
+
+def need_only(sources) -> None:
+    """Say, before the first kernel, which of ``csrc/`` this process will use: where the full library has not been built, only
+    those are compiled."""
+    global _sources
+    _sources = tuple(sources)
 
 
 def lib() -> ctypes.CDLL:
@@ -30,7 +38,7 @@ def lib() -> ctypes.CDLL:
 
             path = _build.LIB_PATH
             if not path.exists():
-                path = _build.build()
+                path = _build.build(only=_sources)
             handle = ctypes.CDLL(str(path), mode=ctypes.RTLD_GLOBAL)
             handle.b2_last_error.restype = ctypes.c_char_p
             handle.b2_status_read_and_clear.restype = ctypes.c_int

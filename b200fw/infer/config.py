@@ -41,6 +41,7 @@ class InferenceConfig:
     inference_mode: str = "mock"         # "kv_cache" (native paged model) | "eager" (full recompute) | "mock"
     use_real_model: bool = False
     model_path: str = ""
+    model_preset: str = ""               # name in b200fw.model.registry.PRESETS (random weights) when there is no model_path
     dtype: str = "bfloat16"
     # ---- additions ---------------------------------------------------------------------------------
     intermediate_size: int = 0
@@ -64,14 +65,21 @@ class InferenceConfig:
                    head_dim=mc.head_dim, hidden_size=mc.hidden_size, vocab_size=mc.vocab_size,
                    intermediate_size=mc.intermediate_size, **kw)
 
+    @classmethod
+    def from_preset(cls, name: str, **kw) -> "InferenceConfig":
+        from ..model.registry import PRESETS
+        return cls.from_model_config(PRESETS[name], model_preset=name, **kw)
+
     def kv_bytes_per_block(self) -> int:
         el = 1 if self.kv_cache_dtype == "fp8" else 2
         return 2 * self.num_layers * self.block_size * self.num_kv_heads * self.head_dim * el
 
     @classmethod
     def auto_from_device(cls, num_layers=32, num_kv_heads=8, head_dim=128, block_size=16,
-                         gpu_memory_fraction=0.3, max_blocks: int = 1 << 20, **kw) -> "InferenceConfig":
-        """Size the block pool from free device memory (a fraction of it); CPU gets a small pool."""
+                         gpu_memory_fraction=0.3, max_blocks: int = 1 << 20, bytes_per_token: int = 0,
+                         **kw) -> "InferenceConfig":
+        """Size the block pool from free device memory (a fraction of it); CPU gets a small pool.  ``bytes_per_token``: cache
+        bytes of one token when the layers are not all alike."""
         base = dict(num_layers=num_layers, num_kv_heads=num_kv_heads, head_dim=head_dim, block_size=block_size)
         if not torch.cuda.is_available():
             return cls(num_blocks=64, enable_cuda_graph=False, **base, **kw)
@@ -80,6 +88,6 @@ class InferenceConfig:
         except (RuntimeError, AssertionError):
             return cls(num_blocks=64, enable_cuda_graph=False, **base, **kw)
         probe = cls(**base, **{k: v for k, v in kw.items() if k == "kv_cache_dtype"})
-        blocks = max(32, int(free * gpu_memory_fraction) // probe.kv_bytes_per_block())
+        blocks = max(32, int(free * gpu_memory_fraction) // (bytes_per_token * block_size or probe.kv_bytes_per_block()))
         kw.setdefault("enable_cuda_graph", total > 12 * 1024 ** 3)
         return cls(num_blocks=min(blocks, max_blocks), **base, **kw)

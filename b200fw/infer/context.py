@@ -31,6 +31,10 @@ class InferenceContext:
     # ---- fields of the reference's context that the kernels here do not need (src/inference/context.py:22-40):
     max_seqlen_k: int = 0                            # filled by prepare_prefill for callers that want it
     slot_mapping: Optional[torch.Tensor] = None      # per-token slot ids; the store kernel takes `store_segments`
+    # ---- models with per-layer caches and recurrent state (b200fw.infer.hybrid) ----------------------------------
+    portions: Optional[object] = None                # b200fw.ops.portions.Portions: the step's rows, in the kernels' order
+    row_order: Optional[torch.Tensor] = None         # int64 [M]: caller's row of every kernel row (None: the same order)
+    row_place: Optional[torch.Tensor] = None         # int64 [M]: kernel row of every caller's row
 
     def slots_from_segments(self, block_size: int = 16) -> Optional[torch.Tensor]:
         """The reference's ``slot_mapping`` (int64 ``[tokens]``: ``block * block_size + offset``, ``-1`` = skip)

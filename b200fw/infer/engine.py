@@ -20,11 +20,13 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..model import ModelConfig, ParallelTransformerModel, load_from_hf_checkpoint, read_hf_config
+from ..model import ModelConfig, ParallelTransformerModel, load_from_hf_checkpoint
+from ..model import registry
 from ..obs import nvtx
 from ..obs.logging import get_logger
 from .config import InferenceConfig
 from .graphs import CUDAGraphRunner
+from .hybrid import HybridModelRunner, make_cache
 from .kv_cache import BlockPool, KVCacheManager
 from .prefix_cache import PrefixCache
 from .radix_cache import RadixAttentionCache
@@ -103,11 +105,17 @@ class InferenceEngine:
         mc = self.model.cfg
         if self.device.type == "cuda" and cfg.block_size != 16:
             raise ValueError(f"block_size={cfg.block_size}: the paged KV kernels are built for 16-token blocks")
-        self.pool = BlockPool(cfg.num_blocks, cfg.block_size, mc.num_layers, mc.num_kv_heads, mc.head_dim,
-                              p0.dtype, self.device, cfg.kv_cache_dtype)
-        self.kv = KVCacheManager(self.pool, cfg.block_size)
-        self.runner = ModelRunner(self.model, self.pool, self.kv, cfg.attention_partition_size,
-                                  cfg.enable_partitioned_attention)
+        if hasattr(self.model, "state_layer_shapes"):
+            self._check_recurrent_config()
+            self.pool, self.kv = make_cache(self.model, cfg.num_blocks, cfg.block_size, cfg.max_num_sequences, p0.dtype,
+                                            self.device)
+            self.runner = HybridModelRunner(self.model, self.pool, self.kv)
+        else:
+            self.pool = BlockPool(cfg.num_blocks, cfg.block_size, mc.num_layers, mc.num_kv_heads, mc.head_dim,
+                                  p0.dtype, self.device, cfg.kv_cache_dtype)
+            self.kv = KVCacheManager(self.pool, cfg.block_size)
+            self.runner = ModelRunner(self.model, self.pool, self.kv, cfg.attention_partition_size,
+                                      cfg.enable_partitioned_attention)
         self.runner.balance_splits = cfg.decode_balance_splits
         if cfg.enable_prefix_caching or cfg.use_radix_cache:
             self.prefix_cache = RadixAttentionCache(cfg.block_size, cfg.radix_cache_max_nodes) if cfg.use_radix_cache \
@@ -123,7 +131,19 @@ class InferenceEngine:
         self.initialized = True
         return self
 
-    def _build_model(self) -> ParallelTransformerModel:
+    def _check_recurrent_config(self):
+        """What a model with recurrent state cannot do: a cached prefix has pages but no state to go on from, a rejected
+        drafted token cannot be taken out of the state, and an fp8 cache wants equal layers."""
+        cfg = self.config
+        bad = [n for n, on in (("speculative_enabled", cfg.speculative_enabled), ("kv_cache_dtype='fp8'", cfg.kv_cache_dtype == "fp8"))
+               if on]
+        if bad:
+            raise ValueError(f"not available for a model with recurrent state: {', '.join(bad)}")
+        if cfg.enable_prefix_caching or cfg.use_radix_cache:
+            logger.warning("prefix caching is off: the model's recurrent state cannot be shared by prefix")
+            cfg.enable_prefix_caching = cfg.use_radix_cache = False
+
+    def _build_model(self):
         cfg = self.config
         dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
         if cfg.dtype == "float16":
@@ -132,14 +152,17 @@ class InferenceEngine:
         if dev.type == "cpu":
             dtype = torch.float32
         if cfg.model_path:
-            mc = read_hf_config(cfg.model_path)
+            mc = registry.read_config(cfg.model_path)
+        elif cfg.model_preset:
+            mc = registry.PRESETS[cfg.model_preset]
         else:
             mc = ModelConfig(cfg.vocab_size, cfg.hidden_size, cfg.num_layers, cfg.num_heads, cfg.num_kv_heads,
                              cfg.head_dim, cfg.intermediate_size or 3 * cfg.hidden_size)
-        model = ParallelTransformerModel(mc, dtype=dtype, device=dev)
-        model.init_weights(cfg.seed)
+        model = registry.build_model(mc, dtype=dtype, device=dev)
+        if not cfg.model_path or not hasattr(model, "checkpoint"):   # a strict loader fills every tensor itself
+            model.init_weights(cfg.seed)
         if cfg.model_path:
-            load_from_hf_checkpoint(model, cfg.model_path)
+            registry.load_checkpoint(model, cfg.model_path)
         for p in model.parameters():
             p.requires_grad_(False)
         return model
@@ -245,11 +268,12 @@ class InferenceEngine:
             return produced
         try:
             decode = [r for r in out.decode_requests if r.request_id not in out.prefill_tokens]
+            mixed = decode if out.prefill_requests and getattr(self.runner, "mixed_batches", False) else []
             if out.prefill_requests:
                 self._resolve_inflight(produced)    # steps with prefill chunks run synchronously
                 with nvtx.range("infer/prefill"):
-                    self._execute_prefill(out, produced)
-            if decode:
+                    self._execute_prefill(out, produced, mixed)
+            if decode and not mixed:
                 with nvtx.range("infer/decode"):
                     self._execute_decode(decode, produced, lookahead=not out.prefill_requests)
         except torch.cuda.OutOfMemoryError:
@@ -339,7 +363,9 @@ class InferenceEngine:
         self.stats["cached_prefix_tokens"] += r.num_cached_tokens
         return True
 
-    def _execute_prefill(self, out: SchedulerOutput, produced: Dict[str, List[int]]):
+    def _execute_prefill(self, out: SchedulerOutput, produced: Dict[str, List[int]], decode: List[Request] = ()):
+        """Run the scheduled prompt portions as one batch.  ``decode``: running requests whose next token joins the same
+        batch (runners with ``mixed_batches``)."""
         cfg = self.config
         batch, starts, counts = [], [], []
         for r in out.prefill_requests:
@@ -366,15 +392,22 @@ class InferenceEngine:
                 counts.append(n)
             except Exception as e:  # noqa: BLE001 - isolate the failing request
                 self._fail(r, e)
-        if cfg.inference_mode == "mock" or not batch:
+        if cfg.inference_mode == "mock" or not (batch or decode):
             self.stats["prefill_tokens"] += out.num_prefill_tokens
             return
+        live = self._reserve_decode(decode, produced) if decode else []
+        if live:        # reserving may have preempted a request that was about to prefill
+            keep = [i for i, r in enumerate(batch) if r.request_id in self.kv.tables]
+            batch, starts, counts = [batch[i] for i in keep], [starts[i] for i in keep], [counts[i] for i in keep]
+        if not (batch or live):
+            return
         ids = [t for r, s, n in zip(batch, starts, counts) for t in r.prompt_tokens[s:s + n]]
-        ctx = self.runner.prepare_prefill([r.request_id for r in batch], starts, counts)
-        tok = torch.tensor(ids, dtype=torch.long)
-        tok = tok.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else tok
-        logits = self.runner.forward(tok, ctx)
         self.stats["prefill_tokens"] += len(ids)
+        self.stats["decode_tokens"] += len(live)
+        ids += [r.output_tokens[-1] for r in live]
+        logits = self._portions_forward([r.request_id for r in batch + live],
+                                        starts + [self.kv.get_seq_token_count(r.request_id) - 1 for r in live],
+                                        counts + [1] * len(live), ids)
         done = [i for i, (r, s, n) in enumerate(zip(batch, starts, counts)) if s + n >= r.num_prompt_tokens]
         for r, n in zip(batch, counts):
             r.num_computed_tokens += n
@@ -389,6 +422,8 @@ class InferenceEngine:
                         self.pool.share(bid)
                     r._prefix_published = True
                     self._drop_inflight(r)
+        done += range(len(batch), len(batch) + len(live))
+        batch = batch + live
         if done:
             rows = torch.tensor(done, device=self.device)
             new, lps = self._sample([batch[i] for i in done], logits.index_select(0, rows))
@@ -399,6 +434,70 @@ class InferenceEngine:
                 produced.setdefault(r.request_id, []).append(t)
                 if self.spec is not None:
                     self._draft_prefill(r)
+
+    def _portions_forward(self, ids: List, starts: List[int], counts: List[int], tokens: List[int], **kw) -> torch.Tensor:
+        """One forward pass over portions of sequences whose pages are reserved; logits as ``ModelRunner.forward``."""
+        ctx = self.runner.prepare_prefill(ids, starts, counts)
+        tok = torch.tensor(tokens, dtype=torch.long)
+        tok = tok.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else tok
+        return self.runner.forward(tok, ctx, **kw)
+
+    # ---- given tokens instead of sampled ones -----------------------------------------------------------------------
+    @_locked
+    def feed(self, entries, want=None) -> Dict[str, torch.Tensor]:
+        """One step over given tokens: ``entries`` is a list of ``(sequence id, tokens)``; a sequence is admitted at its first
+        entry and goes on from its cache and state at later ones, until :meth:`release`.  All entries are one batch, run by
+        the same runner, pages and state slots as generation.  Returns ``{id: logits [n, vocab]}`` of the places ``want[id]``
+        among the entry's tokens (``want`` None: of every token).  Raises, with nothing computed, when the pages or slots do
+        not suffice."""
+        assert self.initialized and self.runner is not None, "feed() needs the kv_cache mode"
+        entries = [(i, [int(t) for t in toks]) for i, toks in entries]
+        V = self.model.cfg.vocab_size
+        if len({i for i, _ in entries}) != len(entries):
+            raise ValueError("feed: one entry per sequence and step")
+        for i, toks in entries:
+            if not toks or min(toks) < 0 or max(toks) >= V:
+                raise ValueError(f"sequence {i!r}: needs at least one token, all inside the vocabulary [0, {V})")
+        undo = []
+        try:
+            for i, toks in entries:
+                fresh = i not in self.kv.tables
+                if fresh and self.kv.allocate_for_sequence(i, 0) is None:
+                    raise RuntimeError(f"no state slot for sequence {i!r}")
+                have = self.kv.get_seq_token_count(i)
+                undo.append((i, fresh, have))
+                if not self.kv.ensure_capacity(i, have + len(toks)):
+                    raise RuntimeError(f"KV cache exhausted at sequence {i!r}")
+                self.kv.set_num_tokens(i, have + len(toks))
+        except RuntimeError:
+            for i, fresh, have in undo:
+                if fresh:
+                    self.kv.free_sequence(i)
+                else:
+                    self.kv.trim(i, have)
+            raise
+        starts, counts = [h for _, _, h in undo], [len(t) for _, t in entries]
+        rows, spans, at = [], {}, 0
+        for (i, toks) in entries:
+            w = list(range(len(toks))) if want is None else list(want.get(i, ()))
+            spans[i] = (len(rows), len(rows) + len(w))
+            rows += [at + k for k in w]
+            at += len(toks)
+        tokens = [t for _, toks in entries for t in toks]
+        ids = [i for i, _ in entries]
+        pick = torch.tensor(rows, dtype=torch.long, device=self.device)
+        self.stats["steps"] += 1
+        if all(c == 1 for c in counts):          # decode step
+            logits = self.runner.forward(self._stage("feed", torch.tensor(tokens, dtype=torch.long)),
+                                         self.runner.prepare_decode(ids), rows=pick)
+        else:
+            logits = self._portions_forward(ids, starts, counts, tokens, rows=pick)
+        return {i: logits[a:b] for i, (a, b) in spans.items()}
+
+    @_locked
+    def release(self, seq_id) -> None:
+        """Give back what a sequence of :meth:`feed` holds."""
+        self.kv.free_sequence(seq_id)
 
     def _draft_prefill(self, r: Request):
         """Bring the draft model's cache level with the target's for a sequence that just finished
@@ -423,22 +522,7 @@ class InferenceEngine:
         if self.spec is not None and self._use_speculation(reqs):
             self._resolve_inflight(produced)
             return self._execute_speculative(reqs, produced)
-        # a request that ended on an EOS found since scheduling needs no further token
-        reqs = [r for r in reqs if not (r.output_tokens and r.output_tokens[-1] != self.PLACEHOLDER and r.is_finished)]
-        live = []
-        for r in reqs:
-            if r.request_id not in self.kv.tables:
-                continue                    # preempted a moment ago to make room for an older request
-            try:
-                room = self._append_token_making_room(r, live, produced)
-                if room is None:
-                    continue                # r itself was the newest holder of blocks: preempted, it retries later
-                if not room:
-                    raise RuntimeError("KV cache exhausted during decode")
-                live.append(r)
-            except Exception as e:  # noqa: BLE001
-                self._resolve_inflight(produced)
-                self._fail(r, e)
+        live = self._reserve_decode(reqs, produced)
         if not live:
             return
         # on a GPU by default; "force" runs the same bookkeeping on the CPU too (tests of the one-step-late logic)
@@ -492,6 +576,26 @@ class InferenceEngine:
         self._resolve_inflight(produced)
         self._inflight = {"reqs": live, "rows": {r.request_id: i for i, r in enumerate(live)}, "slots": slots,
                           "ids_dev": ids_dev, "host_ids": host_ids, "host_lps": host_lps, "event": ev}
+
+    def _reserve_decode(self, reqs: List[Request], produced: Dict[str, List[int]]) -> List[Request]:
+        """Reserve the page slot of every request's next token; returns the requests that got one."""
+        # a request that ended on an EOS found since scheduling needs no further token
+        reqs = [r for r in reqs if not (r.output_tokens and r.output_tokens[-1] != self.PLACEHOLDER and r.is_finished)]
+        live: List[Request] = []
+        for r in reqs:
+            if r.request_id not in self.kv.tables:
+                continue                    # preempted a moment ago to make room for an older request
+            try:
+                room = self._append_token_making_room(r, live, produced)
+                if room is None:
+                    continue                # r itself was the newest holder of blocks: preempted, it retries later
+                if not room:
+                    raise RuntimeError("KV cache exhausted during decode")
+                live.append(r)
+            except Exception as e:  # noqa: BLE001
+                self._resolve_inflight(produced)
+                self._fail(r, e)
+        return live
 
     def _append_token_making_room(self, r: Request, live: List[Request], produced: Dict[str, List[int]]):
         """Reserve the KV slot of ``r``'s next token.  When the pool is dry: first the prefix cache gives up blocks, then
@@ -549,11 +653,14 @@ class InferenceEngine:
         size = gr.padded_size(len(live))
         width = self._graph_table_width()
         ctx = self.runner.prepare_decode(ids, pad_to=size, max_blocks=width)
+        hooks = self.runner if hasattr(self.runner, "graph_inputs") else None
         if ctx.block_tables.shape[1] > width or size is None:
             return self.runner.forward(last, self.runner.prepare_decode(ids))   # longer than the graphs cover
         plan = self._graph_split_plan(width)
         if not gr.has(size):
             def make(n):
+                if hooks is not None:
+                    return hooks.graph_inputs(n, width)
                 return {"tokens": torch.zeros(n, dtype=torch.long, device=self.device),
                         "positions": torch.zeros(n, dtype=torch.int32, device=self.device),
                         "block_tables": torch.full((n, width), -1, dtype=torch.int32, device=self.device),
@@ -562,6 +669,8 @@ class InferenceEngine:
                         "slots": torch.full((n,), -1, dtype=torch.int32, device=self.device)}
 
             def fn(inp):
+                if hooks is not None:
+                    return self.runner.forward(inp["tokens"], hooks.graph_context(inp, width))
                 from .context import InferenceContext
                 c = InferenceContext(False, inp["tokens"].shape[0], inp["block_tables"], inp["context_lens"],
                                      width * self.config.block_size, inp["segments"], positions=inp["positions"],
@@ -571,6 +680,8 @@ class InferenceEngine:
         tokens = torch.zeros(size, dtype=torch.long, device=self.device)
         tokens[:len(live)] = last
         self.stats["graph_replays"] += 1
+        if hooks is not None:
+            return gr.replay(size, {"tokens": tokens, **hooks.graph_values(ctx)})
         return gr.replay(size, {"tokens": tokens, "positions": ctx.positions, "block_tables": ctx.block_tables,
                                 "context_lens": ctx.context_lens, "segments": ctx.store_segments,
                                 "slots": ctx.slot_mapping})
@@ -790,10 +901,15 @@ class InferenceEngine:
     @torch.no_grad()
     def load_weights(self, named_tensors) -> int:
         """Copy HF-named tensors into the live model *in place* (captured graphs keep working)."""
+        self._resolve_inflight()            # the launch in flight reads the weights: let it finish first
+        if hasattr(self.model, "checkpoint"):
+            items = named_tensors.items() if isinstance(named_tensors, dict) else named_tensors
+            n, _ = registry.load_slots(self.model, items, strict=False)
+            self.on_weights_updated()
+            return n
         from ..model.hf_io import hf_named_tensors
         mine = dict(hf_named_tensors(self.model))
         n = 0
-        self._resolve_inflight()            # the launch in flight reads the weights: let it finish first
         for k, v in (named_tensors.items() if isinstance(named_tensors, dict) else named_tensors):
             if k in mine:
                 mine[k].copy_(v.to(mine[k].dtype))

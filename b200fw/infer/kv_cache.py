@@ -10,7 +10,7 @@ from __future__ import annotations
 
 from collections import deque
 from dataclasses import dataclass
-from typing import Deque, Dict, List, Optional
+from typing import Deque, Dict, List, Optional, Tuple
 
 import torch
 
@@ -52,7 +52,11 @@ class Block:
 class BlockPool:
     def __init__(self, num_blocks: int, block_size: int, num_layers: int, num_kv_heads: int, head_dim: int,
                  dtype: torch.dtype = torch.bfloat16, device="cpu", kv_cache_dtype: str = "fp16",
-                 allocate: bool = True, cache_dtype: Optional[str] = None):
+                 allocate: bool = True, cache_dtype: Optional[str] = None,
+                 layer_shapes: Optional[List[Optional[Tuple[int, int, int]]]] = None):
+        """``layer_shapes``: for a model whose layers differ, one ``(kv heads, key size, value size)`` per layer (None: a
+        layer without pages); every layer then has its own K and V tensor ``[blocks, block_size, heads, size]``, and block
+        ``i`` is the same tokens in all of them."""
         kv_cache_dtype = cache_dtype if cache_dtype is not None else kv_cache_dtype     # `cache_dtype`: the reference's name
         self.num_blocks, self.block_size = num_blocks, block_size
         self.num_layers, self.num_kv_heads, self.head_dim = num_layers, num_kv_heads, head_dim
@@ -62,11 +66,20 @@ class BlockPool:
         self.free_list: Deque[int] = deque(range(num_blocks))
         self.kv: Optional[torch.Tensor] = None
         self.scales: Optional[torch.Tensor] = None
+        self.layer_shapes = layer_shapes
+        self.per_layer: List[Optional[Tuple[torch.Tensor, torch.Tensor]]] = []
         self.double_free_count = 0
         if allocate:
             self._allocate()
 
     def _allocate(self):
+        if self.layer_shapes is not None:
+            if self.fp8:
+                raise ValueError("an fp8 KV cache needs equal layers: this model's layers differ")
+            def pages(heads, size):
+                return torch.zeros((self.num_blocks, self.block_size, heads, size), dtype=self.dtype, device=self.device)
+            self.per_layer = [None if s is None else (pages(s[0], s[1]), pages(s[0], s[2])) for s in self.layer_shapes]
+            return
         shape = (2, self.num_layers, self.num_blocks, self.block_size, self.num_kv_heads, self.head_dim)
         try:
             self.kv = torch.zeros(shape, dtype=torch.uint8 if self.fp8 else self.dtype, device=self.device)
@@ -124,6 +137,8 @@ class BlockPool:
 
     # ---- storage views --------------------------------------------------------------------------------
     def layer_kv(self, layer: int):
+        if self.layer_shapes is not None:
+            return self.per_layer[layer]
         return self.kv[0, layer], self.kv[1, layer]
 
     def layer_scales(self, layer: int):
@@ -142,6 +157,40 @@ class BlockPool:
             return None
         two, L, nb, bs = self.kv.shape[:4]
         return self.kv.view(two, L, nb * bs, *self.kv.shape[4:])
+
+
+class StatePool:
+    """Recurrent state of the sequences being served: a fixed number of slots, each with the fp32 tensors of every layer
+    (``layer_shapes[layer] = {name: shape}``).  A slot belongs to one sequence from its admission until it is freed; it is
+    not cleared in between, because a sequence that starts at position 0 starts from zero whatever its slot holds."""
+
+    def __init__(self, num_slots: int, layer_shapes: List[Dict[str, Tuple[int, ...]]], device="cpu"):
+        self.num_slots, self.device = num_slots, torch.device(device)
+        self.layers = [{n: torch.zeros((num_slots, *s), dtype=torch.float32, device=self.device) for n, s in shapes.items()}
+                       for shapes in layer_shapes]
+        self.free_list: Deque[int] = deque(range(num_slots))
+        self.owner: Dict[object, int] = {}
+
+    def allocate(self, seq_id) -> Optional[int]:
+        if not self.free_list:
+            return None
+        self.owner[seq_id] = self.free_list.popleft()
+        return self.owner[seq_id]
+
+    def free(self, seq_id) -> None:
+        slot = self.owner.pop(seq_id, None)
+        if slot is not None:
+            self.free_list.append(slot)
+
+    def slot(self, seq_id) -> int:
+        return self.owner[seq_id]
+
+    @property
+    def num_free_slots(self) -> int:
+        return len(self.free_list)
+
+    def bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for l in self.layers for t in l.values())
 
 
 class BlockTable:
@@ -174,8 +223,9 @@ class BlockTable:
 
 
 class KVCacheManager:
-    def __init__(self, block_pool: BlockPool, block_size: int = 16):
-        self.pool, self.block_size = block_pool, block_size
+    def __init__(self, block_pool: BlockPool, block_size: int = 16, state: Optional[StatePool] = None):
+        """``state``: recurrent-state slots that are handed out and returned together with the block tables."""
+        self.pool, self.block_size, self.state = block_pool, block_size, state
         self.tables: Dict[object, BlockTable] = {}
         self.alloc_failures = 0
 
@@ -183,6 +233,8 @@ class KVCacheManager:
         return (num_tokens + self.block_size - 1) // self.block_size
 
     def can_allocate(self, num_tokens: int) -> bool:
+        if self.state is not None and self.state.num_free_slots == 0:
+            return False
         return self.pool.num_free_blocks >= self.blocks_needed(num_tokens) + 1   # keep one spare
 
     def allocate_for_sequence(self, seq_id, num_initial_tokens: int = 0,
@@ -190,6 +242,9 @@ class KVCacheManager:
         """New table covering ``num_initial_tokens``; ``shared_block_ids`` (a cached prefix) are
         referenced instead of allocated.  Rolls everything back and returns None when the pool runs dry."""
         assert seq_id not in self.tables, f"sequence {seq_id} already has a block table"
+        if self.state is not None and self.state.num_free_slots == 0:
+            self.alloc_failures += 1
+            return None
         table = BlockTable(self.block_size)
         for bid in shared_block_ids or []:
             table.append_block(self.pool.share(bid))
@@ -204,6 +259,8 @@ class KVCacheManager:
             table.append_block(b)
         table.num_tokens = num_initial_tokens
         self.tables[seq_id] = table
+        if self.state is not None:
+            self.state.allocate(seq_id)
         return table
 
     def ensure_capacity(self, seq_id, num_tokens: int) -> bool:
@@ -246,6 +303,8 @@ class KVCacheManager:
             return
         for b in table.blocks:
             self.pool.free(b)
+        if self.state is not None:
+            self.state.free(seq_id)
 
     def get_block_table(self, seq_id) -> List[int]:
         t = self.tables.get(seq_id)
@@ -260,7 +319,9 @@ class KVCacheManager:
             self.free_sequence(sid)
 
     def get_stats(self) -> dict:
-        return {"num_blocks": self.pool.num_blocks, "free_blocks": self.pool.num_free_blocks,
+        extra = {} if self.state is None else {"state_slots": self.state.num_slots,
+                                               "free_state_slots": self.state.num_free_slots}
+        return {**extra, "num_blocks": self.pool.num_blocks, "free_blocks": self.pool.num_free_blocks,
                 "used_blocks": self.pool.num_used_blocks, "utilization": self.pool.utilization,
                 "num_sequences": len(self.tables), "alloc_failures": self.alloc_failures,
                 "double_frees": self.pool.double_free_count}

@@ -186,8 +186,8 @@ class ModelRunner:
 
     @torch.no_grad()
     def forward(self, token_ids: torch.Tensor, ctx: InferenceContext, all_rows: bool = False,
-                split_plan: Optional[Tuple[int, int]] = None) -> torch.Tensor:
-        """Token ids ``[T]`` -> logits ``[num_seqs, V]`` of each sequence's last row (or of every row)."""
+                split_plan: Optional[Tuple[int, int]] = None, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Token ids ``[T]`` -> logits ``[num_seqs, V]`` of each sequence's last row (or of every row, or of ``rows``)."""
         m, cfg = self.model, self.cfg
         self.forward_calls += 1
         Hq, Hkv, D = cfg.num_heads, cfg.num_kv_heads, cfg.head_dim
@@ -230,7 +230,9 @@ class ModelRunner:
             x = ops.rmsnorm(h, layer.post_attention_layernorm.weight, cfg.rms_norm_eps)
             gu = ops.linear(x, layer.mlp.gate_up_proj.weight)
             h = ops.linear(ops.swiglu(gu), layer.mlp.down_proj.weight, h)
-        if ctx.is_prefill and not all_rows:
+        if rows is not None:
+            h = h.index_select(0, rows)
+        elif ctx.is_prefill and not all_rows:
             h = h.index_select(0, ctx.last_token_rows)
         h = ops.rmsnorm(h.contiguous(), m.norm.weight, cfg.rms_norm_eps)
         return m.logits_from_hidden(h)

@@ -12,9 +12,14 @@ from .loss import lm_head_cross_entropy, lm_head_logprob, grpo_token_loss, Vocab
 from .optim import sumsq, fused_adamw
 from .paged import (kv_store, kv_gather, paged_decode_attention, paged_prefill_attention, varlen_attention,
                     topp_sample)
+from .residual import embedding_f32, rmsnorm_f32, merge_norm_add, glu, rope_rows, rope_turns
+from .linear_state import retention, delta_inputs, gated_delta
+from .paged_rows import qk_norm_store, paged_attention, distance_buckets
 
 __all__ = [
     "gemm", "linear", "lora_linear", "grad_into_main", "rmsnorm", "qknorm_rope", "qknorm_rope_store", "swiglu", "embedding", "rope_tables",
     "flash_attention", "VocabShard", "valid_rows", "lm_head_cross_entropy", "lm_head_logprob", "grpo_token_loss", "sumsq",
     "fused_adamw", "kv_store", "kv_gather", "paged_decode_attention", "paged_prefill_attention", "varlen_attention", "topp_sample",
+    "embedding_f32", "rmsnorm_f32", "merge_norm_add", "glu", "rope_rows", "rope_turns", "retention", "delta_inputs",
+    "gated_delta", "qk_norm_store", "paged_attention", "distance_buckets",
 ]

@@ -42,6 +42,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
                 out.copy_(r.to(out.dtype))
             return out
         return r.to(out_dtype if a.dtype == torch.bfloat16 else a.dtype)
+    if a.dtype == torch.float32 and b.dtype == torch.float32:
+        return _gemm_f32(a, b, a_mn, b_mn, out, accumulate, residual, ext)
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16, "gemm: bf16 operands required on CUDA"
     assert a.stride(-1) == 1 and b.stride(-1) == 1 and a.dim() == 2 and b.dim() == 2
     M, K = (a.shape[1], a.shape[0]) if a_mn else (a.shape[0], a.shape[1])
@@ -71,6 +73,21 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
                                a.stride(0), b.stride(0), out.stride(0), int(a_mn), int(b_mn), flags, bn,
                                max_ctas, nv.stream_ptr())
     nv.check(rc, "gemm")
+    nv.count_launch()
+    return out
+
+
+def _gemm_f32(a, b, a_mn, b_mn, out, accumulate, residual, ext) -> torch.Tensor:
+    """``a [M,K] @ b [N,K]^T`` in true 32-bit (plain FMA kernel, no reduced-precision tensor-core mode): inference of a model
+    that was asked to run in float32."""
+    if a_mn or b_mn or residual is not None or ext is not None:
+        raise NotImplementedError("the 32-bit gemm takes [M,K] and [N,K] operands only")
+    assert a.stride(-1) == 1 and b.stride(-1) == 1 and a.dim() == 2 and b.dim() == 2 and a.shape[1] == b.shape[1]
+    if out is None:
+        out = torch.empty((a.shape[0], b.shape[0]), device=a.device, dtype=torch.float32)
+    assert out.shape == (a.shape[0], b.shape[0]) and out.stride(-1) == 1 and out.dtype == torch.float32
+    nv.check(nv.lib().b2_gemm_f32(nv.ptr(a), nv.ptr(b), nv.ptr(out), a.shape[0], b.shape[0], a.shape[1], a.stride(0),
+                                  b.stride(0), out.stride(0), int(accumulate), nv.stream_ptr()), "gemm_f32")
     nv.count_launch()
     return out
 

@@ -1,0 +1,40 @@
+"""Row layout of a batch of sequence portions: what every state-carrying or paged op needs to know about a step."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import List, Optional
+
+import torch
+
+
+def pad8(n: int) -> int:
+    """Feature counts are stored in multiples of eight (16-byte rows for bf16): padding channels hold zeros."""
+    return (n + 7) // 8 * 8
+
+
+@dataclass
+class Portions:
+    """Sequence ``s`` owns rows ``cu[s]:cu[s+1]`` of the step's activations; its first row sits at position
+    ``starts[s]`` and its recurrent state in slot ``slots[s]`` (-1: padding of a graph batch).  The first
+    ``num_short`` sequences (``short_rows`` rows) hold one or a few tokens each and take the row-by-row kernels;
+    the others take the tiled ones.  ``block_tables`` rows are padded with -1."""
+    cu: torch.Tensor                         # int32 [nseq + 1]
+    starts: torch.Tensor                     # int32 [nseq]
+    slots: torch.Tensor                      # int32 [nseq]
+    row_seq: torch.Tensor                    # int32 [M]
+    positions: torch.Tensor                  # int32 [M]
+    tiles: torch.Tensor                      # int32 [n, 4] = (sequence, first row, rows, offset in the portion), <= 16 rows
+    block_tables: torch.Tensor               # int32 [nseq, max_blocks]
+    nseq: int
+    num_short: int
+    short_rows: int
+    max_short: int                           # longest portion among the short ones
+    max_keys: int                            # longest context (tokens) of any sequence after this step
+    long_counts: Optional[List[int]] = None  # rows of each sequence past num_short (host copy)
+    long_chunks: Optional[torch.Tensor] = None   # int32 [n, 4] like tiles, 64-row chunks of the long portions
+    max_long: int = 0
+    ragged: bool = True                      # False: every sequence is one row (decode): row r is sequence r
+
+    @property
+    def rows(self) -> int:
+        return self.positions.shape[0]

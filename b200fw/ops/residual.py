@@ -1,0 +1,91 @@
+"""Ops around a 32-bit residual stream: embedding into it, RMS norm out of it, the weighted sum of two normed branches
+added to it, gated activation over column slices, rotary tables for a batch's positions.
+
+Activations and residual rows are padded to a multiple of eight columns (:func:`pad8`); the padding is zero."""
+from __future__ import annotations
+
+import math
+from typing import Optional, Tuple
+
+import torch
+
+from .. import _native as nv
+
+
+def _f32(t: torch.Tensor) -> int:
+    return int(t.dtype == torch.float32)
+
+
+def embedding_f32(ids: torch.Tensor, table: torch.Tensor, vocab: Optional[int] = None) -> torch.Tensor:
+    """Rows of ``table`` as fp32; an id outside ``[0, vocab)`` (padding rows of a graph batch) gives zeros on a GPU."""
+    if not table.is_cuda:
+        return table[ids].float()
+    x = torch.empty((ids.numel(), table.shape[1]), device=table.device, dtype=torch.float32)
+    nv.check(nv.lib().b2_embed_f32(nv.ptr(ids), nv.ptr(table), nv.ptr(x), ids.numel(), table.shape[1],
+                                   table.shape[0] if vocab is None else vocab, _f32(table), nv.stream_ptr()), "embed_f32")
+    nv.count_launch()
+    return x
+
+
+def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, n: int, eps: float, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x[rows] / sqrt(mean(x^2) + eps) * w`` in ``w``'s dtype; ``n`` real columns, ``w`` zero past them.  ``rows``
+    (int64) selects and orders the rows of ``x``."""
+    if not x.is_cuda:
+        xs = x if rows is None else x[rows]
+        r = torch.rsqrt((xs[:, :n] * xs[:, :n]).mean(-1, keepdim=True) + eps)
+        return (xs * r * w.float()).to(w.dtype)
+    M = x.shape[0] if rows is None else rows.numel()
+    h = torch.empty((M, x.shape[1]), device=x.device, dtype=w.dtype)
+    nv.check(nv.lib().b2_rmsnorm_f32(nv.ptr(x), nv.ptr(w), nv.ptr(h), nv.ptr(rows), M, x.shape[1], n,
+                                     nv.ctypes.c_float(eps), _f32(w), nv.stream_ptr()), "rmsnorm_f32")
+    nv.count_launch()
+    return h
+
+
+def merge_norm_add(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, coef: float,
+                   n: int, eps: float, w_next: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """In place ``x += coef * (rms(a) wa + rms(b) wb)`` (``a``, ``b``, ``x`` fp32); returns ``rms(x) w_next`` when the
+    next norm's weight is given."""
+    if not x.is_cuda:
+        def rms(t):
+            return t * torch.rsqrt((t[:, :n] * t[:, :n]).mean(-1, keepdim=True) + eps)
+        x += coef * (rms(a) * wa.float() + rms(b) * wb.float())
+        return None if w_next is None else (rms(x) * w_next.float()).to(w_next.dtype)
+    h = None if w_next is None else torch.empty(x.shape, device=x.device, dtype=w_next.dtype)
+    nv.check(nv.lib().b2_merge_norm_add(nv.ptr(x), nv.ptr(a), nv.ptr(b), nv.ptr(wa), nv.ptr(wb), nv.ptr(w_next), nv.ptr(h),
+                                        x.shape[0], x.shape[1], n, nv.ctypes.c_float(coef), nv.ctypes.c_float(eps),
+                                        _f32(wa), nv.stream_ptr()), "merge_norm_add")
+    nv.count_launch()
+    return h
+
+
+def glu(gate: torch.Tensor, up: torch.Tensor, out: torch.Tensor) -> None:
+    """``out = silu(gate) * up``; the three are column slices (``gate`` and ``up`` of one matrix)."""
+    if not gate.is_cuda:
+        g = gate.float()
+        out.copy_((g * torch.sigmoid(g) * up.float()).to(out.dtype))
+        return
+    assert gate.stride(0) == up.stride(0)
+    nv.check(nv.lib().b2_glu(nv.ptr(gate), nv.ptr(up), nv.ptr(out), gate.shape[0], gate.shape[1], gate.stride(0),
+                             out.stride(0), _f32(gate), nv.stream_ptr()), "glu")
+    nv.count_launch()
+
+
+def rope_turns(base: float, dims: int, device) -> torch.Tensor:
+    """``base^(-2 i / dims) / (2 pi)`` for i < dims / 2, in double precision."""
+    return torch.tensor([base ** (-2.0 * i / dims) / (2.0 * math.pi) for i in range(dims // 2)], dtype=torch.float64,
+                        device=device)
+
+
+def rope_rows(positions: torch.Tensor, turns: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """fp32 ``cos`` / ``sin`` ``[rows, dims/2]`` of every row's position: no table bounds the context length."""
+    M, half = positions.numel(), turns.numel()
+    if not positions.is_cuda:
+        a = positions.double()[:, None] * turns[None, :] * (2.0 * math.pi)
+        return a.cos().float(), a.sin().float()
+    cs = torch.empty((M, half), device=positions.device, dtype=torch.float32)
+    sn = torch.empty_like(cs)
+    nv.check(nv.lib().b2_rope_rows(nv.ptr(positions), nv.ptr(turns), nv.ptr(cs), nv.ptr(sn), M, half, nv.stream_ptr()),
+             "rope_rows")
+    nv.count_launch()
+    return cs, sn

@@ -1,0 +1,333 @@
+// Paged attention one query row at a time, for any head sizes up to 256, in bf16 or true 32-bit: the decode step and short
+// portions.  Beside plain causal attention it takes, each optional,
+//   * chunked visibility: row at position i sees keys floor(i / chunk) * chunk .. i only;
+//   * a learned additive bias per head and distance bucket: rel[bucket[min(i - j, len - 1)], h];
+//   * a softmax sink per head: exp(sink_h) joins the denominator, with no key and no value;
+//   * an output gate per head: the head's output times sigmoid(gate).
+// And the stage before it: per-head RMS norm of q and k and the store of k and v into their pages.
+//
+// Cache layout of one layer: K [blocks, 16, G, dkp], V [blocks, 16, G, dvp] in the activation type, head sizes padded to a
+// multiple of eight (padding zero).  Row r belongs to sequence row_seq[r], whose pages are block_tables[row_seq[r]][*].
+#include "host.h"
+#include "vec.cuh"
+
+namespace b2 {
+
+constexpr int AR_PAGE = 16;
+constexpr int AR_THREADS = 128;
+constexpr int AR_UNROLL = 4;
+constexpr float AR_LOG2E = 1.4426950408889634f;
+
+struct AttnRowsParams {
+  const void* q;         // T [M, H * dkp]
+  const void* kc;
+  const void* vc;
+  const int* tables;     // [nseq, max_blocks]
+  const int* row_seq;    // [M] or null: row r is sequence r
+  const int* pos;        // [M]
+  const int* slot;       // per sequence, or null: slot < 0 marks a padding row (output zero)
+  const void* gate;      // T [M, ld_gate]: H columns, or null
+  const void* sink;      // T [H] or null
+  const void* rel;       // T [buckets, H] or null
+  const int* bucket;     // [nbucket]
+  void* out;             // T [M, ld_out]
+  float* part_o;         // [M, H, nsplit, dvp]
+  float* part_ml;        // [M, H, nsplit, 2]
+  long long ld_gate, ld_out;
+  int max_blocks, H, G, dkp, dvp, chunk, nbucket, partition, nsplit, groups;
+  float scale;
+};
+
+template <typename T>
+__device__ __forceinline__ float ar_finish(const AttnRowsParams& p, int head, size_t row, float o, float L, float M2) {
+  // M2: running maximum in the base-2 domain
+  if (p.sink) {
+    const float s2 = to_f(static_cast<const T*>(p.sink)[head]) * AR_LOG2E;
+    const float m = fmaxf(M2, s2);
+    const float w = M2 == -INFINITY ? 0.f : exp2f(M2 - m);
+    L = L * w + exp2f(s2 - m);
+    o *= w;
+  }
+  o = L > 0.f ? o / L : 0.f;
+  if (p.gate) o *= sigmoid_f(to_f(static_cast<const T*>(p.gate)[row * p.ld_gate + head]));
+  return o;
+}
+
+// Grid (M, G * groups, nsplit).  A key row is spread over LPT lanes, eight channels each, so one warp-wide step covers
+// 32 / LPT tokens; every lane group runs its own online softmax over the tokens it sees for the GH query heads of this CTA,
+// and groups and warps are merged at the end with the exact log-sum-exp rule.
+template <typename T, int LPT, int GH>
+__global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsParams p) {
+  constexpr int TPW = 32 / LPT, U = AR_UNROLL;
+  __shared__ float sAcc[AR_THREADS / 32][GH][LPT * 8];
+  __shared__ float sM[AR_THREADS / 32][GH], sL[AR_THREADS / 32][GH];
+  const size_t row = blockIdx.x;
+  const int kvh = blockIdx.y / p.groups, hg = blockIdx.y % p.groups, split = blockIdx.z;
+  const int per = p.H / p.G;
+  const int nh = min(GH, per - hg * GH);
+  const int head0 = kvh * per + hg * GH;
+  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row);
+  const bool live = p.slot == nullptr || p.slot[s] >= 0;
+  const int pos = p.pos[row];
+  const int first = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+  const int t_begin = first + split * p.partition;
+  const int t_end = live ? min(pos + 1, t_begin + p.partition) : t_begin;
+  const int* table = p.tables + static_cast<size_t>(s) * p.max_blocks;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, group = lane / LPT, sub = lane % LPT;
+  const bool kin = sub * 8 < p.dkp, vin = sub * 8 < p.dvp;
+  const T* kc = static_cast<const T*>(p.kc) + static_cast<size_t>(kvh) * p.dkp + sub * 8;
+  const T* vc = static_cast<const T*>(p.vc) + static_cast<size_t>(kvh) * p.dvp + sub * 8;
+  const size_t kts = static_cast<size_t>(p.G) * p.dkp, vts = static_cast<size_t>(p.G) * p.dvp;
+
+  float qr[GH][8], acc[GH][8], m[GH], l[GH];
+#pragma unroll
+  for (int g = 0; g < GH; ++g) {
+    float t[8] = {};
+    if (kin && g < nh) vload8(static_cast<const T*>(p.q) + (row * p.H + head0 + g) * p.dkp + sub * 8, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      qr[g][e] = t[e] * (p.scale * AR_LOG2E);
+      acc[g][e] = 0.f;
+    }
+    m[g] = -INFINITY;
+    l[g] = 0.f;
+  }
+  constexpr int STEP = (AR_THREADS / 32) * TPW * U;
+  for (int base = t_begin + warp * (TPW * U); base < t_end; base += STEP) {
+    float kf[U][8], vf[U][8], sc[U][GH];
+    bool valid[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int tok = base + u * TPW + group;
+      valid[u] = tok < t_end;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) kf[u][e] = vf[u][e] = 0.f;
+      if (valid[u]) {
+        const size_t at = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
+        if (kin) vload8(kc + at * kts, kf[u]);
+        if (vin) vload8(vc + at * vts, vf[u]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int tok = base + u * TPW + group;
+      int b = 0;
+      if (p.rel && valid[u]) b = p.bucket[min(pos - tok, p.nbucket - 1)];
+#pragma unroll
+      for (int g = 0; g < GH; ++g) {
+        float d = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) d = fmaf(qr[g][e], kf[u][e], d);
+#pragma unroll
+        for (int o = LPT / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+        if (p.rel && valid[u] && g < nh)
+          d = fmaf(to_f(static_cast<const T*>(p.rel)[static_cast<size_t>(b) * p.H + head0 + g]), AR_LOG2E, d);
+        sc[u][g] = valid[u] ? d : -INFINITY;
+      }
+    }
+#pragma unroll
+    for (int g = 0; g < GH; ++g) {
+      float mn = m[g];
+#pragma unroll
+      for (int u = 0; u < U; ++u) mn = fmaxf(mn, sc[u][g]);
+      if (mn == -INFINITY) continue;   // this lane group has not seen a token yet
+      const float alpha = exp2f(m[g] - mn);
+      m[g] = mn;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[g][e] *= alpha;
+      float ps = 0.f;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const float w = exp2f(sc[u][g] - mn);
+        ps += w;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[g][e] = fmaf(w, vf[u][e], acc[g][e]);
+      }
+      l[g] = l[g] * alpha + ps;
+    }
+  }
+#pragma unroll
+  for (int o = LPT; o < 32; o <<= 1)
+#pragma unroll
+    for (int g = 0; g < GH; ++g) {
+      const float mo = __shfl_xor_sync(0xffffffffu, m[g], o), lo = __shfl_xor_sync(0xffffffffu, l[g], o);
+      const float mn = fmaxf(m[g], mo);
+      const float wa = m[g] == -INFINITY ? 0.f : exp2f(m[g] - mn), wb = mo == -INFINITY ? 0.f : exp2f(mo - mn);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[g][e] = acc[g][e] * wa + __shfl_xor_sync(0xffffffffu, acc[g][e], o) * wb;
+      l[g] = l[g] * wa + lo * wb;
+      m[g] = mn;
+    }
+  if (group == 0)
+#pragma unroll
+    for (int g = 0; g < GH; ++g) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sAcc[warp][g][sub * 8 + e] = acc[g][e];
+      if (sub == 0) {
+        sM[warp][g] = m[g];
+        sL[warp][g] = l[g];
+      }
+    }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nh * p.dvp; i += AR_THREADS) {
+    const int g = i / p.dvp, c = i % p.dvp, head = head0 + g;
+    float M = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < AR_THREADS / 32; ++w) M = fmaxf(M, sM[w][g]);
+    float L = 0.f, o = 0.f;
+#pragma unroll
+    for (int w = 0; w < AR_THREADS / 32; ++w) {
+      const float wt = sM[w][g] == -INFINITY ? 0.f : exp2f(sM[w][g] - M);
+      L += sL[w][g] * wt;
+      o += sAcc[w][g][c] * wt;
+    }
+    if (p.nsplit == 1) {
+      static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(head) * p.dvp + c] = from_f<T>(ar_finish<T>(p, head, row, o, L, M));
+    } else {
+      const size_t at = (row * p.H + head) * p.nsplit + split;
+      p.part_o[at * p.dvp + c] = o;
+      if (c == 0) {
+        p.part_ml[at * 2] = M;
+        p.part_ml[at * 2 + 1] = L;
+      }
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) attn_rows_merge_kernel(const AttnRowsParams p) {
+  const size_t row = blockIdx.x;
+  const int head = blockIdx.y;
+  const size_t at = (row * p.H + head) * p.nsplit;
+  float M = -INFINITY;
+  for (int i = 0; i < p.nsplit; ++i) M = fmaxf(M, p.part_ml[(at + i) * 2]);
+  for (int c = threadIdx.x; c < p.dvp; c += blockDim.x) {
+    float L = 0.f, o = 0.f;
+    for (int i = 0; i < p.nsplit; ++i) {
+      const float mi = p.part_ml[(at + i) * 2];
+      if (mi == -INFINITY) continue;
+      const float w = exp2f(mi - M);
+      L += p.part_ml[(at + i) * 2 + 1] * w;
+      o += p.part_o[(at + i) * p.dvp + c] * w;
+    }
+    static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(head) * p.dvp + c] = from_f<T>(ar_finish<T>(p, head, row, o, L, M));
+  }
+}
+
+// Per-head RMS norm of q and k (optional weights) and the store of k / v.  Grid (M, ceil((H + 2 G) / 4)), one warp per head.
+template <typename T>
+__global__ void __launch_bounds__(128) qk_norm_store_kernel(const T* __restrict__ q, const T* __restrict__ k,
+                                                            const T* __restrict__ v, long long ld, T* __restrict__ q_out,
+                                                            T* __restrict__ kc, T* __restrict__ vc,
+                                                            const int* __restrict__ tables, const int* __restrict__ row_seq,
+                                                            const int* __restrict__ pos, const int* __restrict__ slot,
+                                                            int max_blocks, int H, int G, int dk, int dkp, int dvp,
+                                                            const T* __restrict__ wq, const T* __restrict__ wk, int norm,
+                                                            float eps) {
+  const size_t row = blockIdx.x;
+  const int w = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (w >= H + 2 * G) return;
+  const int s = row_seq ? row_seq[row] : static_cast<int>(row);
+  const bool live = slot == nullptr || slot[s] >= 0;
+  const T* src;
+  T* dst = nullptr;
+  int width = dkp;
+  if (w < H) {
+    src = q + row * ld + static_cast<size_t>(w) * dkp;
+    dst = q_out + (row * H + w) * dkp;
+  } else {
+    const int g = w < H + G ? w - H : w - H - G;
+    const int p = pos[row];
+    if (live) {
+      const size_t at = static_cast<size_t>(tables[static_cast<size_t>(s) * max_blocks + p / AR_PAGE]) * AR_PAGE + p % AR_PAGE;
+      dst = w < H + G ? kc + (at * G + g) * dkp : vc + (at * G + g) * dvp;
+    }
+    width = w < H + G ? dkp : dvp;
+    src = (w < H + G ? k + row * ld + static_cast<size_t>(g) * dkp : v + row * ld + static_cast<size_t>(g) * dvp);
+  }
+  if (dst == nullptr) return;
+  const int c = lane * 8;   // widths up to 256
+  float t[8] = {};
+  if (c < width) vload8(src + c, t);
+  if (w < H + G && norm) {
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
+    const float r = 1.f / sqrtf(warp_sum(ss) / dk + eps);
+    const T* wt = w < H ? wq : wk;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) t[e] *= wt && c + e < dk ? r * to_f(wt[c + e]) : r;
+  }
+  if (c < width) vstore8(dst + c, t);
+}
+
+template <typename T, int LPT>
+static int launch_rows(const AttnRowsParams& p, int M, int GH, cudaStream_t stream) {
+  const dim3 grid(M, p.G * p.groups, p.nsplit);
+  switch (GH) {
+    case 1: attn_rows_kernel<T, LPT, 1><<<grid, AR_THREADS, 0, stream>>>(p); break;
+    case 2: attn_rows_kernel<T, LPT, 2><<<grid, AR_THREADS, 0, stream>>>(p); break;
+    case 3: attn_rows_kernel<T, LPT, 3><<<grid, AR_THREADS, 0, stream>>>(p); break;
+    default: attn_rows_kernel<T, LPT, 4><<<grid, AR_THREADS, 0, stream>>>(p); break;
+  }
+  B2_CHECK_LAUNCH("attn_rows");
+  if (p.nsplit > 1) {
+    attn_rows_merge_kernel<T><<<dim3(M, p.H), 128, 0, stream>>>(p);
+    B2_CHECK_LAUNCH("attn_rows_merge");
+  }
+  return 0;
+}
+
+}  // namespace b2
+
+using namespace b2;
+
+// partition: keys per split, counted from the row's first visible key; nsplit * partition must cover every row's keys.
+B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const int* tables, const int* row_seq,
+                           const int* pos, const int* slot, const void* gate, long long ld_gate, const void* sink,
+                           const void* rel, const int* bucket, int nbucket, void* out, long long ld_out, float* part_o,
+                           float* part_ml, int M, int max_blocks, int H, int G, int dkp, int dvp, int chunk, int partition,
+                           int nsplit, float scale, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || dkp < 8 || dvp < 8 || nsplit < 1 ||
+      nsplit > 65535 || partition < 1 || (nsplit > 1 && (part_o == nullptr || part_ml == nullptr)) ||
+      (rel != nullptr && (bucket == nullptr || nbucket < 1)) || max_blocks < 1 || H > 65535) {
+    set_error("attn_rows: H %% G == 0 and head sizes up to 256 in multiples of 8 (padded) required");
+    return 10;
+  }
+  AttnRowsParams p = {};
+  p.q = q; p.kc = kc; p.vc = vc; p.tables = tables; p.row_seq = row_seq; p.pos = pos; p.slot = slot; p.gate = gate;
+  p.sink = sink; p.rel = rel; p.bucket = bucket; p.out = out; p.part_o = part_o; p.part_ml = part_ml; p.ld_gate = ld_gate;
+  p.ld_out = ld_out; p.max_blocks = max_blocks; p.H = H; p.G = G; p.dkp = dkp; p.dvp = dvp; p.chunk = chunk;
+  p.nbucket = nbucket; p.partition = partition; p.nsplit = nsplit; p.scale = scale;
+  const int per = H / G;
+  p.groups = (per + 3) / 4;
+  const int GH = (per + p.groups - 1) / p.groups;
+  const int w = dkp > dvp ? dkp : dvp;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  B2_DISPATCH_T(is_f32, {
+    if (w <= 64) return (launch_rows<T, 8>(p, M, GH, st));
+    if (w <= 128) return (launch_rows<T, 16>(p, M, GH, st));
+    return (launch_rows<T, 32>(p, M, GH, st));
+  });
+}
+
+B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long long ld, void* q_out, void* kc, void* vc,
+                               const int* tables, const int* row_seq, const int* pos, const int* slot, int M,
+                               int max_blocks, int H, int G, int dk, int dkp, int dvp, const void* wq, const void* wk,
+                               int norm, float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || ld % 8 || dk < 1 || dk > dkp || max_blocks < 1 || H < 1 || G < 1) {
+    set_error("qk_norm_store: head sizes up to 256 in multiples of 8 (padded) required");
+    return 10;
+  }
+  const dim3 grid(M, (H + 2 * G + 3) / 4);
+  B2_DISPATCH_T(is_f32, qk_norm_store_kernel<T><<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), ld, static_cast<T*>(q_out),
+      static_cast<T*>(kc), static_cast<T*>(vc), tables, row_seq, pos, slot, max_blocks, H, G, dk, dkp, dvp,
+      static_cast<const T*>(wq), static_cast<const T*>(wk), norm, eps););
+  B2_CHECK_LAUNCH("qk_norm_store");
+  return 0;
+}

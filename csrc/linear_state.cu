@@ -1,0 +1,391 @@
+// Linear-attention recurrences with a matrix state per head, S [key channel, value channel] in fp32, kept in per-sequence
+// slots and carried from token to token:
+//
+//   retention   S <- a_h S + k v^T                                     o = S^T q     (one fixed decay per head)
+//   delta rule  S <- g . S;  u = beta (v - S^T k);  S <- S + k u^T     o = S^T q     (one decay per head and key channel)
+//
+// followed by a per-head RMS norm over the value channels and an output gate.  This file has the token-by-token form,
+// which is the decode step, the form for short portions, and the one that runs in true 32-bit; it also has the delta
+// rule's input stage (short causal convolution, activation, unit norms, decays, step sizes).
+//
+// A portion of a sequence is a run of rows: sequence s owns rows cu[s]..cu[s+1] of the projections, its first row sits at
+// position start[s], its state in slot[s] (slot < 0: padding of a graph batch, skipped).  start == 0 means the state is
+// zero, whatever the slot holds: a slot needs no clearing between two sequences.
+#include "host.h"
+#include "vec.cuh"
+
+namespace b2 {
+
+struct StateSeqs {
+  const int* cu;
+  const int* start;
+  const int* slot;
+};
+
+struct SerialParams {
+  StateSeqs seq;
+  // retention: projection rows (T), row stride ld; delta: fp32 rows from the input stage
+  const void* q;
+  const void* k;
+  const void* v;      // T in both forms
+  const void* gate;   // retention: T; delta: fp32
+  const float* glog;  // delta: [M, H * dkp] log decays
+  const float* beta;  // delta: [M, H]
+  const float* cs;    // rotary tables [M, rot / 2] (retention)
+  const float* sn;
+  const float* decay;       // retention: [H]
+  const void* norm_w;       // T [dvp] or null
+  void* out;                // T, row stride ld_out
+  float* state;             // [slots, H, dkp, dvp]
+  long long ld_qk, ld_v, ld_gate, ld_out;
+  int H, group;             // head h uses q / k head h / group
+  int dk, dkp, dv, dvp, rot;
+  float kscale, eps;
+  int tile;                 // tokens staged at a time
+};
+
+// One CTA per (head, sequence).  A warp owns eight value columns; its lanes form four groups that split the key rows in
+// quads (lane group r holds rows 16 j + 4 r .. + 3), so the state of a head lives in registers, 4 JJ values a thread, and
+// the two reductions of a token are two shuffles.  q, k and the decays of a tile of tokens are staged in shared memory as
+// fp32 (rotated / exponentiated there once); the outputs of the tile are collected in shared memory, normed, gated, stored.
+template <typename T, int JJ, bool DELTA, int MAXT>
+__global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p) {
+  constexpr int DK = 16 * JJ;
+  extern __shared__ __align__(16) float sm[];
+  const int h = blockIdx.x, s = blockIdx.y;
+  const int slot = p.seq.slot[s];
+  const int row0 = p.seq.cu[s], count = p.seq.cu[s + 1] - row0;
+  if (slot < 0 || count <= 0) return;
+  const int TT = p.tile;
+  float* sk = sm;
+  float* sq = sk + TT * DK;
+  float* sg = sq + TT * DK;                       // delta only
+  float* sv = sg + (DELTA ? TT * DK : 0);
+  float* so = sv + TT * p.dvp;
+  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31;
+  const int rg = lane >> 3, col = warp * 8 + (lane & 7);
+  const int kvh = h / p.group;
+  float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * p.dkp * p.dvp;
+  const bool fresh = p.seq.start[s] == 0;
+
+  float S[4 * JJ];
+#pragma unroll
+  for (int j = 0; j < JJ; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = 16 * j + 4 * rg + e;
+      S[4 * j + e] = (!fresh && i < p.dkp) ? st[static_cast<size_t>(i) * p.dvp + col] : 0.f;
+    }
+  const float a = DELTA ? 0.f : p.decay[h];
+
+  for (int t0 = 0; t0 < count; t0 += TT) {
+    const int nt = min(TT, count - t0);
+    if (DELTA) {
+      const float* q = static_cast<const float*>(p.q);
+      const float* k = static_cast<const float*>(p.k);
+      for (int i = tid; i < nt * DK; i += nthr) {
+        const int t = i / DK, c = i % DK;
+        const size_t row = row0 + t0 + t;
+        const bool in = c < p.dkp;
+        sq[i] = in ? q[row * p.ld_qk + kvh * p.dkp + c] : 0.f;
+        sk[i] = in ? k[row * p.ld_qk + kvh * p.dkp + c] : 0.f;
+        sg[i] = in ? expf(p.glog[(row * p.H + h) * p.dkp + c]) : 0.f;
+      }
+    } else {
+      const T* q = static_cast<const T*>(p.q);
+      const T* k = static_cast<const T*>(p.k);
+      const int half = p.rot / 2;
+      for (int i = tid; i < nt * DK; i += nthr) {
+        const int t = i / DK, c = i % DK;
+        const size_t row = row0 + t0 + t;
+        float qv = 0.f, kv = 0.f;
+        if (c < p.dkp) {
+          const size_t at = row * p.ld_qk + kvh * p.dkp;
+          qv = to_f(q[at + c]);
+          kv = to_f(k[at + c]);
+          if (c < p.rot) {
+            const int f = c < half ? c : c - half;
+            const float cs = p.cs[row * half + f], sn = p.sn[row * half + f];
+            const int o = c < half ? c + half : c - half;
+            const float sgn = c < half ? -sn : sn;
+            qv = qv * cs + to_f(q[at + o]) * sgn;
+            kv = kv * cs + to_f(k[at + o]) * sgn;
+          }
+          kv *= p.kscale;
+        }
+        sq[i] = qv;
+        sk[i] = kv;
+      }
+    }
+    for (int i = tid; i < nt * p.dvp; i += nthr) {
+      const int t = i / p.dvp, c = i % p.dvp;
+      sv[i] = to_f(static_cast<const T*>(p.v)[static_cast<size_t>(row0 + t0 + t) * p.ld_v + static_cast<size_t>(h) * p.dvp + c]);
+    }
+    __syncthreads();
+    for (int t = 0; t < nt; ++t) {
+      const float* kt = sk + t * DK + 4 * rg;
+      const float* qt = sq + t * DK + 4 * rg;
+      float u = sv[t * p.dvp + col];
+      if (DELTA) {
+        const float* gt = sg + t * DK + 4 * rg;
+        float d0 = 0.f, d1 = 0.f;
+#pragma unroll
+        for (int j = 0; j < JJ; ++j) {
+          const float4 g = *reinterpret_cast<const float4*>(gt + 16 * j);
+          const float4 k = *reinterpret_cast<const float4*>(kt + 16 * j);
+          S[4 * j] *= g.x; S[4 * j + 1] *= g.y; S[4 * j + 2] *= g.z; S[4 * j + 3] *= g.w;
+          d0 = fmaf(S[4 * j], k.x, d0);
+          d1 = fmaf(S[4 * j + 1], k.y, d1);
+          d0 = fmaf(S[4 * j + 2], k.z, d0);
+          d1 = fmaf(S[4 * j + 3], k.w, d1);
+        }
+        float d = d0 + d1;
+        d += __shfl_xor_sync(0xffffffffu, d, 8);
+        d += __shfl_xor_sync(0xffffffffu, d, 16);
+        u = p.beta[static_cast<size_t>(row0 + t0 + t) * p.H + h] * (u - d);
+      }
+      float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < JJ; ++j) {
+        const float4 k = *reinterpret_cast<const float4*>(kt + 16 * j);
+        const float4 q = *reinterpret_cast<const float4*>(qt + 16 * j);
+        if (DELTA) {
+          S[4 * j] = fmaf(k.x, u, S[4 * j]);
+          S[4 * j + 1] = fmaf(k.y, u, S[4 * j + 1]);
+          S[4 * j + 2] = fmaf(k.z, u, S[4 * j + 2]);
+          S[4 * j + 3] = fmaf(k.w, u, S[4 * j + 3]);
+        } else {
+          S[4 * j] = fmaf(a, S[4 * j], k.x * u);
+          S[4 * j + 1] = fmaf(a, S[4 * j + 1], k.y * u);
+          S[4 * j + 2] = fmaf(a, S[4 * j + 2], k.z * u);
+          S[4 * j + 3] = fmaf(a, S[4 * j + 3], k.w * u);
+        }
+        o0 = fmaf(S[4 * j], q.x, o0);
+        o1 = fmaf(S[4 * j + 1], q.y, o1);
+        o0 = fmaf(S[4 * j + 2], q.z, o0);
+        o1 = fmaf(S[4 * j + 3], q.w, o1);
+      }
+      float o = o0 + o1;
+      o += __shfl_xor_sync(0xffffffffu, o, 8);
+      o += __shfl_xor_sync(0xffffffffu, o, 16);
+      if (rg == 0) so[t * p.dvp + col] = o;
+    }
+    __syncthreads();
+    for (int t = warp; t < nt; t += nthr >> 5) {
+      float ss = 0.f;
+      for (int c = lane; c < p.dvp; c += 32) ss = fmaf(so[t * p.dvp + c], so[t * p.dvp + c], ss);
+      const float r = 1.f / sqrtf(warp_sum(ss) / p.dv + p.eps);
+      const size_t row = row0 + t0 + t;
+      for (int c = lane; c < p.dvp; c += 32) {
+        float o = so[t * p.dvp + c] * r;
+        const size_t gi = row * p.ld_gate + static_cast<size_t>(h) * p.dvp + c;
+        if (DELTA) {
+          if (p.norm_w) o *= to_f(static_cast<const T*>(p.norm_w)[c]);
+          o *= sigmoid_f(static_cast<const float*>(p.gate)[gi]);
+        } else {
+          o *= silu_f(to_f(static_cast<const T*>(p.gate)[gi]));
+        }
+        static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(h) * p.dvp + c] = from_f<T>(o);
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int j = 0; j < JJ; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = 16 * j + 4 * rg + e;
+      if (i < p.dkp) st[static_cast<size_t>(i) * p.dvp + col] = S[4 * j + e];
+    }
+}
+
+// Input stage of the delta rule.  Grid (tiles, 2 G + H): tile = {sequence, first row, rows, offset of that row in the
+// portion}, at most PREP_TILE rows.  Roles along y: G query heads, G key heads (convolution, silu, unit norm), H value heads
+// (convolution, silu; the head's decays and step size).  The convolution's channels are laid out [q | k | v] in the
+// projection, the taps and the state alike.  Only the portion's first tile reads the sequence's convolution state (taps - 1
+// <= PREP_TILE), so that tile also replaces it, after its own reads.
+constexpr int PREP_TILE = 16;
+constexpr int PREP_THREADS = 128;
+constexpr int PREP_MAXC = 8;   // channels a lane keeps: heads up to 256 wide
+
+struct DeltaPrepParams {
+  StateSeqs seq;
+  const int* tiles;      // [n, 4]
+  const void* x;         // T rows [M, ld]: q | k | v
+  const void* taps;      // T [C, K]
+  const void* b;         // T [M, ld]: H columns
+  const float* a2;       // [M, ld_a2]: H * dkp columns
+  const void* A_log;     // T [H]
+  const void* dt_bias;   // T [H * dkp]
+  float* conv_state;     // [slots, C, K - 1]
+  float* q;              // [M, G * dkp]
+  float* k;
+  void* v;               // T [M, H * dvp]
+  float* glog;           // [M, H * dkp]
+  float* beta;           // [M, H]
+  long long ld, ld_a2;
+  int G, H, dk, dkp, dv, dvp, K;
+  float qscale, unit_eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(const DeltaPrepParams p) {
+  const int* tl = p.tiles + blockIdx.x * 4;
+  const int s = tl[0], row0 = tl[1], rows = tl[2], off = tl[3];
+  const int slot = s < 0 ? -1 : p.seq.slot[s];
+  if (slot < 0 || rows <= 0) return;
+  const int y = blockIdx.y, G = p.G, K = p.K;
+  const bool is_v = y >= 2 * G;
+  const int width = is_v ? p.dvp : p.dkp;
+  const int c0 = is_v ? 2 * G * p.dkp + (y - 2 * G) * p.dvp : y * p.dkp;
+  const int C = 2 * G * p.dkp + p.H * p.dvp;
+  const bool fresh = p.seq.start[s] == 0;
+  const T* x = static_cast<const T*>(p.x) + c0;
+  const T* taps = static_cast<const T*>(p.taps) + static_cast<size_t>(c0) * K;
+  float* cst = p.conv_state + (static_cast<size_t>(slot) * C + c0) * (K - 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  for (int t = warp; t < rows; t += PREP_THREADS / 32) {
+    const size_t row = row0 + t;
+    float val[PREP_MAXC], ss = 0.f;
+#pragma unroll
+    for (int m = 0; m < PREP_MAXC; ++m) {
+      const int c = lane + 32 * m;
+      val[m] = 0.f;
+      if (c < width) {
+        float acc = 0.f;
+        for (int j = 0; j < K; ++j) {           // j tokens back
+          const int at = off + t - j;           // index in the portion
+          float xv = 0.f;
+          if (at >= 0) xv = to_f(x[(row - j) * p.ld + c]);
+          else if (!fresh) xv = cst[static_cast<size_t>(c) * (K - 1) + (K - 1 + at)];
+          acc = fmaf(to_f(taps[static_cast<size_t>(c) * K + K - 1 - j]), xv, acc);
+        }
+        val[m] = silu_f(acc);
+        ss = fmaf(val[m], val[m], ss);
+      }
+    }
+    if (is_v) {
+      const int h = y - 2 * G;
+#pragma unroll
+      for (int m = 0; m < PREP_MAXC; ++m) {
+        const int c = lane + 32 * m;
+        if (c < width) static_cast<T*>(p.v)[(row * p.H + h) * p.dvp + c] = from_f<T>(val[m]);
+      }
+      const float A = -expf(to_f(static_cast<const T*>(p.A_log)[h]));
+      for (int c = lane; c < p.dkp; c += 32) {
+        const float z = p.a2[row * p.ld_a2 + static_cast<size_t>(h) * p.dkp + c] +
+                        to_f(static_cast<const T*>(p.dt_bias)[h * p.dkp + c]);
+        p.glog[(row * p.H + h) * p.dkp + c] = A * softplus_f(z);
+      }
+      if (lane == 0) p.beta[row * p.H + h] = sigmoid_f(to_f(static_cast<const T*>(p.b)[row * p.ld + h]));
+    } else {
+      const float r = (y < G ? p.qscale : 1.f) / sqrtf(warp_sum(ss) + p.unit_eps);
+      float* dst = (y < G ? p.q : p.k) + (row * G + (y < G ? y : y - G)) * p.dkp;
+#pragma unroll
+      for (int m = 0; m < PREP_MAXC; ++m) {
+        const int c = lane + 32 * m;
+        if (c < width) dst[c] = val[m] * r;
+      }
+    }
+  }
+  if (off != 0 || K < 2) return;
+  __syncthreads();
+  const int count = p.seq.cu[s + 1] - p.seq.cu[s];
+  for (int c = threadIdx.x; c < width; c += PREP_THREADS) {
+    float* d = cst + static_cast<size_t>(c) * (K - 1);
+    for (int j = 0; j < K - 1; ++j) {
+      const int at = count - (K - 1) + j;
+      d[j] = at >= 0 ? to_f(x[(static_cast<size_t>(row0) + at) * p.ld + c]) : (fresh ? 0.f : d[j + count]);
+    }
+  }
+}
+
+template <typename T, bool DELTA>
+static int launch_serial(const SerialParams& p, int nseq, cudaStream_t stream) {
+  const int JJ = p.dkp <= 16 ? 1 : p.dkp <= 32 ? 2 : p.dkp <= 64 ? 4 : p.dkp <= 128 ? 8 : 16;
+  const int DK = 16 * JJ;
+  const size_t smem = sizeof(float) * p.tile * ((DELTA ? 3 : 2) * DK + 2 * p.dvp);
+  const dim3 grid(p.H, nseq);
+#define B2_SERIAL(J)                                                                                            \
+  do {                                                                                                          \
+    auto kern = p.dvp <= 128 ? state_serial_kernel<T, J, DELTA, 512> : state_serial_kernel<T, J, DELTA, 1024>;  \
+    if (smem > 48 * 1024)                                                                                       \
+      cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));          \
+    kern<<<grid, p.dvp * 4, smem, stream>>>(p);                                                                 \
+  } while (0)
+  if (JJ == 1) B2_SERIAL(1);
+  else if (JJ == 2) B2_SERIAL(2);
+  else if (JJ == 4) B2_SERIAL(4);
+  else if (JJ == 8) B2_SERIAL(8);
+  else B2_SERIAL(16);
+#undef B2_SERIAL
+  B2_CHECK_LAUNCH("linear_state");
+  return 0;
+}
+
+static bool bad_heads(const char* what, int H, int group, int dk, int dkp, int dv, int dvp, int nseq) {
+  if (dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || dk > dkp || dv > dvp || dk < 1 || dv < 1 || H < 1 || group < 1 ||
+      H % group || nseq > 65535) {
+    set_error("%s: head sizes up to 256 in multiples of 8 (padded) and H %% group == 0 required", what);
+    return true;
+  }
+  return false;
+}
+
+}  // namespace b2
+
+using namespace b2;
+
+B2_EXPORT int b2_retention_serial(const void* q, const void* k, const void* v, const void* gate, void* out, float* state,
+                                  const float* decay, const float* cs, const float* sn, const int* cu, const int* start,
+                                  const int* slot, int nseq, int max_rows, int H, int dk, int dkp, int dv, int dvp, int rot,
+                                  long long ld_in, long long ld_out, float kscale, float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (nseq <= 0) return 0;
+  if (bad_heads("retention", H, 1, dk, dkp, dv, dvp, nseq)) return 10;
+  if (rot < 0 || rot % 2 || rot > dk) { set_error("retention: rotary dims must be even and at most the head size"); return 10; }
+  SerialParams p = {};
+  p.seq = {cu, start, slot};
+  p.q = q; p.k = k; p.v = v; p.gate = gate; p.cs = cs; p.sn = sn; p.decay = decay; p.out = out; p.state = state;
+  p.ld_qk = p.ld_v = p.ld_gate = ld_in; p.ld_out = ld_out;
+  p.H = H; p.group = 1; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.rot = rot; p.kscale = kscale; p.eps = eps;
+  p.tile = max_rows < 16 ? (max_rows < 1 ? 1 : max_rows) : 16;
+  B2_DISPATCH_T(is_f32, return (launch_serial<T, false>(p, nseq, static_cast<cudaStream_t>(stream))););
+}
+
+B2_EXPORT int b2_delta_serial(const float* q, const float* k, const void* v, const float* glog, const float* beta,
+                              const float* gate, const void* norm_w, void* out, float* state, const int* cu, const int* start,
+                              const int* slot, int nseq, int max_rows, int H, int G, int dk, int dkp, int dv, int dvp,
+                              long long ld_gate, long long ld_out, float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (nseq <= 0) return 0;
+  if (G < 1 || H % G || bad_heads("gated_delta", H, H / (G > 0 ? G : 1), dk, dkp, dv, dvp, nseq)) return 10;
+  SerialParams p = {};
+  p.seq = {cu, start, slot};
+  p.q = q; p.k = k; p.v = v; p.gate = gate; p.glog = glog; p.beta = beta; p.norm_w = norm_w; p.out = out; p.state = state;
+  p.ld_qk = static_cast<long long>(G) * dkp; p.ld_v = static_cast<long long>(H) * dvp; p.ld_gate = ld_gate; p.ld_out = ld_out;
+  p.H = H; p.group = H / G; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.eps = eps;
+  p.tile = max_rows < 16 ? (max_rows < 1 ? 1 : max_rows) : 16;
+  B2_DISPATCH_T(is_f32, return (launch_serial<T, true>(p, nseq, static_cast<cudaStream_t>(stream))););
+}
+
+B2_EXPORT int b2_delta_prep(const void* x, const void* taps, const void* b, const float* a2, const void* A_log,
+                            const void* dt_bias, float* conv_state, float* q, float* k, void* v, float* glog, float* beta,
+                            const int* cu, const int* start, const int* slot, const int* tiles, int ntiles, int H, int G,
+                            int dk, int dkp, int dv, int dvp, int K, long long ld, long long ld_a2, float qscale,
+                            float unit_eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (ntiles <= 0) return 0;
+  if (G < 1 || H % G || bad_heads("delta_prep", H, H / (G > 0 ? G : 1), dk, dkp, dv, dvp, 1)) return 10;
+  if (K < 1 || K - 1 > PREP_TILE || 2 * G + H > 65535) { set_error("delta_prep: 1 to %d convolution taps", PREP_TILE + 1); return 10; }
+  DeltaPrepParams p = {};
+  p.seq = {cu, start, slot};
+  p.tiles = tiles; p.x = x; p.taps = taps; p.b = b; p.a2 = a2; p.A_log = A_log; p.dt_bias = dt_bias; p.conv_state = conv_state;
+  p.q = q; p.k = k; p.v = v; p.glog = glog; p.beta = beta; p.ld = ld; p.ld_a2 = ld_a2;
+  p.G = G; p.H = H; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.K = K; p.qscale = qscale; p.unit_eps = unit_eps;
+  const dim3 grid(ntiles, 2 * G + H);
+  B2_DISPATCH_T(is_f32, delta_prep_kernel<T><<<grid, PREP_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(p););
+  B2_CHECK_LAUNCH("delta_prep");
+  return 0;
+}

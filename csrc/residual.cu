@@ -1,0 +1,270 @@
+// Kernels around a 32-bit residual stream: embedding into it, RMS norm out of it, the half-sum of two normed branches
+// added to it (with the next norm in the same pass), gated activation over column slices, rotary tables for a batch's
+// positions, and the 32-bit matrix product used when a model runs without any reduced-precision mode.
+//
+// Rows of the residual and of every activation are padded to a multiple of eight columns; `n` is the real width.  The
+// padding columns are zero (their norm weights are zero), so vector accesses never need a tail.
+#include "host.h"
+#include "vec.cuh"
+
+namespace b2 {
+
+constexpr int RES_THREADS = 256;
+constexpr int RES_VEC = 4;   // 8-column pieces a thread keeps in registers (rows up to 8192 columns); longer rows are re-read
+
+__device__ __forceinline__ float res_block_sum(float v, float* scratch) {
+  v = warp_sum(v);
+  __syncthreads();   // the previous use of scratch has been read
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int lane = threadIdx.x & 31;
+  return warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? scratch[lane] : 0.f);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RES_THREADS) embed_f32_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
+                                                                float* __restrict__ x, int ld, int vocab) {
+  const long long id = ids[blockIdx.x];
+  const bool ok = id >= 0 && id < vocab;   // padding rows of a graph batch carry any id; nothing outside the table is read
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
+    float f[8] = {};
+    if (ok) vload8(table + static_cast<size_t>(id) * ld + c, f);
+    vstore8(x + static_cast<size_t>(blockIdx.x) * ld + c, f);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RES_THREADS) rmsnorm_f32_kernel(const float* __restrict__ x, const T* __restrict__ w,
+                                                                  T* __restrict__ h, const long long* __restrict__ rows, int ld,
+                                                                  int n, float eps) {
+  __shared__ float scratch[32];
+  const size_t src = rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
+  const float* xr = x + src * ld;
+  T* hr = h + static_cast<size_t>(blockIdx.x) * ld;
+  float v[RES_VEC][8], ss = 0.f;
+  int i = 0;
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8, ++i) {
+    float t[8];
+    vload8(xr + c, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
+#pragma unroll
+    for (int k = 0; k < RES_VEC; ++k)
+      if (k == i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = t[e];
+  }
+  const float r = 1.f / sqrtf(res_block_sum(ss, scratch) / n + eps);
+  i = 0;
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8, ++i) {
+    float t[8], wv[8];
+    if (i >= RES_VEC) vload8(xr + c, t);
+#pragma unroll
+    for (int k = 0; k < RES_VEC; ++k)
+      if (k == i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) t[e] = v[k][e];
+    vload8(w + c, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) t[e] *= r * wv[e];
+    vstore8(hr + c, t);
+  }
+}
+
+// x += coef * (rms(a) wa + rms(b) wb); h = rms(x) w_next when w_next is given.  a, b: fp32 [M, ld].
+template <typename T>
+__global__ void __launch_bounds__(RES_THREADS) merge_norm_add_kernel(float* __restrict__ x, const float* __restrict__ a,
+                                                                     const float* __restrict__ b, const T* __restrict__ wa,
+                                                                     const T* __restrict__ wb, const T* __restrict__ w_next,
+                                                                     T* __restrict__ h, int ld, int n, float coef, float eps) {
+  __shared__ float scratch[32];
+  const size_t base = static_cast<size_t>(blockIdx.x) * ld;
+  float sa = 0.f, sb = 0.f;
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
+    float t[8], u[8];
+    vload8(a + base + c, t);
+    vload8(b + base + c, u);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      sa = fmaf(t[e], t[e], sa);
+      sb = fmaf(u[e], u[e], sb);
+    }
+  }
+  const float ra = coef / sqrtf(res_block_sum(sa, scratch) / n + eps);
+  const float rb = coef / sqrtf(res_block_sum(sb, scratch) / n + eps);
+  float ss = 0.f;
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
+    float t[8], u[8], f[8], va[8], vb[8];
+    vload8(a + base + c, t);
+    vload8(b + base + c, u);
+    vload8(wa + c, va);
+    vload8(wb + c, vb);
+    vload8(x + base + c, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      f[e] += t[e] * ra * va[e] + u[e] * rb * vb[e];
+      ss = fmaf(f[e], f[e], ss);
+    }
+    vstore8(x + base + c, f);
+  }
+  if (w_next == nullptr) return;
+  const float r = 1.f / sqrtf(res_block_sum(ss, scratch) / n + eps);
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {   // re-reads what this thread just wrote
+    float f[8], wv[8];
+    vload8(x + base + c, f);
+    vload8(w_next + c, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] *= r * wv[e];
+    vstore8(h + base + c, f);
+  }
+}
+
+// out = silu(gate) * up over column slices (row strides ld_in / ld_out)
+template <typename T>
+__global__ void __launch_bounds__(RES_THREADS) glu_kernel(const T* __restrict__ gate, const T* __restrict__ up,
+                                                          T* __restrict__ out, int ld_in, int ld_out, int nvec, long long total) {
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long row = i / nvec;
+    const int c = static_cast<int>(i - row * nvec) * 8;
+    float g[8], u[8];
+    vload8(gate + row * ld_in + c, g);
+    vload8(up + row * ld_in + c, u);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = silu_f(g[e]) * u[e];
+    vstore8(out + row * ld_out + c, g);
+  }
+}
+
+// cos / sin of position * freq, the angle reduced in double precision: turns[i] = freq_i / (2 pi).
+__global__ void __launch_bounds__(RES_THREADS) rope_rows_kernel(const int* __restrict__ pos, const double* __restrict__ turns,
+                                                                float* __restrict__ cs, float* __restrict__ sn, int half,
+                                                                int total) {
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < total; i += gridDim.x * blockDim.x) {
+    const double t = static_cast<double>(pos[i / half]) * turns[i % half];
+    float s, c;
+    sincospif(2.f * static_cast<float>(t - rint(t)), &s, &c);
+    cs[i] = c;
+    sn[i] = s;
+  }
+}
+
+// C[M,N] (+)= A[M,K] B[N,K]^T in plain fp32 FMA (64 x 64 tile, 4 x 4 per thread).
+constexpr int SG_T = 64, SG_K = 16;
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B,
+                                                       float* __restrict__ C, int M, int N, int K, int lda, int ldb, int ldc,
+                                                       int accumulate) {
+  __shared__ float sA[SG_K][SG_T + 4], sB[SG_K][SG_T + 4];
+  const int m0 = blockIdx.y * SG_T, n0 = blockIdx.x * SG_T;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += SG_K) {
+    for (int i = threadIdx.x; i < SG_T * SG_K; i += 256) {
+      const int r = i / SG_K, k = i % SG_K;
+      const bool in = k0 + k < K;
+      sA[k][r] = in && m0 + r < M ? A[static_cast<size_t>(m0 + r) * lda + k0 + k] : 0.f;
+      sB[k][r] = in && n0 + r < N ? B[static_cast<size_t>(n0 + r) * ldb + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < SG_K; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&sA[k][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&sB[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) continue;
+      float* c = C + static_cast<size_t>(m) * ldc + n;
+      *c = accumulate ? *c + acc[i][j] : acc[i][j];
+    }
+  }
+}
+
+}  // namespace b2
+
+using namespace b2;
+
+B2_EXPORT int b2_embed_f32(const long long* ids, const void* table, float* x, int M, int ld, int vocab, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8) { set_error("embed_f32: row width must be a multiple of 8"); return 10; }
+  B2_DISPATCH_T(is_f32, embed_f32_kernel<T><<<M, RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      ids, static_cast<const T*>(table), x, ld, vocab););
+  B2_CHECK_LAUNCH("embed_f32");
+  return 0;
+}
+
+B2_EXPORT int b2_rmsnorm_f32(const float* x, const void* w, void* h, const long long* rows, int M, int ld, int n, float eps,
+                             int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld) { set_error("rmsnorm_f32: ld %% 8 == 0 and 0 < n <= ld required"); return 10; }
+  B2_DISPATCH_T(is_f32, rmsnorm_f32_kernel<T><<<M, RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      x, static_cast<const T*>(w), static_cast<T*>(h), rows, ld, n, eps););
+  B2_CHECK_LAUNCH("rmsnorm_f32");
+  return 0;
+}
+
+B2_EXPORT int b2_merge_norm_add(float* x, const float* a, const float* b, const void* wa, const void* wb, const void* w_next,
+                                void* h, int M, int ld, int n, float coef, float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld) { set_error("merge_norm_add: ld %% 8 == 0 and 0 < n <= ld required"); return 10; }
+  B2_DISPATCH_T(is_f32, merge_norm_add_kernel<T><<<M, RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      x, a, b, static_cast<const T*>(wa), static_cast<const T*>(wb), static_cast<const T*>(w_next), static_cast<T*>(h), ld, n,
+      coef, eps););
+  B2_CHECK_LAUNCH("merge_norm_add");
+  return 0;
+}
+
+B2_EXPORT int b2_glu(const void* gate, const void* up, void* out, int M, int cols, int ld_in, int ld_out, int is_f32,
+                     void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0 || cols <= 0) return 0;
+  if (cols % 8 || ld_in % 8 || ld_out % 8) { set_error("glu: columns and strides must be multiples of 8"); return 10; }
+  const long long total = static_cast<long long>(M) * (cols / 8);
+  long long blocks = (total + RES_THREADS - 1) / RES_THREADS;
+  const long long cap = static_cast<long long>(num_sms()) * 16;
+  if (blocks > cap) blocks = cap;
+  B2_DISPATCH_T(is_f32, glu_kernel<T><<<static_cast<int>(blocks), RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const T*>(gate), static_cast<const T*>(up), static_cast<T*>(out), ld_in, ld_out, cols / 8, total););
+  B2_CHECK_LAUNCH("glu");
+  return 0;
+}
+
+B2_EXPORT int b2_rope_rows(const int* pos, const double* turns, float* cs, float* sn, int M, int half, void* stream) {
+  b2::ensure_thread_context();
+  const long long total = static_cast<long long>(M) * half;
+  if (total <= 0) return 0;
+  if (total > 0x7fffffffll) { set_error("rope_rows: too many rows"); return 10; }
+  long long blocks = (total + RES_THREADS - 1) / RES_THREADS;
+  const long long cap = static_cast<long long>(num_sms()) * 8;
+  if (blocks > cap) blocks = cap;
+  rope_rows_kernel<<<static_cast<int>(blocks), RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      pos, turns, cs, sn, half, static_cast<int>(total));
+  B2_CHECK_LAUNCH("rope_rows");
+  return 0;
+}
+
+B2_EXPORT int b2_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldb, int ldc,
+                          int accumulate, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  const dim3 grid((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T);
+  if (grid.y > 65535) { set_error("gemm_f32: too many rows (%d)", M); return 10; }
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, B, C, M, N, K, lda, ldb, ldc, accumulate);
+  B2_CHECK_LAUNCH("gemm_f32");
+  return 0;
+}
