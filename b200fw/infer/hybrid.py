@@ -34,45 +34,20 @@ class HybridModelRunner(ModelRunner):
     # ---- metadata ----------------------------------------------------------------------------------------
     def prepare_prefill(self, seq_ids: Sequence, starts: Sequence[int], counts: Sequence[int]) -> InferenceContext:
         """Sequence ``i`` computes positions ``starts[i] .. starts[i] + counts[i] - 1`` (its pages already cover them)."""
+        p, order, place = build_portions(starts, counts, [self.mgr.get_block_table(i) for i in seq_ids],
+                                         [self.state.slot(i) for i in seq_ids], self.dtype == torch.float32, self._np)
         n = len(seq_ids)
-        serial = self.dtype == torch.float32     # 32-bit runs take the token-by-token kernels throughout
-        short = [i for i in range(n) if serial or counts[i] <= SHORT_ROWS]
-        long = [i for i in range(n) if not (serial or counts[i] <= SHORT_ROWS)]
-        order = short + long
-        c = np.asarray([counts[i] for i in order], dtype=np.int32)
-        st = np.asarray([starts[i] for i in order], dtype=np.int32)
-        cu = np.zeros(n + 1, dtype=np.int32)
-        np.cumsum(c, out=cu[1:])
-        M = int(cu[-1])
-        row_seq = np.repeat(np.arange(n, dtype=np.int32), c)
-        pos = (np.arange(M, dtype=np.int32) - cu[row_seq] + st[row_seq]).astype(np.int32)
-        tables = [self.mgr.get_block_table(seq_ids[i]) for i in order]
-        width = max(1, max((len(t) for t in tables), default=1))
-        bt = np.full((n, width), -1, dtype=np.int32)
-        for i, t in enumerate(tables):
-            bt[i, :len(t)] = t
-        slots = np.asarray([self.state.slot(seq_ids[i]) for i in order], dtype=np.int32)
-        place = None
-        if order != list(range(n)):
-            caller = np.zeros(n + 1, dtype=np.int64)
-            np.cumsum(np.asarray(counts, dtype=np.int64), out=caller[1:])
-            rows = np.concatenate([np.arange(caller[i], caller[i + 1]) for i in order])    # caller's row of kernel row r
-            place = np.empty(M, dtype=np.int64)
-            place[rows] = np.arange(M)
+        cu = np.concatenate([[0], np.cumsum([counts[i] for i in order])])
         last = np.zeros(n, dtype=np.int64)
         last[np.asarray(order, dtype=np.int64)] = cu[1:] - 1       # in the caller's sequence order, as kernel rows
-        ns = len(short)
-        p = Portions(
-            cu=self._np(cu), starts=self._np(st), slots=self._np(slots), row_seq=self._np(row_seq), positions=self._np(pos),
-            tiles=self._np(_row_tiles(cu, 0, n, TILE)), block_tables=self._np(bt), nseq=n, num_short=ns,
-            short_rows=int(cu[ns]), max_short=int(c[:ns].max()) if ns else 0, max_keys=int((st + c).max()) if n else 1,
-            long_counts=[int(x) for x in c[ns:]], long_chunks=self._np(_row_tiles(cu, ns, n, CHUNK)) if ns < n else None,
-            max_long=int(c[ns:].max()) if ns < n else 0)
+        back = None
+        if place is not None:
+            back = np.empty_like(place)
+            back[place] = np.arange(len(place))
         return InferenceContext(
-            is_prefill=True, num_seqs=n, total_q=M, max_seqlen_q=int(c.max()) if n else 0, positions=p.positions,
+            is_prefill=True, num_seqs=n, total_q=p.rows, max_seqlen_q=max(counts, default=0), positions=p.positions,
             last_token_rows=self._np(last), portions=p, block_tables=p.block_tables,
-            row_order=None if place is None else self._np(rows.astype(np.int64)),
-            row_place=None if place is None else self._np(place))
+            row_order=None if place is None else self._np(back), row_place=None if place is None else self._np(place))
 
     def prepare_decode(self, seq_ids: Sequence, pad_to: int = 0, max_blocks: int = 0) -> InferenceContext:
         """One decoded token per sequence at position ``len - 1``; rows past the sequences are padding (slot -1)."""
@@ -160,6 +135,40 @@ class HybridModelRunner(ModelRunner):
 
     def run_batch_decode(self, *a, **k):
         raise NotImplementedError("raw-tensor decode knows no state slots: use prepare_decode + forward")
+
+
+def build_portions(starts: Sequence[int], counts: Sequence[int], tables: Sequence[Sequence[int]], slots: Sequence[int],
+                   serial: bool, dev=torch.from_numpy) -> Tuple[Portions, List[int], Optional[np.ndarray]]:
+    """Row layout of one step: sequence ``i`` computes ``counts[i]`` positions from ``starts[i]``.  ``serial``: every portion
+    takes the row-by-row kernels (32-bit runs).  Returns the layout, the kernels' order of the sequences, and the kernel row of
+    every caller's row (None when the orders agree)."""
+    n = len(counts)
+    short = [i for i in range(n) if serial or counts[i] <= SHORT_ROWS]
+    order = short + [i for i in range(n) if not (serial or counts[i] <= SHORT_ROWS)]
+    c = np.asarray([counts[i] for i in order], dtype=np.int32)
+    st = np.asarray([starts[i] for i in order], dtype=np.int32)
+    cu = np.zeros(n + 1, dtype=np.int32)
+    np.cumsum(c, out=cu[1:])
+    M = int(cu[-1])
+    row_seq = np.repeat(np.arange(n, dtype=np.int32), c)
+    pos = (np.arange(M, dtype=np.int32) - cu[row_seq] + st[row_seq]).astype(np.int32)
+    bt = np.full((n, max(1, max((len(t) for t in tables), default=1))), -1, dtype=np.int32)
+    for r, i in enumerate(order):
+        bt[r, :len(tables[i])] = tables[i]
+    place = None
+    if order != list(range(n)):
+        caller = np.zeros(n + 1, dtype=np.int64)
+        np.cumsum(np.asarray(counts, dtype=np.int64), out=caller[1:])
+        place = np.empty(M, dtype=np.int64)
+        place[np.concatenate([np.arange(caller[i], caller[i + 1]) for i in order])] = np.arange(M)
+    ns = len(short)
+    p = Portions(
+        cu=dev(cu), starts=dev(st), slots=dev(np.asarray([slots[i] for i in order], dtype=np.int32)), row_seq=dev(row_seq),
+        positions=dev(pos), tiles=dev(_row_tiles(cu, 0, n, TILE)), block_tables=dev(bt), nseq=n, num_short=ns,
+        short_rows=int(cu[ns]), max_short=int(c[:ns].max()) if ns else 0, max_keys=int((st + c).max()) if n else 1,
+        long_counts=[int(x) for x in c[ns:]], long_chunks=dev(_row_tiles(cu, ns, n, CHUNK)) if ns < n else None,
+        max_long=int(c[ns:].max()) if ns < n else 0)
+    return p, order, place
 
 
 def _row_tiles(cu: np.ndarray, lo: int, hi: int, size: int) -> np.ndarray:
