@@ -425,8 +425,8 @@ def test_stop_and_abort():
     full = greedy(cfg, w, p, 8)
     eng = engine(m, eos_token_id=full[3])
     assert eng.generate([p], max_tokens=8)[0] == full[:full.index(full[3]) + 1]
-    r = eng.add_request("x", p, 50)
-    for _ in range(4):
+    r = eng.add_request("x", p, 50)          # two steps: the prompt and one more token, before the stop token
+    for _ in range(2):
         eng.step()
     assert eng.abort_request("x") and r.output_tokens == full[:len(r.output_tokens)]
     assert eng.kv.pool.num_used_blocks == 0 and eng.kv.state.num_free_slots == 4
