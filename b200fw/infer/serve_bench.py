@@ -1,0 +1,271 @@
+"""Serving throughput of a model preset (prefill and decode through the engine) and the rooflines of its kernels.
+
+Random weights, seeded synthetic prompts.  Phases are timed with CUDA events around engine steps; kernels one by one, with the
+L2 cache flushed before every launch."""
+from __future__ import annotations
+
+import random
+from typing import Callable, Dict, List, Optional, Tuple
+
+import torch
+
+from .. import _native as nv
+from .. import ops
+from ..model.registry import PRESETS, build_model
+from ..obs.profilers import measured_peaks
+from ..ops.portions import pad8
+from .config import InferenceConfig
+from .engine import InferenceEngine
+from .hybrid import build_portions
+
+DEV = "cuda"
+
+
+def _prompts(n: int, length: int, vocab: int, seed: int = 0) -> List[List[int]]:
+    r = random.Random(seed)
+    return [[r.randrange(3, vocab) for _ in range(length)] for _ in range(n)]
+
+
+def throughput(preset: str, batch: int = 256, prompt: int = 1024, new_tokens: int = 64, warmup: int = 3,
+               budget: int = 8192) -> Dict:
+    """``batch`` requests of ``prompt`` tokens, ``new_tokens`` each: tokens/s of the prompt phase and of the decode phase, and
+    the whole call from pinned host ids to host ids."""
+    mc = PRESETS[preset]
+    model = build_model(mc, dtype=torch.bfloat16, device=torch.device(DEV))
+    model.init_weights(0)
+    for p in model.parameters():
+        p.requires_grad_(False)
+    blocks = batch * (-(-(prompt + new_tokens + warmup + 2) // 16) + 1) + 64
+    eng = InferenceEngine(InferenceConfig.from_model_config(
+        mc, num_blocks=blocks, inference_mode="kv_cache", max_num_batched_tokens=budget + batch, max_prefill_tokens=budget,
+        chunk_size=2048, max_num_sequences=batch, enable_cuda_graph=True, temperature=0.0, eos_token_id=None,
+        adaptive_chunking=False), model).initialize()
+    eng.generate(_prompts(batch, prompt, mc.vocab_size, 1), warmup)           # allocator, graphs, tensor maps
+    out = {"model": preset, "params": mc.num_params(), "batch": batch, "prompt": prompt, "new_tokens": new_tokens}
+    for i, p in enumerate(_prompts(batch, prompt, mc.vocab_size)):
+        eng.add_request(f"r{i}", p, new_tokens + 1)
+    ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
+    launches = nv.launch_count
+    torch.cuda.synchronize()
+    ev[0].record()
+    while any(r.num_generated_tokens == 0 for r in eng.requests.values()):
+        eng.step()
+    ev[1].record()
+    before = sum(r.num_generated_tokens for r in eng.requests.values())
+    steps = 0
+    while eng.has_pending():
+        eng.step()
+        steps += 1
+    ev[2].record()
+    torch.cuda.synchronize()
+    pre, dec = ev[0].elapsed_time(ev[1]), ev[1].elapsed_time(ev[2])
+    made = batch * (new_tokens + 1)
+    out.update(prefill_tokens_per_s=batch * prompt / (pre * 1e-3), decode_tokens_per_s=(made - before) / (dec * 1e-3),
+               decode_ms_per_step=dec / max(1, steps), end_to_end_tokens_per_s=made / ((pre + dec) * 1e-3),
+               gpu_launches=nv.launch_count - launches, device_status=nv.read_status())
+    del eng, model
+    torch.cuda.empty_cache()
+    return out
+
+
+def prefill_once(preset: str, lengths: List[int], iters: int = 5) -> Dict:
+    """One forward pass over whole prompts (no scheduler): tokens/s by CUDA events."""
+    mc = PRESETS[preset]
+    model = build_model(mc, dtype=torch.bfloat16, device=torch.device(DEV))
+    model.init_weights(0)
+    for p in model.parameters():
+        p.requires_grad_(False)
+    eng = InferenceEngine(InferenceConfig.from_model_config(
+        mc, num_blocks=sum(-(-n // 16) for n in lengths) + 8, inference_mode="kv_cache", max_num_sequences=len(lengths)),
+        model).initialize()
+    for i, n in enumerate(lengths):
+        eng.kv.allocate_for_sequence(i, n)
+    ids = torch.tensor([t for n in lengths for t in _prompts(1, n, mc.vocab_size)[0]], device=DEV)
+    ctx = eng.runner.prepare_prefill(list(range(len(lengths))), [0] * len(lengths), lengths)
+    for _ in range(3):
+        eng.runner.forward(ids, ctx)
+    s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    s.record()
+    for _ in range(iters):
+        eng.runner.forward(ids, ctx)
+    e.record()
+    torch.cuda.synchronize()
+    ms = s.elapsed_time(e) / iters
+    return {"model": preset, "lengths": lengths, "ms": ms, "tokens_per_s": sum(lengths) / (ms * 1e-3),
+            "device_status": nv.read_status()}
+
+
+# ---- kernels ---------------------------------------------------------------------------------------------------------
+class _Timer:
+    def __init__(self, iters: int = 10):
+        self.iters, self.flush = iters, torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+        self.peaks = measured_peaks()
+        self.rows: Dict[str, Dict] = {}
+
+    def __call__(self, name: str, fn: Callable[[], None], bytes_: float, flops: float = 0.0) -> None:
+        for _ in range(3):
+            fn()
+        ms = []
+        for _ in range(self.iters):
+            self.flush.zero_()
+            s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            s.record()
+            fn()
+            e.record()
+            torch.cuda.synchronize()
+            ms.append(s.elapsed_time(e))
+        t = sorted(ms)[len(ms) // 2]
+        floor = max(bytes_ / (self.peaks["hbm_gbs"] * 1e9), flops / (self.peaks["bf16_tflops"] * 1e12)) * 1e3
+        self.rows[name] = {"us": round(t * 1e3, 1), "roofline_us": round(floor * 1e3, 1), "of_measured": round(floor / t, 3)}
+
+
+def _bf(*shape):
+    return torch.randn(*shape, device=DEV).to(torch.bfloat16) * 0.5
+
+
+def _gemm(t: _Timer, name, M, N, K, out32=False, acc=False, residual=False):
+    a, w = _bf(M, K), _bf(N, K)
+    o = torch.zeros(M, N, device=DEV, dtype=torch.float32 if out32 else torch.bfloat16)
+    r = _bf(M, N) if residual else None
+    by = 2 * (M * K + N * K) + M * N * (4 if out32 else 2) * (2 if acc else 1) + (2 * M * N if residual else 0)
+    t(name, lambda: ops.gemm(a, w, out=o, accumulate=acc, residual=r), by, 2.0 * M * N * K)
+
+
+def _layout(lengths: Optional[List[int]], batch: int, ctx: int):
+    if lengths is None:
+        starts, counts = [ctx - 1] * batch, [1] * batch
+    else:
+        starts, counts = [0] * len(lengths), list(lengths)
+    need = [-(-(s + c) // 16) for s, c in zip(starts, counts)]
+    ids, tables = torch.randperm(sum(need)).tolist(), []
+    for n in need:
+        tables.append(ids[:n])
+        ids = ids[n:]
+    p, _, _ = build_portions(starts, counts, tables, list(range(len(counts))), False,
+                             lambda a: torch.from_numpy(a).to(DEV))
+    return p, sum(need), starts, counts
+
+
+def fetelorn_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    """Every kernel of a layer at the preset's sizes: whole prompts of ``lengths`` tokens, or one decoded token for each of
+    ``batch`` sequences at ``ctx`` tokens."""
+    mc, t = PRESETS[preset], _Timer()
+    W, V = mc.hidden_size, mc.vocab_size
+    ret = next(l for l in mc.layers if l["type"] == "retention")
+    par = next(l for l in mc.layers if l["type"] == "parallel")
+    p, pages, starts, counts = _layout(lengths, batch, ctx)
+    M, n = p.rows, p.nseq
+    x, w = torch.randn(M, W, device=DEV), _bf(W)
+    t("rmsnorm_f32", lambda: ops.rmsnorm_f32(x, w, W, 1e-6), M * W * 6)
+    m, ff = ret["mixer"], ret["mlp"]["ff"]
+    H, dk, dv = m["heads"], m["dim"], m["vdim"]
+    nin = H * 2 * (dk + dv) + 2 * ff
+    _gemm(t, "gemm in (retention + ff)", M, nin, W)
+    _gemm(t, "gemm out (retention + ff), += fp32", M, W, H * dv + ff, True, True)
+    y, buf = _bf(M, nin), _bf(M, H * dv + ff)
+    o = H * 2 * (dk + dv)
+    t("glu", lambda: ops.glu(y[:, o:o + ff], y[:, o + ff:], buf[:, H * dv:]), M * ff * 6)
+    turns = ops.rope_turns(1e4, m["rot"]["dims"], DEV)
+    t("rope_rows", lambda: ops.rope_rows(p.positions, turns), M * m["rot"]["dims"] * 4)
+    cs, sn = ops.rope_rows(p.positions, turns)
+    S, dec = torch.zeros(n, H, dk, dv, device=DEV), torch.tensor(m["decay"], device=DEV)
+    c = [0, H * dk, 2 * H * dk, 2 * H * dk + H * dv, o]
+    flops = M * H * (2.0 * 64 * (dk + dv) / 2 + 4.0 * dk * dv)          # chunked form, 64-token chunks
+    state = n * H * dk * dv * 4 * (1 if lengths else 2)
+    t("retention", lambda: ops.retention(*(y[:, c[i]:c[i + 1]] for i in range(4)), buf[:, :H * dv], S, p, dec, dk, dv, cs, sn,
+                                         dk ** -0.5, 1e-6), M * H * (2 * dk + 3 * dv) * 2 + state, flops if lengths else 0)
+    a, b, r = par["mixer"]["left"], par["mixer"]["right"], mc.ranks[mc.layers.index(par)]
+    ff = par["mlp"]["ff"]
+    lq, lk, lv = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"]
+    rk, rv = b["kv_heads"] * b["dim"], b["heads"] * b["vdim"]
+    nin = lq + lk + lv + pad8(a["heads"]) + 2 * rk + rv + pad8(b["heads"]) + r["decay_rank"] + r["gate_rank"] + 2 * ff
+    _gemm(t, "gemm in (parallel + ff)", M, nin, W)
+    kc, vc = _bf(pages, 16, a["kv_heads"], a["dim"]), _bf(pages, 16, a["kv_heads"], a["vdim"])
+    yy, g = _bf(M, lq + lk + lv), _bf(M, a["heads"])
+    t("qk_norm_store", lambda: ops.qk_norm_store(yy[:, :lq], yy[:, lq:lq + lk], yy[:, lq + lk:], kc, vc, p, a["heads"], a["dim"],
+                                                 True, 1e-6), M * (lq + lk + lv) * 4)
+    q = ops.qk_norm_store(yy[:, :lq], yy[:, lq:lq + lk], yy[:, lq + lk:], kc, vc, p, a["heads"], a["dim"], True, 1e-6)
+    rel, sink = _bf(r["bias_rows"], a["heads"]), _bf(a["heads"])
+    chunk = a["mask"]["size"]
+    bucket = ops.distance_buckets(r["bias_rows"], a["bias_max"], min(chunk, a["bias_max"] + 1), DEV)
+    att = _bf(M, a["heads"] * a["vdim"])
+    seen = 0                                                             # query-key pairs
+    for s, k in zip(starts, counts):
+        seen += sum((i % chunk) + 1 for i in range(s, s + k))
+    by = M * (lq + a["heads"] * a["vdim"]) * 2 + (seen if lengths is None else M) * (lk + lv) * 2
+    t("paged_attention", lambda: ops.paged_attention(q, kc, vc, att, p, a["heads"], a["scale"], chunk, rel, bucket, sink, g), by,
+      2.0 * seen * a["heads"] * (a["dim"] + a["vdim"]))
+    _gemm(t, "gemm left o (fp32)", M, W, a["heads"] * a["vdim"], True)
+    low = r["decay_rank"] + r["gate_rank"]
+    H, G, dk, dv = b["heads"], b["kv_heads"], b["dim"], b["vdim"]
+    _gemm(t, "gemm low-rank second (fp32)", M, H * (dk + dv), low, True)
+    C = 2 * G * dk + H * dv
+    xx, taps, bb, z = _bf(M, C + 8), _bf(C, b["conv"]), None, torch.randn(M, H * (dk + dv), device=DEV)
+    bb = xx[:, C:C + H] if H <= 8 else _bf(M, C + 8)[:, :H]
+    A, dt, nw = _bf(H), _bf(H * dk), _bf(dv)
+    conv, S = torch.zeros(n, C, b["conv"] - 1, device=DEV), torch.zeros(n, H, dk, dv, device=DEV)
+    args = (xx[:, :C], taps, bb, z[:, :H * dk], A, dt, conv, p, G, dk, dv, dk ** -0.5)
+    outs = ops.delta_inputs(*args)
+    io = sum(t_.numel() * t_.element_size() for t_ in outs)
+    t("delta_inputs", lambda: ops.delta_inputs(*args), M * (C * 2 + H * dk * 4 + H * 2) + io)
+    out = _bf(M, H * dv)
+    flops = M * H * (2.0 * 64 * (2 * dk + 2 * dv) / 2 + 6.0 * dk * dv)
+    state = n * H * dk * dv * 4 * (1 if lengths else 2)
+    t("gated_delta", lambda: ops.gated_delta(*outs, z[:, H * dk:], nw, out, S, p, G, dk, dv, 1e-6),
+      io + M * H * dv * (4 + 2) + state, flops if lengths else 0)
+    _gemm(t, "gemm right o (fp32)", M, W, H * dv, True)
+    _gemm(t, "gemm down, += fp32", M, W, ff, True, True)
+    l32, r32 = torch.randn(M, W, device=DEV), torch.randn(M, W, device=DEV)
+    t("merge_norm_add", lambda: ops.merge_norm_add(x, l32, r32, w, w, 0.5, W, 1e-6, w), M * W * (16 + 2))
+    if lengths is None:
+        _gemm(t, "gemm logits (fp32)", M, V, W, True)
+    del t.flush
+    return t.rows
+
+
+def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    """The same for the dense decoder family."""
+    mc, t = PRESETS[preset], _Timer()
+    W, V, H, G, D, ff = mc.hidden_size, mc.vocab_size, mc.num_heads, mc.num_kv_heads, mc.head_dim, mc.intermediate_size
+    p, pages, starts, counts = _layout(lengths, batch, ctx)
+    M = p.rows
+    x, w, wd = _bf(M, W), _bf(W), _bf(D)
+    t("rmsnorm", lambda: ops.rmsnorm(x, w, 1e-6), M * W * 4)
+    nq = (H + 2 * G) * D
+    _gemm(t, "gemm qkv", M, nq, W)
+    kc, vc = _bf(pages, 16, G, D), _bf(pages, 16, G, D)
+    qkv = _bf(M, nq)
+    cos, sin = ops.rope_tables(max(ctx, max(counts)) + 1, D, mc.rope_theta, torch.device(DEV))
+    pos = p.positions
+    blk = p.block_tables[p.row_seq.long(), (pos // 16).long()]
+    slots = (blk * 16 + pos % 16).to(torch.int32)
+
+    def store():
+        return ops.qknorm_rope_store(qkv, wd, wd, pos, cos, sin, H, G, D, 1e-6, kc, vc, slots)
+    t("qknorm_rope_store", store, M * nq * 4)
+    q, k, v = store()
+    if lengths is None:
+        lens = torch.full((batch,), ctx, dtype=torch.int32, device=DEV)
+        t("paged_decode_attention", lambda: ops.paged_decode_attention(q, kc, vc, p.block_tables, lens, H),
+          batch * ctx * 2 * G * D * 2 + M * 2 * H * D * 2)
+    else:
+        cu = torch.tensor([0] + list(torch.tensor(lengths).cumsum(0)), dtype=torch.int32, device=DEV)
+        pairs = sum(n * (n + 1) / 2 for n in lengths)
+        t("paged_prefill_attention", lambda: ops.paged_prefill_attention(q, kc, vc, p.block_tables, cu, cu, max(lengths), H),
+          M * (2 * H + 2 * G) * D * 2, 4.0 * pairs * H * D)
+    _gemm(t, "gemm o (+ residual)", M, W, H * D, residual=True)
+    _gemm(t, "gemm gate_up", M, 2 * ff, W)
+    gu = _bf(M, 2 * ff)
+    t("swiglu", lambda: ops.swiglu(gu), M * ff * 6)
+    _gemm(t, "gemm down (+ residual)", M, W, ff, residual=True)
+    if lengths is None:
+        _gemm(t, "gemm logits", M, V, W)
+    del t.flush
+    return t.rows
+
+
+def kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    with torch.no_grad():
+        f = fetelorn_kernels if hasattr(PRESETS[preset], "kv_bytes_per_token") else dense_kernels
+        return f(preset, lengths, batch, ctx)

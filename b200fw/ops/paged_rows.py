@@ -94,19 +94,31 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                 o = o * torch.sigmoid(gate[r].float())[:, None]
             out[r] = o.reshape(-1).to(out.dtype)
         return
-    f32 = int(q.dtype == torch.float32)
+    lead = M
+    if p.nseq > p.num_short and dkp <= 128 and dvp <= 128 and (bucket is None or bucket.numel() <= 7680):
+        lead, ns = p.short_rows, p.num_short          # the long portions: tensor-core tiles straight over the pages
+        assert out.stride(0) % 8 == 0 and k_cache.is_contiguous() and v_cache.is_contiguous()
+        nv.check(nv.lib().b2_attn_fwd_paged_ext(
+            nv.ptr(q), nv.ptr(k_cache), nv.ptr(v_cache), nv.ptr(out), nv.ctypes.c_longlong(out.stride(0)), p.nseq - ns, H, G, dkp,
+            dvp, nblk, nv.ctypes.c_float(scale), nv.ptr(p.cu[ns:]), nv.ptr(p.starts[ns:]), nv.ptr(p.block_tables[ns:]),
+            p.block_tables.shape[1], p.max_long, M, chunk, nv.ptr(rel), nv.ptr(bucket), 0 if bucket is None else bucket.numel(),
+            nv.ptr(sink), nv.ptr(gate), nv.ctypes.c_longlong(0 if gate is None else gate.stride(0)), nv.stream_ptr()),
+            "attn_fwd_paged_ext")
+        nv.count_launch()
+    if lead == 0:
+        return
     keys = p.max_keys if chunk <= 0 else min(p.max_keys, chunk)
-    part, nsplit = _split(M, G * ((H // G + 3) // 4), keys)
+    part, nsplit = _split(lead, G * ((H // G + 3) // 4), keys)
     po = pm = None
     if nsplit > 1:
-        po = torch.empty((M, H, nsplit, dvp), device=q.device, dtype=torch.float32)
-        pm = torch.empty((M, H, nsplit, 2), device=q.device, dtype=torch.float32)
+        po = torch.empty((lead, H, nsplit, dvp), device=q.device, dtype=torch.float32)
+        pm = torch.empty((lead, H, nsplit, 2), device=q.device, dtype=torch.float32)
     nv.check(nv.lib().b2_attn_rows(
         nv.ptr(q), nv.ptr(k_cache), nv.ptr(v_cache), nv.ptr(p.block_tables), nv.ptr(p.row_seq), nv.ptr(p.positions),
         nv.ptr(p.slots), nv.ptr(gate), nv.ctypes.c_longlong(0 if gate is None else gate.stride(0)), nv.ptr(sink), nv.ptr(rel),
         nv.ptr(bucket), 0 if bucket is None else bucket.numel(), nv.ptr(out), nv.ctypes.c_longlong(out.stride(0)), nv.ptr(po),
-        nv.ptr(pm), M, p.block_tables.shape[1], H, G, dkp, dvp, chunk, part, nsplit, nv.ctypes.c_float(scale), f32,
-        nv.stream_ptr()), "attn_rows")
+        nv.ptr(pm), lead, p.block_tables.shape[1], H, G, dkp, dvp, chunk, part, nsplit, nv.ctypes.c_float(scale),
+        int(q.dtype == torch.float32), nv.stream_ptr()), "attn_rows")
     nv.count_launch(2 if nsplit > 1 else 1)
 
 

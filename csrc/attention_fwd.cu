@@ -17,6 +17,23 @@ constexpr int AT_THREADS = 352;  // warp 0 TMA, warps 1 and 10 MMA issue, warps 
 constexpr int AT_TILE_BYTES = 128 * 128 * 2;  // 32 KiB: two [128 x 64] swizzled halves
 constexpr int AT_HALF_BYTES = 128 * 64 * 2;
 
+// Options of the extended form (EXT): head sizes below 128 (the tensor maps zero-fill up to the tile), chunked visibility,
+// a learned additive bias per distance bucket, a softmax sink and an output gate per head.  Keys are always paged.
+struct FwdExt {
+  const int* start;       // [B] position of each sequence's first query row: it sees start + q_len keys in all
+  int chunk;              // > 0: a query at position i sees keys floor(i / chunk) * chunk .. i
+  const __nv_bfloat16* rel;   // [buckets, Hq] or null
+  const int* bucket;      // [nbucket]: bucket of a distance, the last entry for every larger one
+  int nbucket;
+  const __nv_bfloat16* sink;  // [Hq] or null
+  const __nv_bfloat16* gate;  // [rows, ld_gate] (Hq columns) or null
+  long long ld_gate, ld_out;
+  int dkp, dvp;           // head sizes, multiples of 8
+};
+constexpr int EXT_TAB_NEG = 256;    // table entries below distance 0 (masked keys of a diagonal tile)
+constexpr int EXT_TAB_FAR = 256;    // entries past the last bucketed distance: no clamping inside a tile
+constexpr int EXT_MAX_BUCKETS = 7680;   // the table shares the write-out staging area (32 KiB)
+
 struct AttnFwdSmem {
   // offsets into the 1024-byte aligned dynamic shared memory
   static constexpr int Q = 0;                           // 2 tiles (this item's and the next item's)
@@ -24,7 +41,7 @@ struct AttnFwdSmem {
   static constexpr int V = K + 2 * AT_TILE_BYTES;       // 2 stages
   static constexpr int EPI = V + 2 * AT_TILE_BYTES;     // 8 warps x 4 KiB write-out staging
   static constexpr int BARS = EPI + 8 * 4096;           // barriers (256 B), then the row exchange buffer (1 KiB)
-  static constexpr int TOTAL = BARS + 256 + 1024 + 1024;   // 198912
+  static constexpr int TOTAL = BARS + 256 + 1024 + 1024;   // 231680
 };
 
 // One work item: a 128-row query tile of one (batch, q head).
@@ -46,7 +63,8 @@ struct FwdParams {
 // length mode: sequence b owns query rows cu_q[b]..cu_q[b+1] and key rows cu_k[b]..cu_k[b+1]; its
 // queries are the LAST q_len positions of its kv_len keys (chunked prefill / speculative verify), so
 // query i sees keys 0..(kv_len - q_len + i).
-__device__ __forceinline__ FwdItem fwd_item(int w, const FwdParams& p) {
+template <bool EXT>
+__device__ __forceinline__ FwdItem fwd_item(int w, const FwdParams& p, const FwdExt& x_) {
   FwdItem it;
   const int hb = w % (p.Hq * p.B);
   const int x = w / (p.Hq * p.B);   // tile rank counted from the last (heaviest) tile
@@ -56,21 +74,28 @@ __device__ __forceinline__ FwdItem fwd_item(int w, const FwdParams& p) {
   const int q_begin = p.cu_q ? p.cu_q[batch] : batch * p.S;
   it.q_len = p.cu_q ? p.cu_q[batch + 1] - q_begin : p.S;
   it.k_begin = p.cu_k ? p.cu_k[batch] : batch * p.S;
-  it.kv_len = p.cu_k ? p.cu_k[batch + 1] - it.k_begin : p.S;
+  it.kv_len = EXT ? x_.start[batch] + it.q_len : p.cu_k ? p.cu_k[batch + 1] - it.k_begin : p.S;
   it.kv_off = it.kv_len - it.q_len;
   const int num_q_tiles = (it.q_len + 127) / 128;
   it.qt = num_q_tiles - 1 - x;
   it.active = it.qt >= 0 && it.q_len > 0;
   it.kvh = it.head / (p.Hq / p.Hkv);
   const int last_key = min(it.kv_len, it.kv_off + (it.qt + 1) * 128);  // exclusive
-  it.n_kv = it.active ? (last_key + 127) / 128 : 0;
+  if (EXT) {   // k_begin: first key of tile 0 (page aligned), the chunk start of the tile's first query
+    const int pos0 = it.kv_off + it.qt * 128;
+    it.k_begin = x_.chunk > 0 && it.active ? pos0 / x_.chunk * x_.chunk / 16 * 16 : 0;
+    it.n_kv = it.active ? (last_key - it.k_begin + 127) / 128 : 0;
+  } else {
+    it.n_kv = it.active ? (last_key + 127) / 128 : 0;
+  }
   it.active = it.active && it.n_kv > 0;
   it.row0 = q_begin + it.qt * 128;
   return it;
 }
-__device__ __forceinline__ int fwd_next_active(int w, int n_items, const FwdParams& p) {
+template <bool EXT>
+__device__ __forceinline__ int fwd_next_active(int w, int n_items, const FwdParams& p, const FwdExt& e) {
   int x = snake_next(w);
-  while (x < n_items && !fwd_item(x, p).active) x = snake_next(x);
+  while (x < n_items && !fwd_item<EXT>(x, p, e).active) x = snake_next(x);
   return x;
 }
 
@@ -85,10 +110,11 @@ __device__ __forceinline__ int fwd_next_active(int w, int n_items, const FwdPara
 // double-buffered in TMEM (S 2 x 128 columns, O 128, P 2 x 64 = all 512), so the softmax of tile j+1 never
 // waits for P*V of tile j unless the running maximum grew enough to force a rescale of O.  Q is double-
 // buffered in shared memory: the next item's Q arrives while the current item is still being processed.
+template <bool EXT>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
-                float* __restrict__ lse_out, const FwdParams prm, float scale, int* status) {
+                float* __restrict__ lse_out, const FwdParams prm, const FwdExt ext, float scale, int* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
@@ -107,6 +133,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   uint64_t* q_full2 = bars + 20;  // second Q slot's full barrier
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 21);
   float* xchg = reinterpret_cast<float*>(smem + AttnFwdSmem::BARS + 256);   // [2 column halves][128 rows]
+  uint64_t* tab_bar = bars + 22;   // EXT: all softmax warps, around every change of what the staging area holds
+  float* tab = reinterpret_cast<float*>(smem + AttnFwdSmem::EPI) + EXT_TAB_NEG;   // EXT: bias by distance
+  // EXT: how many 16-channel steps and 64-channel halves the head sizes need
+  const int k_steps = EXT ? (ext.dkp + 15) / 16 : 8;
+  const bool k_half2 = !EXT || ext.dkp > 64, v_half2 = !EXT || ext.dvp > 64;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int Hq = prm.Hq;
@@ -118,6 +149,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     mbar_init(&q_empty[0], 1);
     mbar_init(&q_empty[1], 1);
     mbar_init(o_free, 8);            // every softmax warp, after it has read its part of O
+    mbar_init(tab_bar, 8);
     for (int i = 0; i < 2; ++i) {
       mbar_init(&k_full[i], 1);
       mbar_init(&v_full[i], 1);
@@ -146,21 +178,27 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   const uint32_t tmem_P = tmem_base + 384;  // 2 x 64 columns: P as bf16 pairs, the A operand of P*V
 
   int w0 = blockIdx.x;
-  if (w0 < n_items && !fwd_item(w0, prm).active) w0 = fwd_next_active(w0, n_items, prm);
+  if (w0 < n_items && !fwd_item<EXT>(w0, prm, ext).active) w0 = fwd_next_active<EXT>(w0, n_items, prm, ext);
 
   if (warp == 0) {
     if (lane == 0) {
       int g = 0, n = 0;
       bool ok = true;
-      for (int w = w0; w < n_items && ok; w = fwd_next_active(w, n_items, prm), ++n) {
-        const FwdItem item = fwd_item(w, prm);
+      for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
+        const FwdItem item = fwd_item<EXT>(w, prm, ext);
         // Q slot n & 1: free once the last Q*K^T of item n-2 has retired, i.e. long before item n starts
         uint64_t* qf = (n & 1) ? q_full2 : q_full;
         uint8_t* sQ = smem + AttnFwdSmem::Q + (n & 1) * AT_TILE_BYTES;
         if (!mbar_wait(&q_empty[n & 1], ((n >> 1) & 1) ^ 1, status, ERR_ATTN_WAIT)) break;
-        mbar_expect_tx(qf, AT_TILE_BYTES);
-        tma_load_2d(sQ, &tmQ, qf, item.head * 128, item.row0);
-        tma_load_2d(sQ + AT_HALF_BYTES, &tmQ, qf, item.head * 128 + 64, item.row0);
+        if (EXT) {
+          mbar_expect_tx(qf, k_half2 ? AT_TILE_BYTES : AT_HALF_BYTES);
+          tma_load_3d(sQ, &tmQ, qf, 0, item.head, item.row0);
+          if (k_half2) tma_load_3d(sQ + AT_HALF_BYTES, &tmQ, qf, 64, item.head, item.row0);
+        } else {
+          mbar_expect_tx(qf, AT_TILE_BYTES);
+          tma_load_2d(sQ, &tmQ, qf, item.head * 128, item.row0);
+          tma_load_2d(sQ + AT_HALF_BYTES, &tmQ, qf, item.head * 128 + 64, item.row0);
+        }
         for (int j = 0; j < item.n_kv; ++j, ++g) {
           const int st = g & 1;
           const uint32_t ph = (g >> 1) & 1;
@@ -176,7 +214,23 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
             const int last_page = (item.kv_len - 1) / 16;
             int rows[8];
 #pragma unroll
-            for (int pg = 0; pg < 8; ++pg) rows[pg] = tbl[min(j * 8 + pg, last_page)] * 16;
+            for (int pg = 0; pg < 8; ++pg) rows[pg] = tbl[min((EXT ? item.k_begin / 16 : 0) + j * 8 + pg, last_page)] * 16;
+            if (EXT) {
+              mbar_expect_tx(&k_full[st], k_half2 ? AT_TILE_BYTES : AT_HALF_BYTES);
+#pragma unroll
+              for (int pg = 0; pg < 8; ++pg) {
+                tma_load_3d(sK + pg * 2048, &tmK, &k_full[st], 0, item.kvh, rows[pg]);
+                if (k_half2) tma_load_3d(sK + AT_HALF_BYTES + pg * 2048, &tmK, &k_full[st], 64, item.kvh, rows[pg]);
+              }
+              if (!mbar_wait(&v_empty[st], ph ^ 1, status, ERR_ATTN_WAIT)) { ok = false; break; }
+              mbar_expect_tx(&v_full[st], v_half2 ? AT_TILE_BYTES : AT_HALF_BYTES);
+#pragma unroll
+              for (int pg = 0; pg < 8; ++pg) {
+                tma_load_3d(sV + pg * 2048, &tmV, &v_full[st], 0, item.kvh, rows[pg]);
+                if (v_half2) tma_load_3d(sV + AT_HALF_BYTES + pg * 2048, &tmV, &v_full[st], 64, item.kvh, rows[pg]);
+              }
+              continue;
+            }
             mbar_expect_tx(&k_full[st], AT_TILE_BYTES);
 #pragma unroll
             for (int pg = 0; pg < 8; ++pg) {
@@ -208,8 +262,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     constexpr uint32_t idesc_s = make_idesc_f16(1, 128, 128, 0, 0);
     int g = 0, n = 0;
     bool ok = true;
-    for (int w = w0; w < n_items && ok; w = fwd_next_active(w, n_items, prm), ++n) {
-      const FwdItem item = fwd_item(w, prm);
+    for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
+      const FwdItem item = fwd_item<EXT>(w, prm, ext);
       if (!mbar_wait((n & 1) ? q_full2 : q_full, (n >> 1) & 1, status, ERR_ATTN_WAIT)) break;
       const uint64_t d_q = make_smem_desc_sw128(smem_u32(smem + AttnFwdSmem::Q + (n & 1) * AT_TILE_BYTES), 16, 1024);
       for (int j = 0; j < item.n_kv; ++j, ++g) {
@@ -224,6 +278,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         if (leader) {
 #pragma unroll
           for (int ks = 0; ks < 8; ++ks) {
+            if (EXT && ks >= k_steps) break;
             const uint32_t o = (ks >> 2) * AT_HALF_BYTES + (ks & 3) * 32;
             umma_f16_ss(tmem_S + st * 128, desc_advance(d_q, o), desc_advance(d_k, o), idesc_s, ks != 0);
           }
@@ -236,11 +291,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   } else if (warp == 10) {
     // ---- O += P V of every global iteration ------------------------------------------------------
     const bool leader = elect_one();
-    constexpr uint32_t idesc_pv = make_idesc_f16(1, 128, 128, 0, 1);
+    const uint32_t idesc_pv = v_half2 ? make_idesc_f16(1, 128, 128, 0, 1) : make_idesc_f16(1, 128, 64, 0, 1);
     int g = 0, n = 0;
     bool ok = true;
-    for (int w = w0; w < n_items && ok; w = fwd_next_active(w, n_items, prm), ++n) {
-      const FwdItem item = fwd_item(w, prm);
+    for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
+      const FwdItem item = fwd_item<EXT>(w, prm, ext);
       // the softmax warps must have read the previous item's O before it is overwritten
       if (n > 0 && !mbar_wait(o_free, (n - 1) & 1, status, ERR_ATTN_WAIT)) break;
       for (int j = 0; j < item.n_kv; ++j, ++g) {
@@ -270,7 +325,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const int half = (warp - 2) >> 2;         // which 64 key columns of every tile this thread handles
     const int r = quarter * 32 + lane;        // query row inside the tile
     const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
-    const float sl2 = scale * 1.4426950408889634f;
+    const float sl2_raw = scale * 1.4426950408889634f;
+    const float sl2 = EXT ? 1.f : sl2_raw;    // EXT: scores are scaled to the base-2 domain as the bias is added
     // the two threads of a row meet at a 64-thread named barrier (one per lane quarter)
     auto pair_barrier = [&]() {
       switch (quarter) {
@@ -280,13 +336,31 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         default: asm volatile("bar.sync 4, 64;" ::: "memory"); break;
       }
     };
+    uint32_t tab_phase = 0;
+    auto tab_sync = [&]() {
+      mbar_arrive_warp(tab_bar);
+      const bool done = mbar_wait_warp(tab_bar, tab_phase, status, ERR_ATTN_WAIT);
+      tab_phase ^= 1;
+      return done;
+    };
     bool ok = true;
     int g = 0, n = 0;
-    for (int w = w0; w < n_items && ok; w = fwd_next_active(w, n_items, prm), ++n) {
-      const FwdItem item = fwd_item(w, prm);
+    for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
+      const FwdItem item = fwd_item<EXT>(w, prm, ext);
       const int q_idx = item.qt * 128 + r;      // index among this sequence's queries
       const int q_pos = item.kv_off + q_idx;    // last key this query may see
-      float m_used = -INFINITY, l = 0.f;        // l: this thread's 64 columns only
+      float m_used = EXT ? -1e30f : -INFINITY, l = 0.f;        // l: this thread's 64 columns only
+      const int first_key = EXT && ext.chunk > 0 ? q_pos / ext.chunk * ext.chunk : 0;
+      if (EXT && ext.rel != nullptr) {
+        // this head's bias by distance, constant past the last bucketed one
+        // every warp has written its part of the previous item out
+        if (!tab_sync()) { ok = false; break; }
+        for (int d = static_cast<int>(threadIdx.x) - 64 - EXT_TAB_NEG; d < ext.nbucket + EXT_TAB_FAR; d += 256) {
+          const int b = ext.bucket[min(max(d, 0), ext.nbucket - 1)];
+          tab[d] = __bfloat162float(ext.rel[static_cast<size_t>(b) * Hq + item.head]) * 1.4426950408889634f;
+        }
+        if (!tab_sync()) { ok = false; break; }
+      }
       for (int j = 0; j < item.n_kv; ++j, ++g) {
         const int st = g & 1;
         const uint32_t ph = (g >> 1) & 1;
@@ -303,7 +377,33 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
         tc_fence_before();
         mbar_arrive_warp(&s_empty[st]);
-        const bool need_mask = ((j + 1) * 128 > item.kv_off + item.qt * 128 + 1) || ((j + 1) * 128 > item.kv_len);
+        if (EXT) {
+          const int key0 = item.k_begin + j * 128 + half * 64;
+          const int pos_lo = item.kv_off + item.qt * 128;           // position of the tile's first query
+          if (ext.rel != nullptr) {
+            if (pos_lo - (item.k_begin + j * 128 + 127) >= ext.nbucket - 1) {
+              const float far = tab[ext.nbucket - 1];
+#pragma unroll
+              for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], sl2_raw, far);
+            } else {
+              // distances of this tile lie in -254 .. nbucket + 252: inside the table
+              const float* tp = tab + (q_pos - key0);
+#pragma unroll
+              for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], sl2_raw, tp[-i]);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 64; ++i) s[i] *= sl2_raw;
+          }
+          const bool edge = item.k_begin + (j + 1) * 128 > pos_lo + 1 || item.k_begin + (j + 1) * 128 > item.kv_len ||
+                            (ext.chunk > 0 && item.k_begin + j * 128 < (pos_lo + 127) / ext.chunk * ext.chunk);
+          if (edge) {
+#pragma unroll
+            for (int i = 0; i < 64; ++i)
+              if (key0 + i > q_pos || key0 + i < first_key || key0 + i >= item.kv_len) s[i] = -INFINITY;
+          }
+        }
+        const bool need_mask = !EXT && (((j + 1) * 128 > item.kv_off + item.qt * 128 + 1) || ((j + 1) * 128 > item.kv_len));
         if (need_mask) {
           const int col0 = j * 128 + half * 64;
 #pragma unroll
@@ -333,6 +433,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
             const float alpha = need ? exp2f((m_used - m_new) * sl2) : 1.f;
 #pragma unroll
             for (int c = 0; c < 4; ++c) {   // this thread's 64 columns of O
+              if (EXT && half == 1 && !v_half2) break;
               uint32_t t[16];
               tmem_ld_32x32b_x16(tmem_O + lane_off + half * 64 + c * 16, t);
               tmem_ld_wait();
@@ -380,7 +481,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       pair_barrier();
       const float lsum = xchg[r] + xchg[128 + r];
       pair_barrier();
-      const float inv = 1.f / lsum;
+      float inv = 1.f / lsum;
+      if (EXT) {
+        float den = lsum;
+        if (ext.sink != nullptr) den += exp2f(fmaf(__bfloat162float(ext.sink[item.head]), 1.4426950408889634f, -m_used));
+        inv = 1.f / den;
+        if (ext.gate != nullptr && q_idx < item.q_len)
+          inv /= 1.f + expf(-__bfloat162float(ext.gate[static_cast<size_t>(item.row0 + r) * ext.ld_gate + item.head]));
+      }
       const bool in_range = q_idx < item.q_len;
       uint4 ov[8];
 #pragma unroll
@@ -400,7 +508,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           ov[c * 4 + v].w = pack_bf16x2(__uint_as_float(t[v * 8 + 6]) * inv, __uint_as_float(t[v * 8 + 7]) * inv);
         }
       }
-      {
+      if (EXT) {
+        if (ext.rel != nullptr && !tab_sync()) { ok = false; break; }   // every warp is done with the bias table
+        const int wq0 = item.qt * 128 + quarter * 32;
+        __nv_bfloat16* base = out + static_cast<size_t>(item.row0 + quarter * 32) * ext.ld_out +
+                              static_cast<size_t>(item.head) * ext.dvp + half * 64;
+        warp_store_rows_128B(smem + AttnFwdSmem::EPI + (warp - 2) * 4096, ov, [&](int row) -> uint8_t* {
+          // the lane's 16-byte piece of the row: skipped past the head's last channel
+          if (wq0 + row >= item.q_len || half * 64 + (lane & 7) * 8 >= ext.dvp) return nullptr;
+          return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * ext.ld_out);
+        });
+      } else {
         const int wq0 = item.qt * 128 + quarter * 32;   // index (within the sequence) of this warp's first query row
         __nv_bfloat16* base = out + (static_cast<size_t>(item.row0 + quarter * 32) * Hq + item.head) * 128 + half * 64;
         warp_store_rows_128B(smem + AttnFwdSmem::EPI + (warp - 2) * 4096, ov, [&](int row) -> uint8_t* {
@@ -408,7 +526,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * Hq * 128);
         });
       }
-      if (half == 0 && in_range && lse_out)
+      if (!EXT && half == 0 && in_range && lse_out)
         lse_out[static_cast<size_t>(item.head) * prm.total_q + item.row0 + r] = m_used * scale + __logf(lsum);
     }
   }
@@ -459,7 +577,7 @@ B2_EXPORT int b2_attn_fwd_varlen(const void* q, const void* k, const void* v, vo
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev]) {
-    if (cudaFuncSetAttribute(attn_fwd_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attn_fwd_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              AttnFwdSmem::TOTAL) != cudaSuccess) {
       set_error("attn_fwd: cannot set shared memory size");
       return 1;
@@ -478,8 +596,8 @@ B2_EXPORT int b2_attn_fwd_varlen(const void* q, const void* k, const void* v, vo
   prm.block_tables = nullptr; prm.max_blocks = 0;
   const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
   const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
-  attn_fwd_kernel<<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(
-      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, scale, status);
+  attn_fwd_kernel<false><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(
+      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, FwdExt{}, scale, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_error("attn_fwd launch failed: %s", cudaGetErrorString(e));
@@ -507,7 +625,7 @@ B2_EXPORT int b2_attn_fwd_paged(const void* q, const void* k_cache, const void* 
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev]) {
-    if (cudaFuncSetAttribute(attn_fwd_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attn_fwd_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              AttnFwdSmem::TOTAL) != cudaSuccess) {
       set_error("attn_fwd_paged: cannot set shared memory size");
       return 1;
@@ -527,11 +645,68 @@ B2_EXPORT int b2_attn_fwd_paged(const void* q, const void* k_cache, const void* 
   prm.block_tables = block_tables; prm.max_blocks = max_blocks;
   const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
   const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
-  attn_fwd_kernel<<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(
-      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, scale, status);
+  attn_fwd_kernel<false><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(
+      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, FwdExt{}, scale, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_error("attn_fwd_paged launch failed: %s", cudaGetErrorString(e));
+    return 4;
+  }
+  return 0;
+}
+
+// The extended form over the paged cache (see FwdExt): q [total_q, Hq * dkp], K pages [blocks, 16, Hkv, dkp], V pages
+// [blocks, 16, Hkv, dvp], out rows of stride ld_out.  cu_q: int32 [B+1] row offsets; start: int32 [B].
+B2_EXPORT int b2_attn_fwd_paged_ext(const void* q, const void* k_cache, const void* v_cache, void* out, long long ld_out, int B,
+                                    int Hq, int Hkv, int dkp, int dvp, int num_blocks, float scale, const int* cu_q,
+                                    const int* start, const int* block_tables, int max_blocks, int max_q, int total_q,
+                                    int chunk, const void* rel, const int* bucket, int nbucket, const void* sink,
+                                    const void* gate, long long ld_gate, void* stream_) {
+  b2::ensure_thread_context();
+  if (dkp < 8 || dkp > 128 || dkp % 8 || dvp < 8 || dvp > 128 || dvp % 8 || Hq < 1 || Hkv < 1 || Hq % Hkv || ld_out % 8 ||
+      block_tables == nullptr || cu_q == nullptr || start == nullptr || max_blocks <= 0 ||
+      (rel != nullptr && (bucket == nullptr || nbucket < 1 || nbucket > EXT_MAX_BUCKETS))) {
+    set_error("attn_fwd_paged_ext: head sizes up to 128 in multiples of 8, Hq %% Hkv == 0, at most %d bucketed distances", EXT_MAX_BUCKETS);
+    return 10;
+  }
+  if (B <= 0 || max_q <= 0 || total_q <= 0) return 0;
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  auto map3 = [](const void* base, uint64_t rows, uint64_t heads, uint64_t d, uint32_t box_rows) {
+    const uint64_t dims[3] = {d, heads, rows}, strides[2] = {d * 2, heads * d * 2};
+    const uint32_t box[3] = {64, 1, box_rows};
+    return tensor_map_nd_bf16(base, 3, dims, strides, box, 3);
+  };
+  const CUtensorMap* tq = map3(q, total_q, Hq, dkp, 128);
+  const CUtensorMap* tk = map3(k_cache, static_cast<uint64_t>(num_blocks) * 16, Hkv, dkp, 16);
+  const CUtensorMap* tv = map3(v_cache, static_cast<uint64_t>(num_blocks) * 16, Hkv, dvp, 16);
+  if (!tq || !tk || !tv) return 2;
+  int* status = status_ptr();
+  if (!status) return 3;
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!configured[dev]) {
+    if (cudaFuncSetAttribute(attn_fwd_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnFwdSmem::TOTAL) !=
+        cudaSuccess) {
+      set_error("attn_fwd_paged_ext: cannot set shared memory size");
+      return 1;
+    }
+    configured[dev] = true;
+  }
+  FwdParams prm;
+  prm.S = 0; prm.Hq = Hq; prm.Hkv = Hkv; prm.B = B; prm.max_tiles = (max_q + 127) / 128; prm.total_q = total_q;
+  prm.cu_q = cu_q; prm.cu_k = nullptr; prm.block_tables = block_tables; prm.max_blocks = max_blocks;
+  FwdExt e;
+  e.start = start; e.chunk = chunk; e.rel = static_cast<const __nv_bfloat16*>(rel); e.bucket = bucket; e.nbucket = nbucket;
+  e.sink = static_cast<const __nv_bfloat16*>(sink); e.gate = static_cast<const __nv_bfloat16*>(gate); e.ld_gate = ld_gate;
+  e.ld_out = ld_out; e.dkp = dkp; e.dvp = dvp;
+  const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
+  const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
+  attn_fwd_kernel<true><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(*tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), nullptr, prm, e,
+                                                            scale, status);
+  cudaError_t err = cudaGetLastError();
+  if (err != cudaSuccess) {
+    set_error("attn_fwd_paged_ext launch failed: %s", cudaGetErrorString(err));
     return 4;
   }
   return 0;

@@ -18,7 +18,7 @@ sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 import torch  # noqa: E402
 
 from b200fw.infer import InferenceConfig, InferenceEngine  # noqa: E402
-from b200fw.model import PRESETS, ParallelTransformerModel  # noqa: E402
+from b200fw.model.registry import PRESETS, build_model  # noqa: E402
 from b200fw.obs.clocks import ClockSampler  # noqa: E402
 
 
@@ -70,7 +70,7 @@ def main(argv=None):
     assert torch.cuda.is_available(), "the inference benchmark needs a GPU"
     mc = PRESETS[a.model_preset]
     dev = torch.device("cuda", 0)
-    model = ParallelTransformerModel(mc, dtype=torch.bfloat16, device=dev)
+    model = build_model(mc, dtype=torch.bfloat16, device=dev)
     model.init_weights(a.seed)
     for p in model.parameters():
         p.requires_grad_(False)

@@ -5,6 +5,7 @@
     python scripts/run_inference.py -m /path/to/Qwen3-0.6B --mode kv_cache -p "What is 2+2?" --num-samples 4 -o out.jsonl
     python scripts/run_inference.py -m /path/to/Qwen3-0.6B -i prompts.jsonl --batch-size 32 --enable-prefix-cache
     python scripts/run_inference.py --model-preset tiny128 --interactive
+    python scripts/run_inference.py -m /path/to/fetelorn --num-prompts 8 --max-tokens 64 --cuda-graph
 
 CLI after the reference's (scripts/run_inference.py:39-60); YAML keys as in configs/inference/standalone.yaml.
 """
@@ -21,13 +22,14 @@ import torch  # noqa: E402
 
 from b200fw.config import get_nested, load_yaml_config  # noqa: E402
 from b200fw.infer import InferenceConfig, InferenceEngine  # noqa: E402
-from b200fw.model import PRESETS, read_hf_config  # noqa: E402
+from b200fw.model import ModelConfig  # noqa: E402
+from b200fw.model.registry import PRESETS, read_config  # noqa: E402
 
 
 def parse_args(argv=None):
     ap = argparse.ArgumentParser(description=__doc__)
     ap.add_argument("--config", default=None, help="YAML file (configs/inference/standalone.yaml schema)")
-    ap.add_argument("--model", "-m", "--model-path", dest="model_path", default="", help="HF model directory")
+    ap.add_argument("--model", "-m", "--model-path", dest="model_path", default="", help="model directory (config.json + safetensors)")
     ap.add_argument("--model-preset", default=None, help="random-init architecture preset instead of a directory")
     ap.add_argument("--mode", choices=["kv_cache", "eager", "mock"], default=None)
     ap.add_argument("--prompt", "-p", action="append", default=None, help="text prompt (repeatable)")
@@ -52,6 +54,8 @@ def parse_args(argv=None):
     ap.add_argument("--partitioned-attention", "--enable-partitioned-attn", dest="partitioned_attention",
                     action="store_true", default=None)
     ap.add_argument("--speculative", action="store_true", default=None)
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
+                    help="float32: true 32-bit, for the architectures whose kernels have it")
     ap.add_argument("--seed", type=int, default=0)
     return ap.parse_args(argv)
 
@@ -72,10 +76,11 @@ def create_inference_config(a, y) -> InferenceConfig:
 
     preset = a.model_preset or get_nested(y, "model.preset")
     path = a.model_path or _first(y, ["model.name_or_path", "model.path"], "")
-    mc = PRESETS[preset] if preset else read_hf_config(path)
+    mc = PRESETS[preset] if preset else read_config(path)
     radix = pick(a.radix_cache, ["optimizations.radix_cache", "advanced.use_radix_cache"], False)
     kw = dict(
         inference_mode=pick(a.mode, "inference.mode", "kv_cache"), model_path="" if preset else path,
+        model_preset=preset if preset and not isinstance(mc, ModelConfig) else "", dtype=a.dtype,
         temperature=pick(a.temperature, ["sampling.temperature", "inference.temperature"], 0.7),
         top_p=pick(a.top_p, ["sampling.top_p", "inference.top_p"], 0.9),
         kv_cache_dtype=pick(a.kv_cache_dtype, "kv_cache.dtype", "fp16"),
@@ -98,7 +103,9 @@ def create_inference_config(a, y) -> InferenceConfig:
         speculative_num_tokens=get_nested(y, "speculative.num_tokens", 4), seed=a.seed)
     nb = pick(a.num_blocks, "kv_cache.num_blocks", None)
     if nb is None:
-        nb = InferenceConfig.auto_from_device(mc.num_layers, mc.num_kv_heads, mc.head_dim, kv_cache_dtype=kw["kv_cache_dtype"]).num_blocks
+        per_token = mc.kv_bytes_per_token() if hasattr(mc, "kv_bytes_per_token") else 0
+        nb = InferenceConfig.auto_from_device(mc.num_layers, mc.num_kv_heads, mc.head_dim, kv_cache_dtype=kw["kv_cache_dtype"],
+                                              bytes_per_token=per_token).num_blocks
     return InferenceConfig.from_model_config(mc, num_blocks=int(nb), **kw)
 
 
