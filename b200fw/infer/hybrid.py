@@ -18,7 +18,7 @@ from .kv_cache import BlockPool, KVCacheManager, StatePool
 from .runner import ModelRunner
 
 TILE = 16          # rows per tile of the row-wise input stages
-CHUNK = 64         # rows per chunk of the chunked recurrences
+CHUNKS = (64, 128)     # rows per chunk of the chunked recurrences
 SHORT_ROWS = 16    # portions up to this many rows take the row-by-row kernels
 
 
@@ -166,8 +166,12 @@ def build_portions(starts: Sequence[int], counts: Sequence[int], tables: Sequenc
         cu=dev(cu), starts=dev(st), slots=dev(np.asarray([slots[i] for i in order], dtype=np.int32)), row_seq=dev(row_seq),
         positions=dev(pos), tiles=dev(_row_tiles(cu, 0, n, TILE)), block_tables=dev(bt), nseq=n, num_short=ns,
         short_rows=int(cu[ns]), max_short=int(c[:ns].max()) if ns else 0, max_keys=int((st + c).max()) if n else 1,
-        long_counts=[int(x) for x in c[ns:]], long_chunks=dev(_row_tiles(cu, ns, n, CHUNK)) if ns < n else None,
         max_long=int(c[ns:].max()) if ns < n else 0)
+    if ns < n:
+        for size in CHUNKS:
+            first = np.concatenate([[0], np.cumsum((c[ns:] + size - 1) // size)]).astype(np.int32)
+            setattr(p, f"chunks{size}", dev(_row_tiles(cu, ns, n, size)))
+            setattr(p, f"first{size}", dev(first))
     return p, order, place
 
 

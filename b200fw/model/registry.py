@@ -82,7 +82,7 @@ ARCHITECTURES: Dict[str, Architecture] = {
     "Fetelorn": Architecture("Fetelorn", FetelornConfig,
                              lambda path: FetelornConfig.from_dict(_config_json(path), safetensors_shapes(path)),
                              FetelornModel, _load_fetelorn,
-                             ("host", "gemm", "residual", "linear_state", "attention_rows", "attention_fwd", "sampling"), float32=True),
+                             ("host", "gemm", "residual", "linear_state", "retention_chunk", "delta_chunk", "attention_rows", "attention_fwd", "sampling"), float32=True),
 }
 PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS}
 

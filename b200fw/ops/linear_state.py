@@ -70,10 +70,20 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Ten
             int(q.dtype == torch.float32), nv.stream_ptr()), "retention_serial")
         nv.count_launch()
     if p.nseq > ns:
+        nlong, n = p.nseq - ns, p.chunks128.shape[0]
+        if q.dtype == torch.bfloat16 and dkp <= 128 and dvp <= 128:
+            ws = torch.empty((n, H, dkp, dvp), device=q.device, dtype=torch.float32)
+            nv.check(nv.lib().b2_retention_chunk(
+                nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(out), nv.ptr(ws), nv.ptr(state), nv.ptr(decay), nv.ptr(cos),
+                nv.ptr(sin), nv.ptr(p.chunks128), nv.ptr(p.first128), nv.ptr(p.starts), nv.ptr(p.slots), n, ns, nlong, H, dk, dkp,
+                dv, dvp, rot, nv.ctypes.c_longlong(q.stride(0)), nv.ctypes.c_longlong(out.stride(0)),
+                nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps), nv.stream_ptr()), "retention_chunk")
+            nv.count_launch(3)
+            return
         cu, st, sl = _sub(p, ns)
         nv.check(nv.lib().b2_retention_serial(
             nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(out), nv.ptr(state), nv.ptr(decay), nv.ptr(cos), nv.ptr(sin),
-            cu, st, sl, p.nseq - ns, p.max_long, H, dk, dkp, dv, dvp, rot, nv.ctypes.c_longlong(q.stride(0)),
+            cu, st, sl, nlong, p.max_long, H, dk, dkp, dv, dvp, rot, nv.ctypes.c_longlong(q.stride(0)),
             nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps),
             int(q.dtype == torch.float32), nv.stream_ptr()), "retention_serial")
         nv.count_launch()
@@ -156,6 +166,17 @@ def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: to
     assert gate.dtype == torch.float32
     for lo, n, longest in ((0, p.num_short, p.max_short), (p.num_short, p.nseq - p.num_short, p.max_long)):
         if n <= 0:
+            continue
+        if lo == p.num_short and p.chunks64 is not None and v.dtype == torch.bfloat16 and dkp <= 128 and dvp <= 128:
+            nc = p.chunks64.shape[0]
+            ws = torch.empty(nc * H * nv.lib().b2_delta_chunk_words(dkp, dvp), device=v.device, dtype=torch.int32)
+            o = torch.empty((v.shape[0], H * dvp), device=v.device, dtype=torch.float32)
+            nv.check(nv.lib().b2_delta_chunk(
+                nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(log_decay), nv.ptr(beta), nv.ptr(gate), nv.ptr(norm_w), nv.ptr(out),
+                nv.ptr(state), nv.ptr(ws), nv.ptr(o), nv.ptr(p.chunks64), nv.ptr(p.first64), nv.ptr(p.starts), nv.ptr(p.slots),
+                nc, lo, n, p.short_rows, p.rows - p.short_rows, H, G, dk, dkp, dv, dvp, nv.ctypes.c_longlong(gate.stride(0)),
+                nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(eps), nv.stream_ptr()), "delta_chunk")
+            nv.count_launch(3)
             continue
         cu, st, sl = _sub(p, lo)
         nv.check(nv.lib().b2_delta_serial(

@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import Optional
 
 import torch
 
@@ -30,8 +30,11 @@ class Portions:
     short_rows: int
     max_short: int                           # longest portion among the short ones
     max_keys: int                            # longest context (tokens) of any sequence after this step
-    long_counts: Optional[List[int]] = None  # rows of each sequence past num_short (host copy)
-    long_chunks: Optional[torch.Tensor] = None   # int32 [n, 4] like tiles, 64-row chunks of the long portions
+    # long portions cut into chunks of 64 and of 128 rows: int32 [n, 4] like tiles, and [nlong + 1] first chunk of each sequence
+    chunks64: Optional[torch.Tensor] = None
+    first64: Optional[torch.Tensor] = None
+    chunks128: Optional[torch.Tensor] = None
+    first128: Optional[torch.Tensor] = None
     max_long: int = 0
     ragged: bool = True                      # False: every sequence is one row (decode): row r is sequence r
 
