@@ -123,9 +123,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
 
 
 def _split(rows: int, ctas_per_row: int, keys: int):
-    """Keys per split and number of splits: enough CTAs for a few waves over 148 SMs, at least 256 keys each."""
+    """Keys per split and number of splits: enough CTAs for a few waves over 148 SMs, 256 to 2048 keys each."""
     want = 4 * 148 * 3
-    n = min((keys + 255) // 256, -(-want // max(1, rows * ctas_per_row)))
+    n = max(min((keys + 255) // 256, -(-want // max(1, rows * ctas_per_row))), (keys + 2047) // 2048)
     if n <= 1:
         return max(1, keys), 1
     part = ((keys + n - 1) // n + 63) // 64 * 64

@@ -38,6 +38,12 @@ struct AttnRowsParams {
   float scale;
 };
 
+// softmax weights: the special-function unit's 2^x beside bf16 values, the library's in 32-bit runs
+template <typename T>
+__device__ __forceinline__ float ar_exp2(float x) {
+  return sizeof(T) == 2 ? fast_exp2(x) : exp2f(x);
+}
+
 template <typename T>
 __device__ __forceinline__ float ar_finish(const AttnRowsParams& p, int head, size_t row, float o, float L, float M2) {
   // M2: running maximum in the base-2 domain
@@ -56,9 +62,20 @@ __device__ __forceinline__ float ar_finish(const AttnRowsParams& p, int head, si
 // Grid (M, G * groups, nsplit).  A key row is spread over LPT lanes, eight channels each, so one warp-wide step covers
 // 32 / LPT tokens; every lane group runs its own online softmax over the tokens it sees for the GH query heads of this CTA,
 // and groups and warps are merged at the end with the exact log-sum-exp rule.
+//
+// The bias of every key of the partition is looked up once, into shared memory.  bf16 rows travel through a ring of three
+// stages per warp filled by 16-byte asynchronous copies (a lane reads back the bytes it copied: no barrier); 32-bit rows are
+// loaded into registers.
+constexpr int AR_STAGES = 3;
+template <typename T>
+__host__ __device__ constexpr int ar_ring_bytes() {
+  return sizeof(T) == 2 ? (AR_THREADS / 32) * AR_STAGES * AR_UNROLL * 2 * 512 : 0;
+}
 template <typename T, int LPT, int GH>
 __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsParams p) {
   constexpr int TPW = 32 / LPT, U = AR_UNROLL;
+  constexpr bool RING = sizeof(T) == 2;
+  extern __shared__ __align__(16) uint8_t ar_dyn[];   // ring, then bias [GH][partition]
   __shared__ float sAcc[AR_THREADS / 32][GH][LPT * 8];
   __shared__ float sM[AR_THREADS / 32][GH], sL[AR_THREADS / 32][GH];
   const size_t row = blockIdx.x;
@@ -93,9 +110,43 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
     l[g] = 0.f;
   }
   constexpr int STEP = (AR_THREADS / 32) * TPW * U;
-  for (int base = t_begin + warp * (TPW * U); base < t_end; base += STEP) {
+  float* sBias = reinterpret_cast<float*>(ar_dyn + ar_ring_bytes<T>());
+  const uint32_t ring = smem_u32(ar_dyn) + (warp * AR_STAGES * U * 2 * 32 + lane) * 16;
+  auto issue = [&](int stage, int at) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int tok = at + u * TPW + group;
+      if (tok < t_end) {
+        const size_t a = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
+        const uint32_t dst = ring + ((stage * U + u) * 2) * 512;
+        if (kin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(kc + a * kts) : "memory");
+        if (vin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + 512), "l"(vc + a * vts) : "memory");
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");   // one group per stage, empty ones included
+  };
+  int base = t_begin + warp * (TPW * U);
+  if (RING) {
+#pragma unroll
+    for (int st = 0; st < AR_STAGES - 1; ++st) issue(st, base + st * STEP);
+  }
+  if (p.rel) {
+    for (int i = threadIdx.x; i < t_end - t_begin; i += AR_THREADS) {
+      const T* rel = static_cast<const T*>(p.rel) + static_cast<size_t>(p.bucket[min(pos - t_begin - i, p.nbucket - 1)]) * p.H + head0;
+#pragma unroll
+      for (int g = 0; g < GH; ++g)
+        if (g < nh) sBias[g * p.partition + i] = to_f(rel[g]) * AR_LOG2E;
+    }
+    __syncthreads();
+  }
+  int stage = 0;
+  for (; base < t_end; base += STEP) {
     float kf[U][8], vf[U][8], sc[U][GH];
     bool valid[U];
+    if (RING) {
+      issue(stage == 0 ? AR_STAGES - 1 : stage - 1, base + (AR_STAGES - 1) * STEP);
+      asm volatile("cp.async.wait_group %0;" ::"n"(AR_STAGES - 1) : "memory");
+    }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int tok = base + u * TPW + group;
@@ -103,16 +154,21 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
 #pragma unroll
       for (int e = 0; e < 8; ++e) kf[u][e] = vf[u][e] = 0.f;
       if (valid[u]) {
-        const size_t at = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
-        if (kin) vload8(kc + at * kts, kf[u]);
-        if (vin) vload8(vc + at * vts, vf[u]);
+        if (RING) {
+          const uint8_t* src = ar_dyn + (warp * AR_STAGES * U * 2 * 32 + lane) * 16 + ((stage * U + u) * 2) * 512;
+          if (kin) vload8(reinterpret_cast<const __nv_bfloat16*>(src), kf[u]);
+          if (vin) vload8(reinterpret_cast<const __nv_bfloat16*>(src + 512), vf[u]);
+        } else {
+          const size_t at = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
+          if (kin) vload8(kc + at * kts, kf[u]);
+          if (vin) vload8(vc + at * vts, vf[u]);
+        }
       }
     }
+    stage = stage + 1 == AR_STAGES ? 0 : stage + 1;
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int tok = base + u * TPW + group;
-      int b = 0;
-      if (p.rel && valid[u]) b = p.bucket[min(pos - tok, p.nbucket - 1)];
 #pragma unroll
       for (int g = 0; g < GH; ++g) {
         float d = 0.f;
@@ -120,8 +176,7 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
         for (int e = 0; e < 8; ++e) d = fmaf(qr[g][e], kf[u][e], d);
 #pragma unroll
         for (int o = LPT / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-        if (p.rel && valid[u] && g < nh)
-          d = fmaf(to_f(static_cast<const T*>(p.rel)[static_cast<size_t>(b) * p.H + head0 + g]), AR_LOG2E, d);
+        if (p.rel && valid[u] && g < nh) d += sBias[g * p.partition + tok - t_begin];
         sc[u][g] = valid[u] ? d : -INFINITY;
       }
     }
@@ -131,14 +186,14 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
 #pragma unroll
       for (int u = 0; u < U; ++u) mn = fmaxf(mn, sc[u][g]);
       if (mn == -INFINITY) continue;   // this lane group has not seen a token yet
-      const float alpha = exp2f(m[g] - mn);
+      const float alpha = ar_exp2<T>(m[g] - mn);
       m[g] = mn;
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[g][e] *= alpha;
       float ps = 0.f;
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        const float w = exp2f(sc[u][g] - mn);
+        const float w = ar_exp2<T>(sc[u][g] - mn);
         ps += w;
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[g][e] = fmaf(w, vf[u][e], acc[g][e]);
@@ -264,12 +319,29 @@ __global__ void __launch_bounds__(128) qk_norm_store_kernel(const T* __restrict_
 template <typename T, int LPT>
 static int launch_rows(const AttnRowsParams& p, int M, int GH, cudaStream_t stream) {
   const dim3 grid(M, p.G * p.groups, p.nsplit);
+  const int smem = ar_ring_bytes<T>() + (p.rel ? GH * p.partition * 4 : 0);
+#define B2_ROWS(GHV)                                                                                              \
+  do {                                                                                                            \
+    auto kern = attn_rows_kernel<T, LPT, GHV>;                                                                    \
+    static int set[64] = {0};                                                                                     \
+    int dev = 0;                                                                                                  \
+    cudaGetDevice(&dev);                                                                                          \
+    if (set[dev & 63] < smem) {                                                                                   \
+      if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {         \
+        set_error("attn_rows: cannot set shared memory size (%d)", smem);                                         \
+        return 1;                                                                                                 \
+      }                                                                                                           \
+      set[dev & 63] = smem;                                                                                       \
+    }                                                                                                             \
+    kern<<<grid, AR_THREADS, smem, stream>>>(p);                                                                  \
+  } while (0)
   switch (GH) {
-    case 1: attn_rows_kernel<T, LPT, 1><<<grid, AR_THREADS, 0, stream>>>(p); break;
-    case 2: attn_rows_kernel<T, LPT, 2><<<grid, AR_THREADS, 0, stream>>>(p); break;
-    case 3: attn_rows_kernel<T, LPT, 3><<<grid, AR_THREADS, 0, stream>>>(p); break;
-    default: attn_rows_kernel<T, LPT, 4><<<grid, AR_THREADS, 0, stream>>>(p); break;
+    case 1: B2_ROWS(1); break;
+    case 2: B2_ROWS(2); break;
+    case 3: B2_ROWS(3); break;
+    default: B2_ROWS(4); break;
   }
+#undef B2_ROWS
   B2_CHECK_LAUNCH("attn_rows");
   if (p.nsplit > 1) {
     attn_rows_merge_kernel<T><<<dim3(M, p.H), 128, 0, stream>>>(p);
@@ -282,7 +354,7 @@ static int launch_rows(const AttnRowsParams& p, int M, int GH, cudaStream_t stre
 
 using namespace b2;
 
-// partition: keys per split, counted from the row's first visible key; nsplit * partition must cover every row's keys.
+// partition: keys per split (at most 4096 with a bias), counted from the row's first visible key; nsplit * partition must cover every row's keys.
 B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const int* tables, const int* row_seq,
                            const int* pos, const int* slot, const void* gate, long long ld_gate, const void* sink,
                            const void* rel, const int* bucket, int nbucket, void* out, long long ld_out, float* part_o,
@@ -292,7 +364,7 @@ B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const 
   if (M <= 0) return 0;
   if (H < 1 || G < 1 || H % G || dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || dkp < 8 || dvp < 8 || nsplit < 1 ||
       nsplit > 65535 || partition < 1 || (nsplit > 1 && (part_o == nullptr || part_ml == nullptr)) ||
-      (rel != nullptr && (bucket == nullptr || nbucket < 1)) || max_blocks < 1 || H > 65535) {
+      (rel != nullptr && (bucket == nullptr || nbucket < 1 || partition > 4096)) || max_blocks < 1 || H > 65535) {
     set_error("attn_rows: H %% G == 0 and head sizes up to 256 in multiples of 8 (padded) required");
     return 10;
   }

@@ -199,6 +199,125 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
     }
 }
 
+// One token per sequence (the decode step), one CTA per (head, sequence).  Eight row groups of dvp / 4 threads: a thread holds
+// four neighbouring value channels of every eighth key row, so a warp reads and writes whole state rows; all of a thread's
+// rows are requested before the first is used.
+constexpr int STEP_GROUPS = 8;
+
+template <typename T, int J, bool DELTA, int MAXT>
+__global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_step_kernel(const SerialParams p) {
+  extern __shared__ __align__(16) float sm[];
+  const int h = blockIdx.x, s = blockIdx.y;
+  const int slot = p.seq.slot[s];
+  if (slot < 0) return;
+  const size_t row = p.seq.cu[s];
+  const int DK = p.dkp, DV = p.dvp, quads = DV / 4, tid = threadIdx.x, nthr = blockDim.x;
+  float* sk = sm;
+  float* sq = sk + DK;
+  float* sg = sq + DK;
+  float* red = sg + DK;                       // [STEP_GROUPS][DV]
+  float* so = red + STEP_GROUPS * DV;         // [DV], then one word per warp
+  const int rg = tid / quads, col = tid % quads * 4, kvh = h / p.group;
+  float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * DK * DV + col;
+  const bool fresh = p.seq.start[s] == 0;
+  float4 S[J];
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+    const int i = rg + STEP_GROUPS * j;
+    S[j] = !fresh && i < DK ? *reinterpret_cast<const float4*>(st + static_cast<size_t>(i) * DV) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  for (int c = tid; c < DK; c += nthr) {
+    const size_t at = row * p.ld_qk + static_cast<size_t>(kvh) * DK;
+    if (DELTA) {
+      sq[c] = static_cast<const float*>(p.q)[at + c];
+      sk[c] = static_cast<const float*>(p.k)[at + c];
+      sg[c] = expf(p.glog[(row * p.H + h) * DK + c]);
+    } else {
+      const T* q = static_cast<const T*>(p.q) + at;
+      const T* k = static_cast<const T*>(p.k) + at;
+      float qv = to_f(q[c]), kv = to_f(k[c]);
+      if (c < p.rot) {
+        const int half = p.rot / 2, f = c < half ? c : c - half, o = c < half ? c + half : c - half;
+        const float cs = p.cs[row * half + f], sn = c < half ? -p.sn[row * half + f] : p.sn[row * half + f];
+        qv = qv * cs + to_f(q[o]) * sn;
+        kv = kv * cs + to_f(k[o]) * sn;
+      }
+      sq[c] = qv;
+      sk[c] = kv * p.kscale;
+    }
+  }
+  float4 u;
+  {
+    float v[4];
+    const T* vp = static_cast<const T*>(p.v) + row * p.ld_v + static_cast<size_t>(h) * DV + col;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = to_f(vp[e]);
+    u = make_float4(v[0], v[1], v[2], v[3]);
+  }
+  __syncthreads();
+  if (DELTA) {
+    float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < J; ++j) {
+      const int i = rg + STEP_GROUPS * j;
+      if (i >= DK) break;
+      const float g = sg[i], k = sk[i];
+      S[j].x *= g; S[j].y *= g; S[j].z *= g; S[j].w *= g;
+      d.x = fmaf(S[j].x, k, d.x); d.y = fmaf(S[j].y, k, d.y); d.z = fmaf(S[j].z, k, d.z); d.w = fmaf(S[j].w, k, d.w);
+    }
+    *reinterpret_cast<float4*>(red + rg * DV + col) = d;
+    __syncthreads();
+    float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < STEP_GROUPS; ++r) {
+      const float4 x = *reinterpret_cast<const float4*>(red + r * DV + col);
+      t.x += x.x; t.y += x.y; t.z += x.z; t.w += x.w;
+    }
+    const float b = p.beta[row * p.H + h];
+    u = make_float4(b * (u.x - t.x), b * (u.y - t.y), b * (u.z - t.z), b * (u.w - t.w));
+    __syncthreads();
+  }
+  const float a = DELTA ? 1.f : p.decay[h];
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+    const int i = rg + STEP_GROUPS * j;
+    if (i >= DK) break;
+    const float k = sk[i], q = sq[i];
+    S[j].x = fmaf(a, S[j].x, k * u.x); S[j].y = fmaf(a, S[j].y, k * u.y);
+    S[j].z = fmaf(a, S[j].z, k * u.z); S[j].w = fmaf(a, S[j].w, k * u.w);
+    *reinterpret_cast<float4*>(st + static_cast<size_t>(i) * DV) = S[j];
+    o.x = fmaf(S[j].x, q, o.x); o.y = fmaf(S[j].y, q, o.y); o.z = fmaf(S[j].z, q, o.z); o.w = fmaf(S[j].w, q, o.w);
+  }
+  *reinterpret_cast<float4*>(red + rg * DV + col) = o;
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < DV; c += nthr) {
+    float x = 0.f;
+#pragma unroll
+    for (int r = 0; r < STEP_GROUPS; ++r) x += red[r * DV + c];
+    so[c] = x;
+    ss = fmaf(x, x, ss);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) so[DV + (tid >> 5)] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int w = 0; w < nthr / 32; ++w) tot += so[DV + w];
+  const float r = 1.f / sqrtf(tot / p.dv + p.eps);
+  for (int c = tid; c < DV; c += nthr) {
+    float x = so[c] * r;
+    const size_t gi = row * p.ld_gate + static_cast<size_t>(h) * DV + c;
+    if (DELTA) {
+      if (p.norm_w) x *= to_f(static_cast<const T*>(p.norm_w)[c]);
+      x *= sigmoid_f(static_cast<const float*>(p.gate)[gi]);
+    } else {
+      x *= silu_f(to_f(static_cast<const T*>(p.gate)[gi]));
+    }
+    static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(h) * DV + c] = from_f<T>(x);
+  }
+}
+
 // Input stage of the delta rule.  Grid (tiles, 2 G + H): tile = {sequence, first row, rows, offset of that row in the
 // portion}, at most PREP_TILE rows.  Roles along y: G query heads, G key heads (convolution, silu, unit norm), H value heads
 // (convolution, silu; the head's decays and step size).  The convolution's channels are laid out [q | k | v] in the
@@ -301,8 +420,170 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(const DeltaPre
   }
 }
 
+// The same stage with four taps, a lane per eight channels: LPH lanes hold a head, a warp walks the rows of a tile with the
+// last inputs in registers.  A warp takes one job: 32 / LPH of the 2 G query and key heads, 32 / LPV value heads, or 256
+// decay channels.  (Any other number of taps: the kernel above.)
+template <typename T, int LPH>
+__device__ __forceinline__ void prep_conv_job(const DeltaPrepParams& p, int s, int row0, int rows, int off, int head, int nheads,
+                                              int c_base, int width, bool unit) {
+  constexpr int K = 4;
+  const int lane = threadIdx.x & 31, hd = head + lane / LPH, c = lane % LPH * 8;
+  const bool in = hd < nheads && c < width;
+  const int ch = c_base + (hd < nheads ? hd : 0) * width + (c < width ? c : 0);    // channel in [q | k | v]
+  const int C = 2 * p.G * p.dkp + p.H * p.dvp;
+  const bool fresh = p.seq.start[s] == 0;
+  const T* x = static_cast<const T*>(p.x) + ch;
+  float* cst = p.conv_state + (static_cast<size_t>(p.seq.slot[s]) * C + ch) * (K - 1);
+  float taps[K * 8], w[K - 1][8];     // w[i]: the input i + 1 tokens back
+#pragma unroll
+  for (int i = 0; i < K; ++i) {
+    float t[8];
+    vload8(static_cast<const T*>(p.taps) + static_cast<size_t>(ch) * K + i * 8, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) taps[i * 8 + e] = t[e];
+  }
+#pragma unroll
+  for (int i = 0; i < K - 1; ++i)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w[i][e] = 0.f;
+  float old[8 * (K - 1)];
+#pragma unroll
+  for (int e = 0; e < 8 * (K - 1); ++e) old[e] = 0.f;
+  if (off == 0) {
+    if (!fresh) {
+#pragma unroll
+      for (int i = 0; i < K - 1; ++i) {
+        float t[8];
+        vload8(cst + i * 8, t);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) old[i * 8 + e] = t[e];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < K - 1; ++i)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[i][e] = old[e * (K - 1) + K - 2 - i];
+  } else {
+#pragma unroll
+    for (int i = 0; i < K - 1; ++i) vload8(x + (static_cast<size_t>(row0) - 1 - i) * p.ld, w[i]);   // off >= a tile > K - 1
+  }
+  for (int t = 0; t < rows; ++t) {
+    const size_t row = static_cast<size_t>(row0) + t;
+    float cur[8], y[8], ss = 0.f;
+    vload8(x + row * p.ld, cur);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float a = cur[e] * taps[e * K + K - 1];
+#pragma unroll
+      for (int i = 0; i < K - 1; ++i) a = fmaf(w[i][e], taps[e * K + K - 2 - i], a);
+      y[e] = silu_f(a);
+      ss = fmaf(y[e], y[e], ss);
+    }
+#pragma unroll
+    for (int i = K - 2; i > 0; --i)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[i][e] = w[i - 1][e];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w[0][e] = cur[e];
+    if (unit) {
+      if (!in) ss = 0.f;
+#pragma unroll
+      for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const bool is_q = hd < p.G;
+      const float r = (is_q ? p.qscale : 1.f) / sqrtf(ss + p.unit_eps);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] *= r;
+      if (in) vstore8((is_q ? p.q : p.k) + (row * p.G + (is_q ? hd : hd - p.G)) * p.dkp + c, y);
+    } else if (in) {
+      vstore8(static_cast<T*>(p.v) + (row * p.H + hd) * p.dvp + c, y);
+    }
+  }
+  if (off != 0 || !in) return;
+  const int count = p.seq.cu[s + 1] - p.seq.cu[s];
+  float nw[K - 1][8];   // [j]: the input at index count - (K - 1) + j of the portion
+#pragma unroll
+  for (int j = 0; j < K - 1; ++j) {
+    const int at = count - (K - 1) + j;
+    if (at >= 0) {
+      vload8(x + (static_cast<size_t>(row0) + at) * p.ld, nw[j]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        nw[j][e] = 0.f;
+#pragma unroll
+        for (int m = 0; m < K - 1; ++m)
+          if (m == j + count) nw[j][e] = old[e * (K - 1) + m];
+      }
+    }
+  }
+  float flat[8 * (K - 1)];
+#pragma unroll
+  for (int e = 0; e < 8; ++e)
+#pragma unroll
+    for (int j = 0; j < K - 1; ++j) flat[e * (K - 1) + j] = nw[j][e];
+#pragma unroll
+  for (int i = 0; i < K - 1; ++i) {
+    float t[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) t[e] = flat[i * 8 + e];
+    vstore8(cst + i * 8, t);
+  }
+}
+
+template <typename T, int LPH, int LPV>
+__global__ void __launch_bounds__(PREP_THREADS) delta_prep_vec_kernel(const DeltaPrepParams p) {
+  const int* tl = p.tiles + blockIdx.x * 4;
+  const int s = tl[0], row0 = tl[1], rows = tl[2], off = tl[3];
+  if (s < 0 || rows <= 0 || p.seq.slot[s] < 0) return;
+  const int nq = (2 * p.G * LPH + 31) / 32, nv = (p.H * LPV + 31) / 32, lane = threadIdx.x & 31;
+  int job = blockIdx.y * (PREP_THREADS / 32) + (threadIdx.x >> 5);
+  if (job < nq) return prep_conv_job<T, LPH>(p, s, row0, rows, off, job * (32 / LPH), 2 * p.G, 0, p.dkp, true);
+  job -= nq;
+  if (job < nv) return prep_conv_job<T, LPV>(p, s, row0, rows, off, job * (32 / LPV), p.H, 2 * p.G * p.dkp, p.dvp, false);
+  job -= nv;
+  const int c = job * 256 + lane * 8, width = p.H * p.dkp;
+  if (job == 0)
+    for (int t = 0; t < rows; ++t)
+      for (int h = lane; h < p.H; h += 32) {
+        const size_t row = static_cast<size_t>(row0) + t;
+        p.beta[row * p.H + h] = sigmoid_f(to_f(static_cast<const T*>(p.b)[row * p.ld + h]));
+      }
+  if (c >= width) return;
+  float dt[8];
+  vload8(static_cast<const T*>(p.dt_bias) + c, dt);
+  const float A = -expf(to_f(static_cast<const T*>(p.A_log)[c / p.dkp]));
+  for (int t = 0; t < rows; ++t) {
+    const size_t row = static_cast<size_t>(row0) + t;
+    float z[8];
+    vload8(p.a2 + row * p.ld_a2 + c, z);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) z[e] = A * softplus_f(z[e] + dt[e]);
+    vstore8(p.glog + row * width + c, z);
+  }
+}
+
+template <typename T, bool DELTA>
+static int launch_step(const SerialParams& p, int nseq, cudaStream_t stream) {
+  const int threads = STEP_GROUPS * (p.dvp / 4);    // a multiple of 16; 32 for head sizes in steps of 16
+  const size_t smem = sizeof(float) * (3 * p.dkp + (STEP_GROUPS + 1) * p.dvp + 32);
+  const dim3 grid(p.H, nseq);
+#define B2_STEP(JV)                                                                                          \
+  do {                                                                                                       \
+    auto kern = threads <= 256 ? state_step_kernel<T, JV, DELTA, 256> : state_step_kernel<T, JV, DELTA, 512>; \
+    kern<<<grid, threads, smem, stream>>>(p);                                                                \
+  } while (0)
+  if (p.dkp <= 32) B2_STEP(4);
+  else if (p.dkp <= 64) B2_STEP(8);
+  else if (p.dkp <= 128) B2_STEP(16);
+  else B2_STEP(32);
+#undef B2_STEP
+  B2_CHECK_LAUNCH("linear_state_step");
+  return 0;
+}
+
 template <typename T, bool DELTA>
 static int launch_serial(const SerialParams& p, int nseq, cudaStream_t stream) {
+  if (p.tile == 1 && p.dvp % 16 == 0) return launch_step<T, DELTA>(p, nseq, stream);
   const int JJ = p.dkp <= 16 ? 1 : p.dkp <= 32 ? 2 : p.dkp <= 64 ? 4 : p.dkp <= 128 ? 8 : 16;
   const int DK = 16 * JJ;
   const size_t smem = sizeof(float) * p.tile * ((DELTA ? 3 : 2) * DK + 2 * p.dvp);
@@ -384,6 +665,25 @@ B2_EXPORT int b2_delta_prep(const void* x, const void* taps, const void* b, cons
   p.tiles = tiles; p.x = x; p.taps = taps; p.b = b; p.a2 = a2; p.A_log = A_log; p.dt_bias = dt_bias; p.conv_state = conv_state;
   p.q = q; p.k = k; p.v = v; p.glog = glog; p.beta = beta; p.ld = ld; p.ld_a2 = ld_a2;
   p.G = G; p.H = H; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.K = K; p.qscale = qscale; p.unit_eps = unit_eps;
+  const auto lanes = [](int w) { int l = 1; while (l * 8 < w) l *= 2; return l; };
+  const int lph = lanes(dkp), lpv = lanes(dvp);
+  if (K == 4 && ld % 8 == 0 && ld_a2 % 8 == 0 && lph >= 4 && lpv >= 4) {
+    const int jobs = (2 * G * lph + 31) / 32 + (H * lpv + 31) / 32 + (H * dkp + 255) / 256;
+    const dim3 vgrid(ntiles, (jobs + PREP_THREADS / 32 - 1) / (PREP_THREADS / 32));
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+#define B2_PREP_V(A, B) delta_prep_vec_kernel<T, A, B><<<vgrid, PREP_THREADS, 0, st>>>(p)
+#define B2_PREP_Q(A)                                                                                        \
+  do {                                                                                                      \
+    if (lpv == 4) B2_PREP_V(A, 4); else if (lpv == 8) B2_PREP_V(A, 8); else if (lpv == 16) B2_PREP_V(A, 16); else B2_PREP_V(A, 32); \
+  } while (0)
+    B2_DISPATCH_T(is_f32, {
+      if (lph == 4) B2_PREP_Q(4); else if (lph == 8) B2_PREP_Q(8); else if (lph == 16) B2_PREP_Q(16); else B2_PREP_Q(32);
+    });
+#undef B2_PREP_Q
+#undef B2_PREP_V
+    B2_CHECK_LAUNCH("delta_prep");
+    return 0;
+  }
   const dim3 grid(ntiles, 2 * G + H);
   B2_DISPATCH_T(is_f32, delta_prep_kernel<T><<<grid, PREP_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(p););
   B2_CHECK_LAUNCH("delta_prep");

@@ -37,19 +37,22 @@ struct RetParams {
 
 __device__ __forceinline__ float ret_pow(float l2a, int n) { return n == 0 ? 1.f : exp2f(l2a * n); }
 
-// Rows of one head, rotated, times scale(t), as split words [RET_C][ld]; zero past `n` rows and past dkp channels.
-template <int DK, typename F>
-__device__ __forceinline__ void ret_load_rotated(uint32_t* dst, int ld, const bf16_t* src, size_t row0, int n, const RetParams& p,
-                                                 F scale) {
-  const int half = p.rot / 2, tid = threadIdx.x;
+// Rows of one head, rotated, times scale(t), as hi (and lo) bf16 matrices [RET_C][ld]; zero past `n` rows and dkp channels.
+template <int DK, bool LO, typename F>
+__device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld, const bf16_t* src, size_t row0, int n,
+                                                 const RetParams& p, F scale) {
+  const int half = p.rot / 2, tid = threadIdx.x, nthr = blockDim.x;
+  auto put = [&](int t, int c, const float (&f)[8]) {
+    if (LO) store8_split(hi + t * ld + c, lo + t * ld + c, f);
+    else vstore8(hi + t * ld + c, f);
+  };
   if (half % 8 == 0) {
     const int rv = half / 8, pieces = rv + (DK - p.rot) / 8;   // rotated pairs of 8-channel pieces, then plain pieces
-    for (int i = tid; i < RET_C * pieces; i += RET_THREADS) {
+    for (int i = tid; i < RET_C * pieces; i += nthr) {
       const int t = i / pieces, c = i % pieces;
       const float f = t < n ? scale(t) : 0.f;
-      uint32_t* d = dst + t * ld;
       if (c < rv) {
-        float u[8] = {}, w[8] = {}, cs[8] = {}, sn[8] = {};
+        float u[8] = {}, w[8] = {}, cs[8] = {}, sn[8] = {}, x[8], y[8];
         if (t < n) {
           const bf16_t* s = src + (row0 + t) * p.ld_in + c * 8;
           vload8(s, u);
@@ -59,40 +62,47 @@ __device__ __forceinline__ void ret_load_rotated(uint32_t* dst, int ld, const bf
         }
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          d[c * 8 + e] = split_word((u[e] * cs[e] - w[e] * sn[e]) * f);
-          d[half + c * 8 + e] = split_word((w[e] * cs[e] + u[e] * sn[e]) * f);
+          x[e] = (u[e] * cs[e] - w[e] * sn[e]) * f;
+          y[e] = (w[e] * cs[e] + u[e] * sn[e]) * f;
         }
+        put(t, c * 8, x);
+        put(t, half + c * 8, y);
       } else {
         const int at = p.rot + (c - rv) * 8;
         float u[8] = {};
         if (t < n && at < p.dkp) vload8(src + (row0 + t) * p.ld_in + at, u);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) d[at + e] = split_word(u[e] * f);
+        for (int e = 0; e < 8; ++e) u[e] *= f;
+        put(t, at, u);
       }
     }
     return;
   }
-  for (int i = tid; i < RET_C * DK; i += RET_THREADS) {
-    const int t = i / DK, c = i % DK;
-    float x = 0.f;
-    if (t < n && c < p.dkp) {
+  for (int i = tid; i < RET_C * (DK / 8); i += nthr) {
+    const int t = i / (DK / 8), c8 = i % (DK / 8) * 8;
+    float x[8] = {};
+    if (t < n && c8 < p.dkp) {
       const bf16_t* s = src + (row0 + t) * p.ld_in;
-      x = to_f(s[c]);
-      if (c < p.rot) {
-        const int f = c < half ? c : c - half;
-        const float o = to_f(s[c < half ? c + half : c - half]);
-        x = x * p.cs[(row0 + t) * half + f] + (c < half ? -o : o) * p.sn[(row0 + t) * half + f];
+      const float fs = scale(t);
+      for (int e = 0; e < 8; ++e) {
+        const int c = c8 + e;
+        x[e] = to_f(s[c]);
+        if (c < p.rot) {
+          const int f = c < half ? c : c - half;
+          const float o = to_f(s[c < half ? c + half : c - half]);
+          x[e] = x[e] * p.cs[(row0 + t) * half + f] + (c < half ? -o : o) * p.sn[(row0 + t) * half + f];
+        }
+        x[e] *= fs;
       }
-      x *= scale(t);
     }
-    dst[t * ld + c] = split_word(x);
+    put(t, c8, x);
   }
 }
 
 template <int DV>
 __device__ __forceinline__ void ret_load_v(bf16_t* dst, const bf16_t* src, size_t row0, int n, const RetParams& p) {
   constexpr int LDV = DV + 8;
-  for (int i = threadIdx.x; i < RET_C * (DV / 8); i += RET_THREADS) {
+  for (int i = threadIdx.x; i < RET_C * (DV / 8); i += blockDim.x) {
     const int t = i / (DV / 8), c = i % (DV / 8) * 8;
     uint4 u = make_uint4(0, 0, 0, 0);
     if (t < n && c < p.dvp) u = *reinterpret_cast<const uint4*>(src + (row0 + t) * p.ld_in + c);
@@ -101,31 +111,34 @@ __device__ __forceinline__ void ret_load_v(bf16_t* dst, const bf16_t* src, size_
 }
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(RET_THREADS) ret_contrib_kernel(const RetParams p) {
-  constexpr int LDK = DK + 4, LDV = DV + 8;
+__global__ void __launch_bounds__(RET_THREADS, 2) ret_contrib_kernel(const RetParams p) {
+  constexpr int LDK = DK + 8, LDV = DV + 8;
   constexpr int NT = DV / 8 / (DK == 128 ? 1 : 2);   // n8 tiles per warp
   extern __shared__ __align__(16) uint8_t sm_raw[];
-  uint32_t* sK = reinterpret_cast<uint32_t*>(sm_raw);
-  bf16_t* sV = reinterpret_cast<bf16_t*>(sK + RET_C * LDK);
+  bf16_t* sKh = reinterpret_cast<bf16_t*>(sm_raw);
+  bf16_t* sKl = sKh + RET_C * LDK;
+  bf16_t* sV = sKl + RET_C * LDK;
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, n = ch[2];
   const size_t row0 = ch[1];
   const float l2a = static_cast<float>(log2(static_cast<double>(p.decay[h])));
-  ret_load_rotated<DK>(sK, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p,
-                       [&](int t) { return p.kscale * ret_pow(l2a, n - 1 - t); });
+  ret_load_rotated<DK, true>(sKh, sKl, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p,
+                             [&](int t) { return p.kscale * ret_pow(l2a, n - 1 - t); });
   ret_load_v<DV>(sV, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   const int mt = DK == 128 ? warp : (warp & 3), nb = DK == 128 ? 0 : (warp >> 2) * NT;
   float acc[NT][4] = {};
   for (int k0 = 0; k0 < n; k0 += 16) {
-    const FragA a = lda_km(sK + k0 * LDK + mt * 16, LDK, g, q);
+    uint32_t ah[4], al[4];
+    ldsm_a_km(sKh + k0 * LDK + mt * 16, LDK, lane, ah);
+    ldsm_a_km(sKl + k0 * LDK + mt * 16, LDK, lane, al);
 #pragma unroll
     for (int j = 0; j < NT; j += 2) {
-      uint32_t b0[2], b1[2];
-      ldb_kn_bf16_x2(sV + k0 * LDV + (nb + j) * 8, LDV, lane, b0, b1);
-      mma_split_bx(acc[j], a, b0);
-      mma_split_bx(acc[j + 1], a, b1);
+      uint32_t b[4];
+      ldsm_b_kn(sV + k0 * LDV + (nb + j) * 8, LDV, lane, b);
+      mma_n16(acc[j], acc[j + 1], ah, b);
+      mma_n16(acc[j], acc[j + 1], al, b);
     }
   }
   float* w = p.ws + (static_cast<size_t>(blockIdx.x) * p.H + h) * p.dkp * p.dvp;
@@ -147,13 +160,14 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
   const int size = p.dkp * p.dvp, i = (blockIdx.x * 256 + threadIdx.x) * 4;
   const int slot = p.slot[s];
   if (i >= size || slot < 0) return;
-  const double l2a = log2(static_cast<double>(p.decay[h]));
+  const float l2a = static_cast<float>(log2(static_cast<double>(p.decay[h])));
   float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * size + i;
   float4 S = p.start[s] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
+  const float full = exp2f(l2a * RET_C);
   const size_t step = static_cast<size_t>(p.H) * size;
   float* w = p.ws + (static_cast<size_t>(c0) * p.H + h) * size + i;
-  constexpr int U = 4;
+  constexpr int U = 8;
   for (int c = c0; c < c1; c += U) {
     float4 kv[U];
 #pragma unroll
@@ -163,7 +177,7 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
     for (int u = 0; u < U; ++u) {
       if (c + u >= c1) break;
       *reinterpret_cast<float4*>(w + u * step) = S;
-      const float a = static_cast<float>(exp2(l2a * p.chunks[(c + u) * 4 + 2]));
+      const float a = c + u + 1 < c1 ? full : exp2f(l2a * p.chunks[(c + u) * 4 + 2]);   // only the last chunk may be short
       S.x = fmaf(a, S.x, kv[u].x);
       S.y = fmaf(a, S.y, kv[u].y);
       S.z = fmaf(a, S.z, kv[u].z);
@@ -174,40 +188,59 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
   *reinterpret_cast<float4*>(st) = S;
 }
 
+// 16 warps: eight row tiles of 16 tokens, two warps each that share the contraction (every other k-step of q S, every other
+// block of keys) and add their results at the end.  Products with q take q's hi part only (q enters no recurrence).
+constexpr int RET_OUT_THREADS = 512;
+
 template <int DK, int DV>
-__global__ void __launch_bounds__(RET_THREADS) ret_out_kernel(const RetParams p) {
-  constexpr int LDQ = DK + 8, LDS = DV + 4, LDV = DV + 8, NT = DV / 8, KS = DK / 16;
-  constexpr int KB = RET_C * LDQ > DK * LDS ? RET_C * LDQ : DK * LDS;
+__host__ __device__ constexpr int ret_out_x_bytes() {   // keys, then before them the state, after them the partial results
+  int a = 2 * RET_C * (DK + 8) * 2, b = 2 * DK * (DV + 8) * 2, c = RET_C * (DV + 4) * 4;
+  return a > b ? (a > c ? a : c) : (b > c ? b : c);
+}
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(RET_OUT_THREADS, 1) ret_out_kernel(const RetParams p) {
+  constexpr int LDK = DK + 8, LDV = DV + 8, LDR = DV + 4, NT = DV / 8, KS = DK / 16;
   extern __shared__ __align__(16) uint8_t sm_raw[];
-  uint32_t* sQ = reinterpret_cast<uint32_t*>(sm_raw);
-  uint32_t* sK = sQ + RET_C * LDQ;                       // the state first, then the keys
-  bf16_t* sV = reinterpret_cast<bf16_t*>(sK + KB);
+  bf16_t* sQ = reinterpret_cast<bf16_t*>(sm_raw);
+  bf16_t* sV = sQ + RET_C * LDK;
+  bf16_t* sX = sV + RET_C * LDV;
+  float* sR = reinterpret_cast<float*>(sX);
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, s = ch[0], n = ch[2];
   const size_t row0 = ch[1];
   const bool zero = ch[3] == 0 && p.start[s] == 0;       // nothing before this chunk
   const float l2a = static_cast<float>(log2(static_cast<double>(p.decay[h])));
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
-  ret_load_rotated<DK>(sQ, LDQ, p.q + static_cast<size_t>(h) * p.dkp, row0, n, p, [](int) { return 1.f; });
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3, rt = warp & 7, par = warp >> 3;
+  const bool active = rt * 16 < n;
+  ret_load_rotated<DK, false>(sQ, nullptr, LDK, p.q + static_cast<size_t>(h) * p.dkp, row0, n, p, [](int) { return 1.f; });
   ret_load_v<DV>(sV, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
   float acc[NT][4] = {};
   if (!zero) {
+    bf16_t* hi = sX;
+    bf16_t* lo = sX + DK * LDV;
     const float* w = p.ws + (static_cast<size_t>(blockIdx.x) * p.H + h) * p.dkp * p.dvp;
-    for (int i = threadIdx.x; i < DK * (DV / 4); i += RET_THREADS) {
-      const int r = i / (DV / 4), c = i % (DV / 4) * 4;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (r < p.dkp && c < p.dvp) x = *reinterpret_cast<const float4*>(w + static_cast<size_t>(r) * p.dvp + c);
-      *reinterpret_cast<uint4*>(sK + r * LDS + c) = make_uint4(split_word(x.x), split_word(x.y), split_word(x.z), split_word(x.w));
+    for (int i = threadIdx.x; i < DK * (DV / 8); i += RET_OUT_THREADS) {
+      const int r = i / (DV / 8), c = i % (DV / 8) * 8;
+      float x[8] = {};
+      if (r < p.dkp && c < p.dvp) vload8(w + static_cast<size_t>(r) * p.dvp + c, x);
+      store8_split(hi + r * LDV + c, lo + r * LDV + c, x);
     }
     __syncthreads();
-    if (warp * 16 < n) {
-#pragma unroll 2
-      for (int ks = 0; ks < KS; ++ks) {
-        const FragA a = lda_mk(sQ + warp * 16 * LDQ + ks * 16, LDQ, g, q);
+    if (active) {
+      for (int ks = par; ks < KS; ks += 2) {
+        uint32_t a[4];
+        ldsm_a_mk(sQ + rt * 16 * LDK + ks * 16, LDK, lane, a);
 #pragma unroll
-        for (int j = 0; j < NT; ++j) mma_split(acc[j], a, ldb_kn(sK + ks * 16 * LDS + j * 8, LDS, g, q));
+        for (int j = 0; j < NT; j += 2) {
+          uint32_t b[4];
+          ldsm_b_kn(hi + ks * 16 * LDV + j * 8, LDV, lane, b);
+          mma_n16(acc[j], acc[j + 1], a, b);
+          ldsm_b_kn(lo + ks * 16 * LDV + j * 8, LDV, lane, b);
+          mma_n16(acc[j], acc[j + 1], a, b);
+        }
       }
-      const float f0 = ret_pow(l2a, warp * 16 + g + 1), f1 = ret_pow(l2a, warp * 16 + g + 9);
+      const float f0 = ret_pow(l2a, rt * 16 + g + 1), f1 = ret_pow(l2a, rt * 16 + g + 9);
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
         acc[j][0] *= f0;
@@ -218,38 +251,54 @@ __global__ void __launch_bounds__(RET_THREADS) ret_out_kernel(const RetParams p)
     }
     __syncthreads();
   }
-  ret_load_rotated<DK>(sK, LDQ, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p, [&](int) { return p.kscale; });
+  bf16_t* kh = sX;
+  bf16_t* kl = sX + RET_C * LDK;
+  ret_load_rotated<DK, true>(kh, kl, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p, [&](int) { return p.kscale; });
   __syncthreads();
-  if (warp * 16 >= n) return;
-  for (int kb = 0; kb <= warp; ++kb) {          // 16 keys at a time, up to the diagonal
+  for (int kb = par; active && kb <= rt; kb += 2) {          // 16 keys at a time, up to the diagonal
     float sc[2][4] = {};
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
-      const FragA a = lda_mk(sQ + warp * 16 * LDQ + ks * 16, LDQ, g, q);
-#pragma unroll
-      for (int j = 0; j < 2; ++j) mma_split(sc[j], a, ldb_nk(sK + (kb * 16 + j * 8) * LDQ + ks * 16, LDQ, g, q));
+      uint32_t a[4], b[4];
+      ldsm_a_mk(sQ + rt * 16 * LDK + ks * 16, LDK, lane, a);
+      ldsm_b_nk(kh + kb * 16 * LDK + ks * 16, LDK, lane, b);
+      mma_n16(sc[0], sc[1], a, b);
+      ldsm_b_nk(kl + kb * 16 * LDK + ks * 16, LDK, lane, b);
+      mma_n16(sc[0], sc[1], a, b);
     }
-    FragA pa;
+    uint32_t ph[4], pl[4];
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        const int d = warp * 16 + g + 8 * r - (kb * 16 + j * 8 + 2 * q);     // distance to the first of the two keys
+        const int d = rt * 16 + g + 8 * r - (kb * 16 + j * 8 + 2 * q);     // distance to the first of the two keys
         const float x0 = d >= 0 ? sc[j][2 * r] * ret_pow(l2a, d) : 0.f;
         const float x1 = d >= 1 ? sc[j][2 * r + 1] * ret_pow(l2a, d - 1) : 0.f;
-        split_pair(x0, x1, pa.hi[2 * j + r], pa.lo[2 * j + r]);
+        split_pair(x0, x1, ph[2 * j + r], pl[2 * j + r]);
       }
 #pragma unroll
     for (int j = 0; j < NT; j += 2) {
-      uint32_t b0[2], b1[2];
-      ldb_kn_bf16_x2(sV + kb * 16 * LDV + j * 8, LDV, lane, b0, b1);
-      mma_split_bx(acc[j], pa, b0);
-      mma_split_bx(acc[j + 1], pa, b1);
+      uint32_t b[4];
+      ldsm_b_kn(sV + kb * 16 * LDV + j * 8, LDV, lane, b);
+      mma_n16(acc[j], acc[j + 1], ph, b);
+      mma_n16(acc[j], acc[j + 1], pl, b);
     }
   }
+  __syncthreads();
+  if (par == 1 && active)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+        *reinterpret_cast<float2*>(sR + (rt * 16 + g + 8 * r) * LDR + j * 8 + 2 * q) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
+  __syncthreads();
+  if (par == 1 || !active) return;
   float s0 = 0.f, s1 = 0.f;
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
+    const float2 x = *reinterpret_cast<const float2*>(sR + (rt * 16 + g) * LDR + j * 8 + 2 * q);
+    const float2 y = *reinterpret_cast<const float2*>(sR + (rt * 16 + g + 8) * LDR + j * 8 + 2 * q);
+    acc[j][0] += x.x; acc[j][1] += x.y; acc[j][2] += y.x; acc[j][3] += y.y;
     s0 += acc[j][0] * acc[j][0] + acc[j][1] * acc[j][1];
     s1 += acc[j][2] * acc[j][2] + acc[j][3] * acc[j][3];
   }
@@ -261,7 +310,7 @@ __global__ void __launch_bounds__(RET_THREADS) ret_out_kernel(const RetParams p)
   const float r0 = 1.f / sqrtf(s0 / p.dv + p.eps), r1 = 1.f / sqrtf(s1 / p.dv + p.eps);
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
-    const int t = warp * 16 + g + 8 * r;
+    const int t = rt * 16 + g + 8 * r;
     if (t >= n) continue;
     const bf16_t* gp = p.gate + (row0 + t) * p.ld_in + static_cast<size_t>(h) * p.dvp;
     bf16_t* op = p.out + (row0 + t) * p.ld_out + static_cast<size_t>(h) * p.dvp;
@@ -278,9 +327,8 @@ __global__ void __launch_bounds__(RET_THREADS) ret_out_kernel(const RetParams p)
 
 template <int DK, int DV>
 static int launch_ret(const RetParams& p, int nchunks, int nlong, cudaStream_t stream) {
-  const int sm1 = RET_C * (DK + 4) * 4 + RET_C * (DV + 8) * 2;
-  const int kb = RET_C * (DK + 8) > DK * (DV + 4) ? RET_C * (DK + 8) : DK * (DV + 4);
-  const int sm3 = (RET_C * (DK + 8) + kb) * 4 + RET_C * (DV + 8) * 2;
+  const int sm1 = RET_C * (2 * (DK + 8) + DV + 8) * 2;
+  const int sm3 = RET_C * (DK + 8 + DV + 8) * 2 + ret_out_x_bytes<DK, DV>();
   static bool set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -296,7 +344,7 @@ static int launch_ret(const RetParams& p, int nchunks, int nlong, cudaStream_t s
   B2_CHECK_LAUNCH("ret_contrib");
   ret_scan_kernel<<<dim3((p.dkp * p.dvp / 4 + 255) / 256, p.H, nlong), 256, 0, stream>>>(p);
   B2_CHECK_LAUNCH("ret_scan");
-  ret_out_kernel<DK, DV><<<dim3(nchunks, p.H), RET_THREADS, sm3, stream>>>(p);
+  ret_out_kernel<DK, DV><<<dim3(nchunks, p.H), RET_OUT_THREADS, sm3, stream>>>(p);
   B2_CHECK_LAUNCH("ret_out");
   return 0;
 }
