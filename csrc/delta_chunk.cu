@@ -32,11 +32,12 @@ struct DeltaParams {
   const int* first;      // [nlong + 1]
   const int* start;
   const int* slot;
-  // per chunk and head: split words W, Qs, Ks [64][DK], P [64][64]; fp32 U0 [64][dvp], end [DK]
-  uint32_t* W;
-  uint32_t* Qs;
-  uint32_t* Ks;
-  uint32_t* P;
+  // per chunk and head, bf16 planes hi then lo: W, Ks [2][64][DK], P [2][64][64]; hi only: Qs [64][DK] (q enters no
+  // recurrence); fp32 U0 [64][dvp], end [DK]
+  __nv_bfloat16* W;
+  __nv_bfloat16* Qs;
+  __nv_bfloat16* Ks;
+  __nv_bfloat16* P;
   float* U0;
   float* end;
   float* o;              // [M, H * dvp]
@@ -44,103 +45,127 @@ struct DeltaParams {
   int H, G, dkp, dvp, seq0;
 };
 
+constexpr int FAC_THREADS = 512;
+
 template <int DK>
-__global__ void __launch_bounds__(DEL_THREADS, 1) delta_factor_kernel(const DeltaParams p) {
-  constexpr int LD = DK + 8, SEGS = DEL_THREADS / DK, SEG = DEL_C / SEGS;
+struct DelFactor {
+  static constexpr int LD = DK + 8, LDV = 128 + 8;
+  static constexpr int G = 0;                          // [64][LD] running log2 decays
+  static constexpr int E = G + DEL_C * LD;             // [64][LD] decays; later the hi and lo planes of k e^G
+  static constexpr int K = E + DEL_C * LD;
+  static constexpr int Q = K + DEL_C * LD;
+  static constexpr int A = Q + DEL_C * LD;             // [64][68], beta folded in
+  static constexpr int P = A + DEL_C * DEL_LDA;
+  static constexpr int T = P + DEL_C * DEL_LDA;        // (I + A)^-1
+  static constexpr int V = T + DEL_C * DEL_LDA;        // bf16 [64][LDV]
+  static constexpr int Z = V + DEL_C * LDV / 2;        // [16][68]
+  static constexpr int TOT = Z + 16 * DEL_LDA;         // segment totals
+  static constexpr int B = TOT + FAC_THREADS;          // beta
+  static constexpr int BYTES = (B + DEL_C) * 4;
+};
+
+template <int DK>
+__global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const DeltaParams p) {
+  using L = DelFactor<DK>;
+  constexpr int LD = L::LD, LDV = L::LDV, SEGS = FAC_THREADS / DK, SEG = DEL_C / SEGS;
   extern __shared__ __align__(16) float sm[];
-  float* sG = sm;                      // cumulative log decays
-  float* sE = sG + DEL_C * LD;         // decays
-  float* sK = sE + DEL_C * LD;
-  float* sQ = sK + DEL_C * LD;
-  float* sA = sQ + DEL_C * LD;         // [64][68], beta folded in
-  float* sP = sA + DEL_C * DEL_LDA;
-  float* sT = sP + DEL_C * DEL_LDA;    // [SEGS][DK] segment totals
-  float* sB = sT + SEGS * DK;          // beta
+  float *sG = sm + L::G, *sE = sm + L::E, *sK = sm + L::K, *sQ = sm + L::Q, *sA = sm + L::A, *sP = sm + L::P, *sT = sm + L::T,
+        *sZ = sm + L::Z, *sTot = sm + L::TOT, *sB = sm + L::B;
+  __nv_bfloat16* sV = reinterpret_cast<__nv_bfloat16*>(sm + L::V);
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, n = ch[2], kvh = h / (p.H / p.G);
   const size_t row0 = ch[1], item = static_cast<size_t>(blockIdx.x) * p.H + h;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
 
-  for (int i = tid; i < DEL_C * (DK / 4); i += DEL_THREADS) {
-    const int t = i / (DK / 4), c = i % (DK / 4) * 4;
-    float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
-    if (t < n && c < p.dkp) {
-      const size_t at = ((row0 + t) * p.G + kvh) * p.dkp + c;
-      kv = *reinterpret_cast<const float4*>(p.k + at);
-      qv = *reinterpret_cast<const float4*>(p.q + at);
-    }
-    *reinterpret_cast<float4*>(sK + t * LD + c) = kv;
-    *reinterpret_cast<float4*>(sQ + t * LD + c) = qv;
-  }
-  if (tid < DEL_C) sB[tid] = tid < n ? p.beta[(row0 + tid) * p.H + h] : 0.f;
   {
+    float x[SEG];
     const int c = tid % DK, seg = tid / DK;
-    float sum = 0.f;
-#pragma unroll 16
+#pragma unroll
     for (int i = 0; i < SEG; ++i) {
       const int t = seg * SEG + i;
-      const float x = t < n && c < p.dkp ? p.glog[((row0 + t) * p.H + h) * p.dkp + c] : 0.f;
-      sum += x;
-      sG[t * LD + c] = sum;
-      sE[t * LD + c] = expf(x);
+      x[i] = t < n && c < p.dkp ? p.glog[((row0 + t) * p.H + h) * p.dkp + c] * 1.4426950408889634f : 0.f;
     }
-    sT[seg * DK + c] = sum;
+#pragma unroll 4
+    for (int i = tid; i < DEL_C * (DK / 4); i += FAC_THREADS) {
+      const int t = i / (DK / 4), cc = i % (DK / 4) * 4;
+      float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
+      if (t < n && cc < p.dkp) {
+        const size_t at = ((row0 + t) * p.G + kvh) * p.dkp + cc;
+        kv = *reinterpret_cast<const float4*>(p.k + at);
+        qv = *reinterpret_cast<const float4*>(p.q + at);
+      }
+      *reinterpret_cast<float4*>(sK + t * LD + cc) = kv;
+      *reinterpret_cast<float4*>(sQ + t * LD + cc) = qv;
+    }
+#pragma unroll 2
+    for (int i = tid; i < DEL_C * (128 / 8); i += FAC_THREADS) {
+      const int t = i / 16, cc = i % 16 * 8;
+      uint4 u = make_uint4(0, 0, 0, 0);
+      if (t < n && cc < p.dvp) u = *reinterpret_cast<const uint4*>(p.v + ((row0 + t) * p.H + h) * p.dvp + cc);
+      *reinterpret_cast<uint4*>(sV + t * LDV + cc) = u;
+    }
+    if (tid < DEL_C) sB[tid] = tid < n ? p.beta[(row0 + tid) * p.H + h] : 0.f;
+    for (int i = tid; i < DEL_C * DEL_LDA / 4; i += FAC_THREADS) {
+      reinterpret_cast<float4*>(sA)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      reinterpret_cast<float4*>(sP)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < SEG; ++i) {
+      sE[(seg * SEG + i) * LD + c] = fast_exp2(x[i]);
+      sum += x[i];
+      x[i] = sum;
+    }
+    sTot[seg * DK + c] = sum;
     __syncthreads();
     float before = 0.f;
-    for (int s = 0; s < seg; ++s) before += sT[s * DK + c];
-    if (seg > 0)
-      for (int i = 0; i < SEG; ++i) sG[(seg * SEG + i) * LD + c] += before;
-  }
-  for (int i = tid; i < DEL_C * DEL_C; i += DEL_THREADS) {
-    sA[i / DEL_C * DEL_LDA + i % DEL_C] = 0.f;
-    sP[i / DEL_C * DEL_LDA + i % DEL_C] = 0.f;
+    for (int s = 0; s < seg; ++s) before += sTot[s * DK + c];
+#pragma unroll
+    for (int i = 0; i < SEG; ++i) sG[(seg * SEG + i) * LD + c] = x[i] + before;
   }
   __syncthreads();
 
-  if (warp < 6) {   // blocks below the diagonal: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
-    const int I = warp == 0 ? 1 : warp < 3 ? 2 : 3, J = warp == 0 ? 0 : warp < 3 ? warp - 1 : warp - 3;
-    float ak[2][4] = {}, aq[2][4] = {};
+  if (warp < 12) {   // blocks below the diagonal, (1,0) (2,0) (2,1) (3,0) (3,1) (3,2): of A by the first six warps, of P by the next
+    const int b = warp % 6, I = b == 0 ? 1 : b < 3 ? 2 : 3, J = b == 0 ? 0 : b < 3 ? b - 1 : b - 3;
+    const float* X = warp < 6 ? sK : sQ;
+    float acc[2][4] = {};
     const float* R = sG + (16 * I - 1) * LD;
 #pragma unroll 2
     for (int ks = 0; ks < DK / 16; ++ks) {
-      FragA fk, fq;
+      FragA fa;
       FragB fb[2];
+      float2 R2[2];
+      R2[0] = *reinterpret_cast<const float2*>(R + ks * 16 + 2 * q4);
+      R2[1] = *reinterpret_cast<const float2*>(R + ks * 16 + 2 * q4 + 8);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int t = 16 * I + g + (i & 1) * 8, c = ks * 16 + 2 * q4 + (i >> 1) * 8;
-        const float2 G2 = *reinterpret_cast<const float2*>(sG + t * LD + c), R2 = *reinterpret_cast<const float2*>(R + c);
-        const float e0 = expf(G2.x - R2.x), e1 = expf(G2.y - R2.y);
-        const float2 k2 = *reinterpret_cast<const float2*>(sK + t * LD + c), q2 = *reinterpret_cast<const float2*>(sQ + t * LD + c);
-        split_pair(k2.x * e0, k2.y * e1, fk.hi[i], fk.lo[i]);
-        split_pair(q2.x * e0, q2.y * e1, fq.hi[i], fq.lo[i]);
+        const int at = (16 * I + g + (i & 1) * 8) * LD + ks * 16 + 2 * q4 + (i >> 1) * 8;
+        const float2 G2 = *reinterpret_cast<const float2*>(sG + at), x2 = *reinterpret_cast<const float2*>(X + at);
+        split_pair(x2.x * fast_exp2(G2.x - R2[i >> 1].x), x2.y * fast_exp2(G2.y - R2[i >> 1].y), fa.hi[i], fa.lo[i]);
       }
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-          const int t = 16 * J + j * 8 + g, c = ks * 16 + 2 * q4 + i * 8;
-          const float2 G2 = *reinterpret_cast<const float2*>(sG + t * LD + c), R2 = *reinterpret_cast<const float2*>(R + c);
-          const float2 k2 = *reinterpret_cast<const float2*>(sK + t * LD + c);
-          split_pair(k2.x * expf(R2.x - G2.x), k2.y * expf(R2.y - G2.y), fb[j].hi[i], fb[j].lo[i]);
+          const int at = (16 * J + j * 8 + g) * LD + ks * 16 + 2 * q4 + i * 8;
+          const float2 G2 = *reinterpret_cast<const float2*>(sG + at), k2 = *reinterpret_cast<const float2*>(sK + at);
+          split_pair(k2.x * fast_exp2(R2[i].x - G2.x), k2.y * fast_exp2(R2[i].y - G2.y), fb[j].hi[i], fb[j].lo[i]);
         }
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        mma_split(ak[j], fk, fb[j]);
-        mma_split(aq[j], fq, fb[j]);
-      }
+      mma_split(acc[0], fa, fb[0]);
+      mma_split(acc[1], fa, fb[1]);
     }
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
         const int t = 16 * I + g + (r >> 1) * 8, c = 16 * J + j * 8 + 2 * q4 + (r & 1);
-        sA[t * DEL_LDA + c] = ak[j][r] * sB[t];
-        sP[t * DEL_LDA + c] = aq[j][r];
+        if (warp < 6) sA[t * DEL_LDA + c] = acc[j][r] * sB[t];
+        else sP[t * DEL_LDA + c] = acc[j][r];
       }
   }
-  {   // diagonal blocks: two warps each (halves of the channels), a lane per key j and quarter of the channels
-    constexpr int NC = DK / 4;
-    const int I = warp >> 1, j = lane & 15, c0 = (warp & 1) * (DK / 2) + (lane >> 4) * NC;
+  {   // diagonal blocks: four warps each (quarters of the channels), a lane per key j and half of its warp's channels
+    constexpr int NC = DK / 8;
+    const int I = warp >> 2, j = lane & 15, c0 = (warp & 3) * (DK / 4) + (lane >> 4) * NC;
     float kd[NC];
 #pragma unroll
     for (int c = 0; c < NC; ++c) kd[c] = sK[(16 * I + j) * LD + c0 + c];
@@ -169,73 +194,165 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_factor_kernel(const Delt
       dk[t] += __shfl_xor_sync(0xffffffffu, dk[t], 16);
       dq[t] += __shfl_xor_sync(0xffffffffu, dq[t], 16);
     }
-    // the two warps of a block add up: one writes, the other adds
-    for (int pass = 0; pass < 2; ++pass) {
-      if ((warp & 1) == pass && lane < 16)
+    for (int pass = 0; pass < 4; ++pass) {      // the four warps of a block add up, one after the other
+      if ((warp & 3) == pass)
 #pragma unroll
         for (int t = 0; t < 16; ++t) {
-          const int row = 16 * I + t;
-          float* A = sA + row * DEL_LDA + 16 * I + j;
-          float* P = sP + row * DEL_LDA + 16 * I + j;
-          if (t > j) *A += dk[t] * sB[row];
-          if (t >= j) *P += dq[t];
+          const int row = 16 * I + t, at = row * DEL_LDA + 16 * I + j;
+          if (lane < 16) {
+            if (t > j) sA[at] += dk[t] * sB[row];
+          } else {
+            if (t >= j) sP[at] += dq[t];
+          }
         }
       __syncthreads();
     }
   }
 
-  // scaled q and k, P, the chunk's total decay
-  for (int i = tid; i < DEL_C * DK; i += DEL_THREADS) {
-    const int t = i / DK, c = i % DK;
-    const float G = sG[t * LD + c], Ge = sG[(DEL_C - 1) * LD + c];
-    p.Qs[item * DEL_C * DK + i] = split_word(sQ[t * LD + c] * expf(G));
-    p.Ks[item * DEL_C * DK + i] = split_word(sK[t * LD + c] * expf(Ge - G));
+  // scaled q and k, P, the chunk's total decay; k e^G into the planes where the decays were
+  __nv_bfloat16* pKh = reinterpret_cast<__nv_bfloat16*>(sE);
+  __nv_bfloat16* pKl = pKh + DEL_C * LD;
+#pragma unroll 2
+  for (int i = tid; i < DEL_C * (DK / 8); i += FAC_THREADS) {
+    const int t = i / (DK / 8), c = i % (DK / 8) * 8;
+    float G[8], Ge[8], k[8], q[8], kg[8];
+    vload8(sG + t * LD + c, G);
+    vload8(sG + (DEL_C - 1) * LD + c, Ge);
+    vload8(sK + t * LD + c, k);
+    vload8(sQ + t * LD + c, q);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float f = fast_exp2(G[e]);
+      kg[e] = k[e] * f;
+      q[e] *= f;
+      k[e] *= fast_exp2(Ge[e] - G[e]);
+    }
+    store8_split(pKh + t * LD + c, pKl + t * LD + c, kg);
+    const size_t at = item * DEL_C * DK + t * DK + c;
+    vstore8(p.Qs + at, q);
+    store8_split(p.Ks + at + item * DEL_C * DK, p.Ks + at + (item + 1) * DEL_C * DK, k);
+    if (t == DEL_C - 1) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) p.end[item * DK + c + e] = fast_exp2(Ge[e]);
+    }
   }
-  for (int i = tid; i < DEL_C * DEL_C; i += DEL_THREADS)
-    p.P[item * DEL_C * DEL_C + i] = split_word(sP[i / DEL_C * DEL_LDA + i % DEL_C]);
-  for (int c = tid; c < DK; c += DEL_THREADS) p.end[item * DK + c] = expf(sG[(DEL_C - 1) * LD + c]);
+  for (int i = tid; i < DEL_C * (DEL_C / 8); i += FAC_THREADS) {
+    const int t = i / 8, c = i % 8 * 8;
+    float x[8];
+    vload8(sP + t * DEL_LDA + c, x);
+    const size_t at = 2 * item * DEL_C * DEL_C + t * DEL_C + c;
+    store8_split(p.P + at, p.P + at + DEL_C * DEL_C, x);
+  }
 
-  // (I + A) X = rhs by forward substitution, one column of [W | U0] per thread
-  const bool is_w = tid < DK;
-  const int col = is_w ? tid : tid - DK;
-  if (is_w || col < p.dvp) {
-    float X[DEL_C];
+  // T = (I + A)^-1: the diagonal blocks by substitution, then T_IJ = -T_II sum_K A_IK T_KJ block row by block row
+  if (tid < DEL_C) {
+    const int I = tid >> 4, c = tid & 15;
+    float x[16];
 #pragma unroll
-    for (int t = 0; t < DEL_C; ++t) {
-      float x = 0.f;
-      if (is_w) x = sB[t] * sK[t * LD + col] * expf(sG[t * LD + col]);
-      else if (t < n) x = sB[t] * __bfloat162float(p.v[(row0 + t) * p.H * p.dvp + static_cast<size_t>(h) * p.dvp + col]);
-      float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    for (int i = 0; i < 16; ++i) {
+      float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-      for (int j = 0; j < t; j += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(sA + t * DEL_LDA + j);   // zero on and above the diagonal
-        s0 = fmaf(a.x, X[j], s0);
-        if (j + 1 < t) s1 = fmaf(a.y, X[j + 1], s1);
-        if (j + 2 < t) s2 = fmaf(a.z, X[j + 2], s2);
-        if (j + 3 < t) s3 = fmaf(a.w, X[j + 3], s3);
+      for (int j = 0; j < i; j += 2) {
+        s0 = fmaf(sA[(16 * I + i) * DEL_LDA + 16 * I + j], x[j], s0);
+        if (j + 1 < i) s1 = fmaf(sA[(16 * I + i) * DEL_LDA + 16 * I + j + 1], x[j + 1], s1);
       }
-      X[t] = x - ((s0 + s1) + (s2 + s3));
-      if (is_w) p.W[(item * DEL_C + t) * DK + col] = split_word(X[t]);
-      else p.U0[(item * DEL_C + t) * p.dvp + col] = X[t];
+      x[i] = (i == c ? 1.f : 0.f) - (s0 + s1);
+      sT[(16 * I + i) * DEL_LDA + 16 * I + c] = x[i];
+    }
+  }
+  __syncthreads();
+  for (int I = 1; I < 4; ++I) {
+    for (int i = tid; i < I * 256; i += FAC_THREADS) {
+      const int r = i / (16 * I), c = i % (16 * I);
+      float z = 0.f;
+#pragma unroll 4
+      for (int k = c / 16 * 16; k < 16 * I; ++k) z = fmaf(sA[(16 * I + r) * DEL_LDA + k], sT[k * DEL_LDA + c], z);
+      sZ[r * DEL_LDA + c] = z;
+    }
+    __syncthreads();
+    for (int i = tid; i < I * 256; i += FAC_THREADS) {
+      const int r = i / (16 * I), c = i % (16 * I);
+      float z = 0.f;
+#pragma unroll
+      for (int k = 0; k < 16; ++k) z = fmaf(sT[(16 * I + r) * DEL_LDA + 16 * I + k], sZ[k * DEL_LDA + c], z);
+      sT[(16 * I + r) * DEL_LDA + c] = -z;
+    }
+    __syncthreads();
+  }
+
+  // [W | U0] = (T beta) [k e^G | v]: one row tile of 16 tokens and a quarter of the columns per warp
+  const int mt = warp & 3, grp = warp >> 2;
+  constexpr int WN = DK / 32;                       // n8 tiles of W per warp
+  float aw[WN][4] = {}, au[4][4] = {};
+  for (int ks = 0; ks <= mt; ++ks) {
+    uint32_t th[4], tl[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = ks * 16 + 2 * q4 + (i >> 1) * 8;
+      const float2 x = *reinterpret_cast<const float2*>(sT + (mt * 16 + g + (i & 1) * 8) * DEL_LDA + c);
+      split_pair(x.x * sB[c], x.y * sB[c + 1], th[i], tl[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < WN; j += 2) {
+      uint32_t bh[4], bl[4];
+      ldsm_b_kn(pKh + ks * 16 * LD + (grp * WN + j) * 8, LD, lane, bh);
+      ldsm_b_kn(pKl + ks * 16 * LD + (grp * WN + j) * 8, LD, lane, bl);
+      mma_n16(aw[j], aw[j + 1], th, bh);
+      mma_n16(aw[j], aw[j + 1], th, bl);
+      mma_n16(aw[j], aw[j + 1], tl, bh);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; j += 2) {
+      uint32_t b[4];
+      ldsm_b_kn(sV + ks * 16 * LDV + (grp * 4 + j) * 8, LDV, lane, b);
+      mma_n16(au[j], au[j + 1], th, b);
+      mma_n16(au[j], au[j + 1], tl, b);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int t = mt * 16 + g + 8 * r;
+#pragma unroll
+    for (int j = 0; j < WN; ++j) {
+      uint32_t hi, lo;
+      split_pair(aw[j][2 * r], aw[j][2 * r + 1], hi, lo);
+      const size_t at = 2 * item * DEL_C * DK + t * DK + (grp * WN + j) * 8 + 2 * q4;
+      *reinterpret_cast<uint32_t*>(p.W + at) = hi;
+      *reinterpret_cast<uint32_t*>(p.W + at + DEL_C * DK) = lo;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = (grp * 4 + j) * 8 + 2 * q4;
+      if (c < p.dvp)
+        *reinterpret_cast<float2*>(p.U0 + (item * DEL_C + t) * p.dvp + c) = make_float2(au[j][2 * r], au[j][2 * r + 1]);
     }
   }
 }
 
 // Grid (value slices of 32 channels, H, long sequences).  The state slice [DK x 32] lives in fp32 MMA accumulators and, as
-// split words, transposed in shared memory, where the two products that read it take it from.
+// hi and lo planes, in shared memory, where the two products that read it take it from.
 constexpr int DEL_SLICE = 32;
 
 template <int DK>
+struct DelScan {
+  static constexpr int LDM = DK + 8, LDP = DEL_C + 8, LDN = DEL_SLICE + 8;
+  static constexpr int W = 0;                            // [2][64][LDM]
+  static constexpr int Q = W + 2 * DEL_C * LDM;          // [64][LDM]
+  static constexpr int K = Q + DEL_C * LDM;              // [2][64][LDM]
+  static constexpr int P = K + 2 * DEL_C * LDM;          // [2][64][LDP]
+  static constexpr int S = P + 2 * DEL_C * LDP;          // [2][DK][LDN]
+  static constexpr int U = S + 2 * DK * LDN;             // [2][64][LDN]
+  static constexpr int BYTES = (U + 2 * DEL_C * LDN) * 2;
+};
+
+template <int DK>
 __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaParams p) {
-  constexpr int LDM = DK + 8, LDT = DK + 4, LDP = DEL_C + 8;
+  using L = DelScan<DK>;
+  constexpr int LDM = L::LDM, LDP = L::LDP, LDN = L::LDN;
   constexpr int SN = DK / 32;                  // n8 tiles of the state a warp owns (16 key rows each)
-  extern __shared__ __align__(16) uint32_t smw[];
-  uint32_t* sW = smw;                          // [64][LDM]
-  uint32_t* sQ = sW + DEL_C * LDM;             // [64][LDM]
-  uint32_t* sK = sQ + DEL_C * LDM;             // [64][LDT]
-  uint32_t* sP = sK + DEL_C * LDT;             // [64][LDP]
-  uint32_t* sS = sP + DEL_C * LDP;             // [32][LDM]  state, transposed
-  uint32_t* sU = sS + DEL_SLICE * LDM;         // [32][LDP]  U, transposed
+  extern __shared__ __align__(16) uint8_t sm_raw[];
+  __nv_bfloat16* sm = reinterpret_cast<__nv_bfloat16*>(sm_raw);
+  __nv_bfloat16 *sW = sm + L::W, *sQ = sm + L::Q, *sK = sm + L::K, *sP = sm + L::P, *sS = sm + L::S, *sU = sm + L::U;
   const int h = blockIdx.y, s = p.seq0 + blockIdx.z, n0 = blockIdx.x * DEL_SLICE;
   const int slot = p.slot[s];
   if (slot < 0) return;
@@ -245,19 +362,19 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
   float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * p.dkp * p.dvp;
 
-  auto copy_rows = [&](uint32_t* dst, int ld, const uint32_t* src, int width) {
-    for (int i = tid; i < DEL_C * (width / 4); i += DEL_THREADS)
-      cp_async16(dst + i / (width / 4) * ld + i % (width / 4) * 4, src + static_cast<size_t>(i) * 4);
+  auto copy_rows = [&](__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, int rows, int width) {
+    for (int i = tid; i < rows * (width / 8); i += DEL_THREADS)
+      cp_async16(dst + i / (width / 8) * ld + i % (width / 8) * 8, src + static_cast<size_t>(i) * 8);
   };
   auto load_wq = [&](int c) {
     const size_t at = (static_cast<size_t>(c) * p.H + h) * DEL_C * DK;
-    copy_rows(sW, LDM, p.W + at, DK);
-    copy_rows(sQ, LDM, p.Qs + at, DK);
+    copy_rows(sW, LDM, p.W + 2 * at, 2 * DEL_C, DK);
+    copy_rows(sQ, LDM, p.Qs + at, DEL_C, DK);
   };
   auto load_kp = [&](int c) {
     const size_t item = static_cast<size_t>(c) * p.H + h;
-    copy_rows(sK, LDT, p.Ks + item * DEL_C * DK, DK);
-    copy_rows(sP, LDP, p.P + item * DEL_C * DEL_C, DEL_C);
+    copy_rows(sK, LDM, p.Ks + 2 * item * DEL_C * DK, 2 * DEL_C, DK);
+    copy_rows(sP, LDP, p.P + 2 * item * DEL_C * DEL_C, 2 * DEL_C, DEL_C);
   };
   load_wq(c0);
   load_kp(c0);
@@ -272,14 +389,19 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
       const int i = sm_ * 16 + g + (r >> 1) * 8, c = n0 + (sn + j) * 8 + 2 * q + (r & 1);
       S[j][r] = !fresh && i < p.dkp && c < p.dvp ? st[static_cast<size_t>(i) * p.dvp + c] : 0.f;
     }
-  auto put_state = [&]() {
+  // accumulator tile (rows m0 + g, + 8; two n8 tiles from n) into hi / lo planes [rows][LDN], `lo` elements apart
+  auto put = [&](__nv_bfloat16* plane, int lo, int m0, int n, const float (&x)[4]) {
 #pragma unroll
-    for (int j = 0; j < SN; ++j)
-#pragma unroll
-      for (int r = 0; r < 4; ++r)
-        sS[((sn + j) * 8 + 2 * q + (r & 1)) * LDM + sm_ * 16 + g + (r >> 1) * 8] = split_word(S[j][r]);
+    for (int r = 0; r < 2; ++r) {
+      uint32_t hi, l;
+      split_pair(x[2 * r], x[2 * r + 1], hi, l);
+      __nv_bfloat16* d = plane + (m0 + g + 8 * r) * LDN + n + 2 * q;
+      *reinterpret_cast<uint32_t*>(d) = hi;
+      *reinterpret_cast<uint32_t*>(d + lo) = l;
+    }
   };
-  put_state();
+#pragma unroll
+  for (int j = 0; j < SN; ++j) put(sS, DK * LDN, sm_ * 16, (sn + j) * 8, S[j]);
 
   for (int c = c0; c < c1; ++c) {
     const size_t item = static_cast<size_t>(c) * p.H + h;
@@ -298,22 +420,27 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
     const float d0 = p.end[item * DK + sm_ * 16 + g], d1 = p.end[item * DK + sm_ * 16 + g + 8];
     cp_async_wait<0>();
     __syncthreads();
-    float w[2][4] = {}, o[2][4] = {};
+    float w[2][4] = {}, wl[2][4] = {}, o[2][4] = {};
 #pragma unroll
     for (int ks = 0; ks < DK / 16; ++ks) {
-      const FragA aw = lda_mk(sW + mt * 16 * LDM + ks * 16, LDM, g, q), aq = lda_mk(sQ + mt * 16 * LDM + ks * 16, LDM, g, q);
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const FragB b = ldb_nk(sS + (nb + j) * 8 * LDM + ks * 16, LDM, g, q);
-        mma_split(w[j], aw, b);
-        mma_split(o[j], aq, b);
-      }
+      uint32_t wh[4], wlo[4], qh[4], sh[4], sl[4];
+      ldsm_b_kn(sS + ks * 16 * LDN + nb * 8, LDN, lane, sh);
+      ldsm_b_kn(sS + (DK + ks * 16) * LDN + nb * 8, LDN, lane, sl);
+      ldsm_a_mk(sW + mt * 16 * LDM + ks * 16, LDM, lane, wh);
+      ldsm_a_mk(sW + (DEL_C + mt * 16) * LDM + ks * 16, LDM, lane, wlo);
+      ldsm_a_mk(sQ + mt * 16 * LDM + ks * 16, LDM, lane, qh);
+      mma_n16(w[0], w[1], wh, sh);
+      mma_n16(o[0], o[1], qh, sh);
+      mma_n16(wl[0], wl[1], wlo, sh);
+      mma_n16(o[0], o[1], qh, sl);
+      mma_n16(wl[0], wl[1], wh, sl);
     }
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
+    for (int j = 0; j < 2; ++j) {
 #pragma unroll
-      for (int r = 0; r < 4; ++r)
-        sU[((nb + j) * 8 + 2 * q + (r & 1)) * LDP + mt * 16 + g + (r >> 1) * 8] = split_word(u0[j][r] - w[j][r]);
+      for (int r = 0; r < 4; ++r) u0[j][r] -= w[j][r] + wl[j][r];
+      put(sU, DEL_C * LDN, mt * 16, (nb + j) * 8, u0[j]);
+    }
     __syncthreads();                     // U is complete; W, Q and the old state have been read
     if (c + 1 < c1) load_wq(c + 1);
     cp_async_commit();
@@ -326,16 +453,31 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
     }
 #pragma unroll
     for (int ks = 0; ks < DEL_C / 16; ++ks) {
-      const FragA a = lda_km(sK + ks * 16 * LDT + sm_ * 16, LDT, g, q);
+      uint32_t kh[4], kl[4];
+      ldsm_a_km(sK + ks * 16 * LDM + sm_ * 16, LDM, lane, kh);
+      ldsm_a_km(sK + (DEL_C + ks * 16) * LDM + sm_ * 16, LDM, lane, kl);
 #pragma unroll
-      for (int j = 0; j < SN; ++j) mma_split(S[j], a, ldb_nk(sU + (sn + j) * 8 * LDP + ks * 16, LDP, g, q));
+      for (int j = 0; j < SN; j += 2) {
+        uint32_t uh[4], ul[4];
+        ldsm_b_kn(sU + ks * 16 * LDN + (sn + j) * 8, LDN, lane, uh);
+        ldsm_b_kn(sU + (DEL_C + ks * 16) * LDN + (sn + j) * 8, LDN, lane, ul);
+        mma_n16(S[j], S[j + 1], kh, uh);
+        mma_n16(S[j], S[j + 1], kh, ul);
+        mma_n16(S[j], S[j + 1], kl, uh);
+      }
     }
+#pragma unroll
+    for (int j = 0; j < SN; ++j) put(sS, DK * LDN, sm_ * 16, (sn + j) * 8, S[j]);
     for (int ks = 0; ks <= mt; ++ks) {
-      const FragA a = lda_mk(sP + mt * 16 * LDP + ks * 16, LDP, g, q);
-#pragma unroll
-      for (int j = 0; j < 2; ++j) mma_split(o[j], a, ldb_nk(sU + (nb + j) * 8 * LDP + ks * 16, LDP, g, q));
+      uint32_t ph[4], pl[4], uh[4], ul[4];
+      ldsm_a_mk(sP + mt * 16 * LDP + ks * 16, LDP, lane, ph);
+      ldsm_a_mk(sP + (DEL_C + mt * 16) * LDP + ks * 16, LDP, lane, pl);
+      ldsm_b_kn(sU + ks * 16 * LDN + nb * 8, LDN, lane, uh);
+      ldsm_b_kn(sU + (DEL_C + ks * 16) * LDN + nb * 8, LDN, lane, ul);
+      mma_n16(o[0], o[1], ph, uh);
+      mma_n16(o[0], o[1], ph, ul);
+      mma_n16(o[0], o[1], pl, uh);
     }
-    put_state();
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -385,8 +527,8 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const float* __restri
 
 template <int DK>
 static int launch_delta(const DeltaParams& p, int nchunks, int nlong, cudaStream_t stream) {
-  const int sm1 = (4 * DEL_C * (DK + 8) + 2 * DEL_C * DEL_LDA + DEL_THREADS + DEL_C) * 4;
-  const int sm2 = (2 * DEL_C * (DK + 8) + DEL_C * (DK + 4) + DEL_C * (DEL_C + 8) + DEL_SLICE * (DK + 8) + DEL_SLICE * (DEL_C + 8)) * 4;
+  const int sm1 = DelFactor<DK>::BYTES;
+  const int sm2 = DelScan<DK>::BYTES;
   static bool set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -398,7 +540,7 @@ static int launch_delta(const DeltaParams& p, int nchunks, int nlong, cudaStream
     }
     set[dev & 63] = true;
   }
-  delta_factor_kernel<DK><<<dim3(nchunks, p.H), DEL_THREADS, sm1, stream>>>(p);
+  delta_factor_kernel<DK><<<dim3(nchunks, p.H), FAC_THREADS, sm1, stream>>>(p);
   B2_CHECK_LAUNCH("delta_factor");
   delta_scan_kernel<DK><<<dim3((p.dvp + DEL_SLICE - 1) / DEL_SLICE, p.H, nlong), DEL_THREADS, sm2, stream>>>(p);
   B2_CHECK_LAUNCH("delta_scan");
@@ -412,7 +554,7 @@ using namespace b2;
 // Words the chunked form needs per (chunk, head); the caller allocates nchunks * H times as many 32-bit words.
 B2_EXPORT int b2_delta_chunk_words(int dkp, int dvp) {
   const int DK = dkp <= 64 ? 64 : 128;
-  return 3 * DEL_C * DK + DEL_C * DEL_C + DEL_C * dvp + DK;
+  return (5 * DEL_C * DK + 2 * DEL_C * DEL_C) / 2 + DEL_C * dvp + DK;
 }
 
 // rows: the rows row0 .. row0 + rows - 1 the chunks cover (for the final stage).  o: fp32 [M, H * dvp] scratch.
@@ -432,11 +574,11 @@ B2_EXPORT int b2_delta_chunk(const float* q, const float* k, const void* v, cons
   DeltaParams p;
   p.q = q; p.k = k; p.v = static_cast<const __nv_bfloat16*>(v); p.glog = glog; p.beta = beta; p.chunks = chunks; p.first = first;
   p.start = start; p.slot = slot; p.state = state; p.o = o; p.H = H; p.G = G; p.dkp = dkp; p.dvp = dvp; p.seq0 = seq0;
-  p.W = static_cast<uint32_t*>(ws);
-  p.Qs = p.W + items * DEL_C * DK;
+  p.W = static_cast<__nv_bfloat16*>(ws);
+  p.Qs = p.W + 2 * items * DEL_C * DK;
   p.Ks = p.Qs + items * DEL_C * DK;
-  p.P = p.Ks + items * DEL_C * DK;
-  p.U0 = reinterpret_cast<float*>(p.P + items * DEL_C * DEL_C);
+  p.P = p.Ks + 2 * items * DEL_C * DK;
+  p.U0 = reinterpret_cast<float*>(p.P + 2 * items * DEL_C * DEL_C);
   p.end = p.U0 + items * DEL_C * dvp;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int rc = DK == 64 ? launch_delta<64>(p, nchunks, nlong, st) : launch_delta<128>(p, nchunks, nlong, st);

@@ -37,8 +37,8 @@ struct RetParams {
 
 __device__ __forceinline__ float ret_pow(float l2a, int n) { return n == 0 ? 1.f : exp2f(l2a * n); }
 
-// Rows of one head, rotated, times scale(t), as hi (and lo) bf16 matrices [RET_C][ld]; zero past `n` rows and dkp channels.
-template <int DK, bool LO, typename F>
+// ROWS rows of one head, rotated, times scale(t), as hi (and lo) bf16 matrices [ROWS][ld]; zero past `n` rows and dkp channels.
+template <int DK, int ROWS, bool LO, typename F>
 __device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld, const bf16_t* src, size_t row0, int n,
                                                  const RetParams& p, F scale) {
   const int half = p.rot / 2, tid = threadIdx.x, nthr = blockDim.x;
@@ -48,7 +48,8 @@ __device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld,
   };
   if (half % 8 == 0) {
     const int rv = half / 8, pieces = rv + (DK - p.rot) / 8;   // rotated pairs of 8-channel pieces, then plain pieces
-    for (int i = tid; i < RET_C * pieces; i += nthr) {
+#pragma unroll 2
+    for (int i = tid; i < ROWS * pieces; i += nthr) {
       const int t = i / pieces, c = i % pieces;
       const float f = t < n ? scale(t) : 0.f;
       if (c < rv) {
@@ -78,7 +79,7 @@ __device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld,
     }
     return;
   }
-  for (int i = tid; i < RET_C * (DK / 8); i += nthr) {
+  for (int i = tid; i < ROWS * (DK / 8); i += nthr) {
     const int t = i / (DK / 8), c8 = i % (DK / 8) * 8;
     float x[8] = {};
     if (t < n && c8 < p.dkp) {
@@ -102,6 +103,7 @@ __device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld,
 template <int DV>
 __device__ __forceinline__ void ret_load_v(bf16_t* dst, const bf16_t* src, size_t row0, int n, const RetParams& p) {
   constexpr int LDV = DV + 8;
+#pragma unroll 4
   for (int i = threadIdx.x; i < RET_C * (DV / 8); i += blockDim.x) {
     const int t = i / (DV / 8), c = i % (DV / 8) * 8;
     uint4 u = make_uint4(0, 0, 0, 0);
@@ -121,8 +123,8 @@ __global__ void __launch_bounds__(RET_THREADS, 2) ret_contrib_kernel(const RetPa
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, n = ch[2];
   const size_t row0 = ch[1];
-  const float l2a = static_cast<float>(log2(static_cast<double>(p.decay[h])));
-  ret_load_rotated<DK, true>(sKh, sKl, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p,
+  const float l2a = log2f(p.decay[h]);
+  ret_load_rotated<DK, RET_C, true>(sKh, sKl, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p,
                              [&](int t) { return p.kscale * ret_pow(l2a, n - 1 - t); });
   ret_load_v<DV>(sV, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
   __syncthreads();
@@ -160,7 +162,7 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
   const int size = p.dkp * p.dvp, i = (blockIdx.x * 256 + threadIdx.x) * 4;
   const int slot = p.slot[s];
   if (i >= size || slot < 0) return;
-  const float l2a = static_cast<float>(log2(static_cast<double>(p.decay[h])));
+  const float l2a = log2f(p.decay[h]);
   float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * size + i;
   float4 S = p.start[s] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
@@ -188,117 +190,110 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
   *reinterpret_cast<float4*>(st) = S;
 }
 
-// 16 warps: eight row tiles of 16 tokens, two warps each that share the contraction (every other k-step of q S, every other
-// block of keys) and add their results at the end.  Products with q take q's hi part only (q enters no recurrence).
-constexpr int RET_OUT_THREADS = 512;
+// Eight warps, 16 tokens each.  The state and the keys pass through one buffer in pieces of 64 rows, so that two CTAs fit on
+// an SM and one's loads run under the other's products.  Products with q take q's hi part only (q enters no recurrence).
+constexpr int RET_PIECE = 64;
 
 template <int DK, int DV>
-__host__ __device__ constexpr int ret_out_x_bytes() {   // keys, then before them the state, after them the partial results
-  int a = 2 * RET_C * (DK + 8) * 2, b = 2 * DK * (DV + 8) * 2, c = RET_C * (DV + 4) * 4;
-  return a > b ? (a > c ? a : c) : (b > c ? b : c);
+__host__ __device__ constexpr int ret_piece_elems() {
+  return 2 * RET_PIECE * (DK > DV ? DK + 8 : DV + 8);
 }
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(RET_OUT_THREADS, 1) ret_out_kernel(const RetParams p) {
-  constexpr int LDK = DK + 8, LDV = DV + 8, LDR = DV + 4, NT = DV / 8, KS = DK / 16;
+__global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams p) {
+  constexpr int LDK = DK + 8, LDV = DV + 8, NT = DV / 8, KS = DK / 16;
   extern __shared__ __align__(16) uint8_t sm_raw[];
   bf16_t* sQ = reinterpret_cast<bf16_t*>(sm_raw);
   bf16_t* sV = sQ + RET_C * LDK;
-  bf16_t* sX = sV + RET_C * LDV;
-  float* sR = reinterpret_cast<float*>(sX);
+  bf16_t* hi = sV + RET_C * LDV;
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, s = ch[0], n = ch[2];
   const size_t row0 = ch[1];
   const bool zero = ch[3] == 0 && p.start[s] == 0;       // nothing before this chunk
-  const float l2a = static_cast<float>(log2(static_cast<double>(p.decay[h])));
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3, rt = warp & 7, par = warp >> 3;
+  const float l2a = log2f(p.decay[h]);
+  const int rt = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   const bool active = rt * 16 < n;
-  ret_load_rotated<DK, false>(sQ, nullptr, LDK, p.q + static_cast<size_t>(h) * p.dkp, row0, n, p, [](int) { return 1.f; });
+  ret_load_rotated<DK, RET_C, false>(sQ, nullptr, LDK, p.q + static_cast<size_t>(h) * p.dkp, row0, n, p, [](int) { return 1.f; });
   ret_load_v<DV>(sV, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
   float acc[NT][4] = {};
   if (!zero) {
-    bf16_t* hi = sX;
-    bf16_t* lo = sX + DK * LDV;
+    bf16_t* lo = hi + RET_PIECE * LDV;
     const float* w = p.ws + (static_cast<size_t>(blockIdx.x) * p.H + h) * p.dkp * p.dvp;
-    for (int i = threadIdx.x; i < DK * (DV / 8); i += RET_OUT_THREADS) {
-      const int r = i / (DV / 8), c = i % (DV / 8) * 8;
-      float x[8] = {};
-      if (r < p.dkp && c < p.dvp) vload8(w + static_cast<size_t>(r) * p.dvp + c, x);
-      store8_split(hi + r * LDV + c, lo + r * LDV + c, x);
-    }
-    __syncthreads();
-    if (active) {
-      for (int ks = par; ks < KS; ks += 2) {
-        uint32_t a[4];
-        ldsm_a_mk(sQ + rt * 16 * LDK + ks * 16, LDK, lane, a);
+    for (int r0 = 0; r0 < DK; r0 += RET_PIECE) {
+      if (r0 > 0) __syncthreads();
+#pragma unroll 4
+      for (int i = threadIdx.x; i < RET_PIECE * (DV / 8); i += RET_THREADS) {
+        const int r = i / (DV / 8), c = i % (DV / 8) * 8;
+        float x[8] = {};
+        if (r0 + r < p.dkp && c < p.dvp) vload8(w + static_cast<size_t>(r0 + r) * p.dvp + c, x);
+        store8_split(hi + r * LDV + c, lo + r * LDV + c, x);
+      }
+      __syncthreads();
+      if (active)
 #pragma unroll
-        for (int j = 0; j < NT; j += 2) {
-          uint32_t b[4];
-          ldsm_b_kn(hi + ks * 16 * LDV + j * 8, LDV, lane, b);
-          mma_n16(acc[j], acc[j + 1], a, b);
-          ldsm_b_kn(lo + ks * 16 * LDV + j * 8, LDV, lane, b);
-          mma_n16(acc[j], acc[j + 1], a, b);
+        for (int ks = 0; ks < RET_PIECE / 16; ++ks) {
+          uint32_t a[4];
+          ldsm_a_mk(sQ + rt * 16 * LDK + r0 + ks * 16, LDK, lane, a);
+#pragma unroll
+          for (int j = 0; j < NT; j += 2) {
+            uint32_t b[4];
+            ldsm_b_kn(hi + ks * 16 * LDV + j * 8, LDV, lane, b);
+            mma_n16(acc[j], acc[j + 1], a, b);
+            ldsm_b_kn(lo + ks * 16 * LDV + j * 8, LDV, lane, b);
+            mma_n16(acc[j], acc[j + 1], a, b);
+          }
         }
-      }
-      const float f0 = ret_pow(l2a, rt * 16 + g + 1), f1 = ret_pow(l2a, rt * 16 + g + 9);
+    }
+    const float f0 = ret_pow(l2a, rt * 16 + g + 1), f1 = ret_pow(l2a, rt * 16 + g + 9);
 #pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        acc[j][0] *= f0;
-        acc[j][1] *= f0;
-        acc[j][2] *= f1;
-        acc[j][3] *= f1;
-      }
+    for (int j = 0; j < NT; ++j) {
+      acc[j][0] *= f0;
+      acc[j][1] *= f0;
+      acc[j][2] *= f1;
+      acc[j][3] *= f1;
     }
     __syncthreads();
   }
-  bf16_t* kh = sX;
-  bf16_t* kl = sX + RET_C * LDK;
-  ret_load_rotated<DK, true>(kh, kl, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p, [&](int) { return p.kscale; });
-  __syncthreads();
-  for (int kb = par; active && kb <= rt; kb += 2) {          // 16 keys at a time, up to the diagonal
-    float sc[2][4] = {};
+  bf16_t* lo = hi + RET_PIECE * LDK;
+  for (int k0 = 0; k0 < n; k0 += RET_PIECE) {
+    if (k0 > 0) __syncthreads();
+    ret_load_rotated<DK, RET_PIECE, true>(hi, lo, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0 + k0, n - k0, p,
+                                          [&](int) { return p.kscale; });
+    __syncthreads();
+    for (int kb = 0; active && kb < RET_PIECE / 16 && k0 / 16 + kb <= rt; ++kb) {     // 16 keys at a time, up to the diagonal
+      float sc[2][4] = {};
 #pragma unroll
-    for (int ks = 0; ks < KS; ++ks) {
-      uint32_t a[4], b[4];
-      ldsm_a_mk(sQ + rt * 16 * LDK + ks * 16, LDK, lane, a);
-      ldsm_b_nk(kh + kb * 16 * LDK + ks * 16, LDK, lane, b);
-      mma_n16(sc[0], sc[1], a, b);
-      ldsm_b_nk(kl + kb * 16 * LDK + ks * 16, LDK, lane, b);
-      mma_n16(sc[0], sc[1], a, b);
-    }
-    uint32_t ph[4], pl[4];
-#pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int d = rt * 16 + g + 8 * r - (kb * 16 + j * 8 + 2 * q);     // distance to the first of the two keys
-        const float x0 = d >= 0 ? sc[j][2 * r] * ret_pow(l2a, d) : 0.f;
-        const float x1 = d >= 1 ? sc[j][2 * r + 1] * ret_pow(l2a, d - 1) : 0.f;
-        split_pair(x0, x1, ph[2 * j + r], pl[2 * j + r]);
+      for (int ks = 0; ks < KS; ++ks) {
+        uint32_t a[4], b[4];
+        ldsm_a_mk(sQ + rt * 16 * LDK + ks * 16, LDK, lane, a);
+        ldsm_b_nk(hi + kb * 16 * LDK + ks * 16, LDK, lane, b);
+        mma_n16(sc[0], sc[1], a, b);
+        ldsm_b_nk(lo + kb * 16 * LDK + ks * 16, LDK, lane, b);
+        mma_n16(sc[0], sc[1], a, b);
       }
+      uint32_t ph[4], pl[4];
 #pragma unroll
-    for (int j = 0; j < NT; j += 2) {
-      uint32_t b[4];
-      ldsm_b_kn(sV + kb * 16 * LDV + j * 8, LDV, lane, b);
-      mma_n16(acc[j], acc[j + 1], ph, b);
-      mma_n16(acc[j], acc[j + 1], pl, b);
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int d = rt * 16 + g + 8 * r - (k0 + kb * 16 + j * 8 + 2 * q);     // distance to the first of the two keys
+          const float x0 = d >= 0 ? sc[j][2 * r] * ret_pow(l2a, d) : 0.f;
+          const float x1 = d >= 1 ? sc[j][2 * r + 1] * ret_pow(l2a, d - 1) : 0.f;
+          split_pair(x0, x1, ph[2 * j + r], pl[2 * j + r]);
+        }
+#pragma unroll
+      for (int j = 0; j < NT; j += 2) {
+        uint32_t b[4];
+        ldsm_b_kn(sV + (k0 + kb * 16) * LDV + j * 8, LDV, lane, b);
+        mma_n16(acc[j], acc[j + 1], ph, b);
+        mma_n16(acc[j], acc[j + 1], pl, b);
+      }
     }
   }
-  __syncthreads();
-  if (par == 1 && active)
-#pragma unroll
-    for (int j = 0; j < NT; ++j)
-#pragma unroll
-      for (int r = 0; r < 2; ++r)
-        *reinterpret_cast<float2*>(sR + (rt * 16 + g + 8 * r) * LDR + j * 8 + 2 * q) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
-  __syncthreads();
-  if (par == 1 || !active) return;
+  if (!active) return;
   float s0 = 0.f, s1 = 0.f;
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
-    const float2 x = *reinterpret_cast<const float2*>(sR + (rt * 16 + g) * LDR + j * 8 + 2 * q);
-    const float2 y = *reinterpret_cast<const float2*>(sR + (rt * 16 + g + 8) * LDR + j * 8 + 2 * q);
-    acc[j][0] += x.x; acc[j][1] += x.y; acc[j][2] += y.x; acc[j][3] += y.y;
     s0 += acc[j][0] * acc[j][0] + acc[j][1] * acc[j][1];
     s1 += acc[j][2] * acc[j][2] + acc[j][3] * acc[j][3];
   }
@@ -328,7 +323,7 @@ __global__ void __launch_bounds__(RET_OUT_THREADS, 1) ret_out_kernel(const RetPa
 template <int DK, int DV>
 static int launch_ret(const RetParams& p, int nchunks, int nlong, cudaStream_t stream) {
   const int sm1 = RET_C * (2 * (DK + 8) + DV + 8) * 2;
-  const int sm3 = RET_C * (DK + 8 + DV + 8) * 2 + ret_out_x_bytes<DK, DV>();
+  const int sm3 = (RET_C * (DK + 8 + DV + 8) + ret_piece_elems<DK, DV>()) * 2;
   static bool set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -344,7 +339,7 @@ static int launch_ret(const RetParams& p, int nchunks, int nlong, cudaStream_t s
   B2_CHECK_LAUNCH("ret_contrib");
   ret_scan_kernel<<<dim3((p.dkp * p.dvp / 4 + 255) / 256, p.H, nlong), 256, 0, stream>>>(p);
   B2_CHECK_LAUNCH("ret_scan");
-  ret_out_kernel<DK, DV><<<dim3(nchunks, p.H), RET_OUT_THREADS, sm3, stream>>>(p);
+  ret_out_kernel<DK, DV><<<dim3(nchunks, p.H), RET_THREADS, sm3, stream>>>(p);
   B2_CHECK_LAUNCH("ret_out");
   return 0;
 }
