@@ -377,6 +377,7 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
     copy_rows(sP, LDP, p.P + 2 * item * DEL_C * DEL_C, 2 * DEL_C, DEL_C);
   };
   load_wq(c0);
+  cp_async_commit();
   load_kp(c0);
   cp_async_commit();
 
@@ -418,7 +419,7 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
         u0[j][2 * r + 1] = x.y;
       }
     const float d0 = p.end[item * DK + sm_ * 16 + g], d1 = p.end[item * DK + sm_ * 16 + g + 8];
-    cp_async_wait<0>();
+    cp_async_wait<1>();                  // W and Q of this chunk; K and P may still be on their way
     __syncthreads();
     float w[2][4] = {}, wl[2][4] = {}, o[2][4] = {};
 #pragma unroll
@@ -441,6 +442,7 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
       for (int r = 0; r < 4; ++r) u0[j][r] -= w[j][r] + wl[j][r];
       put(sU, DEL_C * LDN, mt * 16, (nb + j) * 8, u0[j]);
     }
+    cp_async_wait<0>();
     __syncthreads();                     // U is complete; W, Q and the old state have been read
     if (c + 1 < c1) load_wq(c + 1);
     cp_async_commit();

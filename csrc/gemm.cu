@@ -635,9 +635,49 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 #pragma unroll 1
       for (int c = 0; c < BN / 32; ++c) {
         uint32_t r[32];
+        const int col0 = n0 + c * 32;
+        if (out_fp32 && !residual && col0 + 32 <= N) {
+          // fp32 rows through a 4 KiB staging block of this warp: every global access then covers four complete 128-byte
+          // lines (8 lanes a row).  The addend is requested before the accumulator is read.
+          uint8_t* stage = slabs + quarter * 8192 + (c & 1) * 4096;
+          const int chunk = lane & 7, row_w = m_blk * GEMM_BM + quarter * 32;
+          float* cp = reinterpret_cast<float*>(Cout) + static_cast<size_t>(row_w) * ldc + col0 + chunk * 4;
+          float4 p[8];
+          if (accumulate && !atomic_out) {
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+              const int rr = 4 * k + (lane >> 3);
+              p[k] = row_w + rr < M ? *reinterpret_cast<const float4*>(cp + static_cast<size_t>(rr) * ldc)
+                                    : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+          }
+          tmem_ld_32x32b_x32(t_base + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+            *reinterpret_cast<uint4*>(stage + lane * 128 + ((j ^ (lane & 7)) << 4)) =
+                make_uint4(r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
+          __syncwarp();
+#pragma unroll
+          for (int k = 0; k < 8; ++k) {
+            const int rr = 4 * k + (lane >> 3);
+            float4 o = *reinterpret_cast<const float4*>(stage + rr * 128 + ((chunk ^ (rr & 7)) << 4));
+            if (row_w + rr >= M) continue;
+            float4* dst = reinterpret_cast<float4*>(cp + static_cast<size_t>(rr) * ldc);
+            if (atomic_out) {
+              atomicAdd(dst, o);
+              continue;
+            }
+            if (accumulate) {
+              o.x += p[k].x; o.y += p[k].y; o.z += p[k].z; o.w += p[k].w;
+            }
+            *dst = o;
+          }
+          __syncwarp();
+          continue;
+        }
         tmem_ld_32x32b_x32(t_base + c * 32, r);
         tmem_ld_wait();
-        const int col0 = n0 + c * 32;
         if (row < M && col0 < N) {
           const size_t off = static_cast<size_t>(row) * ldc + col0;
           const bool full = (col0 + 32 <= N);
