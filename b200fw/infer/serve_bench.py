@@ -26,8 +26,7 @@ def _prompts(n: int, length: int, vocab: int, seed: int = 0) -> List[List[int]]:
     return [[r.randrange(3, vocab) for _ in range(length)] for _ in range(n)]
 
 
-def throughput(preset: str, batch: int = 256, prompt: int = 1024, new_tokens: int = 64, warmup: int = 3,
-               budget: int = 8192) -> Dict:
+def throughput(preset: str, batch: int = 256, prompt: int = 1024, new_tokens: int = 64, budget: int = 8192) -> Dict:
     """``batch`` requests of ``prompt`` tokens, ``new_tokens`` each: tokens/s of the prompt phase and of the decode phase, and
     the whole call from pinned host ids to host ids."""
     mc = PRESETS[preset]
@@ -35,7 +34,8 @@ def throughput(preset: str, batch: int = 256, prompt: int = 1024, new_tokens: in
     model.init_weights(0)
     for p in model.parameters():
         p.requires_grad_(False)
-    blocks = batch * (-(-(prompt + new_tokens + warmup + 2) // 16) + 1) + 64
+    warmup = -(-batch * prompt // budget) + 4       # long enough that the whole batch decodes together
+    blocks = batch * (-(-(prompt + max(new_tokens, warmup) + 2) // 16) + 1) + 64
     eng = InferenceEngine(InferenceConfig.from_model_config(
         mc, num_blocks=blocks, inference_mode="kv_cache", max_num_batched_tokens=budget + batch, max_prefill_tokens=budget,
         chunk_size=2048, max_num_sequences=batch, enable_cuda_graph=True, temperature=0.0, eos_token_id=None,

@@ -8,6 +8,9 @@ weights.  ``--model qwen3-32b --tp 8`` runs the TP8 large-model configuration on
 One "step" is one optimizer step (all its micro-batches, gradient reduction, clip, AdamW).  Prints one
 JSON line on rank 0.  ``--impl reference`` runs the unmodified reference implementation installed under
 ``baseline/_ref`` on the same workload through its own TrainEngine.
+
+``--serve PRESETS`` instead measures serving (one GPU): prefill and decode throughput of each preset through the inference
+engine, and with ``--serve-kernels`` the roofline of every kernel of a layer.  One JSON line as well.
 """
 from __future__ import annotations
 
@@ -57,7 +60,31 @@ def parse():
                     help="override the preset's layer count (smoke runs of a large architecture; not a benchmark config)")
     ap.add_argument("--fused-tp", action="store_true",
                     help="run the sequence-parallel collectives inside the GEMM kernels (peer memory) instead of NCCL")
+    ap.add_argument("--serve", default="", metavar="PRESETS",
+                    help="serving throughput of these model presets (comma-separated) instead of the training step")
+    ap.add_argument("--serve-kernels", action="store_true", help="with --serve: time every kernel of a layer too")
+    ap.add_argument("--serve-batch", type=int, default=256)
+    ap.add_argument("--serve-prompt", type=int, default=1024)
+    ap.add_argument("--serve-tokens", type=int, default=64)
     return ap.parse_args()
+
+
+def run_serve(a):
+    from b200fw.infer import serve_bench
+    line = {"metric": "serve_tokens_per_s", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16",
+            "data": "synthetic (seeded uniform tokens, random-init weights)", "impl": "b200fw",
+            "l2": "weights and caches larger than L2 (phases); flushed before every launch (kernels)", "models": {}}
+    sampler = ClockSampler(0)
+    sampler.start()
+    for name in a.serve.split(","):
+        m = {"engine": serve_bench.throughput(name, a.serve_batch, a.serve_prompt, a.serve_tokens),
+             "prefill": [serve_bench.prefill_once(name, n) for n in ([2048] * 4, [8192], [256] * 32)]}
+        if a.serve_kernels:
+            m["kernels"] = {"prefill 4 x 2048": serve_bench.kernels(name, lengths=[2048] * 4),
+                            "decode 256 @ 1024": serve_bench.kernels(name), "decode 32 @ 1024": serve_bench.kernels(name, batch=32)}
+        line["models"][name] = m
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line), flush=True)
 
 
 def synthetic_batches(vocab, micro_batch, seq, count, seed, pinned):
@@ -227,6 +254,9 @@ def main():
         return
     if not torch.cuda.is_available():
         print(json.dumps({"impl": "b200fw", "unavailable": "no CUDA device"}))
+        return
+    if a.serve:
+        run_serve(a)
         return
     run_ours(a)
 

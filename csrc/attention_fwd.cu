@@ -355,6 +355,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         // this head's bias by distance, constant past the last bucketed one
         // every warp has written its part of the previous item out
         if (!tab_sync()) { ok = false; break; }
+#pragma unroll 4
         for (int d = static_cast<int>(threadIdx.x) - 64 - EXT_TAB_NEG; d < ext.nbucket + EXT_TAB_FAR; d += 256) {
           const int b = ext.bucket[min(max(d, 0), ext.nbucket - 1)];
           tab[d] = __bfloat162float(ext.rel[static_cast<size_t>(b) * Hq + item.head]) * 1.4426950408889634f;
@@ -484,7 +485,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       float inv = 1.f / lsum;
       if (EXT) {
         float den = lsum;
-        if (ext.sink != nullptr) den += exp2f(fmaf(__bfloat162float(ext.sink[item.head]), 1.4426950408889634f, -m_used));
+        if (ext.sink != nullptr) den += fast_exp2(fmaf(__bfloat162float(ext.sink[item.head]), 1.4426950408889634f, -m_used));
         inv = 1.f / den;
         if (ext.gate != nullptr && q_idx < item.q_len)
           inv /= 1.f + expf(-__bfloat162float(ext.gate[static_cast<size_t>(item.row0 + r) * ext.ld_gate + item.head]));

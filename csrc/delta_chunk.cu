@@ -522,8 +522,8 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const float* __restri
     w1 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(w + c + 2));
   }
   uint2 y;
-  y.x = pack_bf16x2(x.x * r * w0.x * sigmoid_f(gt.x), x.y * r * w0.y * sigmoid_f(gt.y));
-  y.y = pack_bf16x2(x.z * r * w1.x * sigmoid_f(gt.z), x.w * r * w1.y * sigmoid_f(gt.w));
+  y.x = pack_bf16x2(x.x * r * w0.x * sigmoid_fast(gt.x), x.y * r * w0.y * sigmoid_fast(gt.y));
+  y.y = pack_bf16x2(x.z * r * w1.x * sigmoid_fast(gt.z), x.w * r * w1.y * sigmoid_fast(gt.w));
   *reinterpret_cast<uint2*>(out + row * ld_out + static_cast<size_t>(h) * dvp + c) = y;
 }
 

@@ -181,9 +181,9 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
         const size_t gi = row * p.ld_gate + static_cast<size_t>(h) * p.dvp + c;
         if (DELTA) {
           if (p.norm_w) o *= to_f(static_cast<const T*>(p.norm_w)[c]);
-          o *= sigmoid_f(static_cast<const float*>(p.gate)[gi]);
+          o *= sigmoid_t<T>(static_cast<const float*>(p.gate)[gi]);
         } else {
-          o *= silu_f(to_f(static_cast<const T*>(p.gate)[gi]));
+          o *= silu_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
         }
         static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(h) * p.dvp + c] = from_f<T>(o);
       }
@@ -310,9 +310,9 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
     const size_t gi = row * p.ld_gate + static_cast<size_t>(h) * DV + c;
     if (DELTA) {
       if (p.norm_w) x *= to_f(static_cast<const T*>(p.norm_w)[c]);
-      x *= sigmoid_f(static_cast<const float*>(p.gate)[gi]);
+      x *= sigmoid_t<T>(static_cast<const float*>(p.gate)[gi]);
     } else {
-      x *= silu_f(to_f(static_cast<const T*>(p.gate)[gi]));
+      x *= silu_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
     }
     static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(h) * DV + c] = from_f<T>(x);
   }
@@ -380,7 +380,7 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(const DeltaPre
           else if (!fresh) xv = cst[static_cast<size_t>(c) * (K - 1) + (K - 1 + at)];
           acc = fmaf(to_f(taps[static_cast<size_t>(c) * K + K - 1 - j]), xv, acc);
         }
-        val[m] = silu_f(acc);
+        val[m] = silu_t<T>(acc);
         ss = fmaf(val[m], val[m], ss);
       }
     }
@@ -476,7 +476,7 @@ __device__ __forceinline__ void prep_conv_job(const DeltaPrepParams& p, int s, i
       float a = cur[e] * taps[e * K + K - 1];
 #pragma unroll
       for (int i = 0; i < K - 1; ++i) a = fmaf(w[i][e], taps[e * K + K - 2 - i], a);
-      y[e] = silu_f(a);
+      y[e] = silu_t<T>(a);
       ss = fmaf(y[e], y[e], ss);
     }
 #pragma unroll

@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(RES_THREADS) glu_kernel(const T* __restrict__ 
     vload8(gate + row * ld_in + c, g);
     vload8(up + row * ld_in + c, u);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) g[e] = silu_f(g[e]) * u[e];
+    for (int e = 0; e < 8; ++e) g[e] = silu_t<T>(g[e]) * u[e];
     vstore8(out + row * ld_out + c, g);
   }
 }

@@ -35,7 +35,7 @@ struct RetParams {
   float kscale, eps;
 };
 
-__device__ __forceinline__ float ret_pow(float l2a, int n) { return n == 0 ? 1.f : exp2f(l2a * n); }
+__device__ __forceinline__ float ret_pow(float l2a, int n) { return n == 0 ? 1.f : fast_exp2(l2a * n); }
 
 // ROWS rows of one head, rotated, times scale(t), as hi (and lo) bf16 matrices [ROWS][ld]; zero past `n` rows and dkp channels.
 template <int DK, int ROWS, bool LO, typename F>
@@ -315,7 +315,7 @@ __global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams
       if (c >= p.dvp) break;
       const float2 gv = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(gp + c));
       const float f = r ? r1 : r0;
-      *reinterpret_cast<uint32_t*>(op + c) = pack_bf16x2(acc[j][2 * r] * f * silu_f(gv.x), acc[j][2 * r + 1] * f * silu_f(gv.y));
+      *reinterpret_cast<uint32_t*>(op + c) = pack_bf16x2(acc[j][2 * r] * f * silu_fast(gv.x), acc[j][2 * r + 1] * f * silu_fast(gv.y));
     }
   }
 }

@@ -46,6 +46,14 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
+// Forms for values that are rounded to bf16 next (relative error about 2^-21): one special-function 2^x and one reciprocal.
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + fast_exp2(-1.4426950408889634f * z)); }
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + fast_exp2(-1.4426950408889634f * z)); }
+template <typename T>
+__device__ __forceinline__ float silu_t(float z) { return sizeof(T) == 2 ? silu_fast(z) : silu_f(z); }
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float z) { return sizeof(T) == 2 ? sigmoid_fast(z) : sigmoid_f(z); }
+
 }  // namespace b2
 
 // bf16 / fp32 dispatch of a launcher body: `T` is the activation type inside the braces
