@@ -478,3 +478,46 @@ def test_bad_checkpoints_and_configs(tmp_path):
     assert eng.prefix_cache is None
     for name in ("fetelorn-tiny", "fetelorn-0.6b"):
         assert registry.PRESETS[name].num_params() > 0
+
+
+# ---- kernels the model leans on -----------------------------------------------------------------------------------------
+@pytest.mark.gpu
+@pytest.mark.parametrize("M,N,K", [(1, 8, 8), (3, 40, 24), (130, 200, 72), (257, 1000, 640)])
+def test_gemm_32bit_and_fp32_outputs(M, N, K):
+    a, b = torch.randn(M, K, device="cuda"), torch.randn(N, K, device="cuda")
+    c = torch.randn(M, N, device="cuda")
+    want = a.double() @ b.double().t()
+    torch.testing.assert_close(ops.gemm(a, b).double(), want, rtol=1e-5, atol=1e-4)
+    torch.testing.assert_close(ops.gemm(a, b, out=c.clone(), accumulate=True).double(), want + c.double(), rtol=1e-5, atol=1e-4)
+    ah, bh = a.bfloat16(), b.bfloat16()
+    want = ah.double() @ bh.double().t()
+    got = ops.gemm(ah, bh, out=torch.empty(M, N, device="cuda"))
+    torch.testing.assert_close(got.double(), want, rtol=1e-4, atol=1e-3)
+    got = ops.gemm(ah, bh, out=c.clone(), accumulate=True)
+    torch.testing.assert_close(got.double(), want + c.double(), rtol=1e-4, atol=1e-3)
+
+
+@pytest.mark.parametrize("run", RUNS)
+@pytest.mark.parametrize("n", [8, 42, 200, 9000])
+def test_residual_ops(run, n):
+    ld, M, eps = pad8(n), 5, 1e-5
+    x, a, b = (torch.nn.functional.pad(randn(M, n, seed=i), (0, ld - n)) for i in (1, 2, 3))
+    wa, wb, wn = (torch.nn.functional.pad(1 + 0.1 * randn(n, seed=i), (0, ld - n)).to(run[1]).to(run[0]) for i in (4, 5, 6))
+    d = lambda t: t.to(run[0])  # noqa: E731
+    rows = torch.tensor([3, 0, 3], device=run[0])
+    h = ops.rmsnorm_f32(d(x), wn, n, eps, rows)
+    want = O.rms(x[rows.cpu(), :n].double(), eps) * wn[:n].double().cpu()
+    t = dict(rtol=1e-2, atol=1e-2) if run[1] == torch.bfloat16 else dict(rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(h[:, :n].double().cpu(), want, **t)
+    assert not h[:, n:].any()
+    y = d(x).clone()
+    h = ops.merge_norm_add(y, d(a), d(b), wa, wb, 0.5, n, eps, wn)
+    s = x[:, :n].double() + 0.5 * (O.rms(a[:, :n].double(), eps) * wa[:n].double().cpu() + O.rms(b[:, :n].double(), eps) * wb[:n].double().cpu())
+    torch.testing.assert_close(y[:, :n].double().cpu(), s, rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(h[:, :n].double().cpu(), O.rms(s, eps) * wn[:n].double().cpu(), **t)
+    assert not h[:, n:].any() and ops.merge_norm_add(y, d(a), d(b), wa, wb, 0.5, n, eps) is None
+    gu = torch.cat([a, b], 1).to(run[1]).to(run[0])
+    out = torch.empty(M, ld, dtype=run[1], device=run[0])
+    ops.glu(gu[:, :ld], gu[:, ld:], out)
+    g, u = gu[:, :ld].double().cpu(), gu[:, ld:].double().cpu()
+    torch.testing.assert_close(out.double().cpu(), O.silu(g) * u, **t)

@@ -161,3 +161,18 @@ inference_preview: {{enabled: false, max_tokens: 4}}
     assert r.returncode == 0, (r.stdout + r.stderr)[-2000:]
     assert f"continuing at iteration {done} of {done + 2}" in r.stdout + r.stderr
     assert json.loads(r.stdout[r.stdout.index("{"):])["completed_iterations"] == 2
+
+
+def test_run_inference_serves_a_hybrid_model(tmp_path):
+    """The architecture follows from the folder's config.json; the same flags as for any other model."""
+    import torch
+
+    from b200fw.model import registry
+    m = registry.build_model(registry.PRESETS["fetelorn-tiny"], dtype=torch.bfloat16, device="cpu")
+    m.init_weights(3)
+    registry.save_checkpoint(m, str(tmp_path))
+    r = subprocess.run([sys.executable, os.path.join(ROOT, "scripts", "run_inference.py"), "-m", str(tmp_path), "--num-prompts", "3",
+                        "--prompt-len", "20", "--max-tokens", "3", "--temperature", "0", "--num-blocks", "32"],
+                       capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr[-800:]
+    assert json.loads(r.stdout)["generated_tokens"] == 9
