@@ -29,6 +29,7 @@ struct FwdExt {
   const __nv_bfloat16* gate;  // [rows, ld_gate] (Hq columns) or null
   long long ld_gate, ld_out;
   int dkp, dvp;           // head sizes, multiples of 8
+  int tpc;                // > 0: query tiles per chunk; items are then ordered by their place in the chunk, heaviest first
 };
 constexpr int EXT_TAB_NEG = 256;    // table entries below distance 0 (masked keys of a diagonal tile)
 constexpr int EXT_TAB_FAR = 256;    // entries past the last bucketed distance: no clamping inside a tile
@@ -78,6 +79,11 @@ __device__ __forceinline__ FwdItem fwd_item(int w, const FwdParams& p, const Fwd
   it.kv_off = it.kv_len - it.q_len;
   const int num_q_tiles = (it.q_len + 127) / 128;
   it.qt = num_q_tiles - 1 - x;
+  if (EXT && x_.tpc > 0) {   // max_tiles is a multiple of tpc; tiles past the sequence's last one are inactive
+    const int chunks = p.max_tiles / x_.tpc;
+    it.qt = x % chunks * x_.tpc + x_.tpc - 1 - x / chunks;
+    if (it.qt >= num_q_tiles) it.qt = -1;
+  }
   it.active = it.qt >= 0 && it.q_len > 0;
   it.kvh = it.head / (p.Hq / p.Hkv);
   const int last_key = min(it.kv_len, it.kv_off + (it.qt + 1) * 128);  // exclusive
@@ -350,6 +356,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const int q_idx = item.qt * 128 + r;      // index among this sequence's queries
       const int q_pos = item.kv_off + q_idx;    // last key this query may see
       float m_used = EXT ? -1e30f : -INFINITY, l = 0.f;        // l: this thread's 64 columns only
+      // requested now, used at the end of the item
+      const float gate_raw = EXT && ext.gate != nullptr && q_idx < item.q_len
+                                 ? __bfloat162float(ext.gate[static_cast<size_t>(item.row0 + r) * ext.ld_gate + item.head]) : 0.f;
+      const float sink2 = EXT && ext.sink != nullptr ? __bfloat162float(ext.sink[item.head]) * 1.4426950408889634f : 0.f;
       const int first_key = EXT && ext.chunk > 0 ? q_pos / ext.chunk * ext.chunk : 0;
       if (EXT && ext.rel != nullptr) {
         // this head's bias by distance, constant past the last bucketed one
@@ -485,10 +495,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       float inv = 1.f / lsum;
       if (EXT) {
         float den = lsum;
-        if (ext.sink != nullptr) den += fast_exp2(fmaf(__bfloat162float(ext.sink[item.head]), 1.4426950408889634f, -m_used));
-        inv = 1.f / den;
-        if (ext.gate != nullptr && q_idx < item.q_len)
-          inv /= 1.f + expf(-__bfloat162float(ext.gate[static_cast<size_t>(item.row0 + r) * ext.ld_gate + item.head]));
+        if (ext.sink != nullptr) den += fast_exp2(sink2 - m_used);
+        if (ext.gate != nullptr) den *= 1.f + fast_exp2(-1.4426950408889634f * gate_raw);
+        inv = __fdividef(1.f, den);
       }
       const bool in_range = q_idx < item.q_len;
       uint4 ov[8];
@@ -701,6 +710,8 @@ B2_EXPORT int b2_attn_fwd_paged_ext(const void* q, const void* k_cache, const vo
   e.start = start; e.chunk = chunk; e.rel = static_cast<const __nv_bfloat16*>(rel); e.bucket = bucket; e.nbucket = nbucket;
   e.sink = static_cast<const __nv_bfloat16*>(sink); e.gate = static_cast<const __nv_bfloat16*>(gate); e.ld_gate = ld_gate;
   e.ld_out = ld_out; e.dkp = dkp; e.dvp = dvp;
+  e.tpc = chunk >= 256 && chunk < max_q ? (chunk + 127) / 128 : 0;
+  if (e.tpc > 0) prm.max_tiles = (prm.max_tiles + e.tpc - 1) / e.tpc * e.tpc;
   const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
   const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
   attn_fwd_kernel<true><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(*tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), nullptr, prm, e,

@@ -829,7 +829,8 @@ static int launch_gemm(const void* A, const void* B, void* C, const void* R, int
     const char* e = std::getenv("B200FW_DETERMINISTIC");
     return e != nullptr && e[0] == '1';
   }();
-  if (COMM == 0 && out_fp32 && !(flags & GEMM_RESIDUAL) && !deterministic) {
+  // With several waves of tiles anyway the slices' atomic traffic costs more than the shorter last wave saves.
+  if (COMM == 0 && out_fp32 && !(flags & GEMM_RESIDUAL) && !deterministic && num_tiles < 4 * grid) {
     const int num_kb = (K + GEMM_BK - 1) / GEMM_BK;
     double best = static_cast<double>((num_tiles + grid - 1) / grid);
     for (int sk = 2; sk <= 4 && num_kb / sk >= 16; ++sk) {
