@@ -4,7 +4,10 @@
 //   2. the running state at every chunk's start: S_c = a^n S_{c-1} + contribution                   (a scan, element-wise)
 //   3. o = a^{t+1} S_c^T q + sum_{j <= t} a^{t-j} (q . k_j) v_j, per-head norm, gate, store         (all chunks at once)
 //
-// Products run on tensor cores with fp32 operands split into two bf16 numbers (mma_split.cuh); v is exact in bf16.
+// The products are tcgen05 MMAs of one 128-token tile with fp32 accumulators in TMEM.  An fp32 operand that enters the
+// recurrence or weighs a value (k, the state, the weights) is the sum of two bf16 numbers, hi + lo, and takes two MMAs;
+// v is exact in bf16, and q, which enters no recurrence, is rounded to bf16.  The operands are computed on the way in
+// (rotation, decays, split), so the threads write the 128-byte-swizzled tiles themselves instead of TMA.
 #include "host.h"
 #include "mma_split.cuh"
 #include "vec.cuh"
@@ -37,19 +40,27 @@ struct RetParams {
 
 __device__ __forceinline__ float ret_pow(float l2a, int n) { return n == 0 ? 1.f : fast_exp2(l2a * n); }
 
-// ROWS rows of one head, rotated, times scale(t), as hi (and lo) bf16 matrices [ROWS][ld]; zero past `n` rows and dkp channels.
-template <int DK, int ROWS, bool LO, typename F>
-__device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld, const bf16_t* src, size_t row0, int n,
+// Swizzled bf16 tile: halves of 64 columns, each [rows x 128 bytes]; `c` is a multiple of 8.
+__device__ __forceinline__ uint8_t* ret_at(uint8_t* tile, int half_bytes, int row, int c) {
+  return tile + (c >> 6) * half_bytes + row * 128 + ((((c >> 3) & 7) ^ (row & 7)) << 4);
+}
+template <bool LO>
+__device__ __forceinline__ void ret_put(uint8_t* hi, uint8_t* lo, int half_bytes, int row, int c, const float (&f)[8]) {
+  bf16_t* h = reinterpret_cast<bf16_t*>(ret_at(hi, half_bytes, row, c));
+  if (LO) store8_split(h, reinterpret_cast<bf16_t*>(ret_at(lo, half_bytes, row, c)), f);
+  else vstore8(h, f);
+}
+
+// ROWS rows of one head, rotated, times scale(t), as hi (and lo) tiles `width` (64 or 128) columns wide; zero past `n` rows
+// and dkp channels.
+template <int ROWS, bool LO, typename F>
+__device__ __forceinline__ void ret_load_rotated(uint8_t* hi, uint8_t* lo, int width, const bf16_t* src, size_t row0, int n,
                                                  const RetParams& p, F scale) {
-  const int half = p.rot / 2, tid = threadIdx.x, nthr = blockDim.x;
-  auto put = [&](int t, int c, const float (&f)[8]) {
-    if (LO) store8_split(hi + t * ld + c, lo + t * ld + c, f);
-    else vstore8(hi + t * ld + c, f);
-  };
+  const int half = p.rot / 2, tid = threadIdx.x;
   if (half % 8 == 0) {
-    const int rv = half / 8, pieces = rv + (DK - p.rot) / 8;   // rotated pairs of 8-channel pieces, then plain pieces
+    const int rv = half / 8, pieces = rv + (width - p.rot) / 8;   // rotated pairs of 8-channel pieces, then plain pieces
 #pragma unroll 2
-    for (int i = tid; i < ROWS * pieces; i += nthr) {
+    for (int i = tid; i < ROWS * pieces; i += RET_THREADS) {
       const int t = i / pieces, c = i % pieces;
       const float f = t < n ? scale(t) : 0.f;
       if (c < rv) {
@@ -66,21 +77,21 @@ __device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld,
           x[e] = (u[e] * cs[e] - w[e] * sn[e]) * f;
           y[e] = (w[e] * cs[e] + u[e] * sn[e]) * f;
         }
-        put(t, c * 8, x);
-        put(t, half + c * 8, y);
+        ret_put<LO>(hi, lo, ROWS * 128, t, c * 8, x);
+        ret_put<LO>(hi, lo, ROWS * 128, t, half + c * 8, y);
       } else {
         const int at = p.rot + (c - rv) * 8;
         float u[8] = {};
         if (t < n && at < p.dkp) vload8(src + (row0 + t) * p.ld_in + at, u);
 #pragma unroll
         for (int e = 0; e < 8; ++e) u[e] *= f;
-        put(t, at, u);
+        ret_put<LO>(hi, lo, ROWS * 128, t, at, u);
       }
     }
     return;
   }
-  for (int i = tid; i < ROWS * (DK / 8); i += nthr) {
-    const int t = i / (DK / 8), c8 = i % (DK / 8) * 8;
+  for (int i = tid; i < ROWS * (width / 8); i += RET_THREADS) {
+    const int t = i / (width / 8), c8 = i % (width / 8) * 8;
     float x[8] = {};
     if (t < n && c8 < p.dkp) {
       const bf16_t* s = src + (row0 + t) * p.ld_in;
@@ -96,64 +107,129 @@ __device__ __forceinline__ void ret_load_rotated(bf16_t* hi, bf16_t* lo, int ld,
         x[e] *= fs;
       }
     }
-    put(t, c8, x);
+    ret_put<LO>(hi, lo, ROWS * 128, t, c8, x);
   }
 }
 
-template <int DV>
-__device__ __forceinline__ void ret_load_v(bf16_t* dst, const bf16_t* src, size_t row0, int n, const RetParams& p) {
-  constexpr int LDV = DV + 8;
+__device__ __forceinline__ void ret_load_v(uint8_t* tile, int width, const bf16_t* src, size_t row0, int n, const RetParams& p) {
+  const int pieces = width / 8;
 #pragma unroll 4
-  for (int i = threadIdx.x; i < RET_C * (DV / 8); i += blockDim.x) {
-    const int t = i / (DV / 8), c = i % (DV / 8) * 8;
+  for (int i = threadIdx.x; i < RET_C * pieces; i += RET_THREADS) {
+    const int t = i / pieces, c = i % pieces * 8;
     uint4 u = make_uint4(0, 0, 0, 0);
     if (t < n && c < p.dvp) u = *reinterpret_cast<const uint4*>(src + (row0 + t) * p.ld_in + c);
-    *reinterpret_cast<uint4*>(dst + t * LDV + c) = u;
+    *reinterpret_cast<uint4*>(ret_at(tile, RET_C * 128, t, c)) = u;
   }
 }
 
-template <int DK, int DV>
-__global__ void __launch_bounds__(RET_THREADS, 2) ret_contrib_kernel(const RetParams p) {
-  constexpr int LDK = DK + 8, LDV = DV + 8;
-  constexpr int NT = DV / 8 / (DK == 128 ? 1 : 2);   // n8 tiles per warp
-  extern __shared__ __align__(16) uint8_t sm_raw[];
-  bf16_t* sKh = reinterpret_cast<bf16_t*>(sm_raw);
-  bf16_t* sKl = sKh + RET_C * LDK;
-  bf16_t* sV = sKl + RET_C * LDK;
+constexpr int RET_TILE = RET_C * 128 * 2;        // a full [128 x 128] bf16 tile: 32 KiB
+constexpr int RET_HALF = RET_C * 128;
+constexpr int RET_CONTRIB_BYTES = 3 * RET_TILE + 64 + 1024;
+constexpr int RET_OUT_BYTES = 3 * RET_TILE + 64 + 1024 + 1024;
+
+__device__ __forceinline__ uint8_t* ret_align(uint8_t* p) {
+  return reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(p) + 1023) & ~static_cast<uintptr_t>(1023));
+}
+
+// The CTA's barrier and TMEM.  A wait that runs out sets the status word and lets everyone run on to the end (later waits
+// return at once), so TMEM is always freed.
+struct RetMma {
+  uint64_t* bar;
+  uint32_t* slot;
+  int* status;
+  uint32_t phase = 0, tmem = 0;
+  __device__ __forceinline__ void setup(uint8_t* at, int* st, uint32_t cols) {
+    bar = reinterpret_cast<uint64_t*>(at);
+    slot = reinterpret_cast<uint32_t*>(at + 16);
+    status = st;
+    if (threadIdx.x == 0) {
+      mbar_init(bar, 1);
+      mbar_fence_init();
+    }
+    if (threadIdx.x < 32) {
+      tmem_alloc(slot, cols);
+      tmem_relinquish();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    tmem = *reinterpret_cast<volatile uint32_t*>(slot);
+  }
+  // operand tiles have been written by all threads: make them visible to the tensor core, then let warp 0 issue
+  __device__ __forceinline__ void publish() {
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+  }
+  __device__ __forceinline__ void wait() {
+    mbar_wait_warp(bar, phase, status, ERR_ATTN_WAIT);
+    phase ^= 1;
+    tc_fence_after();
+  }
+  __device__ __forceinline__ void release(uint32_t cols) {
+    tc_fence_before();
+    __syncthreads();
+    if (threadIdx.x < 32) {
+      tc_fence_after();
+      tmem_dealloc(tmem, cols);
+    }
+  }
+};
+
+__global__ void __launch_bounds__(RET_THREADS, 2) ret_contrib_kernel(const RetParams p, int* status) {
+  extern __shared__ uint8_t sm_raw[];
+  uint8_t* sm = ret_align(sm_raw);
+  uint8_t *sKh = sm, *sKl = sm + RET_TILE, *sV = sm + 2 * RET_TILE;
+  RetMma mma;
+  mma.setup(sm + 3 * RET_TILE, status, 128);
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, n = ch[2];
   const size_t row0 = ch[1];
   const float l2a = log2f(p.decay[h]);
-  ret_load_rotated<DK, RET_C, true>(sKh, sKl, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p,
-                             [&](int t) { return p.kscale * ret_pow(l2a, n - 1 - t); });
-  ret_load_v<DV>(sV, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
-  __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
-  const int mt = DK == 128 ? warp : (warp & 3), nb = DK == 128 ? 0 : (warp >> 2) * NT;
-  float acc[NT][4] = {};
-  for (int k0 = 0; k0 < n; k0 += 16) {
-    uint32_t ah[4], al[4];
-    ldsm_a_km(sKh + k0 * LDK + mt * 16, LDK, lane, ah);
-    ldsm_a_km(sKl + k0 * LDK + mt * 16, LDK, lane, al);
+  const int wk = p.dkp > 64 ? 128 : 64, wv = p.dvp > 64 ? 128 : 64;
+  ret_load_rotated<RET_C, true>(sKh, sKl, wk, p.k + static_cast<size_t>(h) * p.dkp, row0, n, p,
+                                [&](int t) { return p.kscale * ret_pow(l2a, n - 1 - t); });
+  ret_load_v(sV, wv, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
+  mma.publish();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp == 0) {
+    // D[key channel, value channel]: both operands have the contraction (tokens) along the rows.  With 64 key channels the
+    // accumulator's upper rows come from whatever follows the tile; they are not stored.
+    const bool leader = elect_one();
+    const uint32_t idesc = make_idesc_f16(1, 128, wv, 1, 1);
+    const uint64_t dh = make_smem_desc_sw128(smem_u32(sKh), RET_HALF, 1024), dl = make_smem_desc_sw128(smem_u32(sKl), RET_HALF, 1024),
+                   dv = make_smem_desc_sw128(smem_u32(sV), RET_HALF, 1024);
+    if (leader) {
 #pragma unroll
-    for (int j = 0; j < NT; j += 2) {
-      uint32_t b[4];
-      ldsm_b_kn(sV + k0 * LDV + (nb + j) * 8, LDV, lane, b);
-      mma_n16(acc[j], acc[j + 1], ah, b);
-      mma_n16(acc[j], acc[j + 1], al, b);
+      for (int ks = 0; ks < RET_C / 16; ++ks) {
+        umma_f16_ss(mma.tmem, desc_advance(dh, ks * 2048), desc_advance(dv, ks * 2048), idesc, ks != 0);
+        umma_f16_ss(mma.tmem, desc_advance(dl, ks * 2048), desc_advance(dv, ks * 2048), idesc, 1);
+      }
+      umma_commit(mma.bar);
     }
+    __syncwarp();
   }
+  mma.wait();
+  const int quarter = warp & 3, half = warp >> 2, i0 = quarter * 32;
   float* w = p.ws + (static_cast<size_t>(blockIdx.x) * p.H + h) * p.dkp * p.dvp;
+  uint8_t* stage = sm + warp * 4096;              // the operands have been read
 #pragma unroll
-  for (int j = 0; j < NT; ++j) {
-    const int c = (nb + j) * 8 + 2 * q;
+  for (int c32 = 0; c32 < 2; ++c32) {
+    const int c0 = half * 64 + c32 * 32;
+    if (c0 >= wv) break;
+    uint32_t t[32];
+    tmem_ld_32x32b_x32(mma.tmem + (static_cast<uint32_t>(i0) << 16) + c0, t);
+    tmem_ld_wait();
+    uint4 v[8];
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int i = mt * 16 + g + 8 * r;
-      if (i < p.dkp && c < p.dvp)
-        *reinterpret_cast<float2*>(w + static_cast<size_t>(i) * p.dvp + c) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
-    }
+    for (int j = 0; j < 8; ++j) v[j] = make_uint4(t[4 * j], t[4 * j + 1], t[4 * j + 2], t[4 * j + 3]);
+    warp_store_rows_128B(stage, v, [&](int row) -> uint8_t* {
+      if (i0 + row >= p.dkp || c0 + (lane & 7) * 4 >= p.dvp) return nullptr;
+      return reinterpret_cast<uint8_t*>(w + static_cast<size_t>(i0 + row) * p.dvp + c0);
+    });
   }
+  mma.release(128);
 }
 
 // ws[c] <- state at the start of chunk c; the final state goes to the slot.  Grid (pieces of the state, H, long sequences).
@@ -190,156 +266,206 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
   *reinterpret_cast<float4*>(st) = S;
 }
 
-// Eight warps, 16 tokens each.  The state and the keys pass through one buffer in pieces of 64 rows, so that two CTAs fit on
-// an SM and one's loads run under the other's products.  Products with q take q's hi part only (q enters no recurrence).
+// TMEM: columns 0..127 hold the weights' fp32 scores and then, as bf16 pairs, their hi (64) and lo (64) parts; 128..255 hold o.
+// The state and the keys pass through one 32 KiB buffer in pieces of 64 rows, so that two CTAs fit on an SM and one's loads
+// run under the other's products.
 constexpr int RET_PIECE = 64;
 
-template <int DK, int DV>
-__host__ __device__ constexpr int ret_piece_elems() {
-  return 2 * RET_PIECE * (DK > DV ? DK + 8 : DV + 8);
-}
-
-template <int DK, int DV>
-__global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams p) {
-  constexpr int LDK = DK + 8, LDV = DV + 8, NT = DV / 8, KS = DK / 16;
-  extern __shared__ __align__(16) uint8_t sm_raw[];
-  bf16_t* sQ = reinterpret_cast<bf16_t*>(sm_raw);
-  bf16_t* sV = sQ + RET_C * LDK;
-  bf16_t* hi = sV + RET_C * LDV;
+__global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams p, int* status) {
+  extern __shared__ uint8_t sm_raw[];
+  uint8_t* sm = ret_align(sm_raw);
+  uint8_t *sQ = sm, *sV = sm + RET_TILE, *hi = sm + 2 * RET_TILE, *lo = hi + RET_TILE / 2;
+  float* xchg = reinterpret_cast<float*>(sm + 3 * RET_TILE + 64);     // [2 column halves][128 rows]
+  RetMma mma;
+  mma.setup(sm + 3 * RET_TILE, status, 256);
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, s = ch[0], n = ch[2];
   const size_t row0 = ch[1];
   const bool zero = ch[3] == 0 && p.start[s] == 0;       // nothing before this chunk
   const float l2a = log2f(p.decay[h]);
-  const int rt = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
-  const bool active = rt * 16 < n;
-  ret_load_rotated<DK, RET_C, false>(sQ, nullptr, LDK, p.q + static_cast<size_t>(h) * p.dkp, row0, n, p, [](int) { return 1.f; });
-  ret_load_v<DV>(sV, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
-  float acc[NT][4] = {};
+  const int wk = p.dkp > 64 ? 128 : 64, wv = p.dvp > 64 ? 128 : 64;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quarter = warp & 3, half = warp >> 2;
+  const int r = quarter * 32 + lane;                     // token of this thread, shared with the warp four further on
+  const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
+  const uint32_t tS = mma.tmem, tO = mma.tmem + 128;
+  const bool mine = half * 64 < wv;                      // this thread has columns of o
+  ret_load_rotated<RET_C, false>(sQ, nullptr, wk, p.q + static_cast<size_t>(h) * p.dkp, row0, n, p, [](int) { return 1.f; });
+  ret_load_v(sV, wv, p.v + static_cast<size_t>(h) * p.dvp, row0, n, p);
+  const bool leader = warp == 0 && elect_one();
+  const uint64_t dq = make_smem_desc_sw128(smem_u32(sQ), 16, 1024);
+  const uint32_t idesc_o = make_idesc_f16(1, 128, wv, 0, 1);
+
   if (!zero) {
-    bf16_t* lo = hi + RET_PIECE * LDV;
     const float* w = p.ws + (static_cast<size_t>(blockIdx.x) * p.H + h) * p.dkp * p.dvp;
-    for (int r0 = 0; r0 < DK; r0 += RET_PIECE) {
-      if (r0 > 0) __syncthreads();
+    const int pieces = wv / 8;
+    for (int r0 = 0; r0 < wk; r0 += RET_PIECE) {
+      if (r0 > 0) mma.wait();
 #pragma unroll 4
-      for (int i = threadIdx.x; i < RET_PIECE * (DV / 8); i += RET_THREADS) {
-        const int r = i / (DV / 8), c = i % (DV / 8) * 8;
+      for (int i = threadIdx.x; i < RET_PIECE * pieces; i += RET_THREADS) {
+        const int t = i / pieces, c = i % pieces * 8;
         float x[8] = {};
-        if (r0 + r < p.dkp && c < p.dvp) vload8(w + static_cast<size_t>(r0 + r) * p.dvp + c, x);
-        store8_split(hi + r * LDV + c, lo + r * LDV + c, x);
+        if (r0 + t < p.dkp && c < p.dvp) vload8(w + static_cast<size_t>(r0 + t) * p.dvp + c, x);
+        ret_put<true>(hi, lo, RET_PIECE * 128, t, c, x);
       }
-      __syncthreads();
-      if (active)
+      mma.publish();
+      if (leader) {
+        const uint64_t dh = make_smem_desc_sw128(smem_u32(hi), RET_PIECE * 128, 1024),
+                       dl = make_smem_desc_sw128(smem_u32(lo), RET_PIECE * 128, 1024);
 #pragma unroll
         for (int ks = 0; ks < RET_PIECE / 16; ++ks) {
-          uint32_t a[4];
-          ldsm_a_mk(sQ + rt * 16 * LDK + r0 + ks * 16, LDK, lane, a);
-#pragma unroll
-          for (int j = 0; j < NT; j += 2) {
-            uint32_t b[4];
-            ldsm_b_kn(hi + ks * 16 * LDV + j * 8, LDV, lane, b);
-            mma_n16(acc[j], acc[j + 1], a, b);
-            ldsm_b_kn(lo + ks * 16 * LDV + j * 8, LDV, lane, b);
-            mma_n16(acc[j], acc[j + 1], a, b);
-          }
+          const uint64_t a = desc_advance(dq, (r0 >> 6) * RET_HALF + ks * 32);
+          umma_f16_ss(tO, a, desc_advance(dh, ks * 2048), idesc_o, r0 > 0 || ks > 0);
+          umma_f16_ss(tO, a, desc_advance(dl, ks * 2048), idesc_o, 1);
         }
+        umma_commit(mma.bar);
+      }
+      __syncwarp();
     }
-    const float f0 = ret_pow(l2a, rt * 16 + g + 1), f1 = ret_pow(l2a, rt * 16 + g + 9);
+    mma.wait();
+    if (mine) {                                          // o = a^{t+1} (q S)
+      const float f = ret_pow(l2a, r + 1);
 #pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      acc[j][0] *= f0;
-      acc[j][1] *= f0;
-      acc[j][2] *= f1;
-      acc[j][3] *= f1;
+      for (int c = 0; c < 4; ++c) {
+        uint32_t t[16];
+        tmem_ld_32x32b_x16(tO + lane_off + half * 64 + c * 16, t);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) t[i] = __float_as_uint(__uint_as_float(t[i]) * f);
+        tmem_st_32x32b_x16(tO + lane_off + half * 64 + c * 16, t);
+      }
+      tmem_st_wait();
     }
-    __syncthreads();
   }
-  bf16_t* lo = hi + RET_PIECE * LDK;
   for (int k0 = 0; k0 < n; k0 += RET_PIECE) {
-    if (k0 > 0) __syncthreads();
-    ret_load_rotated<DK, RET_PIECE, true>(hi, lo, LDK, p.k + static_cast<size_t>(h) * p.dkp, row0 + k0, n - k0, p,
-                                          [&](int) { return p.kscale; });
-    __syncthreads();
-    for (int kb = 0; active && kb < RET_PIECE / 16 && k0 / 16 + kb <= rt; ++kb) {     // 16 keys at a time, up to the diagonal
-      float sc[2][4] = {};
-#pragma unroll
-      for (int ks = 0; ks < KS; ++ks) {
-        uint32_t a[4], b[4];
-        ldsm_a_mk(sQ + rt * 16 * LDK + ks * 16, LDK, lane, a);
-        ldsm_b_nk(hi + kb * 16 * LDK + ks * 16, LDK, lane, b);
-        mma_n16(sc[0], sc[1], a, b);
-        ldsm_b_nk(lo + kb * 16 * LDK + ks * 16, LDK, lane, b);
-        mma_n16(sc[0], sc[1], a, b);
+    ret_load_rotated<RET_PIECE, true>(hi, lo, wk, p.k + static_cast<size_t>(h) * p.dkp, row0 + k0, n - k0, p,
+                                      [&](int) { return p.kscale; });
+    mma.publish();
+    if (leader) {
+      const uint32_t idesc = make_idesc_f16(1, 128, RET_PIECE, 0, 0);
+      const uint64_t dh = make_smem_desc_sw128(smem_u32(hi), 16, 1024), dl = make_smem_desc_sw128(smem_u32(lo), 16, 1024);
+      for (int ks = 0; ks < wk / 16; ++ks) {
+        const uint64_t a = desc_advance(dq, (ks >> 2) * RET_HALF + (ks & 3) * 32);
+        const uint32_t b = (ks >> 2) * (RET_PIECE * 128) + (ks & 3) * 32;
+        umma_f16_ss(tS + k0, a, desc_advance(dh, b), idesc, ks != 0);
+        umma_f16_ss(tS + k0, a, desc_advance(dl, b), idesc, 1);
       }
-      uint32_t ph[4], pl[4];
+      umma_commit(mma.bar);
+    }
+    __syncwarp();
+    mma.wait();
+  }
+  {
+    // weights of this thread's 64 keys: decayed, causal, split
+    uint32_t ph[32], pl[32];
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
+    for (int c = 0; c < 2; ++c) {
+      uint32_t t[32];
+      tmem_ld_32x32b_x32(tS + lane_off + half * 64 + c * 32, t);
+      tmem_ld_wait();
+      const int d0 = r - (half * 64 + c * 32);           // distance to the first of these keys
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int d = rt * 16 + g + 8 * r - (k0 + kb * 16 + j * 8 + 2 * q);     // distance to the first of the two keys
-          const float x0 = d >= 0 ? sc[j][2 * r] * ret_pow(l2a, d) : 0.f;
-          const float x1 = d >= 1 ? sc[j][2 * r + 1] * ret_pow(l2a, d - 1) : 0.f;
-          split_pair(x0, x1, ph[2 * j + r], pl[2 * j + r]);
-        }
+      for (int i = 0; i < 16; ++i) {
+        const int d = d0 - 2 * i;
+        // a key past the chunk's end has a distance below zero for every token of the chunk
+        const float x0 = d >= 0 ? __uint_as_float(t[2 * i]) * ret_pow(l2a, d) : 0.f;
+        const float x1 = d >= 1 ? __uint_as_float(t[2 * i + 1]) * ret_pow(l2a, d - 1) : 0.f;
+        split_pair(x0, x1, ph[c * 16 + i], pl[c * 16 + i]);
+      }
+    }
+    tc_fence_before();
+    __syncthreads();                                     // everyone has read its scores
+    tc_fence_after();
 #pragma unroll
-      for (int j = 0; j < NT; j += 2) {
-        uint32_t b[4];
-        ldsm_b_kn(sV + (k0 + kb * 16) * LDV + j * 8, LDV, lane, b);
-        mma_n16(acc[j], acc[j + 1], ph, b);
-        mma_n16(acc[j], acc[j + 1], pl, b);
+    for (int c = 0; c < 2; ++c) {
+      uint32_t a[16], b[16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        a[i] = r < n ? ph[c * 16 + i] : 0u;
+        b[i] = r < n ? pl[c * 16 + i] : 0u;
+      }
+      tmem_st_32x32b_x16(tS + lane_off + half * 32 + c * 16, a);
+      tmem_st_32x32b_x16(tS + lane_off + 64 + half * 32 + c * 16, b);
+    }
+    tmem_st_wait();
+  }
+  mma.publish();
+  if (leader) {
+    const uint64_t dv = make_smem_desc_sw128(smem_u32(sV), RET_HALF, 1024);
+#pragma unroll
+    for (int ks = 0; ks < RET_C / 16; ++ks)
+      umma_f16_ts(tO, tS + ks * 8, desc_advance(dv, ks * 2048), idesc_o, (zero && ks == 0) ? 0u : 1u);
+#pragma unroll
+    for (int ks = 0; ks < RET_C / 16; ++ks) umma_f16_ts(tO, tS + 64 + ks * 8, desc_advance(dv, ks * 2048), idesc_o, 1);
+    umma_commit(mma.bar);
+  }
+  __syncwarp();
+  // the gate, while the tensor core works
+  float o[64];
+  uint4 gv[8];
+  const bool live = mine && r < n;
+  const bf16_t* gp = p.gate + (row0 + r) * p.ld_in + static_cast<size_t>(h) * p.dvp + half * 64;
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+    gv[j] = live && half * 64 + j * 8 < p.dvp ? *reinterpret_cast<const uint4*>(gp + j * 8) : make_uint4(0, 0, 0, 0);
+  mma.wait();
+  float ss = 0.f;
+  if (mine) {
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+      uint32_t t[32];
+      tmem_ld_32x32b_x32(tO + lane_off + half * 64 + c * 32, t);
+      tmem_ld_wait();
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        o[c * 32 + i] = __uint_as_float(t[i]);
+        ss = fmaf(o[c * 32 + i], o[c * 32 + i], ss);
       }
     }
   }
-  if (!active) return;
-  float s0 = 0.f, s1 = 0.f;
+  xchg[half * 128 + r] = ss;
+  __syncthreads();
+  if (mine) {
+    const float f = 1.f / sqrtf((xchg[r] + xchg[128 + r]) / p.dv + p.eps);
+    uint4 ov[8];
 #pragma unroll
-  for (int j = 0; j < NT; ++j) {
-    s0 += acc[j][0] * acc[j][0] + acc[j][1] * acc[j][1];
-    s1 += acc[j][2] * acc[j][2] + acc[j][3] * acc[j][3];
-  }
+    for (int j = 0; j < 8; ++j) {
+      const uint32_t g[4] = {gv[j].x, gv[j].y, gv[j].z, gv[j].w};
+      uint32_t y[4];
 #pragma unroll
-  for (int o = 1; o < 4; o <<= 1) {
-    s0 += __shfl_xor_sync(0xffffffffu, s0, o);
-    s1 += __shfl_xor_sync(0xffffffffu, s1, o);
-  }
-  const float r0 = 1.f / sqrtf(s0 / p.dv + p.eps), r1 = 1.f / sqrtf(s1 / p.dv + p.eps);
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    const int t = rt * 16 + g + 8 * r;
-    if (t >= n) continue;
-    const bf16_t* gp = p.gate + (row0 + t) * p.ld_in + static_cast<size_t>(h) * p.dvp;
-    bf16_t* op = p.out + (row0 + t) * p.ld_out + static_cast<size_t>(h) * p.dvp;
-#pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      const int c = j * 8 + 2 * q;
-      if (c >= p.dvp) break;
-      const float2 gv = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(gp + c));
-      const float f = r ? r1 : r0;
-      *reinterpret_cast<uint32_t*>(op + c) = pack_bf16x2(acc[j][2 * r] * f * silu_fast(gv.x), acc[j][2 * r + 1] * f * silu_fast(gv.y));
+      for (int e = 0; e < 4; ++e) {
+        const float2 g2 = unpack_bf16x2(g[e]);
+        y[e] = pack_bf16x2(o[j * 8 + 2 * e] * f * silu_fast(g2.x), o[j * 8 + 2 * e + 1] * f * silu_fast(g2.y));
+      }
+      ov[j] = make_uint4(y[0], y[1], y[2], y[3]);
     }
+    bf16_t* base = p.out + (row0 + quarter * 32) * p.ld_out + static_cast<size_t>(h) * p.dvp + half * 64;
+    warp_store_rows_128B(hi + warp * 4096, ov, [&](int row) -> uint8_t* {
+      if (quarter * 32 + row >= n || half * 64 + (lane & 7) * 8 >= p.dvp) return nullptr;
+      return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * p.ld_out);
+    });
   }
+  mma.release(256);
 }
 
-template <int DK, int DV>
 static int launch_ret(const RetParams& p, int nchunks, int nlong, cudaStream_t stream) {
-  const int sm1 = RET_C * (2 * (DK + 8) + DV + 8) * 2;
-  const int sm3 = (RET_C * (DK + 8 + DV + 8) + ret_piece_elems<DK, DV>()) * 2;
+  int* status = status_ptr();
+  if (!status) return 3;
   static bool set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!set[dev & 63]) {
-    if (cudaFuncSetAttribute(ret_contrib_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||
-        cudaFuncSetAttribute(ret_out_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) {
+    if (cudaFuncSetAttribute(ret_contrib_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, RET_CONTRIB_BYTES) != cudaSuccess ||
+        cudaFuncSetAttribute(ret_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, RET_OUT_BYTES) != cudaSuccess) {
       set_error("retention_chunk: cannot set shared memory size");
       return 1;
     }
     set[dev & 63] = true;
   }
-  ret_contrib_kernel<DK, DV><<<dim3(nchunks, p.H), RET_THREADS, sm1, stream>>>(p);
+  ret_contrib_kernel<<<dim3(nchunks, p.H), RET_THREADS, RET_CONTRIB_BYTES, stream>>>(p, status);
   B2_CHECK_LAUNCH("ret_contrib");
   ret_scan_kernel<<<dim3((p.dkp * p.dvp / 4 + 255) / 256, p.H, nlong), 256, 0, stream>>>(p);
   B2_CHECK_LAUNCH("ret_scan");
-  ret_out_kernel<DK, DV><<<dim3(nchunks, p.H), RET_THREADS, sm3, stream>>>(p);
+  ret_out_kernel<<<dim3(nchunks, p.H), RET_THREADS, RET_OUT_BYTES, stream>>>(p, status);
   B2_CHECK_LAUNCH("ret_out");
   return 0;
 }
@@ -367,6 +493,5 @@ B2_EXPORT int b2_retention_chunk(const void* q, const void* k, const void* v, co
   p.cs = cs; p.sn = sn; p.chunks = chunks; p.first = first; p.start = start; p.slot = slot; p.ld_in = ld_in; p.ld_out = ld_out;
   p.H = H; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.rot = rot; p.seq0 = seq0; p.kscale = kscale; p.eps = eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dkp <= 64) return dvp <= 64 ? launch_ret<64, 64>(p, nchunks, nlong, st) : launch_ret<64, 128>(p, nchunks, nlong, st);
-  return dvp <= 64 ? launch_ret<128, 64>(p, nchunks, nlong, st) : launch_ret<128, 128>(p, nchunks, nlong, st);
+  return launch_ret(p, nchunks, nlong, st);
 }
