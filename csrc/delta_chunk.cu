@@ -83,26 +83,38 @@ __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const Delt
 #pragma unroll
     for (int i = 0; i < SEG; ++i) {
       const int t = seg * SEG + i;
-      x[i] = t < n && c < p.dkp ? p.glog[((row0 + t) * p.H + h) * p.dkp + c] * 1.4426950408889634f : 0.f;
+      // loads are unconditional, clamped to rows and channels that exist, so that they are all in flight together
+      x[i] = p.glog[((row0 + min(t, n - 1)) * p.H + h) * p.dkp + min(c, p.dkp - 1)];
     }
-#pragma unroll 4
-    for (int i = tid; i < DEL_C * (DK / 4); i += FAC_THREADS) {
-      const int t = i / (DK / 4), cc = i % (DK / 4) * 4;
-      float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
-      if (t < n && cc < p.dkp) {
-        const size_t at = ((row0 + t) * p.G + kvh) * p.dkp + cc;
-        kv = *reinterpret_cast<const float4*>(p.k + at);
-        qv = *reinterpret_cast<const float4*>(p.q + at);
-      }
-      *reinterpret_cast<float4*>(sK + t * LD + cc) = kv;
-      *reinterpret_cast<float4*>(sQ + t * LD + cc) = qv;
+    constexpr int NK = DEL_C * (DK / 4) / FAC_THREADS, NV = DEL_C * 16 / FAC_THREADS;
+    float4 kv[NK], qv[NK];
+    uint4 vv[NV];
+#pragma unroll
+    for (int j = 0; j < NK; ++j) {
+      const int i = tid + j * FAC_THREADS, t = min(i / (DK / 4), n - 1), cc = min(i % (DK / 4) * 4, p.dkp - 4);
+      const size_t at = ((row0 + t) * p.G + kvh) * p.dkp + cc;
+      kv[j] = *reinterpret_cast<const float4*>(p.k + at);
+      qv[j] = *reinterpret_cast<const float4*>(p.q + at);
     }
-#pragma unroll 2
-    for (int i = tid; i < DEL_C * (128 / 8); i += FAC_THREADS) {
-      const int t = i / 16, cc = i % 16 * 8;
-      uint4 u = make_uint4(0, 0, 0, 0);
-      if (t < n && cc < p.dvp) u = *reinterpret_cast<const uint4*>(p.v + ((row0 + t) * p.H + h) * p.dvp + cc);
-      *reinterpret_cast<uint4*>(sV + t * LDV + cc) = u;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int i = tid + j * FAC_THREADS, t = min(i / 16, n - 1), cc = min(i % 16 * 8, p.dvp - 8);
+      vv[j] = *reinterpret_cast<const uint4*>(p.v + ((row0 + t) * p.H + h) * p.dvp + cc);
+    }
+#pragma unroll
+    for (int i = 0; i < SEG; ++i) x[i] = seg * SEG + i < n && c < p.dkp ? x[i] * 1.4426950408889634f : 0.f;
+#pragma unroll
+    for (int j = 0; j < NK; ++j) {
+      const int i = tid + j * FAC_THREADS, t = i / (DK / 4), cc = i % (DK / 4) * 4;
+      const bool in = t < n && cc < p.dkp;
+      const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+      *reinterpret_cast<float4*>(sK + t * LD + cc) = in ? kv[j] : z;
+      *reinterpret_cast<float4*>(sQ + t * LD + cc) = in ? qv[j] : z;
+    }
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int i = tid + j * FAC_THREADS, t = i / 16, cc = i % 16 * 8;
+      *reinterpret_cast<uint4*>(sV + t * LDV + cc) = t < n && cc < p.dvp ? vv[j] : make_uint4(0, 0, 0, 0);
     }
     if (tid < DEL_C) sB[tid] = tid < n ? p.beta[(row0 + tid) * p.H + h] : 0.f;
     for (int i = tid; i < DEL_C * DEL_LDA / 4; i += FAC_THREADS) {

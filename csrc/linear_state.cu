@@ -467,10 +467,20 @@ __device__ __forceinline__ void prep_conv_job(const DeltaPrepParams& p, int s, i
 #pragma unroll
     for (int i = 0; i < K - 1; ++i) vload8(x + (static_cast<size_t>(row0) - 1 - i) * p.ld, w[i]);   // off >= a tile > K - 1
   }
+  constexpr int AHEAD = 4;            // rows requested together
+  float buf[AHEAD][8];
   for (int t = 0; t < rows; ++t) {
     const size_t row = static_cast<size_t>(row0) + t;
+    if (t % AHEAD == 0) {
+#pragma unroll
+      for (int i = 0; i < AHEAD; ++i) vload8(x + (static_cast<size_t>(row0) + min(t + i, rows - 1)) * p.ld, buf[i]);
+    }
     float cur[8], y[8], ss = 0.f;
-    vload8(x + row * p.ld, cur);
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      if (t % AHEAD == i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) cur[e] = buf[i][e];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       float a = cur[e] * taps[e * K + K - 1];
@@ -552,13 +562,18 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_vec_kernel(const Delt
   float dt[8];
   vload8(static_cast<const T*>(p.dt_bias) + c, dt);
   const float A = -expf(to_f(static_cast<const T*>(p.A_log)[c / p.dkp]));
-  for (int t = 0; t < rows; ++t) {
-    const size_t row = static_cast<size_t>(row0) + t;
-    float z[8];
-    vload8(p.a2 + row * p.ld_a2 + c, z);
+  constexpr int AHEAD = 4;
+  for (int t0 = 0; t0 < rows; t0 += AHEAD) {
+    float z[AHEAD][8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) z[e] = A * softplus_f(z[e] + dt[e]);
-    vstore8(p.glog + row * width + c, z);
+    for (int i = 0; i < AHEAD; ++i) vload8(p.a2 + (static_cast<size_t>(row0) + min(t0 + i, rows - 1)) * p.ld_a2 + c, z[i]);
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      if (t0 + i >= rows) break;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) z[i][e] = A * softplus_f(z[i][e] + dt[e]);
+      vstore8(p.glog + (static_cast<size_t>(row0) + t0 + i) * width + c, z[i]);
+    }
   }
 }
 

@@ -58,34 +58,53 @@ __device__ __forceinline__ void ret_load_rotated(uint8_t* hi, uint8_t* lo, int w
                                                  const RetParams& p, F scale) {
   const int half = p.rot / 2, tid = threadIdx.x;
   if (half % 8 == 0) {
-    const int rv = half / 8, pieces = rv + (width - p.rot) / 8;   // rotated pairs of 8-channel pieces, then plain pieces
-#pragma unroll 2
-    for (int i = tid; i < ROWS * pieces; i += RET_THREADS) {
-      const int t = i / pieces, c = i % pieces;
-      const float f = t < n ? scale(t) : 0.f;
-      if (c < rv) {
-        float u[8] = {}, w[8] = {}, cs[8] = {}, sn[8] = {}, x[8], y[8];
-        if (t < n) {
-          const bf16_t* s = src + (row0 + t) * p.ld_in + c * 8;
-          vload8(s, u);
-          vload8(s + half, w);
-          vload8(p.cs + (row0 + t) * half + c * 8, cs);
-          vload8(p.sn + (row0 + t) * half + c * 8, sn);
-        }
+    // Rotated pairs of 8-channel pieces, then plain pieces.  Two items at a time, their loads unconditional (clamped to rows
+    // and channels that exist, the result dropped), so that all of them are in flight together.
+    const int rv = half / 8, pieces = rv + (width - p.rot) / 8, total = ROWS * pieces;
+    for (int i0 = tid; i0 < total; i0 += 2 * RET_THREADS) {
+      uint4 u4[2], w4[2];
+      float4 c4[2][2], s4[2][2];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          x[e] = (u[e] * cs[e] - w[e] * sn[e]) * f;
-          y[e] = (w[e] * cs[e] + u[e] * sn[e]) * f;
+      for (int k = 0; k < 2; ++k) {
+        const int i = min(i0 + k * RET_THREADS, total - 1), t = min(i / pieces, n - 1), c = i % pieces;
+        const int at = c < rv ? c * 8 : min(p.rot + (c - rv) * 8, p.dkp - 8);
+        const bf16_t* s = src + (row0 + t) * p.ld_in + at;
+        u4[k] = *reinterpret_cast<const uint4*>(s);
+        w4[k] = *reinterpret_cast<const uint4*>(c < rv ? s + half : s);
+        if (rv > 0) {
+          const size_t f = (row0 + t) * half + (c < rv ? c * 8 : 0);
+          c4[k][0] = *reinterpret_cast<const float4*>(p.cs + f);
+          c4[k][1] = *reinterpret_cast<const float4*>(p.cs + f + 4);
+          s4[k][0] = *reinterpret_cast<const float4*>(p.sn + f);
+          s4[k][1] = *reinterpret_cast<const float4*>(p.sn + f + 4);
         }
-        ret_put<LO>(hi, lo, ROWS * 128, t, c * 8, x);
-        ret_put<LO>(hi, lo, ROWS * 128, t, half + c * 8, y);
-      } else {
-        const int at = p.rot + (c - rv) * 8;
-        float u[8] = {};
-        if (t < n && at < p.dkp) vload8(src + (row0 + t) * p.ld_in + at, u);
+      }
 #pragma unroll
-        for (int e = 0; e < 8; ++e) u[e] *= f;
-        ret_put<LO>(hi, lo, ROWS * 128, t, at, u);
+      for (int k = 0; k < 2; ++k) {
+        const int i = i0 + k * RET_THREADS, t = i / pieces, c = i % pieces;
+        if (i >= total) break;
+        float u[8], x[8], y[8];
+        unpack8(u4[k], u);
+        if (c < rv) {
+          const float f = t < n ? scale(t) : 0.f;
+          float w[8];
+          unpack8(w4[k], w);
+          const float cs[8] = {c4[k][0].x, c4[k][0].y, c4[k][0].z, c4[k][0].w, c4[k][1].x, c4[k][1].y, c4[k][1].z, c4[k][1].w};
+          const float sn[8] = {s4[k][0].x, s4[k][0].y, s4[k][0].z, s4[k][0].w, s4[k][1].x, s4[k][1].y, s4[k][1].z, s4[k][1].w};
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            x[e] = (u[e] * cs[e] - w[e] * sn[e]) * f;
+            y[e] = (w[e] * cs[e] + u[e] * sn[e]) * f;
+          }
+          ret_put<LO>(hi, lo, ROWS * 128, t, c * 8, x);
+          ret_put<LO>(hi, lo, ROWS * 128, t, half + c * 8, y);
+        } else {
+          const int at = p.rot + (c - rv) * 8;
+          const float f = t < n && at < p.dkp ? scale(t) : 0.f;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) u[e] = f != 0.f ? u[e] * f : 0.f;
+          ret_put<LO>(hi, lo, ROWS * 128, t, at, u);
+        }
       }
     }
     return;
@@ -112,13 +131,19 @@ __device__ __forceinline__ void ret_load_rotated(uint8_t* hi, uint8_t* lo, int w
 }
 
 __device__ __forceinline__ void ret_load_v(uint8_t* tile, int width, const bf16_t* src, size_t row0, int n, const RetParams& p) {
-  const int pieces = width / 8;
-#pragma unroll 4
-  for (int i = threadIdx.x; i < RET_C * pieces; i += RET_THREADS) {
-    const int t = i / pieces, c = i % pieces * 8;
-    uint4 u = make_uint4(0, 0, 0, 0);
-    if (t < n && c < p.dvp) u = *reinterpret_cast<const uint4*>(src + (row0 + t) * p.ld_in + c);
-    *reinterpret_cast<uint4*>(ret_at(tile, RET_C * 128, t, c)) = u;
+  const int pieces = width / 8;                    // RET_C * pieces is a multiple of 4 * RET_THREADS
+  for (int i0 = threadIdx.x; i0 < RET_C * pieces; i0 += 4 * RET_THREADS) {
+    uint4 u[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = i0 + k * RET_THREADS, t = min(i / pieces, n - 1), c = min(i % pieces * 8, p.dvp - 8);
+      u[k] = *reinterpret_cast<const uint4*>(src + (row0 + t) * p.ld_in + c);
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = i0 + k * RET_THREADS, t = i / pieces, c = i % pieces * 8;
+      *reinterpret_cast<uint4*>(ret_at(tile, RET_C * 128, t, c)) = t < n && c < p.dvp ? u[k] : make_uint4(0, 0, 0, 0);
+    }
   }
 }
 
@@ -249,8 +274,7 @@ __global__ void __launch_bounds__(256) ret_scan_kernel(const RetParams p) {
   for (int c = c0; c < c1; c += U) {
     float4 kv[U];
 #pragma unroll
-    for (int u = 0; u < U; ++u)
-      if (c + u < c1) kv[u] = *reinterpret_cast<const float4*>(w + u * step);
+    for (int u = 0; u < U; ++u) kv[u] = *reinterpret_cast<const float4*>(w + min(u, c1 - 1 - c) * step);
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       if (c + u >= c1) break;
@@ -300,12 +324,21 @@ __global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams
     const int pieces = wv / 8;
     for (int r0 = 0; r0 < wk; r0 += RET_PIECE) {
       if (r0 > 0) mma.wait();
-#pragma unroll 4
-      for (int i = threadIdx.x; i < RET_PIECE * pieces; i += RET_THREADS) {
-        const int t = i / pieces, c = i % pieces * 8;
-        float x[8] = {};
-        if (r0 + t < p.dkp && c < p.dvp) vload8(w + static_cast<size_t>(r0 + t) * p.dvp + c, x);
-        ret_put<true>(hi, lo, RET_PIECE * 128, t, c, x);
+      for (int i0 = threadIdx.x; i0 < RET_PIECE * pieces; i0 += 2 * RET_THREADS) {   // a multiple of 2 * RET_THREADS
+        float x[2][8];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          const int i = i0 + k * RET_THREADS, t = min(r0 + i / pieces, p.dkp - 1), c = min(i % pieces * 8, p.dvp - 8);
+          vload8(w + static_cast<size_t>(t) * p.dvp + c, x[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          const int i = i0 + k * RET_THREADS, t = i / pieces, c = i % pieces * 8;
+          const bool in = r0 + t < p.dkp && c < p.dvp;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) x[k][e] = in ? x[k][e] : 0.f;
+          ret_put<true>(hi, lo, RET_PIECE * 128, t, c, x[k]);
+        }
       }
       mma.publish();
       if (leader) {

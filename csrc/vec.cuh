@@ -14,8 +14,7 @@ __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return
 template <>
 __device__ __forceinline__ float from_f<float>(float v) { return v; }
 
-__device__ __forceinline__ void vload8(const __nv_bfloat16* p, float (&f)[8]) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
+__device__ __forceinline__ void unpack8(const uint4& u, float (&f)[8]) {
   const uint32_t w[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -23,6 +22,9 @@ __device__ __forceinline__ void vload8(const __nv_bfloat16* p, float (&f)[8]) {
     f[2 * i] = t.x;
     f[2 * i + 1] = t.y;
   }
+}
+__device__ __forceinline__ void vload8(const __nv_bfloat16* p, float (&f)[8]) {
+  unpack8(*reinterpret_cast<const uint4*>(p), f);
 }
 __device__ __forceinline__ void vload8(const float* p, float (&f)[8]) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
