@@ -263,9 +263,9 @@ def test_chunked_attention(run, H, G, dk, dv, chunk):
 
 
 def test_distance_buckets():
-    b = ops.distance_buckets(16, 240, 300).tolist()
-    assert b == [min(O.distance_bucket(n, 16, 240), 15) for n in range(300)]
-    assert b[:8] == list(range(8)) and b[240] == b[299] == 15
+    b = ops.distance_buckets(12, 90, 200).tolist()
+    assert b == [min(O.distance_bucket(n, 12, 90), 11) for n in range(200)]
+    assert b[:6] == list(range(6)) and b[90] == b[199] == 11
     # a distance exactly on an edge belongs to the upper bucket: 4 * (64 / 4)^(1/2) = 16
     assert ops.distance_buckets(8, 64, 17).tolist()[15:] == [5, 6]
 
