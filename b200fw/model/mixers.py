@@ -10,6 +10,7 @@ Head sizes and feature counts are stored padded to multiples of eight with zeros
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Tuple
 
@@ -167,7 +168,7 @@ class BiasedChunkAttention(nn.Module):
         self.rel = _param(bias_rows, heads, dtype=dtype, device=device)
         self.sink = _param(heads, dtype=dtype, device=device)
         # distances past the last entry share its bucket: everything at `bias_far` or beyond is in the last one
-        length = min(self.chunk, max(int(bias_far), bias_rows) + 1)
+        length = min(self.chunk, max(math.ceil(bias_far), bias_rows) + 1)
         self.register_buffer("bucket", ops.distance_buckets(bias_rows, bias_far, length, device), persistent=False)
         self.o = PackedCols(hidden, [("o", heads, vdim)], dtype, device)
 

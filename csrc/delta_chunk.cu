@@ -32,12 +32,9 @@ struct DeltaParams {
   const int* first;      // [nlong + 1]
   const int* start;
   const int* slot;
-  // per chunk and head, bf16 planes hi then lo: W, Ks [2][64][DK], P [2][64][64]; hi only: Qs [64][DK] (q enters no
-  // recurrence); fp32 U0 [64][dvp], end [DK]
-  __nv_bfloat16* W;
-  __nv_bfloat16* Qs;
-  __nv_bfloat16* Ks;
-  __nv_bfloat16* P;
+  // per chunk and head one record of bf16 planes, exactly as the scan keeps them in shared memory (DelRecord); fp32
+  // U0 [64][dvp], end [DK]
+  __nv_bfloat16* rec;
   float* U0;
   float* end;
   float* o;              // [M, H * dvp]
@@ -64,9 +61,19 @@ struct DelFactor {
   static constexpr int BYTES = (B + DEL_C) * 4;
 };
 
+// W and Ks hi then lo [2][64][DK + 8], P [2][64][64 + 8]; Qs hi only (q enters no recurrence).  The scan copies a record in two
+// pieces, W | Qs and Ks | P.
+template <int DK>
+struct DelRecord {
+  static constexpr int LDM = DK + 8, LDP = DEL_C + 8;
+  static constexpr int W = 0, Q = W + 2 * DEL_C * LDM, K = Q + DEL_C * LDM, P = K + 2 * DEL_C * LDM;
+  static constexpr int ELEMS = P + 2 * DEL_C * LDP;
+};
+
 template <int DK>
 __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const DeltaParams p) {
   using L = DelFactor<DK>;
+  using Rec = DelRecord<DK>;
   constexpr int LD = L::LD, LDV = L::LDV, SEGS = FAC_THREADS / DK, SEG = DEL_C / SEGS;
   extern __shared__ __align__(16) float sm[];
   float *sG = sm + L::G, *sE = sm + L::E, *sK = sm + L::K, *sQ = sm + L::Q, *sA = sm + L::A, *sP = sm + L::P, *sT = sm + L::T,
@@ -75,6 +82,7 @@ __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const Delt
   const int* ch = p.chunks + blockIdx.x * 4;
   const int h = blockIdx.y, n = ch[2], kvh = h / (p.H / p.G);
   const size_t row0 = ch[1], item = static_cast<size_t>(blockIdx.x) * p.H + h;
+  __nv_bfloat16* rec = p.rec + item * Rec::ELEMS;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
 
   {
@@ -240,9 +248,8 @@ __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const Delt
       k[e] *= fast_exp2(Ge[e] - G[e]);
     }
     store8_split(pKh + t * LD + c, pKl + t * LD + c, kg);
-    const size_t at = item * DEL_C * DK + t * DK + c;
-    vstore8(p.Qs + at, q);
-    store8_split(p.Ks + at + item * DEL_C * DK, p.Ks + at + (item + 1) * DEL_C * DK, k);
+    vstore8(rec + Rec::Q + t * Rec::LDM + c, q);
+    store8_split(rec + Rec::K + t * Rec::LDM + c, rec + Rec::K + (DEL_C + t) * Rec::LDM + c, k);
     if (t == DEL_C - 1) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) p.end[item * DK + c + e] = fast_exp2(Ge[e]);
@@ -252,8 +259,7 @@ __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const Delt
     const int t = i / 8, c = i % 8 * 8;
     float x[8];
     vload8(sP + t * DEL_LDA + c, x);
-    const size_t at = 2 * item * DEL_C * DEL_C + t * DEL_C + c;
-    store8_split(p.P + at, p.P + at + DEL_C * DEL_C, x);
+    store8_split(rec + Rec::P + t * Rec::LDP + c, rec + Rec::P + (DEL_C + t) * Rec::LDP + c, x);
   }
 
   // T = (I + A)^-1: the diagonal blocks by substitution, then T_IJ = -T_II sum_K A_IK T_KJ block row by block row
@@ -328,9 +334,9 @@ __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const Delt
     for (int j = 0; j < WN; ++j) {
       uint32_t hi, lo;
       split_pair(aw[j][2 * r], aw[j][2 * r + 1], hi, lo);
-      const size_t at = 2 * item * DEL_C * DK + t * DK + (grp * WN + j) * 8 + 2 * q4;
-      *reinterpret_cast<uint32_t*>(p.W + at) = hi;
-      *reinterpret_cast<uint32_t*>(p.W + at + DEL_C * DK) = lo;
+      __nv_bfloat16* w = rec + Rec::W + t * Rec::LDM + (grp * WN + j) * 8 + 2 * q4;
+      *reinterpret_cast<uint32_t*>(w) = hi;
+      *reinterpret_cast<uint32_t*>(w + DEL_C * Rec::LDM) = lo;
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -346,19 +352,17 @@ __global__ void __launch_bounds__(FAC_THREADS, 1) delta_factor_kernel(const Delt
 constexpr int DEL_SLICE = 32;
 
 template <int DK>
-struct DelScan {
-  static constexpr int LDM = DK + 8, LDP = DEL_C + 8, LDN = DEL_SLICE + 8;
-  static constexpr int W = 0;                            // [2][64][LDM]
-  static constexpr int Q = W + 2 * DEL_C * LDM;          // [64][LDM]
-  static constexpr int K = Q + DEL_C * LDM;              // [2][64][LDM]
-  static constexpr int P = K + 2 * DEL_C * LDM;          // [2][64][LDP]
-  static constexpr int S = P + 2 * DEL_C * LDP;          // [2][DK][LDN]
+struct DelScan : DelRecord<DK> {                         // the record, then
+  static constexpr int LDN = DEL_SLICE + 8;
+  static constexpr int S = DelRecord<DK>::ELEMS;         // [2][DK][LDN]
   static constexpr int U = S + 2 * DK * LDN;             // [2][64][LDN]
-  static constexpr int BYTES = (U + 2 * DEL_C * LDN) * 2;
+  static constexpr int BARS = U + 2 * DEL_C * LDN;       // two mbarriers
+  static constexpr int BYTES = BARS * 2 + 16;
+  static constexpr int WQ_BYTES = DelRecord<DK>::K * 2, KP_BYTES = (DelRecord<DK>::ELEMS - DelRecord<DK>::K) * 2;
 };
 
 template <int DK>
-__global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaParams p, int* status) {
   using L = DelScan<DK>;
   constexpr int LDM = L::LDM, LDP = L::LDP, LDN = L::LDN;
   constexpr int SN = DK / 32;                  // n8 tiles of the state a warp owns (16 key rows each)
@@ -374,24 +378,24 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
   float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * p.dkp * p.dvp;
 
-  auto copy_rows = [&](__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, int rows, int width) {
-    for (int i = tid; i < rows * (width / 8); i += DEL_THREADS)
-      cp_async16(dst + i / (width / 8) * ld + i % (width / 8) * 8, src + static_cast<size_t>(i) * 8);
+  uint64_t* bar = reinterpret_cast<uint64_t*>(sm + L::BARS);
+  if (tid == 0) {
+    mbar_init(&bar[0], 1);
+    mbar_init(&bar[1], 1);
+    mbar_fence_init();
+  }
+  __syncthreads();
+  auto load = [&](int c, int which) {      // one thread: W | Qs or Ks | P of chunk c
+    const __nv_bfloat16* src = p.rec + (static_cast<size_t>(c) * p.H + h) * L::ELEMS;
+    const uint32_t bytes = which ? L::KP_BYTES : L::WQ_BYTES;
+    mbar_expect_tx(&bar[which], bytes);
+    bulk_load(sm + (which ? L::K : 0), src + (which ? L::K : 0), bytes, &bar[which]);
   };
-  auto load_wq = [&](int c) {
-    const size_t at = (static_cast<size_t>(c) * p.H + h) * DEL_C * DK;
-    copy_rows(sW, LDM, p.W + 2 * at, 2 * DEL_C, DK);
-    copy_rows(sQ, LDM, p.Qs + at, DEL_C, DK);
-  };
-  auto load_kp = [&](int c) {
-    const size_t item = static_cast<size_t>(c) * p.H + h;
-    copy_rows(sK, LDM, p.Ks + 2 * item * DEL_C * DK, 2 * DEL_C, DK);
-    copy_rows(sP, LDP, p.P + 2 * item * DEL_C * DEL_C, 2 * DEL_C, DEL_C);
-  };
-  load_wq(c0);
-  cp_async_commit();
-  load_kp(c0);
-  cp_async_commit();
+  if (tid == 0) {
+    load(c0, 0);
+    load(c0, 1);
+  }
+  bool ok = true;
 
   float S[SN][4];
   const bool fresh = p.start[s] == 0;
@@ -431,7 +435,8 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
         u0[j][2 * r + 1] = x.y;
       }
     const float d0 = p.end[item * DK + sm_ * 16 + g], d1 = p.end[item * DK + sm_ * 16 + g + 8];
-    cp_async_wait<1>();                  // W and Q of this chunk; K and P may still be on their way
+    // W and Q of this chunk (K and P may still be on their way), and the state written at the end of the previous one
+    ok = mbar_wait_warp(&bar[0], (c - c0) & 1, status, ERR_ATTN_WAIT) && ok;
     __syncthreads();
     float w[2][4] = {}, wl[2][4] = {}, o[2][4] = {};
 #pragma unroll
@@ -454,10 +459,9 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
       for (int r = 0; r < 4; ++r) u0[j][r] -= w[j][r] + wl[j][r];
       put(sU, DEL_C * LDN, mt * 16, (nb + j) * 8, u0[j]);
     }
-    cp_async_wait<0>();
+    ok = mbar_wait_warp(&bar[1], (c - c0) & 1, status, ERR_ATTN_WAIT) && ok;
     __syncthreads();                     // U is complete; W, Q and the old state have been read
-    if (c + 1 < c1) load_wq(c + 1);
-    cp_async_commit();
+    if (tid == 0 && ok && c + 1 < c1) load(c + 1, 0);
 #pragma unroll
     for (int j = 0; j < SN; ++j) {
       S[j][0] *= d0;
@@ -502,8 +506,7 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
               make_float2(o[j][2 * r], o[j][2 * r + 1]);
       }
     __syncthreads();                     // K, P and U have been read
-    if (c + 1 < c1) load_kp(c + 1);
-    cp_async_commit();
+    if (tid == 0 && ok && c + 1 < c1) load(c + 1, 1);
   }
 #pragma unroll
   for (int j = 0; j < SN; ++j)
@@ -512,6 +515,10 @@ __global__ void __launch_bounds__(DEL_THREADS, 1) delta_scan_kernel(const DeltaP
       const int i = sm_ * 16 + g + (r >> 1) * 8, c = n0 + (sn + j) * 8 + 2 * q + (r & 1);
       if (i < p.dkp && c < p.dvp) st[static_cast<size_t>(i) * p.dvp + c] = S[j][r];
     }
+  if (!ok) {   // a copy may still be on its way into shared memory
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+  }
 }
 
 // out = o / rms(o) * w * sigmoid(gate) per head: one warp per (row, head), at most 128 channels.
@@ -541,6 +548,8 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const float* __restri
 
 template <int DK>
 static int launch_delta(const DeltaParams& p, int nchunks, int nlong, cudaStream_t stream) {
+  int* status = status_ptr();
+  if (!status) return 3;
   const int sm1 = DelFactor<DK>::BYTES;
   const int sm2 = DelScan<DK>::BYTES;
   static bool set[64] = {false};
@@ -556,7 +565,7 @@ static int launch_delta(const DeltaParams& p, int nchunks, int nlong, cudaStream
   }
   delta_factor_kernel<DK><<<dim3(nchunks, p.H), FAC_THREADS, sm1, stream>>>(p);
   B2_CHECK_LAUNCH("delta_factor");
-  delta_scan_kernel<DK><<<dim3((p.dvp + DEL_SLICE - 1) / DEL_SLICE, p.H, nlong), DEL_THREADS, sm2, stream>>>(p);
+  delta_scan_kernel<DK><<<dim3((p.dvp + DEL_SLICE - 1) / DEL_SLICE, p.H, nlong), DEL_THREADS, sm2, stream>>>(p, status);
   B2_CHECK_LAUNCH("delta_scan");
   return 0;
 }
@@ -567,8 +576,7 @@ using namespace b2;
 
 // Words the chunked form needs per (chunk, head); the caller allocates nchunks * H times as many 32-bit words.
 B2_EXPORT int b2_delta_chunk_words(int dkp, int dvp) {
-  const int DK = dkp <= 64 ? 64 : 128;
-  return (5 * DEL_C * DK + 2 * DEL_C * DEL_C) / 2 + DEL_C * dvp + DK;
+  return dkp <= 64 ? DelRecord<64>::ELEMS / 2 + DEL_C * dvp + 64 : DelRecord<128>::ELEMS / 2 + DEL_C * dvp + 128;
 }
 
 // rows: the rows row0 .. row0 + rows - 1 the chunks cover (for the final stage).  o: fp32 [M, H * dvp] scratch.
@@ -588,11 +596,8 @@ B2_EXPORT int b2_delta_chunk(const float* q, const float* k, const void* v, cons
   DeltaParams p;
   p.q = q; p.k = k; p.v = static_cast<const __nv_bfloat16*>(v); p.glog = glog; p.beta = beta; p.chunks = chunks; p.first = first;
   p.start = start; p.slot = slot; p.state = state; p.o = o; p.H = H; p.G = G; p.dkp = dkp; p.dvp = dvp; p.seq0 = seq0;
-  p.W = static_cast<__nv_bfloat16*>(ws);
-  p.Qs = p.W + 2 * items * DEL_C * DK;
-  p.Ks = p.Qs + items * DEL_C * DK;
-  p.P = p.Ks + 2 * items * DEL_C * DK;
-  p.U0 = reinterpret_cast<float*>(p.P + 2 * items * DEL_C * DEL_C);
+  p.rec = static_cast<__nv_bfloat16*>(ws);
+  p.U0 = reinterpret_cast<float*>(p.rec + items * (DK == 64 ? DelRecord<64>::ELEMS : DelRecord<128>::ELEMS));
   p.end = p.U0 + items * DEL_C * dvp;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int rc = DK == 64 ? launch_delta<64>(p, nchunks, nlong, st) : launch_delta<128>(p, nchunks, nlong, st);
