@@ -141,43 +141,39 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
   }
   int stage = 0;
   for (; base < t_end; base += STEP) {
-    float kf[U][8], vf[U][8], sc[U][GH];
-    bool valid[U];
+    float sc[U][GH];
     if (RING) {
       issue(stage == 0 ? AR_STAGES - 1 : stage - 1, base + (AR_STAGES - 1) * STEP);
       asm volatile("cp.async.wait_group %0;" ::"n"(AR_STAGES - 1) : "memory");
     }
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
+    // one K (which = 0) or V (1) piece of this lane; zero past the partition and past the head's channels
+    auto piece = [&](int u, int which, float (&f)[8]) {
       const int tok = base + u * TPW + group;
-      valid[u] = tok < t_end;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) kf[u][e] = vf[u][e] = 0.f;
-      if (valid[u]) {
-        if (RING) {
-          const uint8_t* src = ar_dyn + (warp * AR_STAGES * U * 2 * 32 + lane) * 16 + ((stage * U + u) * 2) * 512;
-          if (kin) vload8(reinterpret_cast<const __nv_bfloat16*>(src), kf[u]);
-          if (vin) vload8(reinterpret_cast<const __nv_bfloat16*>(src + 512), vf[u]);
-        } else {
-          const size_t at = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
-          if (kin) vload8(kc + at * kts, kf[u]);
-          if (vin) vload8(vc + at * vts, vf[u]);
-        }
+      for (int e = 0; e < 8; ++e) f[e] = 0.f;
+      if (tok >= t_end || !(which ? vin : kin)) return;
+      if (RING) {
+        vload8(reinterpret_cast<const __nv_bfloat16*>(ar_dyn + (warp * AR_STAGES * U * 2 * 32 + lane) * 16 +
+                                                      ((stage * U + u) * 2 + which) * 512), f);
+      } else {
+        const size_t at = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
+        vload8(which ? vc + at * vts : kc + at * kts, f);
       }
-    }
-    stage = stage + 1 == AR_STAGES ? 0 : stage + 1;
+    };
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int tok = base + u * TPW + group;
+      float kf[8];
+      piece(u, 0, kf);
 #pragma unroll
       for (int g = 0; g < GH; ++g) {
         float d = 0.f;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) d = fmaf(qr[g][e], kf[u][e], d);
+        for (int e = 0; e < 8; ++e) d = fmaf(qr[g][e], kf[e], d);
 #pragma unroll
         for (int o = LPT / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-        if (p.rel && valid[u] && g < nh) d += sBias[g * p.partition + tok - t_begin];
-        sc[u][g] = valid[u] ? d : -INFINITY;
+        if (p.rel && tok < t_end && g < nh) d += sBias[g * p.partition + tok - t_begin];
+        sc[u][g] = tok < t_end ? d : -INFINITY;
       }
     }
 #pragma unroll
@@ -185,7 +181,11 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
       float mn = m[g];
 #pragma unroll
       for (int u = 0; u < U; ++u) mn = fmaxf(mn, sc[u][g]);
-      if (mn == -INFINITY) continue;   // this lane group has not seen a token yet
+      if (mn == -INFINITY) {   // this lane group has not seen a token yet: its weights are zero
+#pragma unroll
+        for (int u = 0; u < U; ++u) sc[u][g] = 0.f;
+        continue;
+      }
       const float alpha = ar_exp2<T>(m[g] - mn);
       m[g] = mn;
 #pragma unroll
@@ -193,13 +193,21 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
       float ps = 0.f;
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        const float w = ar_exp2<T>(sc[u][g] - mn);
-        ps += w;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[g][e] = fmaf(w, vf[u][e], acc[g][e]);
+        sc[u][g] = ar_exp2<T>(sc[u][g] - mn);
+        ps += sc[u][g];
       }
       l[g] = l[g] * alpha + ps;
     }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      float vf[8];
+      piece(u, 1, vf);
+#pragma unroll
+      for (int g = 0; g < GH; ++g)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[g][e] = fmaf(sc[u][g], vf[e], acc[g][e]);
+    }
+    stage = stage + 1 == AR_STAGES ? 0 : stage + 1;
   }
 #pragma unroll
   for (int o = LPT; o < 32; o <<= 1)
