@@ -438,9 +438,7 @@ class InferenceEngine:
     def _portions_forward(self, ids: List, starts: List[int], counts: List[int], tokens: List[int], **kw) -> torch.Tensor:
         """One forward pass over portions of sequences whose pages are reserved; logits as ``ModelRunner.forward``."""
         ctx = self.runner.prepare_prefill(ids, starts, counts)
-        tok = torch.tensor(tokens, dtype=torch.long)
-        tok = tok.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else tok
-        return self.runner.forward(tok, ctx, **kw)
+        return self.runner.forward(self._stage("tokens", torch.tensor(tokens, dtype=torch.long)), ctx, **kw)
 
     # ---- given tokens instead of sampled ones -----------------------------------------------------------------------
     @_locked
@@ -624,18 +622,10 @@ class InferenceEngine:
                 return None
 
     def _stage(self, name: str, t: torch.Tensor) -> torch.Tensor:
-        """Host tensor -> device through a small ring of pinned staging buffers (no page-locking per call; a ring
-        because the copy of the previous step may not have run yet when this step's values are written)."""
+        """Host tensor -> device through the runner's ring of pinned staging buffers."""
         if self.device.type != "cuda":
             return t
-        ring = self._stage_rings.setdefault((name, t.dtype), {"bufs": [None] * 4, "i": 0})
-        i = ring["i"] = (ring["i"] + 1) % 4
-        buf = ring["bufs"][i]
-        if buf is None or buf.numel() < t.numel():
-            buf = ring["bufs"][i] = torch.empty(max(256, t.numel()), dtype=t.dtype, pin_memory=True)
-        view = buf[:t.numel()].view(t.shape)
-        view.copy_(t)
-        return view.to(self.device, non_blocking=True)
+        return self.runner._stage(t)
 
     def _pinned_out(self, n: int):
         ring = self._stage_rings.setdefault("out", {"bufs": [None] * 4, "i": 0})

@@ -57,16 +57,26 @@ class ModelRunner:
         self.fuse_kv_store = True     # norm + RoPE + cache store in one launch for 16-bit caches (False: two launches)
 
     # ---- metadata ----------------------------------------------------------------------------------------
+    STAGE_RING = 64     # pinned buffers per dtype, reused half a ring at a time
+
     def _stage(self, t: torch.Tensor) -> torch.Tensor:
         """Host tensor -> device through a ring of reusable pinned buffers.  Page-locking a fresh buffer per tensor
         costs more than the copy; a ring (not one buffer) because the engine queues a step's copies while the GPU
-        may still be running the previous step, whose staging memory must stay untouched until its copy has run."""
+        may still be running earlier steps, whose staging memory must stay untouched until its copies have run: before
+        one half of the ring is filled again, the event recorded behind its last copy is waited for (steps that read
+        nothing back - chunks of a long prompt - let the host run far ahead)."""
         if self.device.type != "cuda":
             return t
-        n = t.numel() * t.element_size()
         ring = self.__dict__.setdefault("_rings", {})
-        r = ring.setdefault(t.dtype, {"bufs": [None] * 16, "i": 0})
-        i = r["i"] = (r["i"] + 1) % len(r["bufs"])
+        r = ring.setdefault(t.dtype, {"bufs": [None] * self.STAGE_RING, "i": -1, "events": [None, None]})
+        i = r["i"] = (r["i"] + 1) % self.STAGE_RING
+        if i % (self.STAGE_RING // 2) == 0:
+            half = i // (self.STAGE_RING // 2)
+            ev = torch.cuda.Event()
+            ev.record()
+            r["events"][1 - half] = ev
+            if r["events"][half] is not None:
+                r["events"][half].synchronize()
         if r["bufs"][i] is None or r["bufs"][i].numel() < t.numel():
             r["bufs"][i] = torch.empty(max(1024, t.numel()), dtype=t.dtype, pin_memory=True)
         view = r["bufs"][i][:t.numel()].view(t.shape)

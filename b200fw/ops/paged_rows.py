@@ -108,7 +108,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     if lead == 0:
         return
     keys = p.max_keys if chunk <= 0 else min(p.max_keys, chunk)
-    part, nsplit = _split(lead, G * ((H // G + 3) // 4), keys)
+    groups = (H // G + 3) // 4
+    part, nsplit = _split(lead, G * groups, -(-(H // G) // groups), keys)
     po = pm = None
     if nsplit > 1:
         po = torch.empty((lead, H, nsplit, dvp), device=q.device, dtype=torch.float32)
@@ -122,10 +123,13 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     nv.count_launch(2 if nsplit > 1 else 1)
 
 
-def _split(rows: int, ctas_per_row: int, keys: int):
-    """Keys per split and number of splits: enough CTAs for a few waves over 148 SMs, 256 to 2048 keys each."""
-    want = 4 * 148 * 3
-    n = max(min((keys + 255) // 256, -(-want // max(1, rows * ctas_per_row))), (keys + 2047) // 2048)
+def _split(rows: int, groups_per_row: int, heads: int, keys: int):
+    """Keys per split and number of splits (measured at 8 to 256 rows): one wave of resident CTAs when the rows alone are
+    fewer than that, else three or four splits so that the last wave is short; 128 to 2048 keys each.  ``heads``: query heads
+    of a CTA (three or four leave registers for three CTAs per SM instead of four)."""
+    ctas, resident, few = max(1, rows * groups_per_row), 148 * (3 if heads > 2 else 4), 3 if heads > 2 else 4
+    n = 1 if ctas > 8 * resident else min((keys + 127) // 128, max(resident // ctas, few))
+    n = max(n, (keys + 2047) // 2048)
     if n <= 1:
         return max(1, keys), 1
     part = ((keys + n - 1) // n + 63) // 64 * 64

@@ -418,6 +418,27 @@ def test_graph_decoding_matches_plain_bf16():
     assert outs[0] == outs[1]
 
 
+@pytest.mark.gpu
+def test_host_running_ahead_of_the_gpu():
+    """Chunks of a long prompt read nothing back, so the host queues many steps ahead: the staged row layouts of earlier steps
+    must survive until their copies have run."""
+    cfg, w = case("wide")
+    m = build(cfg, w, ("cuda", torch.bfloat16))
+    prompt = toks(3000, cfg["vocab"], 99)
+    outs = []
+    for sync in (True, False):
+        eng = engine(m, tokens=3200, seqs=2, chunk_size=17, max_prefill_tokens=17, adaptive_chunking=False)
+        r = eng.add_request("a", prompt, 6)
+        if not sync:
+            torch.cuda._sleep(int(2e8))          # about 0.1 s of GPU time in front of the first step
+        while eng.has_pending():
+            eng.step()
+            if sync:
+                torch.cuda.synchronize()
+        outs.append(r.output_tokens)
+    assert outs[0] == outs[1]
+
+
 def test_stop_and_abort():
     cfg, w = case("odd")
     m = build(cfg, w, ("cpu", torch.float32))
