@@ -355,8 +355,7 @@ __device__ __forceinline__ void warp_store_rows_128B(uint8_t* stage, const uint4
 }
 
 // ---- small numeric helpers -----------------------------------------------------------------
-// 2^x on the special-function unit, one instruction (exp2f adds range handling around the same
-// instruction; softmax arguments are <= 0 and -inf maps to 0, so none of it is needed).
+// 2^x on the special-function unit, one instruction: softmax arguments are <= 0 and -inf maps to 0.
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
