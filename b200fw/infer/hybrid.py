@@ -108,7 +108,7 @@ class HybridModelRunner(ModelRunner):
         m, p = self.model, ctx.portions
         self.forward_calls += 1
         ids = token_ids if ctx.row_order is None else token_ids.index_select(0, ctx.row_order)
-        x = ops.embedding_f32(ids, m.embed_tokens, m.cfg.vocab_size)
+        x, h = m.embed(ids)
         tables: Dict[Tuple[float, int], Tuple[torch.Tensor, torch.Tensor]] = {}
 
         def rope(base: float, dims: int):
@@ -119,7 +119,7 @@ class HybridModelRunner(ModelRunner):
                 tables[key] = ops.rope_rows(p.positions, self._turns[key])
             return tables[key]
 
-        h, n = None, len(m.layers)
+        n = len(m.layers)
         for li, layer in enumerate(m.layers):
             after = m.layers[li + 1].norm1 if li + 1 < n else None
             h = layer(x, h, p, self.pool.layer_kv(li), self.state.layers[li], rope, after)
@@ -172,6 +172,11 @@ def build_portions(starts: Sequence[int], counts: Sequence[int], tables: Sequenc
             first = np.concatenate([[0], np.cumsum((c[ns:] + size - 1) // size)]).astype(np.int32)
             setattr(p, f"chunks{size}", dev(_row_tiles(cu, ns, n, size)))
             setattr(p, f"first{size}", dev(first))
+        pages = (st[ns:] + c[ns:] + 15) // 16
+        first = (np.cumsum(pages) - pages).astype(np.int32)
+        p.ctx_counts = pages.tolist()
+        p.ctx_pages = dev(np.concatenate([bt[ns + i, :k] for i, k in enumerate(p.ctx_counts)]))
+        p.ctx_tables = dev(first[:, None] + np.minimum(np.arange(pages.max(), dtype=np.int32)[None, :], pages[:, None].astype(np.int32) - 1))
     return p, order, place
 
 

@@ -230,6 +230,10 @@ class FetelornModel(nn.Module):
         return [l.state_shapes() for l in self.layers]
 
     # ---- pieces the runner calls ------------------------------------------------------------------------------
+    def embed(self, ids: torch.Tensor):
+        """The residual stream's first rows (fp32), and what the first layer reads if that is not its own norm's business."""
+        return ops.embedding_f32(ids, self.embed_tokens, self.cfg.vocab_size), None
+
     def logits_from_hidden(self, h: torch.Tensor) -> torch.Tensor:
         out = torch.empty((h.shape[0], self.embed_tokens.shape[0]), dtype=torch.float32, device=h.device)
         return ops.gemm(h, self.embed_tokens, out=out)[:, :self.cfg.vocab_size]

@@ -34,6 +34,20 @@ class Slot:
         return self.view.detach().reshape(self.shape)
 
 
+@dataclass
+class RowSplitSlot:
+    """A checkpoint tensor whose leading rows live in several places: ``parts`` = (slot, rows) in order."""
+    parts: List[Tuple[Slot, int]]
+    shape: Tuple[int, ...]
+
+    def load(self, t: torch.Tensor) -> None:
+        for (slot, _), piece in zip(self.parts, t.split([n for _, n in self.parts])):
+            slot.load(piece)
+
+    def export(self) -> torch.Tensor:
+        return torch.cat([slot.export() for slot, _ in self.parts])
+
+
 def _param(*shape, dtype, device) -> nn.Parameter:
     return nn.Parameter(torch.zeros(*shape, dtype=dtype, device=device), requires_grad=False)
 
@@ -59,8 +73,14 @@ class PackedRows(nn.Module):
         a, e = self.sections[first], self.sections[last or first]
         return y[:, a[0]:e[0] + e[1] * pad8(e[2])]
 
-    def forward(self, x: torch.Tensor) -> torch.Tensor:
-        return ops.linear(x, self.weight)
+    def end(self, name: str) -> int:
+        """Columns up to and with section ``name``."""
+        at, heads, d = self.sections[name]
+        return at + heads * pad8(d)
+
+    def forward(self, x: torch.Tensor, act: Optional[str] = None, cols: Optional[int] = None) -> torch.Tensor:
+        """``act`` on the first ``cols`` columns, in the product's epilogue (:func:`b200fw.ops.linear_act`)."""
+        return ops.linear_act(x, self.weight, act, cols)
 
 
 class PackedCols(nn.Module):
@@ -109,6 +129,22 @@ class DenseGLU(nn.Module):
 
     def run(self, y: "Sections", out: torch.Tensor) -> None:
         ops.glu(y.cols("gate"), y.cols("up"), out)
+
+
+class SquaredReLU(nn.Module):
+    """``W_down relu(W_up h)^2``, a pair of products of its own: for layers whose feed-forward reads what the mixer left."""
+
+    def __init__(self, hidden: int, inner: int, dtype, device):
+        super().__init__()
+        self.up = PackedRows(hidden, [("up", 1, inner)], dtype, device)
+        self.down = PackedCols(hidden, [("down", 1, inner)], dtype, device)
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        return {prefix + "up": self.up.slot("up"), prefix + "down": self.down.slot("down")}
+
+    def run(self, h: torch.Tensor) -> torch.Tensor:
+        """fp32 ``[M, hidden]``."""
+        return self.down(self.up(h, "relu2"))
 
 
 class Sections:
@@ -247,3 +283,149 @@ class GatedDelta(nn.Module):
         ops.gated_delta(q, k, v, g, beta, z[:, H * dkp:], self.norm, out, state["S"], p, self.kv_heads, self.dim, self.vdim,
                         self.eps)
         return self.o(out)
+
+
+class Lightning(nn.Module):
+    """Linear attention with a fixed decay per head over silu features of q, k and v; one norm over all heads together and a
+    sigmoid gate.  No positions: the decay orders the tokens."""
+
+    def __init__(self, hidden: int, heads: int, dim: int, vdim: int, decay: List[float], eps: float, dtype, device):
+        super().__init__()
+        if len(decay) != heads:
+            raise ValueError(f"lightning: {len(decay)} decays for {heads} heads")
+        self.heads, self.dim, self.vdim, self.eps = heads, dim, vdim, eps
+        self.in_proj = PackedRows(hidden, [("q", heads, dim), ("k", heads, dim), ("v", heads, vdim), ("g", heads, vdim)], dtype,
+                                  device)
+        self.o = PackedCols(hidden, [("o", heads, vdim)], dtype, device)
+        self.norm = _param(heads, pad8(vdim), dtype=dtype, device=device)
+        self.register_buffer("decay", torch.tensor(decay, dtype=torch.float32, device=device), persistent=False)
+
+    def kv_shape(self) -> None:
+        return None
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        return {"S": (self.heads, pad8(self.dim), pad8(self.vdim))}
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        t = {prefix + n: self.in_proj.slot(n) for n in "qkvg"}
+        t[prefix + "o"] = self.o.slot("o")
+        t[prefix + "norm"] = Slot(self.norm.data[:, :self.vdim], (self.heads * self.vdim,))
+        return t
+
+    def run(self, h: torch.Tensor, p, kv, state: Dict[str, torch.Tensor], rope) -> Tuple[torch.Tensor, Dict]:
+        """fp32 ``[M, hidden]``, still to be divided by the heads' common root mean square: that factor of a row commutes with
+        the projection, so the sum after it applies it (:func:`b200fw.ops.post_norm`)."""
+        P = self.in_proj
+        y = P(h, "silu", P.end("v"))
+        out = self.o.buffer(y.shape[0])
+        sumsq = torch.empty((y.shape[0], self.heads), dtype=torch.float32, device=y.device)
+        ops.retention(P.cols(y, "q"), P.cols(y, "k"), P.cols(y, "v"), P.cols(y, "g"), out, state["S"], p, self.decay, self.dim,
+                      self.vdim, None, None, 1.0, self.eps, self.norm.view(-1), sumsq)
+        return self.o(out), {"sumsq": sumsq, "sumsq_n": self.heads * self.vdim}
+
+
+class DifferentialAttention(nn.Module):
+    """Two softmax attentions per head over one set of values, subtracted; sliding window, soft cap, biases, normed and rotated
+    queries and keys (channel pairs), a norm per head without weight and a sigmoid gate per channel.  Grouped query heads."""
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, softcap: float, window: int,
+                 rot_base: float, rot_dims: int, diff: float, eps: float, dtype, device):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"attention: {heads} query heads do not divide over {kv_heads} key/value heads")
+        if rot_dims % 2 or not 0 <= rot_dims <= dim:
+            raise ValueError(f"attention: rotary dims {rot_dims} must be even and at most the head size {dim}")
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.softcap, self.window, self.diff, self.eps = float(scale), float(softcap), int(window), float(diff), eps
+        self.rot = (float(rot_base), int(rot_dims))
+        self.in_proj = PackedRows(hidden, [("q", 2 * heads, dim), ("k", 2 * kv_heads, dim), ("v", kv_heads, vdim), ("g", heads, vdim)],
+                                  dtype, device)
+        self.bias = _param(self.in_proj.end("v"), dtype=dtype, device=device)
+        self.q_norm = _param(dim, dtype=dtype, device=device)
+        self.k_norm = _param(dim, dtype=dtype, device=device)
+        self.lam = _param(4, pad8(dim), dtype=dtype, device=device)
+        self.o = PackedCols(hidden, [("o", heads, vdim)], dtype, device)
+        self.o_bias = _param(pad8(hidden), dtype=dtype, device=device)
+        self.hidden = hidden
+
+    def kv_shape(self) -> Tuple[int, int, int]:
+        return self.kv_heads, 2 * pad8(self.dim), pad8(self.vdim)
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        return {}
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        t = {prefix + n: self.in_proj.slot(n) for n in "qkvg"}
+        for n in "qkv":
+            at, heads, d = self.in_proj.sections[n]
+            t[prefix + n + ".b"] = Slot(self.bias.data[at:at + heads * pad8(d)].view(heads, pad8(d))[:, :d], (heads * d,))
+        t[prefix + "q.norm"] = Slot(self.q_norm.data, (self.dim,))
+        t[prefix + "k.norm"] = Slot(self.k_norm.data, (self.dim,))
+        for i, n in enumerate(("lq1", "lk1", "lq2", "lk2")):
+            t[prefix + n] = Slot(self.lam.data[i, :self.dim], (self.dim,))
+        t[prefix + "o"] = self.o.slot("o")
+        t[prefix + "o.b"] = Slot(self.o_bias.data[:self.hidden], (self.hidden,))
+        return t
+
+    def run(self, h: torch.Tensor, p, kv: Tuple[torch.Tensor, torch.Tensor], state, rope) -> Tuple[torch.Tensor, Dict]:
+        """fp32 ``[M, hidden]`` without the output bias, which the sum after it adds."""
+        kc, vc = kv
+        kc = kc.view(kc.shape[0], kc.shape[1], 2 * self.kv_heads, pad8(self.dim))
+        P = self.in_proj
+        y = P(h)
+        cos, sin = rope(*self.rot) if self.rot[1] else (None, None)
+        q = ops.qk_norm_store(P.cols(y, "q"), P.cols(y, "k"), P.cols(y, "v"), kc, vc, p, 2 * self.heads, self.dim, True, self.eps,
+                              self.q_norm, self.k_norm, self.bias, cos, sin)
+        out = self.o.buffer(y.shape[0])
+        ops.differential_attention(q, kc, vc, out, p, self.heads, self.scale, self.lam, self.diff, self.vdim, self.eps,
+                                   P.cols(y, "g"), self.window, self.softcap)
+        return self.o(out), {"bias": self.o_bias}
+
+
+class LatentAttention(nn.Module):
+    """Softmax attention whose keys and values are made from one cached latent per token, plus one rotated key part that all
+    heads share; a sink per head.  ``w_key`` holds the key projection beside an identity for the rotated part."""
+
+    def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float, rot_base: float,
+                 eps: float, dtype, device):
+        super().__init__()
+        if rot_dim % 2 or rot_dim < 2:
+            raise ValueError(f"latent attention: the rotated size {rot_dim} must be even and positive")
+        self.heads, self.dim, self.rot_dim, self.vdim, self.rank = heads, dim, rot_dim, vdim, rank
+        self.scale, self.eps, self.rot = float(scale), eps, (float(rot_base), int(rot_dim))
+        self.in_proj = PackedRows(hidden, [("q", heads, dim + rot_dim), ("c", 1, rank), ("kr", 1, rot_dim)], dtype, device)
+        self.c_norm = _param(pad8(rank), dtype=dtype, device=device)
+        self.w_key = _param(heads, pad8(dim + rot_dim), pad8(rank) + pad8(rot_dim), dtype=dtype, device=device)
+        i = torch.arange(rot_dim, device=device)
+        self.w_key.data[:, dim + i, pad8(rank) + i] = 1.0
+        self.w_value = _param(heads, pad8(vdim), pad8(rank), dtype=dtype, device=device)
+        self.sink = _param(heads, dtype=dtype, device=device)
+        self.o = PackedCols(hidden, [("o", heads, vdim)], dtype, device)
+
+    def kv_shape(self) -> Tuple[int, int, int]:
+        return 1, pad8(self.rank) + pad8(self.rot_dim), 0
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        return {}
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        H, hidden = self.heads, self.in_proj.in_features
+        t = {prefix + "q": self.in_proj.slot("q"),
+             prefix + "dkv": RowSplitSlot([(self.in_proj.slot("c"), self.rank), (self.in_proj.slot("kr"), self.rot_dim)],
+                                          (self.rank + self.rot_dim, hidden)),
+             prefix + "dkv.norm": Slot(self.c_norm.data[:self.rank], (self.rank,)),
+             prefix + "uk": Slot(self.w_key.data[:, :self.dim, :self.rank], (H * self.dim, self.rank)),
+             prefix + "uv": Slot(self.w_value.data[:, :self.vdim, :self.rank], (H * self.vdim, self.rank)),
+             prefix + "sink": Slot(self.sink.data, (H,)), prefix + "o": self.o.slot("o")}
+        return t
+
+    def run(self, h: torch.Tensor, p, kv: Tuple[torch.Tensor, torch.Tensor], state, rope) -> Tuple[torch.Tensor, Dict]:
+        """fp32 ``[M, hidden]``."""
+        P = self.in_proj
+        y = P(h)
+        q = P.cols(y, "q")
+        ops.latent_store(q, P.cols(y, "c"), P.cols(y, "kr"), kv[0], p, self.heads, self.dim, self.rank, self.rot_dim, self.c_norm,
+                         *rope(*self.rot), self.eps)
+        out = self.o.buffer(y.shape[0])
+        ops.latent_attention(q, kv[0], out, p, self.w_key, self.w_value, self.scale, self.sink)
+        return self.o(out), {}

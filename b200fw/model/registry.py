@@ -15,6 +15,7 @@ from .config import PRESETS as DENSE_PRESETS
 from .config import ModelConfig
 from .fetelorn import FETELORN_PRESETS, FetelornConfig, FetelornModel
 from .qwen3 import ParallelTransformerModel
+from .sotazen import SOTAZEN_PRESETS, SotazenConfig, SotazenModel
 
 
 @dataclass(frozen=True)
@@ -70,7 +71,7 @@ def load_slots(model, tensors: Iterable[Tuple[str, torch.Tensor]], strict: bool 
     return len(copies), missing
 
 
-def _load_fetelorn(model, path: str, strict: bool = True) -> Tuple[int, int]:
+def _load_slots_at(model, path: str, strict: bool = True) -> Tuple[int, int]:
     return load_slots(model, hf_io._load_all(path).items(), strict, path)
 
 
@@ -81,10 +82,13 @@ ARCHITECTURES: Dict[str, Architecture] = {
                                      ("host", "gemm", "norm_rope", "attention_fwd", "paged", "sampling")),
     "Fetelorn": Architecture("Fetelorn", FetelornConfig,
                              lambda path: FetelornConfig.from_dict(_config_json(path), safetensors_shapes(path)),
-                             FetelornModel, _load_fetelorn,
+                             FetelornModel, _load_slots_at,
                              ("host", "gemm", "residual", "linear_state", "retention_chunk", "delta_chunk", "attention_rows", "attention_fwd", "sampling"), float32=True),
+    "Sotazen": Architecture("Sotazen", SotazenConfig, lambda path: SotazenConfig.from_dict(_config_json(path)), SotazenModel,
+                            _load_slots_at, ("host", "gemm", "residual", "linear_state", "retention_chunk", "attention_rows",
+                                             "attention_latent", "attention_fwd", "sampling"), float32=True),
 }
-PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS}
+PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS, **SOTAZEN_PRESETS}
 
 
 def architecture_at(path: str) -> Architecture:

@@ -12,6 +12,29 @@ import torch
 from .. import _native as nv
 
 OUT_FP32, ACCUMULATE, RESIDUAL = 1, 2, 4
+ACTS = {None: 0, "silu": 1, "relu2": 2}
+
+
+def linear_act(a: torch.Tensor, b: torch.Tensor, act: Optional[str], cols: Optional[int] = None) -> torch.Tensor:
+    """``a [M,K] @ b [N,K]^T`` in ``a``'s dtype, the first ``cols`` columns (all by default; a multiple of 8) through an
+    activation inside the product's epilogue, on the 32-bit accumulator: ``silu`` or ``relu2`` (the square of relu)."""
+    N = b.shape[0]
+    cols = N if cols is None else cols
+    if act is None:
+        return linear(a, b)
+    if not a.is_cuda:
+        r = a.float() @ b.float().t()
+        z = r[:, :cols]
+        r[:, :cols] = z * torch.sigmoid(z) if act == "silu" else z.clamp(min=0) ** 2
+        return r.to(a.dtype)
+    if a.dtype == torch.float32:
+        return _gemm_f32(a, b, False, False, None, False, None, None, ACTS[act], cols)
+    assert a.dtype == b.dtype == torch.bfloat16 and a.stride(-1) == 1 and b.stride(-1) == 1 and a.shape[1] == b.shape[1]
+    out = torch.empty((a.shape[0], N), device=a.device, dtype=torch.bfloat16)
+    nv.check(nv.lib().b2_gemm_bf16_act(nv.ptr(a), nv.ptr(b), nv.ptr(out), a.shape[0], N, a.shape[1], a.stride(0), b.stride(0), N,
+                                       ACTS[act], cols, nv.stream_ptr()), "gemm_act")
+    nv.count_launch()
+    return out
 
 
 def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = False,
@@ -77,7 +100,7 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
     return out
 
 
-def _gemm_f32(a, b, a_mn, b_mn, out, accumulate, residual, ext) -> torch.Tensor:
+def _gemm_f32(a, b, a_mn, b_mn, out, accumulate, residual, ext, act=0, act_cols=0) -> torch.Tensor:
     """``a [M,K] @ b [N,K]^T`` in true 32-bit (plain FMA kernel, no reduced-precision tensor-core mode): inference of a model
     that was asked to run in float32."""
     if a_mn or b_mn or residual is not None or ext is not None:
@@ -87,7 +110,7 @@ def _gemm_f32(a, b, a_mn, b_mn, out, accumulate, residual, ext) -> torch.Tensor:
         out = torch.empty((a.shape[0], b.shape[0]), device=a.device, dtype=torch.float32)
     assert out.shape == (a.shape[0], b.shape[0]) and out.stride(-1) == 1 and out.dtype == torch.float32
     nv.check(nv.lib().b2_gemm_f32(nv.ptr(a), nv.ptr(b), nv.ptr(out), a.shape[0], b.shape[0], a.shape[1], a.stride(0),
-                                  b.stride(0), out.stride(0), int(accumulate), nv.stream_ptr()), "gemm_f32")
+                                  b.stride(0), out.stride(0), int(accumulate), act, act_cols, nv.stream_ptr()), "gemm_f32")
     nv.count_launch()
     return out
 

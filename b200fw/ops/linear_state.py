@@ -31,10 +31,13 @@ def _head_rms(o: torch.Tensor, dv: int, eps: float) -> torch.Tensor:
 
 def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, state: torch.Tensor,
               p: Portions, decay: torch.Tensor, dk: int, dv: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
-              k_scale: float, eps: float) -> None:
+              k_scale: float, eps: float, norm_w: Optional[torch.Tensor] = None, sumsq: Optional[torch.Tensor] = None) -> None:
     """``S <- decay_h S + k v^T``, ``o = S^T q`` with rotary positions on q and k and ``k_scale`` on the rotated k; then
     ``out = o / rms(o) * silu(gate)`` per head.  ``q, k [M, H*dkp]``, ``v, gate, out [M, H*dvp]`` are column slices
-    (the first four of one matrix)."""
+    (the first four of one matrix).
+
+    ``sumsq [M, H]`` (fp32, written): the heads are normed together, by whoever reads ``out``'s projection; then
+    ``out = o * norm_w * sigmoid(gate)`` with ``norm_w [H*dvp]``, and ``sumsq`` holds every head's ``sum(o^2)``."""
     H, dkp, dvp = state.shape[1:]
     rot = 0 if cos is None else 2 * cos.shape[1]
     if not q.is_cuda:
@@ -57,6 +60,10 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Ten
                 S = decay[:, None, None] * S + kf[t, :, :, None] * vf[t, :, None, :]
                 o[t] = (S * qf[t, :, :, None]).sum(1)
             state[slot] = S
+        if sumsq is not None:
+            sumsq.copy_((o * o).sum(-1))
+            out.copy_((o * norm_w.float().reshape(H, dvp) * torch.sigmoid(gf)).reshape(M, H * dvp).to(out.dtype))
+            return
         out.copy_((_head_rms(o, dv, eps) * gf * torch.sigmoid(gf)).reshape(M, H * dvp).to(out.dtype))
         return
     assert q.stride(0) == k.stride(0) == v.stride(0) == gate.stride(0)
@@ -66,7 +73,7 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Ten
         nv.check(nv.lib().b2_retention_serial(
             nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(out), nv.ptr(state), nv.ptr(decay), nv.ptr(cos), nv.ptr(sin),
             cu, st, sl, ns, p.max_short, H, dk, dkp, dv, dvp, rot, nv.ctypes.c_longlong(q.stride(0)),
-            nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps),
+            nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps), nv.ptr(norm_w), nv.ptr(sumsq),
             int(q.dtype == torch.float32), nv.stream_ptr()), "retention_serial")
         nv.count_launch()
     if p.nseq > ns:
@@ -77,14 +84,14 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Ten
                 nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(out), nv.ptr(ws), nv.ptr(state), nv.ptr(decay), nv.ptr(cos),
                 nv.ptr(sin), nv.ptr(p.chunks128), nv.ptr(p.first128), nv.ptr(p.starts), nv.ptr(p.slots), n, ns, nlong, H, dk, dkp,
                 dv, dvp, rot, nv.ctypes.c_longlong(q.stride(0)), nv.ctypes.c_longlong(out.stride(0)),
-                nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps), nv.stream_ptr()), "retention_chunk")
+                nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps), nv.ptr(norm_w), nv.ptr(sumsq), nv.stream_ptr()), "retention_chunk")
             nv.count_launch(3)
             return
         cu, st, sl = _sub(p, ns)
         nv.check(nv.lib().b2_retention_serial(
             nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(out), nv.ptr(state), nv.ptr(decay), nv.ptr(cos), nv.ptr(sin),
             cu, st, sl, nlong, p.max_long, H, dk, dkp, dv, dvp, rot, nv.ctypes.c_longlong(q.stride(0)),
-            nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps),
+            nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(k_scale), nv.ctypes.c_float(eps), nv.ptr(norm_w), nv.ptr(sumsq),
             int(q.dtype == torch.float32), nv.stream_ptr()), "retention_serial")
         nv.count_launch()
 

@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
+from typing import List, Optional
 
 import torch
 
@@ -36,6 +36,11 @@ class Portions:
     chunks128: Optional[torch.Tensor] = None
     first128: Optional[torch.Tensor] = None
     max_long: int = 0
+    # contexts of the long portions laid out page after page: int32 [pages] page of the pool, int32 [nlong, max pages] where a
+    # sequence's pages are in that layout, pages per sequence
+    ctx_pages: Optional[torch.Tensor] = None
+    ctx_tables: Optional[torch.Tensor] = None
+    ctx_counts: Optional[List[int]] = None
     ragged: bool = True                      # False: every sequence is one row (decode): row r is sequence r
 
     @property

@@ -16,15 +16,19 @@ def _f32(t: torch.Tensor) -> int:
     return int(t.dtype == torch.float32)
 
 
-def embedding_f32(ids: torch.Tensor, table: torch.Tensor, vocab: Optional[int] = None) -> torch.Tensor:
-    """Rows of ``table`` as fp32; an id outside ``[0, vocab)`` (padding rows of a graph batch) gives zeros on a GPU."""
+def embedding_f32(ids: torch.Tensor, table: torch.Tensor, vocab: Optional[int] = None, scale: float = 1.0, h: bool = False):
+    """Rows of ``table`` times ``scale`` as fp32; an id outside ``[0, vocab)`` (padding rows of a graph batch) gives zeros on a
+    GPU.  ``h``: returns ``(x, x in the table's dtype)``."""
     if not table.is_cuda:
-        return table[ids].float()
+        x = table[ids].float() * scale
+        return (x, x.to(table.dtype)) if h else x
     x = torch.empty((ids.numel(), table.shape[1]), device=table.device, dtype=torch.float32)
-    nv.check(nv.lib().b2_embed_f32(nv.ptr(ids), nv.ptr(table), nv.ptr(x), ids.numel(), table.shape[1],
-                                   table.shape[0] if vocab is None else vocab, _f32(table), nv.stream_ptr()), "embed_f32")
+    low = torch.empty(x.shape, device=x.device, dtype=table.dtype) if h and table.dtype != torch.float32 else None
+    nv.check(nv.lib().b2_embed_f32(nv.ptr(ids), nv.ptr(table), nv.ptr(x), nv.ptr(low), ids.numel(), table.shape[1],
+                                   table.shape[0] if vocab is None else vocab, nv.ctypes.c_float(scale), _f32(table),
+                                   nv.stream_ptr()), "embed_f32")
     nv.count_launch()
-    return x
+    return (x, x if low is None else low) if h else x
 
 
 def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, n: int, eps: float, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -57,6 +61,27 @@ def merge_norm_add(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor, wa: torch.
                                         _f32(wa), nv.stream_ptr()), "merge_norm_add")
     nv.count_launch()
     return h
+
+
+def post_norm(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, alpha: float, n: int, eps: float,
+              bias: Optional[torch.Tensor] = None, sumsq: Optional[torch.Tensor] = None, sumsq_n: int = 0) -> torch.Tensor:
+    """In place ``x = rms(alpha * x + y + bias) * w`` (``x``, ``y`` fp32); returns the new ``x`` in ``w``'s dtype (``x``
+    itself in 32-bit).  ``sumsq [rows, parts]``: ``y`` is first divided by the root mean square (over ``sumsq_n`` channels) of
+    the input it was projected from, whose sums of squares these are."""
+    if not x.is_cuda:
+        if sumsq is not None:
+            y = y * torch.rsqrt(sumsq.sum(-1, keepdim=True) / sumsq_n + eps)
+        t = alpha * x + y
+        if bias is not None:
+            t = t + bias.float()
+        x.copy_(t * torch.rsqrt((t[:, :n] * t[:, :n]).mean(-1, keepdim=True) + eps) * w.float())
+        return x if w.dtype == torch.float32 else x.to(w.dtype)
+    h = None if w.dtype == torch.float32 else torch.empty(x.shape, device=x.device, dtype=w.dtype)
+    nv.check(nv.lib().b2_post_norm(nv.ptr(x), nv.ptr(y), nv.ptr(w), nv.ptr(bias), nv.ptr(sumsq), 0 if sumsq is None else sumsq.shape[1],
+                                   sumsq_n, nv.ptr(h), x.shape[0], x.shape[1], n, nv.ctypes.c_float(alpha), nv.ctypes.c_float(eps),
+                                   _f32(w), nv.stream_ptr()), "post_norm")
+    nv.count_launch()
+    return x if h is None else h
 
 
 def glu(gate: torch.Tensor, up: torch.Tensor, out: torch.Tensor) -> None:

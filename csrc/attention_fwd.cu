@@ -10,6 +10,7 @@
 // out [T, Hq*128], lse [Hq, T] (natural log, scaled scores).  T = B*S; sequence b owns rows b*S..b*S+S-1.
 #include "common.cuh"
 #include "host.h"
+#include "vec.cuh"
 
 namespace b2 {
 
@@ -17,8 +18,13 @@ constexpr int AT_THREADS = 352;  // warp 0 TMA, warps 1 and 10 MMA issue, warps 
 constexpr int AT_TILE_BYTES = 128 * 128 * 2;  // 32 KiB: two [128 x 64] swizzled halves
 constexpr int AT_HALF_BYTES = 128 * 64 * 2;
 
-// Options of the extended form (EXT): head sizes below 128 (the tensor maps zero-fill up to the tile), chunked visibility,
-// a learned additive bias per distance bucket, a softmax sink and an output gate per head.  Keys are always paged.
+// Options of the extended form (EXT): other head sizes (the tensor maps zero-fill up to the tile; keys up to 64 KH channels),
+// chunked visibility or a sliding window, a soft cap on the scores, a learned additive bias per distance bucket, a softmax sink
+// and an output gate per head; or differential heads.  Keys are always paged.
+//
+// Differential heads (maps = 2): an item is one head, done as two passes over the same keys' pages, map 1 and then map 2.  The
+// first pass leaves its normalised output in a scratch tile of this CTA (every thread reads back what it wrote itself, so the tile
+// stays in L2 and needs no synchronisation), the second subtracts, norms over the head's channels, gates and stores.
 struct FwdExt {
   const int* start;       // [B] position of each sequence's first query row: it sees start + q_len keys in all
   int chunk;              // > 0: a query at position i sees keys floor(i / chunk) * chunk .. i
@@ -29,21 +35,35 @@ struct FwdExt {
   const __nv_bfloat16* gate;  // [rows, ld_gate] (Hq columns) or null
   long long ld_gate, ld_out;
   int dkp, dvp;           // head sizes, multiples of 8
+  int window;             // > 0: a query at position i sees keys i - window + 1 .. i
+  float softcap;          // > 0: scores pass through softcap * tanh(score / softcap)
+  int maps;               // 2: differential heads; q has 2 Hq, K pages 2 Hkv rows a token; gate has Hq * dvp columns
+  const __nv_bfloat16* lam;   // [4, dkp]
+  float lam_init, eps;
+  int dv;                 // real value channels, for the differential norm
+  float* scratch;         // [grid, 256, 64] fp32
   int tpc;                // > 0: query tiles per chunk; items are then ordered by their place in the chunk, heaviest first
 };
 constexpr int EXT_TAB_NEG = 256;    // table entries below distance 0 (masked keys of a diagonal tile)
 constexpr int EXT_TAB_FAR = 256;    // entries past the last bucketed distance: no clamping inside a tile
 constexpr int EXT_MAX_BUCKETS = 7680;   // the table shares the write-out staging area (32 KiB)
 
-struct AttnFwdSmem {
+// KH: 64-channel pieces of a query / key row.  Three leave room for one Q tile and half of the write-out staging.
+template <int KH>
+struct AttnFwdSmemT {
   // offsets into the 1024-byte aligned dynamic shared memory
+  static constexpr int QSLOTS = KH == 3 ? 1 : 2;
+  static constexpr int KTILE = KH * AT_HALF_BYTES;
   static constexpr int Q = 0;                           // 2 tiles (this item's and the next item's)
-  static constexpr int K = Q + 2 * AT_TILE_BYTES;       // 2 stages
-  static constexpr int V = K + 2 * AT_TILE_BYTES;       // 2 stages
-  static constexpr int EPI = V + 2 * AT_TILE_BYTES;     // 8 warps x 4 KiB write-out staging
-  static constexpr int BARS = EPI + 8 * 4096;           // barriers (256 B), then the row exchange buffer (1 KiB)
-  static constexpr int TOTAL = BARS + 256 + 1024 + 1024;   // 231680
+  static constexpr int K = Q + QSLOTS * KTILE;          // 2 stages
+  static constexpr int V = K + 2 * KTILE;               // 2 stages
+  static constexpr int STAGE = KH == 3 ? 2048 : 4096;   // write-out staging of a warp
+  static constexpr int EPI = V + 2 * AT_TILE_BYTES;     // 8 warps
+  static constexpr int BARS = EPI + 8 * STAGE;          // barriers (256 B), then the row exchange buffer (1 KiB)
+  static constexpr int TOTAL = BARS + 256 + 1024 + 1024;   // 231680 in both forms
+  static_assert(TOTAL <= 232448, "shared memory of one CTA");
 };
+using AttnFwdSmem = AttnFwdSmemT<2>;
 
 // One work item: a 128-row query tile of one (batch, q head).
 struct FwdItem {
@@ -89,7 +109,8 @@ __device__ __forceinline__ FwdItem fwd_item(int w, const FwdParams& p, const Fwd
   const int last_key = min(it.kv_len, it.kv_off + (it.qt + 1) * 128);  // exclusive
   if (EXT) {   // k_begin: first key of tile 0 (page aligned), the chunk start of the tile's first query
     const int pos0 = it.kv_off + it.qt * 128;
-    it.k_begin = x_.chunk > 0 && it.active ? pos0 / x_.chunk * x_.chunk / 16 * 16 : 0;
+    it.k_begin = !it.active ? 0 : x_.chunk > 0 ? pos0 / x_.chunk * x_.chunk / 16 * 16
+                 : x_.window > 0 ? max(0, pos0 - x_.window + 1) / 16 * 16 : 0;
     it.n_kv = it.active ? (last_key - it.k_begin + 127) / 128 : 0;
   } else {
     it.n_kv = it.active ? (last_key + 127) / 128 : 0;
@@ -104,6 +125,12 @@ __device__ __forceinline__ int fwd_next_active(int w, int n_items, const FwdPara
   while (x < n_items && !fwd_item<EXT>(x, p, e).active) x = snake_next(x);
   return x;
 }
+// A step of the walk: an item, or one map of a differential head's item (map = step % 2).
+template <bool EXT>
+__device__ __forceinline__ int fwd_next_step(int u, int n_items, const FwdParams& p, const FwdExt& e) {
+  if (!EXT || e.maps == 1) return fwd_next_active<EXT>(u, n_items, p, e);
+  return u % 2 == 0 ? u + 1 : 2 * fwd_next_active<EXT>(u / 2, n_items, p, e);
+}
 
 // Persistent: each CTA walks its share of the items (heaviest tiles first, dealt in boustrophedon order).
 // Barriers, TMEM and the K/V ring live across items; the next item's Q is requested as soon as the last
@@ -116,15 +143,17 @@ __device__ __forceinline__ int fwd_next_active(int w, int n_items, const FwdPara
 // double-buffered in TMEM (S 2 x 128 columns, O 128, P 2 x 64 = all 512), so the softmax of tile j+1 never
 // waits for P*V of tile j unless the running maximum grew enough to force a rescale of O.  Q is double-
 // buffered in shared memory: the next item's Q arrives while the current item is still being processed.
-template <bool EXT>
+template <bool EXT, int KH = 2>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
                 float* __restrict__ lse_out, const FwdParams prm, const FwdExt ext, float scale, int* status) {
+  using Smem = AttnFwdSmemT<KH>;
+  constexpr int QS = Smem::QSLOTS;          // Q slots
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + AttnFwdSmem::BARS);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Smem::BARS);
   uint64_t* q_full = bars + 0;    // [2] with q_empty at bars + 17
   uint64_t* k_full = bars + 1;    // [2]
   uint64_t* v_full = bars + 3;    // [2]
@@ -138,16 +167,20 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   uint64_t* o_free = bars + 19;
   uint64_t* q_full2 = bars + 20;  // second Q slot's full barrier
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 21);
-  float* xchg = reinterpret_cast<float*>(smem + AttnFwdSmem::BARS + 256);   // [2 column halves][128 rows]
+  float* xchg = reinterpret_cast<float*>(smem + Smem::BARS + 256);   // [2 column halves][128 rows]
   uint64_t* tab_bar = bars + 22;   // EXT: all softmax warps, around every change of what the staging area holds
-  float* tab = reinterpret_cast<float*>(smem + AttnFwdSmem::EPI) + EXT_TAB_NEG;   // EXT: bias by distance
+  float* tab = reinterpret_cast<float*>(smem + Smem::EPI) + EXT_TAB_NEG;   // EXT: bias by distance
   // EXT: how many 16-channel steps and 64-channel halves the head sizes need
   const int k_steps = EXT ? (ext.dkp + 15) / 16 : 8;
   const bool k_half2 = !EXT || ext.dkp > 64, v_half2 = !EXT || ext.dvp > 64;
+  const bool k_half3 = KH == 3 && ext.dkp > 128;
+  const uint32_t k_bytes = (k_half3 ? 3 : k_half2 ? 2 : 1) * AT_HALF_BYTES;
+  const int maps = EXT ? ext.maps : 1;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int Hq = prm.Hq;
   const int n_items = prm.max_tiles * prm.Hq * prm.B;
+  const int n_steps = n_items * maps;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -185,21 +218,25 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 
   int w0 = blockIdx.x;
   if (w0 < n_items && !fwd_item<EXT>(w0, prm, ext).active) w0 = fwd_next_active<EXT>(w0, n_items, prm, ext);
+  w0 *= maps;
 
   if (warp == 0) {
     if (lane == 0) {
       int g = 0, n = 0;
       bool ok = true;
-      for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
-        const FwdItem item = fwd_item<EXT>(w, prm, ext);
+      for (int w = w0; w < n_steps && ok; w = fwd_next_step<EXT>(w, n_items, prm, ext), ++n) {
+        const FwdItem item = fwd_item<EXT>(EXT ? w / maps : w, prm, ext);
         // Q slot n & 1: free once the last Q*K^T of item n-2 has retired, i.e. long before item n starts
-        uint64_t* qf = (n & 1) ? q_full2 : q_full;
-        uint8_t* sQ = smem + AttnFwdSmem::Q + (n & 1) * AT_TILE_BYTES;
-        if (!mbar_wait(&q_empty[n & 1], ((n >> 1) & 1) ^ 1, status, ERR_ATTN_WAIT)) break;
+        const int qslot = n % QS;
+        uint64_t* qf = qslot ? q_full2 : q_full;
+        uint8_t* sQ = smem + Smem::Q + qslot * Smem::KTILE;
+        const int qrow = item.head * maps + w % maps, krow_ = item.kvh * maps + w % maps;   // EXT: head rows of this step
+        if (!mbar_wait(&q_empty[qslot], ((n / QS) & 1) ^ 1, status, ERR_ATTN_WAIT)) break;
         if (EXT) {
-          mbar_expect_tx(qf, k_half2 ? AT_TILE_BYTES : AT_HALF_BYTES);
-          tma_load_3d(sQ, &tmQ, qf, 0, item.head, item.row0);
-          if (k_half2) tma_load_3d(sQ + AT_HALF_BYTES, &tmQ, qf, 64, item.head, item.row0);
+          mbar_expect_tx(qf, k_bytes);
+          tma_load_3d(sQ, &tmQ, qf, 0, qrow, item.row0);
+          if (k_half2) tma_load_3d(sQ + AT_HALF_BYTES, &tmQ, qf, 64, qrow, item.row0);
+          if (k_half3) tma_load_3d(sQ + 2 * AT_HALF_BYTES, &tmQ, qf, 128, qrow, item.row0);
         } else {
           mbar_expect_tx(qf, AT_TILE_BYTES);
           tma_load_2d(sQ, &tmQ, qf, item.head * 128, item.row0);
@@ -210,8 +247,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           const uint32_t ph = (g >> 1) & 1;
           const int krow = item.k_begin + j * 128;
           if (!mbar_wait(&k_empty[st], ph ^ 1, status, ERR_ATTN_WAIT)) { ok = false; break; }
-          uint8_t* sK = smem + AttnFwdSmem::K + st * AT_TILE_BYTES;
-          uint8_t* sV = smem + AttnFwdSmem::V + st * AT_TILE_BYTES;
+          uint8_t* sK = smem + Smem::K + st * Smem::KTILE;
+          uint8_t* sV = smem + Smem::V + st * AT_TILE_BYTES;
           if (prm.block_tables != nullptr) {
             // a 128-key tile is eight 16-token pages: each lands as a [16 x 64] box at its row offset of the
             // swizzled tile (16 rows x 128 B = 2 KiB, a whole number of swizzle atoms).  Pages past the end of the
@@ -222,11 +259,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
             for (int pg = 0; pg < 8; ++pg) rows[pg] = tbl[min((EXT ? item.k_begin / 16 : 0) + j * 8 + pg, last_page)] * 16;
             if (EXT) {
-              mbar_expect_tx(&k_full[st], k_half2 ? AT_TILE_BYTES : AT_HALF_BYTES);
+              mbar_expect_tx(&k_full[st], k_bytes);
 #pragma unroll
               for (int pg = 0; pg < 8; ++pg) {
-                tma_load_3d(sK + pg * 2048, &tmK, &k_full[st], 0, item.kvh, rows[pg]);
-                if (k_half2) tma_load_3d(sK + AT_HALF_BYTES + pg * 2048, &tmK, &k_full[st], 64, item.kvh, rows[pg]);
+                tma_load_3d(sK + pg * 2048, &tmK, &k_full[st], 0, krow_, rows[pg]);
+                if (k_half2) tma_load_3d(sK + AT_HALF_BYTES + pg * 2048, &tmK, &k_full[st], 64, krow_, rows[pg]);
+                if (k_half3) tma_load_3d(sK + 2 * AT_HALF_BYTES + pg * 2048, &tmK, &k_full[st], 128, krow_, rows[pg]);
               }
               if (!mbar_wait(&v_empty[st], ph ^ 1, status, ERR_ATTN_WAIT)) { ok = false; break; }
               mbar_expect_tx(&v_full[st], v_half2 ? AT_TILE_BYTES : AT_HALF_BYTES);
@@ -268,10 +306,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     constexpr uint32_t idesc_s = make_idesc_f16(1, 128, 128, 0, 0);
     int g = 0, n = 0;
     bool ok = true;
-    for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
-      const FwdItem item = fwd_item<EXT>(w, prm, ext);
-      if (!mbar_wait((n & 1) ? q_full2 : q_full, (n >> 1) & 1, status, ERR_ATTN_WAIT)) break;
-      const uint64_t d_q = make_smem_desc_sw128(smem_u32(smem + AttnFwdSmem::Q + (n & 1) * AT_TILE_BYTES), 16, 1024);
+    for (int w = w0; w < n_steps && ok; w = fwd_next_step<EXT>(w, n_items, prm, ext), ++n) {
+      const FwdItem item = fwd_item<EXT>(EXT ? w / maps : w, prm, ext);
+      if (!mbar_wait(n % QS ? q_full2 : q_full, (n / QS) & 1, status, ERR_ATTN_WAIT)) break;
+      const uint64_t d_q = make_smem_desc_sw128(smem_u32(smem + Smem::Q + (n % QS) * Smem::KTILE), 16, 1024);
       for (int j = 0; j < item.n_kv; ++j, ++g) {
         const int st = g & 1;
         if (!mbar_wait(&k_full[st], (g >> 1) & 1, status, ERR_ATTN_WAIT) ||
@@ -280,17 +318,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           break;
         }
         tc_fence_after();
-        const uint64_t d_k = make_smem_desc_sw128(smem_u32(smem + AttnFwdSmem::K + st * AT_TILE_BYTES), 16, 1024);
+        const uint64_t d_k = make_smem_desc_sw128(smem_u32(smem + Smem::K + st * Smem::KTILE), 16, 1024);
         if (leader) {
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks) {
+          for (int ks = 0; ks < 4 * KH; ++ks) {
             if (EXT && ks >= k_steps) break;
             const uint32_t o = (ks >> 2) * AT_HALF_BYTES + (ks & 3) * 32;
             umma_f16_ss(tmem_S + st * 128, desc_advance(d_q, o), desc_advance(d_k, o), idesc_s, ks != 0);
           }
           umma_commit(&k_empty[st]);
           umma_commit(&s_full[st]);
-          if (j + 1 == item.n_kv) umma_commit(&q_empty[n & 1]);   // last Q*K^T of the item: its Q slot is free
+          if (j + 1 == item.n_kv) umma_commit(&q_empty[n % QS]);   // last Q*K^T of the item: its Q slot is free
         }
       }
     }
@@ -300,8 +338,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const uint32_t idesc_pv = v_half2 ? make_idesc_f16(1, 128, 128, 0, 1) : make_idesc_f16(1, 128, 64, 0, 1);
     int g = 0, n = 0;
     bool ok = true;
-    for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
-      const FwdItem item = fwd_item<EXT>(w, prm, ext);
+    for (int w = w0; w < n_steps && ok; w = fwd_next_step<EXT>(w, n_items, prm, ext), ++n) {
+      const FwdItem item = fwd_item<EXT>(EXT ? w / maps : w, prm, ext);
       // the softmax warps must have read the previous item's O before it is overwritten
       if (n > 0 && !mbar_wait(o_free, (n - 1) & 1, status, ERR_ATTN_WAIT)) break;
       for (int j = 0; j < item.n_kv; ++j, ++g) {
@@ -312,7 +350,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           break;
         }
         tc_fence_after();
-        const uint64_t d_v = make_smem_desc_sw128(smem_u32(smem + AttnFwdSmem::V + st * AT_TILE_BYTES),
+        const uint64_t d_v = make_smem_desc_sw128(smem_u32(smem + Smem::V + st * AT_TILE_BYTES),
                                                   AT_HALF_BYTES, 1024);
         const uint32_t acc0 = j != 0;
         if (leader) {
@@ -349,18 +387,21 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       tab_phase ^= 1;
       return done;
     };
+    const float lam = EXT && maps == 2 ? diff_lambda(ext.lam, ext.dkp, ext.lam_init) : 0.f;
+    const float cap_inv = EXT && ext.softcap > 0.f ? scale / ext.softcap : 0.f;      // raw score -> score / cap
+    const float cap2 = EXT ? ext.softcap * 1.4426950408889634f : 0.f;
     bool ok = true;
     int g = 0, n = 0;
-    for (int w = w0; w < n_items && ok; w = fwd_next_active<EXT>(w, n_items, prm, ext), ++n) {
-      const FwdItem item = fwd_item<EXT>(w, prm, ext);
+    for (int w = w0; w < n_steps && ok; w = fwd_next_step<EXT>(w, n_items, prm, ext), ++n) {
+      const FwdItem item = fwd_item<EXT>(EXT ? w / maps : w, prm, ext);
       const int q_idx = item.qt * 128 + r;      // index among this sequence's queries
       const int q_pos = item.kv_off + q_idx;    // last key this query may see
       float m_used = EXT ? -1e30f : -INFINITY, l = 0.f;        // l: this thread's 64 columns only
       // requested now, used at the end of the item
-      const float gate_raw = EXT && ext.gate != nullptr && q_idx < item.q_len
+      const float gate_raw = EXT && maps == 1 && ext.gate != nullptr && q_idx < item.q_len
                                  ? __bfloat162float(ext.gate[static_cast<size_t>(item.row0 + r) * ext.ld_gate + item.head]) : 0.f;
       const float sink2 = EXT && ext.sink != nullptr ? __bfloat162float(ext.sink[item.head]) * 1.4426950408889634f : 0.f;
-      const int first_key = EXT && ext.chunk > 0 ? q_pos / ext.chunk * ext.chunk : 0;
+      const int first_key = !EXT ? 0 : ext.chunk > 0 ? q_pos / ext.chunk * ext.chunk : ext.window > 0 ? q_pos - ext.window + 1 : 0;
       if (EXT && ext.rel != nullptr) {
         // this head's bias by distance, constant past the last bucketed one
         // every warp has written its part of the previous item out
@@ -402,12 +443,27 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
               for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], sl2_raw, tp[-i]);
             }
+          } else if (ext.softcap > 0.f) {
+            float big = 0.f;
+#pragma unroll
+            for (int i = 0; i < 64; ++i) {
+              s[i] *= cap_inv;
+              big = fmaxf(big, fabsf(s[i]));
+            }
+            if (__any_sync(0xffffffffu, big > SOFTCAP_SERIES)) {
+#pragma unroll
+              for (int i = 0; i < 64; ++i) s[i] = cap2 * tanh_wide(s[i]);
+            } else {
+#pragma unroll
+              for (int i = 0; i < 64; ++i) s[i] = cap2 * tanh_series(s[i]);
+            }
           } else {
 #pragma unroll
             for (int i = 0; i < 64; ++i) s[i] *= sl2_raw;
           }
           const bool edge = item.k_begin + (j + 1) * 128 > pos_lo + 1 || item.k_begin + (j + 1) * 128 > item.kv_len ||
-                            (ext.chunk > 0 && item.k_begin + j * 128 < (pos_lo + 127) / ext.chunk * ext.chunk);
+                            (ext.chunk > 0 && item.k_begin + j * 128 < (pos_lo + 127) / ext.chunk * ext.chunk) ||
+                            (ext.window > 0 && item.k_begin + j * 128 < pos_lo + 128 - ext.window);
           if (edge) {
 #pragma unroll
             for (int i = 0; i < 64; ++i)
@@ -496,13 +552,67 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (EXT) {
         float den = lsum;
         if (ext.sink != nullptr) den += fast_exp2(sink2 - m_used);
-        if (ext.gate != nullptr) den *= 1.f + fast_exp2(-1.4426950408889634f * gate_raw);
+        if (maps == 1 && ext.gate != nullptr) den *= 1.f + fast_exp2(-1.4426950408889634f * gate_raw);
         inv = __fdividef(1.f, den);
       }
       const bool in_range = q_idx < item.q_len;
       uint4 ov[8];
+      if (EXT && maps == 2) {
+        float o[64];
+        const bool mine = half * 64 < ext.dvp;       // this thread has channels of the head
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          uint32_t t[32];
+          tmem_ld_32x32b_x32(tmem_O + lane_off + half * 64 + c * 32, t);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) o[c * 32 + i] = mine ? __uint_as_float(t[i]) * inv : 0.f;
+        }
+        tc_fence_before();
+        mbar_arrive_warp(o_free);
+        float4* tile = reinterpret_cast<float4*>(ext.scratch) + static_cast<size_t>(blockIdx.x) * 4096 + (threadIdx.x - 64);
+        if (w % 2 == 0) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) tile[i * 256] = make_float4(o[4 * i], o[4 * i + 1], o[4 * i + 2], o[4 * i + 3]);
+          continue;
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float4 a1 = tile[i * 256];
+          o[4 * i] = a1.x - lam * o[4 * i];
+          o[4 * i + 1] = a1.y - lam * o[4 * i + 1];
+          o[4 * i + 2] = a1.z - lam * o[4 * i + 2];
+          o[4 * i + 3] = a1.w - lam * o[4 * i + 3];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) ss = fmaf(o[4 * i + e], o[4 * i + e], ss);
+        }
+        xchg[half * 128 + r] = ss;
+        pair_barrier();
+        const float norm = (1.f - ext.lam_init) / sqrtf((xchg[r] + xchg[128 + r]) / ext.dv + ext.eps);
+        pair_barrier();
+        const __nv_bfloat16* gp = ext.gate == nullptr ? nullptr
+            : ext.gate + static_cast<size_t>(item.row0 + r) * ext.ld_gate + static_cast<size_t>(item.head) * ext.dvp + half * 64;
+#pragma unroll
+        for (int v = 0; v < 8; ++v) {
+          float f[8];
+          if (gp != nullptr && in_range && half * 64 + v * 8 < ext.dvp) {
+            vload8(gp + v * 8, f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = sigmoid_fast(f[e]) * norm;
+          } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = norm;
+          }
+          ov[v].x = pack_bf16x2(o[v * 8 + 0] * f[0], o[v * 8 + 1] * f[1]);
+          ov[v].y = pack_bf16x2(o[v * 8 + 2] * f[2], o[v * 8 + 3] * f[3]);
+          ov[v].z = pack_bf16x2(o[v * 8 + 4] * f[4], o[v * 8 + 5] * f[5]);
+          ov[v].w = pack_bf16x2(o[v * 8 + 6] * f[6], o[v * 8 + 7] * f[7]);
+        }
+      }
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
+        if (EXT && maps == 2) break;
         uint32_t t[32];
         tmem_ld_32x32b_x32(tmem_O + lane_off + half * 64 + c * 32, t);
         tmem_ld_wait();
@@ -523,7 +633,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         const int wq0 = item.qt * 128 + quarter * 32;
         __nv_bfloat16* base = out + static_cast<size_t>(item.row0 + quarter * 32) * ext.ld_out +
                               static_cast<size_t>(item.head) * ext.dvp + half * 64;
-        warp_store_rows_128B(smem + AttnFwdSmem::EPI + (warp - 2) * 4096, ov, [&](int row) -> uint8_t* {
+        warp_store_rows_128B<Smem::STAGE / 128>(smem + Smem::EPI + (warp - 2) * Smem::STAGE, ov, [&](int row) -> uint8_t* {
           // the lane's 16-byte piece of the row: skipped past the head's last channel
           if (wq0 + row >= item.q_len || half * 64 + (lane & 7) * 8 >= ext.dvp) return nullptr;
           return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * ext.ld_out);
@@ -531,7 +641,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       } else {
         const int wq0 = item.qt * 128 + quarter * 32;   // index (within the sequence) of this warp's first query row
         __nv_bfloat16* base = out + (static_cast<size_t>(item.row0 + quarter * 32) * Hq + item.head) * 128 + half * 64;
-        warp_store_rows_128B(smem + AttnFwdSmem::EPI + (warp - 2) * 4096, ov, [&](int row) -> uint8_t* {
+        warp_store_rows_128B(smem + Smem::EPI + (warp - 2) * 4096, ov, [&](int row) -> uint8_t* {
           if (wq0 + row >= item.q_len) return nullptr;
           return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * Hq * 128);
         });
@@ -552,6 +662,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     tc_fence_after();
     tmem_dealloc(tmem_base, 512);
   }
+}
+
+static FwdExt no_ext() {
+  FwdExt e = {};
+  e.maps = 1;
+  return e;
 }
 
 }  // namespace b2
@@ -607,7 +723,7 @@ B2_EXPORT int b2_attn_fwd_varlen(const void* q, const void* k, const void* v, vo
   const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
   const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
   attn_fwd_kernel<false><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(
-      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, FwdExt{}, scale, status);
+      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, no_ext(), scale, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_error("attn_fwd launch failed: %s", cudaGetErrorString(e));
@@ -656,7 +772,7 @@ B2_EXPORT int b2_attn_fwd_paged(const void* q, const void* k_cache, const void* 
   const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
   const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
   attn_fwd_kernel<false><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(
-      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, FwdExt{}, scale, status);
+      *tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), lse, prm, no_ext(), scale, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_error("attn_fwd_paged launch failed: %s", cudaGetErrorString(e));
@@ -666,29 +782,35 @@ B2_EXPORT int b2_attn_fwd_paged(const void* q, const void* k_cache, const void* 
 }
 
 // The extended form over the paged cache (see FwdExt): q [total_q, Hq * dkp], K pages [blocks, 16, Hkv, dkp], V pages
-// [blocks, 16, Hkv, dvp], out rows of stride ld_out.  cu_q: int32 [B+1] row offsets; start: int32 [B].
+// [blocks, 16, Hkv, dvp], out rows of stride ld_out, q rows of stride ld_q.  maps = 2: see FwdExt; scratch: fp32 [number of
+// SMs, 256, 64].  cu_q: int32 [B+1] row offsets; start: int32 [B].
 B2_EXPORT int b2_attn_fwd_paged_ext(const void* q, const void* k_cache, const void* v_cache, void* out, long long ld_out, int B,
                                     int Hq, int Hkv, int dkp, int dvp, int num_blocks, float scale, const int* cu_q,
                                     const int* start, const int* block_tables, int max_blocks, int max_q, int total_q,
                                     int chunk, const void* rel, const int* bucket, int nbucket, const void* sink,
-                                    const void* gate, long long ld_gate, void* stream_) {
+                                    const void* gate, long long ld_gate, long long ld_q, int window, float softcap, int maps,
+                                    const void* lam, float lam_init, float eps, int dv, float* scratch, void* stream_) {
   b2::ensure_thread_context();
-  if (dkp < 8 || dkp > 128 || dkp % 8 || dvp < 8 || dvp > 128 || dvp % 8 || Hq < 1 || Hkv < 1 || Hq % Hkv || ld_out % 8 ||
+  if (dkp < 8 || dkp > 192 || dkp % 8 || dvp < 8 || dvp > 128 || dvp % 8 || Hq < 1 || Hkv < 1 || Hq % Hkv || ld_out % 8 ||
       block_tables == nullptr || cu_q == nullptr || start == nullptr || max_blocks <= 0 ||
-      (rel != nullptr && (bucket == nullptr || nbucket < 1 || nbucket > EXT_MAX_BUCKETS))) {
-    set_error("attn_fwd_paged_ext: head sizes up to 128 in multiples of 8, Hq %% Hkv == 0, at most %d bucketed distances", EXT_MAX_BUCKETS);
+      (rel != nullptr && (bucket == nullptr || nbucket < 1 || nbucket > EXT_MAX_BUCKETS || dkp > 128 || softcap > 0.f)) ||
+      ld_q % 8 || (maps != 1 && maps != 2) ||
+      (maps == 2 && (dkp > 128 || lam == nullptr || scratch == nullptr || rel != nullptr || sink != nullptr || dv < 1 || dv > dvp ||
+                     (gate != nullptr && ld_gate % 8)))) {
+    set_error("attn_fwd_paged_ext: head sizes up to 128 (keys without a bias table: 192) in multiples of 8, Hq %% Hkv == 0, at most %d bucketed distances", EXT_MAX_BUCKETS);
     return 10;
   }
   if (B <= 0 || max_q <= 0 || total_q <= 0) return 0;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  auto map3 = [](const void* base, uint64_t rows, uint64_t heads, uint64_t d, uint32_t box_rows) {
-    const uint64_t dims[3] = {d, heads, rows}, strides[2] = {d * 2, heads * d * 2};
+  auto map3 = [](const void* base, uint64_t rows, uint64_t heads, uint64_t d, uint64_t ld, uint32_t box_rows) {
+    const uint64_t dims[3] = {d, heads, rows}, strides[2] = {d * 2, ld * 2};
     const uint32_t box[3] = {64, 1, box_rows};
     return tensor_map_nd_bf16(base, 3, dims, strides, box, 3);
   };
-  const CUtensorMap* tq = map3(q, total_q, Hq, dkp, 128);
-  const CUtensorMap* tk = map3(k_cache, static_cast<uint64_t>(num_blocks) * 16, Hkv, dkp, 16);
-  const CUtensorMap* tv = map3(v_cache, static_cast<uint64_t>(num_blocks) * 16, Hkv, dvp, 16);
+  const CUtensorMap* tq = map3(q, total_q, static_cast<uint64_t>(Hq) * maps, dkp, ld_q, 128);
+  const CUtensorMap* tk = map3(k_cache, static_cast<uint64_t>(num_blocks) * 16, static_cast<uint64_t>(Hkv) * maps, dkp,
+                               static_cast<uint64_t>(Hkv) * maps * dkp, 16);
+  const CUtensorMap* tv = map3(v_cache, static_cast<uint64_t>(num_blocks) * 16, Hkv, dvp, static_cast<uint64_t>(Hkv) * dvp, 16);
   if (!tq || !tk || !tv) return 2;
   int* status = status_ptr();
   if (!status) return 3;
@@ -696,8 +818,10 @@ B2_EXPORT int b2_attn_fwd_paged_ext(const void* q, const void* k_cache, const vo
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev]) {
-    if (cudaFuncSetAttribute(attn_fwd_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnFwdSmem::TOTAL) !=
-        cudaSuccess) {
+    if (cudaFuncSetAttribute(attn_fwd_kernel<true, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnFwdSmemT<2>::TOTAL) !=
+            cudaSuccess ||
+        cudaFuncSetAttribute(attn_fwd_kernel<true, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnFwdSmemT<3>::TOTAL) !=
+            cudaSuccess) {
       set_error("attn_fwd_paged_ext: cannot set shared memory size");
       return 1;
     }
@@ -710,12 +834,17 @@ B2_EXPORT int b2_attn_fwd_paged_ext(const void* q, const void* k_cache, const vo
   e.start = start; e.chunk = chunk; e.rel = static_cast<const __nv_bfloat16*>(rel); e.bucket = bucket; e.nbucket = nbucket;
   e.sink = static_cast<const __nv_bfloat16*>(sink); e.gate = static_cast<const __nv_bfloat16*>(gate); e.ld_gate = ld_gate;
   e.ld_out = ld_out; e.dkp = dkp; e.dvp = dvp;
+  e.window = chunk > 0 ? 0 : window; e.softcap = softcap; e.maps = maps; e.lam = static_cast<const __nv_bfloat16*>(lam);
+  e.lam_init = lam_init; e.eps = eps; e.dv = dv; e.scratch = scratch;
   e.tpc = chunk >= 256 && chunk < max_q ? (chunk + 127) / 128 : 0;
   if (e.tpc > 0) prm.max_tiles = (prm.max_tiles + e.tpc - 1) / e.tpc * e.tpc;
   const long long n_items = static_cast<long long>(prm.max_tiles) * Hq * B;
   const int grid = n_items < num_sms() ? static_cast<int>(n_items) : num_sms();
-  attn_fwd_kernel<true><<<grid, AT_THREADS, AttnFwdSmem::TOTAL, stream>>>(*tq, *tk, *tv, static_cast<__nv_bfloat16*>(out), nullptr, prm, e,
-                                                            scale, status);
+  __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
+  if (dkp > 128)
+    attn_fwd_kernel<true, 3><<<grid, AT_THREADS, AttnFwdSmemT<3>::TOTAL, stream>>>(*tq, *tk, *tv, o, nullptr, prm, e, scale, status);
+  else
+    attn_fwd_kernel<true, 2><<<grid, AT_THREADS, AttnFwdSmemT<2>::TOTAL, stream>>>(*tq, *tk, *tv, o, nullptr, prm, e, scale, status);
   cudaError_t err = cudaGetLastError();
   if (err != cudaSuccess) {
     set_error("attn_fwd_paged_ext launch failed: %s", cudaGetErrorString(err));

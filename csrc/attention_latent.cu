@@ -1,0 +1,573 @@
+// Latent attention: what is cached of a token is one row for all heads, a normed latent c and a rotated key part
+//
+//   [ c (kv_rank, padded to Cp) | rotated part (padded) ]      pages [blocks, 16, Rp], Rp = Cp + padded rotated size
+//
+// from which a head's key is [W_uk c | rotated part] and its value W_uv c.  Two ways to attend, equal but for rounding:
+//   expanded   keys and values of all heads are made from the rows (a GEMM) and attended like ordinary ones: long portions, where
+//              a row serves many queries (latent_gather brings the pages into token order for that GEMM)
+//   absorbed   q_h^T W_uk c = (W_uk^T q_h)^T c, so the query moves into the latent space, every head attends over the same rows,
+//              and W_uv is applied to the result: decoding and short portions (latent_rows, between two products per head,
+//              head_linear)
+// And the stage before either: norm of the latent, rotary positions of the queries' and the key's rotated part, page store.
+#include "host.h"
+#include "mma_split.cuh"
+#include "vec.cuh"
+
+namespace b2 {
+
+constexpr int LA_PAGE = 16;
+constexpr float LA_LOG2E = 1.4426950408889634f;
+typedef __nv_bfloat16 la_bf16;
+
+__device__ __forceinline__ void la_copy16(void* dst, const void* src, bool in) {
+  const int n = in ? 16 : 0;   // zero-filled otherwise
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void la_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void la_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+
+// ---- input stage -----------------------------------------------------------------------------------------------------------
+// One row per CTA.  q [M, H * dqp] is rotated in place: channels dim .. dim + rot - 1 of every head, pairs (2 i, 2 i + 1).
+constexpr int LS_THREADS = 128;
+template <typename T>
+__global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(T* __restrict__ q, const T* __restrict__ c, const T* __restrict__ kr,
+                                                                  long long ld, T* __restrict__ pages, const T* __restrict__ w,
+                                                                  const int* __restrict__ tables, const int* __restrict__ row_seq,
+                                                                  const int* __restrict__ pos, const int* __restrict__ slot,
+                                                                  const float* __restrict__ cs, const float* __restrict__ sn,
+                                                                  int max_blocks, int H, int dim, int dqp, int rank, int Cp, int Rp,
+                                                                  int rot, float eps) {
+  __shared__ float red[LS_THREADS / 32];
+  const size_t row = blockIdx.x;
+  const int s = row_seq ? row_seq[row] : static_cast<int>(row), tid = threadIdx.x, half = rot / 2;
+  const float* cr = cs + row * half;
+  const float* sr = sn + row * half;
+  T* qr = q + row * ld;
+  for (int i = tid; i < H * half; i += LS_THREADS) {
+    const int h = i / half, f = i % half;
+    T* at = qr + static_cast<size_t>(h) * dqp + dim + 2 * f;
+    const float u = to_f(at[0]), v = to_f(at[1]), co = cr[f], si = sr[f];
+    at[0] = from_f<T>(u * co - v * si);
+    at[1] = from_f<T>(v * co + u * si);
+  }
+  if (slot != nullptr && slot[s] < 0) return;
+  const int p = pos[row];
+  T* dst = pages + (static_cast<size_t>(tables[static_cast<size_t>(s) * max_blocks + p / LA_PAGE]) * LA_PAGE + p % LA_PAGE) * Rp;
+  const T* crow = c + row * ld;
+  float ss = 0.f;
+  for (int a = tid * 8; a < Cp; a += LS_THREADS * 8) {
+    float t[8];
+    vload8(crow + a, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  const float r = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / rank + eps);
+  for (int a = tid * 8; a < Cp; a += LS_THREADS * 8) {
+    float t[8], g[8];
+    vload8(crow + a, t);
+    vload8(w + a, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) t[e] *= r * g[e];
+    vstore8(dst + a, t);
+  }
+  const T* krow = kr + row * ld;
+  for (int f = LS_THREADS - 1 - tid; f < (Rp - Cp) / 2; f += LS_THREADS) {
+    float u = to_f(krow[2 * f]), v = to_f(krow[2 * f + 1]);
+    if (f < half) {
+      const float x = u * cr[f] - v * sr[f];
+      v = v * cr[f] + u * sr[f];
+      u = x;
+    }
+    dst[Cp + 2 * f] = from_f<T>(u);
+    dst[Cp + 2 * f + 1] = from_f<T>(v);
+  }
+}
+
+// out page i <- page ids[i], `bytes` a page
+__global__ void __launch_bounds__(128) latent_gather_kernel(const uint8_t* __restrict__ pages, const int* __restrict__ ids,
+                                                            uint8_t* __restrict__ out, int bytes) {
+  const uint8_t* src = pages + static_cast<size_t>(ids[blockIdx.x]) * bytes;
+  uint8_t* dst = out + static_cast<size_t>(blockIdx.x) * bytes;
+  for (int i = threadIdx.x * 16; i < bytes; i += 128 * 16)
+    *reinterpret_cast<uint4*>(dst + i) = *reinterpret_cast<const uint4*>(src + i);
+}
+
+// ---- one small product per head ----------------------------------------------------------------------------------------------
+// out[m, h, :] = W_h x[m, h, :] with W_h [N, K] (KN: W_h stored [K, N]); x rows of stride ld_x with heads xs apart, out likewise.
+struct HeadLinearParams {
+  const void* x;
+  const void* w;
+  void* out;
+  long long ld_x, ld_out;
+  int M, H, N, K, xs, os;
+};
+
+template <bool KN>
+__global__ void __launch_bounds__(256) head_linear_any_kernel(const HeadLinearParams p) {
+  const int n = blockIdx.x * 256 + threadIdx.x, h = blockIdx.y;
+  const float* w = static_cast<const float*>(p.w) + static_cast<size_t>(h) * p.N * p.K;
+  if (n >= p.N) return;
+  for (int m = blockIdx.z; m < p.M; m += gridDim.z) {
+    const float* x = static_cast<const float*>(p.x) + m * p.ld_x + static_cast<size_t>(h) * p.xs;
+    float s = 0.f;
+    for (int k = 0; k < p.K; ++k) s = fmaf(x[k], KN ? w[static_cast<size_t>(k) * p.N + n] : w[static_cast<size_t>(n) * p.K + k], s);
+    static_cast<float*>(p.out)[m * p.ld_out + static_cast<size_t>(h) * p.os + n] = s;
+  }
+}
+
+// bf16: a 64 x 64 output tile of one head per CTA, four warps of 16 rows, K in pieces of 64 through two stages.
+constexpr int HL_T = 64, HL_LD = HL_T + 8;
+template <bool KN>
+__global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearParams p) {
+  __shared__ __align__(16) la_bf16 sA[2][HL_T][HL_LD], sB[2][HL_T][HL_LD];
+  const int n0 = blockIdx.x * HL_T, h = blockIdx.y, m0 = blockIdx.z * HL_T;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const la_bf16* x = static_cast<const la_bf16*>(p.x) + static_cast<size_t>(h) * p.xs;
+  const la_bf16* w = static_cast<const la_bf16*>(p.w) + static_cast<size_t>(h) * p.N * p.K;
+  auto issue = [&](int st, int k0) {
+    for (int i = tid; i < HL_T * (HL_T / 8); i += 128) {
+      const int r = i / 8, c = i % 8 * 8;
+      const bool ia = m0 + r < p.M && k0 + c < p.K;
+      la_copy16(&sA[st][r][c], x + (ia ? (m0 + r) * p.ld_x + k0 + c : 0), ia);
+      const int n = KN ? n0 + c : n0 + r, k = KN ? k0 + r : k0 + c;
+      const bool ib = n < p.N && k < p.K;
+      la_copy16(&sB[st][r][c], w + (ib ? (KN ? static_cast<size_t>(k) * p.N + n : static_cast<size_t>(n) * p.K + k) : 0), ib);
+    }
+    la_commit();
+  };
+  float acc[HL_T / 8][4] = {};
+  issue(0, 0);
+  int st = 0;
+  for (int k0 = 0; k0 < p.K; k0 += HL_T, st ^= 1) {
+    if (k0 + HL_T < p.K) {
+      issue(st ^ 1, k0 + HL_T);
+      la_wait<1>();
+    } else {
+      la_wait<0>();
+    }
+    __syncthreads();
+#pragma unroll
+    for (int ks = 0; ks < HL_T / 16; ++ks) {
+      uint32_t a[4];
+      ldsm_a_mk(&sA[st][warp * 16][ks * 16], HL_LD, lane, a);
+#pragma unroll
+      for (int n = 0; n < HL_T; n += 16) {
+        uint32_t b[4];
+        if (KN) ldsm_b_kn(&sB[st][ks * 16][n], HL_LD, lane, b);
+        else ldsm_b_nk(&sB[st][n][ks * 16], HL_LD, lane, b);
+        mma_n16(acc[n / 8], acc[n / 8 + 1], a, b);
+      }
+    }
+    __syncthreads();
+  }
+  la_bf16* out = static_cast<la_bf16*>(p.out) + static_cast<size_t>(h) * p.os;
+#pragma unroll
+  for (int n = 0; n < HL_T / 8; ++n)
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int m = m0 + warp * 16 + (lane >> 2) + 8 * hh, c = n0 + n * 8 + (lane & 3) * 2;
+      if (m < p.M && c < p.N)
+        *reinterpret_cast<uint32_t*>(out + m * p.ld_out + c) = pack_bf16x2(acc[n][2 * hh], acc[n][2 * hh + 1]);
+    }
+}
+
+// ---- absorbed attention ------------------------------------------------------------------------------------------------------
+struct LatentRowsParams {
+  const void* q;         // T [M, H * Rp]
+  const void* pages;     // T [blocks, 16, Rp]
+  const int* tables;
+  const int* row_seq;    // [M] or null: row r is sequence r
+  const int* pos;
+  const int* slot;       // slot < 0: padding row (output zero)
+  const void* sink;      // T [H] or null
+  void* out;             // T [M, H * Cp]
+  float* part_o;         // [M, H, nsplit, Cp]
+  float* part_ml;        // [M, H, nsplit, 2]
+  int max_blocks, H, Rp, Cp, partition, nsplit;
+  float scale;
+};
+
+template <typename T>
+__device__ __forceinline__ float la_sink(const LatentRowsParams& p, int head, float M2, float L) {
+  // factor on the weighted sum of values: 1 / (L + sink), M2 being the maximum in the base-2 domain
+  if (p.sink == nullptr) return L > 0.f ? 1.f / L : 0.f;
+  const float s2 = to_f(static_cast<const T*>(p.sink)[head]) * LA_LOG2E, m = fmaxf(M2, s2);
+  const float w = M2 == -INFINITY ? 0.f : exp2f(M2 - m);
+  return w / (L * w + exp2f(s2 - m));
+}
+
+// Any sizes, any type: one CTA per (row, head, split); a key per warp at a time, its channels over the lanes.
+constexpr int LR_ANY_WARPS = 4;
+template <typename T, int E>
+__global__ void __launch_bounds__(LR_ANY_WARPS * 32) latent_rows_any_kernel(const LatentRowsParams p) {
+  extern __shared__ __align__(16) float la_any[];     // q [32 E], then accumulators [warps][32 E]
+  __shared__ float sM[LR_ANY_WARPS], sL[LR_ANY_WARPS];
+  const size_t row = blockIdx.x;
+  const int head = blockIdx.y, split = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row);
+  const bool live = p.slot == nullptr || p.slot[s] >= 0;
+  const int t_begin = split * p.partition, t_end = live ? min(p.pos[row] + 1, t_begin + p.partition) : t_begin;
+  const int* table = p.tables + static_cast<size_t>(s) * p.max_blocks;
+  const T* q = static_cast<const T*>(p.q) + (row * p.H + head) * p.Rp;
+  float* sQ = la_any;
+  float* sAcc = la_any + 32 * E;
+  for (int c = threadIdx.x; c < 32 * E; c += LR_ANY_WARPS * 32) sQ[c] = c < p.Rp ? to_f(q[c]) * (p.scale * LA_LOG2E) : 0.f;
+  __syncthreads();
+  float acc[E], m = -INFINITY, l = 0.f;
+#pragma unroll
+  for (int e = 0; e < E; ++e) acc[e] = 0.f;
+  for (int t = t_begin + warp; t < t_end; t += LR_ANY_WARPS) {
+    const T* k = static_cast<const T*>(p.pages) + (static_cast<size_t>(table[t / LA_PAGE]) * LA_PAGE + t % LA_PAGE) * p.Rp;
+    float v[E], d = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int c = lane + 32 * e;
+      v[e] = c < p.Rp ? to_f(k[c]) : 0.f;
+      d = fmaf(v[e], sQ[c], d);
+    }
+    d = warp_sum(d);
+    const float mn = fmaxf(m, d), a = exp2f(m - mn), w = exp2f(d - mn);
+    m = mn;
+    l = l * a + w;
+#pragma unroll
+    for (int e = 0; e < E; ++e) acc[e] = acc[e] * a + w * v[e];
+  }
+#pragma unroll
+  for (int e = 0; e < E; ++e) sAcc[warp * 32 * E + lane + 32 * e] = acc[e];
+  if (lane == 0) {
+    sM[warp] = m;
+    sL[warp] = l;
+  }
+  __syncthreads();
+  float M = -INFINITY, L = 0.f;
+  for (int w = 0; w < LR_ANY_WARPS; ++w) M = fmaxf(M, sM[w]);
+  for (int w = 0; w < LR_ANY_WARPS; ++w) L += sM[w] == -INFINITY ? 0.f : sL[w] * exp2f(sM[w] - M);
+  const size_t at = (row * p.H + head) * p.nsplit + split;
+  const float f = p.nsplit == 1 ? la_sink<T>(p, head, M, L) : 1.f;
+  for (int c = threadIdx.x; c < p.Cp; c += LR_ANY_WARPS * 32) {
+    float o = 0.f;
+    for (int w = 0; w < LR_ANY_WARPS; ++w) o += sM[w] == -INFINITY ? 0.f : sAcc[w * 32 * E + c] * exp2f(sM[w] - M);
+    if (p.nsplit == 1) static_cast<T*>(p.out)[(row * p.H + head) * p.Cp + c] = from_f<T>(o * f);
+    else p.part_o[at * p.Cp + c] = o;
+  }
+  if (p.nsplit > 1 && threadIdx.x == 0) {
+    p.part_ml[at * 2] = M;
+    p.part_ml[at * 2 + 1] = L;
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentRowsParams p) {
+  const size_t row = blockIdx.x;
+  const int head = blockIdx.y;
+  const size_t at = (row * p.H + head) * p.nsplit;
+  float M = -INFINITY, L = 0.f;
+  for (int i = 0; i < p.nsplit; ++i) M = fmaxf(M, p.part_ml[(at + i) * 2]);
+  for (int i = 0; i < p.nsplit; ++i) {
+    const float mi = p.part_ml[(at + i) * 2];
+    L += mi == -INFINITY ? 0.f : p.part_ml[(at + i) * 2 + 1] * exp2f(mi - M);
+  }
+  const float f = la_sink<T>(p, head, M, L);
+  for (int c = threadIdx.x * 8; c < p.Cp; c += 128 * 8) {
+    float o[8] = {};
+    for (int i = 0; i < p.nsplit; ++i) {
+      const float mi = p.part_ml[(at + i) * 2];
+      if (mi == -INFINITY) continue;
+      const float w = exp2f(mi - M);
+      float t[8];
+      vload8(p.part_o + (at + i) * p.Cp + c, t);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = fmaf(t[e], w, o[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) o[e] *= f;
+    vstore8(static_cast<T*>(p.out) + (row * p.H + head) * p.Cp + c, o);
+  }
+}
+
+// bf16 on the tensor cores: one CTA per (row, 16 heads, split).  The sixteen heads are the rows of an m16n8k16 product (the
+// 128-row tcgen05 tile would be seven eighths padding), a tile of 64 keys its columns, and then the weights times the same tile,
+// whose first Cp channels are the values: every cached byte is read once for all heads.  Eight warps: four groups of 16 keys times
+// two halves of the channels for the scores, 16-channel pieces of the latent for the values.
+constexpr int LR_THREADS = 256, LR_KEYS = 64, LR_HEADS = 16, LR_LDP = LR_KEYS + 8, LR_LDS = LR_KEYS + 4;
+__host__ __device__ constexpr int lr_ld(int Rp) { return (Rp + 15) / 16 * 16 + 8; }
+static int lr_bytes(int Rp) {
+  return (LR_HEADS + 2 * LR_KEYS) * lr_ld(Rp) * 2 + 2 * LR_HEADS * LR_LDS * 4 + LR_HEADS * LR_LDP * 2 + 3 * LR_HEADS * 4;
+}
+
+template <int NG>    // 16-channel pieces of the latent per warp: Cp <= 128 NG
+__global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(const LatentRowsParams p) {
+  extern __shared__ __align__(16) uint8_t la_dyn[];
+  const int R16 = (p.Rp + 15) / 16 * 16, LD = R16 + 8, pieces = R16 / 8;
+  la_bf16* sQ = reinterpret_cast<la_bf16*>(la_dyn);            // [16][LD]
+  la_bf16* sC = sQ + LR_HEADS * LD;                            // [2][64][LD]
+  float* sS = reinterpret_cast<float*>(sC + 2 * LR_KEYS * LD); // [2 channel halves][16][LDS]
+  la_bf16* sP = reinterpret_cast<la_bf16*>(sS + 2 * LR_HEADS * LR_LDS);   // [16][LDP]
+  float* sA = reinterpret_cast<float*>(sP + LR_HEADS * LR_LDP);           // [16] rescale, then [16] max, [16] sum
+  const size_t row = blockIdx.x;
+  const int head0 = blockIdx.y * LR_HEADS, nh = min(LR_HEADS, p.H - head0), split = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row);
+  const bool live = p.slot == nullptr || p.slot[s] >= 0;
+  const int t_begin = split * p.partition, t_end = live ? min(p.pos[row] + 1, t_begin + p.partition) : t_begin;
+  const int* table = p.tables + static_cast<size_t>(s) * p.max_blocks;
+  const la_bf16* pages = static_cast<const la_bf16*>(p.pages);
+
+  auto issue = [&](int st, int t0) {
+    if (t0 < t_end) {
+#pragma unroll
+      for (int i = 0; i < LR_KEYS / 8; ++i) {
+        const int key = warp + 8 * i, t = t0 + key;
+        const bool in = t < t_end;
+        const la_bf16* src = pages + (in ? (static_cast<size_t>(table[t / LA_PAGE]) * LA_PAGE + t % LA_PAGE) * p.Rp : 0);
+        la_bf16* dst = sC + (st * LR_KEYS + key) * LD;
+        for (int c = lane; c < pieces; c += 32) {
+          const bool ok = in && c * 8 < p.Rp;
+          la_copy16(dst + c * 8, src + (ok ? c * 8 : 0), ok);
+        }
+      }
+    }
+    la_commit();
+  };
+  {
+    const la_bf16* q = static_cast<const la_bf16*>(p.q) + (row * p.H + head0) * p.Rp;
+    for (int i = tid; i < LR_HEADS * pieces; i += LR_THREADS) {
+      const int h = i / pieces, c = i % pieces * 8;
+      const bool in = h < nh && c < p.Rp;
+      la_copy16(sQ + h * LD + c, q + (in ? static_cast<size_t>(h) * p.Rp + c : 0), in);
+    }
+  }
+  issue(0, t_begin);          // the queries belong to this group
+  issue(1, t_begin + LR_KEYS);
+
+  const int kg = warp & 3, kh = warp >> 2, steps = R16 / 16;
+  const int k_lo = kh ? (steps + 1) / 2 : 0, k_hi = kh ? steps : (steps + 1) / 2;
+  const int sr = tid >> 4, sk = (tid & 15) * 4;          // softmax: row of scores and first of four keys
+  const float sl2 = p.scale * LA_LOG2E;
+  float m = -INFINITY, l = 0.f;
+  float acc[NG][2][4] = {};
+  int st = 0;
+  for (int t0 = t_begin; t0 < t_end; t0 += LR_KEYS, st ^= 1) {
+    la_wait<1>();
+    __syncthreads();
+    const la_bf16* tile = sC + st * LR_KEYS * LD;
+    {
+      float d[2][2][4] = {};
+      for (int k = k_lo; k < k_hi; k += 2) {
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          if (k + u >= k_hi) break;
+          uint32_t a[4], b[4];
+          ldsm_a_mk(sQ + (k + u) * 16, LD, lane, a);
+          ldsm_b_nk(tile + kg * 16 * LD + (k + u) * 16, LD, lane, b);
+          mma_n16(d[u][0], d[u][1], a, b);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+          float* o = sS + (kh * LR_HEADS + (lane >> 2) + 8 * hh) * LR_LDS + kg * 16 + n * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(o) = make_float2(d[0][n][2 * hh] + d[1][n][2 * hh], d[0][n][2 * hh + 1] + d[1][n][2 * hh + 1]);
+        }
+    }
+    __syncthreads();
+    {
+      const float4 x = *reinterpret_cast<const float4*>(sS + sr * LR_LDS + sk);
+      const float4 y = *reinterpret_cast<const float4*>(sS + (LR_HEADS + sr) * LR_LDS + sk);
+      float v[4] = {(x.x + y.x) * sl2, (x.y + y.y) * sl2, (x.z + y.z) * sl2, (x.w + y.w) * sl2};
+      float mx = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (t0 + sk + e >= t_end) v[e] = -INFINITY;
+        mx = fmaxf(mx, v[e]);
+      }
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float mn = fmaxf(m, mx), alpha = fast_exp2(m - mn);    // a tile has at least one key
+      float ps = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[e] = fast_exp2(v[e] - mn);
+        ps += v[e];
+      }
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+      l = l * alpha + ps;
+      m = mn;
+      *reinterpret_cast<uint2*>(sP + sr * LR_LDP + sk) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+      if (sk == 0) sA[sr] = alpha;
+    }
+    __syncthreads();
+    {
+      const float a0 = sA[lane >> 2], a1 = sA[(lane >> 2) + 8];
+#pragma unroll
+      for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          acc[g][n][0] *= a0;
+          acc[g][n][1] *= a0;
+          acc[g][n][2] *= a1;
+          acc[g][n][3] *= a1;
+        }
+#pragma unroll
+      for (int ks = 0; ks < LR_KEYS / 16; ++ks) {
+        uint32_t a[4];
+        ldsm_a_mk(sP + ks * 16, LR_LDP, lane, a);
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+          const int c = (warp + 8 * g) * 16;
+          if (c >= p.Cp) break;
+          uint32_t b[4];
+          ldsm_b_kn(tile + ks * 16 * LD + c, LD, lane, b);
+          mma_n16(acc[g][0], acc[g][1], a, b);
+        }
+      }
+    }
+    __syncthreads();
+    issue(st, t0 + 2 * LR_KEYS);
+  }
+  la_wait<0>();
+  if (sk == 0) {
+    sA[16 + sr] = m;
+    sA[32 + sr] = l;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int hh = 0; hh < 2; ++hh) {
+    const int r = (lane >> 2) + 8 * hh, head = head0 + r;
+    if (r >= nh) continue;
+    const size_t at = (row * p.H + head) * p.nsplit + split;
+    const float f = p.nsplit == 1 ? la_sink<la_bf16>(p, head, sA[16 + r], sA[32 + r]) : 1.f;
+#pragma unroll
+    for (int g = 0; g < NG; ++g)
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        const int c = (warp + 8 * g) * 16 + n * 8 + (lane & 3) * 2;
+        if (c >= p.Cp) continue;
+        const float x = acc[g][n][2 * hh] * f, y = acc[g][n][2 * hh + 1] * f;
+        if (p.nsplit == 1) *reinterpret_cast<uint32_t*>(static_cast<la_bf16*>(p.out) + (row * p.H + head) * p.Cp + c) = pack_bf16x2(x, y);
+        else *reinterpret_cast<float2*>(p.part_o + at * p.Cp + c) = make_float2(x, y);
+      }
+    if (p.nsplit > 1 && warp == 0 && (lane & 3) == 0) {
+      p.part_ml[at * 2] = sA[16 + r];
+      p.part_ml[at * 2 + 1] = sA[32 + r];
+    }
+  }
+}
+
+template <typename K>
+static int la_smem(K kern, int bytes, const char* what) {
+  if (bytes > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess) {
+    set_error("%s: cannot set shared memory size (%d)", what, bytes);
+    return 1;
+  }
+  return 0;
+}
+
+}  // namespace b2
+
+using namespace b2;
+
+B2_EXPORT int b2_latent_store(void* q, const void* c, const void* kr, long long ld, void* pages, const void* w, const int* tables,
+                              const int* row_seq, const int* pos, const int* slot, const float* cs, const float* sn, int M,
+                              int max_blocks, int H, int dim, int dqp, int rank, int Cp, int Rp, int rot, float eps, int is_f32,
+                              void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (H < 1 || dim < 1 || rot < 2 || rot % 2 || dim + rot > dqp || dqp % 8 || Cp % 8 || Rp % 8 || rank < 1 || rank > Cp ||
+      Rp - Cp < rot || ld % 8 || max_blocks < 1) {
+    set_error("latent_store: padded sizes in multiples of 8 and an even rotated size required");
+    return 10;
+  }
+  B2_DISPATCH_T(is_f32, latent_store_kernel<T><<<M, LS_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<T*>(q), static_cast<const T*>(c), static_cast<const T*>(kr), ld, static_cast<T*>(pages), static_cast<const T*>(w),
+      tables, row_seq, pos, slot, cs, sn, max_blocks, H, dim, dqp, rank, Cp, Rp, rot, eps););
+  B2_CHECK_LAUNCH("latent_store");
+  return 0;
+}
+
+// ids: int32 [n] page of the pool for every page of out; page_bytes a multiple of 16
+B2_EXPORT int b2_latent_gather(const void* pages, const int* ids, void* out, int n, int page_bytes, void* stream) {
+  b2::ensure_thread_context();
+  if (n <= 0) return 0;
+  if (page_bytes < 16 || page_bytes % 16) { set_error("latent_gather: pages of a multiple of 16 bytes required"); return 10; }
+  latent_gather_kernel<<<n, 128, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const uint8_t*>(pages), ids,
+                                                                         static_cast<uint8_t*>(out), page_bytes);
+  B2_CHECK_LAUNCH("latent_gather");
+  return 0;
+}
+
+B2_EXPORT int b2_head_linear(const void* x, const void* w, void* out, long long ld_x, long long ld_out, int M, int H, int N, int K,
+                             int xs, int os, int kn, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (H < 1 || H > 65535 || N < 8 || K < 8 || N % 8 || K % 8 || xs % 8 || os % 8 || ld_x % 8 || ld_out % 8) {
+    set_error("head_linear: sizes and strides in multiples of 8 required");
+    return 10;
+  }
+  HeadLinearParams p = {x, w, out, ld_x, ld_out, M, H, N, K, xs, os};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (is_f32) {
+    const dim3 grid((N + 255) / 256, H, M < 65535 ? M : 65535);
+    if (kn) head_linear_any_kernel<true><<<grid, 256, 0, st>>>(p);
+    else head_linear_any_kernel<false><<<grid, 256, 0, st>>>(p);
+  } else {
+    const dim3 grid((N + HL_T - 1) / HL_T, H, (M + HL_T - 1) / HL_T);
+    if (grid.z > 65535) { set_error("head_linear: too many rows (%d)", M); return 10; }
+    if (kn) head_linear_kernel<true><<<grid, 128, 0, st>>>(p);
+    else head_linear_kernel<false><<<grid, 128, 0, st>>>(p);
+  }
+  B2_CHECK_LAUNCH("head_linear");
+  return 0;
+}
+
+// partition: keys per split; nsplit * partition must cover every row's keys.
+B2_EXPORT int b2_latent_rows(const void* q, const void* pages, const int* tables, const int* row_seq, const int* pos,
+                             const int* slot, const void* sink, void* out, float* part_o, float* part_ml, int M, int max_blocks,
+                             int H, int Rp, int Cp, int partition, int nsplit, float scale, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (H < 1 || H > 65535 || Rp % 8 || Cp % 8 || Cp < 8 || Rp < Cp || Rp > 1280 || partition < 1 || nsplit < 1 || nsplit > 65535 ||
+      max_blocks < 1 || (nsplit > 1 && (part_o == nullptr || part_ml == nullptr))) {
+    set_error("latent_rows: rows up to 1280 channels in multiples of 8 required");
+    return 10;
+  }
+  LatentRowsParams p = {q, pages, tables, row_seq, pos, slot, sink, out, part_o, part_ml, max_blocks, H, Rp, Cp, partition, nsplit,
+                        scale};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (!is_f32 && Cp <= 512 && lr_bytes(Rp) <= 232448) {
+    const dim3 grid(M, (H + LR_HEADS - 1) / LR_HEADS, nsplit);
+    const int smem = lr_bytes(Rp);
+#define B2_LR(NGV)                                                                \
+  do {                                                                            \
+    if (int rc = la_smem(latent_rows_kernel<NGV>, smem, "latent_rows")) return rc; \
+    latent_rows_kernel<NGV><<<grid, LR_THREADS, smem, st>>>(p);                   \
+  } while (0)
+    if (Cp <= 128) B2_LR(1);
+    else if (Cp <= 256) B2_LR(2);
+    else B2_LR(4);
+#undef B2_LR
+  } else {
+    const dim3 grid(M, H, nsplit);
+    B2_DISPATCH_T(is_f32, {
+      if (Rp <= 256) {
+        latent_rows_any_kernel<T, 8><<<grid, LR_ANY_WARPS * 32, 5 * 256 * 4, st>>>(p);
+      } else {
+        latent_rows_any_kernel<T, 40><<<grid, LR_ANY_WARPS * 32, 5 * 1280 * 4, st>>>(p);
+      }
+    });
+  }
+  B2_CHECK_LAUNCH("latent_rows");
+  if (nsplit > 1) {
+    B2_DISPATCH_T(is_f32, latent_merge_kernel<T><<<dim3(M, H), 128, 0, st>>>(p););
+    B2_CHECK_LAUNCH("latent_merge");
+  }
+  return 0;
+}

@@ -1,13 +1,17 @@
 // Paged attention one query row at a time, for any head sizes up to 256, in bf16 or true 32-bit: the decode step and short
 // portions.  Beside plain causal attention it takes, each optional,
 //   * chunked visibility: row at position i sees keys floor(i / chunk) * chunk .. i only;
+//   * a sliding window: keys i - window + 1 .. i only;
+//   * a soft cap: scores pass through cap * tanh(score / cap);
 //   * a learned additive bias per head and distance bucket: rel[bucket[min(i - j, len - 1)], h];
 //   * a softmax sink per head: exp(sink_h) joins the denominator, with no key and no value;
-//   * an output gate per head: the head's output times sigmoid(gate).
-// And the stage before it: per-head RMS norm of q and k and the store of k and v into their pages.
+//   * an output gate per head: the head's output times sigmoid(gate);
+//   * differential heads (MAPS = 2): a head has two query rows and two key rows over one value row, two attentions a1 and a2 that
+//     leave as rms(a1 - lambda a2) (1 - lambda_init), times a sigmoid gate per channel.
+// And the stage before it: bias, per-head RMS norm and rotary positions of q and k and the store of k and v into their pages.
 //
 // Cache layout of one layer: K [blocks, 16, G, dkp], V [blocks, 16, G, dvp] in the activation type, head sizes padded to a
-// multiple of eight (padding zero).  Row r belongs to sequence row_seq[r], whose pages are block_tables[row_seq[r]][*].
+// multiple of eight (padding zero); differential: K [blocks, 16, G, 2, dkp], q [M, H, 2, dkp].  Row r belongs to sequence row_seq[r], whose pages are block_tables[row_seq[r]][*].
 #include "host.h"
 #include "vec.cuh"
 
@@ -26,7 +30,7 @@ struct AttnRowsParams {
   const int* row_seq;    // [M] or null: row r is sequence r
   const int* pos;        // [M]
   const int* slot;       // per sequence, or null: slot < 0 marks a padding row (output zero)
-  const void* gate;      // T [M, ld_gate]: H columns, or null
+  const void* gate;      // T [M, ld_gate]: H columns (differential: H * dvp), or null
   const void* sink;      // T [H] or null
   const void* rel;       // T [buckets, H] or null
   const int* bucket;     // [nbucket]
@@ -36,6 +40,10 @@ struct AttnRowsParams {
   long long ld_gate, ld_out;
   int max_blocks, H, G, dkp, dvp, chunk, nbucket, partition, nsplit, groups;
   float scale;
+  int window, dv;        // dv: real value channels (the differential norm divides by it)
+  float softcap;
+  const void* lam;       // differential: T [4, dkp] = lq1, lk1, lq2, lk2
+  float lam_init, eps;
 };
 
 // softmax weights: the special-function unit's 2^x beside bf16 values, the library's in 32-bit runs
@@ -59,6 +67,28 @@ __device__ __forceinline__ float ar_finish(const AttnRowsParams& p, int head, si
   return o;
 }
 
+// Differential heads: o = a1 - lambda a2, normed over the head's channels, times 1 - lambda_init and the gate.  N channels of
+// one head per thread, c0 + i * stride; `sum` adds over the threads that share the head.
+template <typename T, int N, typename F>
+__device__ __forceinline__ void ar_diff_store(const AttnRowsParams& p, float lam, int head, size_t row, const float (&a1)[N],
+                                              const float (&a2)[N], int c0, int stride, F sum) {
+  float o[N], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    o[i] = c0 + i * stride < p.dvp ? a1[i] - lam * a2[i] : 0.f;
+    ss = fmaf(o[i], o[i], ss);
+  }
+  const float r = (1.f - p.lam_init) / sqrtf(sum(ss) / p.dv + p.eps);
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = c0 + i * stride;
+    if (c >= p.dvp) break;
+    float x = o[i] * r;
+    if (p.gate) x *= sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[row * p.ld_gate + static_cast<size_t>(head) * p.dvp + c]));
+    static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(head) * p.dvp + c] = from_f<T>(x);
+  }
+}
+
 // Grid (M, G * groups, nsplit).  A key row is spread over LPT lanes, eight channels each, so one warp-wide step covers
 // 32 / LPT tokens; every lane group runs its own online softmax over the tokens it sees for the GH query heads of this CTA,
 // and groups and warps are merged at the end with the exact log-sum-exp rule.
@@ -68,12 +98,14 @@ __device__ __forceinline__ float ar_finish(const AttnRowsParams& p, int head, si
 // loaded into registers.
 constexpr int AR_STAGES = 3;
 template <typename T>
-__host__ __device__ constexpr int ar_ring_bytes() {
-  return sizeof(T) == 2 ? (AR_THREADS / 32) * AR_STAGES * AR_UNROLL * 2 * 512 : 0;
+__host__ __device__ constexpr int ar_ring_bytes(int maps) {
+  return sizeof(T) == 2 ? (AR_THREADS / 32) * AR_STAGES * AR_UNROLL * (maps + 1) * 512 : 0;
 }
-template <typename T, int LPT, int GH>
+// GH: query rows of a CTA (a differential head has two, of which row g reads key row g % 2)
+template <typename T, int LPT, int GH, int MAPS>
 __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsParams p) {
-  constexpr int TPW = 32 / LPT, U = AR_UNROLL;
+  constexpr int TPW = 32 / LPT, U = AR_UNROLL, PIECES = MAPS + 1;
+  static_assert(GH % MAPS == 0, "a differential head's two query rows belong to one CTA");
   constexpr bool RING = sizeof(T) == 2;
   extern __shared__ __align__(16) uint8_t ar_dyn[];   // ring, then bias [GH][partition]
   __shared__ float sAcc[AR_THREADS / 32][GH][LPT * 8];
@@ -81,46 +113,49 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
   const size_t row = blockIdx.x;
   const int kvh = blockIdx.y / p.groups, hg = blockIdx.y % p.groups, split = blockIdx.z;
   const int per = p.H / p.G;
-  const int nh = min(GH, per - hg * GH);
-  const int head0 = kvh * per + hg * GH;
+  const int nh = min(GH, (per - hg * (GH / MAPS)) * MAPS);
+  const int head0 = (kvh * per + hg * (GH / MAPS)) * MAPS;      // first query row's index among H * MAPS
   const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row);
   const bool live = p.slot == nullptr || p.slot[s] >= 0;
   const int pos = p.pos[row];
-  const int first = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+  const int first = p.chunk > 0 ? pos / p.chunk * p.chunk : p.window > 0 ? max(0, pos - p.window + 1) : 0;
   const int t_begin = first + split * p.partition;
   const int t_end = live ? min(pos + 1, t_begin + p.partition) : t_begin;
   const int* table = p.tables + static_cast<size_t>(s) * p.max_blocks;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, group = lane / LPT, sub = lane % LPT;
   const bool kin = sub * 8 < p.dkp, vin = sub * 8 < p.dvp;
-  const T* kc = static_cast<const T*>(p.kc) + static_cast<size_t>(kvh) * p.dkp + sub * 8;
+  const T* kc = static_cast<const T*>(p.kc) + static_cast<size_t>(kvh) * MAPS * p.dkp + sub * 8;
   const T* vc = static_cast<const T*>(p.vc) + static_cast<size_t>(kvh) * p.dvp + sub * 8;
-  const size_t kts = static_cast<size_t>(p.G) * p.dkp, vts = static_cast<size_t>(p.G) * p.dvp;
+  const size_t kts = static_cast<size_t>(p.G) * MAPS * p.dkp, vts = static_cast<size_t>(p.G) * p.dvp;
 
   float qr[GH][8], acc[GH][8], m[GH], l[GH];
+  const float qscale = p.softcap > 0.f ? p.scale : p.scale * AR_LOG2E;
 #pragma unroll
   for (int g = 0; g < GH; ++g) {
     float t[8] = {};
-    if (kin && g < nh) vload8(static_cast<const T*>(p.q) + (row * p.H + head0 + g) * p.dkp + sub * 8, t);
+    if (kin && g < nh) vload8(static_cast<const T*>(p.q) + (row * p.H * MAPS + head0 + g) * p.dkp + sub * 8, t);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      qr[g][e] = t[e] * (p.scale * AR_LOG2E);
+      qr[g][e] = t[e] * qscale;
       acc[g][e] = 0.f;
     }
     m[g] = -INFINITY;
     l[g] = 0.f;
   }
   constexpr int STEP = (AR_THREADS / 32) * TPW * U;
-  float* sBias = reinterpret_cast<float*>(ar_dyn + ar_ring_bytes<T>());
-  const uint32_t ring = smem_u32(ar_dyn) + (warp * AR_STAGES * U * 2 * 32 + lane) * 16;
+  float* sBias = reinterpret_cast<float*>(ar_dyn + ar_ring_bytes<T>(MAPS));
+  const uint32_t ring = smem_u32(ar_dyn) + (warp * AR_STAGES * U * PIECES * 32 + lane) * 16;
   auto issue = [&](int stage, int at) {
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int tok = at + u * TPW + group;
       if (tok < t_end) {
         const size_t a = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
-        const uint32_t dst = ring + ((stage * U + u) * 2) * 512;
-        if (kin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(kc + a * kts) : "memory");
-        if (vin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + 512), "l"(vc + a * vts) : "memory");
+        const uint32_t dst = ring + ((stage * U + u) * PIECES) * 512;
+#pragma unroll
+        for (int mp = 0; mp < MAPS; ++mp)
+          if (kin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + mp * 512), "l"(kc + a * kts + mp * p.dkp) : "memory");
+        if (vin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + MAPS * 512), "l"(vc + a * vts) : "memory");
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");   // one group per stage, empty ones included
@@ -146,32 +181,34 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
       issue(stage == 0 ? AR_STAGES - 1 : stage - 1, base + (AR_STAGES - 1) * STEP);
       asm volatile("cp.async.wait_group %0;" ::"n"(AR_STAGES - 1) : "memory");
     }
-    // one K (which = 0) or V (1) piece of this lane; zero past the partition and past the head's channels
+    // one K (which < MAPS) or V (MAPS) piece of this lane; zero past the partition and past the head's channels
     auto piece = [&](int u, int which, float (&f)[8]) {
       const int tok = base + u * TPW + group;
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] = 0.f;
-      if (tok >= t_end || !(which ? vin : kin)) return;
+      if (tok >= t_end || !(which == MAPS ? vin : kin)) return;
       if (RING) {
-        vload8(reinterpret_cast<const __nv_bfloat16*>(ar_dyn + (warp * AR_STAGES * U * 2 * 32 + lane) * 16 +
-                                                      ((stage * U + u) * 2 + which) * 512), f);
+        vload8(reinterpret_cast<const __nv_bfloat16*>(ar_dyn + (warp * AR_STAGES * U * PIECES * 32 + lane) * 16 +
+                                                      ((stage * U + u) * PIECES + which) * 512), f);
       } else {
         const size_t at = static_cast<size_t>(table[tok / AR_PAGE]) * AR_PAGE + tok % AR_PAGE;
-        vload8(which ? vc + at * vts : kc + at * kts, f);
+        vload8(which == MAPS ? vc + at * vts : kc + at * kts + which * p.dkp, f);
       }
     };
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int tok = base + u * TPW + group;
-      float kf[8];
-      piece(u, 0, kf);
+      float kf[MAPS][8];
+#pragma unroll
+      for (int mp = 0; mp < MAPS; ++mp) piece(u, mp, kf[mp]);
 #pragma unroll
       for (int g = 0; g < GH; ++g) {
         float d = 0.f;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) d = fmaf(qr[g][e], kf[e], d);
+        for (int e = 0; e < 8; ++e) d = fmaf(qr[g][e], kf[g % MAPS][e], d);
 #pragma unroll
         for (int o = LPT / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+        if (p.softcap > 0.f) d = softcap_t<T>(d, p.softcap) * AR_LOG2E;
         if (p.rel && tok < t_end && g < nh) d += sBias[g * p.partition + tok - t_begin];
         sc[u][g] = tok < t_end ? d : -INFINITY;
       }
@@ -201,7 +238,7 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       float vf[8];
-      piece(u, 1, vf);
+      piece(u, MAPS, vf);
 #pragma unroll
       for (int g = 0; g < GH; ++g)
 #pragma unroll
@@ -232,6 +269,33 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
       }
     }
   __syncthreads();
+  if (MAPS == 2 && p.nsplit == 1) {
+    const float lam = diff_lambda(static_cast<const T*>(p.lam), p.dkp, p.lam_init);
+    for (int hd = warp; hd < nh / 2; hd += AR_THREADS / 32) {
+      constexpr int N = LPT / 4;             // channels of a lane: LPT * 8 / 32
+      float a[2][N];
+#pragma unroll
+      for (int mp = 0; mp < 2; ++mp) {
+        const int g = hd * 2 + mp;
+        float M = -INFINITY, L = 0.f;
+#pragma unroll
+        for (int w = 0; w < AR_THREADS / 32; ++w) M = fmaxf(M, sM[w][g]);
+#pragma unroll
+        for (int i = 0; i < N; ++i) a[mp][i] = 0.f;
+#pragma unroll
+        for (int w = 0; w < AR_THREADS / 32; ++w) {
+          const float wt = sM[w][g] == -INFINITY ? 0.f : exp2f(sM[w][g] - M);
+          L += sL[w][g] * wt;
+#pragma unroll
+          for (int i = 0; i < N; ++i) a[mp][i] += sAcc[w][g][lane + 32 * i] * wt;
+        }
+#pragma unroll
+        for (int i = 0; i < N; ++i) a[mp][i] = L > 0.f ? a[mp][i] / L : 0.f;
+      }
+      ar_diff_store<T>(p, lam, head0 / 2 + hd, row, a[0], a[1], lane, 32, [](float v) { return warp_sum(v); });
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < nh * p.dvp; i += AR_THREADS) {
     const int g = i / p.dvp, c = i % p.dvp, head = head0 + g;
     float M = -INFINITY;
@@ -247,7 +311,7 @@ __global__ void __launch_bounds__(AR_THREADS) attn_rows_kernel(const AttnRowsPar
     if (p.nsplit == 1) {
       static_cast<T*>(p.out)[row * p.ld_out + static_cast<size_t>(head) * p.dvp + c] = from_f<T>(ar_finish<T>(p, head, row, o, L, M));
     } else {
-      const size_t at = (row * p.H + head) * p.nsplit + split;
+      const size_t at = (row * p.H * MAPS + head) * p.nsplit + split;
       p.part_o[at * p.dvp + c] = o;
       if (c == 0) {
         p.part_ml[at * 2] = M;
@@ -277,25 +341,63 @@ __global__ void __launch_bounds__(128) attn_rows_merge_kernel(const AttnRowsPara
   }
 }
 
-// Per-head RMS norm of q and k (optional weights) and the store of k / v.  Grid (M, ceil((H + 2 G) / 4)), one warp per head.
+// Splits of both query rows of a differential head.  Grid (M, H).
+template <typename T>
+__global__ void __launch_bounds__(128) attn_rows_diff_merge_kernel(const AttnRowsParams p) {
+  __shared__ float red[4];
+  const size_t row = blockIdx.x;
+  const int head = blockIdx.y;
+  const float lam = diff_lambda(static_cast<const T*>(p.lam), p.dkp, p.lam_init);
+  float a[2][2];
+#pragma unroll
+  for (int mp = 0; mp < 2; ++mp) {
+    const size_t at = ((row * p.H + head) * 2 + mp) * p.nsplit;
+    float M = -INFINITY, L = 0.f, o0 = 0.f, o1 = 0.f;
+    for (int i = 0; i < p.nsplit; ++i) M = fmaxf(M, p.part_ml[(at + i) * 2]);
+    for (int i = 0; i < p.nsplit; ++i) {
+      const float mi = p.part_ml[(at + i) * 2];
+      if (mi == -INFINITY) continue;
+      const float w = exp2f(mi - M);
+      L += p.part_ml[(at + i) * 2 + 1] * w;
+      const float* o = p.part_o + (at + i) * p.dvp;
+      if (static_cast<int>(threadIdx.x) < p.dvp) o0 += o[threadIdx.x] * w;
+      if (static_cast<int>(threadIdx.x) + 128 < p.dvp) o1 += o[threadIdx.x + 128] * w;
+    }
+    a[mp][0] = L > 0.f ? o0 / L : 0.f;
+    a[mp][1] = L > 0.f ? o1 / L : 0.f;
+  }
+  ar_diff_store<T>(p, lam, head, row, a[0], a[1], threadIdx.x, 128, [&](float v) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    return red[0] + red[1] + red[2] + red[3];
+  });
+}
+
+// Bias, per-head RMS norm of q and k (optional weights), rotary positions on channel pairs (2 i, 2 i + 1), and the store of k / v.
+// Grid (M, ceil((H + Gk + Gv) / 4)), one warp per head.
 template <typename T>
 __global__ void __launch_bounds__(128) qk_norm_store_kernel(const T* __restrict__ q, const T* __restrict__ k,
                                                             const T* __restrict__ v, long long ld, T* __restrict__ q_out,
                                                             T* __restrict__ kc, T* __restrict__ vc,
                                                             const int* __restrict__ tables, const int* __restrict__ row_seq,
                                                             const int* __restrict__ pos, const int* __restrict__ slot,
-                                                            int max_blocks, int H, int G, int dk, int dkp, int dvp,
+                                                            int max_blocks, int H, int G, int Gv, int dk, int dkp, int dvp,
                                                             const T* __restrict__ wq, const T* __restrict__ wk, int norm,
-                                                            float eps) {
+                                                            float eps, const T* __restrict__ bq, const T* __restrict__ bk,
+                                                            const T* __restrict__ bv, const float* __restrict__ cs,
+                                                            const float* __restrict__ sn, int rot) {
   const size_t row = blockIdx.x;
   const int w = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (w >= H + 2 * G) return;
+  if (w >= H + G + Gv) return;
   const int s = row_seq ? row_seq[row] : static_cast<int>(row);
   const bool live = slot == nullptr || slot[s] >= 0;
   const T* src;
   T* dst = nullptr;
+  const T* bias;
   int width = dkp;
   if (w < H) {
+    bias = bq ? bq + static_cast<size_t>(w) * dkp : nullptr;
     src = q + row * ld + static_cast<size_t>(w) * dkp;
     dst = q_out + (row * H + w) * dkp;
   } else {
@@ -303,15 +405,24 @@ __global__ void __launch_bounds__(128) qk_norm_store_kernel(const T* __restrict_
     const int p = pos[row];
     if (live) {
       const size_t at = static_cast<size_t>(tables[static_cast<size_t>(s) * max_blocks + p / AR_PAGE]) * AR_PAGE + p % AR_PAGE;
-      dst = w < H + G ? kc + (at * G + g) * dkp : vc + (at * G + g) * dvp;
+      dst = w < H + G ? kc + (at * G + g) * dkp : vc + (at * Gv + g) * dvp;
     }
+    bias = w < H + G ? (bk ? bk + static_cast<size_t>(g) * dkp : nullptr) : (bv ? bv + static_cast<size_t>(g) * dvp : nullptr);
     width = w < H + G ? dkp : dvp;
     src = (w < H + G ? k + row * ld + static_cast<size_t>(g) * dkp : v + row * ld + static_cast<size_t>(g) * dvp);
   }
   if (dst == nullptr) return;
   const int c = lane * 8;   // widths up to 256
   float t[8] = {};
-  if (c < width) vload8(src + c, t);
+  if (c < width) {
+    vload8(src + c, t);
+    if (bias) {
+      float b[8];
+      vload8(bias + c, b);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) t[e] += b[e];
+    }
+  }
   if (w < H + G && norm) {
     float ss = 0.f;
 #pragma unroll
@@ -321,16 +432,26 @@ __global__ void __launch_bounds__(128) qk_norm_store_kernel(const T* __restrict_
 #pragma unroll
     for (int e = 0; e < 8; ++e) t[e] *= wt && c + e < dk ? r * to_f(wt[c + e]) : r;
   }
+  if (cs && w < H + G) {
+    const size_t at = row * (rot / 2) + c / 2;
+#pragma unroll
+    for (int e = 0; e < 8; e += 2)
+      if (c + e < rot) {
+        const float co = cs[at + e / 2], si = sn[at + e / 2], u = t[e], x = t[e + 1];
+        t[e] = u * co - x * si;
+        t[e + 1] = x * co + u * si;
+      }
+  }
   if (c < width) vstore8(dst + c, t);
 }
 
 template <typename T, int LPT>
 static int launch_rows(const AttnRowsParams& p, int M, int GH, cudaStream_t stream) {
   const dim3 grid(M, p.G * p.groups, p.nsplit);
-  const int smem = ar_ring_bytes<T>() + (p.rel ? GH * p.partition * 4 : 0);
-#define B2_ROWS(GHV)                                                                                              \
+  const int smem = ar_ring_bytes<T>(p.lam ? 2 : 1) + (p.rel ? GH * p.partition * 4 : 0);
+#define B2_ROWS(GHV, MAPSV)                                                                                       \
   do {                                                                                                            \
-    auto kern = attn_rows_kernel<T, LPT, GHV>;                                                                    \
+    auto kern = attn_rows_kernel<T, LPT, GHV, MAPSV>;                                                                    \
     static int set[64] = {0};                                                                                     \
     int dev = 0;                                                                                                  \
     cudaGetDevice(&dev);                                                                                          \
@@ -343,15 +464,23 @@ static int launch_rows(const AttnRowsParams& p, int M, int GH, cudaStream_t stre
     }                                                                                                             \
     kern<<<grid, AR_THREADS, smem, stream>>>(p);                                                                  \
   } while (0)
-  switch (GH) {
-    case 1: B2_ROWS(1); break;
-    case 2: B2_ROWS(2); break;
-    case 3: B2_ROWS(3); break;
-    default: B2_ROWS(4); break;
+  if (p.lam) {
+    if (GH == 2) B2_ROWS(2, 2);
+    else B2_ROWS(4, 2);
+  } else {
+    switch (GH) {
+      case 1: B2_ROWS(1, 1); break;
+      case 2: B2_ROWS(2, 1); break;
+      case 3: B2_ROWS(3, 1); break;
+      default: B2_ROWS(4, 1); break;
+    }
   }
 #undef B2_ROWS
   B2_CHECK_LAUNCH("attn_rows");
-  if (p.nsplit > 1) {
+  if (p.nsplit > 1 && p.lam) {
+    attn_rows_diff_merge_kernel<T><<<dim3(M, p.H), 128, 0, stream>>>(p);
+    B2_CHECK_LAUNCH("attn_rows_diff_merge");
+  } else if (p.nsplit > 1) {
     attn_rows_merge_kernel<T><<<dim3(M, p.H), 128, 0, stream>>>(p);
     B2_CHECK_LAUNCH("attn_rows_merge");
   }
@@ -362,17 +491,20 @@ static int launch_rows(const AttnRowsParams& p, int M, int GH, cudaStream_t stre
 
 using namespace b2;
 
+// lam (T [4, dkp]): differential heads, whose out is normed over dv channels with eps; the gate then has H * dvp columns.
 // partition: keys per split (at most 4096 with a bias), counted from the row's first visible key; nsplit * partition must cover every row's keys.
 B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const int* tables, const int* row_seq,
                            const int* pos, const int* slot, const void* gate, long long ld_gate, const void* sink,
                            const void* rel, const int* bucket, int nbucket, void* out, long long ld_out, float* part_o,
                            float* part_ml, int M, int max_blocks, int H, int G, int dkp, int dvp, int chunk, int partition,
-                           int nsplit, float scale, int is_f32, void* stream) {
+                           int nsplit, float scale, int window, float softcap, const void* lam, float lam_init, float eps, int dv,
+                           int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (H < 1 || G < 1 || H % G || dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || dkp < 8 || dvp < 8 || nsplit < 1 ||
       nsplit > 65535 || partition < 1 || (nsplit > 1 && (part_o == nullptr || part_ml == nullptr)) ||
-      (rel != nullptr && (bucket == nullptr || nbucket < 1 || partition > 4096)) || max_blocks < 1 || H > 65535) {
+      (rel != nullptr && (bucket == nullptr || nbucket < 1 || partition > 4096)) || max_blocks < 1 || H > 65535 ||
+      (lam != nullptr && (rel != nullptr || sink != nullptr || dv < 1 || dv > dvp))) {
     set_error("attn_rows: H %% G == 0 and head sizes up to 256 in multiples of 8 (padded) required");
     return 10;
   }
@@ -381,9 +513,10 @@ B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const 
   p.sink = sink; p.rel = rel; p.bucket = bucket; p.out = out; p.part_o = part_o; p.part_ml = part_ml; p.ld_gate = ld_gate;
   p.ld_out = ld_out; p.max_blocks = max_blocks; p.H = H; p.G = G; p.dkp = dkp; p.dvp = dvp; p.chunk = chunk;
   p.nbucket = nbucket; p.partition = partition; p.nsplit = nsplit; p.scale = scale;
-  const int per = H / G;
-  p.groups = (per + 3) / 4;
-  const int GH = (per + p.groups - 1) / p.groups;
+  p.window = window; p.softcap = softcap; p.lam = lam; p.lam_init = lam_init; p.eps = eps; p.dv = dv;
+  const int per = H / G, most = lam ? 2 : 4;
+  p.groups = (per + most - 1) / most;
+  const int GH = (per + p.groups - 1) / p.groups * (lam ? 2 : 1);
   const int w = dkp > dvp ? dkp : dvp;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   B2_DISPATCH_T(is_f32, {
@@ -395,19 +528,22 @@ B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const 
 
 B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long long ld, void* q_out, void* kc, void* vc,
                                const int* tables, const int* row_seq, const int* pos, const int* slot, int M,
-                               int max_blocks, int H, int G, int dk, int dkp, int dvp, const void* wq, const void* wk,
-                               int norm, float eps, int is_f32, void* stream) {
+                               int max_blocks, int H, int G, int Gv, int dk, int dkp, int dvp, const void* wq, const void* wk,
+                               int norm, float eps, const void* bq, const void* bk, const void* bv, const float* cs,
+                               const float* sn, int rot, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
-  if (dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || ld % 8 || dk < 1 || dk > dkp || max_blocks < 1 || H < 1 || G < 1) {
+  if (dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || ld % 8 || dk < 1 || dk > dkp || max_blocks < 1 || H < 1 || G < 1 || Gv < 1 ||
+      (cs != nullptr && (rot < 2 || rot % 2 || rot > dk))) {
     set_error("qk_norm_store: head sizes up to 256 in multiples of 8 (padded) required");
     return 10;
   }
-  const dim3 grid(M, (H + 2 * G + 3) / 4);
+  const dim3 grid(M, (H + G + Gv + 3) / 4);
   B2_DISPATCH_T(is_f32, qk_norm_store_kernel<T><<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(
       static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), ld, static_cast<T*>(q_out),
-      static_cast<T*>(kc), static_cast<T*>(vc), tables, row_seq, pos, slot, max_blocks, H, G, dk, dkp, dvp,
-      static_cast<const T*>(wq), static_cast<const T*>(wk), norm, eps););
+      static_cast<T*>(kc), static_cast<T*>(vc), tables, row_seq, pos, slot, max_blocks, H, G, Gv, dk, dkp, dvp,
+      static_cast<const T*>(wq), static_cast<const T*>(wk), norm, eps, static_cast<const T*>(bq), static_cast<const T*>(bk),
+      static_cast<const T*>(bv), cs, sn, rot););
   B2_CHECK_LAUNCH("qk_norm_store");
   return 0;
 }

@@ -336,22 +336,27 @@ __host__ __device__ constexpr uint32_t make_idesc_f16(uint32_t fmt, uint32_t M, 
 // bytes each (partial-sector writes: ~2000 cycles for a 32 KiB tile); staged through 4 KiB of shared
 // memory private to the warp, every instruction writes four complete 128-byte lines.
 // row_ptr(row) returns the global address of that row's 128 bytes, or nullptr to skip the row.
-template <typename RowPtr>
+// ROWS: rows the staging block holds (32, or 16 in two passes).
+template <int ROWS = 32, typename RowPtr>
 __device__ __forceinline__ void warp_store_rows_128B(uint8_t* stage, const uint4 (&v)[8], RowPtr row_ptr) {
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & 31, chunk = lane & 7;
 #pragma unroll
-  for (int j = 0; j < 8; ++j)
-    *reinterpret_cast<uint4*>(stage + lane * 128 + ((j ^ (lane & 7)) << 4)) = v[j];
-  __syncwarp();
-  const int chunk = lane & 7;
+  for (int r0 = 0; r0 < 32; r0 += ROWS) {
+    if (ROWS == 32 || lane / ROWS == r0 / ROWS) {
 #pragma unroll
-  for (int k = 0; k < 8; ++k) {
-    const int row = 4 * k + (lane >> 3);
-    const uint4 val = *reinterpret_cast<const uint4*>(stage + row * 128 + ((chunk ^ (row & 7)) << 4));
-    uint8_t* dst = row_ptr(row);
-    if (dst) *reinterpret_cast<uint4*>(dst + chunk * 16) = val;
+      for (int j = 0; j < 8; ++j)
+        *reinterpret_cast<uint4*>(stage + (lane - r0) * 128 + ((j ^ (lane & 7)) << 4)) = v[j];
+    }
+    __syncwarp();
+#pragma unroll
+    for (int k = 0; k < ROWS / 4; ++k) {
+      const int row = 4 * k + (lane >> 3);
+      const uint4 val = *reinterpret_cast<const uint4*>(stage + row * 128 + ((chunk ^ (row & 7)) << 4));
+      uint8_t* dst = row_ptr(r0 + row);
+      if (dst) *reinterpret_cast<uint4*>(dst + chunk * 16) = val;
+    }
+    __syncwarp();
   }
-  __syncwarp();
 }
 
 // ---- small numeric helpers -----------------------------------------------------------------

@@ -23,6 +23,7 @@
 
 #include "common.cuh"
 #include "host.h"
+#include "vec.cuh"
 
 namespace b2 {
 
@@ -186,7 +187,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
                  const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmR,
                  void* __restrict__ Cout, const __nv_bfloat16* __restrict__ R, int M, int N, int K,
                  int ldc, int flags, GemmMnDesc mn, const __grid_constant__ GemmComm comm, int* status,
-                 int split_k, const __grid_constant__ GemmExt ext) {
+                 int split_k, const __grid_constant__ GemmExt ext, int act, int act_cols) {
   using Cfg = GemmCfg<BN>;
   static_assert(COMM == 0 || !A_MN, "fused communication paths take a K-major A operand");
   extern __shared__ uint8_t smem_raw[];
@@ -607,6 +608,26 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
                 }
               }
             }
+            if (act != 0 && col0 < act_cols) {   // act_cols is a multiple of 8
+#pragma unroll
+              for (int c8 = 0; c8 < 8; ++c8) {
+                if (col0 + c8 * 8 >= act_cols) break;
+#pragma unroll
+                for (int e = 0; e < 8; e += 2) {
+                  float x0 = __uint_as_float(v[c8 * 8 + e]), x1 = __uint_as_float(v[c8 * 8 + e + 1]);
+                  if (act == GEMM_ACT_SILU) {
+                    silu_pair_fast(x0, x1);
+                  } else {
+                    x0 = fmaxf(x0, 0.f);
+                    x1 = fmaxf(x1, 0.f);
+                    x0 *= x0;
+                    x1 *= x1;
+                  }
+                  v[c8 * 8 + e] = __float_as_uint(x0);
+                  v[c8 * 8 + e + 1] = __float_as_uint(x1);
+                }
+              }
+            }
 #pragma unroll
             for (int c8 = 0; c8 < 8; ++c8) {
               uint4 o;
@@ -787,7 +808,7 @@ template <int BN, bool A_MN, bool B_MN, int COMM = 0>
 static int launch_gemm(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
                        int lda, int ldb, int ldc, int flags, int max_ctas, cudaStream_t stream,
                        const GemmComm* comm_in = nullptr, const void* A2 = nullptr, const void* B2 = nullptr,
-                       int K2 = 0, int lda2 = 0, int ldb2 = 0) {
+                       int K2 = 0, int lda2 = 0, int ldb2 = 0, int act = 0, int act_cols = 0) {
   using Cfg = GemmCfg<BN>;
   auto kern = gemm_bf16_kernel<BN, A_MN, B_MN, COMM>;
   GemmComm comm;
@@ -868,7 +889,7 @@ static int launch_gemm(const void* A, const void* B, void* C, const void* R, int
   }
   kern<<<grid, GEMM_THREADS + (COMM == 2 ? 128 : COMM == 1 ? 64 : 0), Cfg::SMEM_BYTES, stream>>>(
       *ta, *tb, *tc, *tr, C, reinterpret_cast<const __nv_bfloat16*>(R), M, N, K, ldc, flags, g_mn_desc, comm, status,
-      split_k, ext);
+      split_k, ext, act, act_cols);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_error("gemm launch failed: %s", cudaGetErrorString(e));
@@ -965,6 +986,27 @@ B2_EXPORT int b2_gemm_bf16_ext(const void* A, const void* B, void* C, const void
 #undef B2_GEMM_EXT_CASE
   set_error("gemm_ext: unsupported configuration bn=%d b_mn=%d", bn, b_mn);
   return 11;
+}
+
+// C[M,N] = A[M,K] B[N,K]^T in bf16, the first act_cols columns through an activation (GEMM_ACT_*) before they are rounded.
+B2_EXPORT int b2_gemm_bf16_act(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int act,
+                               int act_cols, void* stream_) {
+  b2::ensure_thread_context();
+  using namespace b2;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((lda % 8) || (ldb % 8) || (ldc % 8) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) ||
+      (reinterpret_cast<uintptr_t>(C) & 15) || (act != GEMM_ACT_SILU && act != GEMM_ACT_RELU2) || (act_cols % 8 && act_cols < N)) {
+    set_error("gemm_act: 16-byte aligned operands, a known activation and act_cols %% 8 == 0 required (lda %d ldb %d ldc %d act_cols %d)",
+              lda, ldb, ldc, act_cols);
+    return 10;
+  }
+  const int tiles256 = ((M + 127) / 128) * ((N + 255) / 256), sms = num_sms();
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if ((tiles256 >= sms || N % 256 == 0) && tiles256 * 2 > sms)
+    return launch_gemm<256, false, false>(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, 0, stream, nullptr, nullptr, nullptr, 0, 0,
+                                          0, act, act_cols);
+  return launch_gemm<128, false, false>(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, 0, stream, nullptr, nullptr, nullptr, 0, 0, 0,
+                                        act, act_cols);
 }
 
 // Test hook: descriptor strides used for MN-major operands (bytes): distance between 64-element

@@ -8,6 +8,10 @@
 
 namespace b2 {
 
+// activations a matrix product can apply to its first output columns
+constexpr int GEMM_ACT_SILU = 1;
+constexpr int GEMM_ACT_RELU2 = 2;    // the square of relu
+
 // Makes the process's device (b2_set_device) current on the calling thread.  Launchers call this
 // first: autograd runs backward passes on worker threads that this library's runtime has never
 // seen, and driver entry points such as the tensor-map encoder need a current context.

@@ -4,7 +4,9 @@
 //   retention   S <- a_h S + k v^T                                     o = S^T q     (one fixed decay per head)
 //   delta rule  S <- g . S;  u = beta (v - S^T k);  S <- S + k u^T     o = S^T q     (one decay per head and key channel)
 //
-// followed by a per-head RMS norm over the value channels and an output gate.  This file has the token-by-token form,
+// followed by a per-head RMS norm over the value channels and an output gate; or, for retention whose heads are normed together,
+// by the norm's weight and a sigmoid gate, with the sum of squares of every head left for the reader of the output projection
+// (the norm is one factor per row, which commutes with that projection).  This file has the token-by-token form,
 // which is the decode step, the form for short portions, and the one that runs in true 32-bit; it also has the delta
 // rule's input stage (short causal convolution, activation, unit norms, decays, step sizes).
 //
@@ -34,7 +36,8 @@ struct SerialParams {
   const float* cs;    // rotary tables [M, rot / 2] (retention)
   const float* sn;
   const float* decay;       // retention: [H]
-  const void* norm_w;       // T [dvp] or null
+  const void* norm_w;       // T [dvp] or null; retention with joint_ss: T [H * dvp]
+  float* joint_ss;          // retention: [M, H], or null for a norm per head
   void* out;                // T, row stride ld_out
   float* state;             // [slots, H, dkp, dvp]
   long long ld_qk, ld_v, ld_gate, ld_out;
@@ -174,14 +177,21 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
     for (int t = warp; t < nt; t += nthr >> 5) {
       float ss = 0.f;
       for (int c = lane; c < p.dvp; c += 32) ss = fmaf(so[t * p.dvp + c], so[t * p.dvp + c], ss);
-      const float r = 1.f / sqrtf(warp_sum(ss) / p.dv + p.eps);
+      ss = warp_sum(ss);
       const size_t row = row0 + t0 + t;
+      float r = 1.f / sqrtf(ss / p.dv + p.eps);
+      if (!DELTA && p.joint_ss) {
+        r = 1.f;
+        if (lane == 0) p.joint_ss[row * p.H + h] = ss;
+      }
       for (int c = lane; c < p.dvp; c += 32) {
         float o = so[t * p.dvp + c] * r;
         const size_t gi = row * p.ld_gate + static_cast<size_t>(h) * p.dvp + c;
         if (DELTA) {
           if (p.norm_w) o *= to_f(static_cast<const T*>(p.norm_w)[c]);
           o *= sigmoid_t<T>(static_cast<const float*>(p.gate)[gi]);
+        } else if (p.joint_ss) {
+          o *= to_f(static_cast<const T*>(p.norm_w)[h * p.dvp + c]) * sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
         } else {
           o *= silu_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
         }
@@ -304,13 +314,19 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
   __syncthreads();
   float tot = 0.f;
   for (int w = 0; w < nthr / 32; ++w) tot += so[DV + w];
-  const float r = 1.f / sqrtf(tot / p.dv + p.eps);
+  float r = 1.f / sqrtf(tot / p.dv + p.eps);
+  if (!DELTA && p.joint_ss) {
+    r = 1.f;
+    if (tid == 0) p.joint_ss[row * p.H + h] = tot;
+  }
   for (int c = tid; c < DV; c += nthr) {
     float x = so[c] * r;
     const size_t gi = row * p.ld_gate + static_cast<size_t>(h) * DV + c;
     if (DELTA) {
       if (p.norm_w) x *= to_f(static_cast<const T*>(p.norm_w)[c]);
       x *= sigmoid_t<T>(static_cast<const float*>(p.gate)[gi]);
+    } else if (p.joint_ss) {
+      x *= to_f(static_cast<const T*>(p.norm_w)[h * DV + c]) * sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
     } else {
       x *= silu_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
     }
@@ -633,17 +649,21 @@ static bool bad_heads(const char* what, int H, int group, int dk, int dkp, int d
 
 using namespace b2;
 
+// joint_ss given: norm_w [H * dvp] and a sigmoid gate instead of the norm per head and the silu gate (see above).
 B2_EXPORT int b2_retention_serial(const void* q, const void* k, const void* v, const void* gate, void* out, float* state,
                                   const float* decay, const float* cs, const float* sn, const int* cu, const int* start,
                                   const int* slot, int nseq, int max_rows, int H, int dk, int dkp, int dv, int dvp, int rot,
-                                  long long ld_in, long long ld_out, float kscale, float eps, int is_f32, void* stream) {
+                                  long long ld_in, long long ld_out, float kscale, float eps, const void* norm_w,
+                                  float* joint_ss, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (nseq <= 0) return 0;
+  if (joint_ss != nullptr && norm_w == nullptr) { set_error("retention: a joint norm needs its weight"); return 10; }
   if (bad_heads("retention", H, 1, dk, dkp, dv, dvp, nseq)) return 10;
   if (rot < 0 || rot % 2 || rot > dk) { set_error("retention: rotary dims must be even and at most the head size"); return 10; }
   SerialParams p = {};
   p.seq = {cu, start, slot};
   p.q = q; p.k = k; p.v = v; p.gate = gate; p.cs = cs; p.sn = sn; p.decay = decay; p.out = out; p.state = state;
+  p.norm_w = norm_w; p.joint_ss = joint_ss;
   p.ld_qk = p.ld_v = p.ld_gate = ld_in; p.ld_out = ld_out;
   p.H = H; p.group = 1; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.rot = rot; p.kscale = kscale; p.eps = eps;
   p.tile = max_rows < 16 ? (max_rows < 1 ? 1 : max_rows) : 16;

@@ -23,13 +23,17 @@ __device__ __forceinline__ float res_block_sum(float v, float* scratch) {
 
 template <typename T>
 __global__ void __launch_bounds__(RES_THREADS) embed_f32_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
-                                                                float* __restrict__ x, int ld, int vocab) {
+                                                                float* __restrict__ x, T* __restrict__ h, int ld, int vocab,
+                                                                float scale) {
   const long long id = ids[blockIdx.x];
   const bool ok = id >= 0 && id < vocab;   // padding rows of a graph batch carry any id; nothing outside the table is read
   for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
     float f[8] = {};
     if (ok) vload8(table + static_cast<size_t>(id) * ld + c, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] *= scale;
     vstore8(x + static_cast<size_t>(blockIdx.x) * ld + c, f);
+    if (h) vstore8(h + static_cast<size_t>(blockIdx.x) * ld + c, f);
   }
 }
 
@@ -68,6 +72,64 @@ __global__ void __launch_bounds__(RES_THREADS) rmsnorm_f32_kernel(const float* _
 #pragma unroll
     for (int e = 0; e < 8; ++e) t[e] *= r * wv[e];
     vstore8(hr + c, t);
+  }
+}
+
+// x <- rms(alpha x + f y + b) w, and the same rounded to T in h (optional).  y: fp32 [M, ld]; b (optional): T [ld]; f is 1, or
+// the root of a norm over the reader's input that was left to this kernel: 1 / sqrt(sum_j ss[row, j] / nss + eps).
+template <typename T>
+__global__ void __launch_bounds__(RES_THREADS) post_norm_kernel(float* __restrict__ x, const float* __restrict__ y,
+                                                                const T* __restrict__ w, const T* __restrict__ b,
+                                                                const float* __restrict__ ss, int parts, int nss,
+                                                                T* __restrict__ h, int ld, int n, float alpha, float eps) {
+  __shared__ float scratch[32];
+  const size_t base = static_cast<size_t>(blockIdx.x) * ld;
+  float f = 1.f;
+  if (ss) {
+    float t = 0.f;
+    for (int j = 0; j < parts; ++j) t += ss[static_cast<size_t>(blockIdx.x) * parts + j];
+    f = 1.f / sqrtf(t / nss + eps);
+  }
+  auto piece = [&](int c, float (&s)[8]) {
+    float t[8];
+    vload8(x + base + c, s);
+    vload8(y + base + c, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s[e] = fmaf(alpha, s[e], f * t[e]);
+    if (b) {
+      vload8(b + c, t);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s[e] += t[e];
+    }
+  };
+  float v[RES_VEC][8], sum = 0.f;
+  int i = 0;
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8, ++i) {
+    float t[8];
+    piece(c, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum = fmaf(t[e], t[e], sum);
+#pragma unroll
+    for (int k = 0; k < RES_VEC; ++k)
+      if (k == i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = t[e];
+  }
+  const float r = 1.f / sqrtf(res_block_sum(sum, scratch) / n + eps);
+  i = 0;
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8, ++i) {
+    float t[8], wv[8];
+    if (i >= RES_VEC) piece(c, t);
+#pragma unroll
+    for (int k = 0; k < RES_VEC; ++k)
+      if (k == i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) t[e] = v[k][e];
+    vload8(w + c, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) t[e] *= r * wv[e];
+    vstore8(x + base + c, t);
+    if (h) vstore8(h + base + c, t);
   }
 }
 
@@ -153,7 +215,7 @@ __global__ void __launch_bounds__(RES_THREADS) rope_rows_kernel(const int* __res
 constexpr int SG_T = 64, SG_K = 16;
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B,
                                                        float* __restrict__ C, int M, int N, int K, int lda, int ldb, int ldc,
-                                                       int accumulate) {
+                                                       int accumulate, int act, int act_cols) {
   __shared__ float sA[SG_K][SG_T + 4], sB[SG_K][SG_T + 4];
   const int m0 = blockIdx.y * SG_T, n0 = blockIdx.x * SG_T;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -187,7 +249,9 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       float* c = C + static_cast<size_t>(m) * ldc + n;
-      *c = accumulate ? *c + acc[i][j] : acc[i][j];
+      float r = accumulate ? *c + acc[i][j] : acc[i][j];
+      if (act != 0 && n < act_cols) r = act == GEMM_ACT_SILU ? silu_f(r) : fmaxf(r, 0.f) * fmaxf(r, 0.f);
+      *c = r;
     }
   }
 }
@@ -196,12 +260,14 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 
 using namespace b2;
 
-B2_EXPORT int b2_embed_f32(const long long* ids, const void* table, float* x, int M, int ld, int vocab, int is_f32, void* stream) {
+// h (optional): the same rows in the table's type.
+B2_EXPORT int b2_embed_f32(const long long* ids, const void* table, float* x, void* h, int M, int ld, int vocab, float scale,
+                           int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (ld % 8) { set_error("embed_f32: row width must be a multiple of 8"); return 10; }
   B2_DISPATCH_T(is_f32, embed_f32_kernel<T><<<M, RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
-      ids, static_cast<const T*>(table), x, ld, vocab););
+      ids, static_cast<const T*>(table), x, static_cast<T*>(h), ld, vocab, scale););
   B2_CHECK_LAUNCH("embed_f32");
   return 0;
 }
@@ -214,6 +280,22 @@ B2_EXPORT int b2_rmsnorm_f32(const float* x, const void* w, void* h, const long 
   B2_DISPATCH_T(is_f32, rmsnorm_f32_kernel<T><<<M, RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
       x, static_cast<const T*>(w), static_cast<T*>(h), rows, ld, n, eps););
   B2_CHECK_LAUNCH("rmsnorm_f32");
+  return 0;
+}
+
+B2_EXPORT int b2_post_norm(float* x, const float* y, const void* w, const void* b, const float* ss, int parts, int nss, void* h,
+                           int M, int ld, int n, float alpha, float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld || (ss != nullptr && (parts < 1 || nss < 1))) {
+    set_error("post_norm: ld %% 8 == 0 and 0 < n <= ld required");
+    return 10;
+  }
+  int threads = (ld / 8 + 31) / 32 * 32;
+  if (threads > RES_THREADS) threads = RES_THREADS;
+  B2_DISPATCH_T(is_f32, post_norm_kernel<T><<<M, threads, 0, static_cast<cudaStream_t>(stream)>>>(
+      x, y, static_cast<const T*>(w), static_cast<const T*>(b), ss, parts, nss, static_cast<T*>(h), ld, n, alpha, eps););
+  B2_CHECK_LAUNCH("post_norm");
   return 0;
 }
 
@@ -259,12 +341,13 @@ B2_EXPORT int b2_rope_rows(const int* pos, const double* turns, float* cs, float
 }
 
 B2_EXPORT int b2_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldb, int ldc,
-                          int accumulate, void* stream) {
+                          int accumulate, int act, int act_cols, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const dim3 grid((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T);
   if (grid.y > 65535) { set_error("gemm_f32: too many rows (%d)", M); return 10; }
-  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, B, C, M, N, K, lda, ldb, ldc, accumulate);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, B, C, M, N, K, lda, ldb, ldc, accumulate, act,
+                                                                     act_cols);
   B2_CHECK_LAUNCH("gemm_f32");
   return 0;
 }

@@ -3,6 +3,7 @@
 //   1. every chunk's own contribution to the state, K^T V with the decays to the chunk's end       (all chunks at once)
 //   2. the running state at every chunk's start: S_c = a^n S_{c-1} + contribution                   (a scan, element-wise)
 //   3. o = a^{t+1} S_c^T q + sum_{j <= t} a^{t-j} (q . k_j) v_j, per-head norm, gate, store         (all chunks at once)
+//      (or, for heads that are normed together, weight, sigmoid gate, store and each head's sum of squares)
 //
 // The products are tcgen05 MMAs of one 128-token tile with fp32 accumulators in TMEM.  An fp32 operand that enters the
 // recurrence or weighs a value (k, the state, the weights) is the sum of two bf16 numbers, hi + lo, and takes two MMAs;
@@ -33,6 +34,8 @@ struct RetParams {
   const int* first;     // [nlong + 1] first chunk of each long sequence
   const int* start;     // [nseq]
   const int* slot;      // [nseq]
+  const bf16_t* norm_w; // joint norm: [H * dvp]
+  float* joint_ss;      // [M, H] sums of squares for the reader, or null: a norm per head and a silu gate
   long long ld_in, ld_out;
   int H, dk, dkp, dv, dvp, rot, seq0;
   float kscale, eps;
@@ -457,8 +460,10 @@ __global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams
   }
   xchg[half * 128 + r] = ss;
   __syncthreads();
+  const float tot = xchg[r] + xchg[128 + r];
+  if (p.joint_ss && half == 0 && r < n) p.joint_ss[(row0 + r) * p.H + h] = tot;
   if (mine) {
-    const float f = 1.f / sqrtf((xchg[r] + xchg[128 + r]) / p.dv + p.eps);
+    const float f = p.joint_ss ? 1.f : 1.f / sqrtf(tot / p.dv + p.eps);
     uint4 ov[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -467,6 +472,12 @@ __global__ void __launch_bounds__(RET_THREADS, 2) ret_out_kernel(const RetParams
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float2 g2 = unpack_bf16x2(g[e]);
+        if (p.joint_ss) {
+          const int c = half * 64 + j * 8 + 2 * e;
+          const float2 w2 = c < p.dvp ? unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p.norm_w + h * p.dvp + c)) : make_float2(0.f, 0.f);
+          y[e] = pack_bf16x2(o[j * 8 + 2 * e] * w2.x * sigmoid_fast(g2.x), o[j * 8 + 2 * e + 1] * w2.y * sigmoid_fast(g2.y));
+          continue;
+        }
         y[e] = pack_bf16x2(o[j * 8 + 2 * e] * f * silu_fast(g2.x), o[j * 8 + 2 * e + 1] * f * silu_fast(g2.y));
       }
       ov[j] = make_uint4(y[0], y[1], y[2], y[3]);
@@ -512,8 +523,9 @@ B2_EXPORT int b2_retention_chunk(const void* q, const void* k, const void* v, co
                                  float* state, const float* decay, const float* cs, const float* sn, const int* chunks,
                                  const int* first, const int* start, const int* slot, int nchunks, int seq0, int nlong, int H,
                                  int dk, int dkp, int dv, int dvp, int rot, long long ld_in, long long ld_out, float kscale,
-                                 float eps, void* stream) {
+                                 float eps, const void* norm_w, float* joint_ss, void* stream) {
   b2::ensure_thread_context();
+  if (joint_ss != nullptr && norm_w == nullptr) { set_error("retention_chunk: a joint norm needs its weight"); return 10; }
   if (nchunks <= 0 || nlong <= 0) return 0;
   if (dkp % 8 || dvp % 8 || dkp < 8 || dvp < 8 || dkp > 128 || dvp > 128 || rot < 0 || rot % 2 || rot > dk || ld_in % 8 ||
       ld_out % 8 || H < 1 || H > 65535 || nlong > 65535) {
@@ -525,6 +537,7 @@ B2_EXPORT int b2_retention_chunk(const void* q, const void* k, const void* v, co
   p.gate = static_cast<const bf16_t*>(gate); p.out = static_cast<bf16_t*>(out); p.ws = ws; p.state = state; p.decay = decay;
   p.cs = cs; p.sn = sn; p.chunks = chunks; p.first = first; p.start = start; p.slot = slot; p.ld_in = ld_in; p.ld_out = ld_out;
   p.H = H; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.rot = rot; p.seq0 = seq0; p.kscale = kscale; p.eps = eps;
+  p.norm_w = static_cast<const bf16_t*>(norm_w); p.joint_ss = joint_ss;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return launch_ret(p, nchunks, nlong, st);
 }

@@ -51,10 +51,52 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 // Forms for values that are rounded to bf16 next (relative error about 2^-21): one special-function 2^x and one reciprocal.
 __device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + fast_exp2(-1.4426950408889634f * z)); }
 __device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + fast_exp2(-1.4426950408889634f * z)); }
+// silu of two values with one reciprocal between them: 1 / (a b) gives 1 / a and 1 / b.  The exponent is bounded so that
+// the product stays finite; past the bound the result is below 1e-17.
+__device__ __forceinline__ void silu_pair_fast(float& x, float& y) {
+  const float a = 1.f + fast_exp2(fminf(-1.4426950408889634f * x, 62.f)), b = 1.f + fast_exp2(fminf(-1.4426950408889634f * y, 62.f));
+  const float r = __fdividef(1.f, a * b);
+  x *= r * b;
+  y *= r * a;
+}
 template <typename T>
 __device__ __forceinline__ float silu_t(float z) { return sizeof(T) == 2 ? silu_fast(z) : silu_f(z); }
 template <typename T>
 __device__ __forceinline__ float sigmoid_t(float z) { return sizeof(T) == 2 ? sigmoid_fast(z) : sigmoid_f(z); }
+
+// cap * tanh(z) for a score s = cap * z pressed softly into (-cap, cap).  Near zero: the Taylor series of tanh (relative error
+// below 1e-7 for |z| <= SOFTCAP_SERIES); elsewhere 1 - 2 / (1 + e^{2 z}), whose absolute error is a rounding of 1.
+constexpr float SOFTCAP_SERIES = 0.4f;
+__device__ __forceinline__ float tanh_series(float z) {
+  const float t = z * z;
+  float r = fmaf(t, 21844.f / 6081075.f, -1382.f / 155925.f);
+  r = fmaf(t, r, 62.f / 2835.f);
+  r = fmaf(t, r, -17.f / 315.f);
+  r = fmaf(t, r, 2.f / 15.f);
+  r = fmaf(t, r, -1.f / 3.f);
+  return fmaf(z * t, r, z);
+}
+__device__ __forceinline__ float tanh_wide(float z) {
+  return 1.f - 2.f * __fdividef(1.f, 1.f + fast_exp2(fminf(2.f * 1.4426950408889634f * z, 126.f)));
+}
+template <typename T>
+__device__ __forceinline__ float softcap_t(float s, float cap) {
+  const float z = s / cap;
+  if (sizeof(T) == 4) return cap * tanhf(z);
+  return cap * (fabsf(z) <= SOFTCAP_SERIES ? tanh_series(z) : tanh_wide(z));
+}
+
+// Weight of the second map of differential attention: exp(lq1 . lk1) - exp(lq2 . lk2) + init, by a whole warp.
+// lam: [4, ld] = lq1, lk1, lq2, lk2, zero past the head size.
+template <typename T>
+__device__ __forceinline__ float diff_lambda(const T* lam, int ld, float init) {
+  float a = 0.f, b = 0.f;
+  for (int c = threadIdx.x & 31; c < ld; c += 32) {
+    a = fmaf(to_f(lam[c]), to_f(lam[ld + c]), a);
+    b = fmaf(to_f(lam[2 * ld + c]), to_f(lam[3 * ld + c]), b);
+  }
+  return expf(warp_sum(a)) - expf(warp_sum(b)) + init;
+}
 
 }  // namespace b2
 
