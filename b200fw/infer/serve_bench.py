@@ -224,6 +224,91 @@ def fetelorn_kernels(preset: str, lengths: Optional[List[int]] = None, batch: in
     return t.rows
 
 
+def sotazen_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    """The same for the differential / latent / lightning decoder."""
+    mc, t = PRESETS[preset], _Timer()
+    W, V, eps = mc.hidden_size, mc.vocab_size, mc.rms_norm_eps
+    kinds = {k: next(l for l in mc.layers if l["type"] == k) for k in ("lightning", "attention", "latent_attention")}
+    ff = kinds["lightning"]["mlp"]["ff"]
+    p, pages, starts, counts = _layout(lengths, batch, ctx)
+    M, n = p.rows, p.nseq
+    x, y32, w, h = torch.randn(M, W, device=DEV), torch.randn(M, W, device=DEV), _bf(W), _bf(M, W)
+    t("post_norm", lambda: ops.post_norm(x, y32, w, 1.5, W, eps), M * W * 14)
+
+    def act(name, N, cols, kind):
+        wt = _bf(N, W)
+        t(name, lambda: ops.linear_act(h, wt, kind, cols), 2 * (M * W + N * W + M * N), 2.0 * M * N * W)
+    act("gemm up, relu^2", ff, ff, "relu2")
+    _gemm(t, "gemm down (fp32)", M, W, ff, True)
+
+    m = kinds["lightning"]["mixer"]
+    H, dk, dv = m["heads"], m["dim"], m["vdim"]
+    c = [0, H * dk, 2 * H * dk, 2 * H * dk + H * dv, 2 * H * (dk + dv)]
+    act("gemm in (lightning), silu", c[4], c[3], "silu")
+    y, out = _bf(M, c[4]), _bf(M, H * dv)
+    S, dec, ss = torch.zeros(n, H, dk, dv, device=DEV), torch.tensor(m["decay"], device=DEV), torch.empty(M, H, device=DEV)
+    nw = _bf(H * dv)
+    flops = M * H * (2.0 * 64 * (dk + dv) / 2 + 4.0 * dk * dv)
+    state = n * H * dk * dv * 4 * (1 if lengths else 2)
+    t("lightning", lambda: ops.retention(*(y[:, c[i]:c[i + 1]] for i in range(4)), out, S, p, dec, dk, dv, None, None, 1.0, eps, nw, ss),
+      M * H * (2 * dk + 3 * dv) * 2 + state, flops if lengths else 0)
+    _gemm(t, "gemm lightning o (fp32)", M, W, H * dv, True)
+
+    a = kinds["attention"]["mixer"]
+    H, G, dk, dv, win = a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["mask"]["size"]
+    lq, lk, lv = 2 * H * dk, 2 * G * dk, G * dv
+    _gemm(t, "gemm in (differential)", M, lq + lk + lv + H * dv, W)
+    kc, vc = _bf(pages, 16, 2 * G, dk), _bf(pages, 16, G, dv)
+    yy, wd, bias = _bf(M, lq + lk + lv + H * dv), _bf(dk), _bf(lq + lk + lv)
+    cs, sn = ops.rope_rows(p.positions, ops.rope_turns(1e4, a["rot"]["dims"], DEV))
+
+    def store():
+        return ops.qk_norm_store(yy[:, :lq], yy[:, lq:lq + lk], yy[:, lq + lk:lq + lk + lv], kc, vc, p, 2 * H, dk, True, eps, wd, wd,
+                                 bias, cs, sn)
+    t("qk_norm_store (bias, rotation)", store, M * ((lq + lk + lv) * 4 + a["rot"]["dims"] * 4))
+    q, lam, gate, out = store(), _bf(4, dk), yy[:, lq + lk + lv:], _bf(M, H * dv)
+    seen = sum(min(i + 1, win) for s, k in zip(starts, counts) for i in range(s, s + k))          # query-key pairs
+    t("differential_attention", lambda: ops.differential_attention(q, kc, vc, out, p, H, a["scale"], lam, a["diff"], dv, eps, gate, win,
+                                                                   a["softcap"]),
+      M * (lq + 2 * H * dv) * 2 + (seen if lengths is None else M) * (lk + lv) * 2, 2.0 * seen * 2 * H * (dk + dv))
+    _gemm(t, "gemm differential o (fp32)", M, W, H * dv, True)
+
+    b = kinds["latent_attention"]["mixer"]
+    H, d, r, dv, C = b["heads"], b["dim"], b["rot_dim"], b["vdim"], b["kv_rank"]
+    dq, R = d + r, C + r
+    _gemm(t, "gemm in (latent)", M, H * dq + R, W)
+    yy, pg = _bf(M, H * dq + R), _bf(pages, 16, 1, R)
+    cs, sn = ops.rope_rows(p.positions, ops.rope_turns(1e4, r, DEV))
+    wc, w_key, w_value, sink, out = _bf(C), _bf(H, dq, R), _bf(H, dv, C), _bf(H), _bf(M, H * dv)
+    q, cc, kr = yy[:, :H * dq], yy[:, H * dq:H * dq + C], yy[:, H * dq + C:]
+    t("latent_store", lambda: ops.latent_store(q, cc, kr, pg, p, H, d, C, r, wc, cs, sn, eps), M * (H * r * 4 + R * 4 + r * 4))
+    pairs = sum((s + k) * (s + k + 1) / 2 - s * (s + 1) / 2 for s, k in zip(starts, counts))
+    if lengths is None:
+        ql, ol = _bf(M, H * R), _bf(M, H * C)
+        t("head_linear (queries to latent)", lambda: ops.head_linear(q, w_key, ql, True), (M * H * (dq + R) + H * dq * R) * 2)
+        t("latent_rows", lambda: ops.latent_rows(ql, pg, ol, p, H, C, b["scale"], sink), (pairs * R + M * H * (R + C)) * 2,
+          2.0 * pairs * H * (R + C))
+        t("head_linear (latent to values)", lambda: ops.head_linear(ol, w_value, out), (M * H * (dv + C) + H * dv * C) * 2)
+    else:
+        _gemm(t, "gemm keys from latents", M, H * dq, R)
+        _gemm(t, "gemm values from latents", M, H * dv, C)
+    t("latent_attention", lambda: ops.latent_attention(q, pg, out, p, w_key, w_value, b["scale"], sink),
+      M * H * (dq + dv) * 2 + (pairs if lengths is None else M) * R * 2,
+      2.0 * pairs * H * (R + C) if lengths is None else 2.0 * (pairs * H * (dq + dv) + M * H * (dq * R + dv * C)))
+    if lengths is not None:
+        from ..ops import latent
+        k, v = _bf(pages * 16, H * dq), _bf(pages * 16, H * dv)
+        t("latent prompt attention alone", lambda: latent.expanded_attention(q, k, v, out, p, H, dq, dv, b["scale"], sink, 0, n, p.ctx_tables),
+          M * H * (dq + dv) * 4, 2.0 * pairs * H * (dq + dv))
+        rows = torch.empty(pages * 16, R, device=DEV, dtype=torch.bfloat16)
+        t("latent_gather", lambda: latent.gather(pg, p.ctx_pages, rows), rows.numel() * 4)
+    _gemm(t, "gemm latent o (fp32)", M, W, H * dv, True)
+    if lengths is None:
+        _gemm(t, "gemm logits (fp32)", M, V, W, True)
+    del t.flush
+    return t.rows
+
+
 def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
     """The same for the dense decoder family."""
     mc, t = PRESETS[preset], _Timer()
@@ -266,6 +351,6 @@ def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int =
 
 
 def kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    by_name = {"Fetelorn": fetelorn_kernels, "Sotazen": sotazen_kernels}
     with torch.no_grad():
-        f = fetelorn_kernels if hasattr(PRESETS[preset], "kv_bytes_per_token") else dense_kernels
-        return f(preset, lengths, batch, ctx)
+        return by_name.get(getattr(PRESETS[preset], "architecture", None), dense_kernels)(preset, lengths, batch, ctx)

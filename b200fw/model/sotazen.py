@@ -248,6 +248,6 @@ SOTAZEN_PRESETS = {
     "sotazen-tiny": sotazen_preset(256, 2, 4, 512, 1024, 1, window=64, rank=64, dim=64, rot=32),
     # the widths, depth and vocabulary of the framework's dense presets of the same size; the feed-forward, which has two matrices
     # instead of three, is wider
-    "sotazen-0.6b": sotazen_preset(1024, 8, 28, 4608, 151936, 4),
-    "sotazen-4b": sotazen_preset(2560, 16, 36, 14592, 151936, 4),
+    "sotazen-0.6b": sotazen_preset(1024, 8, 28, 5120, 151936, 4),
+    "sotazen-4b": sotazen_preset(2560, 16, 36, 15104, 151936, 4),
 }

@@ -130,7 +130,7 @@ def _expanded(q, pages, out, p: Portions, w_key, w_value, scale, sink, max_pages
     """The long portions: their contexts' rows in token order, keys and values of all heads from them, tensor-core attention."""
     H, dqp, Rp = w_key.shape
     dvp, Cp = w_value.shape[1:]
-    ns, counts, a, first = p.num_short, p.ctx_counts, 0, 0
+    counts, a, first = p.ctx_counts, 0, 0
     assert out.stride(0) % 8 == 0 and pages.is_contiguous()
     while a < len(counts):
         b, n = a, 0
@@ -138,17 +138,27 @@ def _expanded(q, pages, out, p: Portions, w_key, w_value, scale, sink, max_pages
             n += counts[b]
             b += 1
         rows = torch.empty((n * 16, Rp), device=q.device, dtype=q.dtype)
-        nv.check(nv.lib().b2_latent_gather(nv.ptr(pages), nv.ptr(p.ctx_pages[first:]), nv.ptr(rows), n, 16 * Rp * rows.element_size(),
-                                           nv.stream_ptr()), "latent_gather")
-        nv.count_launch()
+        gather(pages, p.ctx_pages[first:first + n], rows)
         k = gemm(rows, w_key.view(H * dqp, Rp))
         v = gemm(rows[:, :Cp], w_value.view(H * dvp, Cp))
         tables = p.ctx_tables[a:b] if first == 0 else p.ctx_tables[a:b] - first
-        nv.check(nv.lib().b2_attn_fwd_paged_ext(
-            nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(out), nv.ctypes.c_longlong(out.stride(0)), b - a, H, H, dqp, dvp, n,
-            nv.ctypes.c_float(scale), nv.ptr(p.cu[ns + a:]), nv.ptr(p.starts[ns + a:]), nv.ptr(tables), tables.shape[1], p.max_long,
-            p.rows, 0, None, None, 0, nv.ptr(sink), None, nv.ctypes.c_longlong(0), nv.ctypes.c_longlong(q.stride(0)), 0,
-            nv.ctypes.c_float(0.0), 1, None, nv.ctypes.c_float(0.0), nv.ctypes.c_float(0.0), 0, None, nv.stream_ptr()),
-            "attn_fwd_paged_ext")
-        nv.count_launch()
+        expanded_attention(q, k, v, out, p, H, dqp, dvp, scale, sink, a, b, tables)
         a, first = b, first + n
+
+
+def gather(pages: torch.Tensor, ids: torch.Tensor, rows: torch.Tensor) -> None:
+    """Pages ``ids`` of the pool one after the other: ``rows [16 n, Rp]``."""
+    nv.check(nv.lib().b2_latent_gather(nv.ptr(pages), nv.ptr(ids), nv.ptr(rows), ids.numel(), 16 * rows.shape[1] * rows.element_size(),
+                                       nv.stream_ptr()), "latent_gather")
+    nv.count_launch()
+
+
+def expanded_attention(q, k, v, out, p: Portions, H: int, dqp: int, dvp: int, scale: float, sink, a: int, b: int, tables) -> None:
+    """Long portions ``a .. b - 1`` over keys and values laid out by ``tables`` in pages of 16 rows."""
+    ns, cf, cl = p.num_short, nv.ctypes.c_float, nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_attn_fwd_paged_ext(
+        nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(out), cl(out.stride(0)), b - a, H, H, dqp, dvp, k.shape[0] // 16, cf(scale),
+        nv.ptr(p.cu[ns + a:]), nv.ptr(p.starts[ns + a:]), nv.ptr(tables), tables.shape[1], p.max_long, p.rows, 0, None, None, 0,
+        nv.ptr(sink), None, cl(0), cl(q.stride(0)), 0, cf(0.0), 1, None, cf(0.0), cf(0.0), 0, None, nv.stream_ptr()),
+        "attn_fwd_paged_ext")
+    nv.count_launch()
