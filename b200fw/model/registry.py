@@ -86,7 +86,7 @@ ARCHITECTURES: Dict[str, Architecture] = {
                              ("host", "gemm", "residual", "linear_state", "retention_chunk", "delta_chunk", "attention_rows", "attention_fwd", "sampling"), float32=True),
     "Sotazen": Architecture("Sotazen", SotazenConfig, lambda path: SotazenConfig.from_dict(_config_json(path)), SotazenModel,
                             _load_slots_at, ("host", "gemm", "residual", "linear_state", "retention_chunk", "attention_rows",
-                                             "attention_latent", "attention_fwd", "sampling"), float32=True),
+                                             "attention_decode", "attention_latent", "attention_fwd", "sampling"), float32=True),
 }
 PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS, **SOTAZEN_PRESETS}
 

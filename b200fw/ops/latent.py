@@ -12,7 +12,7 @@ import torch
 
 from .. import _native as nv
 from .gemm import gemm
-from .paged_rows import _split
+from .paged_rows import _split, decode_attention
 from .portions import Portions
 
 MAX_EXPANDED_BYTES = 4 << 30     # keys and values of long portions' contexts, made at once
@@ -104,7 +104,9 @@ def latent_rows(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, p: Port
                 sink: Optional[torch.Tensor]) -> None:
     """Attention of the first rows of the step in the latent space: ``q [m, H*Rp]`` -> ``out [m, H*Cp]``."""
     m, Rp = q.shape[0], pages.shape[-1]
-    part, nsplit = _split_rows(m * ((H + 15) // 16), p.max_keys, Rp) if q.dtype == torch.bfloat16 else (max(1, p.max_keys), 1)
+    if q.dtype == torch.bfloat16 and decode_attention(q, pages, None, out, p, m, H, 1, Rp, Cp, scale, sink):
+        return
+    part, nsplit = _split(m * H, 1, 1, p.max_keys)
     po = pm = None
     if nsplit > 1:
         po = torch.empty((m, H, nsplit, Cp), device=q.device, dtype=torch.float32)
@@ -114,16 +116,6 @@ def latent_rows(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, p: Port
         nv.ptr(out), nv.ptr(po), nv.ptr(pm), m, p.block_tables.shape[1], H, Rp, Cp, part, nsplit, nv.ctypes.c_float(scale),
         int(q.dtype == torch.float32), nv.stream_ptr()), "latent_rows")
     nv.count_launch(2 if nsplit > 1 else 1)
-
-
-def _split_rows(ctas: int, keys: int, Rp: int):
-    """Keys per split and number of splits: whole waves of resident CTAs while a split keeps at least 128 keys."""
-    resident = 148 * (2 if Rp <= 320 else 1)
-    n = max(1, min((keys + 127) // 128, -(-2 * resident // max(1, ctas))))
-    if n == 1:
-        return max(1, keys), 1
-    part = ((keys + n - 1) // n + 63) // 64 * 64
-    return part, (keys + part - 1) // part
 
 
 def _expanded(q, pages, out, p: Portions, w_key, w_value, scale, sink, max_pages: int) -> None:

@@ -171,6 +171,9 @@ def _attention(q, k_cache, v_cache, out, p, H, scale, chunk, rel, bucket, sink, 
         nv.count_launch()
     if lead == 0:
         return
+    if q.dtype == torch.bfloat16 and lam is not None and decode_attention(
+            q, k_cache, v_cache, out, p, lead, H, G, maps * dkp, dvp, scale, None, gate, window, softcap, lam, lam_init, eps, dv):
+        return
     assert q.is_contiguous()
     keys = min(p.max_keys, chunk or window or p.max_keys)
     most = 4 // maps
@@ -186,6 +189,33 @@ def _attention(q, k_cache, v_cache, out, p, H, scale, chunk, rel, bucket, sink, 
         nv.ptr(po), nv.ptr(pm), lead, p.block_tables.shape[1], H, G, dkp, dvp, chunk, part, nsplit, cf(scale), window, cf(softcap),
         nv.ptr(lam), cf(lam_init), cf(eps), dv, int(q.dtype == torch.float32), nv.stream_ptr()), "attn_rows")
     nv.count_launch(2 if nsplit > 1 else 1)
+
+
+def decode_attention(q, k_cache, v_cache, out, p: Portions, rows: int, H: int, G: int, R: int, C: int, scale: float, sink, gate=None,
+                     window: int = 0, softcap: float = 0.0, lam=None, lam_init: float = 0.0, eps: float = 0.0, dv: int = 0) -> bool:
+    """The first ``rows`` rows of the step, one query token each, on the tensor cores with the work split evenly over the SMs
+    (csrc/attention_decode.cu).  ``v_cache`` None: a value is the first ``C`` channels of its key row.  False, with nothing done,
+    for sizes the kernel has no form for."""
+    tile = nv.lib().b2_decode_tile(R, C, int(v_cache is not None))
+    if tile == 0:
+        return False
+    key = (rows, window, tile)
+    if key not in p.plans:
+        p.plans[key] = torch.empty(rows + 1, device=q.device, dtype=torch.int32)
+        nv.check(nv.lib().b2_decode_plan(nv.ptr(p.positions), nv.ptr(p.row_seq), nv.ptr(p.slots), nv.ptr(p.plans[key]), rows, window,
+                                         tile, nv.stream_ptr()), "decode_plan")
+        nv.count_launch()
+    n = _sms(q.device)
+    po = torch.empty((n, 2, 16, C), device=q.device, dtype=torch.float32)
+    pm = torch.empty((n, 2, 16, 2), device=q.device, dtype=torch.float32)
+    cf, cl = nv.ctypes.c_float, nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_decode_attention(
+        nv.ptr(q), nv.ptr(k_cache), nv.ptr(v_cache), nv.ptr(p.block_tables), nv.ptr(p.row_seq), nv.ptr(p.positions),
+        nv.ptr(p.plans[key]), nv.ptr(sink), nv.ptr(gate), nv.ptr(lam), nv.ptr(out), nv.ptr(po), nv.ptr(pm), cl(q.stride(0)),
+        cl(0 if gate is None else gate.stride(0)), cl(out.stride(0)), rows, p.block_tables.shape[1], H, G, R, C, window, dv, cf(scale),
+        cf(softcap), cf(lam_init), cf(eps), nv.stream_ptr()), "decode_attention")
+    nv.count_launch(2)
+    return True
 
 
 def _split(rows: int, groups_per_row: int, heads: int, keys: int):

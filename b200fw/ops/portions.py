@@ -1,8 +1,8 @@
 """Row layout of a batch of sequence portions: what every state-carrying or paged op needs to know about a step."""
 from __future__ import annotations
 
-from dataclasses import dataclass
-from typing import List, Optional
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
@@ -41,6 +41,7 @@ class Portions:
     ctx_pages: Optional[torch.Tensor] = None
     ctx_tables: Optional[torch.Tensor] = None
     ctx_counts: Optional[List[int]] = None
+    plans: Dict[Tuple[int, int, int], torch.Tensor] = field(default_factory=dict)    # decode_plan: (rows, window, tile) -> tile counts
     ragged: bool = True                      # False: every sequence is one row (decode): row r is sequence r
 
     @property

@@ -6,8 +6,8 @@
 //   expanded   keys and values of all heads are made from the rows (a GEMM) and attended like ordinary ones: long portions, where
 //              a row serves many queries (latent_gather brings the pages into token order for that GEMM)
 //   absorbed   q_h^T W_uk c = (W_uk^T q_h)^T c, so the query moves into the latent space, every head attends over the same rows,
-//              and W_uv is applied to the result: decoding and short portions (latent_rows, between two products per head,
-//              head_linear)
+//              and W_uv is applied to the result: decoding and short portions (between two products per head, head_linear); in
+//              bf16 by the kernel of attention_decode.cu, in 32-bit and for sizes beyond it by latent_rows here
 // And the stage before either: norm of the latent, rotary positions of the queries' and the key's rotated part, page store.
 #include "host.h"
 #include "mma_split.cuh"
@@ -46,12 +46,31 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(T* __restrict_
   const float* cr = cs + row * half;
   const float* sr = sn + row * half;
   T* qr = q + row * ld;
-  for (int i = tid; i < H * half; i += LS_THREADS) {
-    const int h = i / half, f = i % half;
-    T* at = qr + static_cast<size_t>(h) * dqp + dim + 2 * f;
-    const float u = to_f(at[0]), v = to_f(at[1]), co = cr[f], si = sr[f];
-    at[0] = from_f<T>(u * co - v * si);
-    at[1] = from_f<T>(v * co + u * si);
+  if (dim % 8 == 0 && rot % 8 == 0) {        // four pairs at a time
+    const int per = rot / 8;
+    for (int i = tid; i < H * per; i += LS_THREADS) {
+      const int h = i / per, f = i % per * 4;
+      T* at = qr + static_cast<size_t>(h) * dqp + dim + 2 * f;
+      float t[8];
+      vload8(at, t);
+      const float4 co = *reinterpret_cast<const float4*>(cr + f), si = *reinterpret_cast<const float4*>(sr + f);
+      const float c4[4] = {co.x, co.y, co.z, co.w}, s4[4] = {si.x, si.y, si.z, si.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float u = t[2 * e], v = t[2 * e + 1];
+        t[2 * e] = u * c4[e] - v * s4[e];
+        t[2 * e + 1] = v * c4[e] + u * s4[e];
+      }
+      vstore8(at, t);
+    }
+  } else {
+    for (int i = tid; i < H * half; i += LS_THREADS) {
+      const int h = i / half, f = i % half;
+      T* at = qr + static_cast<size_t>(h) * dqp + dim + 2 * f;
+      const float u = to_f(at[0]), v = to_f(at[1]), co = cr[f], si = sr[f];
+      at[0] = from_f<T>(u * co - v * si);
+      at[1] = from_f<T>(v * co + u * si);
+    }
   }
   if (slot != nullptr && slot[s] < 0) return;
   const int p = pos[row];
@@ -291,186 +310,6 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentRowsParam
   }
 }
 
-// bf16 on the tensor cores: one CTA per (row, 16 heads, split).  The sixteen heads are the rows of an m16n8k16 product (the
-// 128-row tcgen05 tile would be seven eighths padding), a tile of 64 keys its columns, and then the weights times the same tile,
-// whose first Cp channels are the values: every cached byte is read once for all heads.  Eight warps: four groups of 16 keys times
-// two halves of the channels for the scores, 16-channel pieces of the latent for the values.
-constexpr int LR_THREADS = 256, LR_KEYS = 64, LR_HEADS = 16, LR_LDP = LR_KEYS + 8, LR_LDS = LR_KEYS + 4;
-__host__ __device__ constexpr int lr_ld(int Rp) { return (Rp + 15) / 16 * 16 + 8; }
-static int lr_bytes(int Rp) {
-  return (LR_HEADS + 2 * LR_KEYS) * lr_ld(Rp) * 2 + 2 * LR_HEADS * LR_LDS * 4 + LR_HEADS * LR_LDP * 2 + 3 * LR_HEADS * 4;
-}
-
-template <int NG>    // 16-channel pieces of the latent per warp: Cp <= 128 NG
-__global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(const LatentRowsParams p) {
-  extern __shared__ __align__(16) uint8_t la_dyn[];
-  const int R16 = (p.Rp + 15) / 16 * 16, LD = R16 + 8, pieces = R16 / 8;
-  la_bf16* sQ = reinterpret_cast<la_bf16*>(la_dyn);            // [16][LD]
-  la_bf16* sC = sQ + LR_HEADS * LD;                            // [2][64][LD]
-  float* sS = reinterpret_cast<float*>(sC + 2 * LR_KEYS * LD); // [2 channel halves][16][LDS]
-  la_bf16* sP = reinterpret_cast<la_bf16*>(sS + 2 * LR_HEADS * LR_LDS);   // [16][LDP]
-  float* sA = reinterpret_cast<float*>(sP + LR_HEADS * LR_LDP);           // [16] rescale, then [16] max, [16] sum
-  const size_t row = blockIdx.x;
-  const int head0 = blockIdx.y * LR_HEADS, nh = min(LR_HEADS, p.H - head0), split = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row);
-  const bool live = p.slot == nullptr || p.slot[s] >= 0;
-  const int t_begin = split * p.partition, t_end = live ? min(p.pos[row] + 1, t_begin + p.partition) : t_begin;
-  const int* table = p.tables + static_cast<size_t>(s) * p.max_blocks;
-  const la_bf16* pages = static_cast<const la_bf16*>(p.pages);
-
-  auto issue = [&](int st, int t0) {
-    if (t0 < t_end) {
-#pragma unroll
-      for (int i = 0; i < LR_KEYS / 8; ++i) {
-        const int key = warp + 8 * i, t = t0 + key;
-        const bool in = t < t_end;
-        const la_bf16* src = pages + (in ? (static_cast<size_t>(table[t / LA_PAGE]) * LA_PAGE + t % LA_PAGE) * p.Rp : 0);
-        la_bf16* dst = sC + (st * LR_KEYS + key) * LD;
-        for (int c = lane; c < pieces; c += 32) {
-          const bool ok = in && c * 8 < p.Rp;
-          la_copy16(dst + c * 8, src + (ok ? c * 8 : 0), ok);
-        }
-      }
-    }
-    la_commit();
-  };
-  {
-    const la_bf16* q = static_cast<const la_bf16*>(p.q) + (row * p.H + head0) * p.Rp;
-    for (int i = tid; i < LR_HEADS * pieces; i += LR_THREADS) {
-      const int h = i / pieces, c = i % pieces * 8;
-      const bool in = h < nh && c < p.Rp;
-      la_copy16(sQ + h * LD + c, q + (in ? static_cast<size_t>(h) * p.Rp + c : 0), in);
-    }
-  }
-  issue(0, t_begin);          // the queries belong to this group
-  issue(1, t_begin + LR_KEYS);
-
-  const int kg = warp & 3, kh = warp >> 2, steps = R16 / 16;
-  const int k_lo = kh ? (steps + 1) / 2 : 0, k_hi = kh ? steps : (steps + 1) / 2;
-  const int sr = tid >> 4, sk = (tid & 15) * 4;          // softmax: row of scores and first of four keys
-  const float sl2 = p.scale * LA_LOG2E;
-  float m = -INFINITY, l = 0.f;
-  float acc[NG][2][4] = {};
-  int st = 0;
-  for (int t0 = t_begin; t0 < t_end; t0 += LR_KEYS, st ^= 1) {
-    la_wait<1>();
-    __syncthreads();
-    const la_bf16* tile = sC + st * LR_KEYS * LD;
-    {
-      float d[2][2][4] = {};
-      for (int k = k_lo; k < k_hi; k += 2) {
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          if (k + u >= k_hi) break;
-          uint32_t a[4], b[4];
-          ldsm_a_mk(sQ + (k + u) * 16, LD, lane, a);
-          ldsm_b_nk(tile + kg * 16 * LD + (k + u) * 16, LD, lane, b);
-          mma_n16(d[u][0], d[u][1], a, b);
-        }
-      }
-#pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int hh = 0; hh < 2; ++hh) {
-          float* o = sS + (kh * LR_HEADS + (lane >> 2) + 8 * hh) * LR_LDS + kg * 16 + n * 8 + (lane & 3) * 2;
-          *reinterpret_cast<float2*>(o) = make_float2(d[0][n][2 * hh] + d[1][n][2 * hh], d[0][n][2 * hh + 1] + d[1][n][2 * hh + 1]);
-        }
-    }
-    __syncthreads();
-    {
-      const float4 x = *reinterpret_cast<const float4*>(sS + sr * LR_LDS + sk);
-      const float4 y = *reinterpret_cast<const float4*>(sS + (LR_HEADS + sr) * LR_LDS + sk);
-      float v[4] = {(x.x + y.x) * sl2, (x.y + y.y) * sl2, (x.z + y.z) * sl2, (x.w + y.w) * sl2};
-      float mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        if (t0 + sk + e >= t_end) v[e] = -INFINITY;
-        mx = fmaxf(mx, v[e]);
-      }
-#pragma unroll
-      for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float mn = fmaxf(m, mx), alpha = fast_exp2(m - mn);    // a tile has at least one key
-      float ps = 0.f;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        v[e] = fast_exp2(v[e] - mn);
-        ps += v[e];
-      }
-#pragma unroll
-      for (int o = 8; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
-      l = l * alpha + ps;
-      m = mn;
-      *reinterpret_cast<uint2*>(sP + sr * LR_LDP + sk) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
-      if (sk == 0) sA[sr] = alpha;
-    }
-    __syncthreads();
-    {
-      const float a0 = sA[lane >> 2], a1 = sA[(lane >> 2) + 8];
-#pragma unroll
-      for (int g = 0; g < NG; ++g)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          acc[g][n][0] *= a0;
-          acc[g][n][1] *= a0;
-          acc[g][n][2] *= a1;
-          acc[g][n][3] *= a1;
-        }
-#pragma unroll
-      for (int ks = 0; ks < LR_KEYS / 16; ++ks) {
-        uint32_t a[4];
-        ldsm_a_mk(sP + ks * 16, LR_LDP, lane, a);
-#pragma unroll
-        for (int g = 0; g < NG; ++g) {
-          const int c = (warp + 8 * g) * 16;
-          if (c >= p.Cp) break;
-          uint32_t b[4];
-          ldsm_b_kn(tile + ks * 16 * LD + c, LD, lane, b);
-          mma_n16(acc[g][0], acc[g][1], a, b);
-        }
-      }
-    }
-    __syncthreads();
-    issue(st, t0 + 2 * LR_KEYS);
-  }
-  la_wait<0>();
-  if (sk == 0) {
-    sA[16 + sr] = m;
-    sA[32 + sr] = l;
-  }
-  __syncthreads();
-#pragma unroll
-  for (int hh = 0; hh < 2; ++hh) {
-    const int r = (lane >> 2) + 8 * hh, head = head0 + r;
-    if (r >= nh) continue;
-    const size_t at = (row * p.H + head) * p.nsplit + split;
-    const float f = p.nsplit == 1 ? la_sink<la_bf16>(p, head, sA[16 + r], sA[32 + r]) : 1.f;
-#pragma unroll
-    for (int g = 0; g < NG; ++g)
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        const int c = (warp + 8 * g) * 16 + n * 8 + (lane & 3) * 2;
-        if (c >= p.Cp) continue;
-        const float x = acc[g][n][2 * hh] * f, y = acc[g][n][2 * hh + 1] * f;
-        if (p.nsplit == 1) *reinterpret_cast<uint32_t*>(static_cast<la_bf16*>(p.out) + (row * p.H + head) * p.Cp + c) = pack_bf16x2(x, y);
-        else *reinterpret_cast<float2*>(p.part_o + at * p.Cp + c) = make_float2(x, y);
-      }
-    if (p.nsplit > 1 && warp == 0 && (lane & 3) == 0) {
-      p.part_ml[at * 2] = sA[16 + r];
-      p.part_ml[at * 2 + 1] = sA[32 + r];
-    }
-  }
-}
-
-template <typename K>
-static int la_smem(K kern, int bytes, const char* what) {
-  if (bytes > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess) {
-    set_error("%s: cannot set shared memory size (%d)", what, bytes);
-    return 1;
-  }
-  return 0;
-}
-
 }  // namespace b2
 
 using namespace b2;
@@ -542,28 +381,14 @@ B2_EXPORT int b2_latent_rows(const void* q, const void* pages, const int* tables
   LatentRowsParams p = {q, pages, tables, row_seq, pos, slot, sink, out, part_o, part_ml, max_blocks, H, Rp, Cp, partition, nsplit,
                         scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (!is_f32 && Cp <= 512 && lr_bytes(Rp) <= 232448) {
-    const dim3 grid(M, (H + LR_HEADS - 1) / LR_HEADS, nsplit);
-    const int smem = lr_bytes(Rp);
-#define B2_LR(NGV)                                                                \
-  do {                                                                            \
-    if (int rc = la_smem(latent_rows_kernel<NGV>, smem, "latent_rows")) return rc; \
-    latent_rows_kernel<NGV><<<grid, LR_THREADS, smem, st>>>(p);                   \
-  } while (0)
-    if (Cp <= 128) B2_LR(1);
-    else if (Cp <= 256) B2_LR(2);
-    else B2_LR(4);
-#undef B2_LR
-  } else {
-    const dim3 grid(M, H, nsplit);
-    B2_DISPATCH_T(is_f32, {
-      if (Rp <= 256) {
-        latent_rows_any_kernel<T, 8><<<grid, LR_ANY_WARPS * 32, 5 * 256 * 4, st>>>(p);
-      } else {
-        latent_rows_any_kernel<T, 40><<<grid, LR_ANY_WARPS * 32, 5 * 1280 * 4, st>>>(p);
-      }
-    });
-  }
+  const dim3 grid(M, H, nsplit);
+  B2_DISPATCH_T(is_f32, {
+    if (Rp <= 256) {
+      latent_rows_any_kernel<T, 8><<<grid, LR_ANY_WARPS * 32, 5 * 256 * 4, st>>>(p);
+    } else {
+      latent_rows_any_kernel<T, 40><<<grid, LR_ANY_WARPS * 32, 5 * 1280 * 4, st>>>(p);
+    }
+  });
   B2_CHECK_LAUNCH("latent_rows");
   if (nsplit > 1) {
     B2_DISPATCH_T(is_f32, latent_merge_kernel<T><<<dim3(M, H), 128, 0, st>>>(p););

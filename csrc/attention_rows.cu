@@ -374,75 +374,119 @@ __global__ void __launch_bounds__(128) attn_rows_diff_merge_kernel(const AttnRow
   });
 }
 
+struct NormStoreParams {
+  const void* q;      // T rows of stride ld: H heads; k: G heads, v: Gv heads likewise
+  const void* k;
+  const void* v;
+  void* q_out;        // T [M, H * dkp]
+  void* kc;
+  void* vc;
+  const int* tables;
+  const int* row_seq;
+  const int* pos;
+  const int* slot;
+  const void* wq;     // T [dk] or null
+  const void* wk;
+  const void* bq;     // T, the columns of q, k, v, or null
+  const void* bk;
+  const void* bv;
+  const float* cs;    // [M, rot / 2] or null
+  const float* sn;
+  long long ld;
+  int max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot;
+  float eps;
+};
+
 // Bias, per-head RMS norm of q and k (optional weights), rotary positions on channel pairs (2 i, 2 i + 1), and the store of k / v.
-// Grid (M, ceil((H + Gk + Gv) / 4)), one warp per head.
-template <typename T>
-__global__ void __launch_bounds__(128) qk_norm_store_kernel(const T* __restrict__ q, const T* __restrict__ k,
-                                                            const T* __restrict__ v, long long ld, T* __restrict__ q_out,
-                                                            T* __restrict__ kc, T* __restrict__ vc,
-                                                            const int* __restrict__ tables, const int* __restrict__ row_seq,
-                                                            const int* __restrict__ pos, const int* __restrict__ slot,
-                                                            int max_blocks, int H, int G, int Gv, int dk, int dkp, int dvp,
-                                                            const T* __restrict__ wq, const T* __restrict__ wk, int norm,
-                                                            float eps, const T* __restrict__ bq, const T* __restrict__ bk,
-                                                            const T* __restrict__ bv, const float* __restrict__ cs,
-                                                            const float* __restrict__ sn, int rot) {
+// Grid (M, y).  LPH lanes per head, eight channels each; a lane takes NS_UNROLL heads of its row at a time, their loads together.
+constexpr int NS_UNROLL = 4;
+template <typename T, int LPH>
+__global__ void __launch_bounds__(128) qk_norm_store_kernel(const NormStoreParams p) {
+  constexpr int GROUPS = 128 / LPH;
   const size_t row = blockIdx.x;
-  const int w = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (w >= H + G + Gv) return;
-  const int s = row_seq ? row_seq[row] : static_cast<int>(row);
-  const bool live = slot == nullptr || slot[s] >= 0;
-  const T* src;
-  T* dst = nullptr;
-  const T* bias;
-  int width = dkp;
-  if (w < H) {
-    bias = bq ? bq + static_cast<size_t>(w) * dkp : nullptr;
-    src = q + row * ld + static_cast<size_t>(w) * dkp;
-    dst = q_out + (row * H + w) * dkp;
-  } else {
-    const int g = w < H + G ? w - H : w - H - G;
-    const int p = pos[row];
-    if (live) {
-      const size_t at = static_cast<size_t>(tables[static_cast<size_t>(s) * max_blocks + p / AR_PAGE]) * AR_PAGE + p % AR_PAGE;
-      dst = w < H + G ? kc + (at * G + g) * dkp : vc + (at * Gv + g) * dvp;
-    }
-    bias = w < H + G ? (bk ? bk + static_cast<size_t>(g) * dkp : nullptr) : (bv ? bv + static_cast<size_t>(g) * dvp : nullptr);
-    width = w < H + G ? dkp : dvp;
-    src = (w < H + G ? k + row * ld + static_cast<size_t>(g) * dkp : v + row * ld + static_cast<size_t>(g) * dvp);
-  }
-  if (dst == nullptr) return;
-  const int c = lane * 8;   // widths up to 256
-  float t[8] = {};
-  if (c < width) {
-    vload8(src + c, t);
-    if (bias) {
-      float b[8];
-      vload8(bias + c, b);
+  const int group = threadIdx.x / LPH, c = threadIdx.x % LPH * 8, units = p.H + p.G + p.Gv;
+  const int stride = GROUPS * gridDim.y;
+  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row), pos = p.pos[row];
+  const bool live = p.slot == nullptr || p.slot[s] >= 0;
+  const bool kin = c < p.dkp, vin = c < p.dvp;
+  const size_t at = live ? static_cast<size_t>(p.tables[static_cast<size_t>(s) * p.max_blocks + pos / AR_PAGE]) * AR_PAGE + pos % AR_PAGE : 0;
+  float co[4], si[4];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) t[e] += b[e];
+  for (int e = 0; e < 4; ++e) {
+    co[e] = 1.f;
+    si[e] = 0.f;
+  }
+  if (p.cs && c < p.rot) {
+    const size_t f = row * (p.rot / 2) + c / 2;
+    if (p.rot % 8 == 0) {
+      const float4 a = *reinterpret_cast<const float4*>(p.cs + f), b = *reinterpret_cast<const float4*>(p.sn + f);
+      co[0] = a.x; co[1] = a.y; co[2] = a.z; co[3] = a.w;
+      si[0] = b.x; si[1] = b.y; si[2] = b.z; si[3] = b.w;
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + 2 * e < p.rot) {
+          co[e] = p.cs[f + e];
+          si[e] = p.sn[f + e];
+        }
     }
   }
-  if (w < H + G && norm) {
-    float ss = 0.f;
+  float wq[8], wk[8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
-    const float r = 1.f / sqrtf(warp_sum(ss) / dk + eps);
-    const T* wt = w < H ? wq : wk;
-#pragma unroll
-    for (int e = 0; e < 8; ++e) t[e] *= wt && c + e < dk ? r * to_f(wt[c + e]) : r;
+  for (int e = 0; e < 8; ++e) {
+    wq[e] = p.wq && c + e < p.dk ? to_f(static_cast<const T*>(p.wq)[c + e]) : 1.f;
+    wk[e] = p.wk && c + e < p.dk ? to_f(static_cast<const T*>(p.wk)[c + e]) : 1.f;
   }
-  if (cs && w < H + G) {
-    const size_t at = row * (rot / 2) + c / 2;
+  for (int w0 = blockIdx.y * GROUPS + group; __any_sync(0xffffffffu, w0 < units); w0 += stride * NS_UNROLL) {
+    float t[NS_UNROLL][8];
+    auto part = [&](int w, const void* q, const void* k, const void* v) {      // the head's columns in a row of q | k | v
+      return w < p.H ? static_cast<const T*>(q) + static_cast<size_t>(w) * p.dkp
+                     : w < p.H + p.G ? static_cast<const T*>(k) + static_cast<size_t>(w - p.H) * p.dkp
+                                     : static_cast<const T*>(v) + static_cast<size_t>(w - p.H - p.G) * p.dvp;
+    };
 #pragma unroll
-    for (int e = 0; e < 8; e += 2)
-      if (c + e < rot) {
-        const float co = cs[at + e / 2], si = sn[at + e / 2], u = t[e], x = t[e + 1];
-        t[e] = u * co - x * si;
-        t[e + 1] = x * co + u * si;
+    for (int i = 0; i < NS_UNROLL; ++i) {
+      const int w = w0 + i * stride;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) t[i][e] = 0.f;
+      if (w < units && (w < p.H + p.G ? kin : vin)) vload8(part(w, p.q, p.k, p.v) + row * p.ld + c, t[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < NS_UNROLL; ++i) {
+      const int w = w0 + i * stride;
+      const bool qk = w < p.H + p.G, in = w < units && (qk ? kin : vin);
+      if (p.bq && in) {
+        float b[8];
+        vload8(part(w, p.bq, p.bk, p.bv) + c, b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) t[i][e] += b[e];
       }
+      if (p.norm) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(t[i][e], t[i][e], ss);
+#pragma unroll
+        for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float r = 1.f / sqrtf(ss / p.dk + p.eps);
+        if (qk)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) t[i][e] *= r * (w < p.H ? wq[e] : wk[e]);
+      }
+      if (p.cs && qk) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float u = t[i][2 * e], x = t[i][2 * e + 1];
+          t[i][2 * e] = u * co[e] - x * si[e];
+          t[i][2 * e + 1] = x * co[e] + u * si[e];
+        }
+      }
+      if (!in || (w >= p.H && !live)) continue;
+      T* dst = w < p.H ? static_cast<T*>(p.q_out) + (row * p.H + w) * p.dkp
+                       : qk ? static_cast<T*>(p.kc) + (at * p.G + w - p.H) * p.dkp
+                            : static_cast<T*>(p.vc) + (at * p.Gv + w - p.H - p.G) * p.dvp;
+      vstore8(dst + c, t[i]);
+    }
   }
-  if (c < width) vstore8(dst + c, t);
 }
 
 template <typename T, int LPT>
@@ -538,12 +582,19 @@ B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long
     set_error("qk_norm_store: head sizes up to 256 in multiples of 8 (padded) required");
     return 10;
   }
-  const dim3 grid(M, (H + G + Gv + 3) / 4);
-  B2_DISPATCH_T(is_f32, qk_norm_store_kernel<T><<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), ld, static_cast<T*>(q_out),
-      static_cast<T*>(kc), static_cast<T*>(vc), tables, row_seq, pos, slot, max_blocks, H, G, Gv, dk, dkp, dvp,
-      static_cast<const T*>(wq), static_cast<const T*>(wk), norm, eps, static_cast<const T*>(bq), static_cast<const T*>(bk),
-      static_cast<const T*>(bv), cs, sn, rot););
+  if ((bq == nullptr) != (bk == nullptr) || (bq == nullptr) != (bv == nullptr)) { set_error("qk_norm_store: all biases or none"); return 10; }
+  const NormStoreParams p = {q, k, v, q_out, kc, vc, tables, row_seq, pos, slot, wq, wk, bq, bk, bv, cs, sn, ld,
+                             max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot, eps};
+  const int w = dkp > dvp ? dkp : dvp, lph = w <= 64 ? 8 : w <= 128 ? 16 : 32, groups = 128 / lph;
+  int y = (H + G + Gv + groups - 1) / groups;              // a head per lane group; several when the rows fill the GPU
+  if (M >= 8 * num_sms()) y = (y + NS_UNROLL - 1) / NS_UNROLL;
+  const dim3 grid(M, y);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  B2_DISPATCH_T(is_f32, {
+    if (lph == 8) qk_norm_store_kernel<T, 8><<<grid, 128, 0, st>>>(p);
+    else if (lph == 16) qk_norm_store_kernel<T, 16><<<grid, 128, 0, st>>>(p);
+    else qk_norm_store_kernel<T, 32><<<grid, 128, 0, st>>>(p);
+  });
   B2_CHECK_LAUNCH("qk_norm_store");
   return 0;
 }

@@ -64,6 +64,20 @@ __device__ __forceinline__ float silu_t(float z) { return sizeof(T) == 2 ? silu_
 template <typename T>
 __device__ __forceinline__ float sigmoid_t(float z) { return sizeof(T) == 2 ? sigmoid_fast(z) : sigmoid_f(z); }
 
+// two fp32 multiplications or fused multiply-adds in one instruction
+__device__ __forceinline__ float2 mul_f32x2(float2 a, float2 b) {
+  unsigned long long d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
+  return reinterpret_cast<float2&>(d);
+}
+__device__ __forceinline__ float2 fma_f32x2(float2 a, float2 b, float2 c) {
+  unsigned long long d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;"
+      : "=l"(d)
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)), "l"(reinterpret_cast<unsigned long long&>(c)));
+  return reinterpret_cast<float2&>(d);
+}
+
 // cap * tanh(z) for a score s = cap * z pressed softly into (-cap, cap).  Near zero: the Taylor series of tanh (relative error
 // below 1e-7 for |z| <= SOFTCAP_SERIES); elsewhere 1 - 2 / (1 + e^{2 z}), whose absolute error is a rounding of 1.
 constexpr float SOFTCAP_SERIES = 0.4f;
