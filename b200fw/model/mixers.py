@@ -341,8 +341,8 @@ class DifferentialAttention(nn.Module):
         self.in_proj = PackedRows(hidden, [("q", 2 * heads, dim), ("k", 2 * kv_heads, dim), ("v", kv_heads, vdim), ("g", heads, vdim)],
                                   dtype, device)
         self.bias = _param(self.in_proj.end("v"), dtype=dtype, device=device)
-        self.q_norm = _param(dim, dtype=dtype, device=device)
-        self.k_norm = _param(dim, dtype=dtype, device=device)
+        self.q_norm = _param(pad8(dim), dtype=dtype, device=device)
+        self.k_norm = _param(pad8(dim), dtype=dtype, device=device)
         self.lam = _param(4, pad8(dim), dtype=dtype, device=device)
         self.o = PackedCols(hidden, [("o", heads, vdim)], dtype, device)
         self.o_bias = _param(pad8(hidden), dtype=dtype, device=device)
@@ -359,8 +359,8 @@ class DifferentialAttention(nn.Module):
         for n in "qkv":
             at, heads, d = self.in_proj.sections[n]
             t[prefix + n + ".b"] = Slot(self.bias.data[at:at + heads * pad8(d)].view(heads, pad8(d))[:, :d], (heads * d,))
-        t[prefix + "q.norm"] = Slot(self.q_norm.data, (self.dim,))
-        t[prefix + "k.norm"] = Slot(self.k_norm.data, (self.dim,))
+        t[prefix + "q.norm"] = Slot(self.q_norm.data[:self.dim], (self.dim,))
+        t[prefix + "k.norm"] = Slot(self.k_norm.data[:self.dim], (self.dim,))
         for i, n in enumerate(("lq1", "lk1", "lq2", "lk2")):
             t[prefix + n] = Slot(self.lam.data[i, :self.dim], (self.dim,))
         t[prefix + "o"] = self.o.slot("o")

@@ -36,7 +36,7 @@ def qk_norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: to
                   wk: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None,
                   sin: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``bias`` (one vector over the columns of q, k and v) added, per-head RMS norm of q and k (``norm``; optional weights
-    ``[dk]``), rotary positions of q and k on channel pairs (2 i, 2 i + 1) (``cos, sin [M, dims/2]``), k and v stored into their
+    ``[dkp]``), rotary positions of q and k on channel pairs (2 i, 2 i + 1) (``cos, sin [M, dims/2]``), k and v stored into their
     sequences' pages.  ``q, k, v`` are column slices of one matrix; returns the new q ``[M, H*dkp]``.  K and V pages may have
     different head counts (two key rows over one value row)."""
     nblk, bs, G, dkp = k_cache.shape
@@ -53,7 +53,7 @@ def qk_norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: to
             if norm:
                 x = x * torch.rsqrt((x * x).sum(-1, keepdim=True) / dk + eps)
                 if w is not None:
-                    x = x * torch.nn.functional.pad(w.float(), (0, dkp - dk))
+                    x = x * w.float()
             if cos is not None:
                 rot = 2 * cos.shape[1]
                 u, z, c, s = x[..., 0:rot:2], x[..., 1:rot:2], cos[:, None, :], sin[:, None, :]
@@ -212,7 +212,7 @@ def decode_attention(q, k_cache, v_cache, out, p: Portions, rows: int, H: int, G
     nv.check(nv.lib().b2_decode_attention(
         nv.ptr(q), nv.ptr(k_cache), nv.ptr(v_cache), nv.ptr(p.block_tables), nv.ptr(p.row_seq), nv.ptr(p.positions),
         nv.ptr(p.plans[key]), nv.ptr(sink), nv.ptr(gate), nv.ptr(lam), nv.ptr(out), nv.ptr(po), nv.ptr(pm), cl(q.stride(0)),
-        cl(0 if gate is None else gate.stride(0)), cl(out.stride(0)), rows, p.block_tables.shape[1], H, G, R, C, window, dv, cf(scale),
+        cl(0 if gate is None else gate.stride(0)), cl(out.stride(0)), rows, k_cache.shape[0], p.block_tables.shape[1], H, G, R, C, window, dv, cf(scale),
         cf(softcap), cf(lam_init), cf(eps), nv.stream_ptr()), "decode_attention")
     nv.count_launch(2)
     return True

@@ -6,8 +6,8 @@
 // rows (decode_plan writes the running tile count).  A CTA finishes every (row, group) that lies inside its run; what a cut
 // divides is left as partial sums, two slots per CTA, for the merge kernel, which has one block per cut and head.
 //
-// Inside a CTA one warp copies (a bulk copy per key row, padded to an odd number of 16-byte pieces so that ldmatrix reads without
-// bank conflicts; a ring of stages, running ahead over the ends of rows) and eight compute.  Scores: each warp a group of
+// Inside a CTA one warp copies (TMA boxes of one page by 64 channels into 128-byte-swizzled tiles, a ring of stages that runs ahead
+// over the ends of rows) and eight compute.  Scores: each warp a group of
 // eight keys, and with HALVES = 2 half of the channels.  They meet in shared memory, double-buffered: one barrier per tile.  Every
 // warp then takes the softmax of the whole tile in the layout of its next operand, and multiplies 16-channel pieces of the values.
 #include "host.h"
@@ -22,8 +22,8 @@ typedef __nv_bfloat16 ad_bf16;
 
 struct DecodeParams {
   const ad_bf16* q;      // [M, ld_q]: head h's map m at (h * maps + m) * (R / maps)
-  const ad_bf16* kc;     // pages: a token's key row of kv head g at (token * G + g) * R
-  const ad_bf16* vc;     // pages of values likewise, or null: a value is the first C channels of the key row
+  // pages of keys [tokens, G, R] and of values [tokens, G, C] come by tensor map
+  int apart;             // 0: a value is the first C channels of its key row
   const int* tables;     // [nseq, max_blocks]
   const int* row_seq;    // [M] or null: row r is sequence r
   const int* pos;        // [M]
@@ -41,7 +41,8 @@ struct DecodeParams {
   float scale, softcap, lam_init, eps;
 };
 
-__device__ __forceinline__ int ad_first(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
+// first key of the row's first tile: the page that holds the first visible one
+__device__ __forceinline__ int ad_first(int pos, int window) { return window > 0 ? max(0, pos - window + 1) / AD_PAGE * AD_PAGE : 0; }
 
 // prefix[r] = tiles of the rows before r.  One CTA.
 __global__ void __launch_bounds__(1024) decode_plan_kernel(const int* __restrict__ pos, const int* __restrict__ row_seq,
@@ -113,35 +114,43 @@ __device__ __forceinline__ void ad_next(const DecodeParams& p, int groups, Decod
   } while (a.n == 0 && a.row + 1 < p.M);
 }
 
-__host__ __device__ constexpr int ad_pitch(int channels) { return (((channels * 2 + 63) / 64 * 64) / 16 | 1) * 16; }   // bytes, whole k32 steps
+// Query rows: an odd number of 16-byte pieces apart, so that ldmatrix meets no bank twice; whole 32-channel steps.
+__host__ __device__ constexpr int ad_pitch(int channels) { return (((channels * 2 + 63) / 64 * 64) / 16 | 1) * 16; }
 struct DecodeSmem {
-  int kpitch, vpitch, stage, q, s, bars, total;
-  __host__ __device__ DecodeSmem(int R, int C, bool values, int tile, int halves, int stages) {
-    kpitch = ad_pitch(R);
-    vpitch = values ? ad_pitch(C) : 0;
-    stage = tile * (kpitch + vpitch);
+  int kparts, vparts, stage, pitch, q, s, bars, total;    // parts: 64-channel pieces, [tile keys x 128 bytes] each
+  __host__ __device__ DecodeSmem(int R, int C, bool apart, int tile, int halves, int stages) {
+    kparts = (R + 63) / 64;
+    vparts = apart ? (C + 63) / 64 : 0;
+    stage = (kparts + vparts) * tile * 128;
+    pitch = ad_pitch(R);
     q = stages * stage;                               // 2 x [16] query rows
-    s = q + 2 * 16 * kpitch;                          // 2 x halves x [16][tile + 8] scores
+    s = q + 2 * 16 * pitch;                           // 2 x halves x [16][tile + 8] scores
     bars = s + 2 * halves * 16 * (tile + 8) * 4;      // barriers (256 B), then [16][8] sums
-    total = bars + 256 + 16 * 8 * 4;
+    total = bars + 256 + 16 * 8 * 4 + 1024;
   }
 };
+// channel c (a multiple of 8) of key k in a swizzled tile
+template <int KT>
+__device__ __forceinline__ const ad_bf16* ad_at(const uint8_t* tile, int k, int c) {
+  return reinterpret_cast<const ad_bf16*>(tile + (c >> 6) * (KT * 128) + k * 128 + ((((c >> 3) & 7) ^ (k & 7)) << 4));
+}
 
 __device__ __forceinline__ void ad_consumer_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 template <int HALVES, int QP, int NG>   // QP: 32-channel steps of a warp's share of the keys; NG: 16-channel pieces of values per warp
-__global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const DecodeParams p, int* status) {
-  constexpr int KT = 64 / HALVES, LDS = KT + 8, KS = KT / 16;
-  extern __shared__ __align__(128) uint8_t ad_smem[];
-  const DecodeSmem L(p.R, p.C, p.vc != nullptr, KT, HALVES, p.stages);
+__global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const DecodeParams p, int* status) {
+  constexpr int KT = 64 / HALVES, LDS = KT + 8, KS = KT / 16, PAGES = KT / AD_PAGE;
+  extern __shared__ uint8_t ad_raw[];
+  uint8_t* ad_smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ad_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const DecodeSmem L(p.R, p.C, p.apart, KT, HALVES, p.stages);
   uint64_t* full = reinterpret_cast<uint64_t*>(ad_smem + L.bars);
   uint64_t *empty = full + 8, *q_full = full + 16, *q_empty = full + 18;
   float* sums = reinterpret_cast<float*>(ad_smem + L.bars + 256);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int groups = p.G * p.hgroups, total = p.prefix[p.M] * groups;
   const int quota = (total + gridDim.x - 1) / gridDim.x, x0 = blockIdx.x * quota, x1 = min(x0 + quota, total);
-  // pads and rows that are never copied enter products with zeros: they must be finite
-  for (int i = tid * 16; i < L.bars; i += AD_THREADS * 16) *reinterpret_cast<uint4*>(ad_smem + i) = make_uint4(0, 0, 0, 0);
+  // what no copy ever writes of the query rows (a head's other map, missing heads, padding) is zero
+  for (int i = L.q + tid * 16; i < L.s; i += AD_THREADS * 16) *reinterpret_cast<uint4*>(ad_smem + i) = make_uint4(0, 0, 0, 0);
   if (tid == 0) {
     for (int i = 0; i < 8; ++i) {
       mbar_init(full + i, 1);
@@ -163,7 +172,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
   if (warp == AD_WARPS) {
     int st = 0, seg = 0;
     uint32_t ph = 0;
-    const int kbytes = p.R * 2, vbytes = p.vc ? p.C * 2 : 0;
+    const int parts = L.kparts + L.vparts;
     for (int x = x0; x < x1; ++seg) {
       const int t1 = min(a.n, a.t + x1 - x), kvh = a.group / p.hgroups, head0 = kvh * (p.H / p.G) + a.group % p.hgroups * p.heads;
       const int rows = min(p.heads, (kvh + 1) * (p.H / p.G) - head0) * p.maps, qs = seg & 1;
@@ -173,26 +182,20 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
       if (lane == 0) mbar_expect_tx(&q_full[qs], rows * kq * 2);
       __syncwarp();
       if (lane < rows)
-        bulk_load(ad_smem + L.q + (qs * 16 + lane) * L.kpitch + lane % p.maps * kq * 2,
+        bulk_load(ad_smem + L.q + (qs * 16 + lane) * L.pitch + lane % p.maps * kq * 2,
                   p.q + a.row * p.ld_q + static_cast<size_t>(head0 * p.maps + lane) * kq, kq * 2, &q_full[qs]);
       for (int t = a.t; t < t1; ++t) {
-        const int k0 = first + t * KT, nk = min(KT, pos + 1 - k0);
-        size_t at[KT / 32];
-#pragma unroll
-        for (int i = 0; i < KT / 32; ++i) {
-          const int k = min(k0 + lane + 32 * i, pos);
-          at[i] = (static_cast<size_t>(table[k / AD_PAGE]) * AD_PAGE + k % AD_PAGE) * p.G + kvh;
-        }
+        // boxes (page, part): pages past the row's last repeat it, those keys are masked
+        const int pg0 = (first + t * KT) / AD_PAGE, last = pos / AD_PAGE;
         mbar_wait_warp(&empty[st], ph ^ 1, status, ERR_ATTN_WAIT);
-        if (lane == 0) mbar_expect_tx(&full[st], nk * (kbytes + vbytes));
+        if (lane == 0) mbar_expect_tx(&full[st], parts * KT * 128);
         __syncwarp();
         uint8_t* tile = ad_smem + st * L.stage;
-#pragma unroll
-        for (int i = 0; i < KT / 32; ++i) {
-          const int k = lane + 32 * i;
-          if (k >= nk) continue;
-          bulk_load(tile + k * L.kpitch, p.kc + at[i] * p.R, kbytes, &full[st]);
-          if (vbytes) bulk_load(tile + KT * L.kpitch + k * L.vpitch, p.vc + at[i] * p.C, vbytes, &full[st]);
+        for (int i = lane; i < parts * PAGES; i += 32) {
+          const int pg = i % PAGES, part = i / PAGES, token = table[min(pg0 + pg, last)] * AD_PAGE;
+          uint8_t* dst = tile + part * (KT * 128) + pg * (AD_PAGE * 128);
+          if (part < L.kparts) tma_load_3d(dst, &tmK, &full[st], part * 64, kvh, token);
+          else tma_load_3d(dst, &tmV, &full[st], (part - L.kparts) * 64, kvh, token);
         }
         if (++st == p.stages) {
           st = 0;
@@ -207,22 +210,23 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
     const int steps = (p.R + 31) / 32, mine = HALVES == 1 ? steps : kh ? steps / 2 : (steps + 1) / 2, c0 = kh ? (steps + 1) / 2 * 32 : 0;
     const float lam = p.maps == 2 ? diff_lambda(p.lam, kq, p.lam_init) : 0.f;
     const float sl2 = p.scale * AD_LOG2E;
-    const int kld = L.kpitch / 2, vld = p.vc ? L.vpitch / 2 : kld;      // in elements
+    const int qld = L.pitch / 2;        // in elements
     int st = 0, seg = 0, buf = 0;
     uint32_t ph = 0;
     for (int x = x0; x < x1; ++seg) {
       const int t1 = min(a.n, a.t + x1 - x), kvh = a.group / p.hgroups, head0 = kvh * (p.H / p.G) + a.group % p.hgroups * p.heads;
       const int rows = min(p.heads, (kvh + 1) * (p.H / p.G) - head0) * p.maps, qs = seg & 1;
-      const int keys = p.pos[a.row] + 1 - ad_first(p.pos[a.row], p.window);
+      const int pos = p.pos[a.row], first = ad_first(pos, p.window), keys = pos + 1 - first;
+      const int skip = p.window > 0 ? max(0, pos - p.window + 1) - first : 0;     // keys of the first tile before the window
       uint32_t q[QP][2][4];
       mbar_wait_warp(&q_full[qs], (seg >> 1) & 1, status, ERR_ATTN_WAIT);
       {
-        const ad_bf16* sq = reinterpret_cast<const ad_bf16*>(ad_smem + L.q + qs * 16 * L.kpitch) + c0;
+        const ad_bf16* sq = reinterpret_cast<const ad_bf16*>(ad_smem + L.q + qs * 16 * L.pitch) + c0;
 #pragma unroll
         for (int i = 0; i < QP; ++i)
           if (i < mine) {
-            ldsm_a_mk(sq + i * 32, kld, lane, q[i][0]);
-            ldsm_a_mk(sq + i * 32 + 16, kld, lane, q[i][1]);
+            ldsm_a_mk(sq + i * 32, qld, lane, q[i][0]);
+            ldsm_a_mk(sq + i * 32 + 16, qld, lane, q[i][1]);
           }
       }
       mbar_arrive_warp(&q_empty[qs]);
@@ -233,17 +237,16 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
         for (int i = 0; i < 8; ++i) acc[g][i >> 2][i & 3] = 0.f;
       for (int t = a.t; t < t1; ++t) {
         mbar_wait_warp(&full[st], ph, status, ERR_ATTN_WAIT);
-        const ad_bf16* tile = reinterpret_cast<const ad_bf16*>(ad_smem + st * L.stage);
+        const uint8_t* tile = ad_smem + st * L.stage;
         float* S = reinterpret_cast<float*>(ad_smem + L.s) + buf * HALVES * 16 * LDS;
         buf ^= 1;
         {
           float d[2][4] = {};
-          const ad_bf16* kp = tile + (kg * 8 + (lane & 7)) * kld + c0 + (lane >> 3) * 8;
 #pragma unroll
           for (int i = 0; i < QP; ++i)
             if (i < mine) {
               uint32_t b[4];
-              ldsm_x4(kp + i * 32, b);
+              ldsm_x4(ad_at<KT>(tile, kg * 8 + (lane & 7), c0 + i * 32 + (lane >> 3) * 8), b);
               const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
               mma_bf16(d[0], q[i][0], b0);
               mma_bf16(d[1], q[i][1], b1);
@@ -284,6 +287,13 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
             for (int i = 0; i < 4; ++i)
               if (ks * 16 + (i >> 1) * 8 + (lane & 3) * 2 + (i & 1) >= left) s[ks][0][i] = s[ks][1][i] = -INFINITY;
         }
+        if (t == 0 && skip > 0) {
+#pragma unroll
+          for (int ks = 0; ks < KS; ++ks)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+              if (ks * 16 + (i >> 1) * 8 + (lane & 3) * 2 + (i & 1) < skip) s[ks][0][i] = s[ks][1][i] = -INFINITY;
+        }
         float n0 = m0, n1 = m1;
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks)
@@ -319,7 +329,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
         }
         l0 = l0 * f0 + p0;       // this lane's keys only; added over the four lanes of a row at the end
         l1 = l1 * f1 + p1;
-        const ad_bf16* vt = p.vc ? tile + KT * kld : tile;
+        const uint8_t* vt = tile + (p.apart ? L.kparts * (KT * 128) : 0);
 #pragma unroll
         for (int g = 0; g < NG; ++g) {
           const int c = (warp + 8 * g) * 16;
@@ -334,7 +344,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const Decode
 #pragma unroll
           for (int ks = 0; ks < KS; ++ks) {
             uint32_t b[4];
-            ldsm_b_kn(vt + ks * 16 * vld + c, vld, lane, b);
+            ldsm_x4_t(ad_at<KT>(vt, ks * 16 + (lane & 15), c + (lane >> 4) * 8), b);
             mma_n16(acc[g][0], acc[g][1], pa[ks], b);
           }
         }
@@ -503,20 +513,26 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(const DecodeParams p,
 }
 
 template <int HALVES, int QP, int NG>
-static int launch_decode(DecodeParams& p, int grid, cudaStream_t stream) {
+static int launch_decode(DecodeParams& p, const CUtensorMap* tk, const CUtensorMap* tv, int grid, cudaStream_t stream) {
   constexpr int KT = 64 / HALVES;
   auto kern = decode_attn_kernel<HALVES, QP, NG>;
   int stages = 8;
-  while (stages > 2 && DecodeSmem(p.R, p.C, p.vc != nullptr, KT, HALVES, stages).total > 232448) --stages;
-  const int smem = DecodeSmem(p.R, p.C, p.vc != nullptr, KT, HALVES, stages).total;
+  while (stages > 2 && DecodeSmem(p.R, p.C, p.apart, KT, HALVES, stages).total > 232448) --stages;
+  const int smem = DecodeSmem(p.R, p.C, p.apart, KT, HALVES, stages).total;
   int* status = status_ptr();
   if (!status) return 3;
-  if (smem > 232448 || cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
-    set_error("decode_attention: cannot set shared memory size (%d)", smem);
-    return 1;
+  static int set[64] = {0};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (set[dev & 63] < smem) {
+    if (smem > 232448 || cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+      set_error("decode_attention: cannot set shared memory size (%d)", smem);
+      return 1;
+    }
+    set[dev & 63] = smem;
   }
   p.stages = stages;
-  kern<<<grid, AD_THREADS, smem, stream>>>(p, status);
+  kern<<<grid, AD_THREADS, smem, stream>>>(*tk, *tv, p, status);
   B2_CHECK_LAUNCH("decode_attention");
   decode_merge_kernel<<<dim3(grid - 1, p.heads), 128, 0, stream>>>(p, grid, KT);
   B2_CHECK_LAUNCH("decode_attention_merge");
@@ -549,7 +565,7 @@ B2_EXPORT int b2_decode_plan(const int* pos, const int* row_seq, const int* slot
 B2_EXPORT int b2_decode_attention(const void* q, const void* kc, const void* vc, const int* tables, const int* row_seq,
                                   const int* pos, const int* prefix, const void* sink, const void* gate, const void* lam, void* out,
                                   float* part_o, float* part_ml, long long ld_q, long long ld_gate, long long ld_out, int M,
-                                  int max_blocks, int H, int G, int R, int C, int window, int dv, float scale, float softcap,
+                                  int num_blocks, int max_blocks, int H, int G, int R, int C, int window, int dv, float scale, float softcap,
                                   float lam_init, float eps, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
@@ -560,7 +576,7 @@ B2_EXPORT int b2_decode_attention(const void* q, const void* kc, const void* vc,
     return 10;
   }
   DecodeParams p = {};
-  p.q = static_cast<const ad_bf16*>(q); p.kc = static_cast<const ad_bf16*>(kc); p.vc = static_cast<const ad_bf16*>(vc);
+  p.q = static_cast<const ad_bf16*>(q); p.apart = vc != nullptr;
   p.tables = tables; p.row_seq = row_seq; p.pos = pos; p.prefix = prefix; p.sink = static_cast<const ad_bf16*>(sink);
   p.gate = static_cast<const ad_bf16*>(gate); p.lam = static_cast<const ad_bf16*>(lam); p.out = static_cast<ad_bf16*>(out);
   p.part_o = part_o; p.part_ml = part_ml; p.ld_q = ld_q; p.ld_gate = ld_gate; p.ld_out = ld_out; p.M = M;
@@ -572,7 +588,14 @@ B2_EXPORT int b2_decode_attention(const void* q, const void* kc, const void* vc,
   p.hgroups = (per + p.heads - 1) / p.heads;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int grid = num_sms();
-  if (vc) return launch_decode<1, 8, 1>(p, grid, st);
-  if (R <= 192 && C <= 128) return launch_decode<2, 3, 1>(p, grid, st);
-  return launch_decode<2, 9, 4>(p, grid, st);
+  auto map = [&](const void* base, uint64_t d) {
+    const uint64_t dims[3] = {d, static_cast<uint64_t>(G), static_cast<uint64_t>(num_blocks) * AD_PAGE}, strides[2] = {d * 2, G * d * 2};
+    const uint32_t box[3] = {64, 1, AD_PAGE};
+    return tensor_map_nd_bf16(base, 3, dims, strides, box, 3);
+  };
+  const CUtensorMap *tk = map(kc, R), *tv = vc ? map(vc, C) : tk;
+  if (!tk || !tv) return 2;
+  if (vc) return launch_decode<1, 8, 1>(p, tk, tv, grid, st);
+  if (R <= 192 && C <= 128) return launch_decode<2, 3, 1>(p, tk, tv, grid, st);
+  return launch_decode<2, 9, 4>(p, tk, tv, grid, st);
 }

@@ -385,7 +385,7 @@ struct NormStoreParams {
   const int* row_seq;
   const int* pos;
   const int* slot;
-  const void* wq;     // T [dk] or null
+  const void* wq;     // T [dkp] or null
   const void* wk;
   const void* bq;     // T, the columns of q, k, v, or null
   const void* bk;
@@ -393,7 +393,7 @@ struct NormStoreParams {
   const float* cs;    // [M, rot / 2] or null
   const float* sn;
   long long ld;
-  int max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot;
+  int M, max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot;
   float eps;
 };
 
@@ -403,88 +403,88 @@ constexpr int NS_UNROLL = 4;
 template <typename T, int LPH>
 __global__ void __launch_bounds__(128) qk_norm_store_kernel(const NormStoreParams p) {
   constexpr int GROUPS = 128 / LPH;
-  const size_t row = blockIdx.x;
   const int group = threadIdx.x / LPH, c = threadIdx.x % LPH * 8, units = p.H + p.G + p.Gv;
   const int stride = GROUPS * gridDim.y;
-  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row), pos = p.pos[row];
-  const bool live = p.slot == nullptr || p.slot[s] >= 0;
   const bool kin = c < p.dkp, vin = c < p.dvp;
-  const size_t at = live ? static_cast<size_t>(p.tables[static_cast<size_t>(s) * p.max_blocks + pos / AR_PAGE]) * AR_PAGE + pos % AR_PAGE : 0;
-  float co[4], si[4];
-#pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    co[e] = 1.f;
-    si[e] = 0.f;
-  }
-  if (p.cs && c < p.rot) {
-    const size_t f = row * (p.rot / 2) + c / 2;
-    if (p.rot % 8 == 0) {
-      const float4 a = *reinterpret_cast<const float4*>(p.cs + f), b = *reinterpret_cast<const float4*>(p.sn + f);
-      co[0] = a.x; co[1] = a.y; co[2] = a.z; co[3] = a.w;
-      si[0] = b.x; si[1] = b.y; si[2] = b.z; si[3] = b.w;
-    } else {
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (c + 2 * e < p.rot) {
-          co[e] = p.cs[f + e];
-          si[e] = p.sn[f + e];
-        }
-    }
-  }
   float wq[8], wk[8];
 #pragma unroll
-  for (int e = 0; e < 8; ++e) {
-    wq[e] = p.wq && c + e < p.dk ? to_f(static_cast<const T*>(p.wq)[c + e]) : 1.f;
-    wk[e] = p.wk && c + e < p.dk ? to_f(static_cast<const T*>(p.wk)[c + e]) : 1.f;
-  }
-  for (int w0 = blockIdx.y * GROUPS + group; __any_sync(0xffffffffu, w0 < units); w0 += stride * NS_UNROLL) {
-    float t[NS_UNROLL][8];
-    auto part = [&](int w, const void* q, const void* k, const void* v) {      // the head's columns in a row of q | k | v
-      return w < p.H ? static_cast<const T*>(q) + static_cast<size_t>(w) * p.dkp
-                     : w < p.H + p.G ? static_cast<const T*>(k) + static_cast<size_t>(w - p.H) * p.dkp
-                                     : static_cast<const T*>(v) + static_cast<size_t>(w - p.H - p.G) * p.dvp;
-    };
+  for (int e = 0; e < 8; ++e) wq[e] = wk[e] = 1.f;
+  if (p.wq && kin) vload8(static_cast<const T*>(p.wq) + c, wq);
+  if (p.wk && kin) vload8(static_cast<const T*>(p.wk) + c, wk);
+  for (size_t row = blockIdx.x; row < static_cast<size_t>(p.M); row += gridDim.x) {
+    const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row), pos = p.pos[row];
+    const bool live = p.slot == nullptr || p.slot[s] >= 0;
+    const size_t at = live ? static_cast<size_t>(p.tables[static_cast<size_t>(s) * p.max_blocks + pos / AR_PAGE]) * AR_PAGE + pos % AR_PAGE : 0;
+    float co[4], si[4];
 #pragma unroll
-    for (int i = 0; i < NS_UNROLL; ++i) {
-      const int w = w0 + i * stride;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) t[i][e] = 0.f;
-      if (w < units && (w < p.H + p.G ? kin : vin)) vload8(part(w, p.q, p.k, p.v) + row * p.ld + c, t[i]);
+    for (int e = 0; e < 4; ++e) {
+      co[e] = 1.f;
+      si[e] = 0.f;
     }
+    if (p.cs && c < p.rot) {
+      const size_t f = row * (p.rot / 2) + c / 2;
+      if (p.rot % 8 == 0) {
+        const float4 a = *reinterpret_cast<const float4*>(p.cs + f), b = *reinterpret_cast<const float4*>(p.sn + f);
+        co[0] = a.x; co[1] = a.y; co[2] = a.z; co[3] = a.w;
+        si[0] = b.x; si[1] = b.y; si[2] = b.z; si[3] = b.w;
+      } else {
 #pragma unroll
-    for (int i = 0; i < NS_UNROLL; ++i) {
-      const int w = w0 + i * stride;
-      const bool qk = w < p.H + p.G, in = w < units && (qk ? kin : vin);
-      if (p.bq && in) {
-        float b[8];
-        vload8(part(w, p.bq, p.bk, p.bv) + c, b);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) t[i][e] += b[e];
+        for (int e = 0; e < 4; ++e)
+          if (c + 2 * e < p.rot) {
+            co[e] = p.cs[f + e];
+            si[e] = p.sn[f + e];
+          }
       }
-      if (p.norm) {
-        float ss = 0.f;
+    }
+    for (int w0 = blockIdx.y * GROUPS + group; __any_sync(0xffffffffu, w0 < units); w0 += stride * NS_UNROLL) {
+      float t[NS_UNROLL][8];
+      auto part = [&](int w, const void* q, const void* k, const void* v) {      // the head's columns in a row of q | k | v
+        return w < p.H ? static_cast<const T*>(q) + static_cast<size_t>(w) * p.dkp
+                       : w < p.H + p.G ? static_cast<const T*>(k) + static_cast<size_t>(w - p.H) * p.dkp
+                                       : static_cast<const T*>(v) + static_cast<size_t>(w - p.H - p.G) * p.dvp;
+      };
 #pragma unroll
-        for (int e = 0; e < 8; ++e) ss = fmaf(t[i][e], t[i][e], ss);
+      for (int i = 0; i < NS_UNROLL; ++i) {
+        const int w = w0 + i * stride;
 #pragma unroll
-        for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        const float r = 1.f / sqrtf(ss / p.dk + p.eps);
-        if (qk)
-#pragma unroll
-          for (int e = 0; e < 8; ++e) t[i][e] *= r * (w < p.H ? wq[e] : wk[e]);
+        for (int e = 0; e < 8; ++e) t[i][e] = 0.f;
+        if (w < units && (w < p.H + p.G ? kin : vin)) vload8(part(w, p.q, p.k, p.v) + row * p.ld + c, t[i]);
       }
-      if (p.cs && qk) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float u = t[i][2 * e], x = t[i][2 * e + 1];
-          t[i][2 * e] = u * co[e] - x * si[e];
-          t[i][2 * e + 1] = x * co[e] + u * si[e];
+      for (int i = 0; i < NS_UNROLL; ++i) {
+        const int w = w0 + i * stride;
+        const bool qk = w < p.H + p.G, in = w < units && (qk ? kin : vin);
+        if (p.bq && in) {
+          float b[8];
+          vload8(part(w, p.bq, p.bk, p.bv) + c, b);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) t[i][e] += b[e];
         }
+        if (p.norm) {
+          float ss = 0.f;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) ss = fmaf(t[i][e], t[i][e], ss);
+#pragma unroll
+          for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+          const float r = rsqrtf(ss / p.dk + p.eps);
+          if (qk)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) t[i][e] *= r * (w < p.H ? wq[e] : wk[e]);
+        }
+        if (p.cs && qk) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float u = t[i][2 * e], x = t[i][2 * e + 1];
+            t[i][2 * e] = u * co[e] - x * si[e];
+            t[i][2 * e + 1] = x * co[e] + u * si[e];
+          }
+        }
+        if (!in || (w >= p.H && !live)) continue;
+        T* dst = w < p.H ? static_cast<T*>(p.q_out) + (row * p.H + w) * p.dkp
+                         : qk ? static_cast<T*>(p.kc) + (at * p.G + w - p.H) * p.dkp
+                              : static_cast<T*>(p.vc) + (at * p.Gv + w - p.H - p.G) * p.dvp;
+        vstore8(dst + c, t[i]);
       }
-      if (!in || (w >= p.H && !live)) continue;
-      T* dst = w < p.H ? static_cast<T*>(p.q_out) + (row * p.H + w) * p.dkp
-                       : qk ? static_cast<T*>(p.kc) + (at * p.G + w - p.H) * p.dkp
-                            : static_cast<T*>(p.vc) + (at * p.Gv + w - p.H - p.G) * p.dvp;
-      vstore8(dst + c, t[i]);
     }
   }
 }
@@ -584,11 +584,11 @@ B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long
   }
   if ((bq == nullptr) != (bk == nullptr) || (bq == nullptr) != (bv == nullptr)) { set_error("qk_norm_store: all biases or none"); return 10; }
   const NormStoreParams p = {q, k, v, q_out, kc, vc, tables, row_seq, pos, slot, wq, wk, bq, bk, bv, cs, sn, ld,
-                             max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot, eps};
+                             M, max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot, eps};
   const int w = dkp > dvp ? dkp : dvp, lph = w <= 64 ? 8 : w <= 128 ? 16 : 32, groups = 128 / lph;
   int y = (H + G + Gv + groups - 1) / groups;              // a head per lane group; several when the rows fill the GPU
   if (M >= 8 * num_sms()) y = (y + NS_UNROLL - 1) / NS_UNROLL;
-  const dim3 grid(M, y);
+  const dim3 grid(M < 10 * num_sms() ? M : 10 * num_sms(), y);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   B2_DISPATCH_T(is_f32, {
     if (lph == 8) qk_norm_store_kernel<T, 8><<<grid, 128, 0, st>>>(p);

@@ -257,7 +257,7 @@ def test_differential_attention(run, H, G, dk, dv, window, rot, cap):
             vc = torch.full((pages, 16, G, pad8(dv)), junk, dtype=run[1], device=run[0])
         q, k, v, g = packed(rows_of(data, order, starts, cnt), run)
         cs, sn = ops.rope_rows(p.positions, turns)
-        qn = ops.qk_norm_store(q, k, v, kc, vc, p, 2 * H, dk, True, eps, on(wq), on(wk), b, cs, sn)
+        qn = ops.qk_norm_store(q, k, v, kc, vc, p, 2 * H, dk, True, eps, on(P8(wq)), on(P8(wk)), b, cs, sn)
         out = torch.full((p.rows, H * pad8(dv)), 9.0, dtype=run[1], device=run[0])
         ops.differential_attention(qn, kc, vc, out, p, H, scale, l4, diff, dv, eps, g, window, cap)
         near(out.float().cpu().reshape(p.rows, H, -1)[:, :, :dv],
