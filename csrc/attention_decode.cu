@@ -16,7 +16,11 @@
 
 namespace b2 {
 
-constexpr int AD_PAGE = 16, AD_WARPS = 8, AD_THREADS = (AD_WARPS + 1) * 32;
+constexpr int AD_PAGE = 16, AD_WARPS = 8, AD_THREADS = (AD_WARPS + 4) * 32;
+// registers a thread is launched with (three warps on each quarter of the SM), and what the copying and the computing warpgroups
+// take of them: 128 x 40 + 256 x 232 <= 384 x 168
+constexpr int AD_REGS = 168, AD_REGS_COPY = 40, AD_REGS_MATH = 232;
+static_assert(128 * AD_REGS_COPY + AD_WARPS * 32 * AD_REGS_MATH <= AD_THREADS * AD_REGS, "register split");
 constexpr float AD_LOG2E = 1.4426950408889634f;
 typedef __nv_bfloat16 ad_bf16;
 
@@ -129,12 +133,6 @@ struct DecodeSmem {
     total = bars + 256 + 16 * 8 * 4 + 1024;
   }
 };
-// channel c (a multiple of 8) of key k in a swizzled tile
-template <int KT>
-__device__ __forceinline__ const ad_bf16* ad_at(const uint8_t* tile, int k, int c) {
-  return reinterpret_cast<const ad_bf16*>(tile + (c >> 6) * (KT * 128) + k * 128 + ((((c >> 3) & 7) ^ (k & 7)) << 4));
-}
-
 __device__ __forceinline__ void ad_consumer_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 template <int HALVES, int QP, int NG>   // QP: 32-channel steps of a warp's share of the keys; NG: 16-channel pieces of values per warp
@@ -169,11 +167,12 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
   const int kq = p.R / p.maps;
 
   // A wait that runs out sets the status word; everyone runs on to the end (later waits return at once).
-  if (warp == AD_WARPS) {
+  if (warp >= AD_WARPS) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(AD_REGS_COPY));
     int st = 0, seg = 0;
     uint32_t ph = 0;
     const int parts = L.kparts + L.vparts;
-    for (int x = x0; x < x1; ++seg) {
+    for (int x = warp == AD_WARPS ? x0 : x1; x < x1; ++seg) {      // one warp of the group copies
       const int t1 = min(a.n, a.t + x1 - x), kvh = a.group / p.hgroups, head0 = kvh * (p.H / p.G) + a.group % p.hgroups * p.heads;
       const int rows = min(p.heads, (kvh + 1) * (p.H / p.G) - head0) * p.maps, qs = seg & 1;
       const int pos = p.pos[a.row], first = ad_first(pos, p.window);
@@ -206,11 +205,21 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
       if (x < x1) ad_next(p, groups, a);
     }
   } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(AD_REGS_MATH));
     const int kg = warp % (8 / HALVES), kh = warp / (8 / HALVES);       // this warp's eight keys and half of the channels
-    const int steps = (p.R + 31) / 32, mine = HALVES == 1 ? steps : kh ? steps / 2 : (steps + 1) / 2, c0 = kh ? (steps + 1) / 2 * 32 : 0;
+    const int steps = (p.R + 31) / 32, cut = HALVES == 1 ? steps : (L.kparts + 1) / 2 * 2;      // 32-channel steps of the first half
+    const int mine = kh ? max(steps - cut, 0) : min(cut, steps), c0 = kh * cut * 32;
     const float lam = p.maps == 2 ? diff_lambda(p.lam, kq, p.lam_init) : 0.f;
     const float sl2 = p.scale * AD_LOG2E;
+    const float cap_in = p.softcap > 0.f ? p.scale / p.softcap : 0.f, cap_out = p.softcap * AD_LOG2E;
     const int qld = L.pitch / 2;        // in elements
+    // this lane's rows of the ldmatrix reads inside a [keys x 64 channels] piece: even and odd 32-channel steps of the keys, the
+    // warp's 16-channel pieces of the values
+    uint32_t koff[2], voff[NG];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) koff[i] = (kg * 8 + (lane & 7)) * 128 + (((i * 4 + (lane >> 3)) ^ (lane & 7)) << 4);
+#pragma unroll
+    for (int g = 0; g < NG; ++g) voff[g] = (lane & 15) * 128 + (((((warp + 8 * g) * 2 + (lane >> 4)) & 7) ^ (lane & 7)) << 4);
     int st = 0, seg = 0, buf = 0;
     uint32_t ph = 0;
     for (int x = x0; x < x1; ++seg) {
@@ -235,33 +244,72 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
       for (int g = 0; g < NG; ++g)
 #pragma unroll
         for (int i = 0; i < 8; ++i) acc[g][i >> 2][i & 3] = 0.f;
-      for (int t = a.t; t < t1; ++t) {
-        mbar_wait_warp(&full[st], ph, status, ERR_ATTN_WAIT);
-        const uint8_t* tile = ad_smem + st * L.stage;
-        float* S = reinterpret_cast<float*>(ad_smem + L.s) + buf * HALVES * 16 * LDS;
-        buf ^= 1;
-        {
-          float d[2][4] = {};
+      // Scores of the tile in stage `at`, scaled to the base-2 domain.  The products of one tile run under the softmax of the one
+      // before: nothing waits for them until they are written to the exchange buffer.
+      auto scores = [&](int at, float (&d)[2][4]) {
+        const uint8_t* tile = ad_smem + at * L.stage + c0 * (KT * 2);
 #pragma unroll
-          for (int i = 0; i < QP; ++i)
-            if (i < mine) {
-              uint32_t b[4];
-              ldsm_x4(ad_at<KT>(tile, kg * 8 + (lane & 7), c0 + i * 32 + (lane >> 3) * 8), b);
-              const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
-              mma_bf16(d[0], q[i][0], b0);
-              mma_bf16(d[1], q[i][1], b1);
+        for (int i = 0; i < 8; ++i) d[i >> 2][i & 3] = 0.f;
+        constexpr int BATCH = 4;
+#pragma unroll
+        for (int i0 = 0; i0 < QP; i0 += BATCH) {
+          uint32_t b[BATCH][4];
+#pragma unroll
+          for (int i = 0; i < BATCH; ++i)
+            if (i0 + i < QP && i0 + i < mine) ldsm_x4(reinterpret_cast<const ad_bf16*>(tile + ((i0 + i) >> 1) * (KT * 128) + koff[(i0 + i) & 1]), b[i]);
+#pragma unroll
+          for (int i = 0; i < BATCH; ++i)
+            if (i0 + i < QP && i0 + i < mine) {
+              const uint32_t b0[2] = {b[i][0], b[i][1]}, b1[2] = {b[i][2], b[i][3]};
+              mma_bf16(d[0], q[i0 + i][0], b0);
+              mma_bf16(d[1], q[i0 + i][1], b1);
             }
+        }
+      };
+      auto publish = [&](float (&d)[2][4], float* S) {
+        float v[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] = d[0][i] + d[1][i];
+        if (HALVES == 1 && p.softcap > 0.f) {
+          float big = 0.f;
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            d[0][i] += d[1][i];
-            if (HALVES == 1 && p.softcap > 0.f) d[0][i] = softcap_t<ad_bf16>(d[0][i] * p.scale, p.softcap) * AD_LOG2E;
-            else d[0][i] *= sl2;
+            v[i] *= cap_in;
+            big = fmaxf(big, fabsf(v[i]));
           }
-          float* o = S + (kh * 16 + (lane >> 2)) * LDS + kg * 8 + (lane & 3) * 2;
-          *reinterpret_cast<float2*>(o) = make_float2(d[0][0], d[0][1]);
-          *reinterpret_cast<float2*>(o + 8 * LDS) = make_float2(d[0][2], d[0][3]);
+          if (__any_sync(0xffffffffu, big > SOFTCAP_SERIES)) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[i] = cap_out * tanh_wide(v[i]);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[i] = cap_out * tanh_series(v[i]);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) v[i] *= sl2;
         }
+        float* o = S + (kh * 16 + (lane >> 2)) * LDS + kg * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(o) = make_float2(v[0], v[1]);
+        *reinterpret_cast<float2*>(o + 8 * LDS) = make_float2(v[2], v[3]);
         ad_consumer_barrier();
+      };
+      float* const Sbuf = reinterpret_cast<float*>(ad_smem + L.s);
+      float d[2][4];
+      mbar_wait_warp(&full[st], ph, status, ERR_ATTN_WAIT);
+      scores(st, d);
+      publish(d, Sbuf + buf * (HALVES * 16 * LDS));
+      for (int t = a.t; t < t1; ++t) {
+        const int cur = st;
+        const float* S = Sbuf + buf * (HALVES * 16 * LDS);
+        buf ^= 1;
+        if (++st == p.stages) {
+          st = 0;
+          ph ^= 1;
+        }
+        if (t + 1 < t1) {
+          mbar_wait_warp(&full[st], ph, status, ERR_ATTN_WAIT);
+          scores(st, d);
+        }
         float s[KS][2][4];       // [16 keys][row, row + 8][key pairs 0, 1 and 8, 9 of this lane]
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks)
@@ -329,7 +377,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
         }
         l0 = l0 * f0 + p0;       // this lane's keys only; added over the four lanes of a row at the end
         l1 = l1 * f1 + p1;
-        const uint8_t* vt = tile + (p.apart ? L.kparts * (KT * 128) : 0);
+        const uint8_t* vt = ad_smem + cur * L.stage + (p.apart ? L.kparts * (KT * 128) : 0);
 #pragma unroll
         for (int g = 0; g < NG; ++g) {
           const int c = (warp + 8 * g) * 16;
@@ -344,15 +392,12 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
 #pragma unroll
           for (int ks = 0; ks < KS; ++ks) {
             uint32_t b[4];
-            ldsm_x4_t(ad_at<KT>(vt, ks * 16 + (lane & 15), c + (lane >> 4) * 8), b);
+            ldsm_x4_t(reinterpret_cast<const ad_bf16*>(vt + (c >> 6) * (KT * 128) + ks * 2048 + voff[g]), b);
             mma_n16(acc[g][0], acc[g][1], pa[ks], b);
           }
         }
-        mbar_arrive_warp(&empty[st]);
-        if (++st == p.stages) {
-          st = 0;
-          ph ^= 1;
-        }
+        mbar_arrive_warp(&empty[cur]);
+        if (t + 1 < t1) publish(d, Sbuf + buf * (HALVES * 16 * LDS));
       }
 #pragma unroll
       for (int o = 1; o < 4; o <<= 1) {
@@ -596,6 +641,6 @@ B2_EXPORT int b2_decode_attention(const void* q, const void* kc, const void* vc,
   const CUtensorMap *tk = map(kc, R), *tv = vc ? map(vc, C) : tk;
   if (!tk || !tv) return 2;
   if (vc) return launch_decode<1, 8, 1>(p, tk, tv, grid, st);
-  if (R <= 192 && C <= 128) return launch_decode<2, 3, 1>(p, tk, tv, grid, st);
-  return launch_decode<2, 9, 4>(p, tk, tv, grid, st);
+  if (R <= 192 && C <= 128) return launch_decode<2, 4, 1>(p, tk, tv, grid, st);
+  return launch_decode<2, 10, 4>(p, tk, tv, grid, st);
 }
