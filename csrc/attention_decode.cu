@@ -135,7 +135,9 @@ struct DecodeSmem {
 };
 __device__ __forceinline__ void ad_consumer_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-template <int HALVES, int QP, int NG>   // QP: 32-channel steps of a warp's share of the keys; NG: 16-channel pieces of values per warp
+// QP: 32-channel steps of a warp's share of the keys; NG: 16-channel pieces of values per warp; EXACT: the sizes fill both, so that
+// the loops over them have no conditions.
+template <int HALVES, int QP, int NG, bool EXACT>
 __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const DecodeParams p, int* status) {
   constexpr int KT = 64 / HALVES, LDS = KT + 8, KS = KT / 16, PAGES = KT / AD_PAGE;
   extern __shared__ uint8_t ad_raw[];
@@ -183,16 +185,20 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
       if (lane < rows)
         bulk_load(ad_smem + L.q + (qs * 16 + lane) * L.pitch + lane % p.maps * kq * 2,
                   p.q + a.row * p.ld_q + static_cast<size_t>(head0 * p.maps + lane) * kq, kq * 2, &q_full[qs]);
+      // boxes (page, part): pages past the row's last repeat it, those keys are masked.  A lane always copies the same page of a
+      // tile; its number is fetched one tile ahead.
+      static_assert(32 % PAGES == 0, "a lane's boxes share a page");
+      const int mypage = first / AD_PAGE + lane % PAGES, last = pos / AD_PAGE;
+      int next = table[min(mypage + a.t * PAGES, last)];
       for (int t = a.t; t < t1; ++t) {
-        // boxes (page, part): pages past the row's last repeat it, those keys are masked
-        const int pg0 = (first + t * KT) / AD_PAGE, last = pos / AD_PAGE;
+        const int token = next * AD_PAGE;
+        next = table[min(mypage + (t + 1) * PAGES, last)];
         mbar_wait_warp(&empty[st], ph ^ 1, status, ERR_ATTN_WAIT);
         if (lane == 0) mbar_expect_tx(&full[st], parts * KT * 128);
         __syncwarp();
-        uint8_t* tile = ad_smem + st * L.stage;
-        for (int i = lane; i < parts * PAGES; i += 32) {
-          const int pg = i % PAGES, part = i / PAGES, token = table[min(pg0 + pg, last)] * AD_PAGE;
-          uint8_t* dst = tile + part * (KT * 128) + pg * (AD_PAGE * 128);
+        uint8_t* tile = ad_smem + st * L.stage + lane % PAGES * (AD_PAGE * 128);
+        for (int part = lane / PAGES; part < parts; part += 32 / PAGES) {
+          uint8_t* dst = tile + part * (KT * 128);
           if (part < L.kparts) tma_load_3d(dst, &tmK, &full[st], part * 64, kvh, token);
           else tma_load_3d(dst, &tmV, &full[st], (part - L.kparts) * 64, kvh, token);
         }
@@ -207,17 +213,18 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
   } else {
     asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(AD_REGS_MATH));
     const int kg = warp % (8 / HALVES), kh = warp / (8 / HALVES);       // this warp's eight keys and half of the channels
-    const int steps = (p.R + 31) / 32, cut = HALVES == 1 ? steps : (L.kparts + 1) / 2 * 2;      // 32-channel steps of the first half
-    const int mine = kh ? max(steps - cut, 0) : min(cut, steps), c0 = kh * cut * 32;
+    const int steps = EXACT ? HALVES * QP : (p.R + 31) / 32, cut = HALVES == 1 ? steps : (steps + 1) / 2;   // 32-channel steps of the first half
+    const int mine = kh ? steps - cut : cut, first_step = kh * cut, c0 = first_step * 32;
     const float lam = p.maps == 2 ? diff_lambda(p.lam, kq, p.lam_init) : 0.f;
     const float sl2 = p.scale * AD_LOG2E;
     const float cap_in = p.softcap > 0.f ? p.scale / p.softcap : 0.f, cap_out = p.softcap * AD_LOG2E;
     const int qld = L.pitch / 2;        // in elements
-    // this lane's rows of the ldmatrix reads inside a [keys x 64 channels] piece: even and odd 32-channel steps of the keys, the
+    // this lane's rows of the ldmatrix reads inside a [keys x 64 channels] piece: the warp's even and odd 32-channel steps of the keys, the
     // warp's 16-channel pieces of the values
     uint32_t koff[2], voff[NG];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) koff[i] = (kg * 8 + (lane & 7)) * 128 + (((i * 4 + (lane >> 3)) ^ (lane & 7)) << 4);
+    for (int i = 0; i < 2; ++i)
+      koff[i] = ((first_step + i) >> 1) * (KT * 128) + (kg * 8 + (lane & 7)) * 128 + (((((first_step + i) & 1) * 4 + (lane >> 3)) ^ (lane & 7)) << 4);
 #pragma unroll
     for (int g = 0; g < NG; ++g) voff[g] = (lane & 15) * 128 + (((((warp + 8 * g) * 2 + (lane >> 4)) & 7) ^ (lane & 7)) << 4);
     int st = 0, seg = 0, buf = 0;
@@ -233,7 +240,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
         const ad_bf16* sq = reinterpret_cast<const ad_bf16*>(ad_smem + L.q + qs * 16 * L.pitch) + c0;
 #pragma unroll
         for (int i = 0; i < QP; ++i)
-          if (i < mine) {
+          if (EXACT || i < mine) {
             ldsm_a_mk(sq + i * 32, qld, lane, q[i][0]);
             ldsm_a_mk(sq + i * 32 + 16, qld, lane, q[i][1]);
           }
@@ -247,7 +254,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
       // Scores of the tile in stage `at`, scaled to the base-2 domain.  The products of one tile run under the softmax of the one
       // before: nothing waits for them until they are written to the exchange buffer.
       auto scores = [&](int at, float (&d)[2][4]) {
-        const uint8_t* tile = ad_smem + at * L.stage + c0 * (KT * 2);
+        const uint8_t* tile = ad_smem + at * L.stage;
 #pragma unroll
         for (int i = 0; i < 8; ++i) d[i >> 2][i & 3] = 0.f;
         constexpr int BATCH = 4;
@@ -256,10 +263,10 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
           uint32_t b[BATCH][4];
 #pragma unroll
           for (int i = 0; i < BATCH; ++i)
-            if (i0 + i < QP && i0 + i < mine) ldsm_x4(reinterpret_cast<const ad_bf16*>(tile + ((i0 + i) >> 1) * (KT * 128) + koff[(i0 + i) & 1]), b[i]);
+            if (i0 + i < QP && (EXACT || i0 + i < mine)) ldsm_x4(reinterpret_cast<const ad_bf16*>(tile + ((i0 + i) >> 1) * (KT * 128) + koff[(i0 + i) & 1]), b[i]);
 #pragma unroll
           for (int i = 0; i < BATCH; ++i)
-            if (i0 + i < QP && i0 + i < mine) {
+            if (i0 + i < QP && (EXACT || i0 + i < mine)) {
               const uint32_t b0[2] = {b[i][0], b[i][1]}, b1[2] = {b[i][2], b[i][3]};
               mma_bf16(d[0], q[i0 + i][0], b0);
               mma_bf16(d[1], q[i0 + i][1], b1);
@@ -381,7 +388,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
 #pragma unroll
         for (int g = 0; g < NG; ++g) {
           const int c = (warp + 8 * g) * 16;
-          if (c >= p.C) break;
+          if (!EXACT && c >= p.C) break;
 #pragma unroll
           for (int n = 0; n < 2; ++n) {
             acc[g][n][0] *= f0;
@@ -557,10 +564,10 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(const DecodeParams p,
         make_uint2(pack_bf16x2(o[0][0], o[0][1]), pack_bf16x2(o[0][2], o[0][3]));
 }
 
-template <int HALVES, int QP, int NG>
+template <int HALVES, int QP, int NG, bool EXACT>
 static int launch_decode(DecodeParams& p, const CUtensorMap* tk, const CUtensorMap* tv, int grid, cudaStream_t stream) {
   constexpr int KT = 64 / HALVES;
-  auto kern = decode_attn_kernel<HALVES, QP, NG>;
+  auto kern = decode_attn_kernel<HALVES, QP, NG, EXACT>;
   int stages = 8;
   while (stages > 2 && DecodeSmem(p.R, p.C, p.apart, KT, HALVES, stages).total > 232448) --stages;
   const int smem = DecodeSmem(p.R, p.C, p.apart, KT, HALVES, stages).total;
@@ -640,7 +647,6 @@ B2_EXPORT int b2_decode_attention(const void* q, const void* kc, const void* vc,
   };
   const CUtensorMap *tk = map(kc, R), *tv = vc ? map(vc, C) : tk;
   if (!tk || !tv) return 2;
-  if (vc) return launch_decode<1, 8, 1>(p, tk, tv, grid, st);
-  if (R <= 192 && C <= 128) return launch_decode<2, 4, 1>(p, tk, tv, grid, st);
-  return launch_decode<2, 10, 4>(p, tk, tv, grid, st);
+  if (vc) return R == 256 && C == 128 ? launch_decode<1, 8, 1, true>(p, tk, tv, grid, st) : launch_decode<1, 8, 1, false>(p, tk, tv, grid, st);
+  return R == 576 && C == 512 ? launch_decode<2, 9, 4, true>(p, tk, tv, grid, st) : launch_decode<2, 9, 4, false>(p, tk, tv, grid, st);
 }
