@@ -163,12 +163,13 @@ inference_preview: {{enabled: false, max_tokens: 4}}
     assert json.loads(r.stdout[r.stdout.index("{"):])["completed_iterations"] == 2
 
 
-def test_run_inference_serves_a_hybrid_model(tmp_path):
+@pytest.mark.parametrize("preset", ["fetelorn-tiny", "sotazen-tiny"])
+def test_run_inference_serves_a_hybrid_model(tmp_path, preset):
     """The architecture follows from the folder's config.json; the same flags as for any other model."""
     import torch
 
     from b200fw.model import registry
-    m = registry.build_model(registry.PRESETS["fetelorn-tiny"], dtype=torch.bfloat16, device="cpu")
+    m = registry.build_model(registry.PRESETS[preset], dtype=torch.bfloat16, device="cpu")
     m.init_weights(3)
     registry.save_checkpoint(m, str(tmp_path))
     r = subprocess.run([sys.executable, os.path.join(ROOT, "scripts", "run_inference.py"), "-m", str(tmp_path), "--num-prompts", "3",

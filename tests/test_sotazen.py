@@ -209,7 +209,7 @@ def loud_keys(T, window, seed):
 @pytest.mark.parametrize("H,G,dk,dv,window,rot,cap", [
     (6, 2, 12, 20, 24, 8, 20.0), (5, 1, 9, 7, 37, 6, 3.0), (4, 2, 128, 96, 150, 64, 30.0), (4, 1, 96, 128, 128, 96, 8.0),
     (8, 1, 64, 64, 17, 2, 50.0), (2, 2, 160, 24, 40, 12, 15.0), (3, 3, 128, 128, 1, 128, 50.0), (2, 1, 64, 128, 1000, 32, 100.0),
-    (1, 1, 24, 72, 129, 24, 6.0)])
+    (1, 1, 24, 72, 129, 24, 6.0), (2, 1, 24, 136, 30, 8, 25.0), (9, 1, 32, 40, 33, 16, 9.0)])
 def test_differential_attention(run, H, G, dk, dv, window, rot, cap):
     """One loud key per query and map at a time, the two maps' apart.  A key that is wrongly seen, or missed, takes the whole
     softmax with it; a cap that is left out sharpens every score."""
@@ -266,7 +266,8 @@ def test_differential_attention(run, H, G, dk, dv, window, rot, cap):
 
 @pytest.mark.parametrize("run", RUNS)
 @pytest.mark.parametrize("H,dim,rot,dv,rank", [(3, 11, 6, 13, 20), (4, 64, 16, 64, 64), (2, 128, 64, 128, 512), (18, 96, 32, 64, 128),
-                                               (1, 160, 32, 24, 40), (2, 40, 24, 136, 72), (5, 128, 8, 128, 264), (2, 24, 2, 8, 600)])
+                                               (1, 160, 32, 24, 40), (2, 40, 24, 136, 72), (5, 128, 8, 128, 264), (2, 24, 2, 8, 600),
+                                               (2, 180, 20, 32, 16)])
 def test_latent_attention(run, H, dim, rot, dv, rank):
     """One loud key per query: far away, on page borders, the first token, the query's own; and a sink that weighs in."""
     eps, base = 1e-6, 300.0
@@ -306,6 +307,45 @@ def test_latent_attention(run, H, dim, rot, dv, rank):
         ops.latent_attention(q, pages, out, p, w_key, w_value, scale, snk)
         near(out.float().cpu().reshape(p.rows, H, -1)[:, :, :dv],
              torch.cat([want[s][starts[s]:starts[s] + cnt[s]] for s in order]).float(), run)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("rows,longest", [(1, 900), (3, 40), (300, 500), (1100, 90)])
+def test_decoded_rows_of_ragged_lengths(rows, longest):
+    """One token for each of many sequences, padding rows among them: the work split over the SMs cuts rows anywhere.  Against the
+    32-bit kernels on the same numbers."""
+    r = random.Random(rows)
+    lens = [r.choice([1, 2, 15, 16, 17, 31, 32, 33, 64, 65, r.randrange(1, longest)]) for _ in range(rows)]
+    lens[-1] = longest
+    pads = [i for i in range(rows - 1) if i % 7 == 3]
+    need = [-(-n // 16) for n in lens]
+    ids, tables = list(range(sum(need))), []
+    r.shuffle(ids)
+    for n in need:
+        tables.append(ids[:n])
+        ids = ids[n:]
+    slots = [-1 if i in pads else i for i in range(rows)]
+    p, _, _ = build_portions([n - 1 for n in lens], [1] * rows, tables, slots, False, lambda a: torch.from_numpy(a).to("cuda"))
+    bf = lambda *s, seed: randn(*s, seed=seed).bfloat16().to("cuda")  # noqa: E731
+    live = torch.tensor([i for i in range(rows) if i not in pads], device="cuda")
+
+    def same(f, width):
+        outs = []
+        for dt in (torch.bfloat16, torch.float32):
+            out = torch.full((rows, width), 9.0, dtype=dt, device="cuda")
+            f(out, lambda t: t.to(dt))
+            outs.append(out.float()[live])
+        assert torch.isfinite(outs[0]).all()
+        d = (outs[0] - outs[1]).pow(2).mean(-1).sqrt() / outs[1].std()
+        assert d.max() < 0.05, float(d.max())
+    for H, G, d, dv, window, cap in ((8, 4, 128, 128, 0, 50.0), (6, 2, 24, 40, 37, 2.0), (20, 1, 64, 64, 100, 30.0)):
+        q, kc, vc = bf(rows, 2 * H * d, seed=1) * 2, bf(sum(need), 16, 2 * G, d, seed=2), bf(sum(need), 16, G, dv, seed=3)
+        lam, gate = bf(4, d, seed=4) * 0.1, bf(rows, H * dv, seed=5)
+        same(lambda o, c: ops.differential_attention(c(q), c(kc), c(vc), o, p, H, d ** -0.5, c(lam), 0.4, dv, 1e-6, c(gate), window, cap),
+             H * dv)
+    for H, R, C in ((8, 576, 512), (3, 80, 64), (18, 336, 264), (16, 24, 16)):
+        q, pages, sink = bf(rows, H * R, seed=1), bf(sum(need), 16, 1, R, seed=2), bf(H, seed=3) + 2
+        same(lambda o, c: ops.latent_rows(c(q), c(pages), o, p, H, C, 2 * R ** -0.5, c(sink)), H * C)
 
 
 @pytest.mark.gpu

@@ -10,11 +10,16 @@ import pytest
 import torch
 
 import fetelorn_oracle as O
+import sotazen_oracle as SO
+import test_sotazen as S
 from test_fetelorn import bf16_exact, build, config, parallel, retention, toks
 from b200fw.model import ModelConfig, ParallelTransformerModel, registry
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CFG = config(36, 51, [parallel(2, 1, 16, 8, 20, 12, 2, 1, 16, 24, 5, ff=16), retention(2, 8, 16, 4, ff=16)])
+
+SOTAZEN = S.config(36, 51, [S.latent(2, 16, 8, 12, 24, ff=16), S.lightning(2, 8, 16, ff=None), S.differential(2, 1, 16, 8, 19, 4, ff=16)])
+MODELS = {"Fetelorn": (CFG, O, build), "Sotazen": (SOTAZEN, SO, S.build)}
 
 
 def replay(model_dir, out, steps, max_tokens, device, dtype="float32"):
@@ -58,9 +63,11 @@ def schedule(seqs, cuts_by_seq):
 
 @pytest.mark.parametrize("device,dtype", [("cpu", "float32"), pytest.param("cuda", "float32", marks=pytest.mark.gpu),
                                           pytest.param("cuda", "bfloat16", marks=pytest.mark.gpu)])
-def test_replay(tmp_path, device, dtype):
-    w = bf16_exact(O.random_weights(CFG, 4))
-    registry.save_checkpoint(build(CFG, w, ("cpu", torch.float32)), str(tmp_path / "m"))
+@pytest.mark.parametrize("design", list(MODELS))
+def test_replay(tmp_path, design, device, dtype):
+    cfg, oracle, make = MODELS[design]
+    w = bf16_exact(oracle.random_weights(cfg, 4))
+    registry.save_checkpoint(make(cfg, w, ("cpu", torch.float32)), str(tmp_path / "m"))
     lens = [33, 18, 25, 40, 9]
     seqs = [toks(n, 51, n) for n in lens]
     cuts = [[20, 1, 12], [17, 1], [2, 3, 20], [39, 1], [9]]
@@ -68,7 +75,7 @@ def test_replay(tmp_path, device, dtype):
     # three requests are live at a time at most: the pool is made for that, not for all five
     rc, done, err = replay(tmp_path / "m", tmp_path / "o", steps, 192, device, dtype)
     assert rc == 0 and done == [s["step"] for s in steps], err[-2000:]
-    want = [O.forward(CFG, w, s).float().numpy() for s in seqs]
+    want = [oracle.forward(cfg, w, s).float().numpy() for s in seqs]
     at = {}
     for s in steps:
         rows = []
