@@ -399,18 +399,32 @@ struct NormStoreParams {
 
 // Bias, per-head RMS norm of q and k (optional weights), rotary positions on channel pairs (2 i, 2 i + 1), and the store of k / v.
 // Grid (M, y).  LPH lanes per head, eight channels each; a lane takes NS_UNROLL heads of its row at a time, their loads together.
+// What waits in registers waits packed, so that eight CTAs fit on an SM.
 constexpr int NS_UNROLL = 4;
+template <typename T>
+struct Packed8 {
+  uint4 w[sizeof(T) / 2];
+  __device__ __forceinline__ void load(const T* p) {
+#pragma unroll
+    for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) w[i] = reinterpret_cast<const uint4*>(p)[i];
+  }
+  __device__ __forceinline__ void zero() {
+#pragma unroll
+    for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) w[i] = make_uint4(0, 0, 0, 0);
+  }
+  __device__ __forceinline__ void get(float (&f)[8]) const { vload8(reinterpret_cast<const T*>(w), f); }
+};
 template <typename T, int LPH>
-__global__ void __launch_bounds__(128) qk_norm_store_kernel(const NormStoreParams p) {
+__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 8 : 4) qk_norm_store_kernel(const NormStoreParams p) {
   constexpr int GROUPS = 128 / LPH;
   const int group = threadIdx.x / LPH, c = threadIdx.x % LPH * 8, units = p.H + p.G + p.Gv;
   const int stride = GROUPS * gridDim.y;
   const bool kin = c < p.dkp, vin = c < p.dvp;
-  float wq[8], wk[8];
-#pragma unroll
-  for (int e = 0; e < 8; ++e) wq[e] = wk[e] = 1.f;
-  if (p.wq && kin) vload8(static_cast<const T*>(p.wq) + c, wq);
-  if (p.wk && kin) vload8(static_cast<const T*>(p.wk) + c, wk);
+  Packed8<T> wq, wk;
+  wq.zero();
+  wk.zero();
+  if (p.wq && kin) wq.load(static_cast<const T*>(p.wq) + c);
+  if (p.wk && kin) wk.load(static_cast<const T*>(p.wk) + c);
   for (size_t row = blockIdx.x; row < static_cast<size_t>(p.M); row += gridDim.x) {
     const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row), pos = p.pos[row];
     const bool live = p.slot == nullptr || p.slot[s] >= 0;
@@ -437,7 +451,7 @@ __global__ void __launch_bounds__(128) qk_norm_store_kernel(const NormStoreParam
       }
     }
     for (int w0 = blockIdx.y * GROUPS + group; __any_sync(0xffffffffu, w0 < units); w0 += stride * NS_UNROLL) {
-      float t[NS_UNROLL][8];
+      Packed8<T> raw[NS_UNROLL];
       auto part = [&](int w, const void* q, const void* k, const void* v) {      // the head's columns in a row of q | k | v
         return w < p.H ? static_cast<const T*>(q) + static_cast<size_t>(w) * p.dkp
                        : w < p.H + p.G ? static_cast<const T*>(k) + static_cast<size_t>(w - p.H) * p.dkp
@@ -446,44 +460,52 @@ __global__ void __launch_bounds__(128) qk_norm_store_kernel(const NormStoreParam
 #pragma unroll
       for (int i = 0; i < NS_UNROLL; ++i) {
         const int w = w0 + i * stride;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) t[i][e] = 0.f;
-        if (w < units && (w < p.H + p.G ? kin : vin)) vload8(part(w, p.q, p.k, p.v) + row * p.ld + c, t[i]);
+        raw[i].zero();
+        if (w < units && (w < p.H + p.G ? kin : vin)) raw[i].load(part(w, p.q, p.k, p.v) + row * p.ld + c);
       }
 #pragma unroll
       for (int i = 0; i < NS_UNROLL; ++i) {
         const int w = w0 + i * stride;
+        float t[8];
+        raw[i].get(t);
         const bool qk = w < p.H + p.G, in = w < units && (qk ? kin : vin);
         if (p.bq && in) {
           float b[8];
           vload8(part(w, p.bq, p.bk, p.bv) + c, b);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) t[i][e] += b[e];
+          for (int e = 0; e < 8; ++e) t[e] += b[e];
         }
         if (p.norm) {
           float ss = 0.f;
 #pragma unroll
-          for (int e = 0; e < 8; ++e) ss = fmaf(t[i][e], t[i][e], ss);
+          for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
 #pragma unroll
           for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
           const float r = rsqrtf(ss / p.dk + p.eps);
-          if (qk)
+          if (qk) {
+            if (w < p.H ? p.wq != nullptr : p.wk != nullptr) {
+              float g[8];
+              (w < p.H ? wq : wk).get(g);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) t[i][e] *= r * (w < p.H ? wq[e] : wk[e]);
+              for (int e = 0; e < 8; ++e) t[e] *= g[e];
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) t[e] *= r;
+          }
         }
         if (p.cs && qk) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const float u = t[i][2 * e], x = t[i][2 * e + 1];
-            t[i][2 * e] = u * co[e] - x * si[e];
-            t[i][2 * e + 1] = x * co[e] + u * si[e];
+            const float u = t[2 * e], x = t[2 * e + 1];
+            t[2 * e] = u * co[e] - x * si[e];
+            t[2 * e + 1] = x * co[e] + u * si[e];
           }
         }
         if (!in || (w >= p.H && !live)) continue;
         T* dst = w < p.H ? static_cast<T*>(p.q_out) + (row * p.H + w) * p.dkp
                          : qk ? static_cast<T*>(p.kc) + (at * p.G + w - p.H) * p.dkp
                               : static_cast<T*>(p.vc) + (at * p.Gv + w - p.H - p.G) * p.dvp;
-        vstore8(dst + c, t[i]);
+        vstore8(dst + c, t);
       }
     }
   }
@@ -588,7 +610,7 @@ B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long
   const int w = dkp > dvp ? dkp : dvp, lph = w <= 64 ? 8 : w <= 128 ? 16 : 32, groups = 128 / lph;
   int y = (H + G + Gv + groups - 1) / groups;              // a head per lane group; several when the rows fill the GPU
   if (M >= 8 * num_sms()) y = (y + NS_UNROLL - 1) / NS_UNROLL;
-  const dim3 grid(M < 10 * num_sms() ? M : 10 * num_sms(), y);
+  const dim3 grid(M < 16 * num_sms() ? M : 16 * num_sms(), y);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   B2_DISPATCH_T(is_f32, {
     if (lph == 8) qk_norm_store_kernel<T, 8><<<grid, 128, 0, st>>>(p);
