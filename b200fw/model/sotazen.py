@@ -234,8 +234,8 @@ def sotazen_preset(width: int, heads: int, depth: int, ff: int, vocab: int, kv_h
                 "rot": {"base": 10000.0, "dims": rot}}}
         elif i % every == every - 2:
             l = {"type": "attention", "mixer": {
-                "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
-                "mask": {"size": window}, "rot": {"base": 10000.0, "dims": dim}, "diff": 0.5}}
+                "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 30.0,
+                "mask": {"size": window}, "rot": {"base": 10000.0, "dims": dim}, "diff": 0.4}}
         else:
             l = {"type": "lightning", "mixer": {
                 "heads": heads, "dim": dim, "vdim": dim,

@@ -7,8 +7,7 @@
 // divides is left as partial sums, two slots per CTA, for the merge kernel, which has one block per cut and head.
 //
 // Inside a CTA one warp copies (TMA boxes of one page by 64 channels into 128-byte-swizzled tiles, a ring of stages that runs ahead
-// over the ends of rows) and eight compute.  Scores: each warp a group of
-// eight keys, and with HALVES = 2 half of the channels.  They meet in shared memory, double-buffered: one barrier per tile.  Every
+// over the ends of rows) and eight compute.  Scores: each warp a group of eight keys, and with HALVES = 2 half of the channels.  They meet in shared memory, double-buffered: one barrier per tile.  Every
 // warp then takes the softmax of the whole tile in the layout of its next operand, and multiplies 16-channel pieces of the values.
 #include "host.h"
 #include "mma_split.cuh"

@@ -208,7 +208,7 @@ def loud_keys(T, window, seed):
 @pytest.mark.parametrize("run", RUNS)
 @pytest.mark.parametrize("H,G,dk,dv,window,rot,cap", [
     (6, 2, 12, 20, 24, 8, 20.0), (5, 1, 9, 7, 37, 6, 3.0), (4, 2, 128, 96, 150, 64, 30.0), (4, 1, 96, 128, 128, 96, 8.0),
-    (8, 1, 64, 64, 17, 2, 50.0), (2, 2, 160, 24, 40, 12, 15.0), (3, 3, 128, 128, 1, 128, 50.0), (2, 1, 64, 128, 1000, 32, 100.0),
+    (8, 1, 64, 64, 17, 2, 45.0), (2, 2, 160, 24, 40, 12, 15.0), (3, 3, 128, 128, 1, 128, 35.0), (2, 1, 64, 128, 1000, 32, 100.0),
     (1, 1, 24, 72, 129, 24, 6.0), (2, 1, 24, 136, 30, 8, 25.0), (9, 1, 32, 40, 33, 16, 9.0)])
 def test_differential_attention(run, H, G, dk, dv, window, rot, cap):
     """One loud key per query and map at a time, the two maps' apart.  A key that is wrongly seen, or missed, takes the whole
@@ -265,7 +265,7 @@ def test_differential_attention(run, H, G, dk, dv, window, rot, cap):
 
 
 @pytest.mark.parametrize("run", RUNS)
-@pytest.mark.parametrize("H,dim,rot,dv,rank", [(3, 11, 6, 13, 20), (4, 64, 16, 64, 64), (2, 128, 64, 128, 512), (18, 96, 32, 64, 128),
+@pytest.mark.parametrize("H,dim,rot,dv,rank", [(3, 11, 6, 13, 20), (4, 72, 24, 64, 80), (2, 128, 64, 128, 512), (18, 96, 32, 64, 128),
                                                (1, 160, 32, 24, 40), (2, 40, 24, 136, 72), (5, 128, 8, 128, 264), (2, 24, 2, 8, 600),
                                                (2, 180, 20, 32, 16)])
 def test_latent_attention(run, H, dim, rot, dv, rank):
@@ -338,7 +338,7 @@ def test_decoded_rows_of_ragged_lengths(rows, longest):
         assert torch.isfinite(outs[0]).all()
         d = (outs[0] - outs[1]).pow(2).mean(-1).sqrt() / outs[1].std()
         assert d.max() < 0.05, float(d.max())
-    for H, G, d, dv, window, cap in ((8, 4, 128, 128, 0, 50.0), (6, 2, 24, 40, 37, 2.0), (20, 1, 64, 64, 100, 30.0)):
+    for H, G, d, dv, window, cap in ((8, 4, 128, 128, 0, 40.0), (6, 2, 24, 40, 37, 2.0), (20, 1, 64, 64, 100, 30.0)):
         q, kc, vc = bf(rows, 2 * H * d, seed=1) * 2, bf(sum(need), 16, 2 * G, d, seed=2), bf(sum(need), 16, G, dv, seed=3)
         lam, gate = bf(4, d, seed=4) * 0.1, bf(rows, H * dv, seed=5)
         same(lambda o, c: ops.differential_attention(c(q), c(kc), c(vc), o, p, H, d ** -0.5, c(lam), 0.4, dv, 1e-6, c(gate), window, cap),
