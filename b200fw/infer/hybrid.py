@@ -29,7 +29,9 @@ class HybridModelRunner(ModelRunner):
                  enable_partitioned: bool = False):
         super().__init__(model, pool, manager, partition_size, enable_partitioned)
         self.state: StatePool = manager.state
-        self._turns: Dict[Tuple[float, int], torch.Tensor] = {}
+        self._turns: Dict[tuple, torch.Tensor] = {}
+        # whose pages a layer reads: its own, or those of an earlier layer
+        self._pages = [li if src is None else src for li, src in enumerate(getattr(model, "kv_sources", lambda: [None] * len(model.layers))())]
 
     # ---- metadata ----------------------------------------------------------------------------------------
     def prepare_prefill(self, seq_ids: Sequence, starts: Sequence[int], counts: Sequence[int]) -> InferenceContext:
@@ -108,21 +110,22 @@ class HybridModelRunner(ModelRunner):
         m, p = self.model, ctx.portions
         self.forward_calls += 1
         ids = token_ids if ctx.row_order is None else token_ids.index_select(0, ctx.row_order)
+        p.ids = ids
         x, h = m.embed(ids)
-        tables: Dict[Tuple[float, int], Tuple[torch.Tensor, torch.Tensor]] = {}
+        tables: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
 
-        def rope(base: float, dims: int):
-            key = (base, dims)
+        def rope(base: float, dims: int, stretch: Optional[tuple] = None):
+            key = (base, dims, stretch)
             if key not in tables:
                 if key not in self._turns:
-                    self._turns[key] = ops.rope_turns(base, dims, self.device)
+                    self._turns[key] = ops.rope_turns(base, dims, self.device, stretch)
                 tables[key] = ops.rope_rows(p.positions, self._turns[key])
             return tables[key]
 
         n = len(m.layers)
         for li, layer in enumerate(m.layers):
             after = m.layers[li + 1].norm1 if li + 1 < n else None
-            h = layer(x, h, p, self.pool.layer_kv(li), self.state.layers[li], rope, after)
+            h = layer(x, h, p, self.pool.layer_kv(self._pages[li]), self.state.layers[li], rope, after)
             if on_layer is not None:
                 on_layer(li, x)
         if rows is not None:
@@ -131,7 +134,8 @@ class HybridModelRunner(ModelRunner):
             pick = ctx.row_place
         else:
             pick = ctx.last_token_rows if ctx.is_prefill else None
-        return m.logits_from_hidden(ops.rmsnorm_f32(x, m.norm, m.cfg.hidden_size, m.cfg.rms_norm_eps, pick))
+        return m.logits_from_hidden(ops.rmsnorm_f32(x, m.norm, m.cfg.hidden_size, m.cfg.rms_norm_eps, pick,
+                                                        getattr(m, "logit_scale", 1.0)))
 
     def run_batch_decode(self, *a, **k):
         raise NotImplementedError("raw-tensor decode knows no state slots: use prepare_decode + forward")

@@ -48,6 +48,28 @@ class RowSplitSlot:
         return torch.cat([slot.export() for slot, _ in self.parts])
 
 
+@dataclass
+class HalvesSlot:
+    """Per-head channels (dimension 1 of ``view [heads, d, ...]``) whose first ``rot`` are rotated in pairs of halves (channel i with
+    i + rot / 2) in the checkpoint and stored as neighbours (2 i, 2 i + 1): a score does not change when queries and keys are
+    reordered alike, and the kernels rotate neighbours."""
+    view: torch.Tensor
+    rot: int
+    shape: Tuple[int, ...]
+
+    def _order(self) -> torch.Tensor:
+        half, d = self.rot // 2, self.view.shape[1]
+        return torch.cat([torch.arange(self.rot).reshape(2, half).t().reshape(-1), torch.arange(self.rot, d)]).to(self.view.device)
+
+    def load(self, t: torch.Tensor) -> None:
+        self.view.copy_(t.to(self.view.device).reshape(self.view.shape)[:, self._order()].to(self.view.dtype))
+
+    def export(self) -> torch.Tensor:
+        out = torch.empty(self.view.shape, dtype=self.view.dtype, device=self.view.device)
+        out[:, self._order()] = self.view.detach()
+        return out.reshape(self.shape)
+
+
 def _param(*shape, dtype, device) -> nn.Parameter:
     return nn.Parameter(torch.zeros(*shape, dtype=dtype, device=device), requires_grad=False)
 
@@ -81,6 +103,10 @@ class PackedRows(nn.Module):
     def forward(self, x: torch.Tensor, act: Optional[str] = None, cols: Optional[int] = None) -> torch.Tensor:
         """``act`` on the first ``cols`` columns, in the product's epilogue (:func:`b200fw.ops.linear_act`)."""
         return ops.linear_act(x, self.weight, act, cols)
+
+    def fp32(self, x: torch.Tensor) -> torch.Tensor:
+        """The product with a 32-bit result."""
+        return ops.gemm(x, self.weight, out=torch.empty((x.shape[0], self.weight.shape[0]), dtype=torch.float32, device=x.device))
 
 
 class PackedCols(nn.Module):
@@ -429,3 +455,231 @@ class LatentAttention(nn.Module):
         out = self.o.buffer(y.shape[0])
         ops.latent_attention(q, kv[0], out, p, self.w_key, self.w_value, self.scale, self.sink)
         return self.o(out), {}
+
+
+class GatedFF(nn.Module):
+    """``W_down(silu(W_gate h) * (W_up h))``, a pair of products of its own: for layers whose feed-forward reads what the mixer
+    left and is normed before the sum."""
+
+    def __init__(self, hidden: int, inner: int, dtype, device):
+        super().__init__()
+        self.up = PackedRows(hidden, [("gate", 1, inner), ("up", 1, inner)], dtype, device)
+        self.down = PackedCols(hidden, [("down", 1, inner)], dtype, device)
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        return {prefix + "gate": self.up.slot("gate"), prefix + "up": self.up.slot("up"), prefix + "down": self.down.slot("down")}
+
+    def run(self, h: torch.Tensor) -> torch.Tensor:
+        """fp32 ``[M, hidden]``."""
+        y, a = self.up(h), self.down.buffer(h.shape[0])
+        ops.glu(self.up.cols(y, "gate"), self.up.cols(y, "up"), a)
+        return self.down(a)
+
+    def add(self, x: torch.Tensor, h: torch.Tensor, norm: torch.Tensor, coef: float, n: int, eps: float) -> torch.Tensor:
+        """``x += coef * norm(ff(h))``; the new ``x`` in the activation dtype."""
+        return ops.norm_add(x, self.run(h), norm, coef, n, eps)
+
+
+class ExpertFF(nn.Module):
+    """Mixture of gated feed-forward experts with sigmoid scores, a learned correction of the choice, a choice limited to the best
+    groups, and a shared expert behind a gate of its own.  Router logits and the shared gate are one 32-bit product."""
+
+    def __init__(self, hidden: int, experts: int, inner: int, top: int, groups: int, keep: int, scale: float,
+                 shared_inner: Optional[int], dtype, device):
+        super().__init__()
+        if groups < 1 or experts % groups or not 1 <= keep <= groups:
+            raise ValueError(f"experts: {experts} do not form {groups} equal groups of which {keep} are kept")
+        if not 1 <= top <= keep * (experts // groups):
+            raise ValueError(f"experts: cannot choose {top} among {keep} groups of {experts // groups}")
+        self.hidden, self.n, self.inner, self.top, self.groups, self.keep, self.scale = hidden, experts, inner, top, groups, keep, float(scale)
+        self.w_in = _param(experts, 2, pad8(inner), pad8(hidden), dtype=dtype, device=device)
+        self.w_out = _param(experts, pad8(hidden), pad8(inner), dtype=dtype, device=device)
+        self.correction = _param(experts, dtype=dtype, device=device)
+        self.shared = GatedFF(hidden, shared_inner, dtype, device) if shared_inner is not None else None
+        self.router = PackedRows(hidden, [("router", 1, experts)] + ([("sg", 1, 1)] if self.shared is not None else []), dtype, device)
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        H, F = self.hidden, self.inner
+        t: Dict[str, Slot] = {}
+        for e in range(self.n):
+            p = f"{prefix}e{e}."
+            t[p + "gate"], t[p + "up"] = (Slot(self.w_in.data[e, i, :F, :H], (F, H)) for i in range(2))
+            t[p + "down"] = Slot(self.w_out.data[e, :H, :F], (H, F))
+        t[prefix + "router"] = self.router.slot("router")
+        t[prefix + "correction"] = Slot(self.correction.data, (self.n,))
+        if self.shared is not None:
+            t |= self.shared.tensors(prefix + "shared.")
+            t[prefix + "shared.sg"] = self.router.slot("sg")
+        return t
+
+    def add(self, x: torch.Tensor, h: torch.Tensor, norm: torch.Tensor, coef: float, n: int, eps: float) -> torch.Tensor:
+        """``x += coef * norm(ff(h))``; the new ``x`` in the activation dtype."""
+        z = self.router.fp32(h)
+        r = ops.route(self.router.cols(z, "router"), self.correction, self.top, self.groups, self.keep, self.scale)
+        shared = gate = None
+        if self.shared is not None:
+            shared, gate = self.shared.run(h), self.router.cols(z, "sg")[:, 0]
+        rows = ops.expert_down(ops.expert_glu(h, self.w_in, r), self.w_out, r)
+        return ops.moe_norm_add(x, rows, r, shared, gate, norm, coef, n, eps)
+
+
+class TokenInput(nn.Module):
+    """A layer's own vector of the token, gated by the residual: ``x += coef * norm(W_proj (gelu(W_gate x) * e))``."""
+
+    def __init__(self, hidden: int, dim: int, layer: int, dtype, device):
+        super().__init__()
+        self.hidden, self.first = hidden, layer * pad8(dim)
+        self.gate = PackedRows(hidden, [("gate", 1, dim)], dtype, device)
+        self.proj = PackedCols(hidden, [("proj", 1, dim)], dtype, device)
+        self.norm = _param(pad8(hidden), dtype=dtype, device=device)
+
+    def tensors(self, prefix: str) -> Dict[str, Slot]:
+        return {prefix + "gate": self.gate.slot("gate"), prefix + "proj": self.proj.slot("proj"),
+                prefix + "norm": Slot(self.norm.data[:self.hidden], (self.hidden,))}
+
+    def add(self, x: torch.Tensor, h: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, vocab: int, coef: float, n: int,
+            eps: float) -> torch.Tensor:
+        g = ops.gelu_times_token(self.gate(h), table, ids, self.first, vocab)
+        return ops.norm_add(x, self.proj(g), self.norm, coef, n, eps)
+
+
+class CausalAttention(nn.Module):
+    """Softmax attention over all keys up to the query: grouped query heads, optional biases, weighted norms of q and k per head,
+    rotary positions on channel halves (optionally with stretched low frequencies), an optional sink per head; keys and values of
+    its own, or those of another layer (``shared_kv``).  Sections of the layer's fused projections (``joint``)."""
+    joint = True
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rot_base: float, rot_dims: int,
+                 stretch: Optional[Tuple[float, float, float, float]], bias: bool, sink: bool, shared_kv: bool, eps: float, dtype,
+                 device):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"attention: {heads} query heads do not divide over {kv_heads} key/value heads")
+        if rot_dims % 2 or not 0 <= rot_dims <= dim:
+            raise ValueError(f"attention: rotary dims {rot_dims} must be even and at most the head size {dim}")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = heads, kv_heads, dim, vdim, float(scale), eps
+        self.rot, self.shared_kv = (float(rot_base), int(rot_dims), stretch), shared_kv
+        self.in_sections = [("q", heads, dim)] + ([] if shared_kv else [("k", kv_heads, dim), ("v", kv_heads, vdim)])
+        self.out_section = ("o", heads, vdim)
+        self.bias = _param(sum(n * pad8(d) for _, n, d in self.in_sections), dtype=dtype, device=device) if bias else None
+        self.q_norm = _param(pad8(dim), dtype=dtype, device=device)
+        self.k_norm = None if shared_kv else _param(pad8(dim), dtype=dtype, device=device)
+        self.sink = _param(heads, dtype=dtype, device=device) if sink else None
+
+    def kv_shape(self) -> Optional[Tuple[int, int, int]]:
+        return None if self.shared_kv else (self.kv_heads, pad8(self.dim), pad8(self.vdim))
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        return {}
+
+    def tensors(self, prefix: str, inp: Sections, out_slot: Slot) -> Dict[str, Slot]:
+        t, at, rot = {prefix + "o": out_slot}, 0, self.rot[1]
+
+        for n, heads, d in self.in_sections:
+            s = inp.slot(n)
+            t[prefix + n] = s if n == "v" else HalvesSlot(s.view, rot, s.shape)
+            if self.bias is not None:
+                b = self.bias.data[at:at + heads * pad8(d)].view(heads, pad8(d))[:, :d]
+                t[prefix + n + ".b"] = Slot(b, (heads * d,)) if n == "v" else HalvesSlot(b, rot, (heads * d,))
+            at += heads * pad8(d)
+        t[prefix + "q.norm"] = HalvesSlot(self.q_norm.data[None, :self.dim], rot, (self.dim,))
+        if self.k_norm is not None:
+            t[prefix + "k.norm"] = HalvesSlot(self.k_norm.data[None, :self.dim], rot, (self.dim,))
+        if self.sink is not None:
+            t[prefix + "sink"] = Slot(self.sink.data, (self.heads,))
+        return t
+
+    def run(self, h: torch.Tensor, y: Sections, out: torch.Tensor, p, kv: Tuple[torch.Tensor, torch.Tensor], state, rope,
+            out_scale: float = 1.0) -> None:
+        if out_scale != 1.0:
+            raise ValueError("attention: its output takes no factor")
+        k, v = (None, None) if self.shared_kv else (y.cols("k"), y.cols("v"))
+        cos, sin = rope(*self.rot) if self.rot[1] else (None, None)
+        q = ops.qk_norm_store(y.cols("q"), k, v, *kv, p, self.heads, self.dim, True, self.eps, self.q_norm, self.k_norm, self.bias,
+                              cos, sin)
+        ops.paged_attention(q, *kv, out, p, self.heads, self.scale, sink=self.sink)
+
+
+class MatrixMemory(nn.Module):
+    """Linear attention with exponential input and forget gates per head, a running maximum that keeps them in range and a
+    normaliser; a norm per head with weights over all heads, and a sigmoid gate.  The gates' projections stay in 32-bit."""
+    joint = True
+
+    def __init__(self, hidden: int, heads: int, dim: int, vdim: int, cap: float, eps: float, dtype, device):
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.cap, self.eps = heads, dim, vdim, float(cap), eps
+        self.in_sections = [("q", heads, dim), ("k", heads, dim), ("v", heads, vdim), ("g", heads, vdim)]
+        self.out_section = ("o", heads, vdim)
+        self.gates = PackedRows(hidden, [("i", 1, heads), ("f", 1, heads)], dtype, device)
+        self.bias = _param(2, heads, dtype=dtype, device=device)
+        self.norm = _param(heads, pad8(vdim), dtype=dtype, device=device)
+
+    def kv_shape(self) -> None:
+        return None
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        return {"S": (self.heads, pad8(self.dim), pad8(self.vdim)), "n": (self.heads, pad8(self.dim)), "m": (self.heads,)}
+
+    def tensors(self, prefix: str, inp: Sections, out_slot: Slot) -> Dict[str, Slot]:
+        t = {prefix + n: inp.slot(n) for n in "qkvg"} | {prefix + "o": out_slot}
+        for i, n in enumerate("if"):
+            t[prefix + n], t[prefix + n + ".b"] = self.gates.slot(n), Slot(self.bias.data[i], (self.heads,))
+        t[prefix + "norm"] = Slot(self.norm.data[:, :self.vdim], (self.heads * self.vdim,))
+        return t
+
+    def run(self, h: torch.Tensor, y: Sections, out: torch.Tensor, p, kv, state: Dict[str, torch.Tensor], rope,
+            out_scale: float = 1.0) -> None:
+        z, H = self.gates.fp32(h), self.heads
+        ops.matrix_memory(y.cols("q"), y.cols("k"), y.cols("v"), y.cols("g"), self.gates.cols(z, "i")[:, :H], self.gates.cols(z, "f")[:, :H],
+                          self.bias[0], self.bias[1], out, state["S"], state["n"], state["m"], p, self.norm.view(-1), self.dim, self.vdim,
+                          self.cap, self.dim ** -0.5, out_scale, self.eps)
+
+
+class GatedRecurrence(nn.Module):
+    """A gelu branch times a gated linear recurrence with one state per channel, behind a short convolution; the two gates are
+    block-diagonal products of the convolution's output, in 32-bit."""
+    joint = True
+
+    def __init__(self, hidden: int, width: int, blocks: int, taps: int, dtype, device):
+        super().__init__()
+        if blocks < 1 or width % blocks:
+            raise ValueError(f"recurrence: {width} channels do not form {blocks} equal blocks")
+        if not 1 <= taps <= 17:
+            raise ValueError(f"recurrence: {taps} convolution taps (1 to 17)")
+        self.width, self.blocks, self.size, self.taps_n = width, blocks, width // blocks, taps
+        B, n, np_ = blocks, self.size, pad8(self.size)
+        self.in_sections = [("y", B, n), ("x", B, n)]
+        self.out_section = ("o", B, n)
+
+        def vec(*s):
+            return _param(*s, dtype=dtype, device=device)
+        self.y_bias, self.x_bias, self.conv_bias, self.lam = vec(B, np_), vec(B, np_), vec(B, np_), vec(B, np_)
+        self.taps = vec(B, np_, taps)
+        self.w_gates, self.gate_bias = vec(B, 2, np_, np_), vec(B, 2, np_)
+
+    def kv_shape(self) -> None:
+        return None
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        C = self.blocks * pad8(self.size)
+        return {"S": (C,), "conv": (C, self.taps_n - 1)}
+
+    def tensors(self, prefix: str, inp: Sections, out_slot: Slot) -> Dict[str, Slot]:
+        B, n, C = self.blocks, self.size, self.width
+        t = {prefix + "y": inp.slot("y"), prefix + "x": inp.slot("x"), prefix + "o": out_slot,
+             prefix + "conv": Slot(self.taps.data[:, :n], (C, self.taps_n))}
+        for name, v in (("y.b", self.y_bias), ("x.b", self.x_bias), ("conv.b", self.conv_bias), ("lam", self.lam)):
+            t[prefix + name] = Slot(v.data[:, :n], (C,))
+        for i, name in enumerate(("ra", "ri")):
+            t[prefix + name] = Slot(self.w_gates.data[:, i, :n, :n], (B, n, n))
+            t[prefix + name + ".b"] = Slot(self.gate_bias.data[:, i, :n], (B, n))
+        return t
+
+    def run(self, h: torch.Tensor, y: Sections, out: torch.Tensor, p, kv, state: Dict[str, torch.Tensor], rope,
+            out_scale: float = 1.0) -> None:
+        if out_scale != 1.0:
+            raise ValueError("recurrence: its output takes no factor")
+        C, n = out.shape[1], pad8(self.size)
+        u = ops.causal_conv(y.cols("x"), self.x_bias.view(-1), self.taps.view(C, -1), self.conv_bias.view(-1), state["conv"], p)
+        z = ops.block_gates(u, self.w_gates.view(self.blocks, 2 * n, n))
+        ops.linear_recurrence(u, z, self.gate_bias.view(-1), self.lam.view(-1), y.cols("y"), self.y_bias.view(-1), out, state["S"], p, n)

@@ -15,6 +15,7 @@ from .config import PRESETS as DENSE_PRESETS
 from .config import ModelConfig
 from .fetelorn import FETELORN_PRESETS, FetelornConfig, FetelornModel
 from .qwen3 import ParallelTransformerModel
+from .ruburax import RUBURAX_PRESETS, RuburaxConfig, RuburaxModel
 from .sotazen import SOTAZEN_PRESETS, SotazenConfig, SotazenModel
 
 
@@ -87,8 +88,12 @@ ARCHITECTURES: Dict[str, Architecture] = {
     "Sotazen": Architecture("Sotazen", SotazenConfig, lambda path: SotazenConfig.from_dict(_config_json(path)), SotazenModel,
                             _load_slots_at, ("host", "gemm", "residual", "linear_state", "retention_chunk", "attention_rows",
                                              "attention_decode", "attention_latent", "attention_fwd", "sampling"), float32=True),
+    "Ruburax": Architecture("Ruburax", RuburaxConfig, lambda path: RuburaxConfig.from_dict(_config_json(path)), RuburaxModel,
+                            _load_slots_at, ("host", "gemm", "residual", "linear_state", "retention_chunk", "recurrence", "moe",
+                                             "attention_rows", "attention_decode", "attention_latent", "attention_fwd", "sampling"),
+                            float32=True),
 }
-PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS, **SOTAZEN_PRESETS}
+PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS, **SOTAZEN_PRESETS, **RUBURAX_PRESETS}
 
 
 def architecture_at(path: str) -> Architecture:

@@ -59,7 +59,7 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed:
     assert w.is_contiguous() and x.shape[1] == H * K and out.shape[1] == H * N
     nv.check(nv.lib().b2_head_linear(
         nv.ptr(x), nv.ptr(w), nv.ptr(out), nv.ctypes.c_longlong(x.stride(0)), nv.ctypes.c_longlong(out.stride(0)), x.shape[0], H, N, K,
-        K, N, int(transposed), int(x.dtype == torch.float32), nv.stream_ptr()), "head_linear")
+        K, N, int(transposed), int(x.dtype == torch.float32), 0, nv.stream_ptr()), "head_linear")
     nv.count_launch()
 
 

@@ -1,5 +1,6 @@
-"""Linear-attention recurrences over per-sequence state slots: retention (one fixed decay per head) and the gated delta
-rule (one learned decay per head and key channel), with the delta rule's input stage.
+"""Linear-attention recurrences over per-sequence state slots: retention (one fixed decay per head), the gated delta rule
+(one learned decay per head and key channel), with the delta rule's input stage, and matrix memory (exponential input and
+forget gates per head, normalised).
 
 All head sizes are stored padded to a multiple of eight (``dkp``, ``dvp``); ``dk``, ``dv`` are the real ones.  States are
 fp32 ``[slots, H, dkp, dvp]``; a sequence whose portion starts at position 0 starts from zero whatever its slot holds."""
@@ -191,4 +192,55 @@ def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: to
             nv.ptr(state), cu, st, sl, n, longest, H, G, dk, dkp, dv, dvp, nv.ctypes.c_longlong(gate.stride(0)),
             nv.ctypes.c_longlong(out.stride(0)), nv.ctypes.c_float(eps), int(v.dtype == torch.float32), nv.stream_ptr()),
             "delta_serial")
+        nv.count_launch()
+
+
+MEMORY_EPS = 1e-6     # added to the normaliser
+
+
+def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, zi: torch.Tensor, zf: torch.Tensor,
+                  bi: torch.Tensor, bf: torch.Tensor, out: torch.Tensor, S: torch.Tensor, n: torch.Tensor, m: torch.Tensor,
+                  p: Portions, norm_w: torch.Tensor, dk: int, dv: int, cap: float, q_scale: float, out_scale: float,
+                  eps: float) -> None:
+    """Log gates ``i = cap tanh((zi + bi) / cap)``, ``f = logsigmoid(cap tanh((zf + bf) / cap))`` per head; with a running maximum
+    ``m <- max(f + m, i)`` (from 0), ``S <- e^(f + m_old - m) S + e^(i - m) k v^T`` and ``n`` likewise with k alone,
+    ``o = S^T q / (max(|n . q|, e^-m) + 1e-6)`` for ``q_scale q``; then ``out = rms(o) norm_w sigmoid(gate) out_scale``, the norm
+    per head.  ``q, k [M, H*dkp]``, ``v, gate, out [M, H*dvp]`` are column slices (the first four of one matrix), ``zi, zf
+    [M, H]`` fp32 column slices of one matrix, ``norm_w [H*dvp]``; ``S [slots, H, dkp, dvp]``, ``n [slots, H, dkp]``,
+    ``m [slots, H]``."""
+    H, dkp, dvp = S.shape[1:]
+    if not q.is_cuda:
+        M = q.shape[0]
+        i = cap * torch.tanh((zi + bi.float()) / cap)
+        f = torch.nn.functional.logsigmoid(cap * torch.tanh((zf + bf.float()) / cap))
+        qf, kf = q.reshape(M, H, dkp).float() * q_scale, k.reshape(M, H, dkp).float()
+        vf, gf = v.reshape(M, H, dvp).float(), gate.reshape(M, H, dvp).float()
+        o = torch.zeros(M, H, dvp)
+        for a, b, start, slot in _cpu_sequences(p):
+            fresh = start == 0
+            Ss, ns, ms = (torch.zeros_like(t[slot]) if fresh else t[slot].clone() for t in (S, n, m))
+            for t in range(a, b):
+                mt = torch.maximum(f[t] + ms, i[t])
+                w, u = torch.exp(f[t] + ms - mt), torch.exp(i[t] - mt)
+                Ss = w[:, None, None] * Ss + u[:, None, None] * kf[t, :, :, None] * vf[t, :, None, :]
+                ns = w[:, None] * ns + u[:, None] * kf[t]
+                ms = mt
+                den = torch.maximum((ns * qf[t]).sum(-1).abs(), torch.exp(-ms)) + MEMORY_EPS
+                o[t] = (Ss * qf[t, :, :, None]).sum(1) / den[:, None]
+            S[slot], n[slot], m[slot] = Ss, ns, ms
+        o = _head_rms(o, dv, eps) * norm_w.float().reshape(H, dvp) * torch.sigmoid(gf) * out_scale
+        out.copy_(o.reshape(M, H * dvp).to(out.dtype))
+        return
+    assert q.stride(0) == k.stride(0) == v.stride(0) == gate.stride(0) and zi.stride(0) == zf.stride(0)
+    assert zi.dtype == zf.dtype == torch.float32
+    cf, cl = nv.ctypes.c_float, nv.ctypes.c_longlong
+    for lo, cnt, longest in ((0, p.num_short, p.max_short), (p.num_short, p.nseq - p.num_short, p.max_long)):
+        if cnt <= 0:
+            continue
+        cu, st, sl = _sub(p, lo)
+        nv.check(nv.lib().b2_memory_serial(
+            nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(zi), nv.ptr(zf), cl(zi.stride(0)), nv.ptr(bi), nv.ptr(bf),
+            nv.ptr(norm_w), nv.ptr(out), nv.ptr(S), nv.ptr(n), nv.ptr(m), cu, st, sl, cnt, longest, H, dk, dkp, dv, dvp,
+            cl(q.stride(0)), cl(out.stride(0)), cf(cap), cf(q_scale), cf(out_scale), cf(eps), int(q.dtype == torch.float32),
+            nv.stream_ptr()), "memory_serial")
         nv.count_launch()

@@ -31,22 +31,28 @@ def distance_buckets(rows: int, far: float, length: int, device=None) -> torch.T
     return torch.tensor(out, dtype=torch.int32, device=device)
 
 
-def qk_norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+def qk_norm_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], k_cache: torch.Tensor, v_cache: torch.Tensor,
                   p: Portions, H: int, dk: int, norm: bool, eps: float, wq: Optional[torch.Tensor] = None,
                   wk: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None,
                   sin: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``bias`` (one vector over the columns of q, k and v) added, per-head RMS norm of q and k (``norm``; optional weights
     ``[dkp]``), rotary positions of q and k on channel pairs (2 i, 2 i + 1) (``cos, sin [M, dims/2]``), k and v stored into their
     sequences' pages.  ``q, k, v`` are column slices of one matrix; returns the new q ``[M, H*dkp]``.  K and V pages may have
-    different head counts (two key rows over one value row)."""
+    different head counts (two key rows over one value row).  ``k`` and ``v`` None: queries alone, over pages another layer fills."""
     nblk, bs, G, dkp = k_cache.shape
     Gv, dvp, M = v_cache.shape[2], v_cache.shape[3], q.shape[0]
+    if k is None:
+        G = Gv = 0
     bq = bk = bv = None
     if bias is not None:
         bq, bk, bv = bias[:H * dkp], bias[H * dkp:(H + G) * dkp], bias[(H + G) * dkp:]
+        if k is None:
+            bk = bv = bq
     if not q.is_cuda:
         if bias is not None:
-            q, k, v = q.float() + bq.float(), k.float() + bk.float(), v.float() + bv.float()
+            q = q.float() + bq.float()
+            if k is not None:
+                k, v = k.float() + bk.float(), v.float() + bv.float()
 
         def n(x, w):
             x = x.float()
@@ -59,6 +65,9 @@ def qk_norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: to
                 u, z, c, s = x[..., 0:rot:2], x[..., 1:rot:2], cos[:, None, :], sin[:, None, :]
                 x = torch.cat([torch.stack([u * c - z * s, z * c + u * s], -1).flatten(-2), x[..., rot:]], -1)
             return x
+        qf = n(q.reshape(M, H, dkp), wq).reshape(M, H * dkp).to(k_cache.dtype)
+        if k is None:
+            return qf
         kf = n(k.reshape(M, G, dkp), wk).to(k_cache.dtype)
         vf = v.reshape(M, Gv, dvp).to(v_cache.dtype)
         for r, (s, pos) in enumerate(zip(p.row_seq.tolist(), p.positions.tolist())):
@@ -66,8 +75,8 @@ def qk_norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: to
                 continue
             blk = int(p.block_tables[s, pos // bs])
             k_cache[blk, pos % bs], v_cache[blk, pos % bs] = kf[r], vf[r]
-        return n(q.reshape(M, H, dkp), wq).reshape(M, H * dkp).to(k_cache.dtype)
-    assert bs == 16 and q.stride(0) == k.stride(0) == v.stride(0)
+        return qf
+    assert bs == 16 and (k is None or q.stride(0) == k.stride(0) == v.stride(0))
     out = torch.empty((M, H * dkp), device=q.device, dtype=q.dtype)
     nv.check(nv.lib().b2_qk_norm_store(
         nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ctypes.c_longlong(q.stride(0)), nv.ptr(out), nv.ptr(k_cache), nv.ptr(v_cache),
@@ -171,8 +180,9 @@ def _attention(q, k_cache, v_cache, out, p, H, scale, chunk, rel, bucket, sink, 
         nv.count_launch()
     if lead == 0:
         return
-    if q.dtype == torch.bfloat16 and lam is not None and decode_attention(
-            q, k_cache, v_cache, out, p, lead, H, G, maps * dkp, dvp, scale, None, gate, window, softcap, lam, lam_init, eps, dv):
+    plain = lam is None and gate is None and rel is None and chunk == 0
+    if q.dtype == torch.bfloat16 and (plain or lam is not None) and decode_attention(
+            q, k_cache, v_cache, out, p, lead, H, G, maps * dkp, dvp, scale, sink, gate, window, softcap, lam, lam_init, eps, dv):
         return
     assert q.is_contiguous()
     keys = min(p.max_keys, chunk or window or p.max_keys)

@@ -41,6 +41,7 @@ class Portions:
     ctx_pages: Optional[torch.Tensor] = None
     ctx_tables: Optional[torch.Tensor] = None
     ctx_counts: Optional[List[int]] = None
+    ids: Optional[torch.Tensor] = None       # int64 [M] token of every row, for layers that look tokens up
     plans: Dict[Tuple[int, int, int], torch.Tensor] = field(default_factory=dict)    # decode_plan: (rows, window, tile) -> tile counts
     ragged: bool = True                      # False: every sequence is one row (decode): row r is sequence r
 

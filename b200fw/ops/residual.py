@@ -1,5 +1,5 @@
-"""Ops around a 32-bit residual stream: embedding into it, RMS norm out of it, the weighted sum of two normed branches
-added to it, gated activation over column slices, rotary tables for a batch's positions.
+"""Ops around a 32-bit residual stream: embedding into it, RMS norm out of it, normed branches added to it, gated activations
+over column slices or with a table of per-token vectors, rotary tables for a batch's positions.
 
 Activations and residual rows are padded to a multiple of eight columns (:func:`pad8`); the padding is zero."""
 from __future__ import annotations
@@ -31,17 +31,18 @@ def embedding_f32(ids: torch.Tensor, table: torch.Tensor, vocab: Optional[int] =
     return (x, x if low is None else low) if h else x
 
 
-def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, n: int, eps: float, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``x[rows] / sqrt(mean(x^2) + eps) * w`` in ``w``'s dtype; ``n`` real columns, ``w`` zero past them.  ``rows``
+def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, n: int, eps: float, rows: Optional[torch.Tensor] = None,
+                scale: float = 1.0) -> torch.Tensor:
+    """``x[rows] / sqrt(mean(x^2) + eps) * w * scale`` in ``w``'s dtype; ``n`` real columns, ``w`` zero past them.  ``rows``
     (int64) selects and orders the rows of ``x``."""
     if not x.is_cuda:
         xs = x if rows is None else x[rows]
-        r = torch.rsqrt((xs[:, :n] * xs[:, :n]).mean(-1, keepdim=True) + eps)
+        r = scale * torch.rsqrt((xs[:, :n] * xs[:, :n]).mean(-1, keepdim=True) + eps)
         return (xs * r * w.float()).to(w.dtype)
     M = x.shape[0] if rows is None else rows.numel()
     h = torch.empty((M, x.shape[1]), device=x.device, dtype=w.dtype)
     nv.check(nv.lib().b2_rmsnorm_f32(nv.ptr(x), nv.ptr(w), nv.ptr(h), nv.ptr(rows), M, x.shape[1], n,
-                                     nv.ctypes.c_float(eps), _f32(w), nv.stream_ptr()), "rmsnorm_f32")
+                                     nv.ctypes.c_float(eps), nv.ctypes.c_float(scale), _f32(w), nv.stream_ptr()), "rmsnorm_f32")
     nv.count_launch()
     return h
 
@@ -84,6 +85,37 @@ def post_norm(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, alpha: float, n
     return x if h is None else h
 
 
+def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, coef: float, n: int, eps: float, y_scale: float = 1.0) -> torch.Tensor:
+    """In place ``x += coef * rms(y_scale * y) * w`` (``x``, ``y`` fp32); returns the new ``x`` in ``w``'s dtype (``x`` itself in
+    32-bit)."""
+    if not x.is_cuda:
+        t = y_scale * y
+        x += coef * t * torch.rsqrt((t[:, :n] * t[:, :n]).mean(-1, keepdim=True) + eps) * w.float()
+        return x if w.dtype == torch.float32 else x.to(w.dtype)
+    h = None if w.dtype == torch.float32 else torch.empty(x.shape, device=x.device, dtype=w.dtype)
+    nv.check(nv.lib().b2_norm_add(nv.ptr(x), nv.ptr(y), nv.ptr(w), nv.ptr(h), x.shape[0], x.shape[1], n, nv.ctypes.c_float(coef),
+                                  nv.ctypes.c_float(eps), nv.ctypes.c_float(y_scale), _f32(w), nv.stream_ptr()), "norm_add")
+    nv.count_launch()
+    return x if h is None else h
+
+
+def gelu_tanh(z: torch.Tensor) -> torch.Tensor:
+    return torch.nn.functional.gelu(z, approximate="tanh")
+
+
+def gelu_times_token(gate: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, first: int, vocab: int) -> torch.Tensor:
+    """``gelu_tanh(gate) * table[ids, first : first + n]`` with ``gate [M, n]``; ids outside ``[0, vocab)`` give zeros on a GPU."""
+    M, n = gate.shape
+    if not gate.is_cuda:
+        return (gelu_tanh(gate.float()) * table[ids, first:first + n].float()).to(gate.dtype)
+    out = torch.empty((M, n), device=gate.device, dtype=gate.dtype)
+    assert gate.stride(1) == 1 and table.stride(1) == 1
+    nv.check(nv.lib().b2_gelu_token(nv.ptr(gate), nv.ptr(table), nv.ptr(ids), nv.ptr(out), M, n, gate.stride(0),
+                                    nv.ctypes.c_longlong(table.stride(0)), first, vocab, _f32(gate), nv.stream_ptr()), "gelu_token")
+    nv.count_launch()
+    return out
+
+
 def glu(gate: torch.Tensor, up: torch.Tensor, out: torch.Tensor) -> None:
     """``out = silu(gate) * up``; the three are column slices (``gate`` and ``up`` of one matrix)."""
     if not gate.is_cuda:
@@ -96,10 +128,25 @@ def glu(gate: torch.Tensor, up: torch.Tensor, out: torch.Tensor) -> None:
     nv.count_launch()
 
 
-def rope_turns(base: float, dims: int, device) -> torch.Tensor:
-    """``base^(-2 i / dims) / (2 pi)`` for i < dims / 2, in double precision."""
-    return torch.tensor([base ** (-2.0 * i / dims) / (2.0 * math.pi) for i in range(dims // 2)], dtype=torch.float64,
-                        device=device)
+def rope_turns(base: float, dims: int, device, stretch: Optional[Tuple[float, float, float, float]] = None) -> torch.Tensor:
+    """Turns per position ``base^(-2 i / dims) / (2 pi)`` for i < dims / 2, in double precision.
+
+    ``stretch = (factor, low, high, original)`` slows the low frequencies for contexts longer than ``original``: a pair that turns
+    fewer than ``low`` times over ``original`` positions is slowed by ``factor``, one that turns more than ``high`` times is kept,
+    and between the two the frequency is blended linearly."""
+    out = []
+    for i in range(dims // 2):
+        f = base ** (-2.0 * i / dims) / (2.0 * math.pi)
+        if stretch is not None:
+            factor, low, high, original = stretch
+            turns = original * f
+            if turns < low:
+                f /= factor
+            elif turns <= high:
+                s = (turns - low) / (high - low)
+                f = (1.0 - s) * f / factor + s * f
+        out.append(f)
+    return torch.tensor(out, dtype=torch.float64, device=device)
 
 
 def rope_rows(positions: torch.Tensor, turns: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
