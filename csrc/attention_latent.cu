@@ -142,7 +142,8 @@ __global__ void __launch_bounds__(256) head_linear_any_kernel(const HeadLinearPa
 
 // bf16: a 64 x 64 output tile of one head per CTA, four warps of 16 rows, K in pieces of 64 through two stages.
 constexpr int HL_T = 64, HL_LD = HL_T + 8;
-template <bool KN>
+// O: type of the result
+template <bool KN, typename O>
 __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearParams p) {
   __shared__ __align__(16) la_bf16 sA[2][HL_T][HL_LD], sB[2][HL_T][HL_LD];
   const int n0 = blockIdx.x * HL_T, h = blockIdx.y, m0 = blockIdx.z * HL_T;
@@ -185,14 +186,15 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearParams
     }
     __syncthreads();
   }
-  la_bf16* out = static_cast<la_bf16*>(p.out) + static_cast<size_t>(h) * p.os;
+  O* out = static_cast<O*>(p.out) + static_cast<size_t>(h) * p.os;
 #pragma unroll
   for (int n = 0; n < HL_T / 8; ++n)
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
       const int m = m0 + warp * 16 + (lane >> 2) + 8 * hh, c = n0 + n * 8 + (lane & 3) * 2;
-      if (m < p.M && c < p.N)
-        *reinterpret_cast<uint32_t*>(out + m * p.ld_out + c) = pack_bf16x2(acc[n][2 * hh], acc[n][2 * hh + 1]);
+      if (m >= p.M || c >= p.N) continue;
+      if (sizeof(O) == 4) *reinterpret_cast<float2*>(out + m * p.ld_out + c) = make_float2(acc[n][2 * hh], acc[n][2 * hh + 1]);
+      else *reinterpret_cast<uint32_t*>(out + m * p.ld_out + c) = pack_bf16x2(acc[n][2 * hh], acc[n][2 * hh + 1]);
     }
 }
 
@@ -343,8 +345,9 @@ B2_EXPORT int b2_latent_gather(const void* pages, const int* ids, void* out, int
   return 0;
 }
 
+// out_f32: a 32-bit result of bf16 operands
 B2_EXPORT int b2_head_linear(const void* x, const void* w, void* out, long long ld_x, long long ld_out, int M, int H, int N, int K,
-                             int xs, int os, int kn, int is_f32, void* stream) {
+                             int xs, int os, int kn, int is_f32, int out_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (H < 1 || H > 65535 || N < 8 || K < 8 || N % 8 || K % 8 || xs % 8 || os % 8 || ld_x % 8 || ld_out % 8) {
@@ -360,8 +363,13 @@ B2_EXPORT int b2_head_linear(const void* x, const void* w, void* out, long long 
   } else {
     const dim3 grid((N + HL_T - 1) / HL_T, H, (M + HL_T - 1) / HL_T);
     if (grid.z > 65535) { set_error("head_linear: too many rows (%d)", M); return 10; }
-    if (kn) head_linear_kernel<true><<<grid, 128, 0, st>>>(p);
-    else head_linear_kernel<false><<<grid, 128, 0, st>>>(p);
+    if (out_f32) {
+      if (kn) head_linear_kernel<true, float><<<grid, 128, 0, st>>>(p);
+      else head_linear_kernel<false, float><<<grid, 128, 0, st>>>(p);
+    } else {
+      if (kn) head_linear_kernel<true, la_bf16><<<grid, 128, 0, st>>>(p);
+      else head_linear_kernel<false, la_bf16><<<grid, 128, 0, st>>>(p);
+    }
   }
   B2_CHECK_LAUNCH("head_linear");
   return 0;

@@ -592,6 +592,7 @@ B2_EXPORT int b2_attn_rows(const void* q, const void* kc, const void* vc, const 
   });
 }
 
+// G = Gv = 0: queries alone
 B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long long ld, void* q_out, void* kc, void* vc,
                                const int* tables, const int* row_seq, const int* pos, const int* slot, int M,
                                int max_blocks, int H, int G, int Gv, int dk, int dkp, int dvp, const void* wq, const void* wk,
@@ -599,7 +600,7 @@ B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long
                                const float* sn, int rot, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
-  if (dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || ld % 8 || dk < 1 || dk > dkp || max_blocks < 1 || H < 1 || G < 1 || Gv < 1 ||
+  if (dkp % 8 || dvp % 8 || dkp > 256 || dvp > 256 || ld % 8 || dk < 1 || dk > dkp || max_blocks < 1 || H < 1 || G < 0 || Gv < 0 ||
       (cs != nullptr && (rot < 2 || rot % 2 || rot > dk))) {
     set_error("qk_norm_store: head sizes up to 256 in multiples of 8 (padded) required");
     return 10;

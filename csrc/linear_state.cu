@@ -3,10 +3,13 @@
 //
 //   retention   S <- a_h S + k v^T                                     o = S^T q     (one fixed decay per head)
 //   delta rule  S <- g . S;  u = beta (v - S^T k);  S <- S + k u^T     o = S^T q     (one decay per head and key channel)
+//   memory      m <- max(f + m', i);  S <- e^{f + m' - m} S + e^{i - m} k v^T;  n likewise with k alone
+//               o = S^T q / (max(|n . q|, e^{-m}) + 1e-6)              (log gates i, f per head and token; m from 0)
 //
 // followed by a per-head RMS norm over the value channels and an output gate; or, for retention whose heads are normed together,
 // by the norm's weight and a sigmoid gate, with the sum of squares of every head left for the reader of the output projection
-// (the norm is one factor per row, which commutes with that projection).  This file has the token-by-token form,
+// (the norm is one factor per row, which commutes with that projection); memory has a norm per head with a weight for every channel
+// of every head, and a sigmoid gate.  This file has the token-by-token form,
 // which is the decode step, the form for short portions, and the one that runs in true 32-bit; it also has the delta
 // rule's input stage (short causal convolution, activation, unit norms, decays, step sizes).
 //
@@ -36,7 +39,7 @@ struct SerialParams {
   const float* cs;    // rotary tables [M, rot / 2] (retention)
   const float* sn;
   const float* decay;       // retention: [H]
-  const void* norm_w;       // T [dvp] or null; retention with joint_ss: T [H * dvp]
+  const void* norm_w;       // T [dvp] or null; retention with joint_ss and memory: T [H * dvp]
   float* joint_ss;          // retention: [M, H], or null for a norm per head
   void* out;                // T, row stride ld_out
   float* state;             // [slots, H, dkp, dvp]
@@ -45,15 +48,33 @@ struct SerialParams {
   int dk, dkp, dv, dvp, rot;
   float kscale, eps;
   int tile;                 // tokens staged at a time
+  // memory: gates before bias and cap, fp32 [M, ld_z]; their biases T [H]; normaliser [slots, H, dkp] and running maximum [slots, H]
+  const float* zi;
+  const float* zf;
+  const void* bi;
+  const void* bf;
+  float* n;
+  float* m;
+  long long ld_z;
+  float cap, qscale, oscale;
 };
+enum : int { RETENTION = 0, DELTA_RULE = 1, MEMORY = 2 };
+constexpr float MEMORY_EPS = 1e-6f;
+
+// log input and log forget gate of memory
+__device__ __forceinline__ float2 memory_gates(float zi, float zf, float cap) {
+  const float x = cap * tanhf(zf / cap);
+  return make_float2(cap * tanhf(zi / cap), fminf(x, 0.f) - log1pf(expf(-fabsf(x))));
+}
 
 // One CTA per (head, sequence).  A warp owns eight value columns; its lanes form four groups that split the key rows in
 // quads (lane group r holds rows 16 j + 4 r .. + 3), so the state of a head lives in registers, 4 JJ values a thread, and
 // the two reductions of a token are two shuffles.  q, k and the decays of a tile of tokens are staged in shared memory as
 // fp32 (rotated / exponentiated there once); the outputs of the tile are collected in shared memory, normed, gated, stored.
-template <typename T, int JJ, bool DELTA, int MAXT>
+template <typename T, int JJ, int KIND, int MAXT>
 __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p) {
   constexpr int DK = 16 * JJ;
+  constexpr bool DELTA = KIND == DELTA_RULE, MEM = KIND == MEMORY;
   extern __shared__ __align__(16) float sm[];
   const int h = blockIdx.x, s = blockIdx.y;
   const int slot = p.seq.slot[s];
@@ -65,6 +86,7 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
   float* sg = sq + TT * DK;                       // delta only
   float* sv = sg + (DELTA ? TT * DK : 0);
   float* so = sv + TT * p.dvp;
+  float* sx = so + TT * p.dvp;                    // memory: [4][TT] old weight, new weight, e^{-m}, n . q
   const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31;
   const int rg = lane >> 3, col = warp * 8 + (lane & 7);
   const int kvh = h / p.group;
@@ -79,7 +101,16 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
       const int i = 16 * j + 4 * rg + e;
       S[4 * j + e] = (!fresh && i < p.dkp) ? st[static_cast<size_t>(i) * p.dvp + col] : 0.f;
     }
-  const float a = DELTA ? 0.f : p.decay[h];
+  const float a = KIND == RETENTION ? p.decay[h] : 0.f;
+  // memory: warp 0 keeps the normaliser (channel lane + 32 j) and the maximum
+  constexpr int NJ = (DK + 31) / 32;
+  const size_t head = static_cast<size_t>(slot < 0 ? 0 : slot) * p.H + h;
+  float nrm[NJ], mx = 0.f;
+  if (MEM && warp == 0) {
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) nrm[j] = !fresh && lane + 32 * j < p.dkp ? p.n[head * p.dkp + lane + 32 * j] : 0.f;
+    if (!fresh) mx = p.m[head];
+  }
 
   for (int t0 = 0; t0 < count; t0 += TT) {
     const int nt = min(TT, count - t0);
@@ -115,9 +146,32 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
             kv = kv * cs + to_f(k[at + o]) * sgn;
           }
           kv *= p.kscale;
+          if (MEM) qv *= p.qscale;
         }
         sq[i] = qv;
         sk[i] = kv;
+      }
+    }
+    if (MEM && warp == 0) {
+      float2 g = make_float2(0.f, 0.f);
+      if (lane < nt) {
+        const size_t row = row0 + t0 + lane;
+        g = memory_gates(p.zi[row * p.ld_z + h] + to_f(static_cast<const T*>(p.bi)[h]),
+                         p.zf[row * p.ld_z + h] + to_f(static_cast<const T*>(p.bf)[h]), p.cap);
+      }
+      float old = 0.f, now = 0.f;                  // the maximum before and after this lane's token
+      for (int t = 0; t < nt; ++t) {
+        const float gi = __shfl_sync(0xffffffffu, g.x, t), gf = __shfl_sync(0xffffffffu, g.y, t), next = fmaxf(gf + mx, gi);
+        if (lane == t) {
+          old = mx;
+          now = next;
+        }
+        mx = next;
+      }
+      if (lane < nt) {
+        sx[lane] = expf(g.y + old - now);
+        sx[TT + lane] = expf(g.x - now);
+        sx[2 * TT + lane] = expf(-now);
       }
     }
     for (int i = tid; i < nt * p.dvp; i += nthr) {
@@ -148,6 +202,8 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
         u = p.beta[static_cast<size_t>(row0 + t0 + t) * p.H + h] * (u - d);
       }
       float o0 = 0.f, o1 = 0.f;
+      const float w = MEM ? sx[t] : a;
+      if (MEM) u *= sx[TT + t];
 #pragma unroll
       for (int j = 0; j < JJ; ++j) {
         const float4 k = *reinterpret_cast<const float4*>(kt + 16 * j);
@@ -158,10 +214,10 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
           S[4 * j + 2] = fmaf(k.z, u, S[4 * j + 2]);
           S[4 * j + 3] = fmaf(k.w, u, S[4 * j + 3]);
         } else {
-          S[4 * j] = fmaf(a, S[4 * j], k.x * u);
-          S[4 * j + 1] = fmaf(a, S[4 * j + 1], k.y * u);
-          S[4 * j + 2] = fmaf(a, S[4 * j + 2], k.z * u);
-          S[4 * j + 3] = fmaf(a, S[4 * j + 3], k.w * u);
+          S[4 * j] = fmaf(w, S[4 * j], k.x * u);
+          S[4 * j + 1] = fmaf(w, S[4 * j + 1], k.y * u);
+          S[4 * j + 2] = fmaf(w, S[4 * j + 2], k.z * u);
+          S[4 * j + 3] = fmaf(w, S[4 * j + 3], k.w * u);
         }
         o0 = fmaf(S[4 * j], q.x, o0);
         o1 = fmaf(S[4 * j + 1], q.y, o1);
@@ -173,14 +229,31 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
       o += __shfl_xor_sync(0xffffffffu, o, 16);
       if (rg == 0) so[t * p.dvp + col] = o;
     }
+    if (MEM && warp == 0) {
+      for (int t = 0; t < nt; ++t) {
+        const float w = sx[t], u = sx[TT + t];
+        float d = 0.f;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const int c = lane + 32 * j;
+          if (c < DK) {
+            nrm[j] = fmaf(w, nrm[j], u * sk[t * DK + c]);
+            d = fmaf(nrm[j], sq[t * DK + c], d);
+          }
+        }
+        d = warp_sum(d);
+        if (lane == 0) sx[3 * TT + t] = d;
+      }
+    }
     __syncthreads();
     for (int t = warp; t < nt; t += nthr >> 5) {
       float ss = 0.f;
       for (int c = lane; c < p.dvp; c += 32) ss = fmaf(so[t * p.dvp + c], so[t * p.dvp + c], ss);
       ss = warp_sum(ss);
       const size_t row = row0 + t0 + t;
-      float r = 1.f / sqrtf(ss / p.dv + p.eps);
-      if (!DELTA && p.joint_ss) {
+      const float inv = MEM ? 1.f / (fmaxf(fabsf(sx[3 * TT + t]), sx[2 * TT + t]) + MEMORY_EPS) : 1.f;
+      float r = inv / sqrtf(ss * inv * inv / p.dv + p.eps);
+      if (KIND == RETENTION && p.joint_ss) {
         r = 1.f;
         if (lane == 0) p.joint_ss[row * p.H + h] = ss;
       }
@@ -190,6 +263,8 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
         if (DELTA) {
           if (p.norm_w) o *= to_f(static_cast<const T*>(p.norm_w)[c]);
           o *= sigmoid_t<T>(static_cast<const float*>(p.gate)[gi]);
+        } else if (MEM) {
+          o *= p.oscale * to_f(static_cast<const T*>(p.norm_w)[h * p.dvp + c]) * sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
         } else if (p.joint_ss) {
           o *= to_f(static_cast<const T*>(p.norm_w)[h * p.dvp + c]) * sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
         } else {
@@ -207,6 +282,12 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
       const int i = 16 * j + 4 * rg + e;
       if (i < p.dkp) st[static_cast<size_t>(i) * p.dvp + col] = S[4 * j + e];
     }
+  if (MEM && warp == 0) {
+#pragma unroll
+    for (int j = 0; j < NJ; ++j)
+      if (lane + 32 * j < p.dkp) p.n[head * p.dkp + lane + 32 * j] = nrm[j];
+    if (lane == 0) p.m[head] = mx;
+  }
 }
 
 // One token per sequence (the decode step), one CTA per (head, sequence).  Eight row groups of dvp / 4 threads: a thread holds
@@ -214,8 +295,9 @@ __global__ void __launch_bounds__(MAXT) state_serial_kernel(const SerialParams p
 // rows are requested before the first is used.
 constexpr int STEP_GROUPS = 8;
 
-template <typename T, int J, bool DELTA, int MAXT>
+template <typename T, int J, int KIND, int MAXT>
 __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_step_kernel(const SerialParams p) {
+  constexpr bool DELTA = KIND == DELTA_RULE, MEM = KIND == MEMORY;
   extern __shared__ __align__(16) float sm[];
   const int h = blockIdx.x, s = blockIdx.y;
   const int slot = p.seq.slot[s];
@@ -226,7 +308,7 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
   float* sq = sk + DK;
   float* sg = sq + DK;
   float* red = sg + DK;                       // [STEP_GROUPS][DV]
-  float* so = red + STEP_GROUPS * DV;         // [DV], then one word per warp
+  float* so = red + STEP_GROUPS * DV;         // [DV], then one word per warp; memory: another per warp
   const int rg = tid / quads, col = tid % quads * 4, kvh = h / p.group;
   float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * DK * DV + col;
   const bool fresh = p.seq.start[s] == 0;
@@ -235,6 +317,18 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
   for (int j = 0; j < J; ++j) {
     const int i = rg + STEP_GROUPS * j;
     S[j] = !fresh && i < DK ? *reinterpret_cast<const float4*>(st + static_cast<size_t>(i) * DV) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // memory: every thread works out the head's gates; the normaliser's channels are dealt out like the stores of k
+  float w_old = 0.f, w_new = 0.f, e_neg = 0.f, mx = 0.f, nq = 0.f;
+  const size_t head = static_cast<size_t>(slot) * p.H + h;
+  if (MEM) {
+    const float2 g = memory_gates(p.zi[row * p.ld_z + h] + to_f(static_cast<const T*>(p.bi)[h]),
+                                  p.zf[row * p.ld_z + h] + to_f(static_cast<const T*>(p.bf)[h]), p.cap);
+    const float m0 = fresh ? 0.f : p.m[head];
+    mx = fmaxf(g.y + m0, g.x);
+    w_old = expf(g.y + m0 - mx);
+    w_new = expf(g.x - mx);
+    e_neg = expf(-mx);
   }
   for (int c = tid; c < DK; c += nthr) {
     const size_t at = row * p.ld_qk + static_cast<size_t>(kvh) * DK;
@@ -252,8 +346,14 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
         qv = qv * cs + to_f(q[o]) * sn;
         kv = kv * cs + to_f(k[o]) * sn;
       }
-      sq[c] = qv;
+      sq[c] = MEM ? qv * p.qscale : qv;
       sk[c] = kv * p.kscale;
+      if (MEM) {
+        float* np = p.n + head * DK + c;
+        const float nv = fmaf(w_old, fresh ? 0.f : *np, w_new * sk[c]);
+        *np = nv;
+        nq = fmaf(nv, sq[c], nq);
+      }
     }
   }
   float4 u;
@@ -287,7 +387,10 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
     u = make_float4(b * (u.x - t.x), b * (u.y - t.y), b * (u.z - t.z), b * (u.w - t.w));
     __syncthreads();
   }
-  const float a = DELTA ? 1.f : p.decay[h];
+  if (MEM) {
+    u.x *= w_new; u.y *= w_new; u.z *= w_new; u.w *= w_new;
+  }
+  const float a = DELTA ? 1.f : MEM ? w_old : p.decay[h];
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
   for (int j = 0; j < J; ++j) {
@@ -310,12 +413,23 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
     ss = fmaf(x, x, ss);
   }
   ss = warp_sum(ss);
+  const int warps = (nthr + 31) / 32;
   if ((tid & 31) == 0) so[DV + (tid >> 5)] = ss;
+  if (MEM) {
+    nq = warp_sum(nq);
+    if ((tid & 31) == 0) so[DV + warps + (tid >> 5)] = nq;
+  }
   __syncthreads();
-  float tot = 0.f;
-  for (int w = 0; w < nthr / 32; ++w) tot += so[DV + w];
-  float r = 1.f / sqrtf(tot / p.dv + p.eps);
-  if (!DELTA && p.joint_ss) {
+  float tot = 0.f, inv = 1.f;
+  for (int w = 0; w < warps; ++w) tot += so[DV + w];
+  if (MEM) {
+    float d = 0.f;
+    for (int w = 0; w < warps; ++w) d += so[DV + warps + w];
+    inv = 1.f / (fmaxf(fabsf(d), e_neg) + MEMORY_EPS);
+    if (tid == 0) p.m[head] = mx;              // everyone has read the old one
+  }
+  float r = inv / sqrtf(tot * inv * inv / p.dv + p.eps);
+  if (KIND == RETENTION && p.joint_ss) {
     r = 1.f;
     if (tid == 0) p.joint_ss[row * p.H + h] = tot;
   }
@@ -325,6 +439,8 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && J <= 16 ? 2 : 1) state_st
     if (DELTA) {
       if (p.norm_w) x *= to_f(static_cast<const T*>(p.norm_w)[c]);
       x *= sigmoid_t<T>(static_cast<const float*>(p.gate)[gi]);
+    } else if (MEM) {
+      x *= p.oscale * to_f(static_cast<const T*>(p.norm_w)[h * DV + c]) * sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
     } else if (p.joint_ss) {
       x *= to_f(static_cast<const T*>(p.norm_w)[h * DV + c]) * sigmoid_t<T>(to_f(static_cast<const T*>(p.gate)[gi]));
     } else {
@@ -593,14 +709,14 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_vec_kernel(const Delt
   }
 }
 
-template <typename T, bool DELTA>
+template <typename T, int KIND>
 static int launch_step(const SerialParams& p, int nseq, cudaStream_t stream) {
   const int threads = STEP_GROUPS * (p.dvp / 4);    // a multiple of 16; 32 for head sizes in steps of 16
-  const size_t smem = sizeof(float) * (3 * p.dkp + (STEP_GROUPS + 1) * p.dvp + 32);
+  const size_t smem = sizeof(float) * (3 * p.dkp + (STEP_GROUPS + 1) * p.dvp + 64);
   const dim3 grid(p.H, nseq);
 #define B2_STEP(JV)                                                                                          \
   do {                                                                                                       \
-    auto kern = threads <= 256 ? state_step_kernel<T, JV, DELTA, 256> : state_step_kernel<T, JV, DELTA, 512>; \
+    auto kern = threads <= 256 ? state_step_kernel<T, JV, KIND, 256> : state_step_kernel<T, JV, KIND, 512>; \
     kern<<<grid, threads, smem, stream>>>(p);                                                                \
   } while (0)
   if (p.dkp <= 32) B2_STEP(4);
@@ -612,16 +728,16 @@ static int launch_step(const SerialParams& p, int nseq, cudaStream_t stream) {
   return 0;
 }
 
-template <typename T, bool DELTA>
+template <typename T, int KIND>
 static int launch_serial(const SerialParams& p, int nseq, cudaStream_t stream) {
-  if (p.tile == 1 && p.dvp % 16 == 0) return launch_step<T, DELTA>(p, nseq, stream);
+  if (p.tile == 1 && p.dvp % 16 == 0) return launch_step<T, KIND>(p, nseq, stream);
   const int JJ = p.dkp <= 16 ? 1 : p.dkp <= 32 ? 2 : p.dkp <= 64 ? 4 : p.dkp <= 128 ? 8 : 16;
   const int DK = 16 * JJ;
-  const size_t smem = sizeof(float) * p.tile * ((DELTA ? 3 : 2) * DK + 2 * p.dvp);
+  const size_t smem = sizeof(float) * p.tile * ((KIND == DELTA_RULE ? 3 : 2) * DK + 2 * p.dvp + (KIND == MEMORY ? 4 : 0));
   const dim3 grid(p.H, nseq);
 #define B2_SERIAL(J)                                                                                            \
   do {                                                                                                          \
-    auto kern = p.dvp <= 128 ? state_serial_kernel<T, J, DELTA, 512> : state_serial_kernel<T, J, DELTA, 1024>;  \
+    auto kern = p.dvp <= 128 ? state_serial_kernel<T, J, KIND, 512> : state_serial_kernel<T, J, KIND, 1024>;  \
     if (smem > 48 * 1024)                                                                                       \
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));          \
     kern<<<grid, p.dvp * 4, smem, stream>>>(p);                                                                 \
@@ -667,7 +783,7 @@ B2_EXPORT int b2_retention_serial(const void* q, const void* k, const void* v, c
   p.ld_qk = p.ld_v = p.ld_gate = ld_in; p.ld_out = ld_out;
   p.H = H; p.group = 1; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.rot = rot; p.kscale = kscale; p.eps = eps;
   p.tile = max_rows < 16 ? (max_rows < 1 ? 1 : max_rows) : 16;
-  B2_DISPATCH_T(is_f32, return (launch_serial<T, false>(p, nseq, static_cast<cudaStream_t>(stream))););
+  B2_DISPATCH_T(is_f32, return (launch_serial<T, RETENTION>(p, nseq, static_cast<cudaStream_t>(stream))););
 }
 
 B2_EXPORT int b2_delta_serial(const float* q, const float* k, const void* v, const float* glog, const float* beta,
@@ -683,7 +799,27 @@ B2_EXPORT int b2_delta_serial(const float* q, const float* k, const void* v, con
   p.ld_qk = static_cast<long long>(G) * dkp; p.ld_v = static_cast<long long>(H) * dvp; p.ld_gate = ld_gate; p.ld_out = ld_out;
   p.H = H; p.group = H / G; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.eps = eps;
   p.tile = max_rows < 16 ? (max_rows < 1 ? 1 : max_rows) : 16;
-  B2_DISPATCH_T(is_f32, return (launch_serial<T, true>(p, nseq, static_cast<cudaStream_t>(stream))););
+  B2_DISPATCH_T(is_f32, return (launch_serial<T, DELTA_RULE>(p, nseq, static_cast<cudaStream_t>(stream))););
+}
+
+// zi, zf: fp32 rows of stride ld_z (H columns); n: fp32 [slots, H, dkp]; m: fp32 [slots, H]; norm_w: T [H * dvp].
+B2_EXPORT int b2_memory_serial(const void* q, const void* k, const void* v, const void* gate, const float* zi, const float* zf,
+                               long long ld_z, const void* bi, const void* bf, const void* norm_w, void* out, float* state, float* n,
+                               float* m, const int* cu, const int* start, const int* slot, int nseq, int max_rows, int H, int dk,
+                               int dkp, int dv, int dvp, long long ld_in, long long ld_out, float cap, float qscale, float oscale,
+                               float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (nseq <= 0) return 0;
+  if (bad_heads("matrix_memory", H, 1, dk, dkp, dv, dvp, nseq)) return 10;
+  if (!(cap > 0.f)) { set_error("matrix_memory: the gates' cap must be positive"); return 10; }
+  SerialParams p = {};
+  p.seq = {cu, start, slot};
+  p.q = q; p.k = k; p.v = v; p.gate = gate; p.out = out; p.state = state; p.norm_w = norm_w;
+  p.ld_qk = p.ld_v = p.ld_gate = ld_in; p.ld_out = ld_out;
+  p.H = H; p.group = 1; p.dk = dk; p.dkp = dkp; p.dv = dv; p.dvp = dvp; p.kscale = 1.f; p.eps = eps;
+  p.zi = zi; p.zf = zf; p.bi = bi; p.bf = bf; p.n = n; p.m = m; p.ld_z = ld_z; p.cap = cap; p.qscale = qscale; p.oscale = oscale;
+  p.tile = max_rows < 16 ? (max_rows < 1 ? 1 : max_rows) : 16;
+  B2_DISPATCH_T(is_f32, return (launch_serial<T, MEMORY>(p, nseq, static_cast<cudaStream_t>(stream))););
 }
 
 B2_EXPORT int b2_delta_prep(const void* x, const void* taps, const void* b, const float* a2, const void* A_log,

@@ -1,0 +1,695 @@
+// Mixture of experts.
+//
+//   moe_route / moe_place   sigmoid scores, the choice among the best groups, and the (token, choice) pairs laid out expert after expert
+//   moe_gemm<GLU>           silu(W_gate h) * (W_up h) over every expert's rows, h gathered by token
+//   moe_gemm<DOWN>          W_down of those rows
+//   moe_norm_add            the weighted sum of a token's rows, a gated shared expert, the norm of the sum, the residual
+//
+// The products are persistent tcgen05 kernels over the list of (expert, 128-row tile, column tile): TMA brings the weights (one 3-D
+// map over all experts, so that a tile past an expert's last row is filled with zeros instead of its neighbour's rows), fp32
+// accumulators stay in TMEM, double-buffered.  The GLU form holds gate and up columns of a tile side by side in one accumulator, so
+// the activation happens on the way out; its token rows are gathered by four warps with asynchronous copies into the swizzled layout.
+// How many rows each expert has is known on the device only: every CTA works out the tile list from the offsets.
+#include "host.h"
+#include "vec.cuh"
+
+namespace b2 {
+
+constexpr int MOE_MAX_EXPERTS = 1024;
+constexpr int MOE_MAX_TOP = 32;
+typedef __nv_bfloat16 moe_bf16;
+
+// ---- routing -----------------------------------------------------------------------------------------------------------
+constexpr int MR_WARPS = 4;
+
+struct RouteParams {
+  const float* z;        // [M, ld]
+  const void* corr;      // T [E]
+  float* weights;        // [M, top]
+  int* place;            // [M, top]: rank among the expert's rows, then the row
+  int* count;            // [E], zero
+  int* id;               // [M, top]
+  long long ld;
+  int M, E, top, groups, keep;
+  float scale;
+};
+
+// largest value and, among equals, the lowest index
+__device__ __forceinline__ void argmax_warp(float& v, int& i) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float v2 = __shfl_xor_sync(0xffffffffu, v, o);
+    const int i2 = __shfl_xor_sync(0xffffffffu, i, o);
+    if (v2 > v || (v2 == v && i2 < i)) {
+      v = v2;
+      i = i2;
+    }
+  }
+}
+
+// A warp per token.
+template <typename T>
+__global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RouteParams p) {
+  extern __shared__ float mr_smem[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * MR_WARPS + warp;
+  if (row >= p.M) return;
+  float* c = mr_smem + warp * 2 * p.E;      // choice scores
+  float* gs = c + p.E;                      // group scores; a chosen group's is then marked
+  const float* z = p.z + static_cast<size_t>(row) * p.ld;
+  constexpr float LOW = -3.0e38f;           // in place of what is no number (rows without a sequence): below any score, above "closed"
+  for (int e = lane; e < p.E; e += 32) {
+    const float s = sigmoid_f(z[e]) + to_f(static_cast<const T*>(p.corr)[e]);
+    c[e] = s >= LOW ? s : LOW;
+  }
+  __syncwarp();
+  if (p.keep < p.groups) {
+    const int per = p.E / p.groups;
+    for (int g = lane; g < p.groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = c[e];
+        b = fmaxf(b, fminf(a, v));
+        a = fmaxf(a, v);
+      }
+      gs[g] = per > 1 ? fmaxf(a + b, LOW) : a;
+    }
+    __syncwarp();
+    for (int k = 0; k < p.keep; ++k) {
+      float v = -INFINITY;
+      int at = p.groups;
+      for (int g = lane; g < p.groups; g += 32)
+        if (gs[g] > v && gs[g] != INFINITY) {
+          v = gs[g];
+          at = g;
+        }
+      argmax_warp(v, at);
+      if (lane == 0 && at < p.groups) gs[at] = INFINITY;
+      __syncwarp();
+    }
+    for (int e = lane; e < p.E; e += 32)
+      if (gs[e / per] != INFINITY) c[e] = -INFINITY;
+    __syncwarp();
+  }
+  int mine = 0;
+  for (int k = 0; k < p.top; ++k) {
+    float v = -INFINITY;
+    int at = p.E;
+    for (int e = lane; e < p.E; e += 32)
+      if (c[e] > v) {
+        v = c[e];
+        at = e;
+      }
+    argmax_warp(v, at);
+    at = min(at, p.E - 1);
+    if (lane == k) mine = at;
+    if (lane == 0) c[at] = -INFINITY;
+    __syncwarp();
+  }
+  if (lane < p.top) {
+    const size_t i = static_cast<size_t>(row) * p.top + lane;
+    p.weights[i] = sigmoid_f(z[mine]) * p.scale;
+    p.id[i] = mine;
+    p.place[i] = atomicAdd(p.count + mine, 1);
+  }
+}
+
+// Running sums of f(i) over i < n by a whole warp: out[0 .. n].
+template <typename F>
+__device__ __forceinline__ void warp_prefix(int n, int* out, F f) {
+  const int lane = threadIdx.x & 31;
+  int carry = 0;
+  for (int i0 = 0; i0 < n; i0 += 32) {
+    const int i = i0 + lane;
+    int v = i < n ? f(i) : 0;
+    const int own = v;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int t = __shfl_up_sync(0xffffffffu, v, o);
+      if (lane >= o) v += t;
+    }
+    if (i < n) out[i] = carry + v - own;
+    carry += __shfl_sync(0xffffffffu, v, 31);
+  }
+  if (lane == 0) out[n] = carry;
+}
+
+__global__ void __launch_bounds__(256) moe_place_kernel(const int* __restrict__ count, const int* __restrict__ id, int* __restrict__ place,
+                                                        int* __restrict__ token, int* __restrict__ offsets, int E, int top, int total) {
+  __shared__ int off[MOE_MAX_EXPERTS + 1];
+  if (threadIdx.x < 32) warp_prefix(E, off, [&](int e) { return count[e]; });
+  __syncthreads();
+  if (blockIdx.x == 0)
+    for (int e = threadIdx.x; e <= E; e += 256) offsets[e] = off[e];
+  for (int i = blockIdx.x * 256 + threadIdx.x; i < total; i += gridDim.x * 256) {
+    const int r = off[id[i]] + place[i];
+    place[i] = r;
+    token[r] = i / top;
+  }
+}
+
+// ---- grouped products ----------------------------------------------------------------------------------------------------
+// The tile list: expert e has ceil(rows / tile) row tiles, first[e] of them before it.
+struct MoeTile {
+  int expert, row0, rows, col;       // rows of the layout; column tile
+};
+__device__ __forceinline__ MoeTile moe_tile(int t, const int* off, const int* first, int E, int tile, int ncols) {
+  // tiles of one expert are neighbours, its row tiles innermost: they share the weights' columns
+  int lo = 0, hi = E;
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) / 2;
+    if (first[mid] * ncols <= t) lo = mid;
+    else hi = mid;
+  }
+  const int n = first[lo + 1] - first[lo], in = t - first[lo] * ncols;
+  MoeTile r;
+  r.expert = lo;
+  r.col = in / n;
+  r.row0 = off[lo] + in % n * tile;
+  r.rows = min(tile, off[lo + 1] - r.row0);
+  return r;
+}
+
+// 32-bit form: 64 x 64 tiles of plain FMAs.  Grid (column tiles, an upper bound of the row tiles).
+constexpr int MF_T = 64, MF_K = 16;
+template <bool GLU>
+__global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restrict__ W,
+                                                           const int* __restrict__ token, const int* __restrict__ offsets,
+                                                           float* __restrict__ out, int E, int N, int K) {
+  __shared__ int off[MOE_MAX_EXPERTS + 1], first[MOE_MAX_EXPERTS + 1];
+  __shared__ __align__(16) float sA[MF_K][MF_T + 4], sB[GLU ? 2 : 1][MF_K][MF_T + 4];   // read in vectors of four
+  for (int e = threadIdx.x; e <= E; e += 256) off[e] = offsets[e];
+  __syncthreads();
+  if (threadIdx.x < 32) warp_prefix(E, first, [&](int e) { return (off[e + 1] - off[e] + MF_T - 1) / MF_T; });
+  __syncthreads();
+  if (static_cast<int>(blockIdx.y) >= first[E]) return;
+  const MoeTile tl = moe_tile(blockIdx.y, off, first, E, MF_T, 1);
+  const int n0 = blockIdx.x * MF_T, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const float* w = W + static_cast<size_t>(tl.expert) * (GLU ? 2 : 1) * N * K;
+  float acc[GLU ? 2 : 1][4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += MF_K) {
+    for (int i = threadIdx.x; i < MF_T * MF_K; i += 256) {
+      const int r = i / MF_K, k = i % MF_K;
+      const bool in = k0 + k < K;
+      const size_t row = GLU ? (r < tl.rows ? token[tl.row0 + r] : 0) : tl.row0 + r;
+      sA[k][r] = in && r < tl.rows ? A[row * lda + k0 + k] : 0.f;
+#pragma unroll
+      for (int g = 0; g < (GLU ? 2 : 1); ++g)
+        sB[g][k][r] = in && n0 + r < N ? w[(static_cast<size_t>(g) * N + n0 + r) * K + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < MF_K; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&sA[k][ty * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+      for (int g = 0; g < (GLU ? 2 : 1); ++g) {
+        const float4 b = *reinterpret_cast<const float4*>(&sB[g][k][tx * 4]);
+        const float bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[g][i][j] = fmaf(av[i], bv[j], acc[g][i][j]);
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = ty * 4 + i;
+    if (m >= tl.rows) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n < N) out[static_cast<size_t>(tl.row0 + m) * N + n] = GLU ? silu_f(acc[0][i][j]) * acc[GLU ? 1 : 0][i][j] : acc[0][i][j];
+    }
+  }
+}
+
+constexpr int MG_BM = 128, MG_BK = 64;
+constexpr int MG_LAG = 2;                  // k-blocks whose gathered rows may still be on their way
+
+template <int BN>
+struct MoeCfg {
+  static constexpr int A_BYTES = MG_BM * MG_BK * 2, B_BYTES = BN * MG_BK * 2, STAGE = A_BYTES + B_BYTES;
+  static constexpr int STAGES = BN == 256 ? 4 : BN == 128 ? 6 : 8;
+  static constexpr int STAGING = 4 * 4096;                        // a block per epilogue warp
+  static constexpr int TABLES = 2 * (MOE_MAX_EXPERTS + 1) * 4;
+  static constexpr int SMEM = STAGES * STAGE + STAGING + 256 + TABLES + 1024;
+  static constexpr int TMEM = 2 * BN;
+};
+
+struct MoeGemmParams {
+  const moe_bf16* a;       // GLU: token rows [tokens, lda]
+  long long lda;
+  const int* token;        // GLU: [P]
+  const int* offsets;      // [E + 1]
+  moe_bf16* out;           // [P, N]
+  int E, N, K;             // GLU: N activation columns (half of a tile's accumulator columns each for gate and up)
+};
+
+template <int BN, bool GLU>
+__global__ void __launch_bounds__(GLU ? 320 : 192, 1)
+moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const MoeGemmParams p, int* status) {
+  using Cfg = MoeCfg<BN>;
+  constexpr int STAGES = Cfg::STAGES, COLS = GLU ? BN / 2 : BN;    // output columns of a tile
+  static_assert(MG_LAG < STAGES, "a stage is handed over before it is needed again");
+  extern __shared__ uint8_t mg_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(mg_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  uint8_t* staging = smem + STAGES * Cfg::STAGE;
+  uint64_t* full = reinterpret_cast<uint64_t*>(staging + Cfg::STAGING);
+  uint64_t *empty = full + STAGES, *acc_full = empty + STAGES, *acc_empty = acc_full + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
+  int* off = reinterpret_cast<int*>(staging + Cfg::STAGING + 256);
+  int* first = off + MOE_MAX_EXPERTS + 1;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (tid == 0) {
+    for (int i = 0; i < STAGES; ++i) {
+      mbar_init(full + i, GLU ? 1 + 4 : 1);       // the weights' copy, and the gathering warps
+      mbar_init(empty + i, 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(acc_full + i, 1);
+      mbar_init(acc_empty + i, 4);
+    }
+    mbar_fence_init();
+    tma_prefetch_desc(&tmB);
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, Cfg::TMEM);
+    tmem_relinquish();
+  }
+  for (int e = tid; e <= p.E; e += blockDim.x) off[e] = p.offsets[e];
+  __syncthreads();
+  if (warp == 0) warp_prefix(p.E, first, [&](int e) { return (off[e + 1] - off[e] + MG_BM - 1) / MG_BM; });
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
+  const int ncols = (p.N + COLS - 1) / COLS, tiles = first[p.E] * ncols, nkb = (p.K + MG_BK - 1) / MG_BK;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      int st = 0;
+      uint32_t ph = 0;
+      bool ok = true;
+      for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
+        const MoeTile tl = moe_tile(t, off, first, p.E, MG_BM, ncols);
+        for (int kb = 0; kb < nkb; ++kb) {
+          if (!mbar_wait(empty + st, ph ^ 1, status, ERR_GEMM_PRODUCER_WAIT)) {
+            ok = false;
+            break;
+          }
+          uint8_t *sA = smem + st * Cfg::STAGE, *sB = sA + Cfg::A_BYTES;
+          mbar_expect_tx(full + st, Cfg::B_BYTES + (GLU ? 0 : Cfg::A_BYTES));
+          if (GLU) {
+            tma_load_3d(sB, &tmB, full + st, kb * MG_BK, tl.col * COLS, 2 * tl.expert);
+            tma_load_3d(sB + Cfg::B_BYTES / 2, &tmB, full + st, kb * MG_BK, tl.col * COLS, 2 * tl.expert + 1);
+          } else {
+            tma_load_2d(sA, &tmA, full + st, kb * MG_BK, tl.row0);
+            tma_load_3d(sB, &tmB, full + st, kb * MG_BK, tl.col * COLS, tl.expert);
+          }
+          if (++st == STAGES) {
+            st = 0;
+            ph ^= 1;
+          }
+        }
+      }
+    }
+  } else if (warp == 1) {
+    const bool leader = elect_one();
+    constexpr uint32_t idesc = make_idesc_f16(1, MG_BM, BN, 0, 0);
+    int st = 0, acc = 0;
+    uint32_t ph = 0, acc_ph = 0;
+    bool ok = true;
+    for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
+      if (!mbar_wait(acc_empty + acc, acc_ph ^ 1, status, ERR_GEMM_MMA_WAIT_TMEM)) break;
+      tc_fence_after();
+      for (int kb = 0; kb < nkb; ++kb) {
+        if (!mbar_wait(full + st, ph, status, ERR_GEMM_MMA_WAIT_FULL)) {
+          ok = false;
+          break;
+        }
+        tc_fence_after();
+        const uint32_t a_base = smem_u32(smem + st * Cfg::STAGE);
+        const uint64_t a0 = make_smem_desc_sw128(a_base, 16, 1024), b0 = make_smem_desc_sw128(a_base + Cfg::A_BYTES, 16, 1024);
+        if (leader) {
+#pragma unroll
+          for (int k = 0; k < MG_BK / 16; ++k)
+            umma_f16_ss(tmem + acc * BN, desc_advance(a0, k * 32), desc_advance(b0, k * 32), idesc, kb > 0 || k > 0 ? 1u : 0u);
+          umma_commit(empty + st);
+        }
+        if (++st == STAGES) {
+          st = 0;
+          ph ^= 1;
+        }
+      }
+      if (!ok) break;
+      if (leader) umma_commit(acc_full + acc);
+      acc ^= 1;
+      if (acc == 0) acc_ph ^= 1;
+    }
+  } else if (GLU && warp >= 6) {
+    // Token rows into the swizzled A tile: eight lanes a row (whole 128-byte lines), rows 32 w .. 32 w + 31 of warp w.  A stage is
+    // handed over MG_LAG k-blocks after its copies were issued, once they have landed and are visible to the tensor core.
+    const int w = warp - 6, chunk = lane & 7, sub = lane >> 3;
+    int st = 0, done = 0;            // stages issued into, handed over
+    uint32_t ph = 0;
+    int pending = 0;
+    bool ok = true;
+    auto hand_over = [&]() {
+      fence_proxy_async_smem();
+      mbar_arrive_warp(full + done);
+      if (++done == STAGES) done = 0;
+      --pending;
+    };
+    for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
+      const MoeTile tl = moe_tile(t, off, first, p.E, MG_BM, ncols);
+      const moe_bf16* src[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int r = w * 32 + j * 4 + sub;
+        src[j] = p.a + (r < tl.rows ? static_cast<size_t>(p.token[tl.row0 + r]) * p.lda : 0) + chunk * 8;
+      }
+      for (int kb = 0; kb < nkb; ++kb) {
+        if (!mbar_wait_warp(empty + st, ph ^ 1, status, ERR_GEMM_PRODUCER_WAIT)) {
+          ok = false;
+          break;
+        }
+        const uint32_t base = smem_u32(smem + st * Cfg::STAGE) + (w * 32 + sub) * 128;
+        const int bytes = kb * MG_BK + chunk * 8 < p.K ? 16 : 0;       // zeros past the last column (p.K is a multiple of 8)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const int r = j * 4 + sub;
+          if (w * 32 + r < tl.rows)        // rows past the expert's last one keep what they hold: their results are dropped
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(base + j * 512 + ((chunk ^ (r & 7)) << 4)),
+                         "l"(bytes ? src[j] + kb * MG_BK : p.a), "r"(bytes)
+                         : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        ++pending;
+        if (++st == STAGES) {
+          st = 0;
+          ph ^= 1;
+        }
+        if (pending > MG_LAG) {
+          asm volatile("cp.async.wait_group %0;" ::"n"(MG_LAG) : "memory");
+          hand_over();
+        }
+      }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    while (pending > 0) hand_over();
+  } else {
+    const int quarter = warp & 3;
+    uint8_t* stage = staging + quarter * 4096;
+    int acc = 0;
+    uint32_t acc_ph = 0;
+    for (int t = blockIdx.x; t < tiles; t += gridDim.x) {
+      const MoeTile tl = moe_tile(t, off, first, p.E, MG_BM, ncols);
+      if (!mbar_wait_warp(acc_full + acc, acc_ph, status, ERR_GEMM_EPI_WAIT)) break;
+      tc_fence_after();
+      const uint32_t at = tmem + (static_cast<uint32_t>(quarter * 32) << 16) + acc * BN;
+      const bool live = quarter * 32 < tl.rows;
+#pragma unroll 1
+      for (int c0 = 0; c0 < COLS; c0 += 64) {
+        if (!live || tl.col * COLS + c0 >= p.N) break;
+        uint4 v[8];
+        constexpr int W32 = COLS < 64 ? COLS / 32 : 2;
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+          uint32_t r[32];
+          if (hh >= W32) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[hh * 4 + j] = make_uint4(0, 0, 0, 0);
+            continue;
+          }
+          tmem_ld_32x32b_x32(at + c0 + hh * 32, r);
+          if (GLU) {
+            uint32_t u[32];
+            tmem_ld_32x32b_x32(at + BN / 2 + c0 + hh * 32, u);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+              float x = __uint_as_float(r[i]), y = __uint_as_float(r[i + 1]);
+              silu_pair_fast(x, y);
+              r[i] = __float_as_uint(x * __uint_as_float(u[i]));
+              r[i + 1] = __float_as_uint(y * __uint_as_float(u[i + 1]));
+            }
+          } else {
+            tmem_ld_wait();
+          }
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            uint32_t o[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[e] = pack_bf16x2(__uint_as_float(r[8 * j + 2 * e]), __uint_as_float(r[8 * j + 2 * e + 1]));
+            v[hh * 4 + j] = make_uint4(o[0], o[1], o[2], o[3]);
+          }
+        }
+        const int col = tl.col * COLS + c0;
+        moe_bf16* base = p.out + static_cast<size_t>(tl.row0 + quarter * 32) * p.N + col;
+        warp_store_rows_128B(stage, v, [&](int row) -> uint8_t* {
+          if (quarter * 32 + row >= tl.rows || col + (lane & 7) * 8 >= p.N || c0 + (lane & 7) * 8 >= COLS) return nullptr;
+          return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * p.N);
+        });
+      }
+      tc_fence_before();
+      mbar_arrive_warp(acc_empty + acc);
+      acc ^= 1;
+      if (acc == 0) acc_ph ^= 1;
+    }
+  }
+  if (*reinterpret_cast<volatile int*>(status) != 0) {     // copies and products in flight land before shared memory and TMEM go away
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    __syncwarp();
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::TMEM);
+  }
+}
+
+// ---- weighted sum, norm, residual ---------------------------------------------------------------------------------------------
+struct MoeAddParams {
+  float* x;              // [M, ld]
+  const void* rows;      // T [P, ld]
+  const int* place;      // [M, top]
+  const float* weights;  // [M, top]
+  const float* shared;   // [M, ld] or null
+  const float* sg;       // [M], stride ld_sg: gate before its sigmoid
+  const void* w;         // T [ld]
+  void* h;               // T [M, ld] or null
+  int top, ld_sg, ld, n;
+  float coef, eps;
+};
+
+__device__ __forceinline__ float moe_block_sum(float v, float* scratch) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int lane = threadIdx.x & 31;
+  return warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? scratch[lane] : 0.f);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) moe_norm_add_kernel(const MoeAddParams p) {
+  __shared__ float scratch[32], sw[MOE_MAX_TOP];
+  __shared__ int sr[MOE_MAX_TOP];
+  const size_t base = static_cast<size_t>(blockIdx.x) * p.ld;
+  if (static_cast<int>(threadIdx.x) < p.top) {
+    sw[threadIdx.x] = p.weights[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
+    sr[threadIdx.x] = p.place[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
+  }
+  const float g = p.shared ? sigmoid_f(p.sg[static_cast<size_t>(blockIdx.x) * p.ld_sg]) : 0.f;
+  __syncthreads();
+  const T* rows = static_cast<const T*>(p.rows);
+  float a[V][8], b[V][8], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] = b[k][e] = 0.f;
+    if (c >= p.ld) continue;
+    vload8(p.x + base + c, b[k]);
+    if (p.shared) {
+      vload8(p.shared + base + c, a[k]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[k][e] *= g;
+    }
+    for (int j = 0; j < p.top; j += 4) {
+      float t[4][8];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (j + i < p.top) vload8(rows + static_cast<size_t>(sr[j + i]) * p.ld + c, t[i]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (j + i < p.top)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) a[k][e] = fmaf(sw[j + i], t[i][e], a[k][e]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < V; ++k)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(a[k][e], a[k][e], ss);
+  const float r = p.coef / sqrtf(moe_block_sum(ss, scratch) / p.n + p.eps);
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c >= p.ld) break;
+    float wv[8];
+    vload8(static_cast<const T*>(p.w) + c, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) b[k][e] = fmaf(a[k][e] * r, wv[e], b[k][e]);
+    vstore8(p.x + base + c, b[k]);
+    if (p.h) vstore8(static_cast<T*>(p.h) + base + c, b[k]);
+  }
+}
+
+template <int BN, bool GLU>
+static int launch_moe(const CUtensorMap* ta, const CUtensorMap* tb, const MoeGemmParams& p, int bound, cudaStream_t stream) {
+  using Cfg = MoeCfg<BN>;
+  auto kern = moe_gemm_kernel<BN, GLU>;
+  int* status = status_ptr();
+  if (!status) return 3;
+  static bool set[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!set[dev & 63]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
+      set_error("moe_gemm: cannot set shared memory size (%d)", Cfg::SMEM);
+      return 1;
+    }
+    set[dev & 63] = true;
+  }
+  constexpr int COLS = GLU ? BN / 2 : BN;
+  const long long tiles = static_cast<long long>(bound) * ((p.N + COLS - 1) / COLS);
+  const int grid = tiles < num_sms() ? static_cast<int>(tiles) : num_sms();
+  kern<<<grid, GLU ? 320 : 192, Cfg::SMEM, stream>>>(*ta, *tb, p, status);
+  B2_CHECK_LAUNCH("moe_gemm");
+  return 0;
+}
+
+static int moe_bound(int P, int E, int tile) { return P / tile + (E < P ? E : P); }    // row tiles at most
+
+// Column tile: the widest that still gives every SM a few tiles, by the expected number of row tiles.
+static int moe_columns(int P, int E, int N, int widest) {
+  const int used = E < P ? E : P;
+  const long long rows = static_cast<long long>(used) * ((P / used + MG_BM - 1) / MG_BM);
+  int cols = widest;
+  while (cols > 32 && rows * ((N + cols - 1) / cols) < 4 * num_sms()) cols /= 2;
+  return cols;
+}
+
+}  // namespace b2
+
+using namespace b2;
+
+// z: fp32 [M, ld]; work: int32 [E + M * top]; offsets: int32 [E + 1]; place: int32 [M, top]; token: int32 [M * top].
+B2_EXPORT int b2_moe_route(const float* z, long long ld, const void* corr, float* weights, int* place, int* token, int* offsets,
+                           int* work, int M, int E, int top, int groups, int keep, float scale, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (E < 1 || E > MOE_MAX_EXPERTS || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > MOE_MAX_TOP ||
+      top > keep * (E / groups) || static_cast<long long>(M) * top > 0x7fffffffll || ld < E) {
+    set_error("moe_route: up to %d experts in equal groups and up to %d chosen required", MOE_MAX_EXPERTS, MOE_MAX_TOP);
+    return 10;
+  }
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (cudaMemsetAsync(work, 0, sizeof(int) * E, st) != cudaSuccess) { set_error("moe_route: clearing the counts failed"); return 5; }
+  const RouteParams p = {z, corr, weights, place, work, work + E, ld, M, E, top, groups, keep, scale};
+  B2_DISPATCH_T(is_f32, moe_route_kernel<T><<<(M + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, MR_WARPS * 2 * E * sizeof(float), st>>>(p););
+  B2_CHECK_LAUNCH("moe_route");
+  const int total = M * top, blocks = (total + 255) / 256;
+  moe_place_kernel<<<blocks < 2 * num_sms() ? blocks : 2 * num_sms(), 256, 0, st>>>(work, work + E, place, token, offsets, E, top, total);
+  B2_CHECK_LAUNCH("moe_place");
+  return 0;
+}
+
+// h: T [tokens, ld], w: T [E, 2, F, K], token: int32 [P] -> out T [P, F]
+B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* token, const int* offsets, void* out, int tokens, int P,
+                         int E, int F, int K, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (P <= 0) return 0;
+  if (E < 1 || E > MOE_MAX_EXPERTS || F < 8 || F % 8 || K < 8 || K % 8 || ld % 8 || ld < K || tokens < 1) {
+    set_error("moe_glu: up to %d experts and sizes in multiples of 8 required", MOE_MAX_EXPERTS);
+    return 10;
+  }
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (is_f32) {
+    const int rows = moe_bound(P, E, MF_T);
+    if (rows > 65535) { set_error("moe_glu: too many rows (%d)", P); return 10; }
+    moe_gemm_f32_kernel<true><<<dim3((F + MF_T - 1) / MF_T, rows), 256, 0, st>>>(
+        static_cast<const float*>(h), ld, static_cast<const float*>(w), token, offsets, static_cast<float*>(out), E, F, K);
+    B2_CHECK_LAUNCH("moe_glu");
+    return 0;
+  }
+  const int cols = moe_columns(P, E, F, 128);
+  const uint64_t dims[3] = {static_cast<uint64_t>(K), static_cast<uint64_t>(F), 2ull * E},
+                 strides[2] = {2ull * K, 2ull * F * K};
+  const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
+  const CUtensorMap* tb = tensor_map_nd_bf16(w, 3, dims, strides, box, 3);
+  if (!tb) return 2;
+  MoeGemmParams p = {static_cast<const moe_bf16*>(h), ld, token, offsets, static_cast<moe_bf16*>(out), E, F, K};
+  const int bound = moe_bound(P, E, MG_BM);
+  if (cols == 128) return launch_moe<256, true>(tb, tb, p, bound, st);
+  if (cols == 64) return launch_moe<128, true>(tb, tb, p, bound, st);
+  return launch_moe<64, true>(tb, tb, p, bound, st);
+}
+
+// a: T [P, F], w: T [E, N, F] -> out T [P, N]
+B2_EXPORT int b2_moe_down(const void* a, const void* w, const int* offsets, void* out, int P, int E, int N, int F, int is_f32,
+                          void* stream) {
+  b2::ensure_thread_context();
+  if (P <= 0) return 0;
+  if (E < 1 || E > MOE_MAX_EXPERTS || F < 8 || F % 8 || N < 8 || N % 8) {
+    set_error("moe_down: up to %d experts and sizes in multiples of 8 required", MOE_MAX_EXPERTS);
+    return 10;
+  }
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (is_f32) {
+    const int rows = moe_bound(P, E, MF_T);
+    if (rows > 65535) { set_error("moe_down: too many rows (%d)", P); return 10; }
+    moe_gemm_f32_kernel<false><<<dim3((N + MF_T - 1) / MF_T, rows), 256, 0, st>>>(
+        static_cast<const float*>(a), F, static_cast<const float*>(w), nullptr, offsets, static_cast<float*>(out), E, N, F);
+    B2_CHECK_LAUNCH("moe_down");
+    return 0;
+  }
+  int cols = moe_columns(P, E, N, 256);
+  if (cols < 64) cols = 64;
+  const uint64_t dims[3] = {static_cast<uint64_t>(F), static_cast<uint64_t>(N), static_cast<uint64_t>(E)},
+                 strides[2] = {2ull * F, 2ull * N * F};
+  const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
+  const CUtensorMap *tb = tensor_map_nd_bf16(w, 3, dims, strides, box, 3), *ta = tensor_map_2d_bf16(a, P, F, F, MG_BM, MG_BK);
+  if (!ta || !tb) return 2;
+  MoeGemmParams p = {nullptr, 0, nullptr, offsets, static_cast<moe_bf16*>(out), E, N, F};
+  const int bound = moe_bound(P, E, MG_BM);
+  if (cols == 256) return launch_moe<256, false>(ta, tb, p, bound, st);
+  if (cols == 128) return launch_moe<128, false>(ta, tb, p, bound, st);
+  return launch_moe<64, false>(ta, tb, p, bound, st);
+}
+
+B2_EXPORT int b2_moe_norm_add(float* x, const void* rows, const int* place, const float* weights, int top, const float* shared,
+                              const float* sg, int ld_sg, const void* w, void* h, int M, int ld, int n, float coef, float eps,
+                              int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld || ld > 32768 || top < 1 || top > MOE_MAX_TOP || (shared != nullptr && sg == nullptr)) {
+    set_error("moe_norm_add: ld %% 8 == 0, 0 < n <= ld <= 32768 and up to %d rows a token required", MOE_MAX_TOP);
+    return 10;
+  }
+  const MoeAddParams p = {x, rows, place, weights, shared, sg, w, h, top, ld_sg, ld, n, coef, eps};
+  const int pieces = ld / 8, V = pieces <= 256 ? 1 : pieces <= 512 ? 2 : 4;
+  const int threads = ((pieces + V - 1) / V + 31) / 32 * 32;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  B2_DISPATCH_T(is_f32, {
+    if (V == 1) moe_norm_add_kernel<T, 1><<<M, threads, 0, st>>>(p);
+    else if (V == 2) moe_norm_add_kernel<T, 2><<<M, threads, 0, st>>>(p);
+    else moe_norm_add_kernel<T, 4><<<M, threads, 0, st>>>(p);
+  });
+  B2_CHECK_LAUNCH("moe_norm_add");
+  return 0;
+}

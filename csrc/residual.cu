@@ -1,6 +1,7 @@
 // Kernels around a 32-bit residual stream: embedding into it, RMS norm out of it, the half-sum of two normed branches
-// added to it (with the next norm in the same pass), gated activation over column slices, rotary tables for a batch's
-// positions, and the 32-bit matrix product used when a model runs without any reduced-precision mode.
+// added to it (with the next norm in the same pass), one normed branch added to it, gated activations over column slices or with a
+// table of per-token vectors, rotary tables for a batch's positions, and the 32-bit matrix product used when a model runs without
+// any reduced-precision mode.
 //
 // Rows of the residual and of every activation are padded to a multiple of eight columns; `n` is the real width.  The
 // padding columns are zero (their norm weights are zero), so vector accesses never need a tail.
@@ -40,7 +41,7 @@ __global__ void __launch_bounds__(RES_THREADS) embed_f32_kernel(const long long*
 template <typename T>
 __global__ void __launch_bounds__(RES_THREADS) rmsnorm_f32_kernel(const float* __restrict__ x, const T* __restrict__ w,
                                                                   T* __restrict__ h, const long long* __restrict__ rows, int ld,
-                                                                  int n, float eps) {
+                                                                  int n, float eps, float scale) {
   __shared__ float scratch[32];
   const size_t src = rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
   const float* xr = x + src * ld;
@@ -58,7 +59,7 @@ __global__ void __launch_bounds__(RES_THREADS) rmsnorm_f32_kernel(const float* _
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[k][e] = t[e];
   }
-  const float r = 1.f / sqrtf(res_block_sum(ss, scratch) / n + eps);
+  const float r = scale / sqrtf(res_block_sum(ss, scratch) / n + eps);
   i = 0;
   for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8, ++i) {
     float t[8], wv[8];
@@ -181,6 +182,64 @@ __global__ void __launch_bounds__(RES_THREADS) merge_norm_add_kernel(float* __re
   }
 }
 
+// x += coef * rms(f y) * w, and the new x rounded to T in h (optional).  y: fp32 [M, ld].  A row's pieces (V per thread) stay in
+// registers; both rows are requested before the first is used.
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const T* __restrict__ w,
+                                                        T* __restrict__ h, int ld, int n, float coef, float eps, float f) {
+  __shared__ float scratch[32];
+  const size_t base = static_cast<size_t>(blockIdx.x) * ld;
+  float a[V][8], b[V][8], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] = b[k][e] = 0.f;
+    if (c < ld) {
+      vload8(y + base + c, a[k]);
+      vload8(x + base + c, b[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < V; ++k)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      a[k][e] *= f;
+      ss = fmaf(a[k][e], a[k][e], ss);
+    }
+  const float r = coef / sqrtf(res_block_sum(ss, scratch) / n + eps);
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c >= ld) break;
+    float wv[8];
+    vload8(w + c, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) b[k][e] = fmaf(a[k][e] * r, wv[e], b[k][e]);
+    vstore8(x + base + c, b[k]);
+    if (h) vstore8(h + base + c, b[k]);
+  }
+}
+
+// out = gelu_tanh(gate) * table[id, first ...]: ids outside the vocabulary (padding rows) give zeros
+template <typename T>
+__global__ void __launch_bounds__(RES_THREADS) gelu_token_kernel(const T* __restrict__ gate, const T* __restrict__ table,
+                                                                 const long long* __restrict__ ids, T* __restrict__ out, int n,
+                                                                 int ld_gate, long long ld_table, int first, int vocab, long long total) {
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long row = i / (n / 8);
+    const int c = static_cast<int>(i - row * (n / 8)) * 8;
+    const long long id = ids[row];
+    float g[8], t[8] = {};
+    vload8(gate + row * ld_gate + c, g);
+    if (id >= 0 && id < vocab) vload8(table + id * ld_table + first + c, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = gelu_tanh_t<T>(g[e]) * t[e];
+    vstore8(out + row * n + c, g);
+  }
+}
+
 // out = silu(gate) * up over column slices (row strides ld_in / ld_out)
 template <typename T>
 __global__ void __launch_bounds__(RES_THREADS) glu_kernel(const T* __restrict__ gate, const T* __restrict__ up,
@@ -273,12 +332,12 @@ B2_EXPORT int b2_embed_f32(const long long* ids, const void* table, float* x, vo
 }
 
 B2_EXPORT int b2_rmsnorm_f32(const float* x, const void* w, void* h, const long long* rows, int M, int ld, int n, float eps,
-                             int is_f32, void* stream) {
+                             float scale, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (ld % 8 || n <= 0 || n > ld) { set_error("rmsnorm_f32: ld %% 8 == 0 and 0 < n <= ld required"); return 10; }
   B2_DISPATCH_T(is_f32, rmsnorm_f32_kernel<T><<<M, RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
-      x, static_cast<const T*>(w), static_cast<T*>(h), rows, ld, n, eps););
+      x, static_cast<const T*>(w), static_cast<T*>(h), rows, ld, n, eps, scale););
   B2_CHECK_LAUNCH("rmsnorm_f32");
   return 0;
 }
@@ -296,6 +355,44 @@ B2_EXPORT int b2_post_norm(float* x, const float* y, const void* w, const void* 
   B2_DISPATCH_T(is_f32, post_norm_kernel<T><<<M, threads, 0, static_cast<cudaStream_t>(stream)>>>(
       x, y, static_cast<const T*>(w), static_cast<const T*>(b), ss, parts, nss, static_cast<T*>(h), ld, n, alpha, eps););
   B2_CHECK_LAUNCH("post_norm");
+  return 0;
+}
+
+B2_EXPORT int b2_norm_add(float* x, const float* y, const void* w, void* h, int M, int ld, int n, float coef, float eps, float y_scale,
+                          int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld || ld > 32768) { set_error("norm_add: ld %% 8 == 0, 0 < n <= ld <= 32768 required"); return 10; }
+  const int pieces = ld / 8, V = pieces <= 256 ? 1 : pieces <= 512 ? 2 : 4;
+  const int threads = ((pieces + V - 1) / V + 31) / 32 * 32;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  B2_DISPATCH_T(is_f32, {
+    const T* wt = static_cast<const T*>(w);
+    T* ht = static_cast<T*>(h);
+    if (V == 1) norm_add_kernel<T, 1><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+    else if (V == 2) norm_add_kernel<T, 2><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+    else norm_add_kernel<T, 4><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+  });
+  B2_CHECK_LAUNCH("norm_add");
+  return 0;
+}
+
+// gate [M, n] (row stride ld_gate), table rows of stride ld_table; n, first and the strides multiples of 8
+B2_EXPORT int b2_gelu_token(const void* gate, const void* table, const long long* ids, void* out, int M, int n, int ld_gate,
+                            long long ld_table, int first, int vocab, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (n < 8 || n % 8 || ld_gate % 8 || ld_table % 8 || first % 8 || first < 0 || first + n > ld_table) {
+    set_error("gelu_token: columns and strides must be multiples of 8");
+    return 10;
+  }
+  const long long total = static_cast<long long>(M) * (n / 8);
+  long long blocks = (total + RES_THREADS - 1) / RES_THREADS;
+  const long long cap = static_cast<long long>(num_sms()) * 16;
+  if (blocks > cap) blocks = cap;
+  B2_DISPATCH_T(is_f32, gelu_token_kernel<T><<<static_cast<int>(blocks), RES_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const T*>(gate), static_cast<const T*>(table), ids, static_cast<T*>(out), n, ld_gate, ld_table, first, vocab, total););
+  B2_CHECK_LAUNCH("gelu_token");
   return 0;
 }
 

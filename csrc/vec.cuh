@@ -64,6 +64,13 @@ __device__ __forceinline__ float silu_t(float z) { return sizeof(T) == 2 ? silu_
 template <typename T>
 __device__ __forceinline__ float sigmoid_t(float z) { return sizeof(T) == 2 ? sigmoid_fast(z) : sigmoid_f(z); }
 
+// gelu in its tanh form: 0.5 z (1 + tanh(u)) = z sigmoid(2 u), u = sqrt(2 / pi) (z + 0.044715 z^3)
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_t(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z * sigmoid_t<T>(2.f * u);
+}
+
 // two fp32 multiplications or fused multiply-adds in one instruction
 __device__ __forceinline__ float2 mul_f32x2(float2 a, float2 b) {
   unsigned long long d;
