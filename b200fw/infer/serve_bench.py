@@ -310,6 +310,92 @@ def sotazen_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     return t.rows
 
 
+def ruburax_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    """The same for the attention / parallel / gated-recurrence decoder with experts."""
+    mc, t = PRESETS[preset], _Timer()
+    W, V, eps = mc.hidden_size, mc.vocab_size, mc.rms_norm_eps
+    kinds = {k: next(l["mixer"] for l in mc.layers if l["type"] == k) for k in ("attention", "parallel", "rglru")}
+    p, pages, starts, counts = _layout(lengths, batch, ctx)
+    M, n = p.rows, p.nseq
+    x, y32, w, h = torch.randn(M, W, device=DEV), torch.randn(M, W, device=DEV), _bf(W), _bf(M, W)
+    t("norm_add", lambda: ops.norm_add(x, y32, w, 0.5, W, eps), M * W * 14)
+
+    a = kinds["attention"]
+    H, G, dk, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+    lq, lk, lv = H * dk, G * dk, G * dv
+    _gemm(t, "gemm in (attention)", M, lq + lk + lv, W)
+    _gemm(t, "gemm in (attention, shared keys)", M, lq, W)
+    kc, vc = _bf(pages, 16, G, dk), _bf(pages, 16, G, dv)
+    yy, wd, bias, sink = _bf(M, lq + lk + lv), _bf(dk), _bf(lq + lk + lv), _bf(H)
+    s = a["rot"]["scaling"]
+    cs, sn = ops.rope_rows(p.positions, ops.rope_turns(a["rot"]["base"], a["rot"]["dims"], DEV, (s["factor"], s["low"], s["high"], s["original"])))
+
+    def store():
+        return ops.qk_norm_store(yy[:, :lq], yy[:, lq:lq + lk], yy[:, lq + lk:], kc, vc, p, H, dk, True, eps, wd, wd, bias, cs, sn)
+    t("qk_norm_store", store, M * ((lq + lk + lv) * 4 + a["rot"]["dims"] * 4))
+    t("qk_norm_store (queries alone)", lambda: ops.qk_norm_store(yy[:, :lq], None, None, kc, vc, p, H, dk, True, eps, wd, None, bias[:lq], cs, sn),
+      M * (lq * 4 + a["rot"]["dims"] * 4))
+    q, out = store(), _bf(M, H * dv)
+    pairs = sum((s + k) * (s + k + 1) / 2 - s * (s + 1) / 2 for s, k in zip(starts, counts))
+    t("paged_attention", lambda: ops.paged_attention(q, kc, vc, out, p, H, a["scale"], sink=sink),
+      M * (lq + H * dv) * 2 + (pairs if lengths is None else M) * (lk + lv) * 2, 2.0 * pairs * H * (dk + dv))
+    _gemm(t, "gemm attention o (fp32)", M, W, H * dv, True)
+
+    b = kinds["parallel"]["right"]
+    H2, dk, dv = b["heads"], b["dim"], b["vdim"]
+    c = [0, H2 * dk, 2 * H2 * dk, 2 * H2 * dk + H2 * dv, 2 * H2 * (dk + dv)]
+    _gemm(t, "gemm in (parallel)", M, lq + lk + lv + c[4], W)
+    _gemm(t, "gemm memory gates (fp32)", M, 2 * pad8(H2), W, True)
+    y, out, nw, bz = _bf(M, c[4]), _bf(M, H2 * dv), _bf(H2 * dv), _bf(2, H2)
+    z = torch.randn(M, 2 * pad8(H2), device=DEV)
+    z[:, pad8(H2):] += 4
+    S, nn, mm = torch.zeros(n, H2, dk, dv, device=DEV), torch.zeros(n, H2, dk, device=DEV), torch.zeros(n, H2, device=DEV)
+    flops = M * H2 * (2.0 * 64 * (dk + dv) / 2 + 4.0 * dk * dv)          # chunked form, 64-token chunks
+    state = n * H2 * (dk * dv + dk) * 4 * (1 if lengths else 2)
+    t("matrix_memory", lambda: ops.matrix_memory(*(y[:, c[i]:c[i + 1]] for i in range(4)), z[:, :H2], z[:, pad8(H2):pad8(H2) + H2], bz[0], bz[1], out,
+                                                 S, nn, mm, p, nw, dk, dv, 15.0, dk ** -0.5, 1.0, eps),
+      M * H2 * ((2 * dk + 3 * dv) * 2 + 8) + state, flops if lengths else 0)
+    _gemm(t, "gemm parallel o (fp32)", M, W, H * a["vdim"] + H2 * dv, True)
+
+    r = kinds["rglru"]
+    C, B = r["width"], r["blocks"]
+    _gemm(t, "gemm in (recurrence)", M, 2 * C, W)
+    y, taps, v, gb = _bf(M, 2 * C), _bf(C, r["conv"]), _bf(C), _bf(B, 2, C // B)
+    wg, lam, out = _bf(B, 2, C // B, C // B) * 0.1, torch.full((C,), -5.0, device=DEV, dtype=torch.bfloat16), _bf(M, C)
+    S, conv = torch.zeros(n, C, device=DEV), torch.zeros(n, C, r["conv"] - 1, device=DEV)
+    t("gated_recurrence", lambda: ops.gated_recurrence(y[:, :C], y[:, C:], v, v, taps, v, wg, gb, lam, out, S, conv, p),
+      M * C * 6 + wg.numel() * 2 + n * C * r["conv"] * 4 * 2, 4.0 * M * C * (C // B))
+    _gemm(t, "gemm recurrence o (fp32)", M, W, C, True)
+
+    f = next(l["mlp"] for l in mc.layers if l["mlp"]["kind"] == "moe")
+    ro, F, sh = f["router"], f["expert"]["ff"], f["shared"]["ff"]
+    E, top = ro["experts"], ro["top"]
+    _gemm(t, "gemm router (fp32)", M, pad8(E) + 8, W, True)
+    z, corr = torch.randn(M, pad8(E) + 8, device=DEV), _bf(E) * 0.1
+    t("route", lambda: ops.route(z, corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"]), M * (E * 4 + top * 12))
+    rt = ops.route(z, corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"])
+    w_in, w_out = _bf(E, 2, F, W), _bf(E, W, F)
+    used = int((rt.offsets[1:] > rt.offsets[:-1]).sum())
+    t("expert_glu", lambda: ops.expert_glu(h, w_in, rt), (used * 2 * F * W + M * W + M * top * F) * 2, 4.0 * M * top * F * W)
+    act = ops.expert_glu(h, w_in, rt)
+    t("expert_down", lambda: ops.expert_down(act, w_out, rt), (used * F * W + M * top * (F + W)) * 2, 2.0 * M * top * F * W)
+    rows, sg = ops.expert_down(act, w_out, rt), torch.randn(M, device=DEV)
+    t("moe_norm_add", lambda: ops.moe_norm_add(x, rows, rt, y32, sg, w, 0.5, W, eps), M * W * (14 + 2 * top))
+    _gemm(t, "gemm shared gate, up", M, 2 * sh, W)
+    gu, act = _bf(M, 2 * sh), _bf(M, sh)
+    t("glu", lambda: ops.glu(gu[:, :sh], gu[:, sh:], act), M * sh * 6)
+    _gemm(t, "gemm shared down (fp32)", M, W, sh, True)
+    d = mc.side_dim
+    _gemm(t, "gemm token gate", M, d, W)
+    gate, table, ids = _bf(M, d), _bf(V, 4 * d), torch.randint(0, V, (M,), device=DEV)
+    t("gelu_times_token", lambda: ops.gelu_times_token(gate, table, ids, d, V), M * d * 6)
+    _gemm(t, "gemm token projection (fp32)", M, W, d, True)
+    if lengths is None:
+        _gemm(t, "gemm logits (fp32)", M, V, W, True)
+    del t.flush
+    return t.rows
+
+
 def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
     """The same for the dense decoder family."""
     mc, t = PRESETS[preset], _Timer()
@@ -352,6 +438,6 @@ def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int =
 
 
 def kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
-    by_name = {"Fetelorn": fetelorn_kernels, "Sotazen": sotazen_kernels}
+    by_name = {"Fetelorn": fetelorn_kernels, "Sotazen": sotazen_kernels, "Ruburax": ruburax_kernels}
     with torch.no_grad():
         return by_name.get(getattr(PRESETS[preset], "architecture", None), dense_kernels)(preset, lengths, batch, ctx)

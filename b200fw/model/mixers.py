@@ -679,7 +679,5 @@ class GatedRecurrence(nn.Module):
             out_scale: float = 1.0) -> None:
         if out_scale != 1.0:
             raise ValueError("recurrence: its output takes no factor")
-        C, n = out.shape[1], pad8(self.size)
-        u = ops.causal_conv(y.cols("x"), self.x_bias.view(-1), self.taps.view(C, -1), self.conv_bias.view(-1), state["conv"], p)
-        z = ops.block_gates(u, self.w_gates.view(self.blocks, 2 * n, n))
-        ops.linear_recurrence(u, z, self.gate_bias.view(-1), self.lam.view(-1), y.cols("y"), self.y_bias.view(-1), out, state["S"], p, n)
+        ops.gated_recurrence(y.cols("y"), y.cols("x"), self.y_bias.view(-1), self.x_bias.view(-1), self.taps.view(out.shape[1], -1),
+                             self.conv_bias.view(-1), self.w_gates, self.gate_bias, self.lam.view(-1), out, state["S"], state["conv"], p)

@@ -86,3 +86,14 @@ def linear_recurrence(u: torch.Tensor, z: torch.Tensor, z_bias: torch.Tensor, la
             nv.ptr(out), cl(out.stride(0)), nv.ptr(state), nv.ptr(ws), nv.ptr(p.cu), nv.ptr(p.starts), nv.ptr(p.slots),
             nv.ptr(chunks), nv.ptr(p.first64 if n else None), n, lo, cnt, C, block, _f32(u), nv.stream_ptr()), "linear_recurrence")
         nv.count_launch(3 if n else 1)
+
+
+def gated_recurrence(y: torch.Tensor, x: torch.Tensor, y_bias: torch.Tensor, x_bias: torch.Tensor, taps: torch.Tensor,
+                     conv_bias: torch.Tensor, w_gates: torch.Tensor, gate_bias: torch.Tensor, lam: torch.Tensor, out: torch.Tensor,
+                     state: torch.Tensor, conv_state: torch.Tensor, p: Portions) -> None:
+    """Convolution, gates and recurrence of a step: ``x``, ``y`` and ``out [M, C]`` are column slices, ``w_gates [B, 2, np, np]`` and
+    ``gate_bias [B, 2, np]`` hold the recurrence gate, then the input gate of every block."""
+    B, _, n, _ = w_gates.shape
+    u = causal_conv(x, x_bias, taps, conv_bias, conv_state, p)
+    z = block_gates(u, w_gates.view(B, 2 * n, n))
+    linear_recurrence(u, z, gate_bias.view(-1), lam, y, y_bias, out, state, p, n)

@@ -184,9 +184,25 @@ def route(scores, correction, top, groups):
     return sorted(open_, key=lambda e: -float(c[e]))[:top]
 
 
-def moe(h, w, p, m):
+def margin(scores, correction, top, groups):
+    """How far the choice of one token is from another one: the smaller of the two gaps, between groups and between experts."""
+    c, gap = scores + correction, math.inf
+    per = c.numel() // groups["count"] if groups is not None else c.numel()
+    if groups is not None and groups["keep"] < groups["count"]:
+        g = sorted((sum(sorted(c[i:i + per].tolist(), reverse=True)[:2]) for i in range(0, c.numel(), per)), reverse=True)
+        gap = g[groups["keep"] - 1] - g[groups["keep"]]
+    picked = route(scores, correction, top, groups)
+    rest = set(route(scores, correction, c.numel(), groups)) - set(picked)
+    if rest:
+        gap = min(gap, min(float(c[e]) for e in picked) - max(float(c[e]) for e in rest))
+    return gap
+
+
+def moe(h, w, p, m, margins=None):
     r, out = m["router"], torch.zeros_like(h)
     s = sigmoid(h @ w[p + "router"].T)
+    if margins is not None:
+        margins.append(torch.tensor([margin(x, w[p + "correction"], r["top"], r.get("groups")) for x in s]))
     for t in range(h.shape[0]):
         for e in route(s[t], w[p + "correction"], r["top"], r.get("groups")):
             out[t] += s[t, e] * r["scale"] * glu(h[t], w, f"{p}e{e}.")
@@ -202,8 +218,9 @@ def token_input(x, w, p, tokens, i, dim, eps):
     return rms(y, eps) * w[p + "side.norm"]
 
 
-def forward(cfg, weights, tokens, layers_out=None):
-    """Logits ``[T, vocab]``; ``layers_out`` (a list) receives the residual stream after every layer."""
+def forward(cfg, weights, tokens, layers_out=None, margins=None):
+    """Logits ``[T, vocab]``; ``layers_out`` (a list) receives the residual stream after every layer, ``margins`` every expert
+    layer's margins of choice."""
     w = {n: t.to(F) for n, t in weights.items()}
     eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
     x, keys = w["embed"][torch.as_tensor(tokens)], {}
@@ -219,7 +236,7 @@ def forward(cfg, weights, tokens, layers_out=None):
             y = rglru_mixer(x, w, p + "mix.", m, eps)
         x = x + mult * rms(y, eps) * w[p + "norm1"]
         if layer["mlp"] is not None:
-            y = glu(x, w, p + "mlp.") if layer["mlp"]["kind"] == "dense" else moe(x, w, p + "mlp.", layer["mlp"])
+            y = glu(x, w, p + "mlp.") if layer["mlp"]["kind"] == "dense" else moe(x, w, p + "mlp.", layer["mlp"], margins)
             x = x + mult * rms(y, eps) * w[p + "norm2"]
         if cfg.get("token_side") is not None:
             x = x + mult * token_input(x, w, p, tokens, i, cfg["token_side"]["dim"], eps)
@@ -287,12 +304,16 @@ def random_weights(cfg, seed=0):
             r = 1.0 + 0.2 * r
         elif name.endswith("f.b"):
             r = 4.0 + r
-        elif last in ("b", "correction"):
+        elif last == "b":
             r = r * 0.5
+        elif last == "correction":
+            r = r * 1.2 - 1.0             # most choice scores are negative, and few choices are close
         elif last == "sink":
             r = 1.0 + r
         elif last == "lam":
             r = r - 4.0
+        elif last == "router":
+            r = r * shape[-1] ** -0.5 * 0.7
         elif name in ("embed", "side.embed"):
             r = r
         else:

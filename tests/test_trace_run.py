@@ -10,7 +10,9 @@ import pytest
 import torch
 
 import fetelorn_oracle as O
+import ruburax_oracle as RO
 import sotazen_oracle as SO
+import test_ruburax as R
 import test_sotazen as S
 from test_fetelorn import bf16_exact, build, config, parallel, retention, toks
 from b200fw.model import ModelConfig, ParallelTransformerModel, registry
@@ -19,7 +21,10 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CFG = config(36, 51, [parallel(2, 1, 16, 8, 20, 12, 2, 1, 16, 24, 5, ff=16), retention(2, 8, 16, 4, ff=16)])
 
 SOTAZEN = S.config(36, 51, [S.latent(2, 16, 8, 12, 24, ff=16), S.lightning(2, 8, 16, ff=None), S.differential(2, 1, 16, 8, 19, 4, ff=16)])
-MODELS = {"Fetelorn": (CFG, O, build), "Sotazen": (SOTAZEN, SO, S.build)}
+RUBURAX = R.config(36, 51, [R.rglru(24, 2, 3, ff=R.dense(16)), R.attention(2, 1, 16, 8, R.rot(8, 400.0, (4.0, 1.0, 2.0, 20))),
+                            R.parallel(R.att(2, 1, 8, 8, R.rot(8)), 2, 8, 12, 6.0, 0.7, 1.2, ff=R.moe(6, 2, 12, (3, 2), 8)),
+                            R.attention(4, 1, 16, 8, R.rot(8, 400.0, (4.0, 1.0, 2.0, 20)), kv_from=1, ff=R.dense(16))])
+MODELS = {"Fetelorn": (CFG, O, build), "Sotazen": (SOTAZEN, SO, S.build), "Ruburax": (RUBURAX, RO, R.build)}
 
 
 def replay(model_dir, out, steps, max_tokens, device, dtype="float32"):
