@@ -237,6 +237,18 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch
     for lo, cnt, longest in ((0, p.num_short, p.max_short), (p.num_short, p.nseq - p.num_short, p.max_long)):
         if cnt <= 0:
             continue
+        if lo == p.num_short and p.chunks128 is not None and q.dtype == torch.bfloat16 and dkp <= 128 and dvp <= 128:
+            nc = p.chunks128.shape[0]
+            ws = torch.empty((nc, H, dkp, dvp), device=q.device, dtype=torch.float32)
+            wn = torch.empty((nc, H, dkp), device=q.device, dtype=torch.float32)
+            wg = torch.empty((nc, H, 3), device=q.device, dtype=torch.float32).view(-1)      # (sum of f, largest g), then the maxima
+            nv.check(nv.lib().b2_memory_chunk(
+                nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(zi), nv.ptr(zf), cl(zi.stride(0)), nv.ptr(bi), nv.ptr(bf),
+                nv.ptr(norm_w), nv.ptr(out), nv.ptr(ws), nv.ptr(wn), nv.ptr(wg), nv.ptr(wg[2 * nc * H:]), nv.ptr(S), nv.ptr(n), nv.ptr(m),
+                nv.ptr(p.chunks128), nv.ptr(p.first128), nv.ptr(p.starts), nv.ptr(p.slots), nc, lo, cnt, H, dk, dkp, dv, dvp,
+                cl(q.stride(0)), cl(out.stride(0)), cf(cap), cf(q_scale), cf(out_scale), cf(eps), nv.stream_ptr()), "memory_chunk")
+            nv.count_launch(3)
+            continue
         cu, st, sl = _sub(p, lo)
         nv.check(nv.lib().b2_memory_serial(
             nv.ptr(q), nv.ptr(k), nv.ptr(v), nv.ptr(gate), nv.ptr(zi), nv.ptr(zf), cl(zi.stride(0)), nv.ptr(bi), nv.ptr(bf),

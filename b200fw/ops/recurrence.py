@@ -55,10 +55,10 @@ def block_gates(u: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 
 def linear_recurrence(u: torch.Tensor, z: torch.Tensor, z_bias: torch.Tensor, lam: torch.Tensor, y: torch.Tensor, y_bias: torch.Tensor,
-                      out: torch.Tensor, state: torch.Tensor, p: Portions, block: int) -> None:
+                      out: torch.Tensor, state: torch.Tensor, p: Portions, block: int, short_only: bool = False) -> None:
     """The recurrence over ``u [M, C]`` with gates ``r, i = sigmoid(z + z_bias)`` (``z`` as :func:`block_gates` gives it, ``z_bias``
     in its order, ``block`` = np) and ``out [M, C] = S gelu_tanh(y + y_bias)``; ``y`` and ``out`` are column slices.  ``state
-    [slots, C]`` fp32."""
+    [slots, C]`` fp32.  ``short_only``: the rows of the short portions alone (``z`` may end there)."""
     M, C = u.shape
     if not u.is_cuda:
         zz = (z + z_bias.float()).reshape(M, C // block, 2, block)
@@ -76,11 +76,11 @@ def linear_recurrence(u: torch.Tensor, z: torch.Tensor, z_bias: torch.Tensor, la
         return
     cl = nv.ctypes.c_longlong
     for lo, cnt in ((0, p.num_short), (p.num_short, p.nseq - p.num_short)):
-        if cnt <= 0:
+        if cnt <= 0 or (short_only and lo > 0):
             continue
         chunks = p.chunks64 if lo == p.num_short else None
         n = 0 if chunks is None else chunks.shape[0]
-        ws = torch.empty((n, 2, C), device=u.device, dtype=torch.float32) if n else None
+        ws = torch.empty((n, 2, 2, C), device=u.device, dtype=torch.float32) if n else None
         nv.check(nv.lib().b2_linear_recurrence(
             nv.ptr(u), cl(u.stride(0)), nv.ptr(z), cl(z.stride(0)), nv.ptr(z_bias), nv.ptr(lam), nv.ptr(y), cl(y.stride(0)), nv.ptr(y_bias),
             nv.ptr(out), cl(out.stride(0)), nv.ptr(state), nv.ptr(ws), nv.ptr(p.cu), nv.ptr(p.starts), nv.ptr(p.slots),
@@ -95,5 +95,17 @@ def gated_recurrence(y: torch.Tensor, x: torch.Tensor, y_bias: torch.Tensor, x_b
     ``gate_bias [B, 2, np]`` hold the recurrence gate, then the input gate of every block."""
     B, _, n, _ = w_gates.shape
     u = causal_conv(x, x_bias, taps, conv_bias, conv_state, p)
-    z = block_gates(u, w_gates.view(B, 2 * n, n))
-    linear_recurrence(u, z, gate_bias.view(-1), lam, y, y_bias, out, state, p, n)
+    tiled = u.is_cuda and u.dtype == torch.bfloat16 and p.nseq > p.num_short and n <= 256
+    if tiled:          # the long portions: gates inside the passes over them
+        ns, nc, cl = p.num_short, p.chunks64.shape[0], nv.ctypes.c_longlong
+        C = u.shape[1]
+        ws = torch.empty((nc, 2, 2, C), device=u.device, dtype=torch.float32)
+        nv.check(nv.lib().b2_gated_recurrence(
+            nv.ptr(u), nv.ptr(w_gates), nv.ptr(gate_bias), nv.ptr(lam), nv.ptr(y), cl(y.stride(0)), nv.ptr(y_bias), nv.ptr(out),
+            cl(out.stride(0)), nv.ptr(state), nv.ptr(ws), nv.ptr(p.starts), nv.ptr(p.slots), nv.ptr(p.chunks64), nv.ptr(p.first64), nc,
+            ns, p.nseq - ns, u.shape[0], C, n, nv.stream_ptr()), "gated_recurrence")
+        nv.count_launch(3)
+        if ns == 0:
+            return
+    z = block_gates(u[:p.short_rows] if tiled else u, w_gates.view(B, 2 * n, n))
+    linear_recurrence(u, z, gate_bias.view(-1), lam, y, y_bias, out, state, p, n, tiled)

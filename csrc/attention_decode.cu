@@ -646,6 +646,7 @@ B2_EXPORT int b2_decode_attention(const void* q, const void* kc, const void* vc,
   };
   const CUtensorMap *tk = map(kc, R), *tv = vc ? map(vc, C) : tk;
   if (!tk || !tv) return 2;
+  if (vc && R == 128 && C == 128) return launch_decode<1, 4, 1, true>(p, tk, tv, grid, st);
   if (vc) return R == 256 && C == 128 ? launch_decode<1, 8, 1, true>(p, tk, tv, grid, st) : launch_decode<1, 8, 1, false>(p, tk, tv, grid, st);
   return R == 576 && C == 512 ? launch_decode<2, 9, 4, true>(p, tk, tv, grid, st) : launch_decode<2, 9, 4, false>(p, tk, tv, grid, st);
 }

@@ -226,12 +226,11 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 }
 
 constexpr int MG_BM = 128, MG_BK = 64;
-constexpr int MG_LAG = 2;                  // k-blocks whose gathered rows may still be on their way
-
 template <int BN>
 struct MoeCfg {
   static constexpr int A_BYTES = MG_BM * MG_BK * 2, B_BYTES = BN * MG_BK * 2, STAGE = A_BYTES + B_BYTES;
   static constexpr int STAGES = BN == 256 ? 4 : BN == 128 ? 6 : 8;
+  static constexpr int LAG = STAGES - 2;       // k-blocks whose gathered rows may still be on their way (below STAGES)
   static constexpr int STAGING = 4 * 4096;                        // a block per epilogue warp
   static constexpr int TABLES = 2 * (MOE_MAX_EXPERTS + 1) * 4;
   static constexpr int SMEM = STAGES * STAGE + STAGING + 256 + TABLES + 1024;
@@ -252,7 +251,6 @@ __global__ void __launch_bounds__(GLU ? 320 : 192, 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const MoeGemmParams p, int* status) {
   using Cfg = MoeCfg<BN>;
   constexpr int STAGES = Cfg::STAGES, COLS = GLU ? BN / 2 : BN;    // output columns of a tile
-  static_assert(MG_LAG < STAGES, "a stage is handed over before it is needed again");
   extern __shared__ uint8_t mg_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(mg_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   uint8_t* staging = smem + STAGES * Cfg::STAGE;
@@ -350,7 +348,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
     }
   } else if (GLU && warp >= 6) {
     // Token rows into the swizzled A tile: eight lanes a row (whole 128-byte lines), rows 32 w .. 32 w + 31 of warp w.  A stage is
-    // handed over MG_LAG k-blocks after its copies were issued, once they have landed and are visible to the tensor core.
+    // handed over LAG k-blocks after its copies were issued, once they have landed and are visible to the tensor core.
     const int w = warp - 6, chunk = lane & 7, sub = lane >> 3;
     int st = 0, done = 0;            // stages issued into, handed over
     uint32_t ph = 0;
@@ -391,8 +389,8 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
           st = 0;
           ph ^= 1;
         }
-        if (pending > MG_LAG) {
-          asm volatile("cp.async.wait_group %0;" ::"n"(MG_LAG) : "memory");
+        if (pending > Cfg::LAG) {
+          asm volatile("cp.async.wait_group %0;" ::"n"(Cfg::LAG) : "memory");
           hand_over();
         }
       }
@@ -494,8 +492,8 @@ __device__ __forceinline__ float moe_block_sum(float v, float* scratch) {
   return warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? scratch[lane] : 0.f);
 }
 
-template <typename T, int V>
-__global__ void __launch_bounds__(1024) moe_norm_add_kernel(const MoeAddParams p) {
+template <typename T, int V, int MAXT>
+__global__ void __launch_bounds__(MAXT) moe_norm_add_kernel(const MoeAddParams p) {
   __shared__ float scratch[32], sw[MOE_MAX_TOP];
   __shared__ int sr[MOE_MAX_TOP];
   const size_t base = static_cast<size_t>(blockIdx.x) * p.ld;
@@ -575,13 +573,20 @@ static int launch_moe(const CUtensorMap* ta, const CUtensorMap* tb, const MoeGem
 
 static int moe_bound(int P, int E, int tile) { return P / tile + (E < P ? E : P); }    // row tiles at most
 
-// Column tile: the widest that still gives every SM a few tiles, by the expected number of row tiles.
-static int moe_columns(int P, int E, int N, int widest) {
+// Column tile: the one whose last wave wastes least, by the expected number of row tiles; a tile costs its columns and a fixed part.
+static int moe_columns(int P, int E, int N, int widest, int narrowest) {
   const int used = E < P ? E : P;
   const long long rows = static_cast<long long>(used) * ((P / used + MG_BM - 1) / MG_BM);
-  int cols = widest;
-  while (cols > 32 && rows * ((N + cols - 1) / cols) < 4 * num_sms()) cols /= 2;
-  return cols;
+  int best = widest;
+  long long least = -1;
+  for (int cols = widest; cols >= narrowest; cols /= 2) {
+    const long long tiles = rows * ((N + cols - 1) / cols), cost = (tiles + num_sms() - 1) / num_sms() * (cols + 32);
+    if (least < 0 || cost < least) {
+      least = cost;
+      best = cols;
+    }
+  }
+  return best;
 }
 
 }  // namespace b2
@@ -627,7 +632,7 @@ B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* 
     B2_CHECK_LAUNCH("moe_glu");
     return 0;
   }
-  const int cols = moe_columns(P, E, F, 128);
+  const int cols = moe_columns(P, E, F, 128, 32);
   const uint64_t dims[3] = {static_cast<uint64_t>(K), static_cast<uint64_t>(F), 2ull * E},
                  strides[2] = {2ull * K, 2ull * F * K};
   const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
@@ -658,8 +663,7 @@ B2_EXPORT int b2_moe_down(const void* a, const void* w, const int* offsets, void
     B2_CHECK_LAUNCH("moe_down");
     return 0;
   }
-  int cols = moe_columns(P, E, N, 256);
-  if (cols < 64) cols = 64;
+  const int cols = moe_columns(P, E, N, 256, 64);
   const uint64_t dims[3] = {static_cast<uint64_t>(F), static_cast<uint64_t>(N), static_cast<uint64_t>(E)},
                  strides[2] = {2ull * F, 2ull * N * F};
   const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
@@ -686,9 +690,10 @@ B2_EXPORT int b2_moe_norm_add(float* x, const void* rows, const int* place, cons
   const int threads = ((pieces + V - 1) / V + 31) / 32 * 32;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   B2_DISPATCH_T(is_f32, {
-    if (V == 1) moe_norm_add_kernel<T, 1><<<M, threads, 0, st>>>(p);
-    else if (V == 2) moe_norm_add_kernel<T, 2><<<M, threads, 0, st>>>(p);
-    else moe_norm_add_kernel<T, 4><<<M, threads, 0, st>>>(p);
+    if (V == 1) moe_norm_add_kernel<T, 1, 256><<<M, threads, 0, st>>>(p);
+    else if (V == 2) moe_norm_add_kernel<T, 2, 256><<<M, threads, 0, st>>>(p);
+    else if (threads <= 256) moe_norm_add_kernel<T, 4, 256><<<M, threads, 0, st>>>(p);
+    else moe_norm_add_kernel<T, 4, 1024><<<M, threads, 0, st>>>(p);
   });
   B2_CHECK_LAUNCH("moe_norm_add");
   return 0;

@@ -5,8 +5,10 @@
 //   log a = -8 r softplus(lam);   S <- a S + sqrt(1 - a^2) i u;   out = S gelu(y + yb)
 //
 // States are fp32 per sequence slot; start == 0 means that they are zero, whatever the slot holds.  Short portions are walked token by
-// token.  Long ones are cut into chunks of 64 tokens: every chunk's own transfer (product of the decays, state from zero), the states
-// at the chunks' starts, then the chunks once more from there.
+// token.  Long ones are cut into runs of 32 tokens: every run's own transfer (product of the decays, state from zero), the states
+// at the runs' starts, then the runs once more from there.  In bf16 the gates of both passes are tcgen05 products inside the pass
+// (rec_gates_kernel): the accumulators have a channel per TMEM lane and a token per column, so that a thread finds the gates of its
+// channel's tokens in its own lane and the recurrence never leaves registers; gates are made twice instead of stored.
 #include "host.h"
 #include "vec.cuh"
 
@@ -31,21 +33,24 @@ struct ConvParams {
   int C, K;
 };
 
-// Grid (tiles, channels / (8 * threads)), eight channels a thread.  Only the portion's first tile reads the state, so that tile also
-// replaces it, after its own reads.
-template <typename T>
+// Grid (tiles, channels / 256): 32 groups of eight channels times four groups of four rows.  Only the portion's first tile reads the
+// state, so that tile also replaces it, after its own reads.  KT: taps known to the compiler (0: any number).
+constexpr int GR_ROWS = GR_TILE / 4;
+template <typename T, int KT>
 __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParams p) {
   const int* tl = p.tiles + blockIdx.x * 4;
-  const int s = tl[0], row0 = tl[1], rows = tl[2], off = tl[3], c = (blockIdx.y * GR_THREADS + threadIdx.x) * 8, K = p.K;
+  const int s = tl[0], row0 = tl[1], rows = tl[2], off = tl[3], K = KT > 0 ? KT : p.K;
+  const int c = (blockIdx.y * 32 + (threadIdx.x & 31)) * 8, t0 = (threadIdx.x >> 5) * GR_ROWS;
   const int slot = s < 0 ? -1 : p.slot[s];
-  if (slot < 0 || rows <= 0 || c >= p.C) return;
-  const bool fresh = p.start[s] == 0;
-  const T* x = static_cast<const T*>(p.x) + c;
-  const T* taps = static_cast<const T*>(p.taps) + static_cast<size_t>(c) * K;
-  float* st = p.state + (static_cast<size_t>(slot) * p.C + c) * (K - 1);
+  if (slot < 0 || rows <= 0) return;
+  const bool fresh = p.start[s] == 0, in = c < p.C;
+  const int cc = in ? c : 0;
+  const T* x = static_cast<const T*>(p.x) + cc;
+  const T* taps = static_cast<const T*>(p.taps) + static_cast<size_t>(cc) * K;
+  float* st = p.state + (static_cast<size_t>(slot) * p.C + cc) * (K - 1);
   float xb[8], cb[8];
-  vload8(static_cast<const T*>(p.xb) + c, xb);
-  vload8(static_cast<const T*>(p.cb) + c, cb);
+  vload8(static_cast<const T*>(p.xb) + cc, xb);
+  vload8(static_cast<const T*>(p.cb) + cc, cb);
   auto input = [&](int at, float (&f)[8]) {          // input at index `at` of the portion
     if (at >= 0) {
       vload8(x + (static_cast<size_t>(row0) + at - off) * p.ld, f);
@@ -56,19 +61,54 @@ __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParam
       for (int e = 0; e < 8; ++e) f[e] = fresh ? 0.f : st[e * (K - 1) + K - 1 + at];
     }
   };
-  for (int t = 0; t < rows; ++t) {
-    float acc[8];
+  if (in && t0 < rows) {
+    float acc[GR_ROWS][8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = cb[e];
-    for (int j = 0; j < K; ++j) {
-      float f[8];
-      input(off + t - j, f);
+    for (int i = 0; i < GR_ROWS; ++i)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = fmaf(to_f(taps[e * K + K - 1 - j]), f[e], acc[e]);
+      for (int e = 0; e < 8; ++e) acc[i][e] = cb[e];
+    if constexpr (KT > 0) {
+      float w[KT * 8];                               // a channel's taps are neighbours
+#pragma unroll
+      for (int i = 0; i < KT; ++i) {
+        float f[8];
+        vload8(taps + i * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[i * 8 + e] = f[e];
+      }
+      const int last = rows - 1;
+#pragma unroll
+      for (int i = -(KT - 1); i < GR_ROWS; ++i) {    // each input once, into the outputs that see it
+        float f[8];
+        input(off + min(t0 + i, last), f);
+#pragma unroll
+        for (int o = 0; o < GR_ROWS; ++o)
+          if (o - i >= 0 && o - i < KT)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc[o][e] = fmaf(w[e * KT + KT - 1 - (o - i)], f[e], acc[o][e]);
+      }
+    } else {
+      for (int j = 0; j < K; ++j) {
+        float w[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[e] = to_f(taps[e * K + K - 1 - j]);
+#pragma unroll
+        for (int i = 0; i < GR_ROWS; ++i) {
+          if (t0 + i >= rows) break;
+          float f[8];
+          input(off + t0 + i - j, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(w[e], f[e], acc[i][e]);
+        }
+      }
     }
-    vstore8(static_cast<T*>(p.u) + (static_cast<size_t>(row0) + t) * p.C + c, acc);
+#pragma unroll
+    for (int i = 0; i < GR_ROWS; ++i)
+      if (t0 + i < rows) vstore8(static_cast<T*>(p.u) + (static_cast<size_t>(row0) + t0 + i) * p.C + c, acc[i]);
   }
   if (off != 0 || K < 2) return;
+  __syncthreads();
+  if (!in || threadIdx.x >= 32) return;
   const int count = p.cu[s + 1] - p.cu[s];
   for (int j = 0; j < K - 1; ++j) {                  // in this order an old input is read before its place is written
     float f[8];
@@ -87,11 +127,11 @@ struct RecParams {
   const void* yb;        // T [C]
   void* out;             // T [M, ld_out]
   float* state;          // [slots, C]
-  float* ws;             // [chunks, 2, C]: transfer (product, end state), then [.., 0, ..] the state at the chunk's start
+  float* ws;             // [runs, 2, C]: transfer (product, end state), then [.., 0, ..] the state at the run's start
   const int* cu;
   const int* start;
   const int* slot;
-  const int* chunks;     // [n, 4]
+  const int* chunks;     // [n, 4], two runs each
   const int* first;      // [nlong + 1]
   long long ld_u, ld_z, ld_y, ld_out;
   int C, block, seq0;
@@ -143,16 +183,21 @@ struct RecChannel {
   }
 };
 
+constexpr int GR_RUN = 32;
+
+// Rows of run h (0, 1) of a chunk.
+__device__ __forceinline__ int run_rows(int rows, int h) { return max(0, min(GR_RUN, rows - h * GR_RUN)); }
+
 template <typename T>
 __global__ void __launch_bounds__(GR_THREADS) rec_transfer_kernel(const RecParams p) {
-  const int* ch = p.chunks + blockIdx.x * 4;
-  const int c = blockIdx.y * GR_THREADS + threadIdx.x;
+  const int* ch = p.chunks + (blockIdx.x >> 1) * 4;
+  const int c = blockIdx.y * GR_THREADS + threadIdx.x, h = blockIdx.x & 1, n = run_rows(ch[2], h);
   if (c >= p.C || p.slot[ch[0]] < 0) return;
   const RecChannel<T> k(p, c);
   float A = 1.f, S = 0.f;
 #pragma unroll 4
-  for (int t = 0; t < ch[2]; ++t) {
-    const float2 g = k.step(p, static_cast<size_t>(ch[1]) + t);
+  for (int t = 0; t < n; ++t) {
+    const float2 g = k.step(p, static_cast<size_t>(ch[1]) + h * GR_RUN + t);
     A *= g.x;
     S = fmaf(g.x, S, g.y);
   }
@@ -168,8 +213,8 @@ __global__ void __launch_bounds__(GR_THREADS) rec_carry_kernel(const RecParams p
   if (c >= p.C || slot < 0) return;
   float* st = p.state + static_cast<size_t>(slot) * p.C + c;
   float S = p.start[s] == 0 ? 0.f : *st;
-  const int c0 = p.first[blockIdx.y], c1 = p.first[blockIdx.y + 1];
-  constexpr int U = 8;
+  const int c0 = p.first[blockIdx.y] * 2, c1 = p.first[blockIdx.y + 1] * 2;
+  constexpr int U = 16;
   for (int i = c0; i < c1; i += U) {
     float A[U], B[U];
 #pragma unroll
@@ -188,17 +233,18 @@ __global__ void __launch_bounds__(GR_THREADS) rec_carry_kernel(const RecParams p
   *st = S;
 }
 
-// CHUNKS: grid (chunks, channels), from the states rec_carry left; else grid (sequences, channels), from the slots and back to them.
-template <typename T, bool CHUNKS>
+// RUNS: grid (runs, channels), from the states rec_carry left; else grid (sequences, channels), from the slots and back to them.
+template <typename T, bool RUNS>
 __global__ void __launch_bounds__(GR_THREADS) rec_out_kernel(const RecParams p) {
   const int c = blockIdx.y * GR_THREADS + threadIdx.x;
-  const int s = CHUNKS ? p.chunks[blockIdx.x * 4] : p.seq0 + static_cast<int>(blockIdx.x);
+  const int* ch = RUNS ? p.chunks + (blockIdx.x >> 1) * 4 : nullptr;
+  const int s = RUNS ? ch[0] : p.seq0 + static_cast<int>(blockIdx.x);
   const int slot = p.slot[s];
   if (c >= p.C || slot < 0) return;
-  const size_t row0 = CHUNKS ? p.chunks[blockIdx.x * 4 + 1] : p.cu[s];
-  const int rows = CHUNKS ? p.chunks[blockIdx.x * 4 + 2] : p.cu[s + 1] - p.cu[s];
+  const size_t row0 = RUNS ? ch[1] + (blockIdx.x & 1) * GR_RUN : p.cu[s];
+  const int rows = RUNS ? run_rows(ch[2], blockIdx.x & 1) : p.cu[s + 1] - p.cu[s];
   float* st = p.state + static_cast<size_t>(slot) * p.C + c;
-  float S = CHUNKS ? p.ws[static_cast<size_t>(blockIdx.x) * 2 * p.C + c] : p.start[s] == 0 ? 0.f : *st;
+  float S = RUNS ? p.ws[static_cast<size_t>(blockIdx.x) * 2 * p.C + c] : p.start[s] == 0 ? 0.f : *st;
   const RecChannel<T> k(p, c);
 #pragma unroll 4
   for (int t = 0; t < rows; ++t) {
@@ -208,7 +254,186 @@ __global__ void __launch_bounds__(GR_THREADS) rec_out_kernel(const RecParams p) 
     S = fmaf(g.x, S, g.y);
     static_cast<T*>(p.out)[row * p.ld_out + c] = from_f<T>(S * y);
   }
-  if (!CHUNKS) *st = S;
+  if (!RUNS) *st = S;
+}
+
+// ---- both passes with their gates on the tensor cores ---------------------------------------------------------------------------
+// A CTA keeps the two gates' weights of 128 channels of a block in shared memory (they read all of the block's channels of u) and
+// walks chunks of 64 tokens: u arrives by TMA one chunk ahead, the products of the next chunk run under the recurrence of this one.
+// Warps 0..3 have the chunk's first run, warps 4..7 the second; thread = channel.
+constexpr int RG_THREADS = 256;
+constexpr int RG_MAX_BLOCK = 256;
+typedef __nv_bfloat16 rg_bf16;
+
+struct RecGateSmem {
+  int kc, weights, stage, total;       // 64-channel pieces of a block; bytes
+  __host__ __device__ explicit RecGateSmem(int block) {
+    kc = (block + 63) / 64;
+    weights = 2 * kc * 128 * 128;
+    stage = kc * 64 * 128;
+    total = weights + 2 * stage + 64 + 1024;
+  }
+};
+
+__device__ __forceinline__ float sqrt_fast(float x) {
+  float y;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <bool OUT>
+__global__ void __launch_bounds__(RG_THREADS) rec_gates_kernel(const __grid_constant__ CUtensorMap tmU, const __grid_constant__ CUtensorMap tmW,
+                                                               const RecParams p, int nchunks, int tiles_per_block, int* status) {
+  extern __shared__ uint8_t rg_raw[];
+  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(rg_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const RecGateSmem L(p.block);
+  uint8_t* su = sm + L.weights;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(su + 2 * L.stage);
+  uint64_t *w_full = bars, *u_full = bars + 1, *done = bars + 3;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quarter = warp & 3, run = warp >> 2;
+  const int b = blockIdx.x / tiles_per_block, ct = blockIdx.x % tiles_per_block;
+  if (tid == 0) {
+    for (int i = 0; i < 5; ++i) mbar_init(bars + i, 1);
+    mbar_fence_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(tmem_slot, 256);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
+  const int stride = gridDim.y;
+  auto load_u = [&](int chunk, int st) {            // one thread
+    mbar_expect_tx(u_full + st, L.stage);
+    const int row = p.chunks[chunk * 4 + 1];
+    for (int k = 0; k < L.kc; ++k) tma_load_2d(su + st * L.stage + k * 8192, &tmU, u_full + st, b * p.block + k * 64, row);
+  };
+  if (tid == 0) {
+    mbar_expect_tx(w_full, L.weights);
+    for (int g = 0; g < 2; ++g)
+      for (int k = 0; k < L.kc; ++k) tma_load_3d(sm + (g * L.kc + k) * 16384, &tmW, w_full, k * 64, ct * 128, 2 * b + g);
+    for (int i = 0; i < 2; ++i)
+      if (static_cast<int>(blockIdx.y) + i * stride < nchunks) load_u(blockIdx.y + i * stride, i);
+  }
+  const bool leader = warp == 0 && elect_one();
+  // gates of the chunk in stage st: columns 0..63 of its accumulators the recurrence gate, 64..127 the input gate
+  auto products = [&](int st, uint32_t ph) {        // warp 0
+    mbar_wait_warp(u_full + st, ph, status, ERR_GEMM_MMA_WAIT_FULL);
+    tc_fence_after();
+    if (leader) {
+      constexpr uint32_t idesc = make_idesc_f16(1, 128, 64, 0, 0);
+      for (int g = 0; g < 2; ++g)
+        for (int k = 0; k < L.kc; ++k) {
+          const uint64_t da = make_smem_desc_sw128(smem_u32(sm + (g * L.kc + k) * 16384), 16, 1024),
+                         db = make_smem_desc_sw128(smem_u32(su + st * L.stage + k * 8192), 16, 1024);
+#pragma unroll
+          for (int ks = 0; ks < 4; ++ks)
+            umma_f16_ss(tmem + st * 128 + g * 64, desc_advance(da, ks * 32), desc_advance(db, ks * 32), idesc, k > 0 || ks > 0 ? 1u : 0u);
+        }
+      umma_commit(done + st);
+    }
+    __syncwarp();
+  };
+  if (warp == 0) {
+    mbar_wait_warp(w_full, 0, status, ERR_GEMM_MMA_WAIT_FULL);
+    if (static_cast<int>(blockIdx.y) < nchunks) products(0, 0);
+  }
+  const int c = ct * 128 + quarter * 32 + lane;     // in the block
+  const bool in = c < p.block;
+  const int ch = b * p.block + (in ? c : 0);
+  const RecChannel<rg_bf16> K(p, ch);
+  const uint32_t at = tmem + (static_cast<uint32_t>(quarter * 32) << 16) + run * GR_RUN;
+  const int u_at = (c >> 6) * 8192 + (c & 7) * 2, u_piece = (c >> 3) & 7;
+  int it = 0;
+  for (int chunk = blockIdx.y; chunk < nchunks; chunk += stride, ++it) {
+    const int st = it & 1;
+    const uint32_t ph = (it >> 1) & 1;
+    if (warp == 0 && chunk + stride < nchunks) products(st ^ 1, ((it + 1) >> 1) & 1);
+    const int* cd = p.chunks + chunk * 4;
+    const size_t row0 = cd[1] + run * GR_RUN;
+    const int n = run_rows(cd[2], run);
+    const size_t wi = (static_cast<size_t>(chunk) * 2 + run) * 2 * p.C + ch;
+    float A = 1.f, S = 0.f;
+    if (OUT) S = p.ws[wi];
+    mbar_wait_warp(u_full + st, ph, status, ERR_GEMM_MMA_WAIT_FULL);       // u itself is read below
+    mbar_wait_warp(done + st, ph, status, ERR_GEMM_EPI_WAIT);
+    tc_fence_after();
+    const uint8_t* ut = su + st * L.stage + u_at;
+#pragma unroll 1
+    for (int t0 = 0; t0 < GR_RUN; t0 += 16) {
+      if (t0 >= n) break;                           // the same for the whole warp
+      uint32_t zr[16], zi[16];
+      float y[16];
+      if (OUT) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+          y[i] = __bfloat162float(static_cast<const rg_bf16*>(p.y)[(row0 + min(t0 + i, n - 1)) * p.ld_y + ch]);
+      }
+      tmem_ld_32x32b_x16(at + st * 128 + t0, zr);
+      tmem_ld_32x32b_x16(at + st * 128 + 64 + t0, zi);
+      tmem_ld_wait();
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const int t = run * GR_RUN + t0 + i;
+        const float u = __bfloat162float(*reinterpret_cast<const rg_bf16*>(ut + t * 128 + ((u_piece ^ (t & 7)) << 4)));
+        const float x = -K.sp * sigmoid_fast(__uint_as_float(zr[i]) + K.br);
+        const float a = fast_exp2(1.4426950408889634f * x);
+        const float inc = sqrt_fast(one_minus_exp(2.f * x, a * a)) * sigmoid_fast(__uint_as_float(zi[i]) + K.bi) * u;
+        if (t0 + i < n) {
+          S = fmaf(a, S, inc);
+          if (!OUT) A *= a;
+          if (OUT && in)
+            static_cast<rg_bf16*>(p.out)[(row0 + t0 + i) * p.ld_out + ch] = __float2bfloat16(S * gelu_tanh_t<rg_bf16>(y[i] + K.yb));
+        }
+      }
+    }
+    if (!OUT && in) {
+      p.ws[wi] = A;
+      p.ws[wi + p.C] = S;
+    }
+    tc_fence_before();
+    __syncthreads();                                // the stage and its accumulators have been read
+    tc_fence_after();
+    if (tid == 0 && chunk + 2 * stride < nchunks) load_u(chunk + 2 * stride, st);
+  }
+  if (*reinterpret_cast<volatile int*>(status) != 0) {     // copies and products in flight land before shared memory and TMEM go away
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 256);
+  }
+}
+
+template <bool OUT>
+static int launch_gates(const CUtensorMap* tu, const CUtensorMap* tw, const RecParams& p, int nchunks, cudaStream_t stream) {
+  auto kern = rec_gates_kernel<OUT>;
+  int* status = status_ptr();
+  if (!status) return 3;
+  const RecGateSmem L(p.block);
+  static int set[64] = {0};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (set[dev & 63] < L.total) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total) != cudaSuccess) {
+      set_error("rec_gates: cannot set shared memory size (%d)", L.total);
+      return 1;
+    }
+    set[dev & 63] = L.total;
+  }
+  const int per = (p.block + 127) / 128, x = p.C / p.block * per, resident = num_sms() * (L.total <= 112 * 1024 ? 2 : 1);
+  int y = resident / x;
+  if (y < 1) y = 1;
+  if (y > nchunks) y = nchunks;
+  kern<<<dim3(x, y), RG_THREADS, L.total, stream>>>(*tu, *tw, p, nchunks, per, status);
+  B2_CHECK_LAUNCH("rec_gates");
+  return 0;
 }
 
 }  // namespace b2
@@ -225,13 +450,18 @@ B2_EXPORT int b2_causal_conv(const void* x, long long ld, const void* xb, const 
     return 10;
   }
   const ConvParams p = {x, ld, xb, taps, cb, state, u, cu, start, slot, tiles, C, K};
-  const dim3 grid(ntiles, (C / 8 + GR_THREADS - 1) / GR_THREADS);
-  B2_DISPATCH_T(is_f32, causal_conv_kernel<T><<<grid, GR_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(p););
+  const dim3 grid(ntiles, (C / 8 + 31) / 32);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (K == 4) {
+    B2_DISPATCH_T(is_f32, (causal_conv_kernel<T, 4><<<grid, GR_THREADS, 0, st>>>(p)););
+  } else {
+    B2_DISPATCH_T(is_f32, (causal_conv_kernel<T, 0><<<grid, GR_THREADS, 0, st>>>(p)););
+  }
   B2_CHECK_LAUNCH("causal_conv");
   return 0;
 }
 
-// Sequences seq0 .. seq0 + nseq - 1; nchunks > 0: they are long, chunks / first describe them and ws is fp32 [nchunks, 2, C].
+// Sequences seq0 .. seq0 + nseq - 1; nchunks > 0: they are long, chunks / first describe them and ws is fp32 [nchunks, 2, 2, C].
 B2_EXPORT int b2_linear_recurrence(const void* u, long long ld_u, const float* z, long long ld_z, const void* zb, const void* lam,
                                    const void* y, long long ld_y, const void* yb, void* out, long long ld_out, float* state, float* ws,
                                    const int* cu, const int* start, const int* slot, const int* chunks, const int* first, int nchunks,
@@ -246,14 +476,38 @@ B2_EXPORT int b2_linear_recurrence(const void* u, long long ld_u, const float* z
   const int cy = (C + GR_THREADS - 1) / GR_THREADS;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (nchunks > 0) {
-    B2_DISPATCH_T(is_f32, rec_transfer_kernel<T><<<dim3(nchunks, cy), GR_THREADS, 0, st>>>(p););
+    B2_DISPATCH_T(is_f32, rec_transfer_kernel<T><<<dim3(2 * nchunks, cy), GR_THREADS, 0, st>>>(p););
     B2_CHECK_LAUNCH("rec_transfer");
     rec_carry_kernel<<<dim3(cy, nseq), GR_THREADS, 0, st>>>(p);
     B2_CHECK_LAUNCH("rec_carry");
-    B2_DISPATCH_T(is_f32, (rec_out_kernel<T, true><<<dim3(nchunks, cy), GR_THREADS, 0, st>>>(p)););
+    B2_DISPATCH_T(is_f32, (rec_out_kernel<T, true><<<dim3(2 * nchunks, cy), GR_THREADS, 0, st>>>(p)););
   } else {
     B2_DISPATCH_T(is_f32, (rec_out_kernel<T, false><<<dim3(nseq, cy), GR_THREADS, 0, st>>>(p)););
   }
   B2_CHECK_LAUNCH("linear_recurrence");
   return 0;
+}
+
+// Long sequences in bf16 with the gates' products inside: u [M, C] contiguous, w [C / block, 2, block, block], blocks up to 256
+// channels in multiples of 8; ws as above.
+B2_EXPORT int b2_gated_recurrence(const void* u, const void* w, const void* zb, const void* lam, const void* y, long long ld_y,
+                                  const void* yb, void* out, long long ld_out, float* state, float* ws, const int* start, const int* slot,
+                                  const int* chunks, const int* first, int nchunks, int seq0, int nseq, int M, int C, int block,
+                                  void* stream) {
+  b2::ensure_thread_context();
+  if (nseq <= 0 || nchunks <= 0) return 0;
+  if (block < 8 || block % 8 || block > RG_MAX_BLOCK || C < block || C % block || nseq > 65535) {
+    set_error("gated_recurrence: blocks up to %d channels in multiples of 8 required", RG_MAX_BLOCK);
+    return 10;
+  }
+  const RecParams p = {u, nullptr, zb, lam, y, yb, out, state, ws, nullptr, start, slot, chunks, first, C, 0, ld_y, ld_out, C, block, seq0};
+  const uint64_t n = block, dims[3] = {n, n, 2ull * (C / block)}, strides[2] = {2 * n, 2 * n * n};
+  const uint32_t box[3] = {64, 128, 1};
+  const CUtensorMap *tw = tensor_map_nd_bf16(w, 3, dims, strides, box, 3), *tu = tensor_map_2d_bf16(u, M, C, C, 64, 64);
+  if (!tw || !tu) return 2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (const int rc = launch_gates<false>(tu, tw, p, nchunks, st)) return rc;
+  rec_carry_kernel<<<dim3((C + GR_THREADS - 1) / GR_THREADS, nseq), GR_THREADS, 0, st>>>(p);
+  B2_CHECK_LAUNCH("rec_carry");
+  return launch_gates<true>(tu, tw, p, nchunks, st);
 }

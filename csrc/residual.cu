@@ -184,8 +184,8 @@ __global__ void __launch_bounds__(RES_THREADS) merge_norm_add_kernel(float* __re
 
 // x += coef * rms(f y) * w, and the new x rounded to T in h (optional).  y: fp32 [M, ld].  A row's pieces (V per thread) stay in
 // registers; both rows are requested before the first is used.
-template <typename T, int V>
-__global__ void __launch_bounds__(1024) norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const T* __restrict__ w,
+template <typename T, int V, int MAXT>
+__global__ void __launch_bounds__(MAXT) norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const T* __restrict__ w,
                                                         T* __restrict__ h, int ld, int n, float coef, float eps, float f) {
   __shared__ float scratch[32];
   const size_t base = static_cast<size_t>(blockIdx.x) * ld;
@@ -369,9 +369,10 @@ B2_EXPORT int b2_norm_add(float* x, const float* y, const void* w, void* h, int 
   B2_DISPATCH_T(is_f32, {
     const T* wt = static_cast<const T*>(w);
     T* ht = static_cast<T*>(h);
-    if (V == 1) norm_add_kernel<T, 1><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
-    else if (V == 2) norm_add_kernel<T, 2><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
-    else norm_add_kernel<T, 4><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+    if (V == 1) norm_add_kernel<T, 1, 256><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+    else if (V == 2) norm_add_kernel<T, 2, 256><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+    else if (threads <= 256) norm_add_kernel<T, 4, 256><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
+    else norm_add_kernel<T, 4, 1024><<<M, threads, 0, st>>>(x, y, wt, ht, ld, n, coef, eps, y_scale);
   });
   B2_CHECK_LAUNCH("norm_add");
   return 0;
