@@ -345,7 +345,8 @@ def ruburax_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     H2, dk, dv = b["heads"], b["dim"], b["vdim"]
     c = [0, H2 * dk, 2 * H2 * dk, 2 * H2 * dk + H2 * dv, 2 * H2 * (dk + dv)]
     _gemm(t, "gemm in (parallel)", M, lq + lk + lv + c[4], W)
-    _gemm(t, "gemm memory gates (fp32)", M, 2 * pad8(H2), W, True)
+    wz = _bf(2 * pad8(H2), W)
+    t("memory gates (fp32 product)", lambda: ops.linear_fp32(h, wz), (M * W + wz.numel()) * 2 + M * wz.shape[0] * 4)
     y, out, nw, bz = _bf(M, c[4]), _bf(M, H2 * dv), _bf(H2 * dv), _bf(2, H2)
     z = torch.randn(M, 2 * pad8(H2), device=DEV)
     z[:, pad8(H2):] += 4
@@ -370,10 +371,12 @@ def ruburax_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     f = next(l["mlp"] for l in mc.layers if l["mlp"]["kind"] == "moe")
     ro, F, sh = f["router"], f["expert"]["ff"], f["shared"]["ff"]
     E, top = ro["experts"], ro["top"]
-    _gemm(t, "gemm router (fp32)", M, pad8(E) + 8, W, True)
-    z, corr = torch.randn(M, pad8(E) + 8, device=DEV), _bf(E) * 0.1
-    t("route", lambda: ops.route(z, corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"]), M * (E * 4 + top * 12))
-    rt = ops.route(z, corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"])
+    wr, corr = _bf(pad8(E) + 8, W) * 0.05, _bf(E) * 0.1
+
+    def route():
+        return ops.router(h, wr, pad8(E), corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"])
+    t("router", route, M * (W * 2 + top * 12) + wr.numel() * 2)
+    rt = route()[0]
     w_in, w_out = _bf(E, 2, F, W), _bf(E, W, F)
     used = int((rt.offsets[1:] > rt.offsets[:-1]).sum())
     t("expert_glu", lambda: ops.expert_glu(h, w_in, rt), (used * 2 * F * W + M * W + M * top * F) * 2, 4.0 * M * top * F * W)
@@ -381,9 +384,8 @@ def ruburax_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     t("expert_down", lambda: ops.expert_down(act, w_out, rt), (used * F * W + M * top * (F + W)) * 2, 2.0 * M * top * F * W)
     rows, sg = ops.expert_down(act, w_out, rt), torch.randn(M, device=DEV)
     t("moe_norm_add", lambda: ops.moe_norm_add(x, rows, rt, y32, sg, w, 0.5, W, eps), M * W * (14 + 2 * top))
-    _gemm(t, "gemm shared gate, up", M, 2 * sh, W)
-    gu, act = _bf(M, 2 * sh), _bf(M, sh)
-    t("glu", lambda: ops.glu(gu[:, :sh], gu[:, sh:], act), M * sh * 6)
+    gu, act = _bf(2 * sh, W), _bf(M, sh)
+    t("glu_linear (shared)", lambda: ops.glu_linear(h, gu, act), (M * W + 2 * sh * W + M * sh) * 2, 4.0 * M * sh * W)
     _gemm(t, "gemm shared down (fp32)", M, W, sh, True)
     d = mc.side_dim
     _gemm(t, "gemm token gate", M, d, W)

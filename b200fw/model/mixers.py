@@ -106,7 +106,7 @@ class PackedRows(nn.Module):
 
     def fp32(self, x: torch.Tensor) -> torch.Tensor:
         """The product with a 32-bit result."""
-        return ops.gemm(x, self.weight, out=torch.empty((x.shape[0], self.weight.shape[0]), dtype=torch.float32, device=x.device))
+        return ops.linear_fp32(x, self.weight)
 
 
 class PackedCols(nn.Module):
@@ -471,8 +471,8 @@ class GatedFF(nn.Module):
 
     def run(self, h: torch.Tensor) -> torch.Tensor:
         """fp32 ``[M, hidden]``."""
-        y, a = self.up(h), self.down.buffer(h.shape[0])
-        ops.glu(self.up.cols(y, "gate"), self.up.cols(y, "up"), a)
+        a = self.down.buffer(h.shape[0])
+        ops.glu_linear(h, self.up.weight, a)
         return self.down(a)
 
     def add(self, x: torch.Tensor, h: torch.Tensor, norm: torch.Tensor, coef: float, n: int, eps: float) -> torch.Tensor:
@@ -514,11 +514,9 @@ class ExpertFF(nn.Module):
 
     def add(self, x: torch.Tensor, h: torch.Tensor, norm: torch.Tensor, coef: float, n: int, eps: float) -> torch.Tensor:
         """``x += coef * norm(ff(h))``; the new ``x`` in the activation dtype."""
-        z = self.router.fp32(h)
-        r = ops.route(self.router.cols(z, "router"), self.correction, self.top, self.groups, self.keep, self.scale)
-        shared = gate = None
-        if self.shared is not None:
-            shared, gate = self.shared.run(h), self.router.cols(z, "sg")[:, 0]
+        r, gate = ops.router(h, self.router.weight, -1 if self.shared is None else self.router.sections["sg"][0], self.correction, self.top,
+                             self.groups, self.keep, self.scale)
+        shared = None if self.shared is None else self.shared.run(h)
         rows = ops.expert_down(ops.expert_glu(h, self.w_in, r), self.w_out, r)
         return ops.moe_norm_add(x, rows, r, shared, gate, norm, coef, n, eps)
 

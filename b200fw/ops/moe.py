@@ -8,7 +8,8 @@ from typing import Optional
 import torch
 
 from .. import _native as nv
-from .residual import _f32
+from .gemm import gemm, linear
+from .residual import _f32, glu
 
 
 @dataclass
@@ -47,15 +48,65 @@ def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int,
         offsets = torch.zeros(E + 1, dtype=torch.int32)
         offsets[1:] = torch.bincount(flat, minlength=E).cumsum(0)
         return Routing(s.gather(1, ids) * scale, place.reshape(M, top), (order // top).to(torch.int32), offsets)
-    dev = logits.device
-    r = Routing(torch.empty((M, top), device=dev, dtype=torch.float32), torch.empty((M, top), device=dev, dtype=torch.int32),
-                torch.empty(M * top, device=dev, dtype=torch.int32), torch.empty(E + 1, device=dev, dtype=torch.int32))
-    work = torch.empty(E + M * top, device=dev, dtype=torch.int32)      # rows per expert, then (expert, rank) of every pair
+    r, work = _routing(M, E, top, logits.device)
     nv.check(nv.lib().b2_moe_route(
         nv.ptr(logits), nv.ctypes.c_longlong(logits.stride(0)), nv.ptr(correction), nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token),
         nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep, nv.ctypes.c_float(scale), _f32(correction), nv.stream_ptr()), "moe_route")
-    nv.count_launch(2)
+    nv.count_launch(2 if M * top <= 16384 else 3)
     return r
+
+
+def _routing(M: int, E: int, top: int, dev):
+    r = Routing(torch.empty((M, top), device=dev, dtype=torch.float32), torch.empty((M, top), device=dev, dtype=torch.int32),
+                torch.empty(M * top, device=dev, dtype=torch.int32), torch.empty(E + 1, device=dev, dtype=torch.int32))
+    return r, torch.empty(E + M * top, device=dev, dtype=torch.int32)      # rows per expert, then the expert of every pair
+
+
+def router(h: torch.Tensor, w: torch.Tensor, shared_row: int, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float):
+    """Router product in 32-bit and :func:`route`: ``h [M, K]``, ``w [>= E, K]`` with the experts' rows first; ``shared_row >= 0``: that
+    row's product is the shared expert's gate.  Returns ``(Routing, gate [M] or None)``."""
+    M, E, N = h.shape[0], correction.numel(), w.shape[0]
+    if not h.is_cuda or h.dtype != torch.bfloat16 or N > SKINNY:
+        z = linear_fp32(h, w)
+        return route(z, correction, top, groups, keep, scale), None if shared_row < 0 else z[:, shared_row]
+    r, work = _routing(M, E, top, h.device)
+    gate = torch.empty(M, device=h.device, dtype=torch.float32) if shared_row >= 0 else None
+    cl = nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_moe_router(
+        nv.ptr(h), cl(h.stride(0)), nv.ptr(w), cl(w.stride(0)), N, h.shape[1], shared_row, nv.ptr(gate), nv.ptr(correction),
+        nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep,
+        nv.ctypes.c_float(scale), nv.stream_ptr()), "moe_router")
+    nv.count_launch(2 if M * top <= 16384 else 3)
+    return r, gate
+
+
+GATHER_ROWS = 16  # rows per expert (on average) from which they are laid out before the product
+SKINNY = 72      # outputs of a product that take the kernel for few of them
+
+
+def linear_fp32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``x [M, K] w [N, K]^T`` with a 32-bit result."""
+    z = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+    if not x.is_cuda or x.dtype != torch.bfloat16 or w.shape[0] > SKINNY:
+        return gemm(x, w, out=z)
+    cl = nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_skinny(nv.ptr(x), cl(x.stride(0)), nv.ptr(w), cl(w.stride(0)), nv.ptr(z), cl(z.stride(0)), x.shape[0], w.shape[0],
+                                x.shape[1], nv.stream_ptr()), "skinny")
+    nv.count_launch()
+    return z
+
+
+def glu_linear(h: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """``out [M, F] = silu(W_gate h) * (W_up h)`` with ``w [2 F, K]``: gate rows, then up rows."""
+    F = out.shape[1]
+    if not h.is_cuda or h.dtype != torch.bfloat16:
+        y = linear(h, w)
+        return glu(y[:, :F], y[:, F:], out)
+    assert w.is_contiguous() and w.shape[0] == 2 * F and h.stride(1) == 1
+    cl = nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_rows_glu(nv.ptr(h), cl(h.stride(0)), nv.ptr(w), nv.ptr(out), cl(out.stride(0)), h.shape[0], F, h.shape[1],
+                                  nv.stream_ptr()), "rows_glu")
+    nv.count_launch()
 
 
 def expert_glu(h: torch.Tensor, w: torch.Tensor, r: Routing) -> torch.Tensor:
@@ -71,9 +122,10 @@ def expert_glu(h: torch.Tensor, w: torch.Tensor, r: Routing) -> torch.Tensor:
             out[off[e]:off[e + 1]] = (torch.nn.functional.silu(x @ w[e, 0].float().t()) * (x @ w[e, 1].float().t())).to(h.dtype)
         return out
     assert h.stride(1) == 1 and w.is_contiguous()
-    nv.check(nv.lib().b2_moe_glu(nv.ptr(h), nv.ctypes.c_longlong(h.stride(0)), nv.ptr(w), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(out), h.shape[0], P, E, F,
-                                 K, _f32(h), nv.stream_ptr()), "moe_glu")
-    nv.count_launch()
+    rows = torch.empty((P, K), device=h.device, dtype=h.dtype) if h.dtype == torch.bfloat16 and P >= GATHER_ROWS * E else None
+    nv.check(nv.lib().b2_moe_glu(nv.ptr(h), nv.ctypes.c_longlong(h.stride(0)), nv.ptr(w), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(rows),
+                                 nv.ptr(out), h.shape[0], P, E, F, K, _f32(h), nv.stream_ptr()), "moe_glu")
+    nv.count_launch(1 if rows is None else 2)
     return out
 
 

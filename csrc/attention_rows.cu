@@ -400,7 +400,6 @@ struct NormStoreParams {
 // Bias, per-head RMS norm of q and k (optional weights), rotary positions on channel pairs (2 i, 2 i + 1), and the store of k / v.
 // Grid (M, y).  LPH lanes per head, eight channels each; a lane takes NS_UNROLL heads of its row at a time, their loads together.
 // What waits in registers waits packed, so that eight CTAs fit on an SM.
-constexpr int NS_UNROLL = 4;
 template <typename T>
 struct Packed8 {
   uint4 w[sizeof(T) / 2];
@@ -414,7 +413,7 @@ struct Packed8 {
   }
   __device__ __forceinline__ void get(float (&f)[8]) const { vload8(reinterpret_cast<const T*>(w), f); }
 };
-template <typename T, int LPH>
+template <typename T, int LPH, int NS_UNROLL>
 __global__ void __launch_bounds__(128, sizeof(T) == 2 ? 8 : 4) qk_norm_store_kernel(const NormStoreParams p) {
   constexpr int GROUPS = 128 / LPH;
   const int group = threadIdx.x / LPH, c = threadIdx.x % LPH * 8, units = p.H + p.G + p.Gv;
@@ -610,14 +609,22 @@ B2_EXPORT int b2_qk_norm_store(const void* q, const void* k, const void* v, long
                              M, max_blocks, H, G, Gv, dk, dkp, dvp, norm, rot, eps};
   const int w = dkp > dvp ? dkp : dvp, lph = w <= 64 ? 8 : w <= 128 ? 16 : 32, groups = 128 / lph;
   int y = (H + G + Gv + groups - 1) / groups;              // a head per lane group; several when the rows fill the GPU
-  if (M >= 8 * num_sms()) y = (y + NS_UNROLL - 1) / NS_UNROLL;
+  const int unroll = M < 8 * num_sms() || y == 1 ? 1 : y == 2 ? 2 : 4;
+  y = (y + unroll - 1) / unroll;
   const dim3 grid(M < 16 * num_sms() ? M : 16 * num_sms(), y);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+#define B2_NORM_STORE(L)                                                      \
+  do {                                                                        \
+    if (unroll == 1) qk_norm_store_kernel<T, L, 1><<<grid, 128, 0, st>>>(p);  \
+    else if (unroll == 2) qk_norm_store_kernel<T, L, 2><<<grid, 128, 0, st>>>(p); \
+    else qk_norm_store_kernel<T, L, 4><<<grid, 128, 0, st>>>(p);              \
+  } while (0)
   B2_DISPATCH_T(is_f32, {
-    if (lph == 8) qk_norm_store_kernel<T, 8><<<grid, 128, 0, st>>>(p);
-    else if (lph == 16) qk_norm_store_kernel<T, 16><<<grid, 128, 0, st>>>(p);
-    else qk_norm_store_kernel<T, 32><<<grid, 128, 0, st>>>(p);
+    if (lph == 8) B2_NORM_STORE(8);
+    else if (lph == 16) B2_NORM_STORE(16);
+    else B2_NORM_STORE(32);
   });
+#undef B2_NORM_STORE
   B2_CHECK_LAUNCH("qk_norm_store");
   return 0;
 }

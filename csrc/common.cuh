@@ -178,6 +178,14 @@ __device__ __forceinline__ void tma_load_4d(void* dst, const void* tmap, uint64_
       "l"(tmap), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z), "r"(w)
       : "memory");
 }
+// Four rows y0 .. y3 of a 2-D map whose box is one row high, one below the other.
+__device__ __forceinline__ void tma_gather4(void* dst, const void* tmap, uint64_t* bar, int x, int y0, int y1, int y2, int y3) {
+  asm volatile(
+      "cp.async.bulk.tensor.2d.shared::cta.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6, %7}], [%2];" ::"r"(
+          smem_u32(dst)),
+      "l"(tmap), "r"(smem_u32(bar)), "r"(x), "r"(y0), "r"(y1), "r"(y2), "r"(y3)
+      : "memory");
+}
 // 2-D tiled store shared -> global (bulk async group); rows / columns outside the tensor are clipped.
 __device__ __forceinline__ void tma_store_2d(const void* tmap, const void* src, int x, int y) {
   asm volatile("cp.async.bulk.tensor.2d.global.shared::cta.bulk_group [%0, {%2, %3}], [%1];" ::"l"(tmap),

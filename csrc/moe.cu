@@ -1,16 +1,18 @@
 // Mixture of experts.
 //
 //   moe_route / moe_place   sigmoid scores, the choice among the best groups, and the (token, choice) pairs laid out expert after expert
-//   moe_gemm<GLU>           silu(W_gate h) * (W_up h) over every expert's rows, h gathered by token
-//   moe_gemm<DOWN>          W_down of those rows
+//   moe_gemm (MOE_GLU)      silu(W_gate h) * (W_up h) over every expert's rows, h gathered by token
+//   moe_gemm (MOE_DOWN)     W_down of those rows
+//   moe_gemm (ROWS_GLU)     the first product over rows that are in order already
 //   moe_norm_add            the weighted sum of a token's rows, a gated shared expert, the norm of the sum, the residual
 //
 // The products are persistent tcgen05 kernels over the list of (expert, 128-row tile, column tile): TMA brings the weights (one 3-D
 // map over all experts, so that a tile past an expert's last row is filled with zeros instead of its neighbour's rows), fp32
 // accumulators stay in TMEM, double-buffered.  The GLU form holds gate and up columns of a tile side by side in one accumulator, so
-// the activation happens on the way out; its token rows are gathered by four warps with asynchronous copies into the swizzled layout.
-// How many rows each expert has is known on the device only: every CTA works out the tile list from the offsets.
+// the activation happens on the way out.  With few rows per expert its token rows are gathered by TMA, four rows a copy; that copy's
+// rate would bound the product over long prompts, so there the rows are laid out expert after expert first (moe_gather).  How many rows each expert has is known on the device only: every CTA works out the tile list from the offsets.
 #include "host.h"
+#include "mma_split.cuh"
 #include "vec.cuh"
 
 namespace b2 {
@@ -20,16 +22,10 @@ constexpr int MOE_MAX_TOP = 32;
 typedef __nv_bfloat16 moe_bf16;
 
 // ---- routing -----------------------------------------------------------------------------------------------------------
-constexpr int MR_WARPS = 4;
-
 struct RouteParams {
-  const float* z;        // [M, ld]
   const void* corr;      // T [E]
   float* weights;        // [M, top]
-  int* place;            // [M, top]: rank among the expert's rows, then the row
-  int* count;            // [E], zero
   int* id;               // [M, top]
-  long long ld;
   int M, E, top, groups, keep;
   float scale;
 };
@@ -47,15 +43,10 @@ __device__ __forceinline__ void argmax_warp(float& v, int& i) {
   }
 }
 
-// A warp per token.
+// The choice of one token by a warp.  z: its logits; c, gs: E floats of shared memory each (choice and group scores).
 template <typename T>
-__global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RouteParams p) {
-  extern __shared__ float mr_smem[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * MR_WARPS + warp;
-  if (row >= p.M) return;
-  float* c = mr_smem + warp * 2 * p.E;      // choice scores
-  float* gs = c + p.E;                      // group scores; a chosen group's is then marked
-  const float* z = p.z + static_cast<size_t>(row) * p.ld;
+__device__ __forceinline__ void route_token(const RouteParams& p, int row, const float* z, float* c, float* gs) {
+  const int lane = threadIdx.x & 31;
   constexpr float LOW = -3.0e38f;           // in place of what is no number (rows without a sequence): below any score, above "closed"
   for (int e = lane; e < p.E; e += 32) {
     const float s = sigmoid_f(z[e]) + to_f(static_cast<const T*>(p.corr)[e]);
@@ -74,7 +65,7 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RoutePar
       gs[g] = per > 1 ? fmaxf(a + b, LOW) : a;
     }
     __syncwarp();
-    for (int k = 0; k < p.keep; ++k) {
+    for (int k = 0; k < p.keep; ++k) {      // a chosen group's score becomes +inf
       float v = -INFINITY;
       int at = p.groups;
       for (int g = lane; g < p.groups; g += 32)
@@ -109,8 +100,80 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RoutePar
     const size_t i = static_cast<size_t>(row) * p.top + lane;
     p.weights[i] = sigmoid_f(z[mine]) * p.scale;
     p.id[i] = mine;
-    p.place[i] = atomicAdd(p.count + mine, 1);
   }
+  __syncwarp();
+}
+
+// Logits given: a warp per token.
+constexpr int MR_WARPS = 4;
+template <typename T>
+__global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RouteParams p, const float* __restrict__ z, long long ld) {
+  extern __shared__ float mr_smem[];
+  const int warp = threadIdx.x >> 5, row = blockIdx.x * MR_WARPS + warp;
+  if (row >= p.M) return;
+  float* c = mr_smem + warp * 2 * p.E;
+  route_token<T>(p, row, z + static_cast<size_t>(row) * ld, c, c + p.E);
+}
+
+// Products with few outputs (router logits, gates), bf16 operands and a 32-bit result: 16 rows a CTA, its warps split the contraction.
+// A lane loads eight neighbouring elements of its row of either operand at once and uses them as the fragments of two m16n8k16
+// products: the order of the contraction is free as long as both operands agree on it.  ROUTE: the rows' experts are chosen on the spot.
+struct SkinnyParams {
+  const moe_bf16* h;     // [M, ld_h]
+  const moe_bf16* w;     // [N, ld_w]
+  float* z;              // [M, ld_z]; ROUTE: only column sg is stored (sg < 0: none)
+  long long ld_h, ld_w, ld_z;
+  int M, N, K, sg;
+};
+constexpr int SK_ROWS = 16, SK_WARPS = 8, SK_MAX_TILES = 9;
+
+template <int NT, bool ROUTE>
+__global__ void __launch_bounds__(SK_WARPS * 32) skinny_kernel(const SkinnyParams p, const RouteParams r) {
+  constexpr int NP = NT * 8, LD = NP + 2;
+  __shared__ float part[SK_WARPS][SK_ROWS][LD];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3, m0 = blockIdx.x * SK_ROWS;
+  const moe_bf16* a0 = p.h + static_cast<size_t>(min(m0 + g, p.M - 1)) * p.ld_h;
+  const moe_bf16* a1 = p.h + static_cast<size_t>(min(m0 + g + 8, p.M - 1)) * p.ld_h;
+  float acc[NT][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+#pragma unroll 2
+  for (int k = warp * 32 + t * 8; k - t * 8 < p.K; k += SK_WARPS * 32) {
+    const bool in = k < p.K;                 // p.K is a multiple of 8
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    const uint4 x0 = in ? *reinterpret_cast<const uint4*>(a0 + k) : zero, x1 = in ? *reinterpret_cast<const uint4*>(a1 + k) : zero;
+    uint4 w[NT];
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+      w[n] = in && n * 8 + g < p.N ? *reinterpret_cast<const uint4*>(p.w + static_cast<size_t>(n * 8 + g) * p.ld_w + k) : zero;
+    const uint32_t f0[4] = {x0.x, x1.x, x0.y, x1.y}, f1[4] = {x0.z, x1.z, x0.w, x1.w};
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      const uint32_t b0[2] = {w[n].x, w[n].y}, b1[2] = {w[n].z, w[n].w};
+      mma_bf16(acc[n], f0, b0);
+      mma_bf16(acc[n], f1, b1);
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    *reinterpret_cast<float2*>(&part[warp][g][n * 8 + 2 * t]) = make_float2(acc[n][0], acc[n][1]);
+    *reinterpret_cast<float2*>(&part[warp][g + 8][n * 8 + 2 * t]) = make_float2(acc[n][2], acc[n][3]);
+  }
+  __syncthreads();
+  for (int i = tid; i < SK_ROWS * NP; i += SK_WARPS * 32) {
+    const int row = i / NP, c = i % NP;
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < SK_WARPS; ++w) s += part[w][row][c];
+    if (ROUTE) part[0][row][c] = s;          // read by this thread alone until the barrier
+    if (m0 + row < p.M && (ROUTE ? c == p.sg : c < p.N)) p.z[static_cast<size_t>(m0 + row) * p.ld_z + (ROUTE ? 0 : c)] = s;
+  }
+  if (!ROUTE) return;
+  __syncthreads();
+  for (int row = warp; row < SK_ROWS && m0 + row < p.M; row += SK_WARPS)
+    route_token<moe_bf16>(r, m0 + row, part[0][row], part[1 + (warp >> 1)][(warp & 1) * 8], part[1 + (warp >> 1)][(warp & 1) * 8 + 1]);
 }
 
 // Running sums of f(i) over i < n by a whole warp: out[0 .. n].
@@ -133,8 +196,64 @@ __device__ __forceinline__ void warp_prefix(int n, int* out, F f) {
   if (lane == 0) out[n] = carry;
 }
 
-__global__ void __launch_bounds__(256) moe_place_kernel(const int* __restrict__ count, const int* __restrict__ id, int* __restrict__ place,
-                                                        int* __restrict__ token, int* __restrict__ offsets, int E, int top, int total) {
+// The layout of the (token, choice) pairs.  Up to MP_ONE pairs: one CTA counts in shared memory.
+constexpr int MP_THREADS = 1024, MP_EACH = 16, MP_ONE = MP_THREADS * MP_EACH;
+__global__ void __launch_bounds__(MP_THREADS) moe_place_kernel(const int* __restrict__ id, int* __restrict__ place, int* __restrict__ token,
+                                                               int* __restrict__ offsets, int E, int top, int total) {
+  __shared__ int cnt[MOE_MAX_EXPERTS], off[MOE_MAX_EXPERTS + 1];
+  for (int e = threadIdx.x; e < E; e += MP_THREADS) cnt[e] = 0;
+  __syncthreads();
+  int e[MP_EACH], rank[MP_EACH];
+#pragma unroll
+  for (int j = 0; j < MP_EACH; ++j) {
+    const int i = threadIdx.x + j * MP_THREADS;
+    e[j] = i < total ? id[i] : 0;
+  }
+#pragma unroll
+  for (int j = 0; j < MP_EACH; ++j)
+    if (static_cast<int>(threadIdx.x) + j * MP_THREADS < total) rank[j] = atomicAdd(cnt + e[j], 1);
+  __syncthreads();
+  if (threadIdx.x < 32) warp_prefix(E, off, [&](int k) { return cnt[k]; });
+  __syncthreads();
+  for (int k = threadIdx.x; k <= E; k += MP_THREADS) offsets[k] = off[k];
+#pragma unroll
+  for (int j = 0; j < MP_EACH; ++j) {
+    const int i = threadIdx.x + j * MP_THREADS;
+    if (i >= total) break;
+    const int r = off[e[j]] + rank[j];
+    place[i] = r;
+    token[r] = i / top;
+  }
+}
+
+// More pairs: every CTA counts its own, takes its places among the experts' rows (count, zero before), then the same once the counts
+// are complete.
+__global__ void __launch_bounds__(256) moe_rank_kernel(const int* __restrict__ id, int* __restrict__ place, int* __restrict__ count, int E,
+                                                       int total) {
+  __shared__ int cnt[MOE_MAX_EXPERTS];
+  for (int e = threadIdx.x; e < E; e += 256) cnt[e] = 0;
+  __syncthreads();
+  int e[4], rank[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int i = (blockIdx.x * 4 + j) * 256 + threadIdx.x;
+    if (i < total) {
+      e[j] = id[i];
+      rank[j] = atomicAdd(cnt + e[j], 1);
+    }
+  }
+  __syncthreads();
+  for (int k = threadIdx.x; k < E; k += 256)
+    if (cnt[k] > 0) cnt[k] = atomicAdd(count + k, cnt[k]);
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int i = (blockIdx.x * 4 + j) * 256 + threadIdx.x;
+    if (i < total) place[i] = cnt[e[j]] + rank[j];
+  }
+}
+__global__ void __launch_bounds__(256) moe_layout_kernel(const int* __restrict__ count, const int* __restrict__ id, int* __restrict__ place,
+                                                         int* __restrict__ token, int* __restrict__ offsets, int E, int top, int total) {
   __shared__ int off[MOE_MAX_EXPERTS + 1];
   if (threadIdx.x < 32) warp_prefix(E, off, [&](int e) { return count[e]; });
   __syncthreads();
@@ -230,26 +349,27 @@ template <int BN>
 struct MoeCfg {
   static constexpr int A_BYTES = MG_BM * MG_BK * 2, B_BYTES = BN * MG_BK * 2, STAGE = A_BYTES + B_BYTES;
   static constexpr int STAGES = BN == 256 ? 4 : BN == 128 ? 6 : 8;
-  static constexpr int LAG = STAGES - 2;       // k-blocks whose gathered rows may still be on their way (below STAGES)
   static constexpr int STAGING = 4 * 4096;                        // a block per epilogue warp
   static constexpr int TABLES = 2 * (MOE_MAX_EXPERTS + 1) * 4;
   static constexpr int SMEM = STAGES * STAGE + STAGING + 256 + TABLES + 1024;
   static constexpr int TMEM = 2 * BN;
 };
 
+enum : int { MOE_GLU = 0, MOE_DOWN = 1, ROWS_GLU = 2 };
+
 struct MoeGemmParams {
-  const moe_bf16* a;       // GLU: token rows [tokens, lda]
-  long long lda;
-  const int* token;        // GLU: [P]
-  const int* offsets;      // [E + 1]
-  moe_bf16* out;           // [P, N]
-  int E, N, K;             // GLU: N activation columns (half of a tile's accumulator columns each for gate and up)
+  const int* token;        // MOE_GLU: [P]
+  const int* offsets;      // [E + 1], or null: one expert, all rows
+  moe_bf16* out;           // [P, ld_out]
+  long long ld_out;
+  int P, E, N, K;          // GLU: N activation columns (half of a tile's accumulator columns each for gate and up)
 };
 
-template <int BN, bool GLU>
-__global__ void __launch_bounds__(GLU ? 320 : 192, 1)
+template <int BN, int FORM>
+__global__ void __launch_bounds__(192, 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const MoeGemmParams p, int* status) {
   using Cfg = MoeCfg<BN>;
+  constexpr bool GLU = FORM != MOE_DOWN;
   constexpr int STAGES = Cfg::STAGES, COLS = GLU ? BN / 2 : BN;    // output columns of a tile
   extern __shared__ uint8_t mg_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(mg_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -262,7 +382,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
     for (int i = 0; i < STAGES; ++i) {
-      mbar_init(full + i, GLU ? 1 + 4 : 1);       // the weights' copy, and the gathering warps
+      mbar_init(full + i, 1);
       mbar_init(empty + i, 1);
     }
     for (int i = 0; i < 2; ++i) {
@@ -270,13 +390,14 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
       mbar_init(acc_empty + i, 4);
     }
     mbar_fence_init();
+    tma_prefetch_desc(&tmA);
     tma_prefetch_desc(&tmB);
   }
   if (warp == 1) {
     tmem_alloc(tmem_slot, Cfg::TMEM);
     tmem_relinquish();
   }
-  for (int e = tid; e <= p.E; e += blockDim.x) off[e] = p.offsets[e];
+  for (int e = tid; e <= p.E; e += blockDim.x) off[e] = p.offsets ? p.offsets[e] : e * p.P;
   __syncthreads();
   if (warp == 0) warp_prefix(p.E, first, [&](int e) { return (off[e + 1] - off[e] + MG_BM - 1) / MG_BM; });
   tc_fence_before();
@@ -286,30 +407,39 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
   const int ncols = (p.N + COLS - 1) / COLS, tiles = first[p.E] * ncols, nkb = (p.K + MG_BK - 1) / MG_BK;
 
   if (warp == 0) {
-    if (lane == 0) {
-      int st = 0;
-      uint32_t ph = 0;
-      bool ok = true;
-      for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
-        const MoeTile tl = moe_tile(t, off, first, p.E, MG_BM, ncols);
-        for (int kb = 0; kb < nkb; ++kb) {
-          if (!mbar_wait(empty + st, ph ^ 1, status, ERR_GEMM_PRODUCER_WAIT)) {
-            ok = false;
-            break;
-          }
-          uint8_t *sA = smem + st * Cfg::STAGE, *sB = sA + Cfg::A_BYTES;
-          mbar_expect_tx(full + st, Cfg::B_BYTES + (GLU ? 0 : Cfg::A_BYTES));
+    // Lane l gathers rows 4 l .. 4 l + 3 of a tile; a group that reaches past the expert's last row repeats it, groups further on keep
+    // what they hold: those results are dropped.
+    int st = 0;
+    uint32_t ph = 0;
+    bool ok = true;
+    for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
+      const MoeTile tl = moe_tile(t, off, first, p.E, MG_BM, ncols);
+      const int groups = (tl.rows + 3) / 4;
+      int y[4] = {};
+      if (FORM == MOE_GLU && lane < groups)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) y[i] = p.token[tl.row0 + min(lane * 4 + i, tl.rows - 1)];
+      for (int kb = 0; kb < nkb; ++kb) {
+        if (!mbar_wait_warp(empty + st, ph ^ 1, status, ERR_GEMM_PRODUCER_WAIT)) {
+          ok = false;
+          break;
+        }
+        uint8_t *sA = smem + st * Cfg::STAGE, *sB = sA + Cfg::A_BYTES;
+        if (lane == 0) {
+          mbar_expect_tx(full + st, Cfg::B_BYTES + (FORM == MOE_GLU ? groups * 512 : Cfg::A_BYTES));
           if (GLU) {
             tma_load_3d(sB, &tmB, full + st, kb * MG_BK, tl.col * COLS, 2 * tl.expert);
             tma_load_3d(sB + Cfg::B_BYTES / 2, &tmB, full + st, kb * MG_BK, tl.col * COLS, 2 * tl.expert + 1);
           } else {
-            tma_load_2d(sA, &tmA, full + st, kb * MG_BK, tl.row0);
             tma_load_3d(sB, &tmB, full + st, kb * MG_BK, tl.col * COLS, tl.expert);
           }
-          if (++st == STAGES) {
-            st = 0;
-            ph ^= 1;
-          }
+          if (FORM != MOE_GLU) tma_load_2d(sA, &tmA, full + st, kb * MG_BK, tl.row0);
+        }
+        __syncwarp();
+        if (FORM == MOE_GLU && lane < groups) tma_gather4(sA + lane * 512, &tmA, full + st, kb * MG_BK, y[0], y[1], y[2], y[3]);
+        if (++st == STAGES) {
+          st = 0;
+          ph ^= 1;
         }
       }
     }
@@ -346,57 +476,6 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
       acc ^= 1;
       if (acc == 0) acc_ph ^= 1;
     }
-  } else if (GLU && warp >= 6) {
-    // Token rows into the swizzled A tile: eight lanes a row (whole 128-byte lines), rows 32 w .. 32 w + 31 of warp w.  A stage is
-    // handed over LAG k-blocks after its copies were issued, once they have landed and are visible to the tensor core.
-    const int w = warp - 6, chunk = lane & 7, sub = lane >> 3;
-    int st = 0, done = 0;            // stages issued into, handed over
-    uint32_t ph = 0;
-    int pending = 0;
-    bool ok = true;
-    auto hand_over = [&]() {
-      fence_proxy_async_smem();
-      mbar_arrive_warp(full + done);
-      if (++done == STAGES) done = 0;
-      --pending;
-    };
-    for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
-      const MoeTile tl = moe_tile(t, off, first, p.E, MG_BM, ncols);
-      const moe_bf16* src[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int r = w * 32 + j * 4 + sub;
-        src[j] = p.a + (r < tl.rows ? static_cast<size_t>(p.token[tl.row0 + r]) * p.lda : 0) + chunk * 8;
-      }
-      for (int kb = 0; kb < nkb; ++kb) {
-        if (!mbar_wait_warp(empty + st, ph ^ 1, status, ERR_GEMM_PRODUCER_WAIT)) {
-          ok = false;
-          break;
-        }
-        const uint32_t base = smem_u32(smem + st * Cfg::STAGE) + (w * 32 + sub) * 128;
-        const int bytes = kb * MG_BK + chunk * 8 < p.K ? 16 : 0;       // zeros past the last column (p.K is a multiple of 8)
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const int r = j * 4 + sub;
-          if (w * 32 + r < tl.rows)        // rows past the expert's last one keep what they hold: their results are dropped
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(base + j * 512 + ((chunk ^ (r & 7)) << 4)),
-                         "l"(bytes ? src[j] + kb * MG_BK : p.a), "r"(bytes)
-                         : "memory");
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        ++pending;
-        if (++st == STAGES) {
-          st = 0;
-          ph ^= 1;
-        }
-        if (pending > Cfg::LAG) {
-          asm volatile("cp.async.wait_group %0;" ::"n"(Cfg::LAG) : "memory");
-          hand_over();
-        }
-      }
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    while (pending > 0) hand_over();
   } else {
     const int quarter = warp & 3;
     uint8_t* stage = staging + quarter * 4096;
@@ -445,10 +524,10 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
           }
         }
         const int col = tl.col * COLS + c0;
-        moe_bf16* base = p.out + static_cast<size_t>(tl.row0 + quarter * 32) * p.N + col;
+        moe_bf16* base = p.out + static_cast<size_t>(tl.row0 + quarter * 32) * p.ld_out + col;
         warp_store_rows_128B(stage, v, [&](int row) -> uint8_t* {
           if (quarter * 32 + row >= tl.rows || col + (lane & 7) * 8 >= p.N || c0 + (lane & 7) * 8 >= COLS) return nullptr;
-          return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * p.N);
+          return reinterpret_cast<uint8_t*>(base + static_cast<size_t>(row) * p.ld_out);
         });
       }
       tc_fence_before();
@@ -467,6 +546,25 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
     __syncwarp();
     tc_fence_after();
     tmem_dealloc(tmem, Cfg::TMEM);
+  }
+}
+
+// rows[r] = h[token[r]], a warp per row (16 bytes a lane)
+__global__ void __launch_bounds__(256) moe_gather_kernel(const moe_bf16* __restrict__ h, long long ld, const int* __restrict__ token,
+                                                         moe_bf16* __restrict__ rows, int P, int K) {
+  for (int r = blockIdx.x * 8 + (threadIdx.x >> 5); r < P; r += gridDim.x * 8) {
+    const uint4* src = reinterpret_cast<const uint4*>(h + static_cast<size_t>(token[r]) * ld);
+    uint4* dst = reinterpret_cast<uint4*>(rows + static_cast<size_t>(r) * K);
+    const int n = K / 8;
+    for (int c0 = threadIdx.x & 31; c0 < n; c0 += 128) {
+      uint4 v[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c0 + 32 * i < n) v[i] = src[c0 + 32 * i];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c0 + 32 * i < n) dst[c0 + 32 * i] = v[i];
+    }
   }
 }
 
@@ -547,10 +645,10 @@ __global__ void __launch_bounds__(MAXT) moe_norm_add_kernel(const MoeAddParams p
   }
 }
 
-template <int BN, bool GLU>
+template <int BN, int FORM>
 static int launch_moe(const CUtensorMap* ta, const CUtensorMap* tb, const MoeGemmParams& p, int bound, cudaStream_t stream) {
   using Cfg = MoeCfg<BN>;
-  auto kern = moe_gemm_kernel<BN, GLU>;
+  auto kern = moe_gemm_kernel<BN, FORM>;
   int* status = status_ptr();
   if (!status) return 3;
   static bool set[64] = {false};
@@ -563,12 +661,25 @@ static int launch_moe(const CUtensorMap* ta, const CUtensorMap* tb, const MoeGem
     }
     set[dev & 63] = true;
   }
-  constexpr int COLS = GLU ? BN / 2 : BN;
+  constexpr int COLS = FORM != MOE_DOWN ? BN / 2 : BN;
   const long long tiles = static_cast<long long>(bound) * ((p.N + COLS - 1) / COLS);
   const int grid = tiles < num_sms() ? static_cast<int>(tiles) : num_sms();
-  kern<<<grid, GLU ? 320 : 192, Cfg::SMEM, stream>>>(*ta, *tb, p, status);
+  kern<<<grid, 192, Cfg::SMEM, stream>>>(*ta, *tb, p, status);
   B2_CHECK_LAUNCH("moe_gemm");
   return 0;
+}
+
+// Gate and up [E, 2, F, K] in tiles of `cols` activation columns.
+template <int FORM>
+static int launch_glu(const CUtensorMap* ta, const void* w, const MoeGemmParams& p, int cols, int bound, cudaStream_t stream) {
+  const uint64_t dims[3] = {static_cast<uint64_t>(p.K), static_cast<uint64_t>(p.N), 2ull * p.E},
+                 strides[2] = {2ull * p.K, 2ull * p.N * p.K};
+  const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
+  const CUtensorMap* tb = tensor_map_nd_bf16(w, 3, dims, strides, box, 3);
+  if (!ta || !tb) return 2;
+  if (cols == 128) return launch_moe<256, FORM>(ta, tb, p, bound, stream);
+  if (cols == 64) return launch_moe<128, FORM>(ta, tb, p, bound, stream);
+  return launch_moe<64, FORM>(ta, tb, p, bound, stream);
 }
 
 static int moe_bound(int P, int E, int tile) { return P / tile + (E < P ? E : P); }    // row tiles at most
@@ -593,30 +704,92 @@ static int moe_columns(int P, int E, int N, int widest, int narrowest) {
 
 using namespace b2;
 
+static bool bad_routing(int M, int E, int top, int groups, int keep) {
+  if (E < 1 || E > MOE_MAX_EXPERTS || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > MOE_MAX_TOP ||
+      top > keep * (E / groups) || static_cast<long long>(M) * top > 0x7fffffffll) {
+    set_error("moe_route: up to %d experts in equal groups and up to %d chosen required", MOE_MAX_EXPERTS, MOE_MAX_TOP);
+    return true;
+  }
+  return false;
+}
+
+// work: [E] counts, then [M * top] chosen experts
+static int launch_place(int* place, int* token, int* offsets, int* work, int M, int E, int top, cudaStream_t st) {
+  const int total = M * top;
+  int* id = work + E;
+  if (total <= MP_ONE) {
+    moe_place_kernel<<<1, MP_THREADS, 0, st>>>(id, place, token, offsets, E, top, total);
+    B2_CHECK_LAUNCH("moe_place");
+    return 0;
+  }
+  if (cudaMemsetAsync(work, 0, sizeof(int) * E, st) != cudaSuccess) { set_error("moe_place: clearing the counts failed"); return 5; }
+  moe_rank_kernel<<<(total + 1023) / 1024, 256, 0, st>>>(id, place, work, E, total);
+  B2_CHECK_LAUNCH("moe_rank");
+  moe_layout_kernel<<<2 * num_sms(), 256, 0, st>>>(work, id, place, token, offsets, E, top, total);
+  B2_CHECK_LAUNCH("moe_layout");
+  return 0;
+}
+
 // z: fp32 [M, ld]; work: int32 [E + M * top]; offsets: int32 [E + 1]; place: int32 [M, top]; token: int32 [M * top].
 B2_EXPORT int b2_moe_route(const float* z, long long ld, const void* corr, float* weights, int* place, int* token, int* offsets,
                            int* work, int M, int E, int top, int groups, int keep, float scale, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
-  if (E < 1 || E > MOE_MAX_EXPERTS || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > MOE_MAX_TOP ||
-      top > keep * (E / groups) || static_cast<long long>(M) * top > 0x7fffffffll || ld < E) {
-    set_error("moe_route: up to %d experts in equal groups and up to %d chosen required", MOE_MAX_EXPERTS, MOE_MAX_TOP);
-    return 10;
-  }
+  if (bad_routing(M, E, top, groups, keep)) return 10;
+  if (ld < E) { set_error("moe_route: a logit per expert required"); return 10; }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (cudaMemsetAsync(work, 0, sizeof(int) * E, st) != cudaSuccess) { set_error("moe_route: clearing the counts failed"); return 5; }
-  const RouteParams p = {z, corr, weights, place, work, work + E, ld, M, E, top, groups, keep, scale};
-  B2_DISPATCH_T(is_f32, moe_route_kernel<T><<<(M + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, MR_WARPS * 2 * E * sizeof(float), st>>>(p););
+  const RouteParams p = {corr, weights, work + E, M, E, top, groups, keep, scale};
+  B2_DISPATCH_T(is_f32, moe_route_kernel<T><<<(M + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, MR_WARPS * 2 * E * sizeof(float), st>>>(p, z, ld););
   B2_CHECK_LAUNCH("moe_route");
-  const int total = M * top, blocks = (total + 255) / 256;
-  moe_place_kernel<<<blocks < 2 * num_sms() ? blocks : 2 * num_sms(), 256, 0, st>>>(work, work + E, place, token, offsets, E, top, total);
-  B2_CHECK_LAUNCH("moe_place");
+  return launch_place(place, token, offsets, work, M, E, top, st);
+}
+
+template <bool ROUTE>
+static int launch_skinny(const SkinnyParams& p, const RouteParams& r, cudaStream_t st) {
+  const int grid = (p.M + SK_ROWS - 1) / SK_ROWS, nt = (p.N + 7) / 8;
+#define B2_SKINNY(V) case V: skinny_kernel<V, ROUTE><<<grid, SK_WARPS * 32, 0, st>>>(p, r); break
+  switch (nt) {
+    B2_SKINNY(1); B2_SKINNY(2); B2_SKINNY(3); B2_SKINNY(4); B2_SKINNY(5); B2_SKINNY(6); B2_SKINNY(7); B2_SKINNY(8); B2_SKINNY(9);
+    default: set_error("skinny: up to %d outputs", SK_MAX_TILES * 8); return 10;
+  }
+#undef B2_SKINNY
+  B2_CHECK_LAUNCH("skinny");
   return 0;
 }
 
-// h: T [tokens, ld], w: T [E, 2, F, K], token: int32 [P] -> out T [P, F]
-B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* token, const int* offsets, void* out, int tokens, int P,
-                         int E, int F, int K, int is_f32, void* stream) {
+// z fp32 [M, N] (row stride ld_z) = h bf16 [M, K] w bf16 [N, K]^T for N up to 72
+B2_EXPORT int b2_skinny(const void* h, long long ld_h, const void* w, long long ld_w, float* z, long long ld_z, int M, int N, int K,
+                        void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (N < 1 || K < 8 || K % 8 || ld_h % 8 || ld_w % 8 || ld_z < N) { set_error("skinny: contraction and strides in multiples of 8 required"); return 10; }
+  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), z, ld_h, ld_w, ld_z, M, N, K, -1};
+  return launch_skinny<false>(p, RouteParams{}, static_cast<cudaStream_t>(stream));
+}
+
+// Router product and choice in one kernel, N = E router rows and what follows them in w (up to 72 rows); sg >= 0: row sg's product goes
+// to sg_out fp32 [M].  The rest as b2_moe_route.
+B2_EXPORT int b2_moe_router(const void* h, long long ld_h, const void* w, long long ld_w, int N, int K, int sg, float* sg_out,
+                            const void* corr, float* weights, int* place, int* token, int* offsets, int* work, int M, int E, int top,
+                            int groups, int keep, float scale, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (bad_routing(M, E, top, groups, keep)) return 10;
+  if (N < E || N > SK_MAX_TILES * 8 || K < 8 || K % 8 || ld_h % 8 || ld_w % 8 || sg >= N || (sg >= 0 && sg_out == nullptr)) {
+    set_error("moe_router: up to %d outputs, contraction and strides in multiples of 8 required", SK_MAX_TILES * 8);
+    return 10;
+  }
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), sg_out, ld_h, ld_w, 1, M, N, K, sg};
+  const RouteParams r = {corr, weights, work + E, M, E, top, groups, keep, scale};
+  if (const int rc = launch_skinny<true>(p, r, st)) return rc;
+  return launch_place(place, token, offsets, work, M, E, top, st);
+}
+
+// h: T [tokens, ld], w: T [E, 2, F, K], token: int32 [P] -> out T [P, F].  rows (bf16 [P, K], or null): room for the rows expert after
+// expert, if they are to be laid out before the product.
+B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* token, const int* offsets, void* rows, void* out, int tokens,
+                         int P, int E, int F, int K, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (P <= 0) return 0;
   if (E < 1 || E > MOE_MAX_EXPERTS || F < 8 || F % 8 || K < 8 || K % 8 || ld % 8 || ld < K || tokens < 1) {
@@ -632,17 +805,31 @@ B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* 
     B2_CHECK_LAUNCH("moe_glu");
     return 0;
   }
-  const int cols = moe_columns(P, E, F, 128, 32);
-  const uint64_t dims[3] = {static_cast<uint64_t>(K), static_cast<uint64_t>(F), 2ull * E},
-                 strides[2] = {2ull * K, 2ull * F * K};
-  const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
-  const CUtensorMap* tb = tensor_map_nd_bf16(w, 3, dims, strides, box, 3);
-  if (!tb) return 2;
-  MoeGemmParams p = {static_cast<const moe_bf16*>(h), ld, token, offsets, static_cast<moe_bf16*>(out), E, F, K};
-  const int bound = moe_bound(P, E, MG_BM);
-  if (cols == 128) return launch_moe<256, true>(tb, tb, p, bound, st);
-  if (cols == 64) return launch_moe<128, true>(tb, tb, p, bound, st);
-  return launch_moe<64, true>(tb, tb, p, bound, st);
+  const uint64_t hd[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(tokens)}, hs[1] = {2ull * ld};
+  const uint32_t hbox[2] = {MG_BK, 1};
+  const MoeGemmParams p = {token, offsets, static_cast<moe_bf16*>(out), F, P, E, F, K};
+  if (rows != nullptr) {
+    const int blocks = (P + 7) / 8;
+    moe_gather_kernel<<<blocks < 16 * num_sms() ? blocks : 16 * num_sms(), 256, 0, st>>>(static_cast<const moe_bf16*>(h), ld, token,
+                                                                                        static_cast<moe_bf16*>(rows), P, K);
+    B2_CHECK_LAUNCH("moe_gather");
+    return launch_glu<ROWS_GLU>(tensor_map_2d_bf16(rows, P, K, K, MG_BM, MG_BK), w, p, moe_columns(P, E, F, 128, 32), moe_bound(P, E, MG_BM),
+                                st);
+  }
+  return launch_glu<MOE_GLU>(tensor_map_nd_bf16(h, 2, hd, hs, hbox, 3), w, p, moe_columns(P, E, F, 128, 32), moe_bound(P, E, MG_BM), st);
+}
+
+// One feed-forward for all rows: h bf16 [M, ld], w bf16 [2, F, K] -> out bf16 [M, F] (row stride ld_out)
+B2_EXPORT int b2_rows_glu(const void* h, long long ld, const void* w, void* out, long long ld_out, int M, int F, int K, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (F < 8 || F % 8 || K < 8 || K % 8 || ld % 8 || ld < K || ld_out % 8 || ld_out < F) {
+    set_error("rows_glu: sizes and strides in multiples of 8 required");
+    return 10;
+  }
+  const MoeGemmParams p = {nullptr, nullptr, static_cast<moe_bf16*>(out), ld_out, M, 1, F, K};
+  return launch_glu<ROWS_GLU>(tensor_map_2d_bf16(h, M, K, ld, MG_BM, MG_BK), w, p, moe_columns(M, 1, F, 128, 32), (M + MG_BM - 1) / MG_BM,
+                              static_cast<cudaStream_t>(stream));
 }
 
 // a: T [P, F], w: T [E, N, F] -> out T [P, N]
@@ -669,11 +856,11 @@ B2_EXPORT int b2_moe_down(const void* a, const void* w, const int* offsets, void
   const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
   const CUtensorMap *tb = tensor_map_nd_bf16(w, 3, dims, strides, box, 3), *ta = tensor_map_2d_bf16(a, P, F, F, MG_BM, MG_BK);
   if (!ta || !tb) return 2;
-  MoeGemmParams p = {nullptr, 0, nullptr, offsets, static_cast<moe_bf16*>(out), E, N, F};
+  const MoeGemmParams p = {nullptr, offsets, static_cast<moe_bf16*>(out), N, P, E, N, F};
   const int bound = moe_bound(P, E, MG_BM);
-  if (cols == 256) return launch_moe<256, false>(ta, tb, p, bound, st);
-  if (cols == 128) return launch_moe<128, false>(ta, tb, p, bound, st);
-  return launch_moe<64, false>(ta, tb, p, bound, st);
+  if (cols == 256) return launch_moe<256, MOE_DOWN>(ta, tb, p, bound, st);
+  if (cols == 128) return launch_moe<128, MOE_DOWN>(ta, tb, p, bound, st);
+  return launch_moe<64, MOE_DOWN>(ta, tb, p, bound, st);
 }
 
 B2_EXPORT int b2_moe_norm_add(float* x, const void* rows, const int* place, const float* weights, int top, const float* shared,

@@ -101,7 +101,7 @@ def close(got, want, run, what=""):
     if len(got):
         d = (got - got.mean(-1, keepdim=True)) - (want - want.mean(-1, keepdim=True))
         e = d.pow(2).mean(-1).sqrt() / want.std()
-        assert e.median() < 0.03 and int((e > 0.06).sum()) <= max(2, len(e) // 20) and e.max() < 0.6, f"{what}: {e.topk(min(4, len(e)))}"
+        assert e.median() < 0.03 and int((e > 0.12).sum()) <= max(2, len(e) // 20) and e.max() < 0.6, f"{what}: {e.topk(min(4, len(e)))}"
 
 
 def build(cfg, weights, run):
@@ -283,6 +283,49 @@ def test_routing(run, E, top, groups, keep):
         got = torch.searchsorted(off, place[t], right=True) - 1
         assert sorted(got.tolist()) == sorted(ids) and (token[place[t].long()] == t).all()
         torch.testing.assert_close(w[t].double(), s[t][got.long()] * 2.5, rtol=1e-5, atol=1e-6)
+
+
+@pytest.mark.parametrize("run", RUNS)
+@pytest.mark.parametrize("E,top,groups,keep,W,shared", [(6, 3, 3, 2, 42, True), (32, 4, 8, 4, 1000, True), (64, 6, 8, 3, 264, False), (80, 2, 4, 2, 128, True),
+                                                       (1, 1, 1, 1, 8, True)])
+def test_router_product(run, E, top, groups, keep, W, shared):
+    """The product and the choice together, with rows that fill no tile, and enough of them for both ways of laying out the pairs."""
+    n = pad8(E) + (8 if shared else 0)
+    w = torch.zeros(n, pad8(W))
+    w[:E, :W] = (randn(E, W, seed=1) * W ** -0.5).bfloat16().float()
+    w[pad8(E):, :W] = (randn(n - pad8(E), W, seed=2) * W ** -0.5).bfloat16().float()
+    corr = ((torch.arange(E) * 7 % E) * 1.3 / 8).bfloat16().float()
+    on = lambda t: t.to(run[1]).to(run[0])  # noqa: E731
+    for M in (1, 23, 16384 // top + 5):
+        h = P8(randn(M, W, seed=M)).bfloat16().float()
+        r, gate = ops.router(on(h), on(w), pad8(E) if shared else -1, on(corr), top, groups, keep, 1.5)
+        z = h.double() @ w.double().T
+        if shared:
+            torch.testing.assert_close(gate.double().cpu(), z[:, pad8(E)], rtol=1e-4, atol=1e-4)
+        assert gate is not None or not shared
+        want = ops.route(z[:, :pad8(E)].float(), corr, top, groups, keep, 1.5)
+        same = (r.weights.cpu().sort(-1).values - want.weights.sort(-1).values).abs().max(-1).values < 1e-4
+        assert same.float().mean() > 0.999                       # a choice so close that the order of a sum decides it
+        off, place = r.offsets.cpu(), r.place.cpu()
+        assert off[-1] == M * top and (place.reshape(-1).sort().values == torch.arange(M * top)).all()
+        ids = torch.searchsorted(off, place, right=True) - 1
+        torch.testing.assert_close(r.weights.double().cpu(), O.sigmoid(z.gather(1, ids)) * 1.5, rtol=1e-4, atol=1e-5)
+        assert (r.token.cpu()[place.long()] == torch.arange(M)[:, None]).all()
+    z = ops.linear_fp32(on(h), on(w))
+    torch.testing.assert_close(z.double().cpu(), h.double() @ w.double().T, rtol=1e-4, atol=1e-4)
+
+
+@pytest.mark.parametrize("run", RUNS)
+@pytest.mark.parametrize("M,F,W", [(1, 8, 8), (3, 40, 24), (130, 200, 72), (257, 1000, 328), (300, 136, 128)])
+def test_gated_product(run, M, F, W):
+    h, w = randn(M, W, seed=1).bfloat16().float(), (randn(2 * F, W, seed=2) * W ** -0.5 * 3).bfloat16().float()
+    on = lambda t: t.to(run[1]).to(run[0])  # noqa: E731
+    out = torch.zeros(M, F + 8, dtype=run[1], device=run[0])
+    ops.glu_linear(on(h), on(w), out[:, 8:])
+    want = O.silu(h.double() @ w[:F].double().T) * (h.double() @ w[F:].double().T)
+    tol = dict(rtol=1e-2, atol=1e-2) if run[1] == torch.bfloat16 else dict(rtol=1e-5, atol=1e-4)
+    torch.testing.assert_close(out[:, 8:].double().cpu(), want, **tol)
+    assert not out[:, :8].any()
 
 
 @pytest.mark.parametrize("run", RUNS)
