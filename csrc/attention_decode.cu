@@ -135,8 +135,9 @@ struct DecodeSmem {
 __device__ __forceinline__ void ad_consumer_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 // QP: 32-channel steps of a warp's share of the keys; NG: 16-channel pieces of values per warp; EXACT: the sizes fill both, so that
-// the loops over them have no conditions.
-template <int HALVES, int QP, int NG, bool EXACT>
+// the loops over them have no conditions; FEW: at most eight query rows, so that the upper half of the sixteen is left out of the
+// softmax.
+template <int HALVES, int QP, int NG, bool EXACT, bool FEW>
 __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const DecodeParams p, int* status) {
   constexpr int KT = 64 / HALVES, LDS = KT + 8, KS = KT / 16, PAGES = KT / AD_PAGE;
   extern __shared__ uint8_t ad_raw[];
@@ -296,7 +297,7 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
         }
         float* o = S + (kh * 16 + (lane >> 2)) * LDS + kg * 8 + (lane & 3) * 2;
         *reinterpret_cast<float2*>(o) = make_float2(v[0], v[1]);
-        *reinterpret_cast<float2*>(o + 8 * LDS) = make_float2(v[2], v[3]);
+        if (!FEW) *reinterpret_cast<float2*>(o + 8 * LDS) = make_float2(v[2], v[3]);
         ad_consumer_barrier();
       };
       float* const Sbuf = reinterpret_cast<float*>(ad_smem + L.s);
@@ -316,11 +317,12 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
           mbar_wait_warp(&full[st], ph, status, ERR_ATTN_WAIT);
           scores(st, d);
         }
-        float s[KS][2][4];       // [16 keys][row, row + 8][key pairs 0, 1 and 8, 9 of this lane]
+        constexpr int RH = FEW ? 1 : 2;
+        float s[KS][RH][4];      // [16 keys][row, row + 8][key pairs 0, 1 and 8, 9 of this lane]
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
-          for (int r = 0; r < 2; ++r)
+          for (int r = 0; r < RH; ++r)
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
               const float* at = S + ((lane >> 2) + 8 * r) * LDS + ks * 16 + u * 8 + (lane & 3) * 2;
@@ -339,14 +341,14 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
           for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-              if (ks * 16 + (i >> 1) * 8 + (lane & 3) * 2 + (i & 1) >= left) s[ks][0][i] = s[ks][1][i] = -INFINITY;
+              if (ks * 16 + (i >> 1) * 8 + (lane & 3) * 2 + (i & 1) >= left) s[ks][0][i] = s[ks][RH - 1][i] = -INFINITY;
         }
         if (t == 0 && skip > 0) {
 #pragma unroll
           for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-              if (ks * 16 + (i >> 1) * 8 + (lane & 3) * 2 + (i & 1) < skip) s[ks][0][i] = s[ks][1][i] = -INFINITY;
+              if (ks * 16 + (i >> 1) * 8 + (lane & 3) * 2 + (i & 1) < skip) s[ks][0][i] = s[ks][RH - 1][i] = -INFINITY;
         }
         float n0 = m0, n1 = m1;
 #pragma unroll
@@ -354,14 +356,14 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             n0 = fmaxf(n0, s[ks][0][i]);
-            n1 = fmaxf(n1, s[ks][1][i]);
+            if (!FEW) n1 = fmaxf(n1, s[ks][RH - 1][i]);
           }
 #pragma unroll
         for (int o = 1; o < 4; o <<= 1) {
           n0 = fmaxf(n0, __shfl_xor_sync(0xffffffffu, n0, o));
-          n1 = fmaxf(n1, __shfl_xor_sync(0xffffffffu, n1, o));
+          if (!FEW) n1 = fmaxf(n1, __shfl_xor_sync(0xffffffffu, n1, o));
         }
-        const float f0 = fast_exp2(m0 - n0), f1 = fast_exp2(m1 - n1);      // a tile has at least one key
+        const float f0 = fast_exp2(m0 - n0), f1 = FEW ? 0.f : fast_exp2(m1 - n1);      // a tile has at least one key
         m0 = n0;
         m1 = n1;
         float p0 = 0.f, p1 = 0.f;
@@ -371,14 +373,16 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             s[ks][0][i] = fast_exp2(s[ks][0][i] - n0);
-            s[ks][1][i] = fast_exp2(s[ks][1][i] - n1);
             p0 += s[ks][0][i];
-            p1 += s[ks][1][i];
+            if (!FEW) {
+              s[ks][RH - 1][i] = fast_exp2(s[ks][RH - 1][i] - n1);
+              p1 += s[ks][RH - 1][i];
+            }
           }
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
             pa[ks][2 * u] = pack_bf16x2(s[ks][0][2 * u], s[ks][0][2 * u + 1]);
-            pa[ks][2 * u + 1] = pack_bf16x2(s[ks][1][2 * u], s[ks][1][2 * u + 1]);
+            pa[ks][2 * u + 1] = FEW ? 0u : pack_bf16x2(s[ks][RH - 1][2 * u], s[ks][RH - 1][2 * u + 1]);
           }
         }
         l0 = l0 * f0 + p0;       // this lane's keys only; added over the four lanes of a row at the end
@@ -392,8 +396,10 @@ __global__ void __launch_bounds__(AD_THREADS, 1) decode_attn_kernel(const __grid
           for (int n = 0; n < 2; ++n) {
             acc[g][n][0] *= f0;
             acc[g][n][1] *= f0;
-            acc[g][n][2] *= f1;
-            acc[g][n][3] *= f1;
+            if (!FEW) {
+              acc[g][n][2] *= f1;
+              acc[g][n][3] *= f1;
+            }
           }
 #pragma unroll
           for (int ks = 0; ks < KS; ++ks) {
@@ -563,10 +569,10 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(const DecodeParams p,
         make_uint2(pack_bf16x2(o[0][0], o[0][1]), pack_bf16x2(o[0][2], o[0][3]));
 }
 
-template <int HALVES, int QP, int NG, bool EXACT>
-static int launch_decode(DecodeParams& p, const CUtensorMap* tk, const CUtensorMap* tv, int grid, cudaStream_t stream) {
+template <int HALVES, int QP, int NG, bool EXACT, bool FEW>
+static int launch_form(DecodeParams& p, const CUtensorMap* tk, const CUtensorMap* tv, int grid, cudaStream_t stream) {
   constexpr int KT = 64 / HALVES;
-  auto kern = decode_attn_kernel<HALVES, QP, NG, EXACT>;
+  auto kern = decode_attn_kernel<HALVES, QP, NG, EXACT, FEW>;
   int stages = 8;
   while (stages > 2 && DecodeSmem(p.R, p.C, p.apart, KT, HALVES, stages).total > 232448) --stages;
   const int smem = DecodeSmem(p.R, p.C, p.apart, KT, HALVES, stages).total;
@@ -588,6 +594,11 @@ static int launch_decode(DecodeParams& p, const CUtensorMap* tk, const CUtensorM
   decode_merge_kernel<<<dim3(grid - 1, p.heads), 128, 0, stream>>>(p, grid, KT);
   B2_CHECK_LAUNCH("decode_attention_merge");
   return 0;
+}
+template <int HALVES, int QP, int NG, bool EXACT>
+static int launch_decode(DecodeParams& p, const CUtensorMap* tk, const CUtensorMap* tv, int grid, cudaStream_t stream) {
+  return p.heads * p.maps <= 8 ? launch_form<HALVES, QP, NG, EXACT, true>(p, tk, tv, grid, stream)
+                               : launch_form<HALVES, QP, NG, EXACT, false>(p, tk, tv, grid, stream);
 }
 
 }  // namespace b2

@@ -53,8 +53,9 @@ __device__ __forceinline__ void route_token(const RouteParams& p, int row, const
     c[e] = s >= LOW ? s : LOW;
   }
   __syncwarp();
+  const int per = p.E / p.groups;
+  const bool narrow = p.E <= 4 * 32;        // few enough to find every expert's rank by comparing it with all others
   if (p.keep < p.groups) {
-    const int per = p.E / p.groups;
     for (int g = lane; g < p.groups; g += 32) {
       float a = -INFINITY, b = -INFINITY;
       for (int e = g * per; e < (g + 1) * per; ++e) {
@@ -65,41 +66,75 @@ __device__ __forceinline__ void route_token(const RouteParams& p, int row, const
       gs[g] = per > 1 ? fmaxf(a + b, LOW) : a;
     }
     __syncwarp();
-    for (int k = 0; k < p.keep; ++k) {      // a chosen group's score becomes +inf
-      float v = -INFINITY;
-      int at = p.groups;
-      for (int g = lane; g < p.groups; g += 32)
-        if (gs[g] > v && gs[g] != INFINITY) {
-          v = gs[g];
-          at = g;
+    if (narrow) {
+      float mine[4];                        // +inf for a kept group, -inf for a closed one
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int g = lane + 32 * j;
+        if (g >= p.groups) break;
+        const float v = gs[g];
+        int rank = 0;
+        for (int o = 0; o < p.groups; ++o) {
+          const float w = gs[o];
+          rank += w > v || (w == v && o < g);
         }
-      argmax_warp(v, at);
-      if (lane == 0 && at < p.groups) gs[at] = INFINITY;
+        mine[j] = rank < p.keep ? INFINITY : -INFINITY;
+      }
       __syncwarp();
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (lane + 32 * j < p.groups) gs[lane + 32 * j] = mine[j];
+      __syncwarp();
+    } else {
+      for (int k = 0; k < p.keep; ++k) {    // a kept group's score becomes +inf
+        float v = -INFINITY;
+        int at = p.groups;
+        for (int g = lane; g < p.groups; g += 32)
+          if (gs[g] > v && gs[g] != INFINITY) {
+            v = gs[g];
+            at = g;
+          }
+        argmax_warp(v, at);
+        if (lane == 0 && at < p.groups) gs[at] = INFINITY;
+        __syncwarp();
+      }
     }
     for (int e = lane; e < p.E; e += 32)
       if (gs[e / per] != INFINITY) c[e] = -INFINITY;
     __syncwarp();
   }
-  int mine = 0;
-  for (int k = 0; k < p.top; ++k) {
-    float v = -INFINITY;
-    int at = p.E;
-    for (int e = lane; e < p.E; e += 32)
-      if (c[e] > v) {
-        v = c[e];
-        at = e;
+  auto choose = [&](int k, int e) {
+    const size_t i = static_cast<size_t>(row) * p.top + k;
+    p.weights[i] = sigmoid_f(z[e]) * p.scale;
+    p.id[i] = e;
+  };
+  if (narrow) {
+    for (int e = lane; e < p.E; e += 32) {
+      const float v = c[e];
+      int rank = 0;
+      for (int o = 0; o < p.E; ++o) {
+        const float w = c[o];
+        rank += w > v || (w == v && o < e);
       }
-    argmax_warp(v, at);
-    at = min(at, p.E - 1);
-    if (lane == k) mine = at;
-    if (lane == 0) c[at] = -INFINITY;
-    __syncwarp();
-  }
-  if (lane < p.top) {
-    const size_t i = static_cast<size_t>(row) * p.top + lane;
-    p.weights[i] = sigmoid_f(z[mine]) * p.scale;
-    p.id[i] = mine;
+      if (rank < p.top) choose(rank, e);
+    }
+  } else {
+    int mine = 0;
+    for (int k = 0; k < p.top; ++k) {
+      float v = -INFINITY;
+      int at = p.E;
+      for (int e = lane; e < p.E; e += 32)
+        if (c[e] > v) {
+          v = c[e];
+          at = e;
+        }
+      argmax_warp(v, at);
+      at = min(at, p.E - 1);
+      if (lane == k) mine = at;
+      if (lane == 0) c[at] = -INFINITY;
+      __syncwarp();
+    }
+    if (lane < p.top) choose(lane, mine);
   }
   __syncwarp();
 }

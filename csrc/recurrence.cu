@@ -51,11 +51,29 @@ __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParam
   float xb[8], cb[8];
   vload8(static_cast<const T*>(p.xb) + cc, xb);
   vload8(static_cast<const T*>(p.cb) + cc, cb);
+  // known taps: the state of these channels in registers (neighbours in memory), [channel][input]
+  constexpr int OLD = KT > 1 ? KT - 1 : 1;
+  float old[OLD * 8];
+  if constexpr (KT > 1) {
+#pragma unroll
+    for (int i = 0; i < OLD; ++i) {
+      float f[8] = {};
+      if (off == 0 && !fresh) vload8(st + i * 8, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) old[i * 8 + e] = f[e];
+    }
+  }
   auto input = [&](int at, float (&f)[8]) {          // input at index `at` of the portion
     if (at >= 0) {
       vload8(x + (static_cast<size_t>(row0) + at - off) * p.ld, f);
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] += xb[e];
+    } else if constexpr (KT > 1) {
+#pragma unroll
+      for (int j = 0; j < OLD; ++j)
+        if (j == OLD + at)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = old[e * OLD + j];
     } else {
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] = fresh ? 0.f : st[e * (K - 1) + K - 1 + at];
@@ -110,6 +128,24 @@ __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParam
   __syncthreads();
   if (!in || threadIdx.x >= 32) return;
   const int count = p.cu[s + 1] - p.cu[s];
+  if constexpr (KT > 1) {
+    float now[OLD * 8];
+#pragma unroll
+    for (int j = 0; j < OLD; ++j) {
+      float f[8];
+      input(count - OLD + j, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) now[e * OLD + j] = f[e];
+    }
+#pragma unroll
+    for (int i = 0; i < OLD; ++i) {
+      float f[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = now[i * 8 + e];
+      vstore8(st + i * 8, f);
+    }
+    return;
+  }
   for (int j = 0; j < K - 1; ++j) {                  // in this order an old input is read before its place is written
     float f[8];
     input(count - (K - 1) + j, f);
