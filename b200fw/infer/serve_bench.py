@@ -374,23 +374,26 @@ def ruburax_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     wr, corr = _bf(pad8(E) + 8, W) * 0.05, _bf(E) * 0.1
 
     def route():
-        return ops.router(h, wr, pad8(E), corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"])
+        return ops.router(h, wr, pad8(E), corr, top, ro["groups"]["count"], ro["groups"]["keep"], ro["scale"], joint)
+    joint = sh == F                      # the shared expert is then one more of the experts
     t("router", route, M * (W * 2 + top * 12) + wr.numel() * 2)
     rt = route()[0]
+    E, top = E + int(joint), top + int(joint)
     w_in, w_out = _bf(E, 2, F, W), _bf(E, W, F)
     used = int((rt.offsets[1:] > rt.offsets[:-1]).sum())
     t("expert_glu", lambda: ops.expert_glu(h, w_in, rt), (used * 2 * F * W + M * W + M * top * F) * 2, 4.0 * M * top * F * W)
     act = ops.expert_glu(h, w_in, rt)
     t("expert_down", lambda: ops.expert_down(act, w_out, rt), (used * F * W + M * top * (F + W)) * 2, 2.0 * M * top * F * W)
     rows, sg = ops.expert_down(act, w_out, rt), torch.randn(M, device=DEV)
-    t("moe_norm_add", lambda: ops.moe_norm_add(x, rows, rt, y32, sg, w, 0.5, W, eps), M * W * (14 + 2 * top))
-    gu, act = _bf(2 * sh, W), _bf(M, sh)
-    t("glu_linear (shared)", lambda: ops.glu_linear(h, gu, act), (M * W + 2 * sh * W + M * sh) * 2, 4.0 * M * sh * W)
-    _gemm(t, "gemm shared down (fp32)", M, W, sh, True)
+    sh32, gate = (None, None) if joint else (y32, sg)
+    t("moe_norm_add", lambda: ops.moe_norm_add(x, rows, rt, sh32, gate, w, 0.5, W, eps), M * W * (10 + 2 * top + (0 if joint else 4)))
+    ff = next(l["mlp"]["ff"] for l in mc.layers if l["mlp"]["kind"] == "dense")
+    gu, act = _bf(2 * ff, W), _bf(M, ff)
+    t("glu_linear (dense)", lambda: ops.glu_linear(h, gu, act), (M * W + 2 * ff * W + M * ff) * 2, 4.0 * M * ff * W)
+    _gemm(t, "gemm dense down (fp32)", M, W, ff, True)
     d = mc.side_dim
-    _gemm(t, "gemm token gate", M, d, W)
-    gate, table, ids = _bf(M, d), _bf(V, 4 * d), torch.randint(0, V, (M,), device=DEV)
-    t("gelu_times_token", lambda: ops.gelu_times_token(gate, table, ids, d, V), M * d * 6)
+    wt, table, ids = _bf(d, W), _bf(V, 4 * d), torch.randint(0, V, (M,), device=DEV)
+    t("token_gate", lambda: ops.token_gate(h, wt, table, ids, d, V), (M * W + d * W + 2 * M * d) * 2, 2.0 * M * d * W)
     _gemm(t, "gemm token projection (fp32)", M, W, d, True)
     if lengths is None:
         _gemm(t, "gemm logits (fp32)", M, V, W, True)

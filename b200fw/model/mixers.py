@@ -482,7 +482,8 @@ class GatedFF(nn.Module):
 
 class ExpertFF(nn.Module):
     """Mixture of gated feed-forward experts with sigmoid scores, a learned correction of the choice, a choice limited to the best
-    groups, and a shared expert behind a gate of its own.  Router logits and the shared gate are one 32-bit product."""
+    groups, and a shared expert behind a gate of its own.  Router logits and the shared gate are one 32-bit product.  A shared expert of
+    the experts' size is stored as one more of them, which every token takes."""
 
     def __init__(self, hidden: int, experts: int, inner: int, top: int, groups: int, keep: int, scale: float,
                  shared_inner: Optional[int], dtype, device):
@@ -492,30 +493,33 @@ class ExpertFF(nn.Module):
         if not 1 <= top <= keep * (experts // groups):
             raise ValueError(f"experts: cannot choose {top} among {keep} groups of {experts // groups}")
         self.hidden, self.n, self.inner, self.top, self.groups, self.keep, self.scale = hidden, experts, inner, top, groups, keep, float(scale)
-        self.w_in = _param(experts, 2, pad8(inner), pad8(hidden), dtype=dtype, device=device)
-        self.w_out = _param(experts, pad8(hidden), pad8(inner), dtype=dtype, device=device)
+        self.joint = shared_inner == inner
+        all_ = experts + int(self.joint)
+        self.w_in = _param(all_, 2, pad8(inner), pad8(hidden), dtype=dtype, device=device)
+        self.w_out = _param(all_, pad8(hidden), pad8(inner), dtype=dtype, device=device)
         self.correction = _param(experts, dtype=dtype, device=device)
-        self.shared = GatedFF(hidden, shared_inner, dtype, device) if shared_inner is not None else None
-        self.router = PackedRows(hidden, [("router", 1, experts)] + ([("sg", 1, 1)] if self.shared is not None else []), dtype, device)
+        self.shared = GatedFF(hidden, shared_inner, dtype, device) if shared_inner is not None and not self.joint else None
+        self.router = PackedRows(hidden, [("router", 1, experts)] + ([("sg", 1, 1)] if shared_inner is not None else []), dtype, device)
+        self.shared_row = self.router.sections["sg"][0] if shared_inner is not None else -1
 
     def tensors(self, prefix: str) -> Dict[str, Slot]:
         H, F = self.hidden, self.inner
         t: Dict[str, Slot] = {}
-        for e in range(self.n):
-            p = f"{prefix}e{e}."
+        for e in range(self.n + int(self.joint)):
+            p = f"{prefix}e{e}." if e < self.n else prefix + "shared."
             t[p + "gate"], t[p + "up"] = (Slot(self.w_in.data[e, i, :F, :H], (F, H)) for i in range(2))
             t[p + "down"] = Slot(self.w_out.data[e, :H, :F], (H, F))
         t[prefix + "router"] = self.router.slot("router")
         t[prefix + "correction"] = Slot(self.correction.data, (self.n,))
         if self.shared is not None:
             t |= self.shared.tensors(prefix + "shared.")
+        if self.shared_row >= 0:
             t[prefix + "shared.sg"] = self.router.slot("sg")
         return t
 
     def add(self, x: torch.Tensor, h: torch.Tensor, norm: torch.Tensor, coef: float, n: int, eps: float) -> torch.Tensor:
         """``x += coef * norm(ff(h))``; the new ``x`` in the activation dtype."""
-        r, gate = ops.router(h, self.router.weight, -1 if self.shared is None else self.router.sections["sg"][0], self.correction, self.top,
-                             self.groups, self.keep, self.scale)
+        r, gate = ops.router(h, self.router.weight, self.shared_row, self.correction, self.top, self.groups, self.keep, self.scale, self.joint)
         shared = None if self.shared is None else self.shared.run(h)
         rows = ops.expert_down(ops.expert_glu(h, self.w_in, r), self.w_out, r)
         return ops.moe_norm_add(x, rows, r, shared, gate, norm, coef, n, eps)
@@ -537,7 +541,7 @@ class TokenInput(nn.Module):
 
     def add(self, x: torch.Tensor, h: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, vocab: int, coef: float, n: int,
             eps: float) -> torch.Tensor:
-        g = ops.gelu_times_token(self.gate(h), table, ids, self.first, vocab)
+        g = ops.token_gate(h, self.gate.weight, table, ids, self.first, vocab)
         return ops.norm_add(x, self.proj(g), self.norm, coef, n, eps)
 
 

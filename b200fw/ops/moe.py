@@ -9,7 +9,7 @@ import torch
 
 from .. import _native as nv
 from .gemm import gemm, linear
-from .residual import _f32, glu
+from .residual import _f32, gelu_times_token, glu
 
 
 @dataclass
@@ -26,7 +26,8 @@ class Routing:
         return self.offsets.numel() - 1
 
 
-def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float) -> Routing:
+def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float,
+          joint: Optional[torch.Tensor] = None) -> Routing:
     """``logits [M, >= E]`` fp32, ``correction [E]``: scores ``s = sigmoid(logits)``; the experts are ``groups`` equal groups of
     neighbours, a group counts by the sum of its two largest ``s + correction``, and the ``top`` largest ``s + correction`` of the
     ``keep`` best groups are chosen, with weight ``s * scale``.  Ties go to the lower index."""
@@ -41,18 +42,24 @@ def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int,
             open_ = torch.zeros(M, groups, dtype=torch.bool).scatter_(1, best, True)
             c = c.masked_fill(~open_.repeat_interleave(per, 1), float("-inf"))
         ids = c.sort(dim=-1, descending=True, stable=True).indices[:, :top]
+        weights = s.gather(1, ids) * scale
+        if joint is not None:
+            ids, weights = torch.cat([ids, torch.full((M, 1), E)], 1), torch.cat([weights, torch.sigmoid(joint)[:, None]], 1)
+            E, top = E + 1, top + 1
         flat = ids.reshape(-1)
         order = flat.sort(stable=True).indices
         place = torch.empty(M * top, dtype=torch.int32)
         place[order] = torch.arange(M * top, dtype=torch.int32)
         offsets = torch.zeros(E + 1, dtype=torch.int32)
         offsets[1:] = torch.bincount(flat, minlength=E).cumsum(0)
-        return Routing(s.gather(1, ids) * scale, place.reshape(M, top), (order // top).to(torch.int32), offsets)
-    r, work = _routing(M, E, top, logits.device)
+        return Routing(weights, place.reshape(M, top), (order // top).to(torch.int32), offsets)
+    more = int(joint is not None)
+    r, work = _routing(M, E + more, top + more, logits.device)
     nv.check(nv.lib().b2_moe_route(
-        nv.ptr(logits), nv.ctypes.c_longlong(logits.stride(0)), nv.ptr(correction), nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token),
+        nv.ptr(logits), nv.ctypes.c_longlong(logits.stride(0)), nv.ptr(joint), nv.ctypes.c_longlong(joint.stride(0) if more else 0), more,
+        nv.ptr(correction), nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token),
         nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep, nv.ctypes.c_float(scale), _f32(correction), nv.stream_ptr()), "moe_route")
-    nv.count_launch(2 if M * top <= 16384 else 3)
+    nv.count_launch(2 if M * (top + more) <= 16384 else 3)
     return r
 
 
@@ -62,21 +69,25 @@ def _routing(M: int, E: int, top: int, dev):
     return r, torch.empty(E + M * top, device=dev, dtype=torch.int32)      # rows per expert, then the expert of every pair
 
 
-def router(h: torch.Tensor, w: torch.Tensor, shared_row: int, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float):
+def router(h: torch.Tensor, w: torch.Tensor, shared_row: int, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float,
+           joint: bool = False):
     """Router product in 32-bit and :func:`route`: ``h [M, K]``, ``w [>= E, K]`` with the experts' rows first; ``shared_row >= 0``: that
-    row's product is the shared expert's gate.  Returns ``(Routing, gate [M] or None)``."""
+    row's product is the shared expert's gate, ``joint``: of a shared expert that is expert E.  Returns ``(Routing, gate [M])``, the gate
+    None without a shared expert and with a joint one."""
     M, E, N = h.shape[0], correction.numel(), w.shape[0]
     if not h.is_cuda or h.dtype != torch.bfloat16 or N > SKINNY:
         z = linear_fp32(h, w)
-        return route(z, correction, top, groups, keep, scale), None if shared_row < 0 else z[:, shared_row]
-    r, work = _routing(M, E, top, h.device)
-    gate = torch.empty(M, device=h.device, dtype=torch.float32) if shared_row >= 0 else None
+        gate = None if shared_row < 0 else z[:, shared_row]
+        return route(z, correction, top, groups, keep, scale, gate if joint else None), None if joint else gate
+    more = int(joint)
+    r, work = _routing(M, E + more, top + more, h.device)
+    gate = torch.empty(M, device=h.device, dtype=torch.float32) if shared_row >= 0 and not joint else None
     cl = nv.ctypes.c_longlong
     nv.check(nv.lib().b2_moe_router(
-        nv.ptr(h), cl(h.stride(0)), nv.ptr(w), cl(w.stride(0)), N, h.shape[1], shared_row, nv.ptr(gate), nv.ptr(correction),
-        nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep,
+        nv.ptr(h), cl(h.stride(0)), nv.ptr(w), cl(w.stride(0)), N, h.shape[1], shared_row, nv.ptr(gate), more,
+        nv.ptr(correction), nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep,
         nv.ctypes.c_float(scale), nv.stream_ptr()), "moe_router")
-    nv.count_launch(2 if M * top <= 16384 else 3)
+    nv.count_launch(2 if M * (top + more) <= 16384 else 3)
     return r, gate
 
 
@@ -94,6 +105,19 @@ def linear_fp32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
                                 x.shape[1], nv.stream_ptr()), "skinny")
     nv.count_launch()
     return z
+
+
+def token_gate(h: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, first: int, vocab: int) -> torch.Tensor:
+    """``gelu_tanh(h w^T) * table[ids, first : first + N]``, ``w [N, K]``."""
+    M, N = h.shape[0], w.shape[0]
+    if not h.is_cuda or h.dtype != torch.bfloat16 or M > 1024:
+        return gelu_times_token(linear(h, w), table, ids, first, vocab)
+    out = torch.empty((M, N), device=h.device, dtype=h.dtype)
+    cl = nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_token_gate(nv.ptr(h), cl(h.stride(0)), nv.ptr(w), cl(w.stride(0)), nv.ptr(table), cl(table.stride(0)), nv.ptr(ids),
+                                    nv.ptr(out), M, N, h.shape[1], first, vocab, nv.stream_ptr()), "token_gate")
+    nv.count_launch()
+    return out
 
 
 def glu_linear(h: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
@@ -157,7 +181,7 @@ def moe_norm_add(x: torch.Tensor, rows: torch.Tensor, r: Routing, shared: Option
         return x if w.dtype == torch.float32 else x.to(w.dtype)
     h = None if w.dtype == torch.float32 else torch.empty(x.shape, device=x.device, dtype=w.dtype)
     nv.check(nv.lib().b2_moe_norm_add(
-        nv.ptr(x), nv.ptr(rows), nv.ptr(r.place), nv.ptr(r.weights), r.place.shape[1], nv.ptr(shared), nv.ptr(shared_gate),
+        nv.ptr(x), nv.ptr(rows), nv.ptr(r.place), nv.ptr(r.weights), r.place.shape[1], rows.shape[0], nv.ptr(shared), nv.ptr(shared_gate),
         0 if shared_gate is None else shared_gate.stride(0), nv.ptr(w), nv.ptr(h), x.shape[0], x.shape[1], n, nv.ctypes.c_float(coef),
         nv.ctypes.c_float(eps), _f32(w), nv.stream_ptr()), "moe_norm_add")
     nv.count_launch()

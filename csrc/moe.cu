@@ -24,9 +24,10 @@ typedef __nv_bfloat16 moe_bf16;
 // ---- routing -----------------------------------------------------------------------------------------------------------
 struct RouteParams {
   const void* corr;      // T [E]
-  float* weights;        // [M, top]
-  int* id;               // [M, top]
+  float* weights;        // [M, slots]
+  int* id;               // [M, slots]
   int M, E, top, groups, keep;
+  int slots;             // top, or one more: expert E, which every token takes behind a gate of its own
   float scale;
 };
 
@@ -43,9 +44,10 @@ __device__ __forceinline__ void argmax_warp(float& v, int& i) {
   }
 }
 
-// The choice of one token by a warp.  z: its logits; c, gs: E floats of shared memory each (choice and group scores).
+// The choice of one token by a warp.  z: its logits; sg: the logit of the gate (slots > top); c, gs: E floats of shared memory each
+// (choice and group scores).
 template <typename T>
-__device__ __forceinline__ void route_token(const RouteParams& p, int row, const float* z, float* c, float* gs) {
+__device__ __forceinline__ void route_token(const RouteParams& p, int row, const float* z, const float* sg, float* c, float* gs) {
   const int lane = threadIdx.x & 31;
   constexpr float LOW = -3.0e38f;           // in place of what is no number (rows without a sequence): below any score, above "closed"
   for (int e = lane; e < p.E; e += 32) {
@@ -103,11 +105,15 @@ __device__ __forceinline__ void route_token(const RouteParams& p, int row, const
       if (gs[e / per] != INFINITY) c[e] = -INFINITY;
     __syncwarp();
   }
+  const size_t first = static_cast<size_t>(row) * p.slots;
   auto choose = [&](int k, int e) {
-    const size_t i = static_cast<size_t>(row) * p.top + k;
-    p.weights[i] = sigmoid_f(z[e]) * p.scale;
-    p.id[i] = e;
+    p.weights[first + k] = sigmoid_f(z[e]) * p.scale;
+    p.id[first + k] = e;
   };
+  if (p.slots > p.top && lane == 31) {
+    p.weights[first + p.top] = sigmoid_f(*sg);
+    p.id[first + p.top] = p.E;
+  }
   if (narrow) {
     for (int e = lane; e < p.E; e += 32) {
       const float v = c[e];
@@ -142,29 +148,39 @@ __device__ __forceinline__ void route_token(const RouteParams& p, int row, const
 // Logits given: a warp per token.
 constexpr int MR_WARPS = 4;
 template <typename T>
-__global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RouteParams p, const float* __restrict__ z, long long ld) {
+__global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RouteParams p, const float* __restrict__ z, long long ld,
+                                                                   const float* __restrict__ sg, long long ld_sg) {
   extern __shared__ float mr_smem[];
   const int warp = threadIdx.x >> 5, row = blockIdx.x * MR_WARPS + warp;
   if (row >= p.M) return;
   float* c = mr_smem + warp * 2 * p.E;
-  route_token<T>(p, row, z + static_cast<size_t>(row) * ld, c, c + p.E);
+  route_token<T>(p, row, z + static_cast<size_t>(row) * ld, sg + static_cast<size_t>(row) * ld_sg, c, c + p.E);
 }
 
-// Products with few outputs (router logits, gates), bf16 operands and a 32-bit result: 16 rows a CTA, its warps split the contraction.
-// A lane loads eight neighbouring elements of its row of either operand at once and uses them as the fragments of two m16n8k16
-// products: the order of the contraction is free as long as both operands agree on it.  ROUTE: the rows' experts are chosen on the spot.
+// Products with few outputs or few rows (router logits, gates), bf16 operands and a 32-bit result: 16 rows and up to 72 columns a CTA,
+// whose warps split the contraction.  A lane loads eight neighbouring elements of its row of either operand at once and uses them as the fragments of two m16n8k16
+// products: the order of the contraction is free as long as both operands agree on it.  SK_ROUTE: the rows' experts are chosen on the
+// spot.  SK_TOKEN: the result goes through gelu and times a vector of the row's token, rounded to bf16.
+enum : int { SK_PLAIN = 0, SK_ROUTE = 1, SK_TOKEN = 2 };
 struct SkinnyParams {
   const moe_bf16* h;     // [M, ld_h]
   const moe_bf16* w;     // [N, ld_w]
-  float* z;              // [M, ld_z]; ROUTE: only column sg is stored (sg < 0: none)
+  float* z;              // [M, ld_z]; ROUTE: only column sg is stored, if at all (null, or sg < 0)
   long long ld_h, ld_w, ld_z;
   int M, N, K, sg;
+  const moe_bf16* table; // SK_TOKEN: [vocab, ld_table], columns first .. first + N - 1
+  const long long* ids;  // [M]
+  moe_bf16* out;         // [M, N]
+  long long ld_table;
+  int first, vocab;
 };
 constexpr int SK_ROWS = 16, SK_WARPS = 8, SK_MAX_TILES = 9;
 
-template <int NT, bool ROUTE>
+template <int NT, int FORM>
 __global__ void __launch_bounds__(SK_WARPS * 32) skinny_kernel(const SkinnyParams p, const RouteParams r) {
   constexpr int NP = NT * 8, LD = NP + 2;
+  constexpr bool ROUTE = FORM == SK_ROUTE;
+  const int n0 = blockIdx.y * NP;
   __shared__ float part[SK_WARPS][SK_ROWS][LD];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3, m0 = blockIdx.x * SK_ROWS;
   const moe_bf16* a0 = p.h + static_cast<size_t>(min(m0 + g, p.M - 1)) * p.ld_h;
@@ -182,7 +198,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) skinny_kernel(const SkinnyParam
     uint4 w[NT];
 #pragma unroll
     for (int n = 0; n < NT; ++n)
-      w[n] = in && n * 8 + g < p.N ? *reinterpret_cast<const uint4*>(p.w + static_cast<size_t>(n * 8 + g) * p.ld_w + k) : zero;
+      w[n] = in && n0 + n * 8 + g < p.N ? *reinterpret_cast<const uint4*>(p.w + static_cast<size_t>(n0 + n * 8 + g) * p.ld_w + k) : zero;
     const uint32_t f0[4] = {x0.x, x1.x, x0.y, x1.y}, f1[4] = {x0.z, x1.z, x0.w, x1.w};
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
@@ -203,12 +219,21 @@ __global__ void __launch_bounds__(SK_WARPS * 32) skinny_kernel(const SkinnyParam
 #pragma unroll
     for (int w = 0; w < SK_WARPS; ++w) s += part[w][row][c];
     if (ROUTE) part[0][row][c] = s;          // read by this thread alone until the barrier
-    if (m0 + row < p.M && (ROUTE ? c == p.sg : c < p.N)) p.z[static_cast<size_t>(m0 + row) * p.ld_z + (ROUTE ? 0 : c)] = s;
+    if (FORM == SK_TOKEN) {
+      if (m0 + row < p.M && n0 + c < p.N) {
+        const long long id = p.ids[m0 + row];
+        const float t = id >= 0 && id < p.vocab ? to_f(p.table[id * p.ld_table + p.first + n0 + c]) : 0.f;
+        p.out[static_cast<size_t>(m0 + row) * p.N + n0 + c] = from_f<moe_bf16>(gelu_tanh_t<moe_bf16>(s) * t);
+      }
+      continue;
+    }
+    if (m0 + row < p.M && (ROUTE ? c == p.sg && p.z != nullptr : n0 + c < p.N)) p.z[static_cast<size_t>(m0 + row) * p.ld_z + (ROUTE ? 0 : n0 + c)] = s;
   }
   if (!ROUTE) return;
   __syncthreads();
   for (int row = warp; row < SK_ROWS && m0 + row < p.M; row += SK_WARPS)
-    route_token<moe_bf16>(r, m0 + row, part[0][row], part[1 + (warp >> 1)][(warp & 1) * 8], part[1 + (warp >> 1)][(warp & 1) * 8 + 1]);
+    route_token<moe_bf16>(r, m0 + row, part[0][row], &part[0][row][max(p.sg, 0)], part[1 + (warp >> 1)][(warp & 1) * 8],
+                          part[1 + (warp >> 1)][(warp & 1) * 8 + 1]);
 }
 
 // Running sums of f(i) over i < n by a whole warp: out[0 .. n].
@@ -231,10 +256,16 @@ __device__ __forceinline__ void warp_prefix(int n, int* out, F f) {
   if (lane == 0) out[n] = carry;
 }
 
+// An index that came from memory and is outside its range: recorded, and the access left out.
+__device__ __forceinline__ bool moe_bad(bool bad, int* status) {
+  if (bad) atomicCAS(status, 0, ERR_BAD_ARGUMENT);
+  return bad;
+}
+
 // The layout of the (token, choice) pairs.  Up to MP_ONE pairs: one CTA counts in shared memory.
 constexpr int MP_THREADS = 1024, MP_EACH = 16, MP_ONE = MP_THREADS * MP_EACH;
 __global__ void __launch_bounds__(MP_THREADS) moe_place_kernel(const int* __restrict__ id, int* __restrict__ place, int* __restrict__ token,
-                                                               int* __restrict__ offsets, int E, int top, int total) {
+                                                               int* __restrict__ offsets, int E, int top, int total, int* status) {
   __shared__ int cnt[MOE_MAX_EXPERTS], off[MOE_MAX_EXPERTS + 1];
   for (int e = threadIdx.x; e < E; e += MP_THREADS) cnt[e] = 0;
   __syncthreads();
@@ -243,6 +274,7 @@ __global__ void __launch_bounds__(MP_THREADS) moe_place_kernel(const int* __rest
   for (int j = 0; j < MP_EACH; ++j) {
     const int i = threadIdx.x + j * MP_THREADS;
     e[j] = i < total ? id[i] : 0;
+    if (moe_bad(e[j] < 0 || e[j] >= E, status)) e[j] = 0;
   }
 #pragma unroll
   for (int j = 0; j < MP_EACH; ++j)
@@ -263,8 +295,8 @@ __global__ void __launch_bounds__(MP_THREADS) moe_place_kernel(const int* __rest
 
 // More pairs: every CTA counts its own, takes its places among the experts' rows (count, zero before), then the same once the counts
 // are complete.
-__global__ void __launch_bounds__(256) moe_rank_kernel(const int* __restrict__ id, int* __restrict__ place, int* __restrict__ count, int E,
-                                                       int total) {
+__global__ void __launch_bounds__(256) moe_rank_kernel(int* __restrict__ id, int* __restrict__ place, int* __restrict__ count, int E,
+                                                       int total, int* status) {
   __shared__ int cnt[MOE_MAX_EXPERTS];
   for (int e = threadIdx.x; e < E; e += 256) cnt[e] = 0;
   __syncthreads();
@@ -274,6 +306,7 @@ __global__ void __launch_bounds__(256) moe_rank_kernel(const int* __restrict__ i
     const int i = (blockIdx.x * 4 + j) * 256 + threadIdx.x;
     if (i < total) {
       e[j] = id[i];
+      if (moe_bad(e[j] < 0 || e[j] >= E, status)) id[i] = e[j] = 0;
       rank[j] = atomicAdd(cnt + e[j], 1);
     }
   }
@@ -288,14 +321,16 @@ __global__ void __launch_bounds__(256) moe_rank_kernel(const int* __restrict__ i
   }
 }
 __global__ void __launch_bounds__(256) moe_layout_kernel(const int* __restrict__ count, const int* __restrict__ id, int* __restrict__ place,
-                                                         int* __restrict__ token, int* __restrict__ offsets, int E, int top, int total) {
+                                                         int* __restrict__ token, int* __restrict__ offsets, int E, int top, int total,
+                                                         int* status) {
   __shared__ int off[MOE_MAX_EXPERTS + 1];
   if (threadIdx.x < 32) warp_prefix(E, off, [&](int e) { return count[e]; });
   __syncthreads();
   if (blockIdx.x == 0)
     for (int e = threadIdx.x; e <= E; e += 256) offsets[e] = off[e];
   for (int i = blockIdx.x * 256 + threadIdx.x; i < total; i += gridDim.x * 256) {
-    const int r = off[id[i]] + place[i];
+    int r = off[id[i]] + place[i];
+    if (moe_bad(r < 0 || r >= total, status)) r = 0;
     place[i] = r;
     token[r] = i / top;
   }
@@ -439,7 +474,9 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
-  const int ncols = (p.N + COLS - 1) / COLS, tiles = first[p.E] * ncols, nkb = (p.K + MG_BK - 1) / MG_BK;
+  const bool sound = off[0] == 0 && off[p.E] == p.P;           // else nothing is computed
+  if (tid == 0) moe_bad(!sound, status);
+  const int ncols = (p.N + COLS - 1) / COLS, tiles = sound ? first[p.E] * ncols : 0, nkb = (p.K + MG_BK - 1) / MG_BK;
 
   if (warp == 0) {
     // Lane l gathers rows 4 l .. 4 l + 3 of a tile; a group that reaches past the expert's last row repeats it, groups further on keep
@@ -586,9 +623,11 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
 
 // rows[r] = h[token[r]], a warp per row (16 bytes a lane)
 __global__ void __launch_bounds__(256) moe_gather_kernel(const moe_bf16* __restrict__ h, long long ld, const int* __restrict__ token,
-                                                         moe_bf16* __restrict__ rows, int P, int K) {
+                                                         moe_bf16* __restrict__ rows, int tokens, int P, int K, int* status) {
   for (int r = blockIdx.x * 8 + (threadIdx.x >> 5); r < P; r += gridDim.x * 8) {
-    const uint4* src = reinterpret_cast<const uint4*>(h + static_cast<size_t>(token[r]) * ld);
+    const int from = token[r];
+    if (moe_bad(from < 0 || from >= tokens, status)) continue;
+    const uint4* src = reinterpret_cast<const uint4*>(h + static_cast<size_t>(from) * ld);
     uint4* dst = reinterpret_cast<uint4*>(rows + static_cast<size_t>(r) * K);
     const int n = K / 8;
     for (int c0 = threadIdx.x & 31; c0 < n; c0 += 128) {
@@ -613,8 +652,9 @@ struct MoeAddParams {
   const float* sg;       // [M], stride ld_sg: gate before its sigmoid
   const void* w;         // T [ld]
   void* h;               // T [M, ld] or null
-  int top, ld_sg, ld, n;
+  int top, P, ld_sg, ld, n;
   float coef, eps;
+  int* status;
 };
 
 __device__ __forceinline__ float moe_block_sum(float v, float* scratch) {
@@ -632,7 +672,8 @@ __global__ void __launch_bounds__(MAXT) moe_norm_add_kernel(const MoeAddParams p
   const size_t base = static_cast<size_t>(blockIdx.x) * p.ld;
   if (static_cast<int>(threadIdx.x) < p.top) {
     sw[threadIdx.x] = p.weights[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
-    sr[threadIdx.x] = p.place[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
+    const int r = p.place[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
+    sr[threadIdx.x] = moe_bad(r < 0 || r >= p.P, p.status) ? 0 : r;
   }
   const float g = p.shared ? sigmoid_f(p.sg[static_cast<size_t>(blockIdx.x) * p.ld_sg]) : 0.f;
   __syncthreads();
@@ -739,50 +780,63 @@ static int moe_columns(int P, int E, int N, int widest, int narrowest) {
 
 using namespace b2;
 
-static bool bad_routing(int M, int E, int top, int groups, int keep) {
-  if (E < 1 || E > MOE_MAX_EXPERTS || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > MOE_MAX_TOP ||
-      top > keep * (E / groups) || static_cast<long long>(M) * top > 0x7fffffffll) {
-    set_error("moe_route: up to %d experts in equal groups and up to %d chosen required", MOE_MAX_EXPERTS, MOE_MAX_TOP);
+static bool bad_routing(int M, int E, int top, int groups, int keep, int slots) {
+  if (E < 1 || E + 1 > MOE_MAX_EXPERTS || (slots != top && slots != top + 1) || slots > MOE_MAX_TOP || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 || top > MOE_MAX_TOP ||
+      top > keep * (E / groups) || static_cast<long long>(M) * slots > 0x7fffffffll) {
+    set_error("moe_route: fewer than %d experts in equal groups and up to %d chosen required", MOE_MAX_EXPERTS, MOE_MAX_TOP);
     return true;
   }
   return false;
 }
 
-// work: [E] counts, then [M * top] chosen experts
+// work: [E] counts, then [M * top] chosen experts (both with the expert that every token takes, if there is one)
 static int launch_place(int* place, int* token, int* offsets, int* work, int M, int E, int top, cudaStream_t st) {
   const int total = M * top;
-  int* id = work + E;
+  int *id = work + E, *status = status_ptr();
+  if (!status) return 3;
   if (total <= MP_ONE) {
-    moe_place_kernel<<<1, MP_THREADS, 0, st>>>(id, place, token, offsets, E, top, total);
+    moe_place_kernel<<<1, MP_THREADS, 0, st>>>(id, place, token, offsets, E, top, total, status);
     B2_CHECK_LAUNCH("moe_place");
     return 0;
   }
   if (cudaMemsetAsync(work, 0, sizeof(int) * E, st) != cudaSuccess) { set_error("moe_place: clearing the counts failed"); return 5; }
-  moe_rank_kernel<<<(total + 1023) / 1024, 256, 0, st>>>(id, place, work, E, total);
+  moe_rank_kernel<<<(total + 1023) / 1024, 256, 0, st>>>(id, place, work, E, total, status);
   B2_CHECK_LAUNCH("moe_rank");
-  moe_layout_kernel<<<2 * num_sms(), 256, 0, st>>>(work, id, place, token, offsets, E, top, total);
+  moe_layout_kernel<<<2 * num_sms(), 256, 0, st>>>(work, id, place, token, offsets, E, top, total, status);
   B2_CHECK_LAUNCH("moe_layout");
   return 0;
 }
 
-// z: fp32 [M, ld]; work: int32 [E + M * top]; offsets: int32 [E + 1]; place: int32 [M, top]; token: int32 [M * top].
-B2_EXPORT int b2_moe_route(const float* z, long long ld, const void* corr, float* weights, int* place, int* token, int* offsets,
-                           int* work, int M, int E, int top, int groups, int keep, float scale, int is_f32, void* stream) {
+// z: fp32 [M, ld]; work: int32 [E + M * top]; offsets: int32 [E + 1]; place: int32 [M, top]; token: int32 [M * top].  joint: every token
+// also takes expert E, with the weight sigmoid(sg) (fp32 [M], stride ld_sg); then one more expert and choice in all of these.
+B2_EXPORT int b2_moe_route(const float* z, long long ld, const float* sg, long long ld_sg, int joint, const void* corr, float* weights,
+                           int* place, int* token, int* offsets, int* work, int M, int E, int top, int groups, int keep, float scale,
+                           int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
-  if (bad_routing(M, E, top, groups, keep)) return 10;
+  const int slots = top + (joint ? 1 : 0), all = E + (joint ? 1 : 0);
+  if (bad_routing(M, E, top, groups, keep, slots)) return 10;
+  if (joint && sg == nullptr) { set_error("moe_route: the joint expert needs its gate"); return 10; }
   if (ld < E) { set_error("moe_route: a logit per expert required"); return 10; }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const RouteParams p = {corr, weights, work + E, M, E, top, groups, keep, scale};
-  B2_DISPATCH_T(is_f32, moe_route_kernel<T><<<(M + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, MR_WARPS * 2 * E * sizeof(float), st>>>(p, z, ld););
+  const RouteParams p = {corr, weights, work + all, M, E, top, groups, keep, slots, scale};
+  B2_DISPATCH_T(is_f32, moe_route_kernel<T><<<(M + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, MR_WARPS * 2 * E * sizeof(float), st>>>(
+      p, z, ld, sg, ld_sg););
   B2_CHECK_LAUNCH("moe_route");
-  return launch_place(place, token, offsets, work, M, E, top, st);
+  return launch_place(place, token, offsets, work, M, all, slots, st);
 }
 
-template <bool ROUTE>
+template <int FORM>
 static int launch_skinny(const SkinnyParams& p, const RouteParams& r, cudaStream_t st) {
-  const int grid = (p.M + SK_ROWS - 1) / SK_ROWS, nt = (p.N + 7) / 8;
-#define B2_SKINNY(V) case V: skinny_kernel<V, ROUTE><<<grid, SK_WARPS * 32, 0, st>>>(p, r); break
+  const int nt = (p.N + 7) / 8;
+  const dim3 wide((p.M + SK_ROWS - 1) / SK_ROWS, (p.N + 63) / 64), grid(wide.x);
+  if (FORM == SK_TOKEN) {
+    if (p.N <= 32) skinny_kernel<4, FORM><<<grid, SK_WARPS * 32, 0, st>>>(p, r);
+    else skinny_kernel<8, FORM><<<wide, SK_WARPS * 32, 0, st>>>(p, r);
+    B2_CHECK_LAUNCH("skinny");
+    return 0;
+  }
+#define B2_SKINNY(V) case V: skinny_kernel<V, FORM><<<grid, SK_WARPS * 32, 0, st>>>(p, r); break
   switch (nt) {
     B2_SKINNY(1); B2_SKINNY(2); B2_SKINNY(3); B2_SKINNY(4); B2_SKINNY(5); B2_SKINNY(6); B2_SKINNY(7); B2_SKINNY(8); B2_SKINNY(9);
     default: set_error("skinny: up to %d outputs", SK_MAX_TILES * 8); return 10;
@@ -798,27 +852,43 @@ B2_EXPORT int b2_skinny(const void* h, long long ld_h, const void* w, long long 
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (N < 1 || K < 8 || K % 8 || ld_h % 8 || ld_w % 8 || ld_z < N) { set_error("skinny: contraction and strides in multiples of 8 required"); return 10; }
-  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), z, ld_h, ld_w, ld_z, M, N, K, -1};
-  return launch_skinny<false>(p, RouteParams{}, static_cast<cudaStream_t>(stream));
+  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), z, ld_h, ld_w, ld_z, M, N, K, -1, nullptr, nullptr, nullptr, 0, 0, 0};
+  return launch_skinny<SK_PLAIN>(p, RouteParams{}, static_cast<cudaStream_t>(stream));
 }
 
-// Router product and choice in one kernel, N = E router rows and what follows them in w (up to 72 rows); sg >= 0: row sg's product goes
-// to sg_out fp32 [M].  The rest as b2_moe_route.
+// out bf16 [M, N] = gelu_tanh(h w^T) * table[ids, first ...]: for few rows; ids outside the vocabulary give zeros
+B2_EXPORT int b2_token_gate(const void* h, long long ld_h, const void* w, long long ld_w, const void* table, long long ld_table,
+                            const long long* ids, void* out, int M, int N, int K, int first, int vocab, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (N < 1 || K < 8 || K % 8 || ld_h % 8 || ld_w % 8 || first < 0 || first + N > ld_table) {
+    set_error("token_gate: contraction and strides in multiples of 8 required");
+    return 10;
+  }
+  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), nullptr, ld_h, ld_w, 0, M, N, K, -1,
+                          static_cast<const moe_bf16*>(table), ids, static_cast<moe_bf16*>(out), ld_table, first, vocab};
+  return launch_skinny<SK_TOKEN>(p, RouteParams{}, static_cast<cudaStream_t>(stream));
+}
+
+// Router product and choice in one kernel, N = E router rows and what follows them in w (up to 72 rows); sg >= 0: row sg's product is
+// the gate of the joint expert, or goes to sg_out fp32 [M].  The rest as b2_moe_route.
 B2_EXPORT int b2_moe_router(const void* h, long long ld_h, const void* w, long long ld_w, int N, int K, int sg, float* sg_out,
-                            const void* corr, float* weights, int* place, int* token, int* offsets, int* work, int M, int E, int top,
+                            int joint, const void* corr, float* weights, int* place, int* token, int* offsets, int* work, int M, int E, int top,
                             int groups, int keep, float scale, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
-  if (bad_routing(M, E, top, groups, keep)) return 10;
-  if (N < E || N > SK_MAX_TILES * 8 || K < 8 || K % 8 || ld_h % 8 || ld_w % 8 || sg >= N || (sg >= 0 && sg_out == nullptr)) {
+  const int slots = top + (joint ? 1 : 0), all = E + (joint ? 1 : 0);
+  if (bad_routing(M, E, top, groups, keep, slots)) return 10;
+  if (N < E || N > SK_MAX_TILES * 8 || K < 8 || K % 8 || ld_h % 8 || ld_w % 8 || sg >= N || (sg >= 0 && !joint && sg_out == nullptr) ||
+      (joint && sg < 0)) {
     set_error("moe_router: up to %d outputs, contraction and strides in multiples of 8 required", SK_MAX_TILES * 8);
     return 10;
   }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), sg_out, ld_h, ld_w, 1, M, N, K, sg};
-  const RouteParams r = {corr, weights, work + E, M, E, top, groups, keep, scale};
-  if (const int rc = launch_skinny<true>(p, r, st)) return rc;
-  return launch_place(place, token, offsets, work, M, E, top, st);
+  const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), sg_out, ld_h, ld_w, 1, M, N, K, sg, nullptr, nullptr, nullptr, 0, 0, 0};
+  const RouteParams r = {corr, weights, work + all, M, E, top, groups, keep, slots, scale};
+  if (const int rc = launch_skinny<SK_ROUTE>(p, r, st)) return rc;
+  return launch_place(place, token, offsets, work, M, all, slots, st);
 }
 
 // h: T [tokens, ld], w: T [E, 2, F, K], token: int32 [P] -> out T [P, F].  rows (bf16 [P, K], or null): room for the rows expert after
@@ -846,7 +916,7 @@ B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* 
   if (rows != nullptr) {
     const int blocks = (P + 7) / 8;
     moe_gather_kernel<<<blocks < 16 * num_sms() ? blocks : 16 * num_sms(), 256, 0, st>>>(static_cast<const moe_bf16*>(h), ld, token,
-                                                                                        static_cast<moe_bf16*>(rows), P, K);
+                                                                                        static_cast<moe_bf16*>(rows), tokens, P, K, status_ptr());
     B2_CHECK_LAUNCH("moe_gather");
     return launch_glu<ROWS_GLU>(tensor_map_2d_bf16(rows, P, K, K, MG_BM, MG_BK), w, p, moe_columns(P, E, F, 128, 32), moe_bound(P, E, MG_BM),
                                 st);
@@ -898,7 +968,7 @@ B2_EXPORT int b2_moe_down(const void* a, const void* w, const int* offsets, void
   return launch_moe<64, MOE_DOWN>(ta, tb, p, bound, st);
 }
 
-B2_EXPORT int b2_moe_norm_add(float* x, const void* rows, const int* place, const float* weights, int top, const float* shared,
+B2_EXPORT int b2_moe_norm_add(float* x, const void* rows, const int* place, const float* weights, int top, int P, const float* shared,
                               const float* sg, int ld_sg, const void* w, void* h, int M, int ld, int n, float coef, float eps,
                               int is_f32, void* stream) {
   b2::ensure_thread_context();
@@ -907,7 +977,7 @@ B2_EXPORT int b2_moe_norm_add(float* x, const void* rows, const int* place, cons
     set_error("moe_norm_add: ld %% 8 == 0, 0 < n <= ld <= 32768 and up to %d rows a token required", MOE_MAX_TOP);
     return 10;
   }
-  const MoeAddParams p = {x, rows, place, weights, shared, sg, w, h, top, ld_sg, ld, n, coef, eps};
+  const MoeAddParams p = {x, rows, place, weights, shared, sg, w, h, top, P, ld_sg, ld, n, coef, eps, status_ptr()};
   const int pieces = ld / 8, V = pieces <= 256 ? 1 : pieces <= 512 ? 2 : 4;
   const int threads = ((pieces + V - 1) / V + 31) / 32 * 32;
   cudaStream_t st = static_cast<cudaStream_t>(stream);

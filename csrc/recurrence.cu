@@ -382,7 +382,8 @@ __global__ void __launch_bounds__(RG_THREADS) rec_gates_kernel(const __grid_cons
   const int ch = b * p.block + (in ? c : 0);
   const RecChannel<rg_bf16> K(p, ch);
   const uint32_t at = tmem + (static_cast<uint32_t>(quarter * 32) << 16) + run * GR_RUN;
-  const int u_at = (c >> 6) * 8192 + (c & 7) * 2, u_piece = (c >> 3) & 7;
+  const int cu = in ? c : 0;                         // lanes past the block's last channel read the first one's
+  const int u_at = (cu >> 6) * 8192 + (cu & 7) * 2, u_piece = (cu >> 3) & 7;
   int it = 0;
   for (int chunk = blockIdx.y; chunk < nchunks; chunk += stride, ++it) {
     const int st = it & 1;

@@ -62,7 +62,7 @@ STRETCH = (5.0, 1.0, 3.0, 40)
 ODD = config(42, 67, [
     rglru(27, 3, 5, ff=moe(6, 3, 10, (3, 2), 14)), attention(6, 2, 18, 10, rot(10, 300.0, STRETCH)),
     parallel(att(3, 1, 10, 21, rot(4)), 3, 11, 6, 9.0, 0.8, -1.4, ff=dense(21)), attention(4, 2, 18, 10, rot(10, 300.0, STRETCH), kv_from=1, ff=moe(9, 2, 12)),
-    rglru(20, 1, 2, ff=moe(5, 2, 9, (5, 3), 7, 3.0)), attention(2, 2, 18, 10, rot(10, 300.0, STRETCH), kv_from=1, scale=0.5, ff=dense(13))], side=5)
+    rglru(20, 1, 2, ff=moe(5, 2, 9, (5, 3), 9, 3.0)), attention(2, 2, 18, 10, rot(10, 300.0, STRETCH), kv_from=1, scale=0.5, ff=dense(13))], side=5)
 # every head with its own key, unit constants, no token input, one tap, as many experts as are chosen
 PLAIN = config(64, 96, [attention(4, 4, 32, 32, rot(32), ff=moe(4, 4, 24)), parallel(att(2, 2, 16, 32, rot(0)), 2, 32, 32, 3.0, 1.0, 1.0, ff=dense(48)),
                         rglru(64, 4, 1, ff=moe(8, 1, 40, (2, 1), 16, 1.0))], eps=1e-3, mult=1.0, logit=1.0, side=None)
@@ -70,7 +70,7 @@ PLAIN = config(64, 96, [attention(4, 4, 32, 32, rot(32), ff=moe(4, 4, 24)), para
 WIDE = config(96, 80, [attention(18, 1, 128, 96, rot(64, 5e4, (8.0, 1.0, 4.0, 64)), scale=0.09, ff=dense(200)),
                        parallel(att(4, 2, 128, 128, rot(128)), 2, 128, 64, 15.0, 0.5, 0.9, ff=moe(16, 4, 72, (4, 2), 136)),
                        attention(2, 1, 128, 96, rot(64, 5e4, (8.0, 1.0, 4.0, 64)), scale=0.09, kv_from=0, ff=moe(40, 6, 40, (8, 4))),
-                       rglru(256, 2, 4, ff=moe(12, 3, 48, (4, 3), 24))], side=24)
+                       rglru(256, 2, 4, ff=moe(12, 3, 48, (4, 3), 48))], side=24)
 CONFIGS = {"odd": ODD, "plain": PLAIN, "wide": WIDE}
 _cache = {}
 
@@ -266,23 +266,55 @@ def test_gated_recurrence(run, B, n, K):
             torch.testing.assert_close(state[slot].cpu().reshape(B, np_)[:, :n].double(), core, rtol=1e-4, atol=1e-4)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("B,n", [(2, 160), (3, 24), (1, 256)])
+def test_gated_recurrence_over_many_chunks(B, n):
+    """More chunks than thread blocks, so that every block walks several of them; blocks of channels that leave lanes without one.
+    Against the operators' unfused form on the same numbers."""
+    run, C, np_ = ("cuda", torch.bfloat16), B * n, pad8(n)
+    T = 64 * 148 * 2 // B * 3 + 40
+    on = lambda *s, seed, f=1.0: (randn(*s, seed=seed) * f).bfloat16().to("cuda")  # noqa: E731
+    y, x, bias = on(T, C, seed=1), on(T, C, seed=2), [on(C, seed=3 + i, f=0.5) for i in range(3)]
+    taps, wg, gb, lam = on(C, 4, seed=7, f=0.5), on(B, 2, np_, np_, seed=8, f=n ** -0.5 * 2), on(B, 2, np_, seed=9), on(C, seed=10, f=2.0) - 4
+    p, _, _ = layout([0], [T], run, pages_each=T // 16 + 1)
+    outs, states = [], []
+    for fused in (True, False):
+        out, state, conv = torch.zeros(T, C, dtype=torch.bfloat16, device="cuda"), torch.zeros(1, C, device="cuda"), torch.zeros(1, C, 3, device="cuda")
+        if fused:
+            ops.gated_recurrence(y, x, bias[0], bias[1], taps, bias[2], wg, gb, lam, out, state, conv, p)
+        else:
+            u = ops.causal_conv(x, bias[1], taps, bias[2], conv, p)
+            ops.linear_recurrence(u, ops.block_gates(u, wg.view(B, 2 * np_, np_)), gb.view(-1), lam, y, bias[0], out, state, p, np_)
+        outs.append(out.float())
+        states.append(state)
+    near(outs[0].cpu()[:, None], outs[1].cpu()[:, None], run)
+    torch.testing.assert_close(states[0], states[1], rtol=2e-3, atol=2e-3)
+
+
 @pytest.mark.parametrize("run", RUNS)
 @pytest.mark.parametrize("E,top,groups,keep", [(6, 3, 3, 2), (5, 2, 5, 3), (8, 1, 2, 1), (9, 9, 1, 1), (64, 6, 8, 3), (256, 8, 8, 4), (40, 6, 8, 4), (33, 4, 11, 2),
                                                (1, 1, 1, 1), (1000, 32, 10, 5)])
 def test_routing(run, E, top, groups, keep):
     """Choice scores are negative for most experts (a closed group must not count as zero), and the correction decides the choice but
-    not the weight."""
+    not the weight; with and without an expert that every token takes."""
     M = 37
-    z, corr = randn(M, pad8(E), seed=E), (randn(E, seed=E + 1) - 1.5).bfloat16().float()
-    r = ops.route(z.to(run[0]), corr.to(run[1]).to(run[0]), top, groups, keep, 2.5)
-    place, token, off, w = r.place.cpu(), r.token.cpu(), r.offsets.cpu(), r.weights.cpu()
-    assert off[0] == 0 and off[-1] == M * top and sorted(place.reshape(-1).tolist()) == list(range(M * top))
-    s = O.sigmoid(z[:, :E].double())
-    for t in range(M):
-        ids = O.route(s[t], corr.double(), top, None if keep == groups else {"count": groups, "keep": keep})
-        got = torch.searchsorted(off, place[t], right=True) - 1
-        assert sorted(got.tolist()) == sorted(ids) and (token[place[t].long()] == t).all()
-        torch.testing.assert_close(w[t].double(), s[t][got.long()] * 2.5, rtol=1e-5, atol=1e-6)
+    z, corr = randn(M, pad8(E) + 1, seed=E), (randn(E, seed=E + 1) - 1.5).bfloat16().float()
+    zd = z.to(run[0])
+    for joint in (False, True) if top < 32 else (False,):
+        r = ops.route(zd[:, :-1], corr.to(run[1]).to(run[0]), top, groups, keep, 2.5, zd[:, -1] if joint else None)
+        place, token, off, w = r.place.cpu(), r.token.cpu(), r.offsets.cpu(), r.weights.cpu()
+        n = M * (top + joint)
+        assert off[0] == 0 and off[-1] == n and len(off) == E + joint + 1 and sorted(place.reshape(-1).tolist()) == list(range(n))
+        s = O.sigmoid(z.double())
+        for t in range(M):
+            ids = O.route(s[t, :E], corr.double(), top, None if keep == groups else {"count": groups, "keep": keep})
+            got = torch.searchsorted(off, place[t], right=True) - 1
+            assert sorted(got.tolist()) == sorted(ids + [E] * joint) and (token[place[t].long()] == t).all()
+            want = s[t][got.long()] * 2.5
+            if joint:
+                assert got[-1] == E
+                want[-1] = s[t, -1]
+            torch.testing.assert_close(w[t].double(), want, rtol=1e-5, atol=1e-6)
 
 
 @pytest.mark.parametrize("run", RUNS)
@@ -302,7 +334,12 @@ def test_router_product(run, E, top, groups, keep, W, shared):
         z = h.double() @ w.double().T
         if shared:
             torch.testing.assert_close(gate.double().cpu(), z[:, pad8(E)], rtol=1e-4, atol=1e-4)
-        assert gate is not None or not shared
+            joint, none = ops.router(on(h), on(w), pad8(E), on(corr), top, groups, keep, 1.5, True)
+            assert none is None and joint.place.shape[1] == top + 1 and torch.equal(joint.weights[:, :top], r.weights)
+            torch.testing.assert_close(joint.weights[:, top].double().cpu(), O.sigmoid(z[:, pad8(E)]), rtol=1e-4, atol=1e-5)
+            assert (joint.place[:, top] >= M * top).all() and int(joint.offsets[E]) == M * top
+        else:
+            assert gate is None
         want = ops.route(z[:, :pad8(E)].float(), corr, top, groups, keep, 1.5)
         same = (r.weights.cpu().sort(-1).values - want.weights.sort(-1).values).abs().max(-1).values < 1e-4
         assert same.float().mean() > 0.999                       # a choice so close that the order of a sum decides it
@@ -387,6 +424,12 @@ def test_token_vectors(run):
         got = ops.gelu_times_token(gate[:, d:], table, ids.to(run[0]), layer * d, V).double().cpu()
         want = O.gelu_tanh(gate[:, d:].double().cpu()) * table.double().cpu()[ids, layer * d:(layer + 1) * d]
         torch.testing.assert_close(got, want, rtol=1e-2 if run[1] == torch.bfloat16 else 1e-5, atol=1e-5)
+    for M, d, W in ((1, 8, 8), (37, 24, 72), (300, 128, 200), (1100, 80, 64)):
+        h, w, table = randn(M, W, seed=1).bfloat16().float(), (randn(d, W, seed=2) * W ** -0.5 * 2).bfloat16().float(), randn(V, 2 * d, seed=3).bfloat16().float()
+        ids = torch.randint(0, V, (M,), generator=torch.Generator().manual_seed(M))
+        got = ops.token_gate(on(h), on(w), on(table), ids.to(run[0]), d, V).double().cpu()
+        want = O.gelu_tanh(h.double() @ w.double().T) * table.double()[ids, d:]
+        torch.testing.assert_close(got, want, rtol=2e-2 if run[1] == torch.bfloat16 else 1e-4, atol=2e-2 if run[1] == torch.bfloat16 else 1e-5)
 
 
 # ---- the whole model --------------------------------------------------------------------------------------------------------
