@@ -97,12 +97,12 @@ def gated_recurrence(y: torch.Tensor, x: torch.Tensor, y_bias: torch.Tensor, x_b
     u = causal_conv(x, x_bias, taps, conv_bias, conv_state, p)
     tiled = u.is_cuda and u.dtype == torch.bfloat16 and p.nseq > p.num_short and n <= 256
     if tiled:          # the long portions: gates inside the passes over them
-        ns, nc, cl = p.num_short, p.chunks64.shape[0], nv.ctypes.c_longlong
+        ns, nc, cl = p.num_short, p.chunks128.shape[0], nv.ctypes.c_longlong
         C = u.shape[1]
-        ws = torch.empty((nc, 2, 2, C), device=u.device, dtype=torch.float32)
+        ws = torch.empty((nc, 4, 2, C), device=u.device, dtype=torch.float32)
         nv.check(nv.lib().b2_gated_recurrence(
             nv.ptr(u), nv.ptr(w_gates), nv.ptr(gate_bias), nv.ptr(lam), nv.ptr(y), cl(y.stride(0)), nv.ptr(y_bias), nv.ptr(out),
-            cl(out.stride(0)), nv.ptr(state), nv.ptr(ws), nv.ptr(p.starts), nv.ptr(p.slots), nv.ptr(p.chunks64), nv.ptr(p.first64), nc,
+            cl(out.stride(0)), nv.ptr(state), nv.ptr(ws), nv.ptr(p.starts), nv.ptr(p.slots), nv.ptr(p.chunks128), nv.ptr(p.first128), nc,
             ns, p.nseq - ns, u.shape[0], C, n, nv.stream_ptr()), "gated_recurrence")
         nv.count_launch(3)
         if ns == 0:

@@ -158,8 +158,8 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const RoutePar
 }
 
 // Products with few outputs or few rows (router logits, gates), bf16 operands and a 32-bit result: 16 rows and up to 72 columns a CTA,
-// whose warps split the contraction.  A lane loads eight neighbouring elements of its row of either operand at once and uses them as the fragments of two m16n8k16
-// products: the order of the contraction is free as long as both operands agree on it.  SK_ROUTE: the rows' experts are chosen on the
+// whose warps split the contraction.  A lane loads eight neighbouring elements of its row of either operand at once and uses them as
+// the fragments of two m16n8k16 products: the order of the contraction is free as long as both operands agree on it.  SK_ROUTE: the rows' experts are chosen on the
 // spot.  SK_TOKEN: the result goes through gelu and times a vector of the row's token, rounded to bf16.
 enum : int { SK_PLAIN = 0, SK_ROUTE = 1, SK_TOKEN = 2 };
 struct SkinnyParams {
@@ -190,21 +190,29 @@ __global__ void __launch_bounds__(SK_WARPS * 32) skinny_kernel(const SkinnyParam
   for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-#pragma unroll 2
-  for (int k = warp * 32 + t * 8; k - t * 8 < p.K; k += SK_WARPS * 32) {
-    const bool in = k < p.K;                 // p.K is a multiple of 8
-    const uint4 zero = make_uint4(0, 0, 0, 0);
-    const uint4 x0 = in ? *reinterpret_cast<const uint4*>(a0 + k) : zero, x1 = in ? *reinterpret_cast<const uint4*>(a1 + k) : zero;
-    uint4 w[NT];
+  constexpr int U = NT <= 2 ? 8 : NT <= 5 ? 4 : 2;        // steps whose loads are in flight together
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  for (int k0 = warp * 32; k0 < p.K; k0 += U * SK_WARPS * 32) {
+    uint4 x0[U], x1[U], w[U][NT];
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
-      w[n] = in && n0 + n * 8 + g < p.N ? *reinterpret_cast<const uint4*>(p.w + static_cast<size_t>(n0 + n * 8 + g) * p.ld_w + k) : zero;
-    const uint32_t f0[4] = {x0.x, x1.x, x0.y, x1.y}, f1[4] = {x0.z, x1.z, x0.w, x1.w};
+    for (int u = 0; u < U; ++u) {
+      const int k = k0 + u * (SK_WARPS * 32) + t * 8;
+      const bool in = k < p.K;               // p.K is a multiple of 8
+      x0[u] = in ? *reinterpret_cast<const uint4*>(a0 + k) : zero;
+      x1[u] = in ? *reinterpret_cast<const uint4*>(a1 + k) : zero;
 #pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      const uint32_t b0[2] = {w[n].x, w[n].y}, b1[2] = {w[n].z, w[n].w};
-      mma_bf16(acc[n], f0, b0);
-      mma_bf16(acc[n], f1, b1);
+      for (int n = 0; n < NT; ++n)
+        w[u][n] = in && n0 + n * 8 + g < p.N ? *reinterpret_cast<const uint4*>(p.w + static_cast<size_t>(n0 + n * 8 + g) * p.ld_w + k) : zero;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t f0[4] = {x0[u].x, x1[u].x, x0[u].y, x1[u].y}, f1[4] = {x0[u].z, x1[u].z, x0[u].w, x1[u].w};
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const uint32_t b0[2] = {w[u][n].x, w[u][n].y}, b1[2] = {w[u][n].z, w[u][n].w};
+        mma_bf16(acc[n], f0, b0);
+        mma_bf16(acc[n], f1, b1);
+      }
     }
   }
 #pragma unroll
@@ -830,16 +838,15 @@ template <int FORM>
 static int launch_skinny(const SkinnyParams& p, const RouteParams& r, cudaStream_t st) {
   const int nt = (p.N + 7) / 8;
   const dim3 wide((p.M + SK_ROWS - 1) / SK_ROWS, (p.N + 63) / 64), grid(wide.x);
-  if (FORM == SK_TOKEN) {
+  if constexpr (FORM == SK_TOKEN) {
     if (p.N <= 32) skinny_kernel<4, FORM><<<grid, SK_WARPS * 32, 0, st>>>(p, r);
     else skinny_kernel<8, FORM><<<wide, SK_WARPS * 32, 0, st>>>(p, r);
-    B2_CHECK_LAUNCH("skinny");
-    return 0;
-  }
+  } else {
 #define B2_SKINNY(V) case V: skinny_kernel<V, FORM><<<grid, SK_WARPS * 32, 0, st>>>(p, r); break
-  switch (nt) {
-    B2_SKINNY(1); B2_SKINNY(2); B2_SKINNY(3); B2_SKINNY(4); B2_SKINNY(5); B2_SKINNY(6); B2_SKINNY(7); B2_SKINNY(8); B2_SKINNY(9);
-    default: set_error("skinny: up to %d outputs", SK_MAX_TILES * 8); return 10;
+    switch (nt) {
+      B2_SKINNY(1); B2_SKINNY(2); B2_SKINNY(3); B2_SKINNY(4); B2_SKINNY(5); B2_SKINNY(6); B2_SKINNY(7); B2_SKINNY(8); B2_SKINNY(9);
+      default: set_error("skinny: up to %d outputs", SK_MAX_TILES * 8); return 10;
+    }
   }
 #undef B2_SKINNY
   B2_CHECK_LAUNCH("skinny");

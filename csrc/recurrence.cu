@@ -167,7 +167,7 @@ struct RecParams {
   const int* cu;
   const int* start;
   const int* slot;
-  const int* chunks;     // [n, 4], two runs each
+  const int* chunks;     // [n, 4], several runs each
   const int* first;      // [nlong + 1]
   long long ld_u, ld_z, ld_y, ld_out;
   int C, block, seq0;
@@ -221,7 +221,7 @@ struct RecChannel {
 
 constexpr int GR_RUN = 32;
 
-// Rows of run h (0, 1) of a chunk.
+// Rows of run h of a chunk.
 __device__ __forceinline__ int run_rows(int rows, int h) { return max(0, min(GR_RUN, rows - h * GR_RUN)); }
 
 template <typename T>
@@ -242,14 +242,14 @@ __global__ void __launch_bounds__(GR_THREADS) rec_transfer_kernel(const RecParam
   w[p.C] = S;
 }
 
-// Grid (channels, long sequences)
-__global__ void __launch_bounds__(GR_THREADS) rec_carry_kernel(const RecParams p) {
+// Grid (channels, long sequences); per: runs of a chunk
+__global__ void __launch_bounds__(GR_THREADS) rec_carry_kernel(const RecParams p, int per) {
   const int c = blockIdx.x * GR_THREADS + threadIdx.x, s = p.seq0 + blockIdx.y;
   const int slot = p.slot[s];
   if (c >= p.C || slot < 0) return;
   float* st = p.state + static_cast<size_t>(slot) * p.C + c;
   float S = p.start[s] == 0 ? 0.f : *st;
-  const int c0 = p.first[blockIdx.y] * 2, c1 = p.first[blockIdx.y + 1] * 2;
+  const int c0 = p.first[blockIdx.y] * per, c1 = p.first[blockIdx.y + 1] * per;
   constexpr int U = 16;
   for (int i = c0; i < c1; i += U) {
     float A[U], B[U];
@@ -294,20 +294,23 @@ __global__ void __launch_bounds__(GR_THREADS) rec_out_kernel(const RecParams p) 
 }
 
 // ---- both passes with their gates on the tensor cores ---------------------------------------------------------------------------
-// A CTA keeps the two gates' weights of 128 channels of a block in shared memory (they read all of the block's channels of u) and
-// walks chunks of 64 tokens: u arrives by TMA one chunk ahead, the products of the next chunk run under the recurrence of this one.
-// Warps 0..3 have the chunk's first run, warps 4..7 the second; thread = channel.
-constexpr int RG_THREADS = 256;
+// A CTA keeps the two gates' weights of up to 128 channels of a block in shared memory (they read all of the block's channels of u)
+// and walks chunks of 128 tokens: where there is room u arrives by TMA one chunk ahead, and the products of the next chunk run under
+// the recurrence of this one.  Four warps per run of 32 tokens; thread = channel.
+constexpr int RG_CHUNK = 128, RG_RUNS = RG_CHUNK / GR_RUN, RG_THREADS = 128 * RG_RUNS;
 constexpr int RG_MAX_BLOCK = 256;
+constexpr int RG_TMEM = 512;           // two accumulators of two gates of a chunk: all of it, so one CTA per SM
 typedef __nv_bfloat16 rg_bf16;
 
 struct RecGateSmem {
-  int kc, weights, stage, total;       // 64-channel pieces of a block; bytes
+  int kc, weights, stage, stages, total;       // 64-channel pieces of a block; bytes
   __host__ __device__ explicit RecGateSmem(int block) {
     kc = (block + 63) / 64;
     weights = 2 * kc * 128 * 128;
-    stage = kc * 64 * 128;
-    total = weights + 2 * stage + 64 + 1024;
+    stage = kc * RG_CHUNK * 128;
+    stages = weights + 2 * stage <= 224 * 1024 ? 2 : 1;
+    total = weights + stages * stage + 64 + 1024;
+    if (total < 120 * 1024) total = 120 * 1024;       // more than half of an SM's
   }
 };
 
@@ -318,90 +321,94 @@ __device__ __forceinline__ float sqrt_fast(float x) {
 }
 
 template <bool OUT>
-__global__ void __launch_bounds__(RG_THREADS) rec_gates_kernel(const __grid_constant__ CUtensorMap tmU, const __grid_constant__ CUtensorMap tmW,
-                                                               const RecParams p, int nchunks, int tiles_per_block, int* status) {
+__global__ void __launch_bounds__(RG_THREADS, 1) rec_gates_kernel(const __grid_constant__ CUtensorMap tmU, const __grid_constant__ CUtensorMap tmW,
+                                                                  const RecParams p, int nchunks, int tiles_per_block, int tile_channels, int* status) {
   extern __shared__ uint8_t rg_raw[];
   uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(rg_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const RecGateSmem L(p.block);
   uint8_t* su = sm + L.weights;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(su + 2 * L.stage);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(su + L.stages * L.stage);
   uint64_t *w_full = bars, *u_full = bars + 1, *done = bars + 3;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quarter = warp & 3, run = warp >> 2;
-  const int b = blockIdx.x / tiles_per_block, ct = blockIdx.x % tiles_per_block;
+  const int b = blockIdx.x / tiles_per_block, c0 = blockIdx.x % tiles_per_block * tile_channels;     // first channel, in the block
   if (tid == 0) {
     for (int i = 0; i < 5; ++i) mbar_init(bars + i, 1);
     mbar_fence_init();
   }
   if (warp == 0) {
-    tmem_alloc(tmem_slot, 256);
+    tmem_alloc(tmem_slot, RG_TMEM);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
-  const int stride = gridDim.y;
-  auto load_u = [&](int chunk, int st) {            // one thread
+  const int stride = gridDim.y, mine = (nchunks - static_cast<int>(blockIdx.y) + stride - 1) / stride;      // chunks of this CTA
+  auto chunk_of = [&](int it) { return static_cast<int>(blockIdx.y) + it * stride; };
+  auto load_u = [&](int it) {                       // one thread
+    const int st = it % L.stages, row = p.chunks[chunk_of(it) * 4 + 1];
     mbar_expect_tx(u_full + st, L.stage);
-    const int row = p.chunks[chunk * 4 + 1];
-    for (int k = 0; k < L.kc; ++k) tma_load_2d(su + st * L.stage + k * 8192, &tmU, u_full + st, b * p.block + k * 64, row);
+    for (int k = 0; k < L.kc; ++k)
+      tma_load_2d(su + st * L.stage + k * (RG_CHUNK * 128), &tmU, u_full + st, b * p.block + k * 64, row);
   };
   if (tid == 0) {
     mbar_expect_tx(w_full, L.weights);
     for (int g = 0; g < 2; ++g)
-      for (int k = 0; k < L.kc; ++k) tma_load_3d(sm + (g * L.kc + k) * 16384, &tmW, w_full, k * 64, ct * 128, 2 * b + g);
-    for (int i = 0; i < 2; ++i)
-      if (static_cast<int>(blockIdx.y) + i * stride < nchunks) load_u(blockIdx.y + i * stride, i);
+      for (int k = 0; k < L.kc; ++k) tma_load_3d(sm + (g * L.kc + k) * 16384, &tmW, w_full, k * 64, c0, 2 * b + g);
+    for (int i = 0; i < L.stages && i < mine; ++i) load_u(i);
   }
   const bool leader = warp == 0 && elect_one();
-  // gates of the chunk in stage st: columns 0..63 of its accumulators the recurrence gate, 64..127 the input gate
-  auto products = [&](int st, uint32_t ph) {        // warp 0
-    mbar_wait_warp(u_full + st, ph, status, ERR_GEMM_MMA_WAIT_FULL);
+  // Gates of chunk `it`: of its accumulator (256 columns) the first half is the recurrence gate's, the second the input gate's.
+  auto products = [&](int it) {                     // warp 0
+    const int st = it % L.stages;
+    mbar_wait_warp(u_full + st, (it / L.stages) & 1, status, ERR_GEMM_MMA_WAIT_FULL);
     tc_fence_after();
     if (leader) {
-      constexpr uint32_t idesc = make_idesc_f16(1, 128, 64, 0, 0);
+      constexpr uint32_t idesc = make_idesc_f16(1, 128, RG_CHUNK, 0, 0);
       for (int g = 0; g < 2; ++g)
         for (int k = 0; k < L.kc; ++k) {
           const uint64_t da = make_smem_desc_sw128(smem_u32(sm + (g * L.kc + k) * 16384), 16, 1024),
-                         db = make_smem_desc_sw128(smem_u32(su + st * L.stage + k * 8192), 16, 1024);
+                         db = make_smem_desc_sw128(smem_u32(su + st * L.stage + k * (RG_CHUNK * 128)), 16, 1024);
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks)
-            umma_f16_ss(tmem + st * 128 + g * 64, desc_advance(da, ks * 32), desc_advance(db, ks * 32), idesc, k > 0 || ks > 0 ? 1u : 0u);
+            umma_f16_ss(tmem + (it & 1) * (2 * RG_CHUNK) + g * RG_CHUNK, desc_advance(da, ks * 32), desc_advance(db, ks * 32), idesc,
+                        k > 0 || ks > 0 ? 1u : 0u);
         }
-      umma_commit(done + st);
+      umma_commit(done + (it & 1));
     }
     __syncwarp();
   };
+  const bool ahead = L.stages == 2;
   if (warp == 0) {
     mbar_wait_warp(w_full, 0, status, ERR_GEMM_MMA_WAIT_FULL);
-    if (static_cast<int>(blockIdx.y) < nchunks) products(0, 0);
+    if (ahead && mine > 0) products(0);
   }
-  const int c = ct * 128 + quarter * 32 + lane;     // in the block
-  const bool in = c < p.block;
-  const int ch = b * p.block + (in ? c : 0);
+  const int l = quarter * 32 + lane;                // lane of the accumulator
+  const bool in = l < tile_channels && c0 + l < p.block;
+  const int c = in ? c0 + l : c0, ch = b * p.block + c;      // lanes without a channel read the tile's first one's
   const RecChannel<rg_bf16> K(p, ch);
   const uint32_t at = tmem + (static_cast<uint32_t>(quarter * 32) << 16) + run * GR_RUN;
-  const int cu = in ? c : 0;                         // lanes past the block's last channel read the first one's
-  const int u_at = (cu >> 6) * 8192 + (cu & 7) * 2, u_piece = (cu >> 3) & 7;
-  int it = 0;
-  for (int chunk = blockIdx.y; chunk < nchunks; chunk += stride, ++it) {
-    const int st = it & 1;
-    const uint32_t ph = (it >> 1) & 1;
-    if (warp == 0 && chunk + stride < nchunks) products(st ^ 1, ((it + 1) >> 1) & 1);
+  const int u_at = (c >> 6) * (RG_CHUNK * 128) + (c & 7) * 2, u_piece = (c >> 3) & 7;
+  const bool idle = quarter * 32 >= tile_channels;  // the whole warp
+  for (int it = 0; it < mine; ++it) {
+    const int st = it % L.stages, chunk = chunk_of(it);
+    if (warp == 0) {
+      if (!ahead) products(it);
+      else if (it + 1 < mine) products(it + 1);
+    }
     const int* cd = p.chunks + chunk * 4;
     const size_t row0 = cd[1] + run * GR_RUN;
-    const int n = run_rows(cd[2], run);
-    const size_t wi = (static_cast<size_t>(chunk) * 2 + run) * 2 * p.C + ch;
+    const int n = idle ? 0 : run_rows(cd[2], run);
+    const size_t wi = (static_cast<size_t>(chunk) * RG_RUNS + run) * 2 * p.C + ch;
     float A = 1.f, S = 0.f;
     if (OUT) S = p.ws[wi];
-    mbar_wait_warp(u_full + st, ph, status, ERR_GEMM_MMA_WAIT_FULL);       // u itself is read below
-    mbar_wait_warp(done + st, ph, status, ERR_GEMM_EPI_WAIT);
+    mbar_wait_warp(u_full + st, (it / L.stages) & 1, status, ERR_GEMM_MMA_WAIT_FULL);       // u itself is read below
+    mbar_wait_warp(done + (it & 1), (it >> 1) & 1, status, ERR_GEMM_EPI_WAIT);
     tc_fence_after();
     const uint8_t* ut = su + st * L.stage + u_at;
 #pragma unroll 1
-    for (int t0 = 0; t0 < GR_RUN; t0 += 16) {
-      if (t0 >= n) break;                           // the same for the whole warp
+    for (int t0 = 0; t0 < n; t0 += 16) {            // n is the same for the whole warp
       uint32_t zr[16], zi[16];
       float y[16];
       if (OUT) {
@@ -409,8 +416,8 @@ __global__ void __launch_bounds__(RG_THREADS) rec_gates_kernel(const __grid_cons
         for (int i = 0; i < 16; ++i)
           y[i] = __bfloat162float(static_cast<const rg_bf16*>(p.y)[(row0 + min(t0 + i, n - 1)) * p.ld_y + ch]);
       }
-      tmem_ld_32x32b_x16(at + st * 128 + t0, zr);
-      tmem_ld_32x32b_x16(at + st * 128 + 64 + t0, zi);
+      tmem_ld_32x32b_x16(at + (it & 1) * (2 * RG_CHUNK) + t0, zr);
+      tmem_ld_32x32b_x16(at + (it & 1) * (2 * RG_CHUNK) + RG_CHUNK + t0, zi);
       tmem_ld_wait();
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
@@ -434,7 +441,7 @@ __global__ void __launch_bounds__(RG_THREADS) rec_gates_kernel(const __grid_cons
     tc_fence_before();
     __syncthreads();                                // the stage and its accumulators have been read
     tc_fence_after();
-    if (tid == 0 && chunk + 2 * stride < nchunks) load_u(chunk + 2 * stride, st);
+    if (tid == 0 && it + L.stages < mine) load_u(it + L.stages);
   }
   if (*reinterpret_cast<volatile int*>(status) != 0) {     // copies and products in flight land before shared memory and TMEM go away
     const unsigned long long t0 = globaltimer_ns();
@@ -444,7 +451,7 @@ __global__ void __launch_bounds__(RG_THREADS) rec_gates_kernel(const __grid_cons
   __syncthreads();
   if (warp == 0) {
     tc_fence_after();
-    tmem_dealloc(tmem, 256);
+    tmem_dealloc(tmem, RG_TMEM);
   }
 }
 
@@ -464,11 +471,13 @@ static int launch_gates(const CUtensorMap* tu, const CUtensorMap* tw, const RecP
     }
     set[dev & 63] = L.total;
   }
-  const int per = (p.block + 127) / 128, x = p.C / p.block * per, resident = num_sms() * (L.total <= 112 * 1024 ? 2 : 1);
-  int y = resident / x;
+  // tiles of equal size, in whole warps where that costs none of them
+  const int per = (p.block + 127) / 128, x = p.C / p.block * per;
+  int tile = (p.block + per - 1) / per, y = num_sms() / x;
+  if ((tile + 31) / 32 * 32 * (per - 1) < p.block) tile = (tile + 31) / 32 * 32;
   if (y < 1) y = 1;
   if (y > nchunks) y = nchunks;
-  kern<<<dim3(x, y), RG_THREADS, L.total, stream>>>(*tu, *tw, p, nchunks, per, status);
+  kern<<<dim3(x, y), RG_THREADS, L.total, stream>>>(*tu, *tw, p, nchunks, per, tile, status);
   B2_CHECK_LAUNCH("rec_gates");
   return 0;
 }
@@ -515,7 +524,7 @@ B2_EXPORT int b2_linear_recurrence(const void* u, long long ld_u, const float* z
   if (nchunks > 0) {
     B2_DISPATCH_T(is_f32, rec_transfer_kernel<T><<<dim3(2 * nchunks, cy), GR_THREADS, 0, st>>>(p););
     B2_CHECK_LAUNCH("rec_transfer");
-    rec_carry_kernel<<<dim3(cy, nseq), GR_THREADS, 0, st>>>(p);
+    rec_carry_kernel<<<dim3(cy, nseq), GR_THREADS, 0, st>>>(p, 2);
     B2_CHECK_LAUNCH("rec_carry");
     B2_DISPATCH_T(is_f32, (rec_out_kernel<T, true><<<dim3(2 * nchunks, cy), GR_THREADS, 0, st>>>(p)););
   } else {
@@ -526,7 +535,7 @@ B2_EXPORT int b2_linear_recurrence(const void* u, long long ld_u, const float* z
 }
 
 // Long sequences in bf16 with the gates' products inside: u [M, C] contiguous, w [C / block, 2, block, block], blocks up to 256
-// channels in multiples of 8; ws as above.
+// channels in multiples of 8; chunks of 128 rows, ws fp32 [nchunks, 4, 2, C].
 B2_EXPORT int b2_gated_recurrence(const void* u, const void* w, const void* zb, const void* lam, const void* y, long long ld_y,
                                   const void* yb, void* out, long long ld_out, float* state, float* ws, const int* start, const int* slot,
                                   const int* chunks, const int* first, int nchunks, int seq0, int nseq, int M, int C, int block,
@@ -540,11 +549,11 @@ B2_EXPORT int b2_gated_recurrence(const void* u, const void* w, const void* zb, 
   const RecParams p = {u, nullptr, zb, lam, y, yb, out, state, ws, nullptr, start, slot, chunks, first, C, 0, ld_y, ld_out, C, block, seq0};
   const uint64_t n = block, dims[3] = {n, n, 2ull * (C / block)}, strides[2] = {2 * n, 2 * n * n};
   const uint32_t box[3] = {64, 128, 1};
-  const CUtensorMap *tw = tensor_map_nd_bf16(w, 3, dims, strides, box, 3), *tu = tensor_map_2d_bf16(u, M, C, C, 64, 64);
+  const CUtensorMap *tw = tensor_map_nd_bf16(w, 3, dims, strides, box, 3), *tu = tensor_map_2d_bf16(u, M, C, C, RG_CHUNK, 64);
   if (!tw || !tu) return 2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (const int rc = launch_gates<false>(tu, tw, p, nchunks, st)) return rc;
-  rec_carry_kernel<<<dim3((C + GR_THREADS - 1) / GR_THREADS, nseq), GR_THREADS, 0, st>>>(p);
+  rec_carry_kernel<<<dim3((C + GR_THREADS - 1) / GR_THREADS, nseq), GR_THREADS, 0, st>>>(p, RG_RUNS);
   B2_CHECK_LAUNCH("rec_carry");
   return launch_gates<true>(tu, tw, p, nchunks, st);
 }
