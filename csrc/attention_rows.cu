@@ -400,19 +400,6 @@ struct NormStoreParams {
 // Bias, per-head RMS norm of q and k (optional weights), rotary positions on channel pairs (2 i, 2 i + 1), and the store of k / v.
 // Grid (M, y).  LPH lanes per head, eight channels each; a lane takes NS_UNROLL heads of its row at a time, their loads together.
 // What waits in registers waits packed, so that eight CTAs fit on an SM.
-template <typename T>
-struct Packed8 {
-  uint4 w[sizeof(T) / 2];
-  __device__ __forceinline__ void load(const T* p) {
-#pragma unroll
-    for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) w[i] = reinterpret_cast<const uint4*>(p)[i];
-  }
-  __device__ __forceinline__ void zero() {
-#pragma unroll
-    for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) w[i] = make_uint4(0, 0, 0, 0);
-  }
-  __device__ __forceinline__ void get(float (&f)[8]) const { vload8(reinterpret_cast<const T*>(w), f); }
-};
 template <typename T, int LPH, int NS_UNROLL>
 __global__ void __launch_bounds__(128, sizeof(T) == 2 ? 8 : 4) qk_norm_store_kernel(const NormStoreParams p) {
   constexpr int GROUPS = 128 / LPH;

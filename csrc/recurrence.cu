@@ -9,6 +9,8 @@
 // at the runs' starts, then the runs once more from there.  In bf16 the gates of both passes are tcgen05 products inside the pass
 // (rec_gates_kernel): the accumulators have a channel per TMEM lane and a token per column, so that a thread finds the gates of its
 // channel's tokens in its own lane and the recurrence never leaves registers; gates are made twice instead of stored.
+#include <type_traits>
+
 #include "host.h"
 #include "vec.cuh"
 
@@ -37,7 +39,7 @@ struct ConvParams {
 // state, so that tile also replaces it, after its own reads.  KT: taps known to the compiler (0: any number).
 constexpr int GR_ROWS = GR_TILE / 4;
 template <typename T, int KT>
-__global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParams p) {
+__global__ void __launch_bounds__(GR_THREADS, sizeof(T) == 2 ? 5 : 4) causal_conv_kernel(const ConvParams p) {
   const int* tl = p.tiles + blockIdx.x * 4;
   const int s = tl[0], row0 = tl[1], rows = tl[2], off = tl[3], K = KT > 0 ? KT : p.K;
   const int c = (blockIdx.y * 32 + (threadIdx.x & 31)) * 8, t0 = (threadIdx.x >> 5) * GR_ROWS;
@@ -51,19 +53,36 @@ __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParam
   float xb[8], cb[8];
   vload8(static_cast<const T*>(p.xb) + cc, xb);
   vload8(static_cast<const T*>(p.cb) + cc, cb);
-  // known taps: the state of these channels in registers (neighbours in memory), [channel][input]
-  constexpr int OLD = KT > 1 ? KT - 1 : 1;
-  float old[OLD * 8];
-  if constexpr (KT > 1) {
+  // Only the first rows of the first tile look back into the state.
+  constexpr int KK = KT > 0 ? KT : 1, OLD = KT > 1 ? KT - 1 : 1;
+  const bool head = off == 0 && t0 == 0;
+  float w[KK * 8];                                   // a channel's taps are neighbours
+  if constexpr (KT > 0) {
 #pragma unroll
-    for (int i = 0; i < OLD; ++i) {
-      float f[8] = {};
-      if (off == 0 && !fresh) vload8(st + i * 8, f);
+    for (int i = 0; i < KK; ++i) {
+      float f[8];
+      vload8(taps + i * 8, f);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) old[i * 8 + e] = f[e];
+      for (int e = 0; e < 8; ++e) w[i * 8 + e] = f[e];
     }
   }
-  auto input = [&](int at, float (&f)[8]) {          // input at index `at` of the portion
+  // known taps: the state of these channels as it lies in memory, [channel][input]
+  auto load_old = [&](float (&old)[OLD * 8]) {
+    if constexpr (KT > 1) {
+#pragma unroll
+      for (int i = 0; i < OLD; ++i) {
+        float f[8] = {};
+        if (!fresh) vload8(st + i * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) old[i * 8 + e] = f[e];
+      }
+    }
+  };
+  auto tap = [&](int e, int j) {                     // of channel e, j tokens back
+    if constexpr (KT > 0) return w[e * KT + KT - 1 - j];
+    else return to_f(taps[e * K + K - 1 - j]);
+  };
+  auto input = [&](int at, float (&f)[8], const float (&old)[OLD * 8]) {          // input at index `at` of the portion
     if (at >= 0) {
       vload8(x + (static_cast<size_t>(row0) + at - off) * p.ld, f);
 #pragma unroll
@@ -79,61 +98,74 @@ __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParam
       for (int e = 0; e < 8; ++e) f[e] = fresh ? 0.f : st[e * (K - 1) + K - 1 + at];
     }
   };
+  T* dst = static_cast<T*>(p.u) + (static_cast<size_t>(row0) + t0) * p.C + c;
   if (in && t0 < rows) {
-    float acc[GR_ROWS][8];
+    const int n = min(GR_ROWS, rows - t0);
+    if (KT > 0 && !head) {                           // all inputs are rows of this portion: requested together
+      Packed8<T> raw[GR_ROWS + KK - 1];
 #pragma unroll
-    for (int i = 0; i < GR_ROWS; ++i)
+      for (int i = 0; i < GR_ROWS + KK - 1; ++i) raw[i].load(x + (static_cast<size_t>(row0) + min(t0 + i - (KK - 1), rows - 1)) * p.ld);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[i][e] = cb[e];
-    if constexpr (KT > 0) {
-      float w[KT * 8];                               // a channel's taps are neighbours
+      for (int o = 0; o < GR_ROWS; ++o) {
+        if (o >= n) break;
+        float acc[8];
 #pragma unroll
-      for (int i = 0; i < KT; ++i) {
-        float f[8];
-        vload8(taps + i * 8, f);
+        for (int e = 0; e < 8; ++e) acc[e] = cb[e];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) w[i * 8 + e] = f[e];
+        for (int j = 0; j < KK; ++j) {
+          float f[8];
+          raw[o + KK - 1 - j].get(f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[e] = fmaf(tap(e, j), f[e] + xb[e], acc[e]);
+        }
+        vstore8(dst + static_cast<size_t>(o) * p.C, acc);
       }
-      const int last = rows - 1;
+    } else if constexpr (KT > 0) {                   // the portion's first rows
+      float old[OLD * 8];
+      load_old(old);
 #pragma unroll
-      for (int i = -(KT - 1); i < GR_ROWS; ++i) {    // each input once, into the outputs that see it
-        float f[8];
-        input(off + min(t0 + i, last), f);
+      for (int o = 0; o < GR_ROWS; ++o) {
+        if (o >= n) break;
+        float acc[8];
 #pragma unroll
-        for (int o = 0; o < GR_ROWS; ++o)
-          if (o - i >= 0 && o - i < KT)
+        for (int e = 0; e < 8; ++e) acc[e] = cb[e];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) acc[o][e] = fmaf(w[e * KT + KT - 1 - (o - i)], f[e], acc[o][e]);
+        for (int j = 0; j < KK; ++j) {
+          float f[8];
+          input(o - j, f, old);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[e] = fmaf(tap(e, j), f[e], acc[e]);
+        }
+        vstore8(dst + static_cast<size_t>(o) * p.C, acc);
       }
     } else {
-      for (int j = 0; j < K; ++j) {
-        float w[8];
+      const float old[OLD * 8] = {};
+      for (int o = 0; o < n; ++o) {
+        float acc[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) w[e] = to_f(taps[e * K + K - 1 - j]);
-#pragma unroll
-        for (int i = 0; i < GR_ROWS; ++i) {
-          if (t0 + i >= rows) break;
+        for (int e = 0; e < 8; ++e) acc[e] = cb[e];
+        for (int j = 0; j < K; ++j) {
           float f[8];
-          input(off + t0 + i - j, f);
+          input(off + t0 + o - j, f, old);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(w[e], f[e], acc[i][e]);
+          for (int e = 0; e < 8; ++e) acc[e] = fmaf(tap(e, j), f[e], acc[e]);
         }
+        vstore8(dst + static_cast<size_t>(o) * p.C, acc);
       }
     }
-#pragma unroll
-    for (int i = 0; i < GR_ROWS; ++i)
-      if (t0 + i < rows) vstore8(static_cast<T*>(p.u) + (static_cast<size_t>(row0) + t0 + i) * p.C + c, acc[i]);
   }
   if (off != 0 || K < 2) return;
   __syncthreads();
-  if (!in || threadIdx.x >= 32) return;
+  if (!in || threadIdx.x >= 32) return;              // the warp of the first rows
   const int count = p.cu[s + 1] - p.cu[s];
+  float old[OLD * 8];
   if constexpr (KT > 1) {
+    load_old(old);
     float now[OLD * 8];
 #pragma unroll
     for (int j = 0; j < OLD; ++j) {
       float f[8];
-      input(count - OLD + j, f);
+      input(count - OLD + j, f, old);
 #pragma unroll
       for (int e = 0; e < 8; ++e) now[e * OLD + j] = f[e];
     }
@@ -144,13 +176,13 @@ __global__ void __launch_bounds__(GR_THREADS) causal_conv_kernel(const ConvParam
       for (int e = 0; e < 8; ++e) f[e] = now[i * 8 + e];
       vstore8(st + i * 8, f);
     }
-    return;
-  }
-  for (int j = 0; j < K - 1; ++j) {                  // in this order an old input is read before its place is written
-    float f[8];
-    input(count - (K - 1) + j, f);
+  } else {
+    for (int j = 0; j < K - 1; ++j) {                // in this order an old input is read before its place is written
+      float f[8];
+      input(count - (K - 1) + j, f, old);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) st[e * (K - 1) + j] = f[e];
+      for (int e = 0; e < 8; ++e) st[e * (K - 1) + j] = f[e];
+    }
   }
 }
 
@@ -295,9 +327,9 @@ __global__ void __launch_bounds__(GR_THREADS) rec_out_kernel(const RecParams p) 
 
 // ---- both passes with their gates on the tensor cores ---------------------------------------------------------------------------
 // A CTA keeps the two gates' weights of up to 128 channels of a block in shared memory (they read all of the block's channels of u)
-// and walks chunks of 128 tokens: where there is room u arrives by TMA one chunk ahead, and the products of the next chunk run under
-// the recurrence of this one.  Four warps per run of 32 tokens; thread = channel.
-constexpr int RG_CHUNK = 128, RG_RUNS = RG_CHUNK / GR_RUN, RG_THREADS = 128 * RG_RUNS;
+// and walks chunks of 128 tokens.  Four warps per run of 32 tokens walk it, thread = channel; one more warp brings u by TMA (one chunk
+// ahead, where there is room for two) and issues the products, those of the next chunk under the recurrence of this one.
+constexpr int RG_CHUNK = 128, RG_RUNS = RG_CHUNK / GR_RUN, RG_WARPS = 4 * RG_RUNS, RG_THREADS = 32 * (RG_WARPS + 1);
 constexpr int RG_MAX_BLOCK = 256;
 constexpr int RG_TMEM = 512;           // two accumulators of two gates of a chunk: all of it, so one CTA per SM
 typedef __nv_bfloat16 rg_bf16;
@@ -328,15 +360,16 @@ __global__ void __launch_bounds__(RG_THREADS, 1) rec_gates_kernel(const __grid_c
   const RecGateSmem L(p.block);
   uint8_t* su = sm + L.weights;
   uint64_t* bars = reinterpret_cast<uint64_t*>(su + L.stages * L.stage);
-  uint64_t *w_full = bars, *u_full = bars + 1, *done = bars + 3;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
+  uint64_t *w_full = bars, *u_full = bars + 1, *done = bars + 3, *used = bars + 5;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 7);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quarter = warp & 3, run = warp >> 2;
   const int b = blockIdx.x / tiles_per_block, c0 = blockIdx.x % tiles_per_block * tile_channels;     // first channel, in the block
   if (tid == 0) {
     for (int i = 0; i < 5; ++i) mbar_init(bars + i, 1);
+    for (int i = 0; i < 2; ++i) mbar_init(used + i, RG_WARPS);
     mbar_fence_init();
   }
-  if (warp == 0) {
+  if (warp == RG_WARPS) {
     tmem_alloc(tmem_slot, RG_TMEM);
     tmem_relinquish();
   }
@@ -346,102 +379,121 @@ __global__ void __launch_bounds__(RG_THREADS, 1) rec_gates_kernel(const __grid_c
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
   const int stride = gridDim.y, mine = (nchunks - static_cast<int>(blockIdx.y) + stride - 1) / stride;      // chunks of this CTA
   auto chunk_of = [&](int it) { return static_cast<int>(blockIdx.y) + it * stride; };
-  auto load_u = [&](int it) {                       // one thread
-    const int st = it % L.stages, row = p.chunks[chunk_of(it) * 4 + 1];
-    mbar_expect_tx(u_full + st, L.stage);
-    for (int k = 0; k < L.kc; ++k)
-      tma_load_2d(su + st * L.stage + k * (RG_CHUNK * 128), &tmU, u_full + st, b * p.block + k * 64, row);
-  };
-  if (tid == 0) {
-    mbar_expect_tx(w_full, L.weights);
-    for (int g = 0; g < 2; ++g)
-      for (int k = 0; k < L.kc; ++k) tma_load_3d(sm + (g * L.kc + k) * 16384, &tmW, w_full, k * 64, c0, 2 * b + g);
-    for (int i = 0; i < L.stages && i < mine; ++i) load_u(i);
-  }
-  const bool leader = warp == 0 && elect_one();
-  // Gates of chunk `it`: of its accumulator (256 columns) the first half is the recurrence gate's, the second the input gate's.
-  auto products = [&](int it) {                     // warp 0
-    const int st = it % L.stages;
-    mbar_wait_warp(u_full + st, (it / L.stages) & 1, status, ERR_GEMM_MMA_WAIT_FULL);
-    tc_fence_after();
+  if (warp == RG_WARPS) {
+    const bool leader = elect_one();
+    auto load_u = [&](int it) {
+      if (!leader) return;
+      const int st = it % L.stages, row = p.chunks[chunk_of(it) * 4 + 1];
+      mbar_expect_tx(u_full + st, L.stage);
+      for (int k = 0; k < L.kc; ++k)
+        tma_load_2d(su + st * L.stage + k * (RG_CHUNK * 128), &tmU, u_full + st, b * p.block + k * 64, row);
+    };
     if (leader) {
-      constexpr uint32_t idesc = make_idesc_f16(1, 128, RG_CHUNK, 0, 0);
+      mbar_expect_tx(w_full, L.weights);
       for (int g = 0; g < 2; ++g)
-        for (int k = 0; k < L.kc; ++k) {
-          const uint64_t da = make_smem_desc_sw128(smem_u32(sm + (g * L.kc + k) * 16384), 16, 1024),
-                         db = make_smem_desc_sw128(smem_u32(su + st * L.stage + k * (RG_CHUNK * 128)), 16, 1024);
-#pragma unroll
-          for (int ks = 0; ks < 4; ++ks)
-            umma_f16_ss(tmem + (it & 1) * (2 * RG_CHUNK) + g * RG_CHUNK, desc_advance(da, ks * 32), desc_advance(db, ks * 32), idesc,
-                        k > 0 || ks > 0 ? 1u : 0u);
-        }
-      umma_commit(done + (it & 1));
+        for (int k = 0; k < L.kc; ++k) tma_load_3d(sm + (g * L.kc + k) * 16384, &tmW, w_full, k * 64, c0, 2 * b + g);
     }
-    __syncwarp();
-  };
-  const bool ahead = L.stages == 2;
-  if (warp == 0) {
+    for (int i = 0; i < L.stages && i < mine; ++i) load_u(i);
     mbar_wait_warp(w_full, 0, status, ERR_GEMM_MMA_WAIT_FULL);
-    if (ahead && mine > 0) products(0);
-  }
-  const int l = quarter * 32 + lane;                // lane of the accumulator
-  const bool in = l < tile_channels && c0 + l < p.block;
-  const int c = in ? c0 + l : c0, ch = b * p.block + c;      // lanes without a channel read the tile's first one's
-  const RecChannel<rg_bf16> K(p, ch);
-  const uint32_t at = tmem + (static_cast<uint32_t>(quarter * 32) << 16) + run * GR_RUN;
-  const int u_at = (c >> 6) * (RG_CHUNK * 128) + (c & 7) * 2, u_piece = (c >> 3) & 7;
-  const bool idle = quarter * 32 >= tile_channels;  // the whole warp
-  for (int it = 0; it < mine; ++it) {
-    const int st = it % L.stages, chunk = chunk_of(it);
-    if (warp == 0) {
-      if (!ahead) products(it);
-      else if (it + 1 < mine) products(it + 1);
-    }
-    const int* cd = p.chunks + chunk * 4;
-    const size_t row0 = cd[1] + run * GR_RUN;
-    const int n = idle ? 0 : run_rows(cd[2], run);
-    const size_t wi = (static_cast<size_t>(chunk) * RG_RUNS + run) * 2 * p.C + ch;
-    float A = 1.f, S = 0.f;
-    if (OUT) S = p.ws[wi];
-    mbar_wait_warp(u_full + st, (it / L.stages) & 1, status, ERR_GEMM_MMA_WAIT_FULL);       // u itself is read below
-    mbar_wait_warp(done + (it & 1), (it >> 1) & 1, status, ERR_GEMM_EPI_WAIT);
-    tc_fence_after();
-    const uint8_t* ut = su + st * L.stage + u_at;
-#pragma unroll 1
-    for (int t0 = 0; t0 < n; t0 += 16) {            // n is the same for the whole warp
-      uint32_t zr[16], zi[16];
-      float y[16];
-      if (OUT) {
+    // Gates of chunk `it`: of its accumulator (256 columns, used again two chunks later) the first half is the recurrence gate's, the
+    // second the input gate's.
+    for (int it = 0; it < mine; ++it) {
+      const int st = it % L.stages, next = it + 1;
+      mbar_wait_warp(u_full + st, (it / L.stages) & 1, status, ERR_GEMM_MMA_WAIT_FULL);
+      tc_fence_after();
+      if (leader) {
+        constexpr uint32_t idesc = make_idesc_f16(1, 128, RG_CHUNK, 0, 0);
+        for (int g = 0; g < 2; ++g)
+          for (int k = 0; k < L.kc; ++k) {
+            const uint64_t da = make_smem_desc_sw128(smem_u32(sm + (g * L.kc + k) * 16384), 16, 1024),
+                           db = make_smem_desc_sw128(smem_u32(su + st * L.stage + k * (RG_CHUNK * 128)), 16, 1024);
 #pragma unroll
-        for (int i = 0; i < 16; ++i)
-          y[i] = __bfloat162float(static_cast<const rg_bf16*>(p.y)[(row0 + min(t0 + i, n - 1)) * p.ld_y + ch]);
+            for (int ks = 0; ks < 4; ++ks)
+              umma_f16_ss(tmem + (it & 1) * (2 * RG_CHUNK) + g * RG_CHUNK, desc_advance(da, ks * 32), desc_advance(db, ks * 32), idesc,
+                          k > 0 || ks > 0 ? 1u : 0u);
+          }
+        umma_commit(done + (it & 1));
       }
-      tmem_ld_32x32b_x16(at + (it & 1) * (2 * RG_CHUNK) + t0, zr);
-      tmem_ld_32x32b_x16(at + (it & 1) * (2 * RG_CHUNK) + RG_CHUNK + t0, zi);
-      tmem_ld_wait();
+      __syncwarp();
+      if (next >= L.stages && next < mine) {        // chunk `last` has been read: its stage, and the accumulator before this one
+        const int last = next - L.stages;
+        mbar_wait_warp(used + (last & 1), (last >> 1) & 1, status, ERR_GEMM_PRODUCER_WAIT);
+        tc_fence_after();
+        load_u(next);
+      }
+    }
+  } else {
+    const int l = quarter * 32 + lane;                // lane of the accumulator
+    const bool in = l < tile_channels && c0 + l < p.block;
+    const int c = in ? c0 + l : c0, ch = b * p.block + c;      // lanes without a channel read the tile's first one's
+    const RecChannel<rg_bf16> K(p, ch);
+    const uint32_t at = tmem + (static_cast<uint32_t>(quarter * 32) << 16) + run * GR_RUN;
+    const int u_at = (c >> 6) * (RG_CHUNK * 128) + (c & 7) * 2, u_piece = (c >> 3) & 7;
+    const bool idle = quarter * 32 >= tile_channels;  // the whole warp
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float br2 = -LOG2E * K.br, bi2 = -LOG2E * K.bi, sp2 = -LOG2E * K.sp;
+    for (int it = 0; it < mine; ++it) {
+      const int st = it % L.stages, chunk = chunk_of(it);
+      const int* cd = p.chunks + chunk * 4;
+      const size_t row0 = cd[1] + run * GR_RUN;
+      const int n = idle ? 0 : run_rows(cd[2], run);
+      const size_t wi = (static_cast<size_t>(chunk) * RG_RUNS + run) * 2 * p.C + ch;
+      float A = 1.f, S = 0.f;
+      if (OUT) S = p.ws[wi];
+      mbar_wait_warp(u_full + st, (it / L.stages) & 1, status, ERR_GEMM_MMA_WAIT_FULL);       // u itself is read below
+      mbar_wait_warp(done + (it & 1), (it >> 1) & 1, status, ERR_GEMM_EPI_WAIT);
+      tc_fence_after();
+      const uint8_t* ut = su + st * L.stage + u_at;
+      const rg_bf16* yp = OUT ? static_cast<const rg_bf16*>(p.y) + row0 * p.ld_y + ch : nullptr;
+      rg_bf16* op = OUT ? static_cast<rg_bf16*>(p.out) + row0 * p.ld_out + ch : nullptr;
+      // sixteen tokens from t0 on; WHOLE: all of them exist
+      auto tokens = [&](auto whole, int t0) {
+        constexpr bool WHOLE = decltype(whole)::value;
+        uint32_t zr[16], zi[16];
+        float y[16];
+        if (OUT) {
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int t = run * GR_RUN + t0 + i;
-        const float u = __bfloat162float(*reinterpret_cast<const rg_bf16*>(ut + t * 128 + ((u_piece ^ (t & 7)) << 4)));
-        const float x = -K.sp * sigmoid_fast(__uint_as_float(zr[i]) + K.br);
-        const float a = fast_exp2(1.4426950408889634f * x);
-        const float inc = sqrt_fast(one_minus_exp(2.f * x, a * a)) * sigmoid_fast(__uint_as_float(zi[i]) + K.bi) * u;
-        if (t0 + i < n) {
+          for (int i = 0; i < 16; ++i) y[i] = __bfloat162float(yp[(WHOLE ? t0 + i : min(t0 + i, n - 1)) * p.ld_y]);
+        }
+        tmem_ld_32x32b_x16(at + (it & 1) * (2 * RG_CHUNK) + t0, zr);
+        tmem_ld_32x32b_x16(at + (it & 1) * (2 * RG_CHUNK) + RG_CHUNK + t0, zi);
+        tmem_ld_wait();
+        const uint8_t* ur = ut + (run * GR_RUN + t0) * 128;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float u = __bfloat162float(*reinterpret_cast<const rg_bf16*>(ur + i * 128 + ((u_piece ^ (i & 7)) << 4)));
+          // both sigmoids with one reciprocal: 1 / (A B) gives 1 / A and 1 / B (the exponents are bounded so that A B stays finite)
+          const float ea = 1.f + fast_exp2(fminf(fmaf(-LOG2E, __uint_as_float(zr[i]), br2), 62.f));
+          const float eb = 1.f + fast_exp2(fminf(fmaf(-LOG2E, __uint_as_float(zi[i]), bi2), 62.f));
+          const float q = __fdividef(1.f, ea * eb);
+          const float x = sp2 * (eb * q);             // log2 a
+          const float X = (2.f / LOG2E) * x;
+          float a = fast_exp2(x);
+          // 1 - a^2: where it cancels, the first terms of its series in X = 2 log a (relative error X^2 / 6)
+          const float m = X > -0.01f ? -X * fmaf(0.5f, X, 1.f) : fmaf(-a, a, 1.f);
+          float inc = sqrt_fast(m) * (ea * q) * u;
+          if (!WHOLE && t0 + i >= n) {
+            a = 1.f;
+            inc = 0.f;
+          }
           S = fmaf(a, S, inc);
           if (!OUT) A *= a;
-          if (OUT && in)
-            static_cast<rg_bf16*>(p.out)[(row0 + t0 + i) * p.ld_out + ch] = __float2bfloat16(S * gelu_tanh_t<rg_bf16>(y[i] + K.yb));
+          if (OUT && in && (WHOLE || t0 + i < n))
+            op[static_cast<long long>(t0 + i) * p.ld_out] = __float2bfloat16(S * gelu_tanh_t<rg_bf16>(y[i] + K.yb));
         }
+      };
+#pragma unroll 1
+      for (int t0 = 0; t0 < n; t0 += 16) {            // n is the same for the whole warp
+        if (n - t0 >= 16) tokens(std::true_type{}, t0);
+        else tokens(std::false_type{}, t0);
       }
+      if (!OUT && in) {
+        p.ws[wi] = A;
+        p.ws[wi + p.C] = S;
+      }
+      tc_fence_before();
+      mbar_arrive_warp(used + (it & 1));                         // this warp has read its part of the stage and of the accumulator
     }
-    if (!OUT && in) {
-      p.ws[wi] = A;
-      p.ws[wi + p.C] = S;
-    }
-    tc_fence_before();
-    __syncthreads();                                // the stage and its accumulators have been read
-    tc_fence_after();
-    if (tid == 0 && it + L.stages < mine) load_u(it + L.stages);
   }
   if (*reinterpret_cast<volatile int*>(status) != 0) {     // copies and products in flight land before shared memory and TMEM go away
     const unsigned long long t0 = globaltimer_ns();
@@ -449,7 +501,7 @@ __global__ void __launch_bounds__(RG_THREADS, 1) rec_gates_kernel(const __grid_c
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 0) {
+  if (warp == RG_WARPS) {
     tc_fence_after();
     tmem_dealloc(tmem, RG_TMEM);
   }

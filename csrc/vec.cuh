@@ -44,6 +44,21 @@ __device__ __forceinline__ void vstore8(float* p, const float (&f)[8]) {
   *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
 }
 
+// eight elements that wait in registers as they came from memory
+template <typename T>
+struct Packed8 {
+  uint4 w[sizeof(T) / 2];
+  __device__ __forceinline__ void load(const T* p) {
+#pragma unroll
+    for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) w[i] = reinterpret_cast<const uint4*>(p)[i];
+  }
+  __device__ __forceinline__ void zero() {
+#pragma unroll
+    for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) w[i] = make_uint4(0, 0, 0, 0);
+  }
+  __device__ __forceinline__ void get(float (&f)[8]) const { vload8(reinterpret_cast<const T*>(w), f); }
+};
+
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }

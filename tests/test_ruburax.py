@@ -11,7 +11,7 @@ import torch
 
 import ruburax_oracle as O
 import test_sotazen as S
-from b200fw import ops
+from b200fw import _native, ops
 from b200fw.infer import InferenceConfig, InferenceEngine
 from b200fw.model import registry
 from b200fw.model.ruburax import RuburaxConfig
@@ -287,6 +287,7 @@ def test_gated_recurrence_over_many_chunks(B, n):
             ops.linear_recurrence(u, ops.block_gates(u, wg.view(B, 2 * np_, np_)), gb.view(-1), lam, y, bias[0], out, state, p, np_)
         outs.append(out.float())
         states.append(state)
+    assert _native.read_status() == 0
     near(outs[0].cpu()[:, None], outs[1].cpu()[:, None], run)
     torch.testing.assert_close(states[0], states[1], rtol=2e-3, atol=2e-3)
 
