@@ -21,10 +21,6 @@ class Routing:
     token: torch.Tensor          # int32 [M * top] token of every row
     offsets: torch.Tensor        # int32 [E + 1]
 
-    @property
-    def experts(self) -> int:
-        return self.offsets.numel() - 1
-
 
 def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float,
           joint: Optional[torch.Tensor] = None) -> Routing:
