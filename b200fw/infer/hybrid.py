@@ -30,8 +30,10 @@ class HybridModelRunner(ModelRunner):
         super().__init__(model, pool, manager, partition_size, enable_partitioned)
         self.state: StatePool = manager.state
         self._turns: Dict[tuple, torch.Tensor] = {}
-        # whose pages a layer reads: its own, or those of an earlier layer
-        self._pages = [li if src is None else src for li, src in enumerate(getattr(model, "kv_sources", lambda: [None] * len(model.layers))())]
+        # the layers in the order they run (one may run several times, each time with pages and state of its own), and whose pages
+        # a run reads: its own, or those of an earlier one
+        self._runs = list(getattr(model, "layer_runs", lambda: range(len(model.layers)))())
+        self._pages = [li if src is None else src for li, src in enumerate(getattr(model, "kv_sources", lambda: [None] * len(self._runs))())]
 
     # ---- metadata ----------------------------------------------------------------------------------------
     def prepare_prefill(self, seq_ids: Sequence, starts: Sequence[int], counts: Sequence[int]) -> InferenceContext:
@@ -106,12 +108,12 @@ class HybridModelRunner(ModelRunner):
                 split_plan: Optional[Tuple[int, int]] = None, rows: Optional[torch.Tensor] = None,
                 on_layer=None) -> torch.Tensor:
         """Token ids ``[M]`` (caller's order) -> logits of each sequence's last row, of every row (``all_rows``) or of the
-        caller's rows ``rows`` (int64).  ``on_layer(i, x)`` sees the residual rows (kernel order) after every layer."""
+        caller's rows ``rows`` (int64).  ``on_layer(i, x)`` sees the residual rows (kernel order) after every layer run."""
         m, p = self.model, ctx.portions
         self.forward_calls += 1
         ids = token_ids if ctx.row_order is None else token_ids.index_select(0, ctx.row_order)
         p.ids = ids
-        x, h = m.embed(ids)
+        x, h = m.embed(ids, p, self.state.sequence)
         tables: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
 
         def rope(base: float, dims: int, stretch: Optional[tuple] = None):
@@ -122,9 +124,9 @@ class HybridModelRunner(ModelRunner):
                 tables[key] = ops.rope_rows(p.positions, self._turns[key])
             return tables[key]
 
-        n = len(m.layers)
-        for li, layer in enumerate(m.layers):
-            after = m.layers[li + 1].norm1 if li + 1 < n else None
+        layers = [m.layers[i] for i in self._runs]
+        for li, layer in enumerate(layers):
+            after = layers[li + 1].norm1 if li + 1 < len(layers) else None
             h = layer(x, h, p, self.pool.layer_kv(self._pages[li]), self.state.layers[li], rope, after)
             if on_layer is not None:
                 on_layer(li, x)
@@ -134,6 +136,8 @@ class HybridModelRunner(ModelRunner):
             pick = ctx.row_place
         else:
             pick = ctx.last_token_rows if ctx.is_prefill else None
+        if hasattr(m, "final_norm"):
+            return m.logits_from_hidden(m.final_norm(x, pick))
         return m.logits_from_hidden(ops.rmsnorm_f32(x, m.norm, m.cfg.hidden_size, m.cfg.rms_norm_eps, pick,
                                                         getattr(m, "logit_scale", 1.0)))
 
@@ -176,11 +180,7 @@ def build_portions(starts: Sequence[int], counts: Sequence[int], tables: Sequenc
             first = np.concatenate([[0], np.cumsum((c[ns:] + size - 1) // size)]).astype(np.int32)
             setattr(p, f"chunks{size}", dev(_row_tiles(cu, ns, n, size)))
             setattr(p, f"first{size}", dev(first))
-        pages = (st[ns:] + c[ns:] + 15) // 16
-        first = (np.cumsum(pages) - pages).astype(np.int32)
-        p.ctx_counts = pages.tolist()
-        p.ctx_pages = dev(np.concatenate([bt[ns + i, :k] for i, k in enumerate(p.ctx_counts)]))
-        p.ctx_tables = dev(first[:, None] + np.minimum(np.arange(pages.max(), dtype=np.int32)[None, :], pages[:, None].astype(np.int32) - 1))
+        p.host_long, p.to_device = (st[ns:], c[ns:], bt[ns:]), dev
     return p, order, place
 
 
@@ -200,7 +200,8 @@ def make_cache(model, num_blocks: int, block_size: int, num_slots: int, dtype, d
     mc = model.cfg
     pool = BlockPool(num_blocks, block_size, mc.num_layers, mc.num_kv_heads, mc.head_dim, dtype, device,
                      layer_shapes=model.kv_layer_shapes())
-    return pool, KVCacheManager(pool, block_size, StatePool(num_slots, model.state_layer_shapes(), device))
+    return pool, KVCacheManager(pool, block_size, StatePool(
+        num_slots, model.state_layer_shapes(), device, getattr(model, "state_sequence_shapes", dict)()))
 
 
 @torch.no_grad()

@@ -161,13 +161,15 @@ class BlockPool:
 
 class StatePool:
     """Recurrent state of the sequences being served: a fixed number of slots, each with the fp32 tensors of every layer
-    (``layer_shapes[layer] = {name: shape}``).  A slot belongs to one sequence from its admission until it is freed; it is
+    (``layer_shapes[layer] = {name: shape}``) and what a sequence keeps outside the layers (``sequence = {name: (shape, dtype)}``).  A slot belongs to one sequence from its admission until it is freed; it is
     not cleared in between, because a sequence that starts at position 0 starts from zero whatever its slot holds."""
 
-    def __init__(self, num_slots: int, layer_shapes: List[Dict[str, Tuple[int, ...]]], device="cpu"):
+    def __init__(self, num_slots: int, layer_shapes: List[Dict[str, Tuple[int, ...]]], device="cpu",
+                 sequence: Optional[Dict[str, Tuple[Tuple[int, ...], torch.dtype]]] = None):
         self.num_slots, self.device = num_slots, torch.device(device)
         self.layers = [{n: torch.zeros((num_slots, *s), dtype=torch.float32, device=self.device) for n, s in shapes.items()}
                        for shapes in layer_shapes]
+        self.sequence = {n: torch.zeros((num_slots, *s), dtype=d, device=self.device) for n, (s, d) in (sequence or {}).items()}
         self.free_list: Deque[int] = deque(range(num_slots))
         self.owner: Dict[object, int] = {}
 
@@ -190,7 +192,7 @@ class StatePool:
         return len(self.free_list)
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for l in self.layers for t in l.values())
+        return sum(t.numel() * t.element_size() for l in [*self.layers, self.sequence] for t in l.values())
 
 
 class BlockTable:

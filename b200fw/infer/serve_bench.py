@@ -299,10 +299,10 @@ def sotazen_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     if lengths is not None:
         from ..ops import latent
         k, v = _bf(pages * 16, H * dq), _bf(pages * 16, H * dv)
-        t("latent prompt attention alone", lambda: latent.expanded_attention(q, k, v, out, p, H, dq, dv, b["scale"], sink, 0, n, p.ctx_tables),
+        t("latent prompt attention alone", lambda: latent.expanded_attention(q, k, v, out, p, H, dq, dv, b["scale"], sink, 0, n, p.context().tables),
           M * H * (dq + dv) * 4, 2.0 * pairs * H * (dq + dv))
         rows = torch.empty(pages * 16, R, device=DEV, dtype=torch.bfloat16)
-        t("latent_gather", lambda: latent.gather(pg, p.ctx_pages, rows), rows.numel() * 4)
+        t("latent_gather", lambda: latent.gather(pg, p.context().pages, rows), rows.numel() * 4)
     _gemm(t, "gemm latent o (fp32)", M, W, H * dv, True)
     if lengths is None:
         _gemm(t, "gemm logits (fp32)", M, V, W, True)

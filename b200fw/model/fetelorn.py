@@ -230,7 +230,7 @@ class FetelornModel(nn.Module):
         return [l.state_shapes() for l in self.layers]
 
     # ---- pieces the runner calls ------------------------------------------------------------------------------
-    def embed(self, ids: torch.Tensor):
+    def embed(self, ids: torch.Tensor, p=None, state=None):
         """The residual stream's first rows (fp32), and what the first layer reads if that is not its own norm's business."""
         return ops.embedding_f32(ids, self.embed_tokens, self.cfg.vocab_size), None
 

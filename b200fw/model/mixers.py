@@ -50,16 +50,18 @@ class RowSplitSlot:
 
 @dataclass
 class HalvesSlot:
-    """Per-head channels (dimension 1 of ``view [heads, d, ...]``) whose first ``rot`` are rotated in pairs of halves (channel i with
-    i + rot / 2) in the checkpoint and stored as neighbours (2 i, 2 i + 1): a score does not change when queries and keys are
-    reordered alike, and the kernels rotate neighbours."""
+    """Per-head channels (dimension 1 of ``view [heads, d, ...]``) of which ``rot``, from channel ``at`` on, are rotated in pairs of
+    halves (the i-th of them with the one rot / 2 further) in the checkpoint and stored as neighbours (2 i, 2 i + 1): a score does not
+    change when queries and keys are reordered alike, and the kernels rotate neighbours."""
     view: torch.Tensor
     rot: int
     shape: Tuple[int, ...]
+    at: int = 0
 
     def _order(self) -> torch.Tensor:
-        half, d = self.rot // 2, self.view.shape[1]
-        return torch.cat([torch.arange(self.rot).reshape(2, half).t().reshape(-1), torch.arange(self.rot, d)]).to(self.view.device)
+        half, d, a = self.rot // 2, self.view.shape[1], self.at
+        turned = a + torch.arange(self.rot).reshape(2, half).t().reshape(-1)
+        return torch.cat([torch.arange(a), turned, torch.arange(a + self.rot, d)]).to(self.view.device)
 
     def load(self, t: torch.Tensor) -> None:
         self.view.copy_(t.to(self.view.device).reshape(self.view.shape)[:, self._order()].to(self.view.dtype))
@@ -410,22 +412,29 @@ class DifferentialAttention(nn.Module):
 
 class LatentAttention(nn.Module):
     """Softmax attention whose keys and values are made from one cached latent per token, plus one rotated key part that all
-    heads share; a sink per head.  ``w_key`` holds the key projection beside an identity for the rotated part."""
+    heads share.  ``w_key`` holds the key projection beside an identity for the rotated part.  Options: queries from a normed latent of
+    their own (``q_rank``), a sliding ``window`` (0: none), a ``sink`` per head, a sigmoid ``gate`` per head on the output, rotated
+    channels paired as ``halves`` in the checkpoint instead of as neighbours."""
 
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float, rot_base: float,
-                 eps: float, dtype, device):
+                 eps: float, dtype, device, q_rank: Optional[int] = None, window: int = 0, sink: bool = True, gate: bool = False,
+                 halves: bool = False):
         super().__init__()
         if rot_dim % 2 or rot_dim < 2:
             raise ValueError(f"latent attention: the rotated size {rot_dim} must be even and positive")
-        self.heads, self.dim, self.rot_dim, self.vdim, self.rank = heads, dim, rot_dim, vdim, rank
+        self.heads, self.dim, self.rot_dim, self.vdim, self.rank, self.q_rank = heads, dim, rot_dim, vdim, rank, q_rank
         self.scale, self.eps, self.rot = float(scale), eps, (float(rot_base), int(rot_dim))
-        self.in_proj = PackedRows(hidden, [("q", heads, dim + rot_dim), ("c", 1, rank), ("kr", 1, rot_dim)], dtype, device)
+        self.window, self.halves = int(window), halves
+        query = ("q", heads, dim + rot_dim) if q_rank is None else ("dq", 1, q_rank)
+        self.in_proj = PackedRows(hidden, [query, ("c", 1, rank), ("kr", 1, rot_dim)] + ([("g", 1, heads)] if gate else []), dtype, device)
+        self.q_up = None if q_rank is None else PackedRows(q_rank, [("uq", heads, dim + rot_dim)], dtype, device)
+        self.q_norm = None if q_rank is None else _param(pad8(q_rank), dtype=dtype, device=device)
         self.c_norm = _param(pad8(rank), dtype=dtype, device=device)
         self.w_key = _param(heads, pad8(dim + rot_dim), pad8(rank) + pad8(rot_dim), dtype=dtype, device=device)
         i = torch.arange(rot_dim, device=device)
         self.w_key.data[:, dim + i, pad8(rank) + i] = 1.0
         self.w_value = _param(heads, pad8(vdim), pad8(rank), dtype=dtype, device=device)
-        self.sink = _param(heads, dtype=dtype, device=device)
+        self.sink = _param(heads, dtype=dtype, device=device) if sink else None
         self.o = PackedCols(hidden, [("o", heads, vdim)], dtype, device)
 
     def kv_shape(self) -> Tuple[int, int, int]:
@@ -435,25 +444,39 @@ class LatentAttention(nn.Module):
         return {}
 
     def tensors(self, prefix: str) -> Dict[str, Slot]:
-        H, hidden = self.heads, self.in_proj.in_features
-        t = {prefix + "q": self.in_proj.slot("q"),
-             prefix + "dkv": RowSplitSlot([(self.in_proj.slot("c"), self.rank), (self.in_proj.slot("kr"), self.rot_dim)],
-                                          (self.rank + self.rot_dim, hidden)),
+        H, hidden, P = self.heads, self.in_proj.in_features, self.in_proj
+
+        def turned(s: Slot, at: int):
+            return HalvesSlot(s.view, self.rot_dim, s.shape, at) if self.halves else s
+        t = {prefix + "dkv": RowSplitSlot([(P.slot("c"), self.rank), (turned(P.slot("kr"), 0), self.rot_dim)], (self.rank + self.rot_dim, hidden)),
              prefix + "dkv.norm": Slot(self.c_norm.data[:self.rank], (self.rank,)),
              prefix + "uk": Slot(self.w_key.data[:, :self.dim, :self.rank], (H * self.dim, self.rank)),
-             prefix + "uv": Slot(self.w_value.data[:, :self.vdim, :self.rank], (H * self.vdim, self.rank)),
-             prefix + "sink": Slot(self.sink.data, (H,)), prefix + "o": self.o.slot("o")}
+             prefix + "uv": Slot(self.w_value.data[:, :self.vdim, :self.rank], (H * self.vdim, self.rank)), prefix + "o": self.o.slot("o")}
+        if self.q_up is None:
+            t[prefix + "q"] = turned(P.slot("q"), self.dim)
+        else:
+            t |= {prefix + "dq": P.slot("dq"), prefix + "dq.norm": Slot(self.q_norm.data[:self.q_rank], (self.q_rank,)),
+                  prefix + "uq": turned(self.q_up.slot("uq"), self.dim)}
+        if "g" in P.sections:
+            t[prefix + "g"] = P.slot("g")
+        if self.sink is not None:
+            t[prefix + "sink"] = Slot(self.sink.data, (H,))
         return t
 
     def run(self, h: torch.Tensor, p, kv: Tuple[torch.Tensor, torch.Tensor], state, rope) -> Tuple[torch.Tensor, Dict]:
         """fp32 ``[M, hidden]``."""
-        P = self.in_proj
+        P, (cos, sin) = self.in_proj, rope(*self.rot)
         y = P(h)
-        q = P.cols(y, "q")
-        ops.latent_store(q, P.cols(y, "c"), P.cols(y, "kr"), kv[0], p, self.heads, self.dim, self.rank, self.rot_dim, self.c_norm,
-                         *rope(*self.rot), self.eps)
+        cq = P.cols(y, "dq") if self.q_up is not None else None
+        q = P.cols(y, "q") if cq is None else None
+        ops.latent_store(q, P.cols(y, "c"), P.cols(y, "kr"), kv[0], p, self.heads, self.dim, self.rank, self.rot_dim, self.c_norm, cos, sin,
+                         self.eps, cq, self.q_norm, self.q_rank or 0)
+        turn = None
+        if cq is not None:
+            q, turn = self.q_up(cq), (cos, sin, self.dim)
+        gate = P.cols(y, "g")[:, :self.heads] if "g" in P.sections else None
         out = self.o.buffer(y.shape[0])
-        ops.latent_attention(q, kv[0], out, p, self.w_key, self.w_value, self.scale, self.sink)
+        ops.latent_attention(q, kv[0], out, p, self.w_key, self.w_value, self.scale, self.sink, self.window, gate, turn)
         return self.o(out), {}
 
 
@@ -481,13 +504,16 @@ class GatedFF(nn.Module):
 
 
 class ExpertFF(nn.Module):
-    """Mixture of gated feed-forward experts with sigmoid scores, a learned correction of the choice, a choice limited to the best
-    groups, and a shared expert behind a gate of its own.  Router logits and the shared gate are one 32-bit product.  A shared expert of
-    the experts' size is stored as one more of them, which every token takes."""
+    """Mixture of gated feed-forward experts with sigmoid or softmax scores, a learned correction of the choice, a choice limited to the
+    best groups, and a shared expert behind a gate of its own.  Router logits and the shared gate are one 32-bit product.  A shared expert
+    of the experts' size is stored as one more of them, which every token takes.  ``clamped = (alpha, limit)``: the experts' gated form
+    (:func:`b200fw.ops.expert_glu`).  ``beside``: sections of other projections of the same input, made by the router's product."""
 
     def __init__(self, hidden: int, experts: int, inner: int, top: int, groups: int, keep: int, scale: float,
-                 shared_inner: Optional[int], dtype, device):
+                 shared_inner: Optional[int], dtype, device, score: str = "sigmoid", corrected: bool = True,
+                 clamped: Optional[Tuple[float, float]] = None, beside: List[Tuple[str, int, int]] = ()):
         super().__init__()
+        self.score, self.clamped = score, clamped
         if groups < 1 or experts % groups or not 1 <= keep <= groups:
             raise ValueError(f"experts: {experts} do not form {groups} equal groups of which {keep} are kept")
         if not 1 <= top <= keep * (experts // groups):
@@ -497,9 +523,9 @@ class ExpertFF(nn.Module):
         all_ = experts + int(self.joint)
         self.w_in = _param(all_, 2, pad8(inner), pad8(hidden), dtype=dtype, device=device)
         self.w_out = _param(all_, pad8(hidden), pad8(inner), dtype=dtype, device=device)
-        self.correction = _param(experts, dtype=dtype, device=device)
+        self.correction = _param(experts, dtype=dtype, device=device) if corrected else None
         self.shared = GatedFF(hidden, shared_inner, dtype, device) if shared_inner is not None and not self.joint else None
-        self.router = PackedRows(hidden, [("router", 1, experts)] + ([("sg", 1, 1)] if shared_inner is not None else []), dtype, device)
+        self.router = PackedRows(hidden, [("router", 1, experts)] + ([("sg", 1, 1)] if shared_inner is not None else []) + list(beside), dtype, device)
         self.shared_row = self.router.sections["sg"][0] if shared_inner is not None else -1
 
     def tensors(self, prefix: str) -> Dict[str, Slot]:
@@ -510,7 +536,8 @@ class ExpertFF(nn.Module):
             t[p + "gate"], t[p + "up"] = (Slot(self.w_in.data[e, i, :F, :H], (F, H)) for i in range(2))
             t[p + "down"] = Slot(self.w_out.data[e, :H, :F], (H, F))
         t[prefix + "router"] = self.router.slot("router")
-        t[prefix + "correction"] = Slot(self.correction.data, (self.n,))
+        if self.correction is not None:
+            t[prefix + "correction"] = Slot(self.correction.data, (self.n,))
         if self.shared is not None:
             t |= self.shared.tensors(prefix + "shared.")
         if self.shared_row >= 0:
@@ -521,8 +548,54 @@ class ExpertFF(nn.Module):
         """``x += coef * norm(ff(h))``; the new ``x`` in the activation dtype."""
         r, gate = ops.router(h, self.router.weight, self.shared_row, self.correction, self.top, self.groups, self.keep, self.scale, self.joint)
         shared = None if self.shared is None else self.shared.run(h)
-        rows = ops.expert_down(ops.expert_glu(h, self.w_in, r), self.w_out, r)
-        return ops.moe_norm_add(x, rows, r, shared, gate, norm, coef, n, eps)
+        return ops.moe_norm_add(x, self._experts(h, r), r, shared, gate, norm, coef, n, eps)
+
+    def _experts(self, h: torch.Tensor, r: "ops.Routing") -> torch.Tensor:
+        return ops.expert_down(ops.expert_glu(h, self.w_in, r, self.clamped), self.w_out, r)
+
+    def run(self, h: torch.Tensor) -> Tuple[Tuple[torch.Tensor, "ops.Routing"], torch.Tensor]:
+        """``(rows, routing)`` for the weighted sum of a token's experts, and the router's whole product (fp32), ``beside`` sections
+        included.  Without a shared expert."""
+        assert self.shared_row < 0
+        z = self.router.fp32(h)
+        r = ops.route(z, self.correction, self.top, self.groups, self.keep, self.scale, score=self.score, experts=self.n)
+        return (self._experts(h, r), r), z
+
+
+class LayerNorm(nn.Module):
+    """Weight and bias of a layer norm over ``hidden`` channels, zero in the padding."""
+
+    def __init__(self, hidden: int, dtype, device):
+        super().__init__()
+        self.hidden = hidden
+        self.weight, self.bias = (_param(pad8(hidden), dtype=dtype, device=device) for _ in range(2))
+
+    @property
+    def pair(self) -> Tuple[torch.Tensor, torch.Tensor]:
+        return self.weight, self.bias
+
+    def tensors(self, name: str) -> Dict[str, Slot]:
+        return {name: Slot(self.weight.data[:self.hidden], (self.hidden,)), name + ".b": Slot(self.bias.data[:self.hidden], (self.hidden,))}
+
+
+class InputConv(nn.Module):
+    """A short causal convolution of a sublayer's input per channel, added to it: ``h + conv(h)``."""
+
+    def __init__(self, hidden: int, taps: int, dtype, device):
+        super().__init__()
+        if not 1 <= taps <= 17:
+            raise ValueError(f"input convolution: {taps} taps (1 to 17)")
+        self.hidden = hidden
+        self.taps = _param(pad8(hidden), taps, dtype=dtype, device=device)
+
+    def state_shape(self) -> Tuple[int, ...]:
+        return (self.taps.shape[0], self.taps.shape[1] - 1)
+
+    def slot(self) -> Slot:
+        return Slot(self.taps.data[:self.hidden], (self.hidden, self.taps.shape[1]))
+
+    def forward(self, h: torch.Tensor, state: torch.Tensor, p) -> torch.Tensor:
+        return ops.causal_conv(h, None, self.taps, None, state, p, add_input=True)
 
 
 class TokenInput(nn.Module):

@@ -14,6 +14,7 @@ from . import hf_io
 from .config import PRESETS as DENSE_PRESETS
 from .config import ModelConfig
 from .fetelorn import FETELORN_PRESETS, FetelornConfig, FetelornModel
+from .lufivik import LUFIVIK_PRESETS, LufivikConfig, LufivikModel
 from .qwen3 import ParallelTransformerModel
 from .ruburax import RUBURAX_PRESETS, RuburaxConfig, RuburaxModel
 from .sotazen import SOTAZEN_PRESETS, SotazenConfig, SotazenModel
@@ -92,8 +93,11 @@ ARCHITECTURES: Dict[str, Architecture] = {
                             _load_slots_at, ("host", "gemm", "residual", "linear_state", "retention_chunk", "recurrence", "moe",
                                              "attention_rows", "attention_decode", "attention_latent", "attention_fwd", "sampling"),
                             float32=True),
+    "Lufivik": Architecture("Lufivik", LufivikConfig, lambda path: LufivikConfig.from_dict(_config_json(path)), LufivikModel,
+                            _load_slots_at, ("host", "gemm", "residual", "recurrence", "moe", "attention_decode", "attention_latent",
+                                             "attention_fwd", "sampling"), float32=True),
 }
-PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS, **SOTAZEN_PRESETS, **RUBURAX_PRESETS}
+PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **FETELORN_PRESETS, **SOTAZEN_PRESETS, **RUBURAX_PRESETS, **LUFIVIK_PRESETS}
 
 
 def architecture_at(path: str) -> Architecture:

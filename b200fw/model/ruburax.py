@@ -291,7 +291,7 @@ class RuburaxModel(nn.Module):
         return [l.state_shapes() for l in self.layers]
 
     # ---- pieces the runner calls ------------------------------------------------------------------------------
-    def embed(self, ids: torch.Tensor):
+    def embed(self, ids: torch.Tensor, p=None, state=None):
         """The residual stream's first rows (fp32) and the same in the activation dtype, which the first layer reads."""
         return ops.embedding_f32(ids, self.embed_tokens, self.cfg.vocab_size, h=True)
 

@@ -1,9 +1,10 @@
-"""Mixture of experts: sigmoid scores, a choice limited to the best groups of experts, grouped products over the rows each expert
-was given, and the weighted sum of a token's experts (with a gated shared expert) added to the residual through a norm."""
+"""Mixture of experts: sigmoid or softmax scores, a choice limited to the best groups of experts, grouped products over the rows each
+expert was given, and the weighted sum of a token's experts (with a gated shared expert) added to the residual through a norm
+(:func:`b200fw.ops.branch_add` does the same through a layer norm, with a gate per channel)."""
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -22,15 +23,18 @@ class Routing:
     offsets: torch.Tensor        # int32 [E + 1]
 
 
-def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float,
-          joint: Optional[torch.Tensor] = None) -> Routing:
-    """``logits [M, >= E]`` fp32, ``correction [E]``: scores ``s = sigmoid(logits)``; the experts are ``groups`` equal groups of
-    neighbours, a group counts by the sum of its two largest ``s + correction``, and the ``top`` largest ``s + correction`` of the
-    ``keep`` best groups are chosen, with weight ``s * scale``.  Ties go to the lower index."""
-    M, E = logits.shape[0], correction.numel()
+def route(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int, scale: float,
+          joint: Optional[torch.Tensor] = None, score: str = "sigmoid", experts: int = 0) -> Routing:
+    """``logits [M, >= E]`` fp32, ``correction [E]`` (None: zero, ``experts`` then says how many there are): scores ``s =
+    sigmoid(logits)``, or their ``softmax`` over all experts; the experts are ``groups`` equal groups of neighbours, a group counts by
+    the sum of its two largest ``s + correction``, and the ``top`` largest ``s + correction`` of the ``keep`` best groups are chosen,
+    with weight ``s * scale``.  Ties go to the lower index."""
+    M, E = logits.shape[0], experts if correction is None else correction.numel()
+    assert score in ("sigmoid", "softmax") and E > 0
     if not logits.is_cuda:
-        s = torch.sigmoid(logits[:, :E])
-        c = s + correction.float()
+        z = logits[:, :E]
+        s = torch.softmax(z, -1) if score == "softmax" else torch.sigmoid(z)
+        c = s + correction.float() if correction is not None else z if keep == groups else s
         if keep < groups:
             per = E // groups
             gs = c.reshape(M, groups, per).topk(min(2, per), -1).values.sum(-1)
@@ -54,7 +58,8 @@ def route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int,
     nv.check(nv.lib().b2_moe_route(
         nv.ptr(logits), nv.ctypes.c_longlong(logits.stride(0)), nv.ptr(joint), nv.ctypes.c_longlong(joint.stride(0) if more else 0), more,
         nv.ptr(correction), nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token),
-        nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep, nv.ctypes.c_float(scale), _f32(correction), nv.stream_ptr()), "moe_route")
+        nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep, nv.ctypes.c_float(scale), int(score == "softmax"),
+        int(correction is not None and correction.dtype == torch.float32), nv.stream_ptr()), "moe_route")
     nv.count_launch(2 if M * (top + more) <= 16384 else 3)
     return r
 
@@ -82,7 +87,7 @@ def router(h: torch.Tensor, w: torch.Tensor, shared_row: int, correction: torch.
     nv.check(nv.lib().b2_moe_router(
         nv.ptr(h), cl(h.stride(0)), nv.ptr(w), cl(w.stride(0)), N, h.shape[1], shared_row, nv.ptr(gate), more,
         nv.ptr(correction), nv.ptr(r.weights), nv.ptr(r.place), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(work), M, E, top, groups, keep,
-        nv.ctypes.c_float(scale), nv.stream_ptr()), "moe_router")
+        nv.ctypes.c_float(scale), 0, nv.stream_ptr()), "moe_router")
     nv.count_launch(2 if M * (top + more) <= 16384 else 3)
     return r, gate
 
@@ -129,9 +134,10 @@ def glu_linear(h: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     nv.count_launch()
 
 
-def expert_glu(h: torch.Tensor, w: torch.Tensor, r: Routing) -> torch.Tensor:
+def expert_glu(h: torch.Tensor, w: torch.Tensor, r: Routing, clamped: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """``silu(W_gate h) * (W_up h)`` of every (token, choice) pair in the routing's row order; ``h [M, K]``, ``w [E, 2, F, K]``
-    (gate, up): ``[M * top, F]``."""
+    (gate, up): ``[M * top, F]``.  ``clamped = (alpha, limit)``: with ``g = min(W_gate h, limit)`` and ``u = clamp(W_up h, -limit,
+    limit)`` it is ``g sigmoid(alpha g) (u + 1)`` instead."""
     E, _, F, K = w.shape
     P = r.token.numel()
     out = torch.empty((P, F), device=h.device, dtype=h.dtype)
@@ -139,12 +145,21 @@ def expert_glu(h: torch.Tensor, w: torch.Tensor, r: Routing) -> torch.Tensor:
         off = r.offsets.tolist()
         for e in range(E):
             x = h[r.token[off[e]:off[e + 1]].long()].float()
-            out[off[e]:off[e + 1]] = (torch.nn.functional.silu(x @ w[e, 0].float().t()) * (x @ w[e, 1].float().t())).to(h.dtype)
+            g, u = x @ w[e, 0].float().t(), x @ w[e, 1].float().t()
+            if clamped is not None:
+                alpha, limit = clamped
+                g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+                y = g * torch.sigmoid(alpha * g) * (u + 1.0)
+            else:
+                y = torch.nn.functional.silu(g) * u
+            out[off[e]:off[e + 1]] = y.to(h.dtype)
         return out
+    alpha, limit = clamped if clamped is not None else (0.0, 0.0)
     assert h.stride(1) == 1 and w.is_contiguous()
     rows = torch.empty((P, K), device=h.device, dtype=h.dtype) if h.dtype == torch.bfloat16 and P >= GATHER_ROWS * E else None
     nv.check(nv.lib().b2_moe_glu(nv.ptr(h), nv.ctypes.c_longlong(h.stride(0)), nv.ptr(w), nv.ptr(r.token), nv.ptr(r.offsets), nv.ptr(rows),
-                                 nv.ptr(out), h.shape[0], P, E, F, K, _f32(h), nv.stream_ptr()), "moe_glu")
+                                 nv.ptr(out), h.shape[0], P, E, F, K, int(clamped is not None), nv.ctypes.c_float(alpha),
+                                 nv.ctypes.c_float(limit), _f32(h), nv.stream_ptr()), "moe_glu")
     nv.count_launch(1 if rows is None else 2)
     return out
 

@@ -2,8 +2,9 @@
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Tuple
+from typing import Callable, Dict, List, Optional, Tuple
 
+import numpy as np
 import torch
 
 
@@ -36,11 +37,10 @@ class Portions:
     chunks128: Optional[torch.Tensor] = None
     first128: Optional[torch.Tensor] = None
     max_long: int = 0
-    # contexts of the long portions laid out page after page: int32 [pages] page of the pool, int32 [nlong, max pages] where a
-    # sequence's pages are in that layout, pages per sequence
-    ctx_pages: Optional[torch.Tensor] = None
-    ctx_tables: Optional[torch.Tensor] = None
-    ctx_counts: Optional[List[int]] = None
+    # the long portions on the host: int32 [nlong] starts and counts, [nlong, max_blocks] pages; and the copy to the device
+    host_long: Optional[Tuple[np.ndarray, np.ndarray, np.ndarray]] = None
+    to_device: Optional[Callable[[np.ndarray], torch.Tensor]] = None
+    contexts: Dict[int, "Context"] = field(default_factory=dict)
     ids: Optional[torch.Tensor] = None       # int64 [M] token of every row, for layers that look tokens up
     plans: Dict[Tuple[int, int, int], torch.Tensor] = field(default_factory=dict)    # decode_plan: (rows, window, tile) -> tile counts
     ragged: bool = True                      # False: every sequence is one row (decode): row r is sequence r
@@ -48,3 +48,25 @@ class Portions:
     @property
     def rows(self) -> int:
         return self.positions.shape[0]
+
+    def context(self, window: int = 0) -> "Context":
+        """What the long portions see (``window > 0``: of so many tokens back), laid out page after page."""
+        if window not in self.contexts:
+            starts, counts, tables = self.host_long
+            first = np.maximum(starts - window + 1, 0) // 16 if window > 0 else np.zeros_like(starts)
+            end = (starts + counts + 15) // 16
+            n = end - first
+            base = (np.cumsum(n) - n).astype(np.int32)
+            page = np.arange(end.max(), dtype=np.int32)[None, :]
+            place = base[:, None] + np.clip(page - first[:, None], 0, n[:, None] - 1)
+            self.contexts[window] = Context(
+                self.to_device(np.concatenate([tables[i, a:e] for i, (a, e) in enumerate(zip(first, end))])),
+                self.to_device(place.astype(np.int32)), n.tolist())
+        return self.contexts[window]
+
+
+@dataclass
+class Context:
+    pages: torch.Tensor                      # int32 [sum of counts] page of the pool
+    tables: torch.Tensor                     # int32 [nlong, max pages] where a sequence's pages are in that layout
+    counts: List[int]                        # pages per sequence

@@ -5,6 +5,8 @@
 Channels are laid out in blocks padded to a multiple of eight (``np`` channels each); padding channels stay zero."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import _native as nv
@@ -15,28 +17,32 @@ from .residual import _f32, gelu_tanh
 DECAY_RATE = 8.0      # a = sigmoid-gated exp(-DECAY_RATE softplus(lam))
 
 
-def causal_conv(x: torch.Tensor, x_bias: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, conv_state: torch.Tensor,
-                p: Portions) -> torch.Tensor:
-    """Per channel ``sum_j taps[:, K-1-j] (x + x_bias)[t - j] + bias``, zeros before the sequence's start.  ``x [M, C]`` (a column
-    slice), ``taps [C, K]``; the K - 1 inputs before the portion come from ``conv_state [slots, C, K-1]``, which is replaced."""
+def causal_conv(x: torch.Tensor, x_bias: Optional[torch.Tensor], taps: torch.Tensor, bias: Optional[torch.Tensor],
+                conv_state: torch.Tensor, p: Portions, add_input: bool = False) -> torch.Tensor:
+    """Per channel ``sum_j taps[:, K-1-j] (x + x_bias)[t - j] + bias``, zeros before the sequence's start; ``add_input``: and the
+    input itself, ``(x + x_bias)[t]``.  ``x [M, C]`` (a column slice), ``taps [C, K]``; the K - 1 inputs before the portion come from
+    ``conv_state [slots, C, K-1]``, which is replaced."""
     M, C = x.shape
     K = taps.shape[1]
     if not x.is_cuda:
-        xf, tf = x.float() + x_bias.float(), taps.float()
+        xf, tf = x.float() + (0 if x_bias is None else x_bias.float()), taps.float()
         u = torch.zeros(M, C)
         for a, e, start, slot in _cpu_sequences(p):
             past = torch.zeros(K - 1, C) if start == 0 else conv_state[slot].t()
             full = torch.cat([past, xf[a:e]], 0)
             for j in range(K):
                 u[a:e] += tf[:, j] * full[j:j + e - a]
-            u[a:e] += bias.float()
+            if bias is not None:
+                u[a:e] += bias.float()
+            if add_input:
+                u[a:e] += xf[a:e]
             conv_state[slot] = full[full.shape[0] - (K - 1):].t()
         return u.to(x.dtype)
     u = torch.empty((M, C), device=x.device, dtype=x.dtype)
     nv.check(nv.lib().b2_causal_conv(
         nv.ptr(x), nv.ctypes.c_longlong(x.stride(0)), nv.ptr(x_bias), nv.ptr(taps), nv.ptr(bias), nv.ptr(conv_state), nv.ptr(u),
-        nv.ptr(p.cu), nv.ptr(p.starts), nv.ptr(p.slots), nv.ptr(p.tiles), p.tiles.shape[0], C, K, _f32(x), nv.stream_ptr()),
-        "causal_conv")
+        nv.ptr(p.cu), nv.ptr(p.starts), nv.ptr(p.slots), nv.ptr(p.tiles), p.tiles.shape[0], C, K, int(add_input), _f32(x),
+        nv.stream_ptr()), "causal_conv")
     nv.count_launch()
     return u
 
@@ -49,7 +55,7 @@ def block_gates(u: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     out = torch.empty((u.shape[0], B * n2), device=u.device, dtype=torch.float32)
     nv.check(nv.lib().b2_head_linear(
         nv.ptr(u), nv.ptr(w), nv.ptr(out), nv.ctypes.c_longlong(u.stride(0)), nv.ctypes.c_longlong(out.stride(0)), u.shape[0], B, n2, n,
-        n, n2, 0, _f32(u), 1, nv.stream_ptr()), "head_linear")
+        n, n2, 0, None, None, 0, 0, None, nv.ctypes.c_longlong(0), _f32(u), 1, nv.stream_ptr()), "head_linear")
     nv.count_launch()
     return out
 

@@ -1,5 +1,6 @@
-"""Ops around a 32-bit residual stream: embedding into it, RMS norm out of it, normed branches added to it, gated activations
-over column slices or with a table of per-token vectors, rotary tables for a batch's positions.
+"""Ops around a 32-bit residual stream: embedding into it (of tokens, or of tokens and pairs of neighbours), RMS norm or layer norm
+out of it, normed branches added to it, gated activations over column slices or with a table of per-token vectors, rotary tables for
+a batch's positions.
 
 Activations and residual rows are padded to a multiple of eight columns (:func:`pad8`); the padding is zero."""
 from __future__ import annotations
@@ -10,6 +11,7 @@ from typing import Optional, Tuple
 import torch
 
 from .. import _native as nv
+from .portions import Portions
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -97,6 +99,83 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, coef: float, n: 
                                   nv.ctypes.c_float(eps), nv.ctypes.c_float(y_scale), _f32(w), nv.stream_ptr()), "norm_add")
     nv.count_launch()
     return x if h is None else h
+
+
+Norm = Tuple[torch.Tensor, torch.Tensor]      # weight and bias of a layer norm, zero past the real columns
+
+
+def _layer_norm(x: torch.Tensor, w: Norm, n: int, eps: float) -> torch.Tensor:
+    """fp32 rows ``x [M, ld]``, zero past ``n``."""
+    d = x - x[:, :n].mean(-1, keepdim=True)
+    return d * torch.rsqrt((d[:, :n] * d[:, :n]).mean(-1, keepdim=True) + eps) * w[0].float() + w[1].float()
+
+
+def layernorm_f32(x: torch.Tensor, w: Norm, n: int, eps: float, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Layer norm of ``x[rows]`` (``rows`` int64 selects and orders) over its ``n`` real columns, in the weight's dtype."""
+    if not x.is_cuda:
+        return _layer_norm(x if rows is None else x[rows], w, n, eps).to(w[0].dtype)
+    M = x.shape[0] if rows is None else rows.numel()
+    h = torch.empty((M, x.shape[1]), device=x.device, dtype=w[0].dtype)
+    nv.check(nv.lib().b2_layernorm_f32(nv.ptr(x), nv.ptr(w[0]), nv.ptr(w[1]), nv.ptr(h), nv.ptr(rows), M, x.shape[1], n, nv.ctypes.c_float(eps),
+                                       _f32(h), nv.stream_ptr()), "layernorm_f32")
+    nv.count_launch()
+    return h
+
+
+def embedding_pairs(ids: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, last: torch.Tensor, p: Portions, vocab: int,
+                    mul_prev: int, mul_cur: int, w: Norm, n: int, eps: float, next_norm: Norm) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Layer norm of ``table[id] + pairs[(before * mul_prev + id * mul_cur) mod buckets]``, ``before`` being the sequence's token before
+    this one; the first token of a sequence takes the last of the ``buckets + 1`` rows.  ``last [slots]`` int32 keeps every sequence's
+    last token between steps.  Returns the rows in 32-bit and their layer norm with ``next_norm`` in the table's dtype."""
+    buckets = pairs.shape[0] - 1
+    if not table.is_cuda:
+        cu, slots, row = p.cu.tolist(), p.slots.tolist(), torch.full((ids.numel(),), buckets)
+        for s, start in enumerate(p.starts.tolist()):
+            a, e = cu[s], cu[s + 1]
+            if e > a and slots[s] >= 0:
+                before = torch.cat([last[slots[s]].reshape(1).long(), ids[a:e - 1].long()])
+                row[a:e] = (before * mul_prev + ids[a:e].long() * mul_cur) % buckets
+                if start == 0:
+                    row[a] = buckets
+                last[slots[s]] = ids[e - 1]
+        x = _layer_norm(table[ids].float() + pairs[row].float(), w, n, eps)
+        return x, _layer_norm(x, next_norm, n, eps).to(table.dtype)
+    x = torch.empty((ids.numel(), table.shape[1]), device=table.device, dtype=torch.float32)
+    h = torch.empty(x.shape, device=x.device, dtype=table.dtype)
+    cl = nv.ctypes.c_longlong
+    nv.check(nv.lib().b2_embed_pairs(
+        nv.ptr(ids), nv.ptr(table), nv.ptr(pairs), nv.ptr(last), nv.ptr(p.cu), nv.ptr(p.row_seq), nv.ptr(p.positions), nv.ptr(p.slots),
+        nv.ptr(w[0]), nv.ptr(w[1]), nv.ptr(next_norm[0]), nv.ptr(next_norm[1]), nv.ptr(x), nv.ptr(h), ids.numel(), x.shape[1], n, vocab,
+        cl(buckets), cl(mul_prev), cl(mul_cur), nv.ctypes.c_float(eps), _f32(table), nv.stream_ptr()), "embed_pairs")
+    nv.count_launch()
+    return x, h
+
+
+def branch_add(x: torch.Tensor, y, w: Norm, n: int, eps: float, gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None,
+               scale: Optional[torch.Tensor] = None, next_norm: Optional[Norm] = None) -> Optional[torch.Tensor]:
+    """In place ``x += scale * norm(y * sigmoid(gate + gate_bias))``, the layer norm having weight and bias ``w``; returns the layer norm
+    of the new ``x`` with ``next_norm`` in the weights' dtype when that is given.  ``y``: fp32 ``[M, ld]``, or ``(rows, routing)``: the
+    weighted sum of every token's expert rows.  ``gate [M, ld]`` (a column slice, fp32 or the weights' dtype), ``gate_bias`` and
+    ``scale [ld]`` are optional."""
+    rows, r = y if isinstance(y, tuple) else (None, None)
+    if not x.is_cuda:
+        t = y if r is None else (rows[r.place.long()].float() * r.weights[:, :, None]).sum(1)
+        if gate is not None:
+            t = t * torch.sigmoid(gate.float() + gate_bias.float())
+        t = _layer_norm(t, w, n, eps)
+        x += t if scale is None else scale.float() * t
+        return None if next_norm is None else _layer_norm(x, next_norm, n, eps).to(w[0].dtype)
+    h = None if next_norm is None else torch.empty(x.shape, device=x.device, dtype=w[0].dtype)
+    nw, nb = (None, None) if next_norm is None else next_norm
+    assert gate is None or (gate.stride(1) == 1 and gate.dtype in (torch.float32, w[0].dtype))
+    nv.check(nv.lib().b2_branch_add(
+        nv.ptr(x), nv.ptr(None if r is not None else y), nv.ptr(rows), nv.ptr(None if r is None else r.place),
+        nv.ptr(None if r is None else r.weights), 0 if r is None else r.place.shape[1], 0 if r is None else rows.shape[0], nv.ptr(gate),
+        nv.ctypes.c_longlong(0 if gate is None else gate.stride(0)), int(gate is not None and gate.dtype == torch.float32),
+        nv.ptr(gate_bias), nv.ptr(w[0]), nv.ptr(w[1]), nv.ptr(scale), nv.ptr(nw), nv.ptr(nb), nv.ptr(h), x.shape[0], x.shape[1], n,
+        nv.ctypes.c_float(eps), _f32(w[0]), nv.stream_ptr()), "branch_add")
+    nv.count_launch()
+    return h
 
 
 def gelu_tanh(z: torch.Tensor) -> torch.Tensor:

@@ -8,7 +8,10 @@
 //   absorbed   q_h^T W_uk c = (W_uk^T q_h)^T c, so the query moves into the latent space, every head attends over the same rows,
 //              and W_uv is applied to the result: decoding and short portions (between two products per head, head_linear); in
 //              bf16 by the kernel of attention_decode.cu, in 32-bit and for sizes beyond it by latent_rows here
-// And the stage before either: norm of the latent, rotary positions of the queries' and the key's rotated part, page store.
+// And the stage before either: norm of the latent (and of the one queries are made from, where they have one), rotary positions of the
+// queries' and the key's rotated part, page store.  Queries made from a latent are turned later: by the product that moves them into
+// the latent space, or in place for the expanded way (latent_turn).  A window limits how far back a query sees; a gate per head
+// scales its output.
 #include "host.h"
 #include "mma_split.cuh"
 #include "vec.cuh"
@@ -30,22 +33,11 @@ __device__ __forceinline__ void la_wait() {
 }
 
 // ---- input stage -----------------------------------------------------------------------------------------------------------
-// One row per CTA.  q [M, H * dqp] is rotated in place: channels dim .. dim + rot - 1 of every head, pairs (2 i, 2 i + 1).
+// The rotated part of a row's queries: channels dim .. dim + rot - 1 of every head, pairs (2 i, 2 i + 1).
 constexpr int LS_THREADS = 128;
 template <typename T>
-__global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(T* __restrict__ q, const T* __restrict__ c, const T* __restrict__ kr,
-                                                                  long long ld, T* __restrict__ pages, const T* __restrict__ w,
-                                                                  const int* __restrict__ tables, const int* __restrict__ row_seq,
-                                                                  const int* __restrict__ pos, const int* __restrict__ slot,
-                                                                  const float* __restrict__ cs, const float* __restrict__ sn,
-                                                                  int max_blocks, int H, int dim, int dqp, int rank, int Cp, int Rp,
-                                                                  int rot, float eps) {
-  __shared__ float red[LS_THREADS / 32];
-  const size_t row = blockIdx.x;
-  const int s = row_seq ? row_seq[row] : static_cast<int>(row), tid = threadIdx.x, half = rot / 2;
-  const float* cr = cs + row * half;
-  const float* sr = sn + row * half;
-  T* qr = q + row * ld;
+__device__ __forceinline__ void turn_heads(T* qr, const float* cr, const float* sr, int H, int dim, int dqp, int rot) {
+  const int tid = threadIdx.x, half = rot / 2;
   if (dim % 8 == 0 && rot % 8 == 0) {        // four pairs at a time
     const int per = rot / 8;
     for (int i = tid; i < H * per; i += LS_THREADS) {
@@ -72,39 +64,83 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(T* __restrict_
       at[1] = from_f<T>(v * co + u * si);
     }
   }
-  if (slot != nullptr && slot[s] < 0) return;
-  const int p = pos[row];
-  T* dst = pages + (static_cast<size_t>(tables[static_cast<size_t>(s) * max_blocks + p / LA_PAGE]) * LA_PAGE + p % LA_PAGE) * Rp;
-  const T* crow = c + row * ld;
-  float ss = 0.f;
-  for (int a = tid * 8; a < Cp; a += LS_THREADS * 8) {
-    float t[8];
-    vload8(crow + a, t);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(LS_THREADS) latent_turn_kernel(T* __restrict__ q, long long ld, const float* __restrict__ cs,
+                                                                 const float* __restrict__ sn, int H, int dim, int dqp, int rot) {
+  const size_t row = blockIdx.x;
+  turn_heads(q + row * ld, cs + row * (rot / 2), sn + row * (rot / 2), H, dim, dqp, rot);
+}
+
+struct LatentStoreParams {
+  void* q;               // T [M, ld] H * dqp columns, turned in place, or null
+  void* cq;              // T [M, ld] Qp columns, normed in place (weight wq, q_rank real channels), or null
+  const void* c;         // T [M, ld] Cp columns
+  const void* kr;        // T [M, ld] Rp - Cp columns
+  void* pages;
+  const void *w, *wq;
+  const int *tables, *row_seq, *pos, *slot;
+  const float *cs, *sn;
+  long long ld;
+  int max_blocks, H, dim, dqp, rank, Cp, Rp, rot, q_rank, Qp;
+  float eps;
+};
+
+// One row per CTA.
+template <typename T>
+__global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentStoreParams p) {
+  __shared__ float red[2][LS_THREADS / 32];
+  const size_t row = blockIdx.x;
+  const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row), tid = threadIdx.x, half = p.rot / 2;
+  const float* cr = p.cs + row * half;
+  const float* sr = p.sn + row * half;
+  if (p.q) turn_heads(static_cast<T*>(p.q) + row * p.ld, cr, sr, p.H, p.dim, p.dqp, p.rot);
+  const T* crow = static_cast<const T*>(p.c) + row * p.ld;
+  T* qrow = static_cast<T*>(p.cq) + row * p.ld;
+  auto sum_squares = [&](const T* v, int n) {
+    float ss = 0.f;
+    for (int a = tid * 8; a < n; a += LS_THREADS * 8) {
+      float t[8];
+      vload8(v + a, t);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
+      for (int e = 0; e < 8; ++e) ss = fmaf(t[e], t[e], ss);
+    }
+    return warp_sum(ss);
+  };
+  auto scaled = [&](const T* v, const T* w, T* dst, int n, float r) {
+    for (int a = tid * 8; a < n; a += LS_THREADS * 8) {
+      float t[8], g[8];
+      vload8(v + a, t);
+      vload8(w + a, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) t[e] *= r * g[e];
+      vstore8(dst + a, t);
+    }
+  };
+  const float ss = sum_squares(crow, p.Cp), sq = p.cq ? sum_squares(qrow, p.Qp) : 0.f;
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = ss;
+    red[1][tid >> 5] = sq;
   }
-  ss = warp_sum(ss);
-  if ((tid & 31) == 0) red[tid >> 5] = ss;
   __syncthreads();
-  const float r = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / rank + eps);
-  for (int a = tid * 8; a < Cp; a += LS_THREADS * 8) {
-    float t[8], g[8];
-    vload8(crow + a, t);
-    vload8(w + a, g);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) t[e] *= r * g[e];
-    vstore8(dst + a, t);
-  }
-  const T* krow = kr + row * ld;
-  for (int f = LS_THREADS - 1 - tid; f < (Rp - Cp) / 2; f += LS_THREADS) {
+  if (p.cq)
+    scaled(qrow, static_cast<const T*>(p.wq), qrow, p.Qp, 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / p.q_rank + p.eps));
+  if (p.slot != nullptr && p.slot[s] < 0) return;
+  const int pos = p.pos[row];
+  T* dst = static_cast<T*>(p.pages) + (static_cast<size_t>(p.tables[static_cast<size_t>(s) * p.max_blocks + pos / LA_PAGE]) * LA_PAGE +
+                                       pos % LA_PAGE) * p.Rp;
+  scaled(crow, static_cast<const T*>(p.w), dst, p.Cp, 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / p.rank + p.eps));
+  const T* krow = static_cast<const T*>(p.kr) + row * p.ld;
+  for (int f = LS_THREADS - 1 - tid; f < (p.Rp - p.Cp) / 2; f += LS_THREADS) {
     float u = to_f(krow[2 * f]), v = to_f(krow[2 * f + 1]);
     if (f < half) {
       const float x = u * cr[f] - v * sr[f];
       v = v * cr[f] + u * sr[f];
       u = x;
     }
-    dst[Cp + 2 * f] = from_f<T>(u);
-    dst[Cp + 2 * f + 1] = from_f<T>(v);
+    dst[p.Cp + 2 * f] = from_f<T>(u);
+    dst[p.Cp + 2 * f + 1] = from_f<T>(v);
   }
 }
 
@@ -118,13 +154,19 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const uint8_t* __res
 }
 
 // ---- one small product per head ----------------------------------------------------------------------------------------------
-// out[m, h, :] = W_h x[m, h, :] with W_h [N, K] (KN: W_h stored [K, N]); x rows of stride ld_x with heads xs apart, out likewise.
+// out[m, h, :] = W_h x[m, h, :] with W_h [N, K] (KN: W_h stored [K, N]); x rows of stride ld_x with heads xs apart, out likewise.  On
+// the 32-bit result: columns turn_at .. turn_at + 2 half - 1 turned in pairs by the row's angles (cs given), the head's columns
+// times sigmoid(gate[m, h]) (gate given).
 struct HeadLinearParams {
   const void* x;
   const void* w;
   void* out;
   long long ld_x, ld_out;
   int M, H, N, K, xs, os;
+  const float *cs, *sn;  // [M, half]
+  const void* gate;      // type of x, [M, ld_gate]
+  long long ld_gate;
+  int turn_at, half;
 };
 
 template <bool KN>
@@ -134,8 +176,18 @@ __global__ void __launch_bounds__(256) head_linear_any_kernel(const HeadLinearPa
   if (n >= p.N) return;
   for (int m = blockIdx.z; m < p.M; m += gridDim.z) {
     const float* x = static_cast<const float*>(p.x) + m * p.ld_x + static_cast<size_t>(h) * p.xs;
-    float s = 0.f;
-    for (int k = 0; k < p.K; ++k) s = fmaf(x[k], KN ? w[static_cast<size_t>(k) * p.N + n] : w[static_cast<size_t>(n) * p.K + k], s);
+    auto dot = [&](int col) {
+      float s = 0.f;
+      for (int k = 0; k < p.K; ++k) s = fmaf(x[k], KN ? w[static_cast<size_t>(k) * p.N + col] : w[static_cast<size_t>(col) * p.K + k], s);
+      return s;
+    };
+    float s = dot(n);
+    const int f = n - p.turn_at;
+    if (p.cs != nullptr && f >= 0 && f < 2 * p.half) {
+      const float other = dot(p.turn_at + (f ^ 1)), co = p.cs[static_cast<size_t>(m) * p.half + f / 2], si = p.sn[static_cast<size_t>(m) * p.half + f / 2];
+      s = f & 1 ? s * co + other * si : s * co - other * si;
+    }
+    if (p.gate != nullptr) s *= sigmoid_f(static_cast<const float*>(p.gate)[m * p.ld_gate + h]);
     static_cast<float*>(p.out)[m * p.ld_out + static_cast<size_t>(h) * p.os + n] = s;
   }
 }
@@ -188,14 +240,25 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearParams
   }
   O* out = static_cast<O*>(p.out) + static_cast<size_t>(h) * p.os;
 #pragma unroll
-  for (int n = 0; n < HL_T / 8; ++n)
+  for (int hh = 0; hh < 2; ++hh) {
+    const int m = m0 + warp * 16 + (lane >> 2) + 8 * hh;
+    if (m >= p.M) continue;
+    const float g = p.gate ? sigmoid_fast(to_f(static_cast<const la_bf16*>(p.gate)[m * p.ld_gate + h])) : 1.f;
 #pragma unroll
-    for (int hh = 0; hh < 2; ++hh) {
-      const int m = m0 + warp * 16 + (lane >> 2) + 8 * hh, c = n0 + n * 8 + (lane & 3) * 2;
-      if (m >= p.M || c >= p.N) continue;
-      if (sizeof(O) == 4) *reinterpret_cast<float2*>(out + m * p.ld_out + c) = make_float2(acc[n][2 * hh], acc[n][2 * hh + 1]);
-      else *reinterpret_cast<uint32_t*>(out + m * p.ld_out + c) = pack_bf16x2(acc[n][2 * hh], acc[n][2 * hh + 1]);
+    for (int n = 0; n < HL_T / 8; ++n) {
+      const int c = n0 + n * 8 + (lane & 3) * 2;
+      if (c >= p.N) continue;
+      float u = acc[n][2 * hh] * g, v = acc[n][2 * hh + 1] * g;
+      const int f = (c - p.turn_at) / 2;
+      if (p.cs != nullptr && c >= p.turn_at && f < p.half) {
+        const float co = p.cs[static_cast<size_t>(m) * p.half + f], si = p.sn[static_cast<size_t>(m) * p.half + f], t = u * co - v * si;
+        v = v * co + u * si;
+        u = t;
+      }
+      if (sizeof(O) == 4) *reinterpret_cast<float2*>(out + m * p.ld_out + c) = make_float2(u, v);
+      else *reinterpret_cast<uint32_t*>(out + m * p.ld_out + c) = pack_bf16x2(u, v);
     }
+  }
 }
 
 // ---- absorbed attention ------------------------------------------------------------------------------------------------------
@@ -211,6 +274,7 @@ struct LatentRowsParams {
   float* part_o;         // [M, H, nsplit, Cp]
   float* part_ml;        // [M, H, nsplit, 2]
   int max_blocks, H, Rp, Cp, partition, nsplit;
+  int window;            // > 0: keys pos - window + 1 .. pos; partitions count from the first visible key
   float scale;
 };
 
@@ -233,7 +297,8 @@ __global__ void __launch_bounds__(LR_ANY_WARPS * 32) latent_rows_any_kernel(cons
   const int head = blockIdx.y, split = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int s = p.row_seq ? p.row_seq[row] : static_cast<int>(row);
   const bool live = p.slot == nullptr || p.slot[s] >= 0;
-  const int t_begin = split * p.partition, t_end = live ? min(p.pos[row] + 1, t_begin + p.partition) : t_begin;
+  const int seen = p.window > 0 ? max(0, p.pos[row] - p.window + 1) : 0;
+  const int t_begin = seen + split * p.partition, t_end = live ? min(p.pos[row] + 1, t_begin + p.partition) : t_begin;
   const int* table = p.tables + static_cast<size_t>(s) * p.max_blocks;
   const T* q = static_cast<const T*>(p.q) + (row * p.H + head) * p.Rp;
   float* sQ = la_any;
@@ -316,21 +381,38 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentRowsParam
 
 using namespace b2;
 
-B2_EXPORT int b2_latent_store(void* q, const void* c, const void* kr, long long ld, void* pages, const void* w, const int* tables,
-                              const int* row_seq, const int* pos, const int* slot, const float* cs, const float* sn, int M,
-                              int max_blocks, int H, int dim, int dqp, int rank, int Cp, int Rp, int rot, float eps, int is_f32,
-                              void* stream) {
+// q null: the queries are made later, from cq (Qp columns of which q_rank are real), which is normed here
+B2_EXPORT int b2_latent_store(void* q, void* cq, const void* c, const void* kr, long long ld, void* pages, const void* w, const void* wq,
+                              const int* tables, const int* row_seq, const int* pos, const int* slot, const float* cs, const float* sn,
+                              int M, int max_blocks, int H, int dim, int dqp, int rank, int Cp, int Rp, int rot, int q_rank, int Qp,
+                              float eps, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
-  if (H < 1 || dim < 1 || rot < 2 || rot % 2 || dim + rot > dqp || dqp % 8 || Cp % 8 || Rp % 8 || rank < 1 || rank > Cp ||
-      Rp - Cp < rot || ld % 8 || max_blocks < 1) {
+  if (rot < 2 || rot % 2 || Cp % 8 || Rp % 8 || rank < 1 || rank > Cp || Rp - Cp < rot || ld % 8 || max_blocks < 1 ||
+      (q != nullptr && (H < 1 || dim < 1 || dim + rot > dqp || dqp % 8)) ||
+      (cq != nullptr && (wq == nullptr || q_rank < 1 || q_rank > Qp || Qp % 8))) {
     set_error("latent_store: padded sizes in multiples of 8 and an even rotated size required");
     return 10;
   }
-  B2_DISPATCH_T(is_f32, latent_store_kernel<T><<<M, LS_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<T*>(q), static_cast<const T*>(c), static_cast<const T*>(kr), ld, static_cast<T*>(pages), static_cast<const T*>(w),
-      tables, row_seq, pos, slot, cs, sn, max_blocks, H, dim, dqp, rank, Cp, Rp, rot, eps););
+  const LatentStoreParams p = {q, cq, c, kr, pages, w, wq, tables, row_seq, pos, slot, cs, sn, ld, max_blocks, H, dim, dqp, rank, Cp, Rp, rot,
+                               q_rank, Qp, eps};
+  B2_DISPATCH_T(is_f32, latent_store_kernel<T><<<M, LS_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(p););
   B2_CHECK_LAUNCH("latent_store");
+  return 0;
+}
+
+// q [M, ld]: the rotated part of every head, in place
+B2_EXPORT int b2_latent_turn(void* q, long long ld, const float* cs, const float* sn, int M, int H, int dim, int dqp, int rot, int is_f32,
+                             void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (H < 1 || dim < 1 || rot < 2 || rot % 2 || dim + rot > dqp || dqp % 8 || ld % 8) {
+    set_error("latent_turn: padded sizes in multiples of 8 and an even rotated size required");
+    return 10;
+  }
+  B2_DISPATCH_T(is_f32, latent_turn_kernel<T><<<M, LS_THREADS, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<T*>(q), ld, cs, sn, H, dim,
+                                                                                                      dqp, rot););
+  B2_CHECK_LAUNCH("latent_turn");
   return 0;
 }
 
@@ -345,16 +427,21 @@ B2_EXPORT int b2_latent_gather(const void* pages, const int* ids, void* out, int
   return 0;
 }
 
-// out_f32: a 32-bit result of bf16 operands
+// out_f32: a 32-bit result of bf16 operands; cs, sn, gate: see HeadLinearParams
 B2_EXPORT int b2_head_linear(const void* x, const void* w, void* out, long long ld_x, long long ld_out, int M, int H, int N, int K,
-                             int xs, int os, int kn, int is_f32, int out_f32, void* stream) {
+                             int xs, int os, int kn, const float* cs, const float* sn, int turn_at, int half, const void* gate,
+                             long long ld_gate, int is_f32, int out_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (H < 1 || H > 65535 || N < 8 || K < 8 || N % 8 || K % 8 || xs % 8 || os % 8 || ld_x % 8 || ld_out % 8) {
     set_error("head_linear: sizes and strides in multiples of 8 required");
     return 10;
   }
-  HeadLinearParams p = {x, w, out, ld_x, ld_out, M, H, N, K, xs, os};
+  if (cs != nullptr && (sn == nullptr || half < 1 || turn_at < 0 || turn_at % 2 || turn_at + 2 * half > N)) {
+    set_error("head_linear: turned columns outside the result");
+    return 10;
+  }
+  HeadLinearParams p = {x, w, out, ld_x, ld_out, M, H, N, K, xs, os, cs, sn, gate, ld_gate, turn_at, half};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (is_f32) {
     const dim3 grid((N + 255) / 256, H, M < 65535 ? M : 65535);
@@ -375,10 +462,10 @@ B2_EXPORT int b2_head_linear(const void* x, const void* w, void* out, long long 
   return 0;
 }
 
-// partition: keys per split; nsplit * partition must cover every row's keys.
+// partition: keys per split; nsplit * partition must cover every row's visible keys.
 B2_EXPORT int b2_latent_rows(const void* q, const void* pages, const int* tables, const int* row_seq, const int* pos,
                              const int* slot, const void* sink, void* out, float* part_o, float* part_ml, int M, int max_blocks,
-                             int H, int Rp, int Cp, int partition, int nsplit, float scale, int is_f32, void* stream) {
+                             int H, int Rp, int Cp, int partition, int nsplit, int window, float scale, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   if (H < 1 || H > 65535 || Rp % 8 || Cp % 8 || Cp < 8 || Rp < Cp || Rp > 1280 || partition < 1 || nsplit < 1 || nsplit > 65535 ||
@@ -387,7 +474,7 @@ B2_EXPORT int b2_latent_rows(const void* q, const void* pages, const int* tables
     return 10;
   }
   LatentRowsParams p = {q, pages, tables, row_seq, pos, slot, sink, out, part_o, part_ml, max_blocks, H, Rp, Cp, partition, nsplit,
-                        scale};
+                        window, scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const dim3 grid(M, H, nsplit);
   B2_DISPATCH_T(is_f32, {

@@ -1,7 +1,8 @@
 // Mixture of experts.
 //
-//   moe_route / moe_place   sigmoid scores, the choice among the best groups, and the (token, choice) pairs laid out expert after expert
-//   moe_gemm (MOE_GLU)      silu(W_gate h) * (W_up h) over every expert's rows, h gathered by token
+//   moe_route / moe_place   sigmoid or softmax scores, the choice among the best groups, and the (token, choice) pairs laid out expert
+//                           after expert
+//   moe_gemm (MOE_GLU)      silu(W_gate h) * (W_up h), or its clamped form, over every expert's rows, h gathered by token
 //   moe_gemm (MOE_DOWN)     W_down of those rows
 //   moe_gemm (ROWS_GLU)     the first product over rows that are in order already
 //   moe_norm_add            the weighted sum of a token's rows, a gated shared expert, the norm of the sum, the residual
@@ -22,13 +23,15 @@ constexpr int MOE_MAX_TOP = 32;
 typedef __nv_bfloat16 moe_bf16;
 
 // ---- routing -----------------------------------------------------------------------------------------------------------
+enum : int { SCORE_SIGMOID = 0, SCORE_SOFTMAX = 1 };
 struct RouteParams {
-  const void* corr;      // T [E]
+  const void* corr;      // T [E] or null
   float* weights;        // [M, slots]
   int* id;               // [M, slots]
   int M, E, top, groups, keep;
   int slots;             // top, or one more: expert E, which every token takes behind a gate of its own
   float scale;
+  int score;             // SCORE_*; softmax over all experts
 };
 
 // largest value and, among equals, the lowest index
@@ -50,8 +53,17 @@ template <typename T>
 __device__ __forceinline__ void route_token(const RouteParams& p, int row, const float* z, const float* sg, float* c, float* gs) {
   const int lane = threadIdx.x & 31;
   constexpr float LOW = -3.0e38f;           // in place of what is no number (rows without a sequence): below any score, above "closed"
+  float most = -INFINITY, total = 0.f;
+  if (p.score == SCORE_SOFTMAX) {
+    for (int e = lane; e < p.E; e += 32) most = fmaxf(most, z[e]);
+    most = warp_max(most);
+    for (int e = lane; e < p.E; e += 32) total += expf(z[e] - most);
+    total = warp_sum(total);
+  }
+  auto score = [&](float v) { return p.score == SCORE_SOFTMAX ? expf(v - most) / total : sigmoid_f(v); };
+  const bool by_logit = p.corr == nullptr && p.keep == p.groups;      // the order of the scores is that of the logits
   for (int e = lane; e < p.E; e += 32) {
-    const float s = sigmoid_f(z[e]) + to_f(static_cast<const T*>(p.corr)[e]);
+    const float s = by_logit ? z[e] : score(z[e]) + (p.corr ? to_f(static_cast<const T*>(p.corr)[e]) : 0.f);
     c[e] = s >= LOW ? s : LOW;
   }
   __syncwarp();
@@ -107,7 +119,7 @@ __device__ __forceinline__ void route_token(const RouteParams& p, int row, const
   }
   const size_t first = static_cast<size_t>(row) * p.slots;
   auto choose = [&](int k, int e) {
-    p.weights[first + k] = sigmoid_f(z[e]) * p.scale;
+    p.weights[first + k] = score(z[e]) * p.scale;
     p.id[first + k] = e;
   };
   if (p.slots > p.top && lane == 31) {
@@ -366,12 +378,36 @@ __device__ __forceinline__ MoeTile moe_tile(int t, const int* off, const int* fi
   return r;
 }
 
+// What a gated product does with gate and up: silu(g) u, or with g = min(g, limit), u = clamp(u, -limit, limit): g sigmoid(alpha g) (u + 1)
+enum : int { GLU_SILU = 0, GLU_CLAMPED = 1 };
+struct GluAct {
+  int kind;
+  float alpha, limit;
+};
+__device__ __forceinline__ float clamped_glu(float g, float u, const GluAct& a) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return g * sigmoid_f(a.alpha * g) * (u + 1.f);
+}
+// two values with one reciprocal between them, for results that are rounded to bf16 next
+__device__ __forceinline__ void clamped_glu_pair_fast(float& g0, float& g1, float u0, float u1, const GluAct& a) {
+  g0 = fminf(g0, a.limit);
+  g1 = fminf(g1, a.limit);
+  u0 = fminf(fmaxf(u0, -a.limit), a.limit);
+  u1 = fminf(fmaxf(u1, -a.limit), a.limit);
+  const float k = -1.4426950408889634f * a.alpha;
+  const float d0 = 1.f + fast_exp2(fminf(k * g0, 62.f)), d1 = 1.f + fast_exp2(fminf(k * g1, 62.f));
+  const float r = __fdividef(1.f, d0 * d1);
+  g0 *= r * d1 * (u0 + 1.f);
+  g1 *= r * d0 * (u1 + 1.f);
+}
+
 // 32-bit form: 64 x 64 tiles of plain FMAs.  Grid (column tiles, an upper bound of the row tiles).
 constexpr int MF_T = 64, MF_K = 16;
 template <bool GLU>
 __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restrict__ W,
                                                            const int* __restrict__ token, const int* __restrict__ offsets,
-                                                           float* __restrict__ out, int E, int N, int K) {
+                                                           float* __restrict__ out, int E, int N, int K, const GluAct act) {
   __shared__ int off[MOE_MAX_EXPERTS + 1], first[MOE_MAX_EXPERTS + 1];
   __shared__ __align__(16) float sA[MF_K][MF_T + 4], sB[GLU ? 2 : 1][MF_K][MF_T + 4];   // read in vectors of four
   for (int e = threadIdx.x; e <= E; e += 256) off[e] = offsets[e];
@@ -417,7 +453,9 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) out[static_cast<size_t>(tl.row0 + m) * N + n] = GLU ? silu_f(acc[0][i][j]) * acc[GLU ? 1 : 0][i][j] : acc[0][i][j];
+      if (n >= N) continue;
+      const float g = acc[0][i][j], u = acc[GLU ? 1 : 0][i][j];
+      out[static_cast<size_t>(tl.row0 + m) * N + n] = !GLU ? g : act.kind == GLU_CLAMPED ? clamped_glu(g, u, act) : silu_f(g) * u;
     }
   }
 }
@@ -441,6 +479,7 @@ struct MoeGemmParams {
   moe_bf16* out;           // [P, ld_out]
   long long ld_out;
   int P, E, N, K;          // GLU: N activation columns (half of a tile's accumulator columns each for gate and up)
+  GluAct act;
 };
 
 template <int BN, int FORM>
@@ -588,9 +627,15 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
               float x = __uint_as_float(r[i]), y = __uint_as_float(r[i + 1]);
-              silu_pair_fast(x, y);
-              r[i] = __float_as_uint(x * __uint_as_float(u[i]));
-              r[i + 1] = __float_as_uint(y * __uint_as_float(u[i + 1]));
+              if (p.act.kind == GLU_CLAMPED) {
+                clamped_glu_pair_fast(x, y, __uint_as_float(u[i]), __uint_as_float(u[i + 1]), p.act);
+              } else {
+                silu_pair_fast(x, y);
+                x *= __uint_as_float(u[i]);
+                y *= __uint_as_float(u[i + 1]);
+              }
+              r[i] = __float_as_uint(x);
+              r[i + 1] = __float_as_uint(y);
             }
           } else {
             tmem_ld_wait();
@@ -816,10 +861,11 @@ static int launch_place(int* place, int* token, int* offsets, int* work, int M, 
 }
 
 // z: fp32 [M, ld]; work: int32 [E + M * top]; offsets: int32 [E + 1]; place: int32 [M, top]; token: int32 [M * top].  joint: every token
-// also takes expert E, with the weight sigmoid(sg) (fp32 [M], stride ld_sg); then one more expert and choice in all of these.
+// also takes expert E, with the weight sigmoid(sg) (fp32 [M], stride ld_sg); then one more expert and choice in all of these.  softmax:
+// scores are a softmax over all experts instead of a sigmoid each; corr may be null.
 B2_EXPORT int b2_moe_route(const float* z, long long ld, const float* sg, long long ld_sg, int joint, const void* corr, float* weights,
                            int* place, int* token, int* offsets, int* work, int M, int E, int top, int groups, int keep, float scale,
-                           int is_f32, void* stream) {
+                           int softmax, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   const int slots = top + (joint ? 1 : 0), all = E + (joint ? 1 : 0);
@@ -827,7 +873,7 @@ B2_EXPORT int b2_moe_route(const float* z, long long ld, const float* sg, long l
   if (joint && sg == nullptr) { set_error("moe_route: the joint expert needs its gate"); return 10; }
   if (ld < E) { set_error("moe_route: a logit per expert required"); return 10; }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const RouteParams p = {corr, weights, work + all, M, E, top, groups, keep, slots, scale};
+  const RouteParams p = {corr, weights, work + all, M, E, top, groups, keep, slots, scale, softmax ? SCORE_SOFTMAX : SCORE_SIGMOID};
   B2_DISPATCH_T(is_f32, moe_route_kernel<T><<<(M + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, MR_WARPS * 2 * E * sizeof(float), st>>>(
       p, z, ld, sg, ld_sg););
   B2_CHECK_LAUNCH("moe_route");
@@ -881,7 +927,7 @@ B2_EXPORT int b2_token_gate(const void* h, long long ld_h, const void* w, long l
 // the gate of the joint expert, or goes to sg_out fp32 [M].  The rest as b2_moe_route.
 B2_EXPORT int b2_moe_router(const void* h, long long ld_h, const void* w, long long ld_w, int N, int K, int sg, float* sg_out,
                             int joint, const void* corr, float* weights, int* place, int* token, int* offsets, int* work, int M, int E, int top,
-                            int groups, int keep, float scale, void* stream) {
+                            int groups, int keep, float scale, int softmax, void* stream) {
   b2::ensure_thread_context();
   if (M <= 0) return 0;
   const int slots = top + (joint ? 1 : 0), all = E + (joint ? 1 : 0);
@@ -893,33 +939,35 @@ B2_EXPORT int b2_moe_router(const void* h, long long ld_h, const void* w, long l
   }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const SkinnyParams p = {static_cast<const moe_bf16*>(h), static_cast<const moe_bf16*>(w), sg_out, ld_h, ld_w, 1, M, N, K, sg, nullptr, nullptr, nullptr, 0, 0, 0};
-  const RouteParams r = {corr, weights, work + all, M, E, top, groups, keep, slots, scale};
+  const RouteParams r = {corr, weights, work + all, M, E, top, groups, keep, slots, scale, softmax ? SCORE_SOFTMAX : SCORE_SIGMOID};
   if (const int rc = launch_skinny<SK_ROUTE>(p, r, st)) return rc;
   return launch_place(place, token, offsets, work, M, all, slots, st);
 }
 
 // h: T [tokens, ld], w: T [E, 2, F, K], token: int32 [P] -> out T [P, F].  rows (bf16 [P, K], or null): room for the rows expert after
-// expert, if they are to be laid out before the product.
+// expert, if they are to be laid out before the product.  clamped: the gated form with alpha and limit instead of silu.
 B2_EXPORT int b2_moe_glu(const void* h, long long ld, const void* w, const int* token, const int* offsets, void* rows, void* out, int tokens,
-                         int P, int E, int F, int K, int is_f32, void* stream) {
+                         int P, int E, int F, int K, int clamped, float alpha, float limit, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (P <= 0) return 0;
   if (E < 1 || E > MOE_MAX_EXPERTS || F < 8 || F % 8 || K < 8 || K % 8 || ld % 8 || ld < K || tokens < 1) {
     set_error("moe_glu: up to %d experts and sizes in multiples of 8 required", MOE_MAX_EXPERTS);
     return 10;
   }
+  if (clamped && !(limit > 0.f)) { set_error("moe_glu: a positive limit required"); return 10; }
+  const GluAct act = {clamped ? GLU_CLAMPED : GLU_SILU, alpha, limit};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (is_f32) {
     const int rows = moe_bound(P, E, MF_T);
     if (rows > 65535) { set_error("moe_glu: too many rows (%d)", P); return 10; }
     moe_gemm_f32_kernel<true><<<dim3((F + MF_T - 1) / MF_T, rows), 256, 0, st>>>(
-        static_cast<const float*>(h), ld, static_cast<const float*>(w), token, offsets, static_cast<float*>(out), E, F, K);
+        static_cast<const float*>(h), ld, static_cast<const float*>(w), token, offsets, static_cast<float*>(out), E, F, K, act);
     B2_CHECK_LAUNCH("moe_glu");
     return 0;
   }
   const uint64_t hd[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(tokens)}, hs[1] = {2ull * ld};
   const uint32_t hbox[2] = {MG_BK, 1};
-  const MoeGemmParams p = {token, offsets, static_cast<moe_bf16*>(out), F, P, E, F, K};
+  const MoeGemmParams p = {token, offsets, static_cast<moe_bf16*>(out), F, P, E, F, K, act};
   if (rows != nullptr) {
     const int blocks = (P + 7) / 8;
     moe_gather_kernel<<<blocks < 16 * num_sms() ? blocks : 16 * num_sms(), 256, 0, st>>>(static_cast<const moe_bf16*>(h), ld, token,
@@ -939,7 +987,7 @@ B2_EXPORT int b2_rows_glu(const void* h, long long ld, const void* w, void* out,
     set_error("rows_glu: sizes and strides in multiples of 8 required");
     return 10;
   }
-  const MoeGemmParams p = {nullptr, nullptr, static_cast<moe_bf16*>(out), ld_out, M, 1, F, K};
+  const MoeGemmParams p = {nullptr, nullptr, static_cast<moe_bf16*>(out), ld_out, M, 1, F, K, {GLU_SILU, 0.f, 0.f}};
   return launch_glu<ROWS_GLU>(tensor_map_2d_bf16(h, M, K, ld, MG_BM, MG_BK), w, p, moe_columns(M, 1, F, 128, 32), (M + MG_BM - 1) / MG_BM,
                               static_cast<cudaStream_t>(stream));
 }
@@ -958,7 +1006,7 @@ B2_EXPORT int b2_moe_down(const void* a, const void* w, const int* offsets, void
     const int rows = moe_bound(P, E, MF_T);
     if (rows > 65535) { set_error("moe_down: too many rows (%d)", P); return 10; }
     moe_gemm_f32_kernel<false><<<dim3((N + MF_T - 1) / MF_T, rows), 256, 0, st>>>(
-        static_cast<const float*>(a), F, static_cast<const float*>(w), nullptr, offsets, static_cast<float*>(out), E, N, F);
+        static_cast<const float*>(a), F, static_cast<const float*>(w), nullptr, offsets, static_cast<float*>(out), E, N, F, GluAct{});
     B2_CHECK_LAUNCH("moe_down");
     return 0;
   }
@@ -968,7 +1016,7 @@ B2_EXPORT int b2_moe_down(const void* a, const void* w, const int* offsets, void
   const uint32_t box[3] = {MG_BK, static_cast<uint32_t>(cols), 1};
   const CUtensorMap *tb = tensor_map_nd_bf16(w, 3, dims, strides, box, 3), *ta = tensor_map_2d_bf16(a, P, F, F, MG_BM, MG_BK);
   if (!ta || !tb) return 2;
-  const MoeGemmParams p = {nullptr, offsets, static_cast<moe_bf16*>(out), N, P, E, N, F};
+  const MoeGemmParams p = {nullptr, offsets, static_cast<moe_bf16*>(out), N, P, E, N, F, GluAct{}};
   const int bound = moe_bound(P, E, MG_BM);
   if (cols == 256) return launch_moe<256, MOE_DOWN>(ta, tb, p, bound, st);
   if (cols == 128) return launch_moe<128, MOE_DOWN>(ta, tb, p, bound, st);

@@ -23,9 +23,9 @@ constexpr float GR_RATE = 8.f;
 struct ConvParams {
   const void* x;         // T [M, ld]
   long long ld;
-  const void* xb;        // T [C]
+  const void* xb;        // T [C] or null
   const void* taps;      // T [C, K], last column: the current token
-  const void* cb;        // T [C]
+  const void* cb;        // T [C] or null
   float* state;          // [slots, C, K - 1] inputs, bias included
   void* u;               // T [M, C]
   const int* cu;
@@ -33,6 +33,7 @@ struct ConvParams {
   const int* slot;
   const int* tiles;      // [n, 4] = (sequence, first row, rows, offset in the portion)
   int C, K;
+  int add;               // 1: the input itself is added to the result
 };
 
 // Grid (tiles, channels / 256): 32 groups of eight channels times four groups of four rows.  Only the portion's first tile reads the
@@ -50,9 +51,9 @@ __global__ void __launch_bounds__(GR_THREADS, sizeof(T) == 2 ? 5 : 4) causal_con
   const T* x = static_cast<const T*>(p.x) + cc;
   const T* taps = static_cast<const T*>(p.taps) + static_cast<size_t>(cc) * K;
   float* st = p.state + (static_cast<size_t>(slot) * p.C + cc) * (K - 1);
-  float xb[8], cb[8];
-  vload8(static_cast<const T*>(p.xb) + cc, xb);
-  vload8(static_cast<const T*>(p.cb) + cc, cb);
+  float xb[8] = {}, cb[8] = {};
+  if (p.xb) vload8(static_cast<const T*>(p.xb) + cc, xb);
+  if (p.cb) vload8(static_cast<const T*>(p.cb) + cc, cb);
   // Only the first rows of the first tile look back into the state.
   constexpr int KK = KT > 0 ? KT : 1, OLD = KT > 1 ? KT - 1 : 1;
   const bool head = off == 0 && t0 == 0;
@@ -78,9 +79,13 @@ __global__ void __launch_bounds__(GR_THREADS, sizeof(T) == 2 ? 5 : 4) causal_con
       }
     }
   };
+  if constexpr (KT > 0) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w[e * KT + KT - 1] += p.add ? 1.f : 0.f;
+  }
   auto tap = [&](int e, int j) {                     // of channel e, j tokens back
     if constexpr (KT > 0) return w[e * KT + KT - 1 - j];
-    else return to_f(taps[e * K + K - 1 - j]);
+    else return to_f(taps[e * K + K - 1 - j]) + (j == 0 && p.add ? 1.f : 0.f);
   };
   auto input = [&](int at, float (&f)[8], const float (&old)[OLD * 8]) {          // input at index `at` of the portion
     if (at >= 0) {
@@ -540,14 +545,14 @@ using namespace b2;
 
 B2_EXPORT int b2_causal_conv(const void* x, long long ld, const void* xb, const void* taps, const void* cb, float* state, void* u,
                              const int* cu, const int* start, const int* slot, const int* tiles, int ntiles, int C, int K,
-                             int is_f32, void* stream) {
+                             int add, int is_f32, void* stream) {
   b2::ensure_thread_context();
   if (ntiles <= 0) return 0;
   if (C < 8 || C % 8 || ld % 8 || K < 1 || K - 1 > GR_TILE) {
     set_error("causal_conv: channels in multiples of 8 and 1 to %d taps required", GR_TILE + 1);
     return 10;
   }
-  const ConvParams p = {x, ld, xb, taps, cb, state, u, cu, start, slot, tiles, C, K};
+  const ConvParams p = {x, ld, xb, taps, cb, state, u, cu, start, slot, tiles, C, K, add};
   const dim3 grid(ntiles, (C / 8 + 31) / 32);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (K == 4) {

@@ -1,7 +1,8 @@
-// Kernels around a 32-bit residual stream: embedding into it, RMS norm out of it, the half-sum of two normed branches
-// added to it (with the next norm in the same pass), one normed branch added to it, gated activations over column slices or with a
-// table of per-token vectors, rotary tables for a batch's positions, and the 32-bit matrix product used when a model runs without
-// any reduced-precision mode.
+// Kernels around a 32-bit residual stream: embedding into it (of the token alone, or of the token and of the pair it forms with the one
+// before, normed), RMS norm or layer norm out of it, the half-sum of two normed branches added to it (with the next norm in the same
+// pass), one normed branch added to it (plain, or gated, layer-normed and scaled per channel with the next layer norm in the same
+// pass), gated activations over column slices or with a table of per-token vectors, rotary tables for a batch's positions, and the
+// 32-bit matrix product used when a model runs without any reduced-precision mode.
 //
 // Rows of the residual and of every activation are padded to a multiple of eight columns; `n` is the real width.  The
 // padding columns are zero (their norm weights are zero), so vector accesses never need a tail.
@@ -220,6 +221,236 @@ __global__ void __launch_bounds__(MAXT) norm_add_kernel(float* __restrict__ x, c
     if (h) vstore8(h + base + c, b[k]);
   }
 }
+
+// ---- layer norms ---------------------------------------------------------------------------------------------------------------
+// A row lies in the registers of a block, V pieces of eight channels a thread, zero past its n channels.  The mean is taken off
+// before anything is squared.
+__device__ __forceinline__ float row_sum(float v, float* scratch) {      // scratch: 32 floats that nothing else uses
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int lane = threadIdx.x & 31;
+  return warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? scratch[lane] : 0.f);
+}
+__device__ __forceinline__ int row_piece(int k) { return (threadIdx.x + k * blockDim.x) * 8; }
+
+// a <- (a - mean) / sqrt(variance + eps)
+template <int V>
+__device__ __forceinline__ void row_standardise(float (&a)[V][8], int n, float eps, float (*scratch)[32]) {
+  float s = 0.f;
+#pragma unroll
+  for (int k = 0; k < V; ++k)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s += a[k][e];
+  const float mean = row_sum(s, scratch[0]) / n;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < V; ++k)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      a[k][e] = row_piece(k) + e < n ? a[k][e] - mean : 0.f;
+      ss = fmaf(a[k][e], a[k][e], ss);
+    }
+  const float r = 1.f / sqrtf(row_sum(ss, scratch[1]) / n + eps);
+#pragma unroll
+  for (int k = 0; k < V; ++k)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] *= r;
+}
+
+// a <- a * w + b, the weights' padding being zero
+template <typename T, int V>
+__device__ __forceinline__ void row_affine(float (&a)[V][8], const T* w, const T* b, int ld) {
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = row_piece(k);
+    if (c >= ld) break;
+    float wv[8], bv[8];
+    vload8(w + c, wv);
+    vload8(b + c, bv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] = fmaf(a[k][e], wv[e], bv[e]);
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void row_store(const float (&a)[V][8], T* dst, int ld) {
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = row_piece(k);
+    if (c >= ld) break;
+    vstore8(dst + c, a[k]);
+  }
+}
+
+// h = layer norm of x[rows]
+template <typename T, int V, int MAXT>
+__global__ void __launch_bounds__(MAXT) layernorm_f32_kernel(const float* __restrict__ x, const T* __restrict__ w, const T* __restrict__ b,
+                                                             T* __restrict__ h, const long long* __restrict__ rows, int ld, int n,
+                                                             float eps) {
+  __shared__ float scratch[2][32];
+  const float* xr = x + (rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x) * ld;
+  float a[V][8];
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] = 0.f;
+    if (row_piece(k) < ld) vload8(xr + row_piece(k), a[k]);
+  }
+  row_standardise(a, n, eps, scratch);
+  row_affine(a, w, b, ld);
+  row_store(a, h + static_cast<size_t>(blockIdx.x) * ld, ld);
+}
+
+// x = layer norm of table[id] + pairs[(before * mul_prev + id * mul_cur) mod buckets], `before` the sequence's token before this one; the
+// first token of a sequence takes row `buckets` of pairs.  h = layer norm of x with the reader's weights.  Between steps the last
+// token of a sequence waits in its slot: the block of the portion's first row reads it and puts the portion's last token there.
+struct EmbedPairsParams {
+  const long long* ids;
+  const void *table, *pairs;
+  int* last;             // [slots]
+  const int *cu, *row_seq, *pos, *slot;
+  const void *w, *b, *next_w, *next_b;
+  float* x;
+  void* h;
+  long long mul_prev, mul_cur, buckets;
+  int ld, n, vocab;
+  float eps;
+};
+template <typename T, int V, int MAXT>
+__global__ void __launch_bounds__(MAXT) embed_pairs_kernel(const EmbedPairsParams p) {
+  __shared__ float scratch[4][32];
+  const int row = blockIdx.x, s = p.row_seq[row], first = p.cu[s], slot = p.slot[s];
+  const long long id = p.ids[row];
+  const bool ok = id >= 0 && id < p.vocab;      // padding rows of a graph batch carry any id; nothing outside the tables is read
+  long long pair = p.buckets;
+  if (p.pos[row] > 0) {
+    const long long before = row > first ? p.ids[row - 1] : slot >= 0 ? p.last[slot] : 0;
+    pair = (before * p.mul_prev + id * p.mul_cur) % p.buckets;
+    if (pair < 0) pair += p.buckets;
+  }
+  const T* tr = static_cast<const T*>(p.table) + static_cast<size_t>(ok ? id : 0) * p.ld;
+  const T* pr = static_cast<const T*>(p.pairs) + static_cast<size_t>(pair) * p.ld;
+  float a[V][8];
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = row_piece(k);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] = 0.f;
+    if (c >= p.ld || !ok) continue;
+    float t[8];
+    vload8(tr + c, a[k]);
+    vload8(pr + c, t);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] += t[e];
+  }
+  row_standardise(a, p.n, p.eps, scratch);      // its barriers: every thread has read `last`
+  if (row == first && slot >= 0 && threadIdx.x == 0) p.last[slot] = static_cast<int>(p.ids[p.cu[s + 1] - 1]);
+  row_affine(a, static_cast<const T*>(p.w), static_cast<const T*>(p.b), p.ld);
+  row_store(a, p.x + static_cast<size_t>(row) * p.ld, p.ld);
+  if (p.h == nullptr) return;
+  row_standardise(a, p.n, p.eps, scratch + 2);
+  row_affine(a, static_cast<const T*>(p.next_w), static_cast<const T*>(p.next_b), p.ld);
+  row_store(a, static_cast<T*>(p.h) + static_cast<size_t>(row) * p.ld, p.ld);
+}
+
+// x += s * layer norm(y * sigmoid(gate + gate_b)), h = layer norm of the new x with the reader's weights.  y: fp32 rows, or (ROWS) the
+// weighted sum of a token's expert rows.  Gate and s are optional.
+constexpr int BA_MAX_TOP = 32;
+struct BranchParams {
+  float* x;              // [M, ld]
+  const float* y;        // [M, ld]
+  const void* rows;      // ROWS: T [P, ld]
+  const int* place;      // [M, top]
+  const float* weights;  // [M, top]
+  const void* gate;      // G [M, ld_gate] or null
+  const void *gate_b, *w, *b, *s, *next_w, *next_b;     // T [ld]; gate_b with gate, s or null, next_* with h
+  void* h;               // T [M, ld] or null
+  long long ld_gate;
+  int top, P, ld, n;
+  float eps;
+  int* status;
+};
+template <typename T, typename G, int V, int MAXT, bool ROWS>
+__global__ void __launch_bounds__(MAXT) branch_add_kernel(const BranchParams p) {
+  __shared__ float scratch[4][32], sw[BA_MAX_TOP];
+  __shared__ int sr[BA_MAX_TOP];
+  const size_t base = static_cast<size_t>(blockIdx.x) * p.ld;
+  if (ROWS) {
+    if (static_cast<int>(threadIdx.x) < p.top) {
+      sw[threadIdx.x] = p.weights[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
+      int r = p.place[static_cast<size_t>(blockIdx.x) * p.top + threadIdx.x];
+      if (r < 0 || r >= p.P) {                  // an index that came from memory: recorded, and the access left out
+        atomicCAS(p.status, 0, ERR_BAD_ARGUMENT);
+        r = 0;
+      }
+      sr[threadIdx.x] = r;
+    }
+    __syncthreads();
+  }
+  const T* rows = static_cast<const T*>(p.rows);
+  float a[V][8], x[V][8];
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = row_piece(k);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[k][e] = x[k][e] = 0.f;
+    if (c >= p.ld) continue;
+    vload8(p.x + base + c, x[k]);
+    float g[8] = {}, gb[8] = {};
+    if (p.gate) {
+      vload8(static_cast<const G*>(p.gate) + blockIdx.x * p.ld_gate + c, g);
+      vload8(static_cast<const T*>(p.gate_b) + c, gb);
+    }
+    if (ROWS) {
+      for (int j = 0; j < p.top; j += 4) {
+        Packed8<T> t[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (j + i < p.top) t[i].load(rows + static_cast<size_t>(sr[j + i]) * p.ld + c);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (j + i < p.top) {
+            float f[8];
+            t[i].get(f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) a[k][e] = fmaf(sw[j + i], f[e], a[k][e]);
+          }
+      }
+    } else {
+      vload8(p.y + base + c, a[k]);
+    }
+    if (p.gate)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[k][e] *= sigmoid_t<T>(g[e] + gb[e]);
+  }
+  row_standardise(a, p.n, p.eps, scratch);
+  row_affine(a, static_cast<const T*>(p.w), static_cast<const T*>(p.b), p.ld);
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    const int c = row_piece(k);
+    if (c >= p.ld) break;
+    float f[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+    if (p.s) vload8(static_cast<const T*>(p.s) + c, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[k][e] = fmaf(a[k][e], f[e], x[k][e]);
+  }
+  row_store(x, p.x + base, p.ld);
+  if (p.h == nullptr) return;
+  row_standardise(x, p.n, p.eps, scratch + 2);
+  row_affine(x, static_cast<const T*>(p.next_w), static_cast<const T*>(p.next_b), p.ld);
+  row_store(x, static_cast<T*>(p.h) + base, p.ld);
+}
+
+// A block for a row of ld channels: pieces a thread and threads; FN<V, MAXT>
+#define B2_ROW_LAUNCH(ld, ...)                                                          \
+  do {                                                                                  \
+    const int pieces_ = (ld) / 8, v_ = pieces_ <= 256 ? 1 : pieces_ <= 512 ? 2 : 4;     \
+    const int threads = ((pieces_ + v_ - 1) / v_ + 31) / 32 * 32;                       \
+    if (v_ == 1) { constexpr int V = 1, MAXT = 256; __VA_ARGS__; }                      \
+    else if (v_ == 2) { constexpr int V = 2, MAXT = 256; __VA_ARGS__; }                 \
+    else if (threads <= 256) { constexpr int V = 4, MAXT = 256; __VA_ARGS__; }          \
+    else { constexpr int V = 4, MAXT = 1024; __VA_ARGS__; }                             \
+  } while (0)
 
 // out = gelu_tanh(gate) * table[id, first ...]: ids outside the vocabulary (padding rows) give zeros
 template <typename T>
@@ -447,5 +678,62 @@ B2_EXPORT int b2_gemm_f32(const float* A, const float* B, float* C, int M, int N
   gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, B, C, M, N, K, lda, ldb, ldc, accumulate, act,
                                                                      act_cols);
   B2_CHECK_LAUNCH("gemm_f32");
+  return 0;
+}
+
+B2_EXPORT int b2_layernorm_f32(const float* x, const void* w, const void* b, void* h, const long long* rows, int M, int ld, int n, float eps,
+                               int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld || ld > 32768) { set_error("layernorm_f32: ld %% 8 == 0, 0 < n <= ld <= 32768 required"); return 10; }
+  B2_DISPATCH_T(is_f32, B2_ROW_LAUNCH(ld, (layernorm_f32_kernel<T, V, MAXT><<<M, threads, 0, static_cast<cudaStream_t>(stream)>>>(
+      x, static_cast<const T*>(w), static_cast<const T*>(b), static_cast<T*>(h), rows, ld, n, eps))););
+  B2_CHECK_LAUNCH("layernorm_f32");
+  return 0;
+}
+
+// table T [vocab, ld], pairs T [buckets + 1, ld], last int32 [slots] (slot < 0: a padding row), h and next_* together or not at all
+B2_EXPORT int b2_embed_pairs(const long long* ids, const void* table, const void* pairs, int* last, const int* cu, const int* row_seq,
+                             const int* pos, const int* slot, const void* w, const void* b, const void* next_w, const void* next_b, float* x,
+                             void* h, int M, int ld, int n, int vocab, long long buckets, long long mul_prev, long long mul_cur, float eps,
+                             int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld || ld > 32768 || vocab < 1 || buckets < 1 || (h != nullptr && (next_w == nullptr || next_b == nullptr))) {
+    set_error("embed_pairs: ld %% 8 == 0, 0 < n <= ld <= 32768 and a bucket required");
+    return 10;
+  }
+  const EmbedPairsParams p = {ids, table, pairs, last, cu, row_seq, pos, slot, w, b, next_w, next_b, x, h, mul_prev, mul_cur, buckets, ld, n, vocab, eps};
+  B2_DISPATCH_T(is_f32, B2_ROW_LAUNCH(ld, (embed_pairs_kernel<T, V, MAXT><<<M, threads, 0, static_cast<cudaStream_t>(stream)>>>(p))););
+  B2_CHECK_LAUNCH("embed_pairs");
+  return 0;
+}
+
+// rows given: the weighted sum of top rows a token (P rows in all) in place of y.  gate_f32: a 32-bit gate beside bf16 weights.
+B2_EXPORT int b2_branch_add(float* x, const float* y, const void* rows, const int* place, const float* weights, int top, int P, const void* gate,
+                            long long ld_gate, int gate_f32, const void* gate_b, const void* w, const void* b, const void* s, const void* next_w,
+                            const void* next_b, void* h, int M, int ld, int n, float eps, int is_f32, void* stream) {
+  b2::ensure_thread_context();
+  if (M <= 0) return 0;
+  if (ld % 8 || n <= 0 || n > ld || ld > 32768 || (rows == nullptr) == (y == nullptr) ||
+      (rows != nullptr && (top < 1 || top > BA_MAX_TOP || place == nullptr || weights == nullptr)) ||
+      (gate != nullptr && (gate_b == nullptr || ld_gate % 8)) || (h != nullptr && (next_w == nullptr || next_b == nullptr))) {
+    set_error("branch_add: ld %% 8 == 0, 0 < n <= ld <= 32768 and up to %d rows a token required", BA_MAX_TOP);
+    return 10;
+  }
+  int* status = status_ptr();
+  if (!status) return 3;
+  const BranchParams p = {x, y, rows, place, weights, gate, gate_b, w, b, s, next_w, next_b, h, ld_gate, top, P, ld, n, eps, status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  B2_DISPATCH_T(is_f32, B2_ROW_LAUNCH(ld, {
+    if (rows != nullptr) {
+      if (gate_f32) branch_add_kernel<T, float, V, MAXT, true><<<M, threads, 0, st>>>(p);
+      else branch_add_kernel<T, T, V, MAXT, true><<<M, threads, 0, st>>>(p);
+    } else {
+      if (gate_f32) branch_add_kernel<T, float, V, MAXT, false><<<M, threads, 0, st>>>(p);
+      else branch_add_kernel<T, T, V, MAXT, false><<<M, threads, 0, st>>>(p);
+    }
+  }););
+  B2_CHECK_LAUNCH("branch_add");
   return 0;
 }
