@@ -163,7 +163,7 @@ inference_preview: {{enabled: false, max_tokens: 4}}
     assert json.loads(r.stdout[r.stdout.index("{"):])["completed_iterations"] == 2
 
 
-@pytest.mark.parametrize("preset", ["fetelorn-tiny", "sotazen-tiny", "ruburax-tiny"])
+@pytest.mark.parametrize("preset", ["fetelorn-tiny", "sotazen-tiny", "ruburax-tiny", "lufivik-tiny"])
 def test_run_inference_serves_a_hybrid_model(tmp_path, preset):
     """The architecture follows from the folder's config.json; the same flags as for any other model."""
     import torch
