@@ -42,7 +42,7 @@ def throughput(preset: str, batch: int = 256, prompt: int = 1024, new_tokens: in
         adaptive_chunking=False), model).initialize()
     eng.generate(_prompts(batch, prompt, mc.vocab_size, 1), warmup)           # allocator, graphs, tensor maps
     eng.generate(_prompts(batch, prompt, mc.vocab_size, 2), warmup)           # capturing the graphs gave the allocator's memory back
-    out = {"model": preset, "params": mc.num_params(), "batch": batch, "prompt": prompt, "new_tokens": new_tokens}
+    out = {"model": preset, "params": mc.num_params(), "params_per_token": getattr(mc, "num_active_params", mc.num_params)(), "batch": batch, "prompt": prompt, "new_tokens": new_tokens}
     for i, p in enumerate(_prompts(batch, prompt, mc.vocab_size)):
         eng.add_request(f"r{i}", p, new_tokens + 1)
     ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
@@ -401,6 +401,79 @@ def ruburax_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int
     return t.rows
 
 
+def lufivik_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
+    """The same for the windowed latent-attention decoder with softmax-routed experts."""
+    from ..ops import latent
+    mc, t = PRESETS[preset], _Timer()
+    W, V, eps = mc.hidden_size, mc.vocab_size, mc.norm_eps
+    m, f = mc.layers[0]["mixer"], mc.layers[0]["mlp"]
+    p, pages, starts, counts = _layout(lengths, batch, ctx)
+    M, n = p.rows, p.nseq
+    x, y32, w, b, h = torch.randn(M, W, device=DEV), torch.randn(M, W, device=DEV), _bf(W), _bf(W), _bf(M, W)
+
+    table, pairs, last = _bf(V, W), _bf(mc.buckets + 1, W), torch.zeros(n, dtype=torch.int32, device=DEV)
+    ids = torch.randint(0, V, (M,), device=DEV)
+    t("embedding_pairs", lambda: ops.embedding_pairs(ids, table, pairs, last, p, V, mc.mul_prev, mc.mul_cur, (w, b), W, eps, (w, b)), M * W * 10)
+    taps, conv = _bf(W, mc.taps), torch.zeros(n, W, mc.taps - 1, device=DEV)
+    t("input convolution", lambda: ops.causal_conv(h, None, taps, None, conv, p, add_input=True),
+      M * W * 4 + n * W * (mc.taps - 1) * 4 * (1 if lengths else 2))
+    _gemm(t, "gemm residual gate", M, W, W)
+    g16 = _bf(M, W)
+    t("branch_add", lambda: ops.branch_add(x, y32, (w, b), W, eps, g16, b, w, (w, b)), M * W * 16)
+
+    H, d, r, dv, C, Q, win = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"], m["mask"]["size"]
+    dq, R = d + r, C + r
+    _gemm(t, "gemm in (latents)", M, Q + R + pad8(H), W)
+    yy, pg = _bf(M, Q + R + pad8(H)), _bf(pages, 16, 1, R)
+    cs, sn = ops.rope_rows(p.positions, ops.rope_turns(m["rot"]["base"], r, DEV))
+    wq, wc, w_key, w_value, out = _bf(Q), _bf(C), _bf(H, dq, R), _bf(H, dv, C), _bf(M, H * dv)
+    cq, cc, kr, gate = yy[:, :Q], yy[:, Q:Q + C], yy[:, Q + C:Q + R], yy[:, Q + R:Q + R + H]
+    t("latent_store (both latents)", lambda: ops.latent_store(None, cc, kr, pg, p, H, d, C, r, wc, cs, sn, eps, cq, wq, Q),
+      M * (Q * 4 + R * 4 + r * 4))
+    _gemm(t, "gemm queries", M, H * dq, Q)
+    q, turn = _bf(M, H * dq), (cs, sn, d)
+    seen = sum(min(i + 1, win) for s, k in zip(starts, counts) for i in range(s, s + k))          # query-key pairs
+    if lengths is None:
+        ql, ol = _bf(M, H * R), _bf(M, H * C)
+        t("head_linear (queries to latent, turned)", lambda: ops.head_linear(q, w_key, ql, True, (cs, sn, C)), (M * H * (dq + R) + H * dq * R) * 2)
+        t("latent_rows", lambda: ops.latent_rows(ql, pg, ol, p, H, C, m["scale"], None, win), (seen * R + M * H * (R + C)) * 2,
+          2.0 * seen * H * (R + C))
+        t("head_linear (latent to values, gated)", lambda: ops.head_linear(ol, w_value, out, gate=gate), (M * H * (dv + C) + H * dv * C) * 2)
+        flops = 2.0 * seen * H * (R + C)
+    else:
+        _gemm(t, "gemm keys from latents", M, H * dq, R)
+        _gemm(t, "gemm values from latents", M, H * dv, C)
+        t("latent_turn", lambda: ops.latent_turn(q, H, d, cs, sn), M * (H * r * 4 + r * 4))
+        k, v, c = _bf(pages * 16, H * dq), _bf(pages * 16, H * dv), p.context(win)
+        t("latent prompt attention alone", lambda: latent.expanded_attention(q, k, v, out, p, H, dq, dv, m["scale"], None, 0, n, c.tables, win, gate),
+          M * H * (dq + dv) * 4, 2.0 * seen * H * (dq + dv))
+        rows = torch.empty(pages * 16, R, device=DEV, dtype=torch.bfloat16)
+        t("latent_gather", lambda: latent.gather(pg, c.pages, rows), rows.numel() * 4)
+        flops = 2.0 * (seen * H * (dq + dv) + M * H * (dq * R + dv * C))
+    t("latent_attention", lambda: ops.latent_attention(q, pg, out, p, w_key, w_value, m["scale"], None, win, gate, turn),
+      M * H * (dq + dv) * 2 + (seen if lengths is None else M) * R * 2, flops)
+    _gemm(t, "gemm latent o (fp32)", M, W, H * dv, True)
+
+    E, top, F = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+    wr = _bf(pad8(E) + W, W) * 0.05
+    t("router and gate product (fp32)", lambda: ops.linear_fp32(h, wr), (M * W + wr.numel()) * 2 + M * wr.shape[0] * 4, 2.0 * M * wr.numel())
+    z = ops.linear_fp32(h, wr)
+    t("choice and layout", lambda: ops.route(z, None, top, 1, 1, 1.0, score="softmax", experts=E), M * (E * 4 + top * 12))
+    rt = ops.route(z, None, top, 1, 1, 1.0, score="softmax", experts=E)
+    w_in, w_out, act = _bf(E, 2, F, W), _bf(E, W, F), (1.702, f["expert"]["limit"])
+    used = int((rt.offsets[1:] > rt.offsets[:-1]).sum())
+    t("expert_glu (clamped)", lambda: ops.expert_glu(h, w_in, rt, act), (used * 2 * F * W + M * W + M * top * F) * 2, 4.0 * M * top * F * W)
+    a = ops.expert_glu(h, w_in, rt, act)
+    t("expert_down", lambda: ops.expert_down(a, w_out, rt), (used * F * W + M * top * (F + W)) * 2, 2.0 * M * top * F * W)
+    rows = ops.expert_down(a, w_out, rt)
+    t("branch_add (experts)", lambda: ops.branch_add(x, (rows, rt), (w, b), W, eps, z[:, pad8(E):], b, w, (w, b)), M * W * (14 + 2 * top))
+    if lengths is None:
+        t("layernorm_f32", lambda: ops.layernorm_f32(x, (w, b), W, eps), M * W * 6)
+        _gemm(t, "gemm logits (fp32)", M, V, W, True)
+    del t.flush
+    return t.rows
+
+
 def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
     """The same for the dense decoder family."""
     mc, t = PRESETS[preset], _Timer()
@@ -443,6 +516,6 @@ def dense_kernels(preset: str, lengths: Optional[List[int]] = None, batch: int =
 
 
 def kernels(preset: str, lengths: Optional[List[int]] = None, batch: int = 256, ctx: int = 1024) -> Dict:
-    by_name = {"Fetelorn": fetelorn_kernels, "Sotazen": sotazen_kernels, "Ruburax": ruburax_kernels}
+    by_name = {"Fetelorn": fetelorn_kernels, "Sotazen": sotazen_kernels, "Ruburax": ruburax_kernels, "Lufivik": lufivik_kernels}
     with torch.no_grad():
         return by_name.get(getattr(PRESETS[preset], "architecture", None), dense_kernels)(preset, lengths, batch, ctx)

@@ -301,6 +301,6 @@ LUFIVIK_PRESETS = {
     "lufivik-tiny": lufivik_preset(256, 2, 3, 1024, 96, 8, 2, 128, (1, 2, 2), window=64, rank=64, dim=64, rot=32),
     # the widths, head counts, layer runs and vocabulary of the framework's other presets of the same size; as many feed-forward channels
     # per token as theirs, in four chosen experts
-    "lufivik-0.6b": lufivik_preset(1024, 8, 20, 151936, 512, 32, 4, 800, (8, 12, 3)),
-    "lufivik-4b": lufivik_preset(2560, 16, 24, 151936, 1024, 32, 4, 2400, (8, 14, 3)),
+    "lufivik-0.6b": lufivik_preset(1024, 8, 20, 151936, 512, 32, 4, 768, (8, 12, 3)),
+    "lufivik-4b": lufivik_preset(2560, 16, 24, 151936, 1024, 32, 4, 2432, (8, 14, 3)),
 }

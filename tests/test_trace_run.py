@@ -26,7 +26,8 @@ SOTAZEN = S.config(36, 51, [S.latent(2, 16, 8, 12, 24, ff=16), S.lightning(2, 8,
 RUBURAX = R.config(36, 51, [R.rglru(24, 2, 3, ff=R.dense(16)), R.attention(2, 1, 16, 8, R.rot(8, 400.0, (4.0, 1.0, 2.0, 20))),
                             R.parallel(R.att(2, 1, 8, 8, R.rot(8)), 2, 8, 12, 6.0, 0.7, 1.2, ff=R.moe(6, 2, 12, (3, 2), 8)),
                             R.attention(4, 1, 16, 8, R.rot(8, 400.0, (4.0, 1.0, 2.0, 20)), kv_from=1, ff=R.dense(16))])
-LUFIVIK = L.config(36, 51, [L.latent(2, 16, 8, 12, 20, 24, 11, L.moe(6, 2, 12)), L.latent(3, 8, 4, 10, 12, 16, 7), L.latent(1, 8, 8, 8, 8, 8, 30, L.moe(5, 3, 8))],
+# every expert is chosen: no position rests on a close choice
+LUFIVIK = L.config(36, 51, [L.latent(2, 16, 8, 12, 20, 24, 11, L.moe(6, 6, 12)), L.latent(3, 8, 4, 10, 12, 16, 7), L.latent(1, 8, 8, 8, 8, 8, 30, L.moe(5, 5, 8))],
                    loop=(1, 3, 2))
 MODELS = {"Fetelorn": (CFG, O, build), "Sotazen": (SOTAZEN, SO, S.build), "Ruburax": (RUBURAX, RO, R.build), "Lufivik": (LUFIVIK, LO, L.build)}
 
